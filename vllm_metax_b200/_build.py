@@ -1,8 +1,10 @@
 """In-tree build of the native extensions for sm_100a.
 
-Two shared objects are produced next to this file:
+The shared objects are produced next to this file:
 
 * ``_b200_C.so``            - CUDA kernels + ``torch.ops.b200`` bindings
+* ``_b200_core.so``         - the core set of them alone (``CORE_UNITS`` + ``bindings_core.cpp``): all that a model class
+  with ``native_units = "core"`` calls; built on demand where the full library does not exist yet
 * ``cumem_allocator.so``    - sleep-mode VMM allocator (CPython module, driver API)
 
 Every ``.cu`` is compiled with ``-gencode arch=compute_100a,code=sm_100a`` by a
@@ -27,10 +29,18 @@ ROOT = Path(__file__).resolve().parent
 CSRC = ROOT / "csrc"
 OBJ = ROOT / "_obj"
 LIB = ROOT / "_b200_C.so"
+CORE_LIB = ROOT / "_b200_core.so"
 CUMEM_LIB = ROOT / "cumem_allocator.so"
 
+# the units behind bindings_core.cpp
+CORE_UNITS = ("attn_prefill_pingpong", "attn_prefill_tcgen05", "causal_conv1d", "fused_misc", "gemm_grouped_tcgen05",
+              "gemm_pair_tcgen05", "gemm_simt", "gemm_splitk_tcgen05", "gemm_streamk_tcgen05", "gemm_tcgen05", "gla",
+              "latent_attn", "mla_decode", "mla_decode_tcgen05", "moe", "residual_conv", "rglru", "sampling")
+# units whose arithmetic is 32-bit by contract (recurrences, norms, angles, fp32 products): no fast-math substitutions
+PRECISE_UNITS = ("gemm_simt", "gla", "latent_attn", "residual_conv", "rglru")
+
 NVCC_FLAGS = [
-    "-gencode", "arch=compute_100a,code=sm_100a", "-std=c++17", "-O3", "-lineinfo", "--use_fast_math",
+    "-gencode", "arch=compute_100a,code=sm_100a", "-std=c++17", "-O3", "-lineinfo",
     "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr", "-DNDEBUG",
 ]
 
@@ -56,9 +66,14 @@ def sources() -> list[Path]:
     return sorted(CSRC.glob("*.cu"))
 
 
-def build(verbose: bool = False, force: bool = False) -> Optional[Path]:
+def _unit_flags(unit: str) -> list[str]:
+    return NVCC_FLAGS if unit in PRECISE_UNITS else NVCC_FLAGS + ["--use_fast_math"]
+
+
+def build(verbose: bool = False, force: bool = False, core_only: bool = False) -> Optional[Path]:
     """Compile ``csrc/*.cu`` for sm_100a and link ``_b200_C.so`` in-tree.  ``B200_TARGET_DEVICE=empty`` skips the
-    native build (a CPU-only checkout that runs the PyTorch reference ops; the reference's ``VLLM_TARGET_DEVICE``)."""
+    native build (a CPU-only checkout that runs the PyTorch reference ops; the reference's ``VLLM_TARGET_DEVICE``).
+    ``core_only`` compiles the core units and links ``_b200_core.so`` instead."""
     if os.environ.get("B200_TARGET_DEVICE", "cuda").lower() in ("empty", "cpu"):
         return None
     import torch
@@ -70,21 +85,26 @@ def build(verbose: bool = False, force: bool = False) -> Optional[Path]:
     jobs = []
     objs = []
     for src in sources():
+        if core_only and src.stem not in CORE_UNITS:
+            continue
         obj = OBJ / (src.stem + ".o")
         objs.append(obj)
         if force or _newer([src, *headers], obj):
-            jobs.append([nvcc, *NVCC_FLAGS, "-I", str(CSRC), "-c", str(src), "-o", str(obj)])
-    bind_src = CSRC / "bindings.cpp"
-    bind_obj = OBJ / "bindings.o"
-    objs.append(bind_obj)
+            jobs.append([nvcc, *_unit_flags(src.stem), "-I", str(CSRC), "-c", str(src), "-o", str(obj)])
+    binds = [CSRC / "bindings_core.cpp"] + ([] if core_only else [CSRC / "bindings.cpp"])
     inc = []
     for p in include_paths(device_type="cuda") if "device_type" in include_paths.__code__.co_varnames else include_paths(cuda=True):
         inc += ["-I", p]
     inc += ["-I", os.path.join(_cuda_home(), "include"), "-I", sysconfig.get_paths()["include"]]
     cxx_abi = int(torch._C._GLIBCXX_USE_CXX11_ABI)
-    if force or _newer([bind_src, *headers], bind_obj):
-        jobs.append(["g++", "-std=c++17", "-O2", "-fPIC", f"-D_GLIBCXX_USE_CXX11_ABI={cxx_abi}",
-                     "-DTORCH_EXTENSION_NAME=_b200_C", *inc, "-I", str(CSRC), "-c", str(bind_src), "-o", str(bind_obj)])
+    for bind_src in binds:
+        bind_obj = OBJ / (bind_src.stem + ".o")
+        objs.append(bind_obj)
+        if force or _newer([bind_src, *headers], bind_obj):
+            jobs.insert(0, ["g++", "-std=c++17", "-O2", "-fPIC", f"-D_GLIBCXX_USE_CXX11_ABI={cxx_abi}",
+                            "-DTORCH_EXTENSION_NAME=_b200_C", *inc, "-I", str(CSRC), "-c", str(bind_src), "-o",
+                            str(bind_obj)])
+    lib = CORE_LIB if core_only else LIB
     if jobs:
         workers = int(os.environ.get("MAX_JOBS", "0")) or min(8, os.cpu_count() or 4)
         import json
@@ -107,14 +127,15 @@ def build(verbose: bool = False, force: bool = False) -> Optional[Path]:
         times_file.write_text(json.dumps(times, indent=1, sort_keys=True))
         if verbose:
             print(f"[b200 build] compiled {len(jobs)} translation units")
-    if force or jobs or not LIB.exists():
+    if force or jobs or not lib.exists():
         libdirs = []
         for p in library_paths(device_type="cuda") if "device_type" in library_paths.__code__.co_varnames else library_paths(cuda=True):
             libdirs += ["-L", p, f"-Wl,-rpath,{p}"]
-        _run(["g++", "-shared", "-o", str(LIB), *map(str, objs), *libdirs, "-L", os.path.join(_cuda_home(), "lib64"),
+        _run(["g++", "-shared", "-o", str(lib), *map(str, objs), *libdirs, "-L", os.path.join(_cuda_home(), "lib64"),
               "-lc10", "-lc10_cuda", "-ltorch_cpu", "-ltorch_cuda", "-ltorch", "-lcudart"])
-    build_cumem(verbose=verbose, force=force)
-    return LIB
+    if not core_only:
+        build_cumem(verbose=verbose, force=force)
+    return lib
 
 
 def build_cumem(verbose: bool = False, force: bool = False) -> Path | None:

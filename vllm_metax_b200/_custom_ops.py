@@ -20,26 +20,38 @@ from . import envs
 from .ops import reference as ref
 
 _LIB = Path(__file__).resolve().parent / "_b200_C.so"
+_CORE_LIB = Path(__file__).resolve().parent / "_b200_core.so"
 _loaded = False
+_loaded_units = ""
 
 ACT_CODES = {"silu": 0, "gelu": 1, "gelu_tanh": 2, "fatrelu": 3, "relu2": 4, "mul_silu": 5, "swigluoai": 6,
              "swiglustep": 7, "gelu_new": 8, "gelu_fast": 9, "gelu_quick": 10}
+# GEMM epilogues (csrc/gemm_epilogue.cuh)
+EPI_CODES = {None: 0, "silu_gate": 1, "gelu": 2, "gelu_tanh": 3, "xielu": 4}
 CACHE_KIND = {"same": 0, "fp8_static": 1, "int8_dyn": 2, "fp8_dyn": 3}
 
 
-def load_native(build_if_missing: bool = True) -> bool:
-    """Load ``_b200_C.so`` (building it in-tree when absent and allowed)."""
-    global _loaded
-    if _loaded:
+def load_native(build_if_missing: bool = True, units: str = "all") -> bool:
+    """Load ``_b200_C.so`` (building it in-tree when absent and allowed).  ``units="core"``: the caller needs the core set
+    only - where the full library has not been built, the core library is built and loaded instead."""
+    global _loaded, _loaded_units
+    if _loaded and (units == "core" or _loaded_units == "all"):
         return True
+    if _loaded:
+        raise RuntimeError("this process serves a model on the core kernel library; build the full one "
+                           "(python -m vllm_metax_b200._build) to use other ops beside it")
+    lib, got = _LIB, "all"
     if not _LIB.exists():
-        if not build_if_missing or envs.B200_USE_PREBUILT_KERNELS:
-            return False
-        from ._build import build
+        if units == "core":
+            lib, got = _CORE_LIB, "core"
+        if not lib.exists():
+            if not build_if_missing or envs.B200_USE_PREBUILT_KERNELS:
+                return False
+            from ._build import build
 
-        build()
-    torch.ops.load_library(str(_LIB))
-    _loaded = True
+            build(core_only=got == "core")
+    torch.ops.load_library(str(lib))
+    _loaded, _loaded_units = True, got
     return True
 
 
@@ -68,7 +80,7 @@ def _use_cuda(t: torch.Tensor) -> bool:
         _force_ref = bool(envs.B200_FORCE_REFERENCE_OPS)
     if _force_ref:
         return False
-    if not _loaded and not load_native():
+    if not _loaded and not load_native():      # (the runner loads what its model needs before the first op)
         raise RuntimeError("CUDA tensor given but the native library _b200_C.so is not built; "
                            "run `python -m vllm_metax_b200._build`")
     _launches += 1
@@ -95,13 +107,28 @@ def check_kernel_status(device: int = 0) -> None:
 
 
 # --------------------------------------------------------------------------- GEMM
+def _tma_ok(*ts: torch.Tensor) -> bool:
+    """Rows (and batches) that start on 16 bytes: what the tensor-core GEMMs load and store."""
+    return all(t.data_ptr() % 16 == 0 and all(s % 8 == 0 for s in t.stride()[:-1]) for t in ts)
+
+
 def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
          residual: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
-         force_bn: int = 0) -> torch.Tensor:
-    """``a [M,K] @ w [N,K]^T (+bias) (+residual)``."""
-    if _use_cuda(a) and a.dtype in (torch.bfloat16, torch.float16):
+         force_bn: int = 0, act: Optional[str] = None, act_params: Optional[torch.Tensor] = None,
+         out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+    """``act(a [M,K] @ w [N,K]^T (+bias)) (+residual)``.  ``act``: None, gelu, gelu_tanh, xielu (``act_params`` = its two
+    fp32 coefficients), applied to the fp32 accumulators in the epilogue; ``out_dtype=torch.float32`` stores those."""
+    if _use_cuda(a):
         if out is None:
-            out = torch.empty(a.shape[0], w.shape[0], dtype=a.dtype, device=a.device)
+            out = torch.empty(a.shape[0], w.shape[0], dtype=out_dtype or a.dtype, device=a.device)
+        if a.dtype == torch.float32 or a.shape[1] % 8 != 0 or not _tma_ok(a, w, out):
+            torch.ops.b200.gemm_simt(out, a, w, bias, EPI_CODES[act], act_params, None, None)
+            if residual is not None:
+                out.add_(residual)
+            return out
+        if act is not None or out.dtype != a.dtype:
+            torch.ops.b200.gemm(out, a, w, bias, residual, 128 if batch_invariant() else force_bn, EPI_CODES[act], act_params)
+            return out
         global _tc_gemm
         if _tc_gemm is None:
             _tc_gemm = bool(envs.B200_TCGEN05_GEMM)
@@ -114,13 +141,30 @@ def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
             if residual is not None:
                 out.add_(residual)
         return out
-    y = ref.gemm(a, w, bias)
+    y = ref.gemm(a, w, bias, torch.float32 if act is not None else out_dtype)
+    if act is not None:
+        y = ref.epilogue_activation(y, act, act_params).to(out_dtype or a.dtype)
     if residual is not None:
         y = (y.float() + residual.float()).to(a.dtype)
     if out is not None:
         out.copy_(y)
         return out
     return y
+
+
+def gemm_batched(a: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``out[z] = a[z] @ w[z]^T`` for ``a [Z,M,K]``, ``w [Z,N,K]`` and ``out [Z,M,N]`` (strided views; ``out`` of a's dtype
+    or fp32): block-diagonal gates, per-head absorption products."""
+    if out is None:
+        out = torch.empty(a.shape[0], a.shape[1], w.shape[1], dtype=a.dtype, device=a.device)
+    if _use_cuda(a):
+        if a.dtype != torch.float32 and a.shape[2] % 8 == 0 and _tma_ok(a, w, out):
+            torch.ops.b200.gemm_batched(out, a, w, 0)
+        else:
+            torch.ops.b200.gemm_simt(out, a, w, None, 0, None, None, None)
+        return out
+    out.copy_(torch.bmm(a.float(), w.float().transpose(1, 2)))
+    return out
 
 
 def gemm_silu_mul(a: torch.Tensor, w_interleaved: torch.Tensor, bias: Optional[torch.Tensor] = None,
@@ -546,7 +590,7 @@ def advance_step(input_ids, positions, seq_lens, slot_mapping, sampled, block_ta
 
 
 def embedding(table, ids, out=None, vocab_start: int = 0):
-    if _use_cuda(table) and table.dtype in (torch.bfloat16, torch.float16):
+    if _use_cuda(table) and table.dtype in (torch.bfloat16, torch.float16) and table.shape[1] % 8 == 0:
         out = torch.empty(ids.numel(), table.shape[1], dtype=table.dtype, device=table.device) if out is None else out
         torch.ops.b200.embedding(out, table, ids, vocab_start)
         return out
@@ -656,11 +700,14 @@ def moe_gather(x, sorted_ids, total_padded, topk: int):
 
 def gemm_grouped(a, w, block_expert, total_padded, epi: int = 0):
     """Per-row-block expert GEMM: ``a [R, K]`` (R multiple of 128), ``w [E, N, K]`` -> ``[R, N]`` (``N/2`` with the
-    SiLU-gate epilogue over row-interleaved gate/up weights)."""
+    SiLU-gate epilogue over row-interleaved gate/up weights).  ``epi``: a code of ``EPI_CODES``."""
     if _use_cuda(a):
         n_out = w.shape[1] // 2 if epi == 1 else w.shape[1]
         out = torch.empty(a.shape[0], n_out, dtype=a.dtype, device=a.device)
-        torch.ops.b200.gemm_grouped(out, a, w, block_expert, total_padded, epi)
+        if a.dtype == torch.float32 or a.shape[1] % 8 != 0 or not _tma_ok(a, w, out):
+            torch.ops.b200.gemm_simt(out, a, w, None, epi, None, block_expert, total_padded)
+        else:
+            torch.ops.b200.gemm_grouped(out, a, w, block_expert, total_padded, epi)
         return out
     R = a.shape[0]
     nblk = R // 128
@@ -674,6 +721,9 @@ def gemm_grouped(a, w, block_expert, total_padded, epi: int = 0):
         y = ref.gemm(a[b * 128:(b + 1) * 128], w[e])
         if epi == 1:
             y = (torch.nn.functional.silu(y[:, 0::2].float()) * y[:, 1::2].float()).to(a.dtype)
+        elif epi > 1:
+            y = ref.epilogue_activation(ref.gemm(a[b * 128:(b + 1) * 128], w[e], out_dtype=torch.float32),
+                                        {v: k for k, v in EPI_CODES.items()}[epi], None).to(a.dtype)
         out[b * 128:(b + 1) * 128] = y
     return out
 
@@ -868,16 +918,20 @@ def wna16_gemm(x, qweight, scales, zeros, bits: int, group: int, *, bias=None, b
 
 # --------------------------------------------------------------------------- MLA
 def mla_decode(q, mla_cache, block_table, seq_lens, scale, *, query_start_loc=None, topk_indices=None, out=None,
-               lse_out=None, num_splits: int = 0, max_seq_len: int = 0, impl: int = 0):
+               lse_out=None, num_splits: int = 0, max_seq_len: int = 0, impl: int = 0, window: int = 0,
+               kv_rank: int = 512):
     """Absorbed MLA over the latent cache (dense, or sparse with ``topk_indices [T, topk]``).
     ``q [T, H, 576]`` -> ``[T, H, 512]``.  ``impl``: 0 = choose, 1 = mma.sync kernel, 2 = tcgen05 kernel (dense 16-bit
     caches; csrc/mla_decode_tcgen05.cu) or fail.  "Choose" takes the tcgen05 kernel for 64 heads per rank or more only
-    with ``B200_MLA_TCGEN05=1``."""
+    with ``B200_MLA_TCGEN05=1``.  Other sizes: cache rows ``[kv_rank latent | rotated part | padding]``, queries of the same
+    row length, output ``[T, H, kv_rank]``.  ``window`` > 0: only the last ``window`` visible positions."""
     if _use_cuda(q):
         T, H, _ = q.shape
+        if q.dtype == torch.float32 or kv_rank > 512:      # CUDA-core kernel: one pass
+            num_splits = 1
         if impl == 0 and not envs.B200_MLA_TCGEN05:
             impl = 1
-        out = torch.empty(T, H, 512, dtype=q.dtype, device=q.device) if out is None else out
+        out = torch.empty(T, H, kv_rank, dtype=q.dtype, device=q.device) if out is None else out
         if num_splits <= 0 and batch_invariant():
             num_splits = 1
         if num_splits <= 0:
@@ -887,19 +941,64 @@ def mla_decode(q, mla_cache, block_table, seq_lens, scale, *, query_start_loc=No
             if impl != 1 and topk_indices is None and mla_cache.dtype != torch.uint8 and (impl == 2 or H >= 64):
                 ctas = 2 * T * ((H + 127) // 128)            # tcgen05 kernel: 128 heads x half the latent per CTA
             kv = topk_indices.shape[1] if topk_indices is not None else (max_seq_len or 4096)
+            if window > 0:
+                kv = min(kv, window)
             num_splits = 1 if ctas >= 148 else max(1, min((296 + ctas - 1) // ctas, kv // 256, 16))
-        ws = _decode_workspace(q.device, num_splits * T * H * 513) if num_splits > 1 else None
+        ws = _decode_workspace(q.device, num_splits * T * H * (kv_rank + 1)) if num_splits > 1 else None
         torch.ops.b200.mla_decode(out, q, mla_cache, block_table, seq_lens, query_start_loc, topk_indices, scale,
-                                  lse_out, ws, num_splits, impl)
+                                  lse_out, ws, num_splits, impl, window)
         return out
-    res, lse = ref.mla_decode(q, mla_cache, block_table, seq_lens, scale, query_start_loc=query_start_loc,
-                              topk_indices=topk_indices)
+    res, lse = ref.mla_decode(q, mla_cache, block_table, seq_lens, scale, kv_lora_rank=kv_rank,
+                              query_start_loc=query_start_loc, topk_indices=topk_indices, window=window)
     if lse_out is not None:
         lse_out.copy_(lse)
     if out is not None:
         out.copy_(res)
         return out
     return res
+
+
+def latent_insert(a, q_off: int, kv_off: int, q_weight, kv_weight, rot_dim: int, inv_freq, positions, cache, slot_mapping,
+                  eps: float):
+    """Epilogue of the merged latent down-projection ``a``: returns the normed query latent ``[T, q_rank]`` and writes
+    ``[normed key latent | rotated key part]`` into the paged cache rows ``slot_mapping`` names (-1: none)."""
+    T, qr, kr = a.shape[0], q_weight.numel(), kv_weight.numel()
+    if _use_cuda(a):
+        cq = torch.empty(T, qr, dtype=a.dtype, device=a.device)
+        torch.ops.b200.latent_insert(cq, cache, a, q_off, kv_off, q_weight, kv_weight, rot_dim, inv_freq, positions,
+                                     slot_mapping, eps)
+        return cq
+    cq = ref.rms_norm(a[:, q_off: q_off + qr], q_weight, eps)
+    rows = torch.zeros(T, cache.shape[-1], dtype=a.dtype, device=a.device)
+    rows[:, :kr] = ref.rms_norm(a[:, kv_off: kv_off + kr], kv_weight, eps)
+    rows[:, kr: kr + rot_dim] = ref.rotate_half(a[:, kv_off + kr: kv_off + kr + rot_dim][:, None], inv_freq, positions)[:, 0]
+    ok = slot_mapping[:T] >= 0
+    cache.view(-1, cache.shape[-1])[slot_mapping[:T][ok]] = rows[ok]
+    return cq
+
+
+def latent_rope(dst, src, inv_freq, positions, rot_dim: int, pad: int = 0):
+    """Rotates ``src [T, H, rot_dim]`` into ``dst`` (may be the same memory) and zeroes ``pad`` entries behind."""
+    if _use_cuda(src):
+        torch.ops.b200.latent_rope(dst, src, inv_freq, positions, rot_dim, pad)
+        return dst
+    dst[..., :rot_dim] = ref.rotate_half(src[..., :rot_dim], inv_freq, positions)
+    dst[..., rot_dim: rot_dim + pad] = 0
+    return dst
+
+
+def gather_mla_cache(cache, block_table, cu_rows, first, total: int):
+    """Rows ``first[b] ..`` of every request's latent cache, ``cu_rows[b+1] - cu_rows[b]`` of them: ``[total, row]``."""
+    if _use_cuda(cache):
+        dst = torch.empty(total, cache.shape[-1], dtype=cache.dtype, device=cache.device)
+        torch.ops.b200.gather_mla_cache(dst, cache, block_table, cu_rows, first)
+        return dst
+    bs, cu = cache.shape[1], cu_rows.tolist()
+    parts = []
+    for b in range(len(cu) - 1):
+        pos = torch.arange(cu[b + 1] - cu[b]) + int(first[b])
+        parts.append(cache[block_table[b].long()[pos // bs], pos % bs])
+    return torch.cat(parts)
 
 
 # --------------------------------------------------------------------------- DSA indexer

@@ -183,7 +183,23 @@ class ModelConfig:
         return i >= self.first_k_dense_replace and (i % max(self.moe_layer_freq, 1) == 0)
 
     @classmethod
+    def from_layer_list(cls, d: dict, **overrides: Any) -> "ModelConfig":
+        """Configs that name their ``architecture`` and list the ``layers`` one by one, each with its own mixer and
+        feed-forward sizes; the model class reads the details from ``hf_config``."""
+        heads = max([int(l["mixer"].get("heads", 1)) for l in d["layers"]], default=1)
+        kw: dict[str, Any] = dict(
+            architecture=d["architecture"], hf_config=dict(d), vocab_size=int(d["vocab"]), hidden_size=int(d["width"]),
+            intermediate_size=max([int((l.get("mlp") or {}).get("ff", 0)) for l in d["layers"]], default=0),
+            num_hidden_layers=len(d["layers"]), num_attention_heads=heads, head_dim=max(1, int(d["width"]) // heads),
+            rms_norm_eps=float(d["norm"]["eps"]), max_position_embeddings=int(d.get("max_position", 1 << 20)),
+            dtype=d.get("dtype", "bfloat16"), eos_token_id=d.get("eos_token_id"))
+        kw.update(overrides)
+        return cls(**kw)
+
+    @classmethod
     def from_hf_dict(cls, d: dict, **overrides: Any) -> "ModelConfig":
+        if isinstance(d.get("layers"), list) and "architecture" in d:
+            return cls.from_layer_list(d, **overrides)
         raw = d
         if isinstance(d.get("llm_config"), dict) and "text_config" not in d:      # InternVL's original export
             d = dict(d, text_config=d["llm_config"])

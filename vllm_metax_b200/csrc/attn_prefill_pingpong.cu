@@ -19,7 +19,8 @@
 //   The three warp groups re-balance the register file at start-up (setmaxnreg): the producer / issuer
 //   group gives registers up, the softmax groups take them so that a 128-wide row of S fits.
 //
-// Query heads must be 16-bit (bf16/fp16); (D_qk, D_v) in {(128,128), (64,64), (192,128)}.
+// Query heads must be 16-bit (bf16/fp16); the tiles are (D_qk, D_v) in {(128,128), (64,64), (192,128)}.  Contiguous K / V
+// may have smaller heads (multiples of 8): the TMA maps end at the real sizes and the fill pads the tile with zeros.
 // Causal offset: row token i of a sequence with q_len new tokens and kv_len total sits at position
 // kv_len - q_len + i.  Sliding window, soft-cap, ALiBi and attention sinks are supported; LSE can be
 // returned for later merges.  TMA loads touch this GPU's memory only.
@@ -383,7 +384,7 @@ attn_prefill_pp_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       tc_fence_after_sync();
     }
     if (ok && n_mine > 0) {
-      T* dst = reinterpret_cast<T*>(p.out) + ((int64_t)(q_begin + tok) * p.num_q_heads + hq) * DV;
+      T* dst = reinterpret_cast<T*>(p.out) + ((int64_t)(q_begin + tok) * p.num_q_heads + hq) * p.dv;
 #pragma unroll 1
       for (int c = 0; c < DV; c += 32) {
         uint32_t v[32];
@@ -395,14 +396,14 @@ attn_prefill_pp_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
             float f[8];
 #pragma unroll
             for (int i = 0; i < 8; ++i) f[i] = __uint_as_float(v[g8 * 8 + i]) * o_acc_scale;
-            *reinterpret_cast<uint4*>(dst + c + g8 * 8) = pack8<T>(f);
+            if (c + g8 * 8 < p.dv) *reinterpret_cast<uint4*>(dst + c + g8 * 8) = pack8<T>(f);
           }
         }
       }
     } else if (ok && row_valid) {
       // a row whose tile sees no key at all (empty context): zeros
-      T* dst = reinterpret_cast<T*>(p.out) + ((int64_t)(q_begin + tok) * p.num_q_heads + hq) * DV;
-      for (int c = 0; c < DV; c += 8) *reinterpret_cast<uint4*>(dst + c) = make_uint4(0, 0, 0, 0);
+      T* dst = reinterpret_cast<T*>(p.out) + ((int64_t)(q_begin + tok) * p.num_q_heads + hq) * p.dv;
+      for (int c = 0; c < p.dv; c += 8) *reinterpret_cast<uint4*>(dst + c) = make_uint4(0, 0, 0, 0);
     }
     if (ok && row_valid && p.lse_out)
       p.lse_out[(int64_t)hq * p.total_q + q_begin + tok] =
@@ -426,8 +427,8 @@ static void launch_prefill_pp(const PrefillParams& p, const void* q, int64_t q_s
   const CUtensorMapDataType dt =
       std::is_same<T, __half>::value ? CU_TENSOR_MAP_DATA_TYPE_FLOAT16 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
   // Q: [T, Hq, DQK], box [128/gp tokens, gp heads, 64]
-  uint64_t qd[3] = {(uint64_t)DQK, (uint64_t)p.num_q_heads, (uint64_t)p.total_q};
-  uint64_t qs[2] = {(uint64_t)DQK * 2, (uint64_t)q_stride * 2};
+  uint64_t qd[3] = {(uint64_t)p.dqk, (uint64_t)p.num_q_heads, (uint64_t)p.total_q};
+  uint64_t qs[2] = {(uint64_t)p.dqk * 2, (uint64_t)q_stride * 2};
   uint32_t qb[3] = {64, (uint32_t)p.gp, (uint32_t)(kPpBM / p.gp)};
   CUtensorMap tmQ = make_tmap_nd(q, dt, 3, qd, qs, qb, CU_TENSOR_MAP_SWIZZLE_128B);
   CUtensorMap tmK, tmV;
@@ -441,12 +442,12 @@ static void launch_prefill_pp(const PrefillParams& p, const void* q, int64_t q_s
     tmK = make_tmap_nd(k_src, dt, 4, kd, ks, kb, CU_TENSOR_MAP_SWIZZLE_128B);
     tmV = tmK;
   } else {
-    uint64_t kd[3] = {(uint64_t)DQK, (uint64_t)p.num_kv_heads, (uint64_t)total_kv};
-    uint64_t ks[2] = {(uint64_t)DQK * 2, (uint64_t)kv_tok_stride_k * 2};
+    uint64_t kd[3] = {(uint64_t)p.dqk, (uint64_t)p.num_kv_heads, (uint64_t)total_kv};
+    uint64_t ks[2] = {(uint64_t)p.k_head_stride * 2, (uint64_t)kv_tok_stride_k * 2};
     uint32_t kb[3] = {64, 1, (uint32_t)BN};
     tmK = make_tmap_nd(k_src, dt, 3, kd, ks, kb, CU_TENSOR_MAP_SWIZZLE_128B);
-    uint64_t vd[3] = {(uint64_t)DV, (uint64_t)p.num_kv_heads, (uint64_t)total_kv};
-    uint64_t vs[2] = {(uint64_t)DV * 2, (uint64_t)kv_tok_stride_v * 2};
+    uint64_t vd[3] = {(uint64_t)p.dv, (uint64_t)p.num_kv_heads, (uint64_t)total_kv};
+    uint64_t vs[2] = {(uint64_t)p.v_head_stride * 2, (uint64_t)kv_tok_stride_v * 2};
     tmV = make_tmap_nd(v_src, dt, 3, vd, vs, kb, CU_TENSOR_MAP_SWIZZLE_128B);
   }
   auto kern = attn_prefill_pp_kernel<T, DQK, DV, BN>;
@@ -468,6 +469,12 @@ int attention_prefill_pp(const PrefillParams& p, const void* q, int64_t q_stride
                          int64_t k_tok_stride, int64_t v_tok_stride, int64_t total_kv, int dqk, int dv, int dtype,
                          int batch, int max_q_len, cudaStream_t stream) {
   if (batch <= 0 || max_q_len <= 0) return 0;
+  if (!p.paged) {                                // contiguous K / V: round the heads up to the tile sizes
+    if (dqk % 8 != 0 || dv % 8 != 0) return -1;
+    if (dqk <= 64 && dv <= 64) dqk = dv = 64;
+    else if (dqk <= 128 && dv <= 128) dqk = dv = 128;
+    else if (dqk <= 192 && dv <= 128) dqk = 192, dv = 128;
+  }
 #define PF(T)                                                                                                        \
   if (dqk == 128 && dv == 128)                                                                                       \
     launch_prefill_pp<T, 128, 128, 128>(p, q, q_stride, k_src, v_src, k_tok_stride, v_tok_stride, total_kv, batch, max_q_len, stream); \

@@ -1,144 +1,11 @@
-// torch.ops.b200.* : adapts torch tensors to the torch-free launchers in ops.h.
-// Every op writes into caller-provided tensors (no allocation here), so the ops can
-// be captured in CUDA graphs.
-#include <ATen/cuda/CUDAContext.h>
-#include <c10/cuda/CUDAGuard.h>
-#include <torch/library.h>
-#include <torch/types.h>
-
-#include <cstdlib>
-#include <cstring>
-#include <tuple>
-
-#include "comm_params.h"
-#include "ops.h"
+// torch.ops.b200.*, the ops beyond the core set (bindings_core.cpp): quantised GEMMs, other caches and attention forms,
+// fused norm / rope kernels, collectives over peer memory.
+#include "bindings_common.h"
 
 namespace {
 
-using at::Tensor;
-using c10::optional;
+using namespace b200_bind;
 
-inline cudaStream_t cur_stream() { return at::cuda::getCurrentCUDAStream().stream(); }
-
-inline int dtype_code(const Tensor& t) {
-  switch (t.scalar_type()) {
-    case at::kBFloat16: return 0;
-    case at::kHalf: return 1;
-    case at::kFloat: return 2;
-    default: TORCH_CHECK(false, "unsupported dtype ", t.scalar_type());
-  }
-}
-inline int dtype16(const Tensor& t) {
-  const int c = dtype_code(t);
-  TORCH_CHECK(c < 2, "expected a bf16 / fp16 tensor");
-  return c;
-}
-template <typename T = void>
-inline T* ptr(const optional<Tensor>& t) {
-  return t.has_value() && t->defined() ? reinterpret_cast<T*>(t->data_ptr()) : nullptr;
-}
-
-// One status word per device, zero-initialised on first use.
-Tensor& status_tensor(int device) {
-  static std::vector<Tensor> words(64);
-  if (!words[device].defined())
-    words[device] = torch::zeros({4}, torch::dtype(torch::kInt32).device(torch::kCUDA, device));
-  return words[device];
-}
-inline void* status_ptr(const Tensor& any) { return status_tensor(any.get_device()).data_ptr(); }
-
-Tensor get_status(int64_t device) { return status_tensor((int)device); }
-
-// ------------------------------------------------------------------ GEMM
-// Scratch of the stream-K GEMM (partial tiles + arrival counters): allocated once per device, stream-ordered use.
-struct StkScratch {
-  float* ws;
-  int* counters;
-  int sms;
-};
-static StkScratch stk_scratch(const Tensor& like) {
-  // leaked on purpose: destroying CUDA tensors from static destructors can outlive the allocator
-  static Tensor* ws = new Tensor[64];
-  static Tensor* counters = new Tensor[64];
-  static int sms_k[64] = {};
-  const int dev = like.get_device();
-  TORCH_CHECK(dev >= 0 && dev < 64);
-  if (sms_k[dev] == 0) cudaDeviceGetAttribute(&sms_k[dev], cudaDevAttrMultiProcessorCount, dev);
-  if (!ws[dev].defined()) {
-    ws[dev] = torch::empty({(int64_t)(b200::gemm_streamk_workspace_bytes(sms_k[dev]) / 4)},
-                           like.options().dtype(at::kFloat));
-    counters[dev] = torch::zeros({2 * (int64_t)b200::gemm_streamk_max_tiles()}, like.options().dtype(at::kInt));
-  }
-  return {ws[dev].data_ptr<float>(), counters[dev].data_ptr<int>(), sms_k[dev]};
-}
-
-void gemm(Tensor& out, const Tensor& a, const Tensor& w, const optional<Tensor>& bias,
-          const optional<Tensor>& residual, int64_t force_bn, int64_t epi) {
-  TORCH_CHECK(a.dim() == 2 && w.dim() == 2 && out.dim() == 2, "gemm expects 2-D tensors");
-  TORCH_CHECK(a.stride(1) == 1 && w.stride(1) == 1 && out.stride(1) == 1, "inner dims must be contiguous");
-  const int M = a.size(0), K = a.size(1), N = w.size(0);
-  TORCH_CHECK(w.size(1) == K && out.size(0) == M && out.size(1) == (epi == 1 ? N / 2 : N), "gemm shape mismatch");
-  TORCH_CHECK(epi == 0 || (!residual.has_value() && N % 16 == 0), "gated epilogue: no residual, N % 16 == 0");
-  TORCH_CHECK(K % 8 == 0 && a.stride(0) % 8 == 0 && w.stride(0) % 8 == 0 && out.stride(0) % 8 == 0,
-              "gemm: K and row pitches must be multiples of 8 elements");
-  TORCH_CHECK(a.scalar_type() == w.scalar_type() && a.scalar_type() == out.scalar_type(), "gemm dtype mismatch");
-  int ldr = 0;
-  if (residual.has_value()) {
-    TORCH_CHECK(residual->stride(1) == 1 && residual->size(0) == M && residual->size(1) == N);
-    ldr = residual->stride(0);
-  }
-  const c10::cuda::CUDAGuard guard(a.device());
-  // CTA-pair (cta_group::2) kernel for large problems: at least one 256 x 256 tile per pair of SMs.
-  static const bool pair_default = [] {
-    const char* e = std::getenv("B200_GEMM_PAIR");
-    return e == nullptr || std::atoi(e) != 0;
-  }();
-  const int64_t pair_tiles = ((M + 255) / 256) * (int64_t)((N + 255) / 256);
-  // (a full 256-token decode batch against a wide weight, e.g. gate_up, already gives every CTA pair a tile)
-  if (force_bn == 512 || (force_bn == 0 && pair_default && ((M >= 512 && pair_tiles >= 64) ||
-                                                             (M >= 256 && pair_tiles >= 96)))) {
-    b200::gemm_tn_pair(a.data_ptr(), w.data_ptr(), out.data_ptr(), ptr(bias), ptr(residual), M, N, K, a.stride(0),
-                       w.stride(0), out.stride(0), ldr, dtype16(a), cur_stream(), status_ptr(a), (int)epi);
-    return;
-  }
-  // stream-K over CTA pairs for skinny problems: decode batches and narrow tensor-parallel shards (force_bn 2000
-  // pins it).  Its scratch (partial tiles + arrival counters) is allocated once per device and stream-ordered
-  // use is assumed, like every other op of this library.
-  static const bool streamk_default = [] {
-    const char* e = std::getenv("B200_GEMM_STREAMK");
-    return e == nullptr || std::atoi(e) != 0;
-  }();
-  {
-    StkScratch sk = stk_scratch(a);
-    const int64_t tiles = ((M + 255) / 256) * (int64_t)((N + 255) / 256);
-    // measured inside replayed graphs: with up to 64 tokens the partial tiles are small and streaming over all SMs
-    // wins; at 256 tokens the 128 KB partials make the fix-up cost more than the balanced stream saves
-    if (force_bn == 2000 || (force_bn == 0 && streamk_default && M <= 64 && K >= 1024 && tiles <= 2 * sk.sms)) {
-      const int rc = b200::gemm_tn_streamk(a.data_ptr(), w.data_ptr(), out.data_ptr(), ptr(bias), ptr(residual), M, N,
-                                           K, a.stride(0), w.stride(0), out.stride(0), ldr, dtype16(a), cur_stream(),
-                                           status_ptr(a), (int)epi, sk.ws, sk.counters, sk.sms);
-      if (rc == 0) return;
-      TORCH_CHECK(force_bn != 2000, "gemm: shape outside the stream-K kernel's scratch");
-    }
-  }
-  // cluster split-K for medium M with too few tiles to cover the GPU (force_bn 1002 / 1004 pins the split count)
-  static const bool splitk_default = [] {
-    const char* e = std::getenv("B200_GEMM_SPLITK");
-    return e == nullptr || std::atoi(e) != 0;
-  }();
-  static int sms = 0;
-  if (sms == 0) cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, a.get_device());
-  int splits = 1;
-  if (force_bn == 1002 || force_bn == 1004) splits = (int)force_bn - 1000;
-  else if (force_bn == 0 && splitk_default && M > 64 && M <= 1024) splits = b200::gemm_splitk_choice(M, N, K, sms);
-  if (splits > 1) {
-    b200::gemm_tn_splitk(a.data_ptr(), w.data_ptr(), out.data_ptr(), ptr(bias), ptr(residual), M, N, K, a.stride(0),
-                         w.stride(0), out.stride(0), ldr, dtype16(a), cur_stream(), status_ptr(a), (int)epi, splits);
-    return;
-  }
-  b200::gemm_tn(a.data_ptr(), w.data_ptr(), out.data_ptr(), ptr(bias), ptr(residual), M, N, K, a.stride(0),
-                w.stride(0), out.stride(0), ldr, dtype16(a), cur_stream(), status_ptr(a), (int)force_bn, (int)epi);
-}
 
 // ------------------------------------------------------------------ norms
 void rms_norm(Tensor& out, const Tensor& x, const Tensor& weight, double eps, bool gemma) {
@@ -315,174 +182,9 @@ void paged_attention_decode(Tensor& out, const Tensor& q, const Tensor& kv_cache
   TORCH_CHECK(rc == 0, "paged_attention_decode: unsupported head_dim ", D);
 }
 
-void attention_prefill(Tensor& out, const Tensor& q, const Tensor& k_src, const optional<Tensor>& v_src,
-                       const optional<Tensor>& block_table, const optional<Tensor>& seq_lens,
-                       const Tensor& query_start_loc, const optional<Tensor>& kv_start_loc, double scale,
-                       int64_t window, double softcap, const optional<Tensor>& sinks,
-                       const optional<Tensor>& lse_out, int64_t batch, int64_t max_q_len, bool causal,
-                       const optional<Tensor>& alibi_slopes) {
-  TORCH_CHECK(q.dim() == 3 && q.stride(2) == 1 && q.stride(1) == q.size(2));
-  b200::PrefillParams p{};
-  p.alibi_slopes = ptr<float>(alibi_slopes);
-  const int T = q.size(0), Hq = q.size(1), DQK = q.size(2);
-  const bool paged = block_table.has_value();
-  int Hkv, DV;
-  int64_t total_kv = 0, ks = 0, vs = 0;
-  const void* kptr = k_src.data_ptr();
-  const void* vptr = nullptr;
-  if (paged) {
-    TORCH_CHECK(k_src.dim() == 5 && k_src.is_contiguous(), "paged mode expects the [nb,2,bs,Hkv,D] cache");
-    TORCH_CHECK(k_src.scalar_type() == q.scalar_type(), "tcgen05 prefill needs a 16-bit cache of the query dtype");
-    Hkv = k_src.size(3);
-    DV = k_src.size(4);
-    p.block_size = k_src.size(2);
-    p.num_blocks = k_src.size(0);
-    p.max_blocks = block_table->size(1);
-    p.block_table = block_table->data_ptr<int>();
-    p.seq_lens = seq_lens->data_ptr<int>();
-    TORCH_CHECK(p.block_size % 16 == 0 && (128 % p.block_size == 0 || p.block_size % 128 == 0),
-                "block_size must be 16/32/64 or a multiple of 128");
-    vptr = kptr;
-  } else {
-    TORCH_CHECK(v_src.has_value() && kv_start_loc.has_value());
-    TORCH_CHECK(k_src.dim() == 3 && k_src.stride(2) == 1 && k_src.stride(1) == k_src.size(2));
-    TORCH_CHECK(v_src->dim() == 3 && v_src->stride(2) == 1 && v_src->stride(1) == v_src->size(2));
-    Hkv = k_src.size(1);
-    DV = v_src->size(2);
-    total_kv = k_src.size(0);
-    ks = k_src.stride(0);
-    vs = v_src->stride(0);
-    vptr = v_src->data_ptr();
-    p.kv_start_loc = kv_start_loc->data_ptr<int>();
-  }
-  p.out = out.data_ptr();
-  p.lse_out = ptr<float>(lse_out);
-  p.query_start_loc = query_start_loc.data_ptr<int>();
-  p.sinks = ptr<float>(sinks);
-  p.num_q_heads = Hq;
-  p.num_kv_heads = Hkv;
-  const int g = Hq / Hkv;
-  p.gp = (128 % g == 0) ? g : 1;
-  p.total_q = T;
-  p.scale = (float)scale;
-  p.softcap = (float)softcap;
-  p.window = (int)window;
-  p.causal = causal;
-  p.paged = paged;
-  p.status = reinterpret_cast<b200::StatusWord*>(status_ptr(q));
-  TORCH_CHECK(out.is_contiguous() && out.size(-1) == DV);
-  TORCH_CHECK(q.stride(0) % 8 == 0, "q token stride must be a multiple of 8 elements");
-  const c10::cuda::CUDAGuard guard(q.device());
-  // B200_ATTN_PREFILL_SINGLE=1 selects the one-tile-per-CTA kernel (P through shared memory)
-  static const bool single_tile = [] {
-    const char* e = std::getenv("B200_ATTN_PREFILL_SINGLE");
-    return e != nullptr && std::atoi(e) != 0;
-  }();
-  const int rc = single_tile
-                     ? b200::attention_prefill(p, q.data_ptr(), q.stride(0), kptr, vptr, ks, vs, total_kv, DQK, DV,
-                                               dtype16(q), batch, max_q_len, cur_stream())
-                     : b200::attention_prefill_pp(p, q.data_ptr(), q.stride(0), kptr, vptr, ks, vs, total_kv, DQK, DV,
-                                                  dtype16(q), batch, max_q_len, cur_stream());
-  TORCH_CHECK(rc == 0, "attention_prefill: unsupported head dims ", DQK, "/", DV);
-}
-
-// ------------------------------------------------------------------ sampling
-void argmax(Tensor& out, const Tensor& logits) {
-  TORCH_CHECK(logits.dim() == 2 && logits.stride(1) == 1 && out.scalar_type() == at::kLong);
-  const c10::cuda::CUDAGuard guard(logits.device());
-  b200::argmax(out.data_ptr<int64_t>(), logits.data_ptr(), logits.size(0), logits.size(1), logits.stride(0),
-               dtype_code(logits), cur_stream());
-}
-void sample(Tensor& out, const Tensor& logits, const Tensor& temperature, const optional<Tensor>& top_k,
-            const optional<Tensor>& top_p, const optional<Tensor>& min_p, const Tensor& uniform) {
-  TORCH_CHECK(logits.dim() == 2 && logits.stride(1) == 1 && out.scalar_type() == at::kLong);
-  const c10::cuda::CUDAGuard guard(logits.device());
-  b200::sample(out.data_ptr<int64_t>(), logits.data_ptr(), logits.size(0), logits.size(1), logits.stride(0),
-               temperature.data_ptr<float>(), ptr<int>(top_k), ptr<float>(top_p), ptr<float>(min_p),
-               uniform.data_ptr<float>(), dtype_code(logits), cur_stream());
-}
-void apply_penalties(Tensor& logits, const optional<Tensor>& prompt_mask, const optional<Tensor>& output_counts,
-                     const optional<Tensor>& rep, const optional<Tensor>& presence,
-                     const optional<Tensor>& frequency) {
-  const c10::cuda::CUDAGuard guard(logits.device());
-  b200::apply_penalties(logits.data_ptr(), ptr<int>(prompt_mask), ptr<int>(output_counts), ptr<float>(rep),
-                        ptr<float>(presence), ptr<float>(frequency), logits.size(0), logits.size(1), logits.stride(0),
-                        dtype_code(logits), cur_stream());
-}
-void advance_step(Tensor& input_ids, Tensor& positions, Tensor& seq_lens, Tensor& slot_mapping, const Tensor& sampled,
-                  const Tensor& block_table, int64_t block_size, int64_t batch, const optional<Tensor>& token_log,
-                  int64_t log_col) {
-  const c10::cuda::CUDAGuard guard(input_ids.device());
-  b200::advance_step(input_ids.data_ptr<int64_t>(), positions.data_ptr<int64_t>(), seq_lens.data_ptr<int>(),
-                     slot_mapping.data_ptr<int64_t>(), sampled.data_ptr<int64_t>(), block_table.data_ptr<int>(),
-                     block_table.size(1), block_size, batch, ptr<int64_t>(token_log), log_col,
-                     token_log.has_value() ? token_log->stride(0) : 0, cur_stream());
-}
-void embedding(Tensor& out, const Tensor& table, const Tensor& ids, int64_t vocab_start) {
-  TORCH_CHECK(table.is_contiguous() && out.is_contiguous() && ids.scalar_type() == at::kLong);
-  TORCH_CHECK(table.size(1) % 8 == 0);
-  const c10::cuda::CUDAGuard guard(table.device());
-  b200::embedding(out.data_ptr(), table.data_ptr(), ids.data_ptr<int64_t>(), ids.numel(), table.size(1), table.size(0),
-                  vocab_start, dtype16(table), cur_stream());
-}
 
 
-// ------------------------------------------------------------------ MoE
-void topk_gating(Tensor& weights, Tensor& ids, const Tensor& gating, const optional<Tensor>& bias, int64_t mode,
-                 bool renorm, double scale) {
-  TORCH_CHECK(gating.dim() == 2 && gating.is_contiguous() && gating.size(1) <= 1024 && ids.size(1) <= 32);
-  TORCH_CHECK(weights.scalar_type() == at::kFloat && ids.scalar_type() == at::kInt);
-  const c10::cuda::CUDAGuard guard(gating.device());
-  b200::topk_gating(weights.data_ptr<float>(), ids.data_ptr<int>(), gating.data_ptr(), ptr<float>(bias),
-                    gating.size(0), gating.size(1), ids.size(1), mode, renorm, (float)scale, dtype_code(gating),
-                    cur_stream());
-}
-void grouped_topk(Tensor& weights, Tensor& ids, const Tensor& gating, const optional<Tensor>& bias, int64_t n_group,
-                  int64_t topk_group, bool sigmoid, bool renorm, double scale) {
-  TORCH_CHECK(gating.dim() == 2 && gating.is_contiguous() && gating.size(1) <= 1024 && ids.size(1) <= 32);
-  TORCH_CHECK(n_group <= 32 && gating.size(1) % n_group == 0);
-  const c10::cuda::CUDAGuard guard(gating.device());
-  b200::grouped_topk(weights.data_ptr<float>(), ids.data_ptr<int>(), gating.data_ptr(), ptr<float>(bias),
-                     gating.size(0), gating.size(1), ids.size(1), n_group, topk_group, sigmoid, renorm, (float)scale,
-                     dtype_code(gating), cur_stream());
-}
-void moe_align(Tensor& sorted_ids, Tensor& block_expert, Tensor& total_padded, const optional<Tensor>& inv_pos,
-               const Tensor& topk_ids, const optional<Tensor>& expert_map, int64_t experts, int64_t block) {
-  TORCH_CHECK(topk_ids.scalar_type() == at::kInt && topk_ids.is_contiguous());
-  TORCH_CHECK(sorted_ids.numel() % block == 0 && block_expert.numel() >= sorted_ids.numel() / block);
-  const c10::cuda::CUDAGuard guard(topk_ids.device());
-  b200::moe_align(sorted_ids.data_ptr<int>(), block_expert.data_ptr<int>(), total_padded.data_ptr<int>(),
-                  ptr<int>(inv_pos), topk_ids.data_ptr<int>(), ptr<int>(expert_map), topk_ids.numel(), experts, block,
-                  sorted_ids.numel(), cur_stream());
-}
-void moe_gather(Tensor& out, const Tensor& x, const Tensor& sorted_ids, const Tensor& total_padded, int64_t topk) {
-  TORCH_CHECK(x.is_contiguous() && out.is_contiguous() && x.size(1) % 8 == 0);
-  const c10::cuda::CUDAGuard guard(x.device());
-  b200::moe_gather(out.data_ptr(), x.data_ptr(), sorted_ids.data_ptr<int>(), total_padded.data_ptr<int>(),
-                   out.size(0), x.size(0) * topk, topk, x.size(1), dtype16(x), cur_stream());
-}
-void moe_combine(Tensor& out, const Tensor& y, const Tensor& weights, const Tensor& inv_pos,
-                 const optional<Tensor>& shared) {
-  TORCH_CHECK(y.is_contiguous() && out.is_contiguous() && weights.scalar_type() == at::kFloat);
-  const c10::cuda::CUDAGuard guard(y.device());
-  b200::moe_combine(out.data_ptr(), y.data_ptr(), weights.data_ptr<float>(), inv_pos.data_ptr<int>(), ptr(shared),
-                    out.size(0), weights.size(1), out.size(1), dtype16(y), cur_stream());
-}
-void moe_sum(Tensor& out, const Tensor& in) {
-  TORCH_CHECK(in.dim() == 3 && in.is_contiguous() && out.is_contiguous());
-  const c10::cuda::CUDAGuard guard(in.device());
-  b200::moe_sum(out.data_ptr(), in.data_ptr(), in.size(0), in.size(1), in.size(2), dtype16(in), cur_stream());
-}
-void gemm_grouped(Tensor& out, const Tensor& a, const Tensor& w, const Tensor& block_expert,
-                  const Tensor& total_padded, int64_t epi) {
-  TORCH_CHECK(a.dim() == 2 && w.dim() == 3 && a.stride(1) == 1 && w.is_contiguous() && out.stride(1) == 1);
-  TORCH_CHECK(a.size(0) % 128 == 0 && a.size(1) == w.size(2) && a.size(1) % 8 == 0 && a.stride(0) % 8 == 0);
-  TORCH_CHECK(out.size(0) == a.size(0) && out.size(1) == (epi == 1 ? w.size(1) / 2 : w.size(1)));
-  const c10::cuda::CUDAGuard guard(a.device());
-  b200::gemm_grouped(a.data_ptr(), a.size(0), a.stride(0), w.data_ptr(), w.size(0), w.size(1), w.size(2),
-                     out.data_ptr(), out.stride(0), block_expert.data_ptr<int>(), total_padded.data_ptr<int>(), epi,
-                     dtype16(a), cur_stream(), status_ptr(a));
-}
+
 
 // ------------------------------------------------------------------ quantisation
 void per_token_group_quant(Tensor& q, Tensor& scales, const Tensor& x, int64_t group, bool ue8m0, bool col_major,
@@ -587,44 +289,6 @@ void wna16_gemm(Tensor& out, const Tensor& a, const Tensor& q, const Tensor& sca
                    status_ptr(a));
 }
 
-// ------------------------------------------------------------------ MLA
-void mla_decode(Tensor& out, const Tensor& q, const Tensor& cache, const Tensor& block_table, const Tensor& seq_lens,
-                const optional<Tensor>& query_start_loc, const optional<Tensor>& topk_indices, double scale,
-                const optional<Tensor>& lse_out, const optional<Tensor>& workspace, int64_t num_splits, int64_t impl) {
-  TORCH_CHECK(q.dim() == 3 && q.size(2) == 576 && q.stride(2) == 1 && q.stride(1) == 576);
-  TORCH_CHECK(cache.is_contiguous() && cache.dim() == 3 && out.is_contiguous() && out.size(2) == 512);
-  const bool rec = cache.scalar_type() == at::kByte;
-  TORCH_CHECK(rec ? cache.size(2) == 656 : (cache.size(2) == 576 && cache.scalar_type() == q.scalar_type()));
-  b200::MlaDecodeParams p{};
-  p.out = out.data_ptr();
-  p.lse_out = ptr<float>(lse_out);
-  p.q = q.data_ptr();
-  p.q_stride = q.stride(0);
-  p.cache = cache.data_ptr();
-  p.block_table = block_table.data_ptr<int>();
-  p.seq_lens = seq_lens.data_ptr<int>();
-  p.query_start_loc = ptr<int>(query_start_loc);
-  p.topk_indices = ptr<int>(topk_indices);
-  p.topk = topk_indices.has_value() ? topk_indices->size(1) : 0;
-  p.num_heads = q.size(1);
-  p.block_size = cache.size(1);
-  p.num_blocks = cache.size(0);
-  p.max_blocks = block_table.size(1);
-  p.num_splits = std::max<int64_t>(1, num_splits);
-  p.total_tokens = q.size(0);
-  p.batch = seq_lens.size(0);
-  p.scale = (float)scale;
-  if (p.num_splits > 1) {
-    const int64_t need = p.num_splits * (int64_t)p.total_tokens * p.num_heads * 513;
-    TORCH_CHECK(workspace.has_value() && workspace->numel() >= need, "mla_decode workspace too small");
-    p.part_out = workspace->data_ptr<float>();
-    p.part_lse = p.part_out + p.num_splits * (int64_t)p.total_tokens * p.num_heads * 512;
-  }
-  p.status = reinterpret_cast<b200::StatusWord*>(status_ptr(q));
-  const c10::cuda::CUDAGuard guard(q.device());
-  const int rc = b200::mla_decode(p, rec, dtype16(q), cur_stream(), (int)impl);
-  TORCH_CHECK(rc == 0, "mla_decode: the tcgen05 kernel was asked for (impl = 2) but does not serve this call");
-}
 
 // ------------------------------------------------------------------ DSA indexer
 void indexer_logits(Tensor& logits, const Tensor& q, const Tensor& w, const Tensor& cache, const Tensor& block_table,
@@ -920,16 +584,6 @@ void permute_cols(Tensor& out, const Tensor& a, const Tensor& perm) {
                      dtype16(a), cur_stream());
 }
 
-void gather_mla_cache(Tensor& dst, const Tensor& cache, const Tensor& block_table, const Tensor& cu_seq_lens,
-                      const optional<Tensor>& seq_starts) {
-  TORCH_CHECK(dst.is_contiguous() && dst.size(1) == 576 && cache.is_contiguous() && cache.dim() == 3);
-  const bool rec = cache.scalar_type() == at::kByte;
-  TORCH_CHECK(rec ? cache.size(2) == 656 : (cache.size(2) == 576 && cache.scalar_type() == dst.scalar_type()));
-  const c10::cuda::CUDAGuard guard(dst.device());
-  b200::gather_mla_cache(dst.data_ptr(), cache.data_ptr(), block_table.data_ptr<int>(), cu_seq_lens.data_ptr<int>(),
-                         ptr<int>(seq_starts), cu_seq_lens.numel() - 1, block_table.size(1), cache.size(1), dst.size(0),
-                         rec, dtype16(dst), cur_stream());
-}
 
 void gather_indexer_k(Tensor& dst_k, Tensor& dst_s, const Tensor& cache, const Tensor& block_table,
                       const Tensor& cu_seq_lens, int64_t block_size) {
@@ -1076,33 +730,6 @@ void gdn_recurrent(Tensor& out, Tensor& state, const Tensor& q, const Tensor& k,
   TORCH_CHECK(rc == 0, "gdn_recurrent: head sizes must be 128 and value heads a multiple of q/k heads");
 }
 
-// x [T, C] (row pitch free), w [C, K], state [slots, K-1, C] (in / out), all of one dtype (bf16 / fp16 / fp32)
-void causal_conv1d(Tensor& out, const Tensor& x, const Tensor& w, const optional<Tensor>& bias,
-                   const optional<Tensor>& state, const Tensor& query_start_loc, const optional<Tensor>& state_idx,
-                   const optional<Tensor>& has_initial, bool silu) {
-  TORCH_CHECK(x.dim() == 2 && x.stride(1) == 1 && out.is_contiguous() && out.sizes() == x.sizes() &&
-              out.scalar_type() == x.scalar_type());
-  const int64_t T = x.size(0), C = x.size(1), K = w.size(1);
-  TORCH_CHECK(w.dim() == 2 && w.size(0) == C && w.is_contiguous() && w.scalar_type() == x.scalar_type());
-  if (bias.has_value()) TORCH_CHECK(bias->is_contiguous() && bias->numel() == C && bias->scalar_type() == x.scalar_type());
-  TORCH_CHECK(query_start_loc.scalar_type() == at::kInt && query_start_loc.is_contiguous());
-  const int64_t B = query_start_loc.numel() - 1;
-  if (state.has_value()) {
-    TORCH_CHECK(state_idx.has_value(), "a carry needs state indices");
-    TORCH_CHECK(state->is_contiguous() && state->dim() == 3 && state->size(1) == K - 1 && state->size(2) == C &&
-                state->scalar_type() == x.scalar_type());
-  }
-  if (state_idx.has_value()) TORCH_CHECK(state_idx->scalar_type() == at::kInt && state_idx->numel() >= B);
-  if (has_initial.has_value()) TORCH_CHECK(has_initial->scalar_type() == at::kInt && has_initial->numel() >= B);
-  const c10::cuda::CUDAGuard guard(x.device());
-  const int rc = b200::causal_conv1d(out.data_ptr(), x.data_ptr(), x.stride(0), w.data_ptr(),
-                                     bias.has_value() ? bias->data_ptr() : nullptr,
-                                     state.has_value() ? state->data_ptr() : nullptr, query_start_loc.data_ptr<int>(),
-                                     state_idx.has_value() ? state_idx->data_ptr<int>() : nullptr,
-                                     has_initial.has_value() ? has_initial->data_ptr<int>() : nullptr, (int)B, (int)T,
-                                     (int)C, (int)K, silu ? 1 : 0, dtype_code(x), cur_stream());
-  TORCH_CHECK(rc == 0, "causal_conv1d: kernel width must be 2..8");
-}
 
 // TurboQuant cache: uint8 [blocks, block_size, kv_heads, slot_bytes]; k, v [T, kv_heads * 128] (any row pitch)
 int64_t tq_slot_bytes(int64_t kbits, int64_t vbits) { return b200::tq_slot_bytes((int)kbits, (int)vbits); }
@@ -1347,12 +974,11 @@ void gather_rows(Tensor& dst, const Tensor& src, const Tensor& idx, const Tensor
 
 }  // namespace
 
-TORCH_LIBRARY(b200, m) {
+TORCH_LIBRARY_FRAGMENT(b200, m) {
   m.def("moe_a2a_dispatch(Tensor x, Tensor topk_ids, Tensor topk_w, Tensor ptrs, int ep, int rank, int experts_per_rank, int cap, bool quant, Tensor(a!) local_sync, int wait_cycles) -> ()", &moe_a2a_dispatch);
   m.def("moe_a2a_combine(Tensor(a!) out, Tensor y, Tensor topk_ids, Tensor? shared_out, Tensor ptrs, int ep, int rank, int experts_per_rank, int cap, Tensor(b!) local_sync, int wait_cycles) -> ()", &moe_a2a_combine);
   m.def("v4_qnorm_rope_kv_insert(Tensor(a!) q_out, Tensor(b!) cache, Tensor q, Tensor kv, Tensor slot_mapping, Tensor positions, Tensor cos_sin, float eps, int block_size) -> ()", &v4_qnorm_rope_kv_insert);
   m.def("v4_gather_dequant(Tensor(a!) dst, Tensor cache, Tensor slots, int block_size) -> ()", &v4_gather_dequant);
-  m.def("causal_conv1d(Tensor(a!) out, Tensor x, Tensor w, Tensor? bias, Tensor(b!)? state, Tensor query_start_loc, Tensor? state_idx, Tensor? has_initial, bool silu) -> ()", &causal_conv1d);
   m.def("gdn_recurrent(Tensor(a!) out, Tensor(b!) state, Tensor q, Tensor k, Tensor v, Tensor g, Tensor beta, Tensor query_start_loc, Tensor? state_idx, Tensor? has_initial, float scale, bool l2norm) -> ()", &gdn_recurrent);
   m.def("tq_slot_bytes(int kbits, int vbits) -> int", &tq_slot_bytes);
   m.def("tq_store(Tensor(a!) cache, Tensor k, Tensor v, Tensor slot_mapping, int kbits, int vbits, bool nc) -> ()", &tq_store);
@@ -1371,19 +997,10 @@ TORCH_LIBRARY(b200, m) {
   m.def("mla_rope_and_cache(Tensor(a!) q_pe, Tensor(b!) k_pe, Tensor kv_c, Tensor(c!) cache, Tensor cos_sin, Tensor positions, Tensor slot_mapping, bool is_neox) -> ()", &mla_rope_and_cache);
   m.def("concat_mla_q(Tensor(a!) out, Tensor nope, Tensor pe) -> ()", &concat_mla_q);
   m.def("permute_cols(Tensor(a!) out, Tensor a, Tensor perm) -> ()", &permute_cols);
-  m.def("gather_mla_cache(Tensor(a!) dst, Tensor cache, Tensor block_table, Tensor cu_seq_lens, Tensor? seq_starts) -> ()", &gather_mla_cache);
   m.def("gather_indexer_k(Tensor(a!) dst_k, Tensor(b!) dst_s, Tensor cache, Tensor block_table, Tensor cu_seq_lens, int block_size) -> ()", &gather_indexer_k);
   m.def("selective_scan(Tensor(a!) out, Tensor u, Tensor delta, Tensor A, Tensor B, Tensor C, Tensor? D, Tensor? z, Tensor? delta_bias, bool delta_softplus, Tensor(b!) state, Tensor? query_start_loc, Tensor? cache_indices, Tensor? has_initial_state, int pad_slot) -> ()", &selective_scan);
   m.def("p2p_copy(int dst_ptr, Tensor src, int ctas, int mode) -> ()", &p2p_copy);
   m.def("gather_rows(Tensor(a!) dst, Tensor src, Tensor idx, Tensor count, int div) -> ()", &gather_rows);
-  m.def("get_status(int device) -> Tensor", &get_status);
-  m.def("topk_gating(Tensor(a!) weights, Tensor(b!) ids, Tensor gating, Tensor? bias, int mode, bool renorm, float scale) -> ()", &topk_gating);
-  m.def("grouped_topk(Tensor(a!) weights, Tensor(b!) ids, Tensor gating, Tensor? bias, int n_group, int topk_group, bool sigmoid, bool renorm, float scale) -> ()", &grouped_topk);
-  m.def("moe_align(Tensor(a!) sorted_ids, Tensor(b!) block_expert, Tensor(c!) total_padded, Tensor(d!)? inv_pos, Tensor topk_ids, Tensor? expert_map, int experts, int block) -> ()", &moe_align);
-  m.def("moe_gather(Tensor(a!) out, Tensor x, Tensor sorted_ids, Tensor total_padded, int topk) -> ()", &moe_gather);
-  m.def("moe_combine(Tensor(a!) out, Tensor y, Tensor weights, Tensor inv_pos, Tensor? shared) -> ()", &moe_combine);
-  m.def("moe_sum(Tensor(a!) out, Tensor inp) -> ()", &moe_sum);
-  m.def("gemm_grouped(Tensor(a!) out, Tensor a, Tensor w, Tensor block_expert, Tensor total_padded, int epi) -> ()", &gemm_grouped);
   m.def("per_token_group_quant(Tensor(a!) q, Tensor(b!) scales, Tensor x, int group, bool ue8m0, bool col_major, float eps) -> ()", &per_token_group_quant);
   m.def("scaled_fp8_quant(Tensor(a!) q, Tensor(b!) scale, Tensor x, int mode, float scale_ub) -> ()", &scaled_fp8_quant);
   m.def("scaled_int8_quant(Tensor(a!) q, Tensor(b!) scale, Tensor(c!)? azp, Tensor x, int mode) -> ()", &scaled_int8_quant);
@@ -1391,7 +1008,6 @@ TORCH_LIBRARY(b200, m) {
   m.def("gemm_fp8_blockscale(Tensor(a!) out, Tensor a, Tensor a_scale, Tensor w, Tensor w_scale, Tensor? block_expert, Tensor? total_padded) -> ()", &gemm_fp8_blockscale);
   m.def("scaled_mm(Tensor(a!) out, Tensor a, Tensor w, Tensor a_scale, Tensor w_scale, Tensor? azp, Tensor? azp_adj, Tensor? bias, Tensor? block_expert, Tensor? total_padded) -> ()", &scaled_mm);
   m.def("wna16_gemm(Tensor(a!) out, Tensor a, Tensor q, Tensor scales, Tensor? zeros, int bits, int group, Tensor? bias, Tensor? block_expert, Tensor? total_padded, int token_tile, int epi) -> ()", &wna16_gemm);
-  m.def("mla_decode(Tensor(a!) out, Tensor q, Tensor cache, Tensor block_table, Tensor seq_lens, Tensor? query_start_loc, Tensor? topk_indices, float scale, Tensor(b!)? lse_out, Tensor(c!)? workspace, int num_splits, int impl=1) -> ()", &mla_decode);
   m.def("indexer_logits(Tensor(a!) logits, Tensor q, Tensor w, Tensor cache, Tensor block_table, Tensor seq_lens, Tensor query_start_loc, int block_size, int max_len, bool int8, int max_query_len, int impl) -> ()", &indexer_logits);
   m.def("topk_per_row(Tensor(a!) out, Tensor x, Tensor? row_len, int cols) -> ()", &topk_per_row);
   m.def("symm_alloc(int nbytes, int device) -> (Tensor, Tensor)", &symm_alloc);
@@ -1416,7 +1032,6 @@ TORCH_LIBRARY(b200, m) {
       "int rank, int rows_per_rank, int rows_cap, int rb_cap, Tensor(b!) local_sync, bool add_residual, "
       "int wait_cycles) -> ()",
       &gemm_ar_norm);
-  m.def("gemm(Tensor(a!) out, Tensor a, Tensor w, Tensor? bias, Tensor? residual, int force_bn, int epi) -> ()", &gemm);
   m.def("rms_norm(Tensor(a!) out, Tensor x, Tensor weight, float eps, bool gemma) -> ()", &rms_norm);
   m.def("fused_add_rms_norm(Tensor(a!) x, Tensor(b!) residual, Tensor weight, float eps, bool gemma) -> ()",
         &fused_add_rms_norm);
@@ -1448,24 +1063,5 @@ TORCH_LIBRARY(b200, m) {
       "Tensor(b!)? lse_out, Tensor(c!)? workspace, int num_splits, int batch, int max_q_len, float k_scale, "
       "float v_scale, bool causal, Tensor? alibi_slopes=None) -> ()",
       &paged_attention_decode);
-  m.def(
-      "attention_prefill(Tensor(a!) out, Tensor q, Tensor k_src, Tensor? v_src, Tensor? block_table, "
-      "Tensor? seq_lens, Tensor query_start_loc, Tensor? kv_start_loc, float scale, int window, float softcap, "
-      "Tensor? sinks, Tensor(b!)? lse_out, int batch, int max_q_len, bool causal, Tensor? alibi_slopes=None) -> ()",
-      &attention_prefill);
-  m.def("argmax(Tensor(a!) out, Tensor logits) -> ()", &argmax);
-  m.def(
-      "sample(Tensor(a!) out, Tensor logits, Tensor temperature, Tensor? top_k, Tensor? top_p, Tensor? min_p, "
-      "Tensor uniform) -> ()",
-      &sample);
-  m.def(
-      "apply_penalties(Tensor(a!) logits, Tensor? prompt_mask, Tensor? output_counts, Tensor? rep, Tensor? presence, "
-      "Tensor? frequency) -> ()",
-      &apply_penalties);
-  m.def(
-      "advance_step(Tensor(a!) input_ids, Tensor(b!) positions, Tensor(c!) seq_lens, Tensor(d!) slot_mapping, "
-      "Tensor sampled, Tensor block_table, int block_size, int batch, Tensor(e!)? token_log, int log_col) -> ()",
-      &advance_step);
-  m.def("embedding(Tensor(a!) out, Tensor table, Tensor ids, int vocab_start) -> ()", &embedding);
   m.def("weak_ref_tensor(Tensor input) -> Tensor", &weak_ref_tensor);
 }

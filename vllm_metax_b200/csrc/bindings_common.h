@@ -1,0 +1,73 @@
+// Helpers shared by the binding units: current stream, dtype codes, optional pointers, the per-device status word.
+#pragma once
+#include <ATen/cuda/CUDAContext.h>
+#include <c10/cuda/CUDAGuard.h>
+#include <torch/library.h>
+#include <torch/types.h>
+
+#include <cstdlib>
+#include <cstring>
+#include <tuple>
+
+#include "comm_params.h"
+#include "ops.h"
+
+namespace b200_bind {
+
+using at::Tensor;
+using c10::optional;
+
+inline cudaStream_t cur_stream() { return at::cuda::getCurrentCUDAStream().stream(); }
+
+inline int dtype_code(const Tensor& t) {
+  switch (t.scalar_type()) {
+    case at::kBFloat16: return 0;
+    case at::kHalf: return 1;
+    case at::kFloat: return 2;
+    default: TORCH_CHECK(false, "unsupported dtype ", t.scalar_type());
+  }
+}
+inline int dtype16(const Tensor& t) {
+  const int c = dtype_code(t);
+  TORCH_CHECK(c < 2, "expected a bf16 / fp16 tensor");
+  return c;
+}
+template <typename T = void>
+inline T* ptr(const optional<Tensor>& t) {
+  return t.has_value() && t->defined() ? reinterpret_cast<T*>(t->data_ptr()) : nullptr;
+}
+
+// One status word per device, zero-initialised on first use.
+inline Tensor& status_tensor(int device) {
+  static std::vector<Tensor> words(64);
+  if (!words[device].defined())
+    words[device] = torch::zeros({4}, torch::dtype(torch::kInt32).device(torch::kCUDA, device));
+  return words[device];
+}
+inline void* status_ptr(const Tensor& any) { return status_tensor(any.get_device()).data_ptr(); }
+
+inline Tensor get_status(int64_t device) { return status_tensor((int)device); }
+
+// Scratch of the stream-K GEMM (partial tiles + arrival counters): allocated once per device, stream-ordered use.
+struct StkScratch {
+  float* ws;
+  int* counters;
+  int sms;
+};
+inline StkScratch stk_scratch(const Tensor& like) {
+  // leaked on purpose: destroying CUDA tensors from static destructors can outlive the allocator
+  static Tensor* ws = new Tensor[64];
+  static Tensor* counters = new Tensor[64];
+  static int sms_k[64] = {};
+  const int dev = like.get_device();
+  TORCH_CHECK(dev >= 0 && dev < 64);
+  if (sms_k[dev] == 0) cudaDeviceGetAttribute(&sms_k[dev], cudaDevAttrMultiProcessorCount, dev);
+  if (!ws[dev].defined()) {
+    ws[dev] = torch::empty({(int64_t)(b200::gemm_streamk_workspace_bytes(sms_k[dev]) / 4)},
+                           like.options().dtype(at::kFloat));
+    counters[dev] = torch::zeros({2 * (int64_t)b200::gemm_streamk_max_tiles()}, like.options().dtype(at::kInt));
+  }
+  return {ws[dev].data_ptr<float>(), counters[dev].data_ptr<int>(), sms_k[dev]};
+}
+
+}  // namespace b200_bind

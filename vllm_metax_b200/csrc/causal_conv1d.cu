@@ -127,7 +127,7 @@ void launch(void* out, const void* x, int64_t x_stride, const void* w, const voi
   conv1d_fwd_kernel<T><<<grid, threads, 0, stream>>>((T*)out, (const T*)x, x_stride, (const T*)w, (const T*)bias,
                                                      (const T*)state, qsl, state_idx, has_init, batch, tokens, channels,
                                                      K, silu);
-  if (state != nullptr && state_idx != nullptr) {
+  if (state != nullptr && state_idx != nullptr && K > 1) {
     dim3 g2((channels + threads - 1) / threads, batch);
     conv1d_state_kernel<T><<<g2, threads, 0, stream>>>((T*)state, (const T*)x, x_stride, qsl, state_idx, has_init,
                                                        channels, K);
@@ -139,7 +139,7 @@ void launch(void* out, const void* x, int64_t x_stride, const void* w, const voi
 int causal_conv1d(void* out, const void* x, int64_t x_stride, const void* w, const void* bias, void* state,
                   const int* query_start_loc, const int* state_idx, const int* has_init, int batch, int tokens,
                   int channels, int K, int silu, int dtype, cudaStream_t stream) {
-  if (K < 2 || K > kMaxK || batch <= 0 || tokens <= 0) return K < 2 || K > kMaxK ? 1 : 0;
+  if (K < 1 || K > kMaxK || batch <= 0 || tokens <= 0) return K < 1 || K > kMaxK ? 1 : 0;
   if (dtype == 0)
     launch<__nv_bfloat16>(out, x, x_stride, w, bias, state, query_start_loc, state_idx, has_init, batch, tokens,
                           channels, K, silu, stream);

@@ -135,7 +135,7 @@ template <typename T>
 __global__ void gather_mla_cache_kernel(T* __restrict__ dst, const uint8_t* __restrict__ cache,
                                         const int* __restrict__ block_table, const int* __restrict__ cu_seq_lens,
                                         const int* __restrict__ seq_starts, int batch, int max_blocks, int block_size,
-                                        int records) {
+                                        int records, int row_elems) {
   const int gw = (blockIdx.x * blockDim.x + threadIdx.x) >> 5;
   const int lane = threadIdx.x & 31;
   const int total = cu_seq_lens[batch];
@@ -149,10 +149,10 @@ __global__ void gather_mla_cache_kernel(T* __restrict__ dst, const uint8_t* __re
   const int pos = gw - cu_seq_lens[b] + (seq_starts ? seq_starts[b] : 0);
   const int64_t blk = block_table[(size_t)b * max_blocks + pos / block_size];
   const int64_t slot = blk * block_size + pos % block_size;
-  T* out = dst + (size_t)gw * 576;
+  T* out = dst + (size_t)gw * row_elems;
   if (!records) {
-    const uint4* src = reinterpret_cast<const uint4*>(cache + (size_t)slot * 576 * sizeof(T));
-    for (int v = lane; v < 72; v += 32) reinterpret_cast<uint4*>(out)[v] = src[v];
+    const uint4* src = reinterpret_cast<const uint4*>(cache + (size_t)slot * row_elems * sizeof(T));
+    for (int v = lane; v < row_elems / 8; v += 32) reinterpret_cast<uint4*>(out)[v] = src[v];
     return;
   }
   const uint8_t* rec = cache + (size_t)slot * 656;
@@ -404,13 +404,13 @@ void permute_cols(void* out, const void* a, const int* perm, int64_t rows, int c
 
 void gather_mla_cache(void* dst, const void* cache, const int* block_table, const int* cu_seq_lens,
                       const int* seq_starts, int batch, int max_blocks, int block_size, int max_total, int records,
-                      int dtype, cudaStream_t stream) {
+                      int row_elems, int dtype, cudaStream_t stream) {
   if (max_total <= 0) return;
   const int blocks = ceil_div(max_total * 32, 256);
   if (dtype == 0)
-    gather_mla_cache_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>((__nv_bfloat16*)dst, (const uint8_t*)cache, block_table, cu_seq_lens, seq_starts, batch, max_blocks, block_size, records);
+    gather_mla_cache_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>((__nv_bfloat16*)dst, (const uint8_t*)cache, block_table, cu_seq_lens, seq_starts, batch, max_blocks, block_size, records, row_elems);
   else
-    gather_mla_cache_kernel<__half><<<blocks, 256, 0, stream>>>((__half*)dst, (const uint8_t*)cache, block_table, cu_seq_lens, seq_starts, batch, max_blocks, block_size, records);
+    gather_mla_cache_kernel<__half><<<blocks, 256, 0, stream>>>((__half*)dst, (const uint8_t*)cache, block_table, cu_seq_lens, seq_starts, batch, max_blocks, block_size, records, row_elems);
 }
 
 void gather_indexer_k(void* dst_k, float* dst_s, const void* cache, const int* block_table, const int* cu_seq_lens,

@@ -36,7 +36,7 @@ template <typename T, int BN, int STAGES>
 __global__ void __launch_bounds__(192, 1)
 gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmW,
                     T* __restrict__ C, const int* __restrict__ block_expert, const int* __restrict__ total_padded,
-                    int N, int K, int ldc, int epi, int num_experts, StatusWord* status) {
+                    int N, int K, int ldc, Epi epi, int num_experts, StatusWord* status) {
   using L = GgSmem<BN, STAGES>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -168,7 +168,7 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
 
 template <typename T, int BN, int STAGES>
 static void launch_grouped(const void* A, int max_rows, int lda, const void* W, int E, int N, int K, void* C, int ldc,
-                           const int* block_expert, const int* total_padded, int epi, cudaStream_t stream,
+                           const int* block_expert, const int* total_padded, Epi epi, cudaStream_t stream,
                            StatusWord* status) {
   using L = GgSmem<BN, STAGES>;
   const CUtensorMapDataType dt =
@@ -195,7 +195,7 @@ static void launch_grouped(const void* A, int max_rows, int lda, const void* W, 
 
 // A [max_rows, K] (max_rows multiple of 128), W [E, N, K], C [max_rows, N] (or N/2 with epi 1).
 void gemm_grouped(const void* A, int max_rows, int lda, const void* W, int E, int N, int K, void* C, int ldc,
-                  const int* block_expert, const int* total_padded, int epi, int dtype, cudaStream_t stream,
+                  const int* block_expert, const int* total_padded, Epi epi, int dtype, cudaStream_t stream,
                   void* status) {
   if (max_rows <= 0 || N <= 0) return;
   StatusWord* st = reinterpret_cast<StatusWord*>(status);

@@ -58,7 +58,7 @@ template <typename T, int STAGES, bool BULK>
 __global__ void __launch_bounds__(192, 1)
 gemm_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB,
                  T* __restrict__ C, const T* __restrict__ bias, const T* __restrict__ residual, int M, int N, int K,
-                 int ldc, int ldr, int epi, StatusWord* status, const __grid_constant__ RowScatter sc) {
+                 int ldc, int ldr, Epi epi, StatusWord* status, const __grid_constant__ RowScatter sc) {
   using L = PairSmem<STAGES, BULK>;
   constexpr int kPairStages = STAGES;
   extern __shared__ uint8_t smem_raw[];
@@ -271,7 +271,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
 
 template <typename T, int STAGES, bool BULK>
 static void launch_pair(const void* A, const void* W, void* C, const void* bias, const void* residual, int M, int N,
-                        int K, int lda, int ldw, int ldc, int ldr, int epi, cudaStream_t stream, StatusWord* status,
+                        int K, int lda, int ldw, int ldc, int ldr, Epi epi, cudaStream_t stream, StatusWord* status,
                         const RowScatter& sc) {
   const CUtensorMapDataType dt =
       std::is_same<T, __half>::value ? CU_TENSOR_MAP_DATA_TYPE_FLOAT16 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
@@ -312,7 +312,7 @@ static void launch_pair(const void* A, const void* W, void* C, const void* bias,
 }
 
 void gemm_tn_pair(const void* A, const void* W, void* C, const void* bias, const void* residual, int M, int N, int K,
-                  int lda, int ldw, int ldc, int ldr, int dtype, cudaStream_t stream, void* status, int epi,
+                  int lda, int ldw, int ldc, int ldr, int dtype, cudaStream_t stream, void* status, Epi epi,
                   const RowScatter* scatter) {
   if (M <= 0 || N <= 0) return;
   RowScatter sc{};
@@ -323,7 +323,7 @@ void gemm_tn_pair(const void* A, const void* W, void* C, const void* bias, const
     const char* e = std::getenv("B200_SCATTER_BULK");
     return e == nullptr || std::atoi(e) != 0;
   }();
-  const bool bulk = sc.tp > 0 && bulk_default && epi == 0 && residual == nullptr && N % 8 == 0 && ldc % 8 == 0;
+  const bool bulk = sc.tp > 0 && bulk_default && epi.code == 0 && residual == nullptr && N % 8 == 0 && ldc % 8 == 0;
 #define B200_PAIR(T)                                                                                              \
   do {                                                                                                            \
     if (bulk) launch_pair<T, 4, true>(A, W, C, bias, residual, M, N, K, lda, ldw, ldc, ldr, epi, stream, st, sc);  \

@@ -41,7 +41,7 @@ template <typename T>
 __global__ void __launch_bounds__(192, 1)
 gemm_splitk_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB,
                    T* __restrict__ C, const T* __restrict__ bias, const T* __restrict__ residual, int M, int N, int K,
-                   int ldc, int ldr, int epi, int splits, StatusWord* status) {
+                   int ldc, int ldr, Epi epi, int splits, StatusWord* status) {
   using L = SkSmem;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -196,7 +196,7 @@ gemm_splitk_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constan
 
 template <typename T>
 static void launch_sk(const void* A, const void* W, void* C, const void* bias, const void* residual, int M, int N, int K,
-                      int lda, int ldw, int ldc, int ldr, int epi, int splits, cudaStream_t stream, StatusWord* status) {
+                      int lda, int ldw, int ldc, int ldr, Epi epi, int splits, cudaStream_t stream, StatusWord* status) {
   const CUtensorMapDataType dt =
       std::is_same<T, __half>::value ? CU_TENSOR_MAP_DATA_TYPE_FLOAT16 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
   CUtensorMap tmA = make_tmap_2d(A, dt, 2, M, K, lda, kSkBM, kSkBK);
@@ -231,7 +231,7 @@ int gemm_splitk_choice(int M, int N, int K, int sms) {
 }
 
 void gemm_tn_splitk(const void* A, const void* W, void* C, const void* bias, const void* residual, int M, int N, int K,
-                    int lda, int ldw, int ldc, int ldr, int dtype, cudaStream_t stream, void* status, int epi,
+                    int lda, int ldw, int ldc, int ldr, int dtype, cudaStream_t stream, void* status, Epi epi,
                     int splits) {
   if (M <= 0 || N <= 0) return;
   StatusWord* st = reinterpret_cast<StatusWord*>(status);

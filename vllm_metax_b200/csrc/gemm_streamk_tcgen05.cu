@@ -18,6 +18,7 @@
 // All mbarrier waits are bounded.  Replaces the library GEMM behind every unquantised linear layer at decode
 // batch sizes (torch.nn.functional.linear in the reference's model files).
 #include <type_traits>
+#include "gemm_epilogue.cuh"
 #include "comm_fused.cuh"
 #include "ptx_sm100.cuh"
 #include "tma_host.h"
@@ -65,7 +66,7 @@ template <typename T>
 __global__ void __launch_bounds__(192, 1)
 gemm_streamk_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmX,
                     T* __restrict__ C, const T* __restrict__ bias, const T* __restrict__ residual, const StkShape sh,
-                    int ldc, int ldr, int epi, float* __restrict__ ws, int* __restrict__ counters,
+                    int ldc, int ldr, Epi epi, float* __restrict__ ws, int* __restrict__ counters,
                     StatusWord* status, const __grid_constant__ RowScatter sc) {
   using L = StkSmem;
   extern __shared__ uint8_t smem_raw[];
@@ -280,7 +281,7 @@ gemm_streamk_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_consta
             } else {
               crow = C + (size_t)tok * ldc;
             }
-            if (epi == 1) {
+            if (epi.code == 1) {
               // interleaved (gate, up) features: two outputs per four lanes
               T o2[2];
 #pragma unroll
@@ -290,6 +291,10 @@ gemm_streamk_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_consta
               }
               if (ra + 3 < sh.N) *reinterpret_cast<uint32_t*>(crow + (ra >> 1)) = *reinterpret_cast<const uint32_t*>(o2);
               else if (ra + 1 < sh.N) crow[ra >> 1] = o2[0];
+            } else if (epi.code > 1) {
+#pragma unroll
+              for (int e = 0; e < 4; ++e)
+                if (ra + e < sh.N) epi_store1<T>(C, (size_t)tok * ldc + ra + e, f[e], epi);
             } else {
               if (residual && sc.tp == 0) {
 #pragma unroll
@@ -319,7 +324,7 @@ gemm_streamk_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_consta
 #pragma unroll
           for (int i = 0; i < 16; ++i) a[i] = __uint_as_float(r[i]);
           const int tok0 = tt * kStkBT + c;
-          if (epi == 1) {
+          if (epi.code == 1) {
             // lanes hold interleaved (gate, up) features: even lane = gate, odd lane = up
 #pragma unroll
             for (int i = 0; i < 16; ++i) {
@@ -327,6 +332,12 @@ gemm_streamk_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_consta
               const float up = __shfl_down_sync(0xffffffffu, g, 1);
               if ((lane & 1) == 0 && ra_ok && tok0 + i < sh.M)
                 C[(size_t)(tok0 + i) * ldc + (ra >> 1)] = from_f<T>(g / (1.f + __expf(-g)) * up);
+            }
+          } else if (epi.code > 1) {
+            if (ra_ok) {
+#pragma unroll
+              for (int i = 0; i < 16; ++i)
+                if (tok0 + i < sh.M) epi_store1<T>(C, (size_t)(tok0 + i) * ldc + ra, a[i] + bv, epi);
             }
           } else if (ra_ok) {
 #pragma unroll
@@ -397,7 +408,7 @@ int gemm_streamk_max_tiles() { return 8192; }
 
 template <typename T>
 static void launch_stk(const void* A, const void* W, void* C, const void* bias, const void* residual,
-                       const StkShape& sh, int lda, int ldw, int ldc, int ldr, int epi, float* ws, int* counters,
+                       const StkShape& sh, int lda, int ldw, int ldc, int ldr, Epi epi, float* ws, int* counters,
                        cudaStream_t stream, StatusWord* status, const RowScatter& sc) {
   const CUtensorMapDataType dt =
       std::is_same<T, __half>::value ? CU_TENSOR_MAP_DATA_TYPE_FLOAT16 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
@@ -430,7 +441,7 @@ static void launch_stk(const void* A, const void* W, void* C, const void* bias, 
 // Returns 0 when launched, -1 when the shape is outside what the scratch buffers cover.
 // `ws` must hold gemm_streamk_workspace_bytes(sms) bytes, `counters` 2 * gemm_streamk_max_tiles() zeroed ints.
 int gemm_tn_streamk(const void* A, const void* W, void* C, const void* bias, const void* residual, int M, int N, int K,
-                    int lda, int ldw, int ldc, int ldr, int dtype, cudaStream_t stream, void* status, int epi,
+                    int lda, int ldw, int ldc, int ldr, int dtype, cudaStream_t stream, void* status, Epi epi,
                     float* ws, int* counters, int sms, const RowScatter* scatter) {
   if (M <= 0 || N <= 0) return 0;
   RowScatter sc{};

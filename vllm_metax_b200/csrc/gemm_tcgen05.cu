@@ -24,6 +24,7 @@
 // the CTA drains and frees its TMEM.
 #include <type_traits>
 #include "common.cuh"
+#include "gemm_epilogue.cuh"
 #include "ptx_sm100.cuh"
 #include "tma_host.h"
 
@@ -44,12 +45,15 @@ struct GemmSmemLayout {
   static constexpr int kDynSmem = kTotal + 1024;  // slack for 1024-byte alignment
 };
 
-template <typename T, int BN, int STAGES, bool SWAP>
+// BATCHED: both operand maps are 3-D and the tile index runs over `batches` products of one shape (C advances by
+// `c_batch` elements from one to the next).
+template <typename T, int BN, int STAGES, bool SWAP, bool BATCHED>
 __global__ void __launch_bounds__(192, 1)
 gemm_tn_kernel(const __grid_constant__ CUtensorMap tmA,   // 128-row operand
                const __grid_constant__ CUtensorMap tmB,   // BN-row operand
-               T* __restrict__ C, const T* __restrict__ bias, const T* __restrict__ residual,
-               int rows_a, int rows_b, int K, int ldc, int ldr, int epi, StatusWord* status) {
+               T* __restrict__ C0, const T* __restrict__ bias, const T* __restrict__ residual,
+               int rows_a, int rows_b, int K, int ldc, int ldr, Epi epi, StatusWord* status, int batches,
+               int64_t c_batch) {
   using L = GemmSmemLayout<BN, STAGES>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -63,7 +67,8 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmA,   // 128-row operand
   const int lane = threadIdx.x & 31;
   const int num_a = ceil_div(rows_a, kBM);
   const int num_b = ceil_div(rows_b, BN);
-  const int num_tiles = num_a * num_b;
+  const int per_batch = num_a * num_b;
+  const int num_tiles = BATCHED ? per_batch * batches : per_batch;
   const int num_k = ceil_div(K, kBK);
   constexpr uint32_t kTmemCols = (2 * BN < 32) ? 32 : 2 * BN;
 
@@ -97,7 +102,8 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmA,   // 128-row operand
       bool ok = true;
       for (int tile = blockIdx.x; tile < num_tiles && ok; tile += gridDim.x) {
         // consecutive CTAs share the BN-row operand tile (same tb) and walk the 128-row operand
-        const int ta = tile % num_a, tb = tile / num_a;
+        const int tz = BATCHED ? tile / per_batch : 0, tr = BATCHED ? tile % per_batch : tile;
+        const int ta = tr % num_a, tb = tr / num_a;
         for (int kb = 0; kb < num_k; ++kb) {
           if (!mbar_wait(&empty_bar[stage], phase ^ 1)) {
             report_status(status, kWaitTimeout, 1, tile, kb);
@@ -107,8 +113,13 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmA,   // 128-row operand
           uint8_t* sa = smem + stage * L::kStageBytes;
           uint8_t* sb = sa + L::kABytes;
           mbar_expect_tx(&full_bar[stage], L::kStageBytes);
-          tma_load_2d(sa, &tmA, &full_bar[stage], kb * kBK, ta * kBM);
-          tma_load_2d(sb, &tmB, &full_bar[stage], kb * kBK, tb * BN);
+          if constexpr (BATCHED) {
+            tma_load_3d(sa, &tmA, &full_bar[stage], kb * kBK, ta * kBM, tz);
+            tma_load_3d(sb, &tmB, &full_bar[stage], kb * kBK, tb * BN, tz);
+          } else {
+            tma_load_2d(sa, &tmA, &full_bar[stage], kb * kBK, ta * kBM);
+            tma_load_2d(sb, &tmB, &full_bar[stage], kb * kBK, tb * BN);
+          }
           if (++stage == STAGES) { stage = 0; phase ^= 1; }
         }
       }
@@ -157,7 +168,11 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmA,   // 128-row operand
     const int quarter = warp & 3;  // TMEM lane quarter this warp may read
     int it = 0;
     for (int tile = blockIdx.x; tile < num_tiles; tile += gridDim.x, ++it) {
-      const int ta = tile % num_a, tb = tile / num_a;
+      const int tz = BATCHED ? tile / per_batch : 0, tr = BATCHED ? tile % per_batch : tile;
+      const int ta = tr % num_a, tb = tr / num_a;
+      // (an fp32 output matrix counts its elements in floats)
+      T* const C = !BATCHED ? C0 : (epi.code & kEpiF32) ? reinterpret_cast<T*>(reinterpret_cast<float*>(C0) + tz * c_batch)
+                                                        : C0 + tz * c_batch;
       const int acc = it & 1;
       const uint32_t acc_phase = (it >> 1) & 1;
       if (!mbar_wait(&tmem_full[acc], acc_phase)) {
@@ -183,7 +198,9 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmA,   // 128-row operand
         const int cb0 = tb * BN + c;  // first index in the BN-row operand
         if constexpr (!SWAP) {
           // row = token (ra), columns = output features cb0..cb0+CH
-          if (ra < rows_a && epi == 1) {
+          if (epi.code > 1) {
+            if (ra < rows_a) epi_store_row<T, CH>(r, ra, cb0, rows_b, C, ldc, bias, epi);
+          } else if (ra < rows_a && epi.code == 1) {
             // columns hold interleaved (gate, up) pairs: out[:, j] = silu(gate_j) * up_j
             T* dst = C + (size_t)ra * ldc + (cb0 >> 1);
 #pragma unroll
@@ -246,7 +263,7 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmA,   // 128-row operand
         } else {
           // row = output feature (ra), columns = tokens cb0..cb0+CH; C is [tokens, features]
           const float bv = (bias && ra < rows_a) ? to_f(bias[ra]) : 0.f;
-          if (epi == 1) {
+          if (epi.code == 1) {
             // lanes hold interleaved (gate, up) features: even lane = gate, odd lane = up
 #pragma unroll
             for (int i = 0; i < CH; ++i) {
@@ -255,6 +272,12 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmA,   // 128-row operand
               const float u = __shfl_down_sync(0xffffffffu, g, 1);
               if ((lane & 1) == 0 && ra < rows_a && tok < rows_b)
                 C[(size_t)tok * ldc + (ra >> 1)] = from_f<T>(g / (1.f + __expf(-g)) * u);
+            }
+          } else if (epi.code > 1) {
+            if (ra < rows_a) {
+#pragma unroll
+              for (int i = 0; i < CH; ++i)
+                if (cb0 + i < rows_b) epi_store1<T>(C, (size_t)(cb0 + i) * ldc + ra, __uint_as_float(r[i]) + bv, epi);
             }
           } else if (ra < rows_a) {
 #pragma unroll
@@ -295,7 +318,7 @@ static int num_sms() {
 
 template <typename T, int BN, int STAGES, bool SWAP>
 static void launch_cfg(const void* a_op, int rows_a, int lda, const void* b_op, int rows_b, int ldb, void* C,
-                       const void* bias, const void* residual, int K, int ldc, int ldr, int epi, cudaStream_t stream,
+                       const void* bias, const void* residual, int K, int ldc, int ldr, Epi epi, cudaStream_t stream,
                        StatusWord* status) {
   using L = GemmSmemLayout<BN, STAGES>;
   static_assert(L::kDynSmem <= 232448, "shared memory budget exceeded");
@@ -303,18 +326,66 @@ static void launch_cfg(const void* a_op, int rows_a, int lda, const void* b_op, 
       std::is_same<T, __half>::value ? CU_TENSOR_MAP_DATA_TYPE_FLOAT16 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
   CUtensorMap tmA = make_tmap_2d(a_op, dt, 2, rows_a, K, lda, kBM, kBK);
   CUtensorMap tmB = make_tmap_2d(b_op, dt, 2, rows_b, K, ldb, BN, kBK);
-  auto kern = gemm_tn_kernel<T, BN, STAGES, SWAP>;
+  auto kern = gemm_tn_kernel<T, BN, STAGES, SWAP, false>;
   // a per-device attribute of the kernel: set on every launch (cheap) rather than once per process
   cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kDynSmem);
   const int tiles = ceil_div(rows_a, kBM) * ceil_div(rows_b, BN);
   const int grid = tiles < num_sms() ? tiles : num_sms();
   kern<<<grid, 192, L::kDynSmem, stream>>>(tmA, tmB, reinterpret_cast<T*>(C), reinterpret_cast<const T*>(bias),
-                                           reinterpret_cast<const T*>(residual), rows_a, rows_b, K, ldc, ldr, epi, status);
+                                           reinterpret_cast<const T*>(residual), rows_a, rows_b, K, ldc, ldr, epi, status, 1, 0);
+}
+
+template <typename T, int BN, int STAGES, bool SWAP>
+static void launch_batched(const void* a_op, int rows_a, int lda, int64_t a_batch, const void* b_op, int rows_b, int ldb,
+                           int64_t b_batch, void* C, int ldc, int64_t c_batch, int batches, int K, Epi epi,
+                           cudaStream_t stream, StatusWord* status) {
+  using L = GemmSmemLayout<BN, STAGES>;
+  const CUtensorMapDataType dt =
+      std::is_same<T, __half>::value ? CU_TENSOR_MAP_DATA_TYPE_FLOAT16 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
+  auto map3 = [&](const void* base, int rows, int ld, int64_t batch, int box_rows) {
+    uint64_t d[3] = {(uint64_t)K, (uint64_t)rows, (uint64_t)batches};
+    uint64_t s[2] = {(uint64_t)ld * 2, (uint64_t)batch * 2};
+    uint32_t b[3] = {(uint32_t)kBK, (uint32_t)box_rows, 1};
+    return make_tmap_nd(base, dt, 3, d, s, b, CU_TENSOR_MAP_SWIZZLE_128B);
+  };
+  CUtensorMap tmA = map3(a_op, rows_a, lda, a_batch, kBM);
+  CUtensorMap tmB = map3(b_op, rows_b, ldb, b_batch, BN);
+  auto kern = gemm_tn_kernel<T, BN, STAGES, SWAP, true>;
+  cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kDynSmem);
+  const int tiles = ceil_div(rows_a, kBM) * ceil_div(rows_b, BN) * batches;
+  const int grid = tiles < num_sms() ? tiles : num_sms();
+  kern<<<grid, 192, L::kDynSmem, stream>>>(tmA, tmB, reinterpret_cast<T*>(C), nullptr, nullptr, rows_a, rows_b, K, ldc, 0,
+                                           epi, status, batches, c_batch);
+}
+
+template <typename T>
+static void batched_dispatch(const void* A, const void* W, void* C, int batches, int M, int N, int K, int lda, int ldw,
+                             int ldc, int64_t a_batch, int64_t w_batch, int64_t c_batch, Epi epi, cudaStream_t stream,
+                             StatusWord* st) {
+  if (M <= 16)
+    launch_batched<T, 16, 8, true>(W, N, ldw, w_batch, A, M, lda, a_batch, C, ldc, c_batch, batches, K, epi, stream, st);
+  else if (M <= 64)
+    launch_batched<T, 64, 8, true>(W, N, ldw, w_batch, A, M, lda, a_batch, C, ldc, c_batch, batches, K, epi, stream, st);
+  else if (N >= 96)
+    launch_batched<T, 128, 6, false>(A, M, lda, a_batch, W, N, ldw, w_batch, C, ldc, c_batch, batches, K, epi, stream, st);
+  else
+    launch_batched<T, 64, 8, false>(A, M, lda, a_batch, W, N, ldw, w_batch, C, ldc, c_batch, batches, K, epi, stream, st);
+}
+
+void gemm_tn_batched(const void* A, const void* W, void* C, int batches, int M, int N, int K, int lda, int ldw, int ldc,
+                     int64_t a_batch, int64_t w_batch, int64_t c_batch, int dtype, cudaStream_t stream, void* status,
+                     Epi epi) {
+  if (M <= 0 || N <= 0 || batches <= 0) return;
+  StatusWord* st = reinterpret_cast<StatusWord*>(status);
+  if (dtype == 0)
+    batched_dispatch<__nv_bfloat16>(A, W, C, batches, M, N, K, lda, ldw, ldc, a_batch, w_batch, c_batch, epi, stream, st);
+  else
+    batched_dispatch<__half>(A, W, C, batches, M, N, K, lda, ldw, ldc, a_batch, w_batch, c_batch, epi, stream, st);
 }
 
 template <typename T>
 static void gemm_dispatch(const void* A, const void* W, void* C, const void* bias, const void* residual, int M, int N,
-                          int K, int lda, int ldw, int ldc, int ldr, int epi, cudaStream_t stream, StatusWord* status,
+                          int K, int lda, int ldw, int ldc, int ldr, Epi epi, cudaStream_t stream, StatusWord* status,
                           int force_bn) {
   const int sms = num_sms();
   if (M <= 64 && force_bn <= 0 || force_bn < 0) {
@@ -350,7 +421,7 @@ static void gemm_dispatch(const void* A, const void* W, void* C, const void* bia
 // epi: 0 = plain, 1 = SiLU-gate epilogue over interleaved (gate, up) output features (C is [M, N/2]).
 // dtype: 0 = bf16, 1 = fp16.  force_bn: 0 = heuristic, >0 = that BN without swap, <0 = swap with |BN| tokens.
 void gemm_tn(const void* A, const void* W, void* C, const void* bias, const void* residual, int M, int N, int K,
-             int lda, int ldw, int ldc, int ldr, int dtype, cudaStream_t stream, void* status, int force_bn, int epi) {
+             int lda, int ldw, int ldc, int ldr, int dtype, cudaStream_t stream, void* status, int force_bn, Epi epi) {
   if (M <= 0 || N <= 0) return;
   if (dtype == 0)
     gemm_dispatch<__nv_bfloat16>(A, W, C, bias, residual, M, N, K, lda, ldw, ldc, ldr, epi, stream,

@@ -1,0 +1,195 @@
+// Pieces around latent (low-rank key / value) attention for any sizes:
+//   latent_insert     one CTA per token: RMS norms of the query latent and of the key latent, rotation of the shared key
+//                     part, and the paged-cache write of [key latent | rotated part] - the epilogue of the merged
+//                     down-projection
+//   latent_rope       rotation of the queries' rotated parts, in place (prompt path) or into the absorbed query rows
+//                     (decode path), one warp per (token, head)
+//   latent_attn_simt  absorbed attention on the CUDA cores: fp32 caches, and 16-bit sizes the tensor-core kernel
+//                     (mla_decode.cu) does not take
+// Angles are position * inv_freq in fp32; pairs are (i, i + rot_dims / 2).
+#include "common.cuh"
+#include "ops.h"
+
+namespace b200 {
+namespace {
+
+__device__ __forceinline__ void rotate_pair(float& u, float& v, float pos, float f) {
+  float s, c;
+  sincosf(pos * f, &s, &c);
+  const float a = u * c - v * s, b = v * c + u * s;
+  u = a;
+  v = b;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(128)
+latent_insert_kernel(const LatentInsertParams p) {
+  __shared__ float red[32];
+  const int64_t t = blockIdx.x;
+  const T* row = reinterpret_cast<const T*>(p.a) + t * p.a_stride;
+  const T* aq = row + p.q_off;
+  const T* ak = row + p.kv_off;
+  float sq = 0.f, sk = 0.f;
+  for (int i = threadIdx.x; i < p.q_rank; i += blockDim.x) { const float v = to_f(aq[i]); sq = fmaf(v, v, sq); }
+  for (int i = threadIdx.x; i < p.kv_rank; i += blockDim.x) { const float v = to_f(ak[i]); sk = fmaf(v, v, sk); }
+  sq = block_sum(sq, red);
+  sk = block_sum(sk, red);
+  const float iq = 1.f / sqrtf(sq / (float)p.q_rank + p.eps), ik = 1.f / sqrtf(sk / (float)p.kv_rank + p.eps);
+  T* cq = reinterpret_cast<T*>(p.cq) + t * p.q_rank;
+  const T* wq = reinterpret_cast<const T*>(p.q_w);
+  for (int i = threadIdx.x; i < p.q_rank; i += blockDim.x) cq[i] = from_f<T>(to_f(aq[i]) * iq * to_f(wq[i]));
+  const int64_t slot = p.slots[t];
+  if (slot < 0) return;
+  if (slot >= p.num_slots) {
+    if (threadIdx.x == 0) report_status(p.status, kBadIndex, 120, (int)p.num_slots, (int)slot);
+    return;
+  }
+  T* dst = reinterpret_cast<T*>(p.cache) + slot * p.row_elems;
+  const T* wk = reinterpret_cast<const T*>(p.kv_w);
+  for (int i = threadIdx.x; i < p.kv_rank; i += blockDim.x) dst[i] = from_f<T>(to_f(ak[i]) * ik * to_f(wk[i]));
+  const T* kr = ak + p.kv_rank;
+  const int half = p.rot_dims / 2;
+  const float pos = (float)p.positions[t];
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float u = to_f(kr[i]), v = to_f(kr[i + half]);
+    rotate_pair(u, v, pos, p.inv_freq[i]);
+    dst[p.kv_rank + i] = from_f<T>(u);
+    dst[p.kv_rank + half + i] = from_f<T>(v);
+  }
+  for (int i = 2 * half + threadIdx.x; i < p.rot_dim; i += blockDim.x) dst[p.kv_rank + i] = kr[i];
+  for (int i = p.kv_rank + p.rot_dim + threadIdx.x; i < p.row_elems; i += blockDim.x) dst[i] = from_f<T>(0.f);
+}
+
+template <typename T>
+__global__ void latent_rope_kernel(const T* src, int64_t src_tok, int64_t src_head, T* dst, int64_t dst_tok,
+                                   int64_t dst_head, const int64_t* __restrict__ positions,
+                                   const float* __restrict__ inv_freq, int tokens, int heads, int rot_dim, int rot_dims,
+                                   int pad) {
+  const int64_t w = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (w >= (int64_t)tokens * heads) return;
+  const int64_t t = w / heads, h = w % heads;
+  const T* s = src + t * src_tok + h * src_head;
+  T* d = dst + t * dst_tok + h * dst_head;
+  const int half = rot_dims / 2;
+  const float pos = (float)positions[t];
+  for (int i = lane; i < half; i += 32) {
+    float u = to_f(s[i]), v = to_f(s[i + half]);
+    rotate_pair(u, v, pos, inv_freq[i]);
+    d[i] = from_f<T>(u);
+    d[i + half] = from_f<T>(v);
+  }
+  if (s != d)
+    for (int i = 2 * half + lane; i < rot_dim; i += 32) d[i] = s[i];
+  for (int i = rot_dim + lane; i < rot_dim + pad; i += 32) d[i] = from_f<T>(0.f);
+}
+
+// One CTA per (token, head): 128 keys at a time, a thread per key for the scores, a thread per column for the values.
+constexpr int kSimtKeys = 128, kSimtCols = 8;
+
+template <typename T>
+__global__ void __launch_bounds__(kSimtKeys)
+latent_attn_simt_kernel(const MlaDecodeParams p) {
+  extern __shared__ float s_q[];                             // [q_dim]
+  __shared__ float s_p[kSimtKeys], red[32];
+  __shared__ int64_t s_row[kSimtKeys];
+  const int t = blockIdx.y, h = blockIdx.x;
+  int lo = 0;
+  if (p.query_start_loc) {
+    for (int hi = p.batch - 1; lo < hi;) {
+      const int mid = (lo + hi + 1) >> 1;
+      if (p.query_start_loc[mid] <= t) lo = mid; else hi = mid - 1;
+    }
+  } else {
+    lo = t;
+  }
+  const int q0 = p.query_start_loc ? p.query_start_loc[lo] : lo, q1 = p.query_start_loc ? p.query_start_loc[lo + 1] : lo + 1;
+  const int lim = p.seq_lens[lo] - (q1 - q0) + (t - q0) + 1;
+  const int first = p.window > 0 ? max(0, lim - p.window) : 0;
+  const int* btab = p.block_table + (int64_t)lo * p.max_blocks;
+  const T* q = reinterpret_cast<const T*>(p.q) + (int64_t)t * p.q_stride + (int64_t)h * p.q_dim;
+  const int depth = min(p.q_dim, p.row_elems);
+  for (int i = threadIdx.x; i < depth; i += blockDim.x) s_q[i] = to_f(q[i]);
+  const T* cache = reinterpret_cast<const T*>(p.cache);
+  float m = -INFINITY, l = 0.f, acc[kSimtCols];
+#pragma unroll
+  for (int i = 0; i < kSimtCols; ++i) acc[i] = 0.f;
+  __syncthreads();
+  for (int k0 = first; k0 < lim; k0 += kSimtKeys) {
+    const int pos = k0 + threadIdx.x;
+    float s = -INFINITY;
+    int64_t row = -1;
+    if (pos < lim && pos < (int64_t)p.max_blocks * p.block_size) {
+      const int page = btab[pos / p.block_size];
+      if (page < 0 || page >= p.num_blocks) report_status(p.status, kBadIndex, 121, (int)p.num_blocks, page);
+      else row = (int64_t)page * p.block_size + pos % p.block_size;
+    }
+    if (row >= 0) {
+      const T* c = cache + row * p.row_elems;
+      float d = 0.f;
+      for (int i = 0; i < depth; ++i) d = fmaf(s_q[i], to_f(c[i]), d);
+      s = d * p.scale;
+    }
+    const float mx = block_max(s, red);
+    const float mn = fmaxf(m, mx), ms = mn == -INFINITY ? 0.f : mn;
+    const float corr = m == -INFINITY ? 0.f : expf(m - ms);
+    const float e = s == -INFINITY ? 0.f : expf(s - ms);
+    m = mn;
+    s_p[threadIdx.x] = e;
+    s_row[threadIdx.x] = row < 0 ? 0 : row;
+    l = l * corr + block_sum(e, red);                        // (its barriers publish s_p and s_row)
+    const int nk = min(kSimtKeys, lim - k0);
+#pragma unroll
+    for (int i = 0; i < kSimtCols; ++i) {
+      const int c = threadIdx.x + i * kSimtKeys;
+      if (c < p.kv_rank) {
+        float a = acc[i] * corr;
+        for (int k = 0; k < nk; ++k) a = fmaf(s_p[k], to_f(cache[s_row[k] * p.row_elems + c]), a);
+        acc[i] = a;
+      }
+    }
+    __syncthreads();
+  }
+  const float inv = l > 0.f ? 1.f / l : 0.f;
+  T* out = reinterpret_cast<T*>(p.out) + ((int64_t)t * p.num_heads + h) * p.kv_rank;
+#pragma unroll
+  for (int i = 0; i < kSimtCols; ++i) {
+    const int c = threadIdx.x + i * kSimtKeys;
+    if (c < p.kv_rank) out[c] = from_f<T>(acc[i] * inv);
+  }
+}
+
+}  // namespace
+
+#define BY_DTYPE(CALL)                                   \
+  if (dtype == 0) { using T = __nv_bfloat16; CALL; }     \
+  else if (dtype == 1) { using T = __half; CALL; }       \
+  else { using T = float; CALL; }
+
+int latent_insert(const LatentInsertParams& p, int dtype, cudaStream_t stream) {
+  if (p.tokens <= 0) return 0;
+  BY_DTYPE((latent_insert_kernel<T><<<p.tokens, 128, 0, stream>>>(p)))
+  return 0;
+}
+
+int latent_rope(const void* src, int64_t src_tok, int64_t src_head, void* dst, int64_t dst_tok, int64_t dst_head,
+                const int64_t* positions, const float* inv_freq, int tokens, int heads, int rot_dim, int rot_dims, int pad,
+                int dtype, cudaStream_t stream) {
+  const int64_t warps = (int64_t)tokens * heads;
+  if (warps <= 0) return 0;
+  BY_DTYPE((latent_rope_kernel<T><<<(unsigned)((warps + 3) / 4), 128, 0, stream>>>(
+      (const T*)src, src_tok, src_head, (T*)dst, dst_tok, dst_head, positions, inv_freq, tokens, heads, rot_dim, rot_dims,
+      pad)))
+  return 0;
+}
+
+// Returns 1 for a latent wider than 1024 or more tokens than the grid holds.
+int latent_attn_simt(const MlaDecodeParams& p, int dtype, cudaStream_t stream) {
+  if (p.total_tokens <= 0) return 0;
+  if (p.kv_rank > kSimtKeys * kSimtCols || p.total_tokens > 65535 || p.q_dim > 8192) return 1;
+  const dim3 grid(p.num_heads, p.total_tokens);
+  BY_DTYPE((latent_attn_simt_kernel<T><<<grid, kSimtKeys, p.q_dim * sizeof(float), stream>>>(p)))
+  return 0;
+}
+
+}  // namespace b200

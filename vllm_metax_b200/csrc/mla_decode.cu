@@ -5,7 +5,12 @@
 //          512 e4m3 | 4 f32 scales, one per 128 | 64 bf16 rope)
 //   out    [T, H, 512],  lse [H, T]
 //
-// Dense: token t of sequence b sees cache positions < seq_len - q_len + i + 1.
+// The sizes above are the DeepSeek ones, compiled in; other latent models run the same kernel with their own: a row is
+// [kv_rank latent | rotated key part], padded to `row_elems` (a multiple of 8), q has `q_dim` entries per head and out
+// `kv_rank` columns.
+//
+// Dense: token t of sequence b sees cache positions < seq_len - q_len + i + 1, with `window` > 0 only the last
+// `window` of them.
 // Sparse (DeepSeek sparse attention): only the positions listed in topk_indices[t, :] (-1 = none).
 //
 // One CTA = one query token x 16 / 32 / 64 heads x one KV split; 8 warps walk 64-token latent tiles through a
@@ -63,6 +68,7 @@ __device__ __forceinline__ uint32_t mla_pack2(float a, float b) {
 constexpr int kMlaTok = 64;                       // latent rows per tile
 constexpr int kMlaThreads = 256;                  // 8 warps: warp w owns tile tokens [8w, 8w+8) and output columns [64w, 64w+64)
 constexpr int kMlaTileB = kMlaTok * kMlaRowBytes; // 72 KB
+constexpr int kMlaMaxSmem = 232448;
 
 // Shared-memory plan for MT m16 row tiles (16 * MT heads per CTA).
 template <int MT, bool FP8>
@@ -82,15 +88,38 @@ struct MlaSmem2 {
   static constexpr int kTotal = kPos + 2 * kMlaTok * 4 + 16;
 };
 
+// The same plan with the row length at run time (16-bit caches): `rb` = bytes of a shared-memory row, 128-byte multiples
+// so that the chunk swizzle stays inside the row.
+struct MlaPlan {
+  int q, ring, p, max, pos, total;
+  __host__ __device__ MlaPlan(int mt, int rb) {
+    q = 0;
+    ring = q + 16 * mt * rb;
+    p = ring + 2 * kMlaTok * rb;
+    max = p + 16 * mt * kMlaTok * 2;
+    pos = max + 8 * 16 * mt * 4;
+    total = pos + 2 * kMlaTok * 4 + 16;
+  }
+};
+
 // One CTA = one query token x 16 MT heads x one KV split.  Per 64-token tile: every warp multiplies ALL of the CTA's
 // rows with ITS 8 tokens over the full 576-wide contraction (no cross-warp reduction of partial scores), the row
 // maxima are exchanged through shared memory, P goes to shared memory once, and every warp multiplies P into ITS 64
 // of the 512 value columns - the value operand is the first 512 columns of the very tile that served as K
 // (ldmatrix.trans).  Four CTA barriers per 64 tokens; the latent rows of a token are read once per 16 MT heads.
-template <typename T, bool FP8, int MT>
+// DV: value columns computed (>= kv_rank; the excess is not stored).  GEN: sizes from the parameters.
+template <typename T, bool FP8, int MT, int DV, bool GEN>
 __global__ void __launch_bounds__(kMlaThreads, 1)
 mla_decode_kernel(const MlaDecodeParams p) {
   using S = MlaSmem2<MT, FP8>;
+  static_assert(!(GEN && FP8), "records have fixed sizes");
+  constexpr int NV = DV / 64;                              // 8-column groups of V per warp
+  const int RB = GEN ? p.smem_row_bytes : kMlaRowBytes;    // shared-memory row
+  const int CPR = RB / 16;
+  const int CROW = GEN ? p.row_elems / 8 : kMlaCPR;        // 16-byte chunks of a cache row
+  const int QD = GEN ? p.q_dim : kMlaD;
+  const int KV = GEN ? p.kv_rank : kMlaDV;
+  const MlaPlan plan(MT, RB);
   extern __shared__ __align__(128) uint8_t smem[];
   __shared__ int s_seq, s_lim;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -115,7 +144,8 @@ mla_decode_kernel(const MlaDecodeParams p) {
   }
   __syncthreads();
   const int seq = s_seq, lim = s_lim;
-  const int n_entries = p.topk_indices ? p.topk : lim;     // logical kv list length
+  const int lo0 = p.window > 0 ? max(0, lim - p.window) : 0;
+  const int n_entries = p.topk_indices ? p.topk : lim - lo0;   // logical kv list length
   const int tiles_total = (n_entries + kMlaTok - 1) / kMlaTok;
   const int tiles_per_split = (tiles_total + p.num_splits - 1) / p.num_splits;
   const int tile_begin = split * tiles_per_split;
@@ -123,26 +153,28 @@ mla_decode_kernel(const MlaDecodeParams p) {
   const int* btab = p.block_table + (int64_t)seq * p.max_blocks;
   const int* idx_row = p.topk_indices ? p.topk_indices + (int64_t)t * p.topk : nullptr;
   uint8_t* q_smem = smem + S::kQ;
-  uint8_t* p_smem = smem + S::kP;
-  float* s_max = reinterpret_cast<float*>(smem + S::kMax);
-  int* s_pos = reinterpret_cast<int*>(smem + S::kPos);
+  uint8_t* p_smem = smem + (GEN ? plan.p : S::kP);
+  float* s_max = reinterpret_cast<float*>(smem + (GEN ? plan.max : S::kMax));
+  int* s_pos = reinterpret_cast<int*>(smem + (GEN ? plan.pos : S::kPos));
+  const int ring0 = GEN ? plan.ring : S::kRing;
   const long long kv_cap = (long long)p.max_blocks * p.block_size;
 
   // ---- Q rows (heads h0 .. h0 + 16 MT - 1 of token t), swizzled; rows beyond the head count are zero
   {
     const T* qb = reinterpret_cast<const T*>(p.q) + (int64_t)t * p.q_stride;
-    for (int i = threadIdx.x; i < 16 * MT * kMlaCPR; i += blockDim.x) {
-      const int r = i / kMlaCPR, c = i % kMlaCPR;
+    for (int i = threadIdx.x; i < 16 * MT * CPR; i += blockDim.x) {
+      const int r = i / CPR, c = i % CPR;
       uint4 v = make_uint4(0, 0, 0, 0);
-      if (h0 + r < p.num_heads) v = *reinterpret_cast<const uint4*>(qb + (int64_t)(h0 + r) * kMlaD + c * 8);
-      *reinterpret_cast<uint4*>(q_smem + r * kMlaRowBytes + ((c ^ (r & 7)) * 16)) = v;
+      if (h0 + r < p.num_heads && (!GEN || c < QD / 8))
+        v = *reinterpret_cast<const uint4*>(qb + (int64_t)(h0 + r) * QD + c * 8);
+      *reinterpret_cast<uint4*>(q_smem + r * RB + ((c ^ (r & 7)) * 16)) = v;
     }
   }
 
   // cache position of entry e of the kv list, or -1 (beyond the list, masked by causality, or a bad index)
   auto pos_of = [&](int e) -> int {
     if (e >= n_entries) return -1;
-    int v = e;
+    int v = e + lo0;
     if (idx_row) v = idx_row[e];
     return (v >= 0 && v < lim && v < kv_cap) ? v : -1;
   };
@@ -163,26 +195,28 @@ mla_decode_kernel(const MlaDecodeParams p) {
   auto issue_rows = [&](int tile, int slot) {
     if (tile >= tile_end) return;
     const uint8_t* cache = reinterpret_cast<const uint8_t*>(p.cache);
-    constexpr int CH = FP8 ? 41 : kMlaCPR;                   // 16-byte chunks per stored row
-    constexpr int RB = FP8 ? kMlaRecBytes : kMlaRowBytes;
-    uint8_t* dst = smem + S::kRing + slot * (FP8 ? S::kRawStage : kMlaTileB);
+    const int CH = FP8 ? 41 : CPR;                           // 16-byte chunks per row in shared memory
+    const int SB = FP8 ? kMlaRecBytes : RB;
+    const int64_t gb = FP8 ? kMlaRecBytes : CROW * 16;       // bytes of a stored row
+    uint8_t* dst = smem + ring0 + slot * (FP8 ? S::kRawStage : kMlaTok * RB);
     for (int i = threadIdx.x; i < kMlaTok * CH; i += blockDim.x) {
       const int r = i / CH, c = i % CH;
       const int row = s_pos[slot * kMlaTok + r];
       const int dc = FP8 ? c : (c ^ (r & 7));
-      mla_cp16(dst + r * RB + dc * 16, cache + (row >= 0 ? (int64_t)row * RB + c * 16 : 0), row >= 0);
+      const bool ok = row >= 0 && (!GEN || c < CROW);        // chunks beyond the stored row: zeros
+      mla_cp16(dst + r * SB + dc * 16, cache + (ok ? row * gb + c * 16 : 0), ok);
     }
   };
 
   const float sl2 = p.scale * 1.4426950408889634f;
   float m_run[MT][2], l_run[MT][2];
-  float o[MT][8][4];
+  float o[MT][NV][4];
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt) {
     m_run[mt][0] = m_run[mt][1] = -INFINITY;
     l_run[mt][0] = l_run[mt][1] = 0.f;
 #pragma unroll
-    for (int i = 0; i < 8; ++i) o[mt][i][0] = o[mt][i][1] = o[mt][i][2] = o[mt][i][3] = 0.f;
+    for (int i = 0; i < NV; ++i) o[mt][i][0] = o[mt][i][1] = o[mt][i][2] = o[mt][i][3] = 0.f;
   }
 
   stage_positions(tile_begin, 0);
@@ -197,7 +231,7 @@ mla_decode_kernel(const MlaDecodeParams p) {
     asm volatile("cp.async.commit_group;" ::: "memory");
     asm volatile("cp.async.wait_group 1;" ::: "memory");
     __syncthreads();
-    const uint8_t* kt = smem + S::kRing + slot * kMlaTileB;
+    const uint8_t* kt = smem + ring0 + slot * kMlaTok * RB;
     if (FP8) {
       // dequantise the 64 records of this slot into the swizzled 16-bit tile
       const uint8_t* raw = smem + S::kRing + slot * S::kRawStage;
@@ -238,11 +272,11 @@ mla_decode_kernel(const MlaDecodeParams p) {
       const int mat = lane >> 3;
       const int kr = warp * 8 + (lane & 7);                  // my token row of the tile
 #pragma unroll 2
-      for (int kp = 0; kp < 18; ++kp) {
+      for (int kp = 0; kp < CPR / 4; ++kp) {
         uint32_t kf[4];
         {
           const int c = 4 * kp + mat;                         // chunks 4kp .. 4kp+3 = two k-steps
-          mla_ldm(kf, kt + kr * kMlaRowBytes + ((c ^ (kr & 7)) * 16));
+          mla_ldm(kf, kt + kr * RB + ((c ^ (kr & 7)) * 16));
         }
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
@@ -251,7 +285,7 @@ mla_decode_kernel(const MlaDecodeParams p) {
           for (int mt = 0; mt < MT; ++mt) {
             uint32_t qf[4];
             const int r = mt * 16 + (mat & 1) * 8 + (lane & 7), c = 2 * ks + (mat >> 1);
-            mla_ldm(qf, q_smem + r * kMlaRowBytes + ((c ^ (r & 7)) * 16));
+            mla_ldm(qf, q_smem + r * RB + ((c ^ (r & 7)) * 16));
             if (half == 0) mla_mma<T>(sc[mt], qf, kf[0], kf[1]);
             else mla_mma<T>(sc2[mt], qf, kf[2], kf[3]);
           }
@@ -307,7 +341,7 @@ mla_decode_kernel(const MlaDecodeParams p) {
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
-      for (int nd = 0; nd < 8; ++nd) {
+      for (int nd = 0; nd < NV; ++nd) {
         o[mt][nd][0] *= corr[mt][0]; o[mt][nd][1] *= corr[mt][0];
         o[mt][nd][2] *= corr[mt][1]; o[mt][nd][3] *= corr[mt][1];
       }
@@ -321,11 +355,11 @@ mla_decode_kernel(const MlaDecodeParams p) {
         mla_ldm(pf[mt], p_smem + r * (kMlaTok * 2) + ((c ^ (r & 7)) * 16));
       }
 #pragma unroll
-      for (int nd = 0; nd < 8; nd += 2) {
+      for (int nd = 0; nd < NV; nd += 2) {
         uint32_t vf[4];
         const int r = kk * 16 + (mat & 1) * 8 + (lane & 7);
-        const int c = warp * 8 + nd + (mat >> 1);
-        mla_ldm_t(vf, kt + r * kMlaRowBytes + ((c ^ (r & 7)) * 16));
+        const int c = warp * NV + nd + (mat >> 1);
+        mla_ldm_t(vf, kt + r * RB + ((c ^ (r & 7)) * 16));
 #pragma unroll
         for (int mt = 0; mt < MT; ++mt) {
           mla_mma<T>(o[mt][nd], pf[mt], vf[0], vf[1]);
@@ -363,20 +397,22 @@ mla_decode_kernel(const MlaDecodeParams p) {
       const float inv = L > 0.f ? 1.f / L : 0.f;
       const float lse = L > 0.f ? Ms * 0.6931471805599453f + logf(L) : -INFINITY;
       if (p.num_splits == 1) {
-        T* dst = reinterpret_cast<T*>(p.out) + ((int64_t)t * p.num_heads + h) * kMlaDV + warp * 64;
+        T* dst = reinterpret_cast<T*>(p.out) + ((int64_t)t * p.num_heads + h) * KV;
 #pragma unroll
-        for (int nd = 0; nd < 8; ++nd) {
-          const int col = nd * 8 + 2 * (lane & 3);
-          *reinterpret_cast<uint32_t*>(dst + col) =
-              mla_pack2<T>(o[mt][nd][half * 2] * inv, o[mt][nd][half * 2 + 1] * inv);
+        for (int nd = 0; nd < NV; ++nd) {
+          const int col = warp * (DV / 8) + nd * 8 + 2 * (lane & 3);
+          if (!GEN || col < KV)                        // (kv_rank is even)
+            *reinterpret_cast<uint32_t*>(dst + col) =
+                mla_pack2<T>(o[mt][nd][half * 2] * inv, o[mt][nd][half * 2 + 1] * inv);
         }
         if (warp == 0 && (lane & 3) == 0 && p.lse_out) p.lse_out[(int64_t)h * p.total_tokens + t] = lse;
       } else {
         const int64_t prow = ((int64_t)split * p.total_tokens + t) * p.num_heads + h;
-        float* dst = p.part_out + prow * kMlaDV + warp * 64;
+        float* dst = p.part_out + prow * KV;
 #pragma unroll
-        for (int nd = 0; nd < 8; ++nd) {
-          const int col = nd * 8 + 2 * (lane & 3);
+        for (int nd = 0; nd < NV; ++nd) {
+          const int col = warp * (DV / 8) + nd * 8 + 2 * (lane & 3);
+          if (GEN && col >= KV) continue;
           dst[col] = o[mt][nd][half * 2] * inv;
           dst[col + 1] = o[mt][nd][half * 2 + 1] * inv;
         }
@@ -388,7 +424,7 @@ mla_decode_kernel(const MlaDecodeParams p) {
 template <typename T>
 __global__ void mla_split_reduce_kernel(T* __restrict__ out, float* __restrict__ lse_out,
                                         const float* __restrict__ part_out, const float* __restrict__ part_lse,
-                                        int num_splits, int total_tokens, int heads) {
+                                        int num_splits, int total_tokens, int heads, int kv) {
   const int64_t row = blockIdx.x;
   const int64_t stride = (int64_t)total_tokens * heads;
   float M = -INFINITY;
@@ -396,11 +432,11 @@ __global__ void mla_split_reduce_kernel(T* __restrict__ out, float* __restrict__
   const float Ms = (M == -INFINITY) ? 0.f : M;
   float L = 0.f;
   for (int s = 0; s < num_splits; ++s) L += __expf(part_lse[s * stride + row] - Ms);
-  for (int c = threadIdx.x; c < kMlaDV; c += blockDim.x) {
+  for (int c = threadIdx.x; c < kv; c += blockDim.x) {
     float acc = 0.f;
     for (int s = 0; s < num_splits; ++s)
-      acc += part_out[(s * stride + row) * kMlaDV + c] * __expf(part_lse[s * stride + row] - Ms);
-    out[row * kMlaDV + c] = from_f<T>(L > 0.f ? acc / L : 0.f);
+      acc += part_out[(s * stride + row) * kv + c] * __expf(part_lse[s * stride + row] - Ms);
+    out[row * kv + c] = from_f<T>(L > 0.f ? acc / L : 0.f);
   }
   if (threadIdx.x == 0 && lse_out)
     lse_out[(row % heads) * (int64_t)total_tokens + row / heads] = L > 0.f ? Ms + logf(L) : -INFINITY;
@@ -410,11 +446,41 @@ template <typename T, bool FP8, int MT>
 static void launch_mla_mt(const MlaDecodeParams& p, cudaStream_t stream) {
   using S = MlaSmem2<MT, FP8>;
   static_assert(S::kTotal <= 232448, "shared memory budget exceeded");
-  auto kern = mla_decode_kernel<T, FP8, MT>;
+  auto kern = mla_decode_kernel<T, FP8, MT, kMlaDV, false>;
   // a per-device attribute of the kernel: set on every launch (cheap) rather than once per process
   cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, S::kTotal);
   dim3 grid((p.num_heads + 16 * MT - 1) / (16 * MT), p.total_tokens, p.num_splits);
   kern<<<grid, kMlaThreads, S::kTotal, stream>>>(p);
+}
+
+template <typename T, int MT, int DV>
+static void launch_mla_gen(const MlaDecodeParams& p, cudaStream_t stream) {
+  auto kern = mla_decode_kernel<T, false, MT, DV, true>;
+  const int smem = MlaPlan(MT, p.smem_row_bytes).total;
+  cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  dim3 grid((p.num_heads + 16 * MT - 1) / (16 * MT), p.total_tokens, p.num_splits);
+  kern<<<grid, kMlaThreads, smem, stream>>>(p);
+}
+
+// Sizes other than 512 + 64.  Returns -1 when the tensor-core kernel does not take them.
+template <typename T>
+static int launch_mla_sizes(MlaDecodeParams p, cudaStream_t stream) {
+  if (p.kv_rank > 512 || p.kv_rank % 2 != 0 || p.row_elems % 8 != 0 || p.q_dim % 8 != 0 || p.q_dim < p.kv_rank ||
+      p.row_elems < p.kv_rank)
+    return -1;
+  const int dv = p.kv_rank <= 128 ? 128 : p.kv_rank <= 256 ? 256 : 512;
+  const int widest = p.row_elems > p.q_dim ? p.row_elems : p.q_dim;
+  const int cols = widest > dv ? widest : dv;             // the value columns are read from the same rows
+  p.smem_row_bytes = (cols + 63) / 64 * 128;
+  const int mt = p.num_heads <= 16 ? 1 : (p.num_heads <= 32 ? 2 : 4);
+  if (MlaPlan(mt, p.smem_row_bytes).total > kMlaMaxSmem) return -1;
+#define MLA_GEN(DV)                                                  \
+  if (mt == 1) launch_mla_gen<T, 1, DV>(p, stream);                  \
+  else if (mt == 2) launch_mla_gen<T, 2, DV>(p, stream);             \
+  else launch_mla_gen<T, 4, DV>(p, stream);
+  if (dv == 128) { MLA_GEN(128) } else if (dv == 256) { MLA_GEN(256) } else { MLA_GEN(512) }
+#undef MLA_GEN
+  return 0;
 }
 
 // Heads per CTA: the latent rows are re-read once per 16 MT heads, so as many heads as shared memory allows.
@@ -438,13 +504,21 @@ static void launch_mla(const MlaDecodeParams& p, cudaStream_t stream) {
 template <typename T>
 static void launch_mla_reduce(const MlaDecodeParams& p, cudaStream_t stream) {
   mla_split_reduce_kernel<T><<<(unsigned)((int64_t)p.total_tokens * p.num_heads), 256, 0, stream>>>(
-      (T*)p.out, p.lse_out, p.part_out, p.part_lse, p.num_splits, p.total_tokens, p.num_heads);
+      (T*)p.out, p.lse_out, p.part_out, p.part_lse, p.num_splits, p.total_tokens, p.num_heads, p.kv_rank);
 }
 
 int mla_decode(const MlaDecodeParams& p, int fp8_records, int dtype, cudaStream_t stream, int impl) {
   if (p.total_tokens <= 0) return 0;
   bool done = false;
-  if (impl != 1 && !fp8_records && (impl == 2 || p.num_heads >= 64)) done = mla_decode_tc(p, dtype, stream) == 0;
+  if (p.kv_rank != kMlaDV || p.q_dim != kMlaD || (!fp8_records && p.row_elems != kMlaD)) {
+    if (fp8_records) return -1;
+    const int rc = dtype == 0 ? launch_mla_sizes<__nv_bfloat16>(p, stream) : launch_mla_sizes<__half>(p, stream);
+    if (rc != 0) return rc;
+    done = true;
+  } else if (p.window > 0) {
+    impl = 1;                                   // the tcgen05 kernel has no window
+  }
+  if (!done && impl != 1 && !fp8_records && (impl == 2 || p.num_heads >= 64)) done = mla_decode_tc(p, dtype, stream) == 0;
   if (!done && impl == 2) return -1;
   if (!done) {
     if (dtype == 0) {

@@ -6,6 +6,7 @@
 #include <stdint.h>
 #include "status.h"
 #include "comm_params.h"
+#include "epi.h"
 
 namespace b200 {
 
@@ -46,6 +47,8 @@ struct PrefillParams {
   int total_q;
   float scale, softcap;
   int window, causal, paged;
+  int dqk, dv;                   // head sizes (the kernel's tiles are padded up to 64 / 128 / 192 by the TMA fill)
+  int64_t k_head_stride, v_head_stride;   // contiguous mode, elements
   StatusWord* status;
 };
 
@@ -61,6 +64,9 @@ struct MlaDecodeParams {
   const int* query_start_loc;  // [B+1] or null (one token per sequence)
   const int* topk_indices;     // [T, topk] per-request positions (-1 = none) or null (dense)
   int64_t q_stride;
+  int window;                  // > 0: only the last `window` visible positions
+  int kv_rank, row_elems, q_dim;   // latent columns; elements of a cache row; entries of a query head (512, 576, 576)
+  int smem_row_bytes;          // set by the launcher
   int num_heads, block_size, max_blocks, num_splits, total_tokens, batch, topk;
   int64_t num_blocks;
   float scale;
@@ -69,15 +75,32 @@ struct MlaDecodeParams {
 
 // ---- gemm_tcgen05.cu
 void gemm_tn(const void* A, const void* W, void* C, const void* bias, const void* residual, int M, int N, int K,
-             int lda, int ldw, int ldc, int ldr, int dtype, cudaStream_t stream, void* status, int force_bn, int epi);
+             int lda, int ldw, int ldc, int ldr, int dtype, cudaStream_t stream, void* status, int force_bn, Epi epi);
+// `batches` independent products of one shape (16-bit operands; strides in elements; 1 = the plain product)
+void gemm_tn_batched(const void* A, const void* W, void* C, int batches, int M, int N, int K, int lda, int ldw, int ldc,
+                     int64_t a_batch, int64_t w_batch, int64_t c_batch, int dtype, cudaStream_t stream, void* status,
+                     Epi epi);
+// gemm_simt.cu: any shape, pitch and alignment, 16-bit or fp32 operands, fp32 accumulation on the CUDA cores; plain,
+// batched, or grouped over expert-sorted 128-row blocks (block_expert / total_padded)
+struct SimtGemmParams {
+  const void* A; const void* W; void* C;
+  const void* bias;              // [N] or null
+  int batches, M, N, K;
+  int64_t lda, ldw, ldc, a_batch, w_batch, c_batch;   // elements
+  const int* block_expert;       // grouped: expert of every 128-row block (w_batch = elements per expert)
+  const int* total_padded;
+  int experts;
+  Epi epi;
+};
+int gemm_simt(const SimtGemmParams& p, int dtype, cudaStream_t stream);
 // gemm_streamk_tcgen05.cu: swap-AB CTA-pair stream-K for skinny problems (scratch supplied by the caller)
 size_t gemm_streamk_workspace_bytes(int sms);
 int gemm_streamk_max_tiles();
 int gemm_tn_streamk(const void* A, const void* W, void* C, const void* bias, const void* residual, int M, int N, int K,
-                    int lda, int ldw, int ldc, int ldr, int dtype, cudaStream_t stream, void* status, int epi,
+                    int lda, int ldw, int ldc, int ldr, int dtype, cudaStream_t stream, void* status, Epi epi,
                     float* ws, int* counters, int sms, const struct RowScatter* scatter = nullptr);
 void gemm_tn_pair(const void* A, const void* W, void* C, const void* bias, const void* residual, int M, int N, int K,
-                  int lda, int ldw, int ldc, int ldr, int dtype, cudaStream_t stream, void* status, int epi,
+                  int lda, int ldw, int ldc, int ldr, int dtype, cudaStream_t stream, void* status, Epi epi,
                   const struct RowScatter* scatter = nullptr);
 // ---- comm_ar_norm.cu
 int ar_norm_gather(const ArNormParams& p, int dtype, cudaStream_t stream);
@@ -85,7 +108,7 @@ int nvls_ar_norm(const NvlsArNormParams& p, int dtype, cudaStream_t stream);
 // ---- gemm_splitk_tcgen05.cu
 int gemm_splitk_choice(int M, int N, int K, int sms);
 void gemm_tn_splitk(const void* A, const void* W, void* C, const void* bias, const void* residual, int M, int N, int K,
-                    int lda, int ldw, int ldc, int ldr, int dtype, cudaStream_t stream, void* status, int epi,
+                    int lda, int ldw, int ldc, int ldr, int dtype, cudaStream_t stream, void* status, Epi epi,
                     int splits);
 // ---- norm.cu
 void rms_norm(void* out, void* x, void* residual, const void* weight, float eps, int tokens, int hidden,
@@ -151,7 +174,7 @@ void moe_combine(void* out, const void* y, const float* weights, const int* inv_
                  int topk, int hidden, int dtype, cudaStream_t stream);
 void moe_sum(void* out, const void* in, int tokens, int topk, int hidden, int dtype, cudaStream_t stream);
 void gemm_grouped(const void* A, int max_rows, int lda, const void* W, int E, int N, int K, void* C, int ldc,
-                  const int* block_expert, const int* total_padded, int epi, int dtype, cudaStream_t stream,
+                  const int* block_expert, const int* total_padded, Epi epi, int dtype, cudaStream_t stream,
                   void* status);
 // ---- quant.cu / gemm_fp8_blockscale.cu
 void per_token_group_quant(void* q, float* scales, const void* x, int64_t rows, int K, int group, int int8, int ue8m0,
@@ -199,7 +222,7 @@ void permute_cols(void* out, const void* a, const int* perm, int64_t rows, int c
                   cudaStream_t stream);
 void gather_mla_cache(void* dst, const void* cache, const int* block_table, const int* cu_seq_lens,
                       const int* seq_starts, int batch, int max_blocks, int block_size, int max_total, int records,
-                      int dtype, cudaStream_t stream);
+                      int row_elems, int dtype, cudaStream_t stream);
 void gather_indexer_k(void* dst_k, float* dst_s, const void* cache, const int* block_table, const int* cu_seq_lens,
                       int batch, int max_blocks, int block_size, int max_total, cudaStream_t stream);
 // ---- mamba_scan.cu
@@ -268,6 +291,73 @@ int gdn_recurrent(void* out, float* state, const void* q, const void* k, const v
 int causal_conv1d(void* out, const void* x, int64_t x_stride, const void* w, const void* bias, void* state,
                   const int* query_start_loc, const int* state_idx, const int* has_init, int batch, int tokens,
                   int channels, int K, int silu, int dtype, cudaStream_t stream);
+// ---- residual_conv.cu (post-norm residual add + short input convolution, fp32 residual stream)
+struct ResidualConvParams {
+  const void* y;           // [tokens, D] sublayer output (or the embedding rows when x is null)
+  const float* x;          // [tokens, D] residual stream or null
+  float* x_out;            // [tokens, D] new residual stream (another buffer than x)
+  void* h;                 // [tokens, D] what the next sublayer reads
+  const void* gain;        // 1 or D numbers, or null
+  const void* w;           // [D, K]
+  float* carry;            // [slots, K-1, D] or null
+  const int* qsl;          // [batch + 1]
+  const int* state_idx;    // [batch] or null
+  const int* has_init;     // [batch] or null
+  int gain_per_channel, batch, tokens, D, K, vec;
+  float eps;
+};
+int residual_conv(const ResidualConvParams& p, int dtype, cudaStream_t stream);
+int residual_norm(void* out, const float* x, const void* y, const void* gain, const void* gain2, int gain_n, int gain2_n,
+                  float eps, int tokens, int D, int vec, int dtype, cudaStream_t stream);
+// ---- gla.cu (gated linear attention: decay per key channel)
+struct GlaParams {
+  const void* qkvg;            // [tokens, row_stride]: q | k | v | gate at the given element offsets
+  int64_t row_stride;
+  int q_off, k_off, v_off, g_off;
+  const float* z;              // [tokens, heads * dim] decay logits without their bias
+  const void* z_bias;          // [heads * dim] or null
+  const void* norm_w;          // [vdim]
+  float* state;                // [slots, heads, dim, vdim]
+  float* o_raw;                // [tokens, heads * vdim] scratch of the split form (columns of a head over several CTAs)
+  void* out;                   // [tokens, heads * vdim]
+  const int* qsl; const int* state_idx; const int* has_init;
+  int batch, tokens, heads, dim, vdim, col_block;
+  float scale, inv_tau, eps;
+};
+int gla_recurrent(GlaParams p, int max_query_len, int sms, int dtype, cudaStream_t stream);
+bool gla_needs_scratch(int batch, int heads, int dim, int vdim, int max_query_len, int sms);
+// ---- rglru.cu (real-gated linear recurrent unit)
+struct RgLruParams {
+  const void* u; int64_t u_stride;       // [tokens, width] recurrence input
+  const void* y; int64_t y_stride;       // [tokens, width] gate branch before its gelu
+  float* gates;                          // [tokens, blocks, 2, width / blocks] logits without bias; overwritten
+  const float* r_bias; const float* i_bias; const float* decay;   // [width]; decay = -8 softplus(lambda)
+  float* state;                          // [slots, width]
+  float* summary;                        // [chunks, 2, width] scratch, needed when a sequence spans several chunks
+  void* out;                             // [tokens, width]
+  const int* qsl; const int* state_idx; const int* has_init;
+  int batch, tokens, width, block_width;
+};
+int rglru_chunk();                       // tokens per chunk
+int rglru_scan(const RgLruParams& p, int max_query_len, int dtype, cudaStream_t stream);
+// ---- latent_attn.cu (latent attention of any sizes: projection epilogues, fp32 attention)
+struct LatentInsertParams {
+  const void* a; int64_t a_stride; int q_off, kv_off;   // [tokens, ...]: query latent | key latent, rotated key part
+  const void* q_w; const void* kv_w;                    // norm weights
+  void* cq;                                             // [tokens, q_rank]
+  void* cache; int64_t row_elems, num_slots;            // [slots, row_elems]
+  const int64_t* slots; const int64_t* positions;
+  const float* inv_freq;                                // [rot_dims / 2]
+  int tokens, q_rank, kv_rank, rot_dim, rot_dims;
+  float eps;
+  StatusWord* status;
+};
+int latent_insert(const LatentInsertParams& p, int dtype, cudaStream_t stream);
+// Rotates the first rot_dims of the rot_dim entries at src (per token and head) into dst and zeroes `pad` entries behind.
+int latent_rope(const void* src, int64_t src_tok, int64_t src_head, void* dst, int64_t dst_tok, int64_t dst_head,
+                const int64_t* positions, const float* inv_freq, int tokens, int heads, int rot_dim, int rot_dims, int pad,
+                int dtype, cudaStream_t stream);
+int latent_attn_simt(const MlaDecodeParams& p, int dtype, cudaStream_t stream);
 // ---- tq_cache.cu (TurboQuant KV cache, head_dim 128)
 int tq_slot_bytes(int kbits, int vbits);
 int tq_store(void* cache, const void* k, const void* v, int64_t k_stride, int64_t v_stride, const int64_t* slot_mapping,

@@ -389,7 +389,8 @@ def _resolve_model(model: Union[str, dict, ModelConfig], **overrides) -> tuple[M
             setattr(mc, k, v)
         mc.__post_init__()
     elif isinstance(model, dict):
-        mc = ModelConfig.from_hf_dict(model, **overrides) if "hidden_size" in model and "architectures" in model \
+        mc = ModelConfig.from_hf_dict(model, **overrides) if ("hidden_size" in model and "architectures" in model) \
+            or isinstance(model.get("layers"), list) \
             else ModelConfig(**{**model, **overrides})
     elif isinstance(model, str) and model.endswith(".gguf"):       # llama.cpp single-file checkpoint
         from .gguf import config_from_gguf, read_gguf

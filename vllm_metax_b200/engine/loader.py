@@ -107,6 +107,17 @@ def iter_safetensors(path: str) -> Iterator[tuple[str, torch.Tensor]]:
                 yield k, f.get_tensor(k)
 
 
+def safetensors_shapes(path: str) -> dict[str, tuple]:
+    """Tensor name -> shape of every safetensors file under ``path``, from the file headers alone."""
+    out: dict[str, tuple] = {}
+    for fn in sorted(glob.glob(os.path.join(path, "*.safetensors"))):
+        with open(fn, "rb") as f:
+            n = int.from_bytes(f.read(8), "little")
+            head = json.loads(f.read(n))
+        out.update({k: tuple(v["shape"]) for k, v in head.items() if k != "__metadata__"})
+    return out
+
+
 def save_sharded_state(model: nn.Module, path: str, rank: int) -> None:
     from safetensors.torch import save_file
 

@@ -27,6 +27,7 @@ from ..attention.metadata import AttentionMetadata, ForwardContext, set_forward_
 from ..config import EngineConfig
 from ..layers.attention import PagedGQABackend
 from ..parallel import state as ps
+from ..models import get_model_class
 from .loader import build_model
 from .scheduler import SchedulerOutput
 
@@ -48,7 +49,7 @@ class ModelRunner:
         if cfg.device == "cuda":
             self.device = torch.device("cuda", ps.local_rank() if torch.cuda.device_count() > 1 else 0)
             torch.cuda.set_device(self.device)
-            if not ops.load_native():
+            if not ops.load_native(units=getattr(get_model_class(cfg.model.architecture), "native_units", "all")):
                 raise RuntimeError("native library missing on a GPU box; run python -m vllm_metax_b200._build")
         else:
             self.device = torch.device("cpu")
@@ -270,6 +271,8 @@ class ModelRunner:
 
     def release_request(self, req) -> None:
         """Called when a request gives its KV blocks back (finished, aborted or preempted for re-computation)."""
+        # a pre-empted request may come back to the same batch row with other blocks: write that row's table anew
+        self._bt_owner = [None if o is not None and o[0] is req else o for o in self._bt_owner]
         if self.state_slots is not None:
             slot = self.state_slots.pop(req.request_id, None)
             if slot is not None:
@@ -470,6 +473,8 @@ class ModelRunner:
             block_table=self.block_table[:B_eff], slot_mapping=self.slot_mapping[:T], max_query_len=max_q,
             max_seq_len=max_seq, block_size=bs, prefill_query_start_loc=self.prefill_qsl[:B_eff - nd_eff + 1],
             max_prefill_query_len=max_q if B_eff > nd_eff else 0)
+        if B_eff > nd_eff:        # prompt portions: layers that size buffers by their context read these on the host
+            md.seq_lens_cpu, md.query_start_loc_cpu = torch.from_numpy(sl[:B_eff].copy()), torch.from_numpy(qsl[:B_eff + 1].copy())
         # MLA: prefill requests without cached context may take the up-projected MHA path
         md.extra["prefill_no_context"] = all(s.start_pos == 0 for s in so.scheduled[nd:])
         if self.cascade and B >= 2 and pad_to <= B:
@@ -793,7 +798,9 @@ class ModelRunner:
             bucket = next((b for b in self.buckets if b >= B), 0)
             if bucket and self.cascade and self._cascade_applies(so):
                 bucket = 0        # the shared prefix is worth more than the captured graph: this step runs eagerly
+        self._await_staging()
         md, T, rows, reqs = self._prepare(so, pad_to=bucket)
+        self._mark_staged()
         all_greedy = all(r.params.greedy and not r.params.needs_penalties and not r.params.constrained for r in reqs)
         n = len(rows)
         logits = None
@@ -847,6 +854,42 @@ class ModelRunner:
             if s.num_spec and s.samples and not isinstance(out.get(s.request.request_id), list):
                 out[s.request.request_id] = [out[s.request.request_id]]
         return out
+
+    def _await_staging(self) -> None:
+        """The pinned staging areas may be rewritten once the previous step's copies have read them (a step that samples
+        nothing returns without waiting for the device)."""
+        if self.is_cuda and self._prep_done is not None:
+            self._prep_done.synchronize()
+
+    def _mark_staged(self) -> None:
+        if self.is_cuda:
+            self._prep_done = torch.cuda.Event()
+            self._prep_done.record()
+
+    @torch.no_grad()
+    def execute_logits(self, so: SchedulerOutput, places: list[list[int]]) -> Optional[torch.Tensor]:
+        """One step like ``execute`` that samples nothing: returns the logits ``[n, vocab]`` (fp32, on the host) at
+        ``places[i]`` - offsets among the tokens that ``so.scheduled[i]`` brings - in that order, or None if there are
+        none.  Decode-only steps replay the captured graphs, as they do when generating."""
+        B = len(so.scheduled)
+        bucket = 0
+        if self.use_graphs and so.num_decode == B and B > 0 and self.graphs:
+            bucket = next((b for b in self.buckets if b >= B), 0)
+        self._await_staging()
+        md, T, _, _ = self._prepare(so, pad_to=bucket)
+        self._mark_staged()
+        rows, t = [], 0
+        for s, ps_ in zip(so.scheduled, places):
+            rows += [t + p for p in ps_]
+            t += s.num_new_tokens
+        if bucket:
+            g, logits, _ = self.graphs[bucket]
+            g.replay()
+            return logits[torch.as_tensor(rows, device=self.device)].float().cpu() if rows else None
+        h = self._forward(md, T)
+        if not rows:
+            return None
+        return self.model.compute_logits(h[torch.as_tensor(rows, device=self.device)]).float().cpu()
 
     @torch.no_grad()
     def execute_dummy(self) -> None:

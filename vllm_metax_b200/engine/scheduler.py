@@ -198,6 +198,40 @@ class Scheduler:
         out.num_decode = len(dec)
         return out
 
+    # ------------------------------------------------------------------ steps dictated from outside
+    def schedule_portions(self, portions: list[tuple[Request, int]]) -> SchedulerOutput:
+        """A step over exactly these requests and token counts (replaying a recorded schedule): the next ``n`` tokens of
+        each, blocks taken from the same pool, decode rows first.  A request is admitted at its first portion; it may sit
+        out steps in between.  Nothing is pre-empted: running out of blocks is an error."""
+        out = SchedulerOutput()
+        for req, n in portions:
+            if n <= 0 or req.num_computed_tokens + n > req.num_tokens:
+                raise ValueError(f"request {req.request_id}: a portion of {n} tokens does not exist")
+            if req.num_computed_tokens + n > self.cfg.max_model_len:
+                raise ValueError(f"request {req.request_id} exceeds max_model_len {self.cfg.max_model_len}")
+            if req not in self.running:
+                if len(self.running) >= self.cfg.max_num_seqs:
+                    raise RuntimeError("more live requests than max_num_seqs")
+                req.status = RequestStatus.RUNNING
+                self.running.append(req)
+            self.kv.allocate(req, n)
+            out.scheduled.append(ScheduledRequest(req, n, req.num_computed_tokens, False))
+        dec = [s for s in out.scheduled if s.num_new_tokens == 1 and s.start_pos > 0]
+        out.scheduled = dec + [s for s in out.scheduled if not (s.num_new_tokens == 1 and s.start_pos > 0)]
+        out.num_decode = len(dec)
+        return out
+
+    def advance_portions(self, out: SchedulerOutput) -> None:
+        for s in out.scheduled:
+            s.request.num_computed_tokens += s.num_new_tokens
+
+    def retire(self, req: Request) -> None:
+        """Give back everything a request holds."""
+        if req in self.running:
+            self.running.remove(req)
+        req.status = RequestStatus.FINISHED_STOPPED
+        self.kv.free(req)
+
     # ------------------------------------------------------------------ two-phase update (overlapped host work)
     # The engine may prepare step k + 1 on the host while the device still runs step k.  ``begin_step`` applies what
     # step k changes without knowing its tokens (computed-token counts, a provisional output token per sampling

@@ -11,7 +11,8 @@ Data flow on one rank (bf16):
     out            = sum_k w_k * Y[pos(t, k)] (+ shared expert)
 
 Weights: ``w13 [E_local, 2I, H]`` with gate/up rows interleaved (row 2j = gate_j, 2j+1 = up_j),
-``w2 [E_local, H, I]``.
+``w2 [E_local, H, I]``.  Experts without a gate (``gated=False``) hold ``w13 [E_local, I, H]`` and apply their activation
+in the same epilogue.
 
 Expert parallelism: experts are sharded over the EP group (``E_local = E / ep``).
 
@@ -51,7 +52,7 @@ BLOCK_M = 128
 
 def fused_experts(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_weights: torch.Tensor,
                   topk_ids: torch.Tensor, num_local_experts: int, expert_map: Optional[torch.Tensor] = None,
-                  shared_out: Optional[torch.Tensor] = None) -> torch.Tensor:
+                  shared_out: Optional[torch.Tensor] = None, epi: int = ops.EPI_CODES["silu_gate"]) -> torch.Tensor:
     """Expert MLPs for the pairs routed to this rank's experts; returns ``[T, H]`` (partial sum
     when ``expert_map`` drops pairs owned by other ranks)."""
     T, H = x.shape
@@ -59,7 +60,7 @@ def fused_experts(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_wei
     sorted_ids, block_expert, total, inv = ops.moe_align_block_size(topk_ids, BLOCK_M, num_local_experts,
                                                                     expert_map, want_inverse=True)
     a = ops.moe_gather(x, sorted_ids, total, topk)
-    h = ops.gemm_grouped(a, w13, block_expert, total, epi=1)
+    h = ops.gemm_grouped(a, w13, block_expert, total, epi=epi)
     y = ops.gemm_grouped(h, w2, block_expert, total, epi=0)
     return ops.moe_combine(y, topk_weights, inv, T, shared_out)
 
@@ -69,8 +70,14 @@ class FusedMoE(nn.Module):
                  dtype=torch.bfloat16, renormalize: bool = True, scoring_func: str = "softmax",
                  use_grouped_topk: bool = False, num_expert_group: int = 1, topk_group: int = 1,
                  routed_scaling_factor: float = 1.0, e_score_correction_bias: bool = False,
-                 reduce_results: bool = True, quant_method=None, prefix: str = ""):
+                 reduce_results: bool = True, quant_method=None, prefix: str = "",
+                 gated: bool = True, activation: str = "silu"):
         super().__init__()
+        # gated: SiLU(gate) * up over interleaved rows; otherwise one up projection through `activation`
+        assert not gated or activation == "silu", "gated experts use the SiLU gate"
+        assert gated or quant_method is None, "quantised experts are gated"
+        self.gated = gated
+        self.epi = ops.EPI_CODES["silu_gate" if gated else activation]
         self.num_experts, self.top_k = num_experts, top_k
         self.hidden_size, self.intermediate_size = hidden_size, intermediate_size
         self.renormalize, self.scoring_func = renormalize, scoring_func
@@ -93,7 +100,7 @@ class FusedMoE(nn.Module):
         if quant_method is not None:
             quant_method.create_weights(self, self.num_local, hidden_size, intermediate_size, dtype)
         else:
-            self.w13_weight = nn.Parameter(torch.empty(self.num_local, 2 * intermediate_size, hidden_size, dtype=dtype),
+            self.w13_weight = nn.Parameter(torch.empty(self.num_local, (2 if gated else 1) * intermediate_size, hidden_size, dtype=dtype),
                                            requires_grad=False)
             self.w2_weight = nn.Parameter(torch.empty(self.num_local, hidden_size, intermediate_size, dtype=dtype),
                                           requires_grad=False)
@@ -179,6 +186,8 @@ class FusedMoE(nn.Module):
         for e in self._local_slots(expert_id):
             if self.quant_method is not None and hasattr(self.quant_method, "load_expert_weight"):
                 self.quant_method.load_expert_weight(self, param, loaded, e, shard)
+            elif not self.gated and shard in ("w1", "w3"):
+                param.data[e].copy_(loaded)
             elif shard == "w1":
                 param.data[e, 0::2].copy_(loaded)
             elif shard == "w3":
@@ -214,7 +223,7 @@ class FusedMoE(nn.Module):
         qm = self.quant_method
         if qm is not None:
             return qm.apply_sorted(self, a, a_scale, block_expert, total)
-        h = ops.gemm_grouped(a, self.w13_weight, block_expert, total, epi=1)
+        h = ops.gemm_grouped(a, self.w13_weight, block_expert, total, epi=self.epi)
         return ops.gemm_grouped(h, self.w2_weight, block_expert, total)
 
     def _forward_sp(self, x: torch.Tensor, router_logits: torch.Tensor,
@@ -261,7 +270,7 @@ class FusedMoE(nn.Module):
                 part = qm.apply(self, h_all, w_all, ids_all.to(torch.int32), None)
             else:
                 part = fused_experts(h_all, self.w13_weight, self.w2_weight, w_all, ids_all.to(torch.int32),
-                                     self.num_local, self.expert_map, None)
+                                     self.num_local, self.expert_map, None, self.epi)
             mine = mgr.combine(part)
         y = tpg.all_gatherv(mine.contiguous(), sizes)
         if shared_out is not None:       # shared experts are tensor-parallel: their partial sums still need the reduction
@@ -309,7 +318,7 @@ class FusedMoE(nn.Module):
         def experts(xs, ws, idss, shared):
             if self.quant_method is not None:
                 return self.quant_method.apply(self, xs, ws, idss, shared)
-            return fused_experts(xs, self.w13_weight, self.w2_weight, ws, idss, self.num_local, self.expert_map, shared)
+            return fused_experts(xs, self.w13_weight, self.w2_weight, ws, idss, self.num_local, self.expert_map, shared, self.epi)
 
         chunk = int(envs.B200_FUSED_MOE_CHUNK_SIZE)
         T = x.shape[0]

@@ -52,6 +52,7 @@ _MODELS: dict[str, tuple[str, str]] = {
     "InternVLForConditionalGeneration": ("internvl", "InternVLForConditionalGeneration"),
     "InternVLChatModel": ("internvl", "InternVLChatModel"),
     "InternS1ForConditionalGeneration": ("internvl", "InternVLForConditionalGeneration"),    # the same graph, other decoder
+    "Naguzen": ("naguzen", "NaguzenForCausalLM"),
     "MambaForCausalLM": ("mamba", "MambaForCausalLM"),
     "Qwen3NextForCausalLM": ("qwen3_next", "Qwen3NextForCausalLM"),
     "Glm4MoeForCausalLM": ("moe_family", "Glm4MoeForCausalLM"),

@@ -188,7 +188,7 @@ def causal_conv1d(x, w, bias=None, state=None, query_start_loc=None, state_indic
         return causal_conv1d_ref(x, w, bias, state, query_start_loc, state_indices, has_initial_state, silu)
     from .. import _custom_ops as ops
 
-    ops.load_native()
+    ops.load_native(units="core")
     out = torch.empty(x.shape, dtype=x.dtype, device=x.device)
     ops._launches += 2 if state is not None else 1
     torch.ops.b200.causal_conv1d(out, x, w.contiguous(), bias, state, query_start_loc.int().contiguous(),

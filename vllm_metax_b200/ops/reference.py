@@ -324,6 +324,25 @@ def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
     return y.to(out_dtype or a.dtype)
 
 
+def epilogue_activation(y: torch.Tensor, act: str, params: Optional[torch.Tensor]) -> torch.Tensor:
+    """The activations of the GEMM epilogues, fp32.  xIELU: ``params`` = (quadratic, exponential) coefficients."""
+    if act == "gelu":
+        return torch.nn.functional.gelu(y)
+    if act == "gelu_tanh":
+        return torch.nn.functional.gelu(y, approximate="tanh")
+    a, b = params.float()
+    return torch.where(y > 0, a * y * y, b * (torch.expm1(y.clamp(max=0)) - y)) + 0.5 * y
+
+
+def rotate_half(x: torch.Tensor, inv_freq: torch.Tensor, positions: torch.Tensor) -> torch.Tensor:
+    """Rotation of the first ``2 * len(inv_freq)`` entries of ``x [T, H, D]``, pairs (i, i + half), angles in fp32."""
+    half = inv_freq.numel()
+    a = positions[: x.shape[0]].float()[:, None] * inv_freq[None]
+    c, s = torch.cos(a)[:, None], torch.sin(a)[:, None]
+    u, v = x[..., :half].float(), x[..., half: 2 * half].float()
+    return torch.cat([(u * c - v * s).to(x.dtype), (v * c + u * s).to(x.dtype), x[..., 2 * half:]], -1)
+
+
 def dequant_block_fp8_weight(wq: torch.Tensor, scale_inv: torch.Tensor, block: Sequence[int] = (128, 128)):
     """``wq [N,K]`` e4m3 with ``scale_inv [ceil(N/bn), ceil(K/bk)]`` -> fp32."""
     N, K = wq.shape[-2:]
@@ -568,7 +587,7 @@ def gather_mla_cache(mla_cache, block_table_row, kv_len):
 
 
 def mla_decode(q, mla_cache, block_table, seq_lens, scale, kv_lora_rank: int = 512,
-               query_start_loc=None, topk_indices: Optional[torch.Tensor] = None):
+               query_start_loc=None, topk_indices: Optional[torch.Tensor] = None, window: int = 0):
     """Absorbed MLA (MQA over the latent cache).
 
     ``q [T, H, 576]`` (``q_nope @ W_UK`` | ``q_pe``); output ``[T, H, 512]`` and
@@ -596,6 +615,8 @@ def mla_decode(q, mla_cache, block_table, seq_lens, scale, kv_lora_rank: int = 5
         kpos = torch.arange(L, device=q.device)[None, :]
         qpos = (L - Lq + torch.arange(Lq, device=q.device))[:, None]
         mask = kpos > qpos
+        if window > 0:
+            mask = mask | (kpos <= qpos - window)
         if topk_indices is not None:
             idx = topk_indices[s0:s1].long()
             sel = torch.zeros(Lq, L + 1, dtype=torch.bool, device=q.device)
