@@ -6,6 +6,7 @@
 #include <torch/types.h>
 
 #include <cstdlib>
+#include <initializer_list>
 #include <cstring>
 #include <tuple>
 
@@ -35,6 +36,16 @@ inline int dtype16(const Tensor& t) {
 template <typename T = void>
 inline T* ptr(const optional<Tensor>& t) {
   return t.has_value() && t->defined() ? reinterpret_cast<T*>(t->data_ptr()) : nullptr;
+}
+
+// Every tensor of a call must live on `ref`'s GPU: a host pointer in a kernel is a fault.
+inline void on_device_of(const Tensor& ref, std::initializer_list<const Tensor*> ts,
+                         std::initializer_list<const optional<Tensor>*> os = {}) {
+  TORCH_CHECK(ref.is_cuda(), "expected a CUDA tensor");
+  for (const Tensor* t : ts) TORCH_CHECK(t->device() == ref.device(), "tensors on ", t->device(), " and ", ref.device());
+  for (const optional<Tensor>* o : os)
+    if (o->has_value() && (*o)->defined())
+      TORCH_CHECK((*o)->device() == ref.device(), "tensors on ", (*o)->device(), " and ", ref.device());
 }
 
 // One status word per device, zero-initialised on first use.

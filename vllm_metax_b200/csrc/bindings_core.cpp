@@ -29,6 +29,7 @@ b200::Epi make_epi(const Tensor& out, const Tensor& a, int64_t act, const option
 
 void gemm(Tensor& out, const Tensor& a, const Tensor& w, const optional<Tensor>& bias,
           const optional<Tensor>& residual, int64_t force_bn, int64_t act, const optional<Tensor>& act_params) {
+  on_device_of(a, {&out, &w}, {&bias, &residual, &act_params});
   TORCH_CHECK(a.dim() == 2 && w.dim() == 2 && out.dim() == 2, "gemm expects 2-D tensors");
   TORCH_CHECK(a.stride(1) == 1 && w.stride(1) == 1 && out.stride(1) == 1, "inner dims must be contiguous");
   const int M = a.size(0), K = a.size(1), N = w.size(0);
@@ -196,6 +197,7 @@ void moe_sum(Tensor& out, const Tensor& in) {
 
 void gemm_grouped(Tensor& out, const Tensor& a, const Tensor& w, const Tensor& block_expert,
                   const Tensor& total_padded, int64_t act) {
+  on_device_of(a, {&out, &w, &block_expert, &total_padded});
   const b200::Epi epi = make_epi(out, a, act, c10::nullopt);
   TORCH_CHECK(a.dim() == 2 && w.dim() == 3 && a.stride(1) == 1 && w.is_contiguous() && out.stride(1) == 1);
   TORCH_CHECK(a.size(0) % 128 == 0 && a.size(1) == w.size(2) && a.size(1) % 8 == 0 && a.stride(0) % 8 == 0);
@@ -210,6 +212,7 @@ void gemm_grouped(Tensor& out, const Tensor& a, const Tensor& w, const Tensor& b
 void causal_conv1d(Tensor& out, const Tensor& x, const Tensor& w, const optional<Tensor>& bias,
                    const optional<Tensor>& state, const Tensor& query_start_loc, const optional<Tensor>& state_idx,
                    const optional<Tensor>& has_initial, bool silu) {
+  on_device_of(x, {&out, &w, &query_start_loc}, {&bias, &state, &state_idx, &has_initial});
   TORCH_CHECK(x.dim() == 2 && x.stride(1) == 1 && out.is_contiguous() && out.sizes() == x.sizes() &&
               out.scalar_type() == x.scalar_type());
   const int64_t T = x.size(0), C = x.size(1), K = w.size(1);
@@ -317,6 +320,7 @@ void mla_decode(Tensor& out, const Tensor& q, const Tensor& cache, const Tensor&
                 const optional<Tensor>& query_start_loc, const optional<Tensor>& topk_indices, double scale,
                 const optional<Tensor>& lse_out, const optional<Tensor>& workspace, int64_t num_splits, int64_t impl,
                 int64_t window) {
+  on_device_of(q, {&out, &cache, &block_table, &seq_lens}, {&query_start_loc, &topk_indices, &lse_out, &workspace});
   TORCH_CHECK(q.dim() == 3 && q.stride(2) == 1 && q.stride(1) == q.size(2));
   TORCH_CHECK(cache.is_contiguous() && cache.dim() == 3 && out.is_contiguous() && out.size(2) <= q.size(2));
   const bool rec = cache.scalar_type() == at::kByte;
@@ -365,6 +369,7 @@ void mla_decode(Tensor& out, const Tensor& q, const Tensor& cache, const Tensor&
 
 void gather_mla_cache(Tensor& dst, const Tensor& cache, const Tensor& block_table, const Tensor& cu_seq_lens,
                       const optional<Tensor>& seq_starts) {
+  on_device_of(dst, {&cache, &block_table, &cu_seq_lens}, {&seq_starts});
   TORCH_CHECK(dst.is_contiguous() && dst.size(1) % 8 == 0 && cache.is_contiguous() && cache.dim() == 3);
   const bool rec = cache.scalar_type() == at::kByte;
   TORCH_CHECK(rec ? (cache.size(2) == 656 && dst.size(1) == 576) : (cache.size(2) == dst.size(1) && cache.scalar_type() == dst.scalar_type()));
@@ -376,6 +381,7 @@ void gather_mla_cache(Tensor& dst, const Tensor& cache, const Tensor& block_tabl
 
 // out[z] = act(a[z] @ w[z]^T): a [Z, M, K], w [Z, N, K], out [Z, M, N] (strided views; 16-bit operands)
 void gemm_batched(Tensor& out, const Tensor& a, const Tensor& w, int64_t act) {
+  on_device_of(a, {&out, &w});
   TORCH_CHECK(a.dim() == 3 && w.dim() == 3 && out.dim() == 3 && a.stride(2) == 1 && w.stride(2) == 1 && out.stride(2) == 1);
   const int64_t Z = a.size(0), M = a.size(1), K = a.size(2), N = w.size(1);
   TORCH_CHECK(w.size(0) == Z && w.size(2) == K && out.size(0) == Z && out.size(1) == M && out.size(2) == N &&
@@ -395,6 +401,7 @@ void gemm_batched(Tensor& out, const Tensor& a, const Tensor& w, int64_t act) {
 void gemm_simt(Tensor& out, const Tensor& a, const Tensor& w, const optional<Tensor>& bias, int64_t act,
                const optional<Tensor>& act_params, const optional<Tensor>& block_expert,
                const optional<Tensor>& total_padded) {
+  on_device_of(a, {&out, &w}, {&bias, &act_params, &block_expert, &total_padded});
   const bool grouped = block_expert.has_value();
   TORCH_CHECK(a.dim() == out.dim() && (grouped ? (a.dim() == 2 && w.dim() == 3) : w.dim() == a.dim()));
   TORCH_CHECK(a.stride(-1) == 1 && w.stride(-1) == 1 && out.stride(-1) == 1 && a.scalar_type() == w.scalar_type());
@@ -436,6 +443,7 @@ StepRefs step_refs(const Tensor& qsl, const optional<Tensor>& idx, const optiona
 void residual_conv(Tensor& x_out, Tensor& h, const Tensor& y, const optional<Tensor>& x, const optional<Tensor>& gain,
                    const Tensor& w, const optional<Tensor>& carry, const Tensor& qsl, const optional<Tensor>& state_idx,
                    const optional<Tensor>& has_init, double eps) {
+  on_device_of(y, {&x_out, &h, &w, &qsl}, {&x, &gain, &carry, &state_idx, &has_init});
   const int64_t T = y.size(0), D = y.size(1), K = w.size(1);
   TORCH_CHECK(y.dim() == 2 && y.is_contiguous() && h.is_contiguous() && h.sizes() == y.sizes() && h.scalar_type() == y.scalar_type());
   TORCH_CHECK(x_out.is_contiguous() && x_out.sizes() == y.sizes() && x_out.scalar_type() == at::kFloat);
@@ -461,6 +469,7 @@ void residual_conv(Tensor& x_out, Tensor& h, const Tensor& y, const optional<Ten
 
 void residual_norm(Tensor& out, const Tensor& y, const optional<Tensor>& x, const optional<Tensor>& gain,
                    const Tensor& gain2, double eps) {
+  on_device_of(y, {&out, &gain2}, {&x, &gain});
   const int64_t T = y.size(0), D = y.size(1);
   TORCH_CHECK(y.dim() == 2 && y.is_contiguous() && out.is_contiguous() && out.sizes() == y.sizes() && out.scalar_type() == y.scalar_type());
   TORCH_CHECK(gain2.scalar_type() == y.scalar_type() && (gain2.numel() == 1 || gain2.numel() == D));
@@ -492,6 +501,7 @@ void gla_recurrent(Tensor& out, Tensor& state, const Tensor& qkvg, int64_t q_off
                    int64_t g_off, const Tensor& z, const optional<Tensor>& z_bias, const Tensor& norm_w,
                    const optional<Tensor>& scratch, const Tensor& qsl, const optional<Tensor>& state_idx,
                    const optional<Tensor>& has_init, double scale, double inv_tau, double eps, int64_t max_query_len) {
+  on_device_of(qkvg, {&out, &state, &z, &norm_w, &qsl}, {&z_bias, &scratch, &state_idx, &has_init});
   TORCH_CHECK(state.dim() == 4 && state.is_contiguous() && state.scalar_type() == at::kFloat);
   const int64_t T = qkvg.size(0), H = state.size(1), D = state.size(2), V = state.size(3);
   TORCH_CHECK(qkvg.dim() == 2 && qkvg.stride(1) == 1 && out.is_contiguous() && out.size(0) == T && out.size(1) == H * V &&
@@ -524,6 +534,7 @@ void rglru_scan(Tensor& out, Tensor& state, Tensor& gates, const Tensor& u, cons
                 const Tensor& i_bias, const Tensor& decay, int64_t block_width, const optional<Tensor>& summary,
                 const Tensor& qsl, const optional<Tensor>& state_idx, const optional<Tensor>& has_init,
                 int64_t max_query_len) {
+  on_device_of(u, {&out, &state, &gates, &y, &r_bias, &i_bias, &decay, &qsl}, {&summary, &state_idx, &has_init});
   const int64_t T = u.size(0), W = u.size(1);
   TORCH_CHECK(u.dim() == 2 && u.stride(1) == 1 && y.dim() == 2 && y.stride(1) == 1 && y.sizes() == u.sizes() &&
               y.scalar_type() == u.scalar_type() && out.is_contiguous() && out.sizes() == u.sizes() && out.scalar_type() == u.scalar_type());
@@ -549,6 +560,7 @@ void rglru_scan(Tensor& out, Tensor& state, Tensor& gates, const Tensor& u, cons
 void latent_insert(Tensor& cq, Tensor& cache, const Tensor& a, int64_t q_off, int64_t kv_off, const Tensor& q_w,
                    const Tensor& kv_w, int64_t rot_dim, const Tensor& inv_freq, const Tensor& positions,
                    const Tensor& slot_mapping, double eps) {
+  on_device_of(a, {&cq, &cache, &q_w, &kv_w, &inv_freq, &positions, &slot_mapping});
   const int64_t T = a.size(0), QR = cq.size(1), KR = kv_w.numel();
   TORCH_CHECK(a.dim() == 2 && a.stride(1) == 1 && cq.is_contiguous() && cq.size(0) == T && cq.scalar_type() == a.scalar_type());
   TORCH_CHECK(cache.dim() == 3 && cache.is_contiguous() && cache.scalar_type() == a.scalar_type() && cache.size(2) >= KR + rot_dim);
@@ -572,6 +584,7 @@ void latent_insert(Tensor& cq, Tensor& cache, const Tensor& a, int64_t q_off, in
 // src, dst [T, H, >= rot_dim] views (last dimension contiguous; may be the same memory)
 void latent_rope(Tensor& dst, const Tensor& src, const Tensor& inv_freq, const Tensor& positions, int64_t rot_dim,
                  int64_t pad) {
+  on_device_of(src, {&dst, &inv_freq, &positions});
   TORCH_CHECK(src.dim() == 3 && dst.dim() == 3 && src.stride(2) == 1 && dst.stride(2) == 1 && src.size(0) == dst.size(0) &&
               src.size(1) == dst.size(1) && src.size(2) >= rot_dim && dst.size(2) >= rot_dim + pad);
   TORCH_CHECK(src.scalar_type() == dst.scalar_type() && positions.scalar_type() == at::kLong && positions.numel() >= src.size(0));

@@ -719,6 +719,7 @@ class ModelRunner:
             md.decode_workspace = torch.empty(md.decode_num_splits * bucket * hq * (spec["head_size"] + 1),
                                               dtype=torch.float32, device=self.device)
         # safe dummy inputs for warm-up
+        self.query_start_loc[:bucket + 1].copy_(torch.arange(bucket + 1, dtype=torch.int32))
         self.seq_lens[:bucket].fill_(1)
         self.slot_mapping[:bucket].fill_(-1)
         self.block_table[:bucket].zero_()

@@ -72,7 +72,8 @@ class LatentAttention(nn.Module):
         self.up_v = _param(heads * vdim, kv_rank, dtype=dtype)
         self.out_proj = _param(width, heads * vdim, dtype=dtype)
         i = torch.arange(rot_dims // 2, dtype=torch.float64, device="cpu")
-        self.register_buffer("inv_freq", (float(rot_base) ** (-2.0 * i / rot_dims)).float(), persistent=False)
+        freq = (float(rot_base) ** (-2.0 * i / rot_dims)).float().to(torch.get_default_device())
+        self.register_buffer("inv_freq", freq, persistent=False)
         # filled by finalize_weights: W_UK transposed per head, and the prompt path's [k | rotated k | v] matrix
         self.register_buffer("absorb_k", torch.zeros(heads, kv_rank, dim, dtype=dtype), persistent=False)
         qk = dim + rot_dim
