@@ -279,4 +279,11 @@ def random_weights(cfg, seed=0):
             if leaf == "router":
                 t = 2.0 * t
         w[name] = t.to(torch.bfloat16)
+    # the experts of a layer are variations of one: where rounding decides between two of equal score, the output moves
+    # little (a wrong expert still stands far above the fp32 limits)
+    for name in w:
+        head, _, leaf = name.rpartition(".")
+        if ".mlp.e" in name and not head.endswith(".e0"):
+            first = head[: head.rindex(".e")] + ".e0." + leaf
+            w[name] = (w[first].float() + 0.25 * w[name].float()).to(torch.bfloat16)
     return w

@@ -175,7 +175,7 @@ void moe_align(Tensor& sorted_ids, Tensor& block_expert, Tensor& total_padded, c
 }
 
 void moe_gather(Tensor& out, const Tensor& x, const Tensor& sorted_ids, const Tensor& total_padded, int64_t topk) {
-  TORCH_CHECK(x.is_contiguous() && out.is_contiguous() && (x.size(1) % 8 == 0 || x.scalar_type() == at::kFloat));
+  TORCH_CHECK(x.is_contiguous() && out.is_contiguous());
   const c10::cuda::CUDAGuard guard(x.device());
   b200::moe_gather(out.data_ptr(), x.data_ptr(), sorted_ids.data_ptr<int>(), total_padded.data_ptr<int>(),
                    out.size(0), x.size(0) * topk, topk, x.size(1), dtype_code(x), cur_stream());

@@ -321,28 +321,30 @@ __global__ void moe_combine_kernel(T* __restrict__ out, const T* __restrict__ y,
   }
 }
 
-// fp32 rows (a model served in 32-bit): one element per thread and trip.
-__global__ void moe_gather_f32_kernel(float* __restrict__ out, const float* __restrict__ x,
-                                      const int* __restrict__ sorted_ids, const int* __restrict__ total_padded, int numel,
-                                      int topk, int hidden) {
+// Rows of fp32, or of a width that 16-byte vectors do not divide: one element per thread and trip.
+template <typename T>
+__global__ void moe_gather_scalar_kernel(T* __restrict__ out, const T* __restrict__ x,
+                                         const int* __restrict__ sorted_ids, const int* __restrict__ total_padded,
+                                         int numel, int topk, int hidden) {
   const int row = blockIdx.x;
   if (row >= *total_padded) return;
   const int id = sorted_ids[row];
   for (int i = threadIdx.x; i < hidden; i += blockDim.x)
-    out[(size_t)row * hidden + i] = id < numel ? x[(size_t)(id / topk) * hidden + i] : 0.f;
+    out[(size_t)row * hidden + i] = id < numel ? x[(size_t)(id / topk) * hidden + i] : from_f<T>(0.f);
 }
 
-__global__ void moe_combine_f32_kernel(float* __restrict__ out, const float* __restrict__ y,
-                                       const float* __restrict__ weights, const int* __restrict__ inv_pos,
-                                       const float* __restrict__ shared, int topk, int hidden) {
+template <typename T>
+__global__ void moe_combine_scalar_kernel(T* __restrict__ out, const T* __restrict__ y,
+                                          const float* __restrict__ weights, const int* __restrict__ inv_pos,
+                                          const T* __restrict__ shared, int topk, int hidden) {
   const size_t t = blockIdx.x;
   for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
-    float acc = shared ? shared[t * hidden + i] : 0.f;
+    float acc = shared ? to_f(shared[t * hidden + i]) : 0.f;
     for (int k = 0; k < topk; ++k) {
       const int pos = inv_pos[t * topk + k];
-      if (pos >= 0) acc = fmaf(weights[t * topk + k], y[(size_t)pos * hidden + i], acc);
+      if (pos >= 0) acc = fmaf(weights[t * topk + k], to_f(y[(size_t)pos * hidden + i]), acc);
     }
-    out[t * hidden + i] = acc;
+    out[t * hidden + i] = from_f<T>(acc);
   }
 }
 
@@ -392,8 +394,11 @@ void moe_align(int* sorted_ids, int* block_expert, int* total_padded, int* inv_p
 void moe_gather(void* out, const void* x, const int* sorted_ids, const int* total_padded, int max_padded, int numel,
                 int topk, int hidden, int dtype, cudaStream_t stream) {
   if (max_padded <= 0) return;
-  if (dtype == 2) {
-    moe_gather_f32_kernel<<<max_padded, 128, 0, stream>>>((float*)out, (const float*)x, sorted_ids, total_padded, numel, topk, hidden);
+  if (dtype == 2 || hidden % 8 != 0) {
+    DISPATCH_16(dtype,
+                (moe_gather_scalar_kernel<<<max_padded, 128, 0, stream>>>((__nv_bfloat16*)out, (const __nv_bfloat16*)x, sorted_ids, total_padded, numel, topk, hidden)),
+                (moe_gather_scalar_kernel<<<max_padded, 128, 0, stream>>>((__half*)out, (const __half*)x, sorted_ids, total_padded, numel, topk, hidden)),
+                (moe_gather_scalar_kernel<<<max_padded, 128, 0, stream>>>((float*)out, (const float*)x, sorted_ids, total_padded, numel, topk, hidden)))
     return;
   }
   const int th = hidden / 8 < 256 ? (hidden / 8 < 32 ? 32 : hidden / 8) : 256;
@@ -406,8 +411,11 @@ void moe_gather(void* out, const void* x, const int* sorted_ids, const int* tota
 void moe_combine(void* out, const void* y, const float* weights, const int* inv_pos, const void* shared, int tokens,
                  int topk, int hidden, int dtype, cudaStream_t stream) {
   if (tokens <= 0) return;
-  if (dtype == 2) {
-    moe_combine_f32_kernel<<<tokens, 128, 0, stream>>>((float*)out, (const float*)y, weights, inv_pos, (const float*)shared, topk, hidden);
+  if (dtype == 2 || hidden % 8 != 0) {
+    DISPATCH_16(dtype,
+                (moe_combine_scalar_kernel<<<tokens, 128, 0, stream>>>((__nv_bfloat16*)out, (const __nv_bfloat16*)y, weights, inv_pos, (const __nv_bfloat16*)shared, topk, hidden)),
+                (moe_combine_scalar_kernel<<<tokens, 128, 0, stream>>>((__half*)out, (const __half*)y, weights, inv_pos, (const __half*)shared, topk, hidden)),
+                (moe_combine_scalar_kernel<<<tokens, 128, 0, stream>>>((float*)out, (const float*)y, weights, inv_pos, (const float*)shared, topk, hidden)))
     return;
   }
   const int th = hidden / 8 < 256 ? (hidden / 8 < 32 ? 32 : hidden / 8) : 256;

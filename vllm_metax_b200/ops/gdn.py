@@ -174,7 +174,7 @@ def causal_conv1d_ref(x, w, bias=None, state=None, query_start_loc=None, state_i
         if bias is not None:
             y = y + bias.float()
         out[s:e] = torch.nn.functional.silu(y) if silu else y
-        if slot >= 0 and state is not None:
+        if slot >= 0 and state is not None and K > 1:
             state[slot] = ext[-(K - 1):].to(state.dtype)
     return out.to(x.dtype)
 
