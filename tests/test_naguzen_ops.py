@@ -110,14 +110,17 @@ def test_short_convolution_over_portions(device, dt, taps):
 # ------------------------------------------------------------------ recurrences
 @pytest.mark.parametrize("device", DEVICES)
 @pytest.mark.parametrize("dt", DTYPES)
-@pytest.mark.parametrize("H,D,V,tau", [(3, 20, 12, 9.0), (2, 64, 48, 16.0), (1, 33, 7, 1.0), (2, 96, 136, 4.0),
-                                       (1, 130, 40, 16.0), (1, 250, 260, 2.0)])
-def test_gated_linear_attention_over_portions(device, dt, H, D, V, tau):
+@pytest.mark.parametrize("H,D,V,tau,long", [(3, 20, 12, 9.0, 0), (2, 64, 48, 16.0, 0), (1, 33, 7, 1.0, 0), (2, 96, 136, 4.0, 0),
+                                            (1, 130, 40, 16.0, 0), (1, 250, 260, 2.0, 0), (2, 40, 24, 16.0, 1),
+                                            (1, 33, 150, 200.0, 1), (1, 170, 30, 50.0, 1)])
+def test_gated_linear_attention_over_portions(device, dt, H, D, V, tau, long):
+    """``long``: portions of several segments beside short ones (edges at 256 tokens), slow decays."""
     eps = 1e-5
+    lens, cuts = ([300, 1, 800, 257], [1, 2, 258, 262, 775]) if long else (LENS, CUTS)
     widths = [H * D, H * D, H * V, H * V]
     off = [8, 8 + widths[0], 8 + 2 * widths[0], 8 + 2 * widths[0] + widths[2]]
-    rows = [rnd(n, off[3] + widths[3] + 5, dt=dt, seed=n) for n in LENS]
-    zs = [rnd(n, H * D, seed=50 + n) * 2 for n in LENS]
+    rows = [rnd(n, off[3] + widths[3] + 5, dt=dt, seed=n) for n in lens]
+    zs = [rnd(n, H * D, seed=50 + n) * 2 for n in lens]
     zb, nw = rnd(H * D, dt=dt) + 3, rnd(V, dt=dt) + 1
     want = []
     for r, z in zip(rows, zs):
@@ -128,7 +131,7 @@ def test_gated_linear_attention_over_portions(device, dt, H, D, V, tau):
         g = p[:, off[3]: off[3] + widths[3]]
         want.append((O.unit_rms(o, eps) * nw.double()).reshape(n, H * V) * g * O.sigmoid(g))
     state = rnd(6, H, D, V).to(device)
-    for step in split_steps(LENS, CUTS):
+    for step in split_steps(lens, cuts):
         qsl, idx, init = step_args(step, SLOTS, device)
         x = torch.cat([rows[s][lo:hi] for s, lo, hi in step]).to(device)
         z = torch.cat([zs[s][lo:hi] for s, lo, hi in step]).to(device)

@@ -462,9 +462,9 @@ void residual_conv(Tensor& x_out, Tensor& h, const Tensor& y, const optional<Ten
   p.w = w.data_ptr(); p.carry = K > 1 ? ptr<float>(carry) : nullptr;
   p.qsl = s.qsl; p.state_idx = s.idx; p.has_init = s.init;
   p.batch = s.batch; p.tokens = T; p.D = D; p.K = K; p.eps = (float)eps;
-  p.vec = D % (D > 4096 ? 16 : D > 2048 ? 8 : 4) == 0;
+  p.vec = D % 8 == 0;
   const c10::cuda::CUDAGuard guard(y.device());
-  TORCH_CHECK(b200::residual_conv(p, dtype_code(y), cur_stream()) == 0, "residual_conv: width up to 8192, 1 to 8 taps");
+  TORCH_CHECK(b200::residual_conv(p, dtype_code(y), cur_stream()) == 0, "residual_conv: 1 to 8 taps");
 }
 
 void residual_norm(Tensor& out, const Tensor& y, const optional<Tensor>& x, const optional<Tensor>& gain,
@@ -480,7 +480,7 @@ void residual_norm(Tensor& out, const Tensor& y, const optional<Tensor>& x, cons
   const c10::cuda::CUDAGuard guard(y.device());
   const int rc = b200::residual_norm(out.data_ptr(), ptr<float>(x), y.data_ptr(), ptr(gain), gain2.data_ptr(),
                                      gain.has_value() ? gain->numel() : 1, gain2.numel(), (float)eps, T, D,
-                                     D % (D > 4096 ? 16 : D > 2048 ? 8 : 4) == 0, dtype_code(y), cur_stream());
+                                     D % (D <= 2048 ? 8 : 16) == 0, dtype_code(y), cur_stream());
   TORCH_CHECK(rc == 0, "residual_norm: width up to 8192");
 }
 
@@ -492,8 +492,10 @@ int device_sms(const Tensor& t) {
   return sms[d];
 }
 
-bool gla_needs_scratch(const Tensor& like, int64_t batch, int64_t heads, int64_t dim, int64_t vdim, int64_t max_query_len) {
-  return b200::gla_needs_scratch((int)batch, (int)heads, (int)dim, (int)vdim, (int)max_query_len, device_sms(like));
+int64_t gla_scratch_floats(const Tensor& like, int64_t batch, int64_t heads, int64_t dim, int64_t vdim, int64_t max_query_len) {
+  const b200::GlaScratch g = b200::gla_scratch((int)batch, (int)like.size(0), (int)heads, (int)dim, (int)vdim,
+                                               (int)max_query_len, device_sms(like));
+  return g.raw + g.segments + 4 * ((g.raw + g.segments) > 0);
 }
 
 // qkvg [T, >= ...]: q, k at [q_off, k_off], v at v_off, gate at g_off (each heads * size wide)
@@ -513,18 +515,20 @@ void gla_recurrent(Tensor& out, Tensor& state, const Tensor& qkvg, int64_t q_off
   if (z_bias.has_value()) TORCH_CHECK(z_bias->numel() == H * D && z_bias->scalar_type() == qkvg.scalar_type());
   const StepRefs s = step_refs(qsl, state_idx, has_init);
   const int sms = device_sms(qkvg);
-  if (b200::gla_needs_scratch(s.batch, H, D, V, (int)max_query_len, sms))
-    TORCH_CHECK(scratch.has_value() && scratch->scalar_type() == at::kFloat && scratch->numel() >= T * H * V, "gla scratch");
+  const int64_t need = gla_scratch_floats(qkvg, s.batch, H, D, V, max_query_len);
+  if (need > 0)
+    TORCH_CHECK(scratch.has_value() && scratch->scalar_type() == at::kFloat && scratch->numel() >= need &&
+                reinterpret_cast<uintptr_t>(scratch->data_ptr()) % 16 == 0, "gla scratch");
   b200::GlaParams p{};
   p.qkvg = qkvg.data_ptr(); p.row_stride = qkvg.stride(0);
   p.q_off = q_off; p.k_off = k_off; p.v_off = v_off; p.g_off = g_off;
   p.z = z.data_ptr<float>(); p.z_bias = ptr(z_bias); p.norm_w = norm_w.data_ptr(); p.state = state.data_ptr<float>();
-  p.o_raw = ptr<float>(scratch); p.out = out.data_ptr();
+  p.out = out.data_ptr();
   p.qsl = s.qsl; p.state_idx = s.idx; p.has_init = s.init; p.batch = s.batch; p.tokens = T;
   p.heads = H; p.dim = D; p.vdim = V;
   p.scale = (float)scale; p.inv_tau = (float)inv_tau; p.eps = (float)eps;
   const c10::cuda::CUDAGuard guard(qkvg.device());
-  TORCH_CHECK(b200::gla_recurrent(p, (int)max_query_len, sms, dtype_code(qkvg), cur_stream()) == 0,
+  TORCH_CHECK(b200::gla_recurrent(p, ptr<float>(scratch), (int)max_query_len, sms, dtype_code(qkvg), cur_stream()) == 0,
               "gla_recurrent: key dimension up to 256");
 }
 
@@ -602,7 +606,7 @@ TORCH_LIBRARY(b200, m) {
   m.def("gemm_simt(Tensor(a!) out, Tensor a, Tensor w, Tensor? bias, int act, Tensor? act_params, Tensor? block_expert, Tensor? total_padded) -> ()", &gemm_simt);
   m.def("residual_conv(Tensor(a!) x_out, Tensor(b!) h, Tensor y, Tensor? x, Tensor? gain, Tensor w, Tensor(c!)? carry, Tensor query_start_loc, Tensor? state_idx, Tensor? has_initial, float eps) -> ()", &residual_conv);
   m.def("residual_norm(Tensor(a!) out, Tensor y, Tensor? x, Tensor? gain, Tensor gain2, float eps) -> ()", &residual_norm);
-  m.def("gla_needs_scratch(Tensor like, int batch, int heads, int dim, int vdim, int max_query_len) -> bool", &gla_needs_scratch);
+  m.def("gla_scratch_floats(Tensor like, int batch, int heads, int dim, int vdim, int max_query_len) -> int", &gla_scratch_floats);
   m.def("gla_recurrent(Tensor(a!) out, Tensor(b!) state, Tensor qkvg, int q_off, int k_off, int v_off, int g_off, Tensor z, Tensor? z_bias, Tensor norm_w, Tensor(c!)? scratch, Tensor query_start_loc, Tensor? state_idx, Tensor? has_initial, float scale, float inv_tau, float eps, int max_query_len) -> ()", &gla_recurrent);
   m.def("rglru_chunk() -> int", &rglru_chunk);
   m.def("rglru_scan(Tensor(a!) out, Tensor(b!) state, Tensor(c!) gates, Tensor u, Tensor y, Tensor r_bias, Tensor i_bias, Tensor decay, int block_width, Tensor(d!)? summary, Tensor query_start_loc, Tensor? state_idx, Tensor? has_initial, int max_query_len) -> ()", &rglru_scan);

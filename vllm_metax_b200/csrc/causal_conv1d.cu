@@ -23,14 +23,14 @@ namespace b200 {
 namespace {
 
 constexpr int kMaxK = 8;
-constexpr int kTokPerCta = 32;
 
 template <typename T>
 __device__ __forceinline__ float ld(const T* p) { return (float)*p; }
 template <typename T>
 __device__ __forceinline__ void st(T* p, float v) { *p = (T)v; }
 
-template <typename T>
+// kTokPerCta: 32 for prompts; a handful for decode steps, whose few tokens must still fill the GPU.
+template <typename T, int kTokPerCta>
 __global__ void conv1d_fwd_kernel(T* __restrict__ out, const T* __restrict__ x, int64_t x_stride,
                                   const T* __restrict__ w, const T* __restrict__ bias, const T* __restrict__ state,
                                   const int* __restrict__ qsl, const int* __restrict__ state_idx,
@@ -123,10 +123,14 @@ void launch(void* out, const void* x, int64_t x_stride, const void* w, const voi
             const int* state_idx, const int* has_init, int batch, int tokens, int channels, int K, int silu,
             cudaStream_t stream) {
   const int threads = 128;
-  dim3 grid((channels + threads - 1) / threads, (tokens + kTokPerCta - 1) / kTokPerCta);
-  conv1d_fwd_kernel<T><<<grid, threads, 0, stream>>>((T*)out, (const T*)x, x_stride, (const T*)w, (const T*)bias,
-                                                     (const T*)state, qsl, state_idx, has_init, batch, tokens, channels,
-                                                     K, silu);
+#define CONV_FWD(TOK)                                                                                              \
+  conv1d_fwd_kernel<T, TOK><<<dim3((channels + threads - 1) / threads, (tokens + TOK - 1) / TOK), threads, 0, stream>>>( \
+      (T*)out, (const T*)x, x_stride, (const T*)w, (const T*)bias, (const T*)state, qsl, state_idx, has_init, batch, tokens, \
+      channels, K, silu)
+  if (tokens <= 64) CONV_FWD(1);
+  else if (tokens <= 1024) CONV_FWD(4);
+  else CONV_FWD(32);
+#undef CONV_FWD
   if (state != nullptr && state_idx != nullptr && K > 1) {
     dim3 g2((channels + threads - 1) / threads, batch);
     conv1d_state_kernel<T><<<g2, threads, 0, stream>>>((T*)state, (const T*)x, x_stride, qsl, state_idx, has_init,

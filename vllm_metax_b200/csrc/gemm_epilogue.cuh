@@ -11,6 +11,52 @@
 
 namespace b200 {
 
+// erf to 1.5e-7 (absolute): formula 7.1.26 of Abramowitz and Stegun, Handbook of Mathematical Functions.  A dozen
+// branch-free instructions, so that the epilogue warps keep up with the tensor core.
+__device__ __forceinline__ float erf_as(float x) {
+  const float ax = fabsf(x);
+  const float t = __fdividef(1.f, fmaf(0.3275911f, ax, 1.f));
+  float p = fmaf(1.061405429f, t, -1.453152027f);
+  p = fmaf(p, t, 1.421413741f);
+  p = fmaf(p, t, -0.284496736f);
+  p = fmaf(p, t, 0.254829592f);
+  return copysignf(fmaf(-p * t, __expf(-ax * ax), 1.f), x);
+}
+
+// What a 16-bit result needs: the same functions with absolute errors of some 1e-7.
+__device__ __forceinline__ float epi_activate16(float f, int act, const float* __restrict__ prm) {
+  if (act == kEpiGelu) return 0.5f * f * (1.f + erf_as(f * 0.70710678118654752f));
+  if (act == kEpiGeluTanh) {                     // (1 + tanh(u)) / 2 = 1 / (1 + exp(-2 u))
+    const float u = 1.5957691216057308f * (f + 0.044715f * f * f * f);
+    return __fdividef(f, 1.f + __expf(-u));
+  }
+  if (act == kEpiXielu) {
+    const float neg = __ldg(prm + 1) * (__expf(fminf(f, 0.f)) - 1.f - f), pos = __ldg(prm) * f * f;
+    return fmaf(0.5f, f, f > 0.f ? pos : neg);
+  }
+  return f;
+}
+
+// N elements at once: one branch on the activation outside the element loop (a branch per element multiplies the code of
+// the unrolled epilogue until it no longer fits the instruction cache).
+template <int N>
+__device__ __forceinline__ void epi_activate16_n(float (&f)[N], int act, const float* __restrict__ prm) {
+  if (act == kEpiXielu) {
+    const float cp = __ldg(prm), cn = __ldg(prm + 1);
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      const float neg = cn * (__expf(fminf(f[i], 0.f)) - 1.f - f[i]), pos = cp * f[i] * f[i];
+      f[i] = fmaf(0.5f, f[i], f[i] > 0.f ? pos : neg);
+    }
+  } else if (act == kEpiGelu) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) f[i] = 0.5f * f[i] * (1.f + erf_as(f[i] * 0.70710678118654752f));
+  } else if (act == kEpiGeluTanh) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) f[i] = epi_activate16(f[i], kEpiGeluTanh, prm);
+  }
+}
+
 __device__ __forceinline__ float epi_activate(float f, int act, const float* __restrict__ prm) {
   if (act == kEpiGelu) return 0.5f * f * (1.f + erff(f * 0.70710678118654752f));
   if (act == kEpiGeluTanh) return 0.5f * f * (1.f + tanhf(0.79788456080286536f * (f + 0.044715f * f * f * f)));
@@ -29,48 +75,100 @@ __device__ __forceinline__ void epi_store1(T* __restrict__ C, size_t idx, float 
   else C[idx] = from_f<T>(f);
 }
 
-// CH consecutive elements of a row (columns cb0 ..), the vector form of epi_store1.
+// N tokens of one output feature (transposed tiles: lane = feature): element k goes to C[(tok0 + k) * ldc + feature].
+template <typename T, int N>
+__device__ __forceinline__ void epi_store_tokens(float (&f)[N], T* __restrict__ C, int feature, int tok0, int tokens, int ldc,
+                                                 const Epi& epi) {
+  epi_activate16_n<N>(f, epi.code & kEpiActMask, epi.act);
+  const size_t at = (size_t)tok0 * ldc + feature;
+  if (epi.code & kEpiF32) {
+#pragma unroll
+    for (int k = 0; k < N; ++k)
+      if (tok0 + k < tokens) reinterpret_cast<float*>(C)[at + (size_t)k * ldc] = f[k];
+  } else {
+#pragma unroll
+    for (int k = 0; k < N; ++k)
+      if (tok0 + k < tokens) C[at + (size_t)k * ldc] = from_f<T>(f[k]);
+  }
+}
+
+// CH consecutive elements of a row (columns cb0 ..), 16-bit output: the vector form of epi_store1.
 template <typename T, int CH>
 __device__ __forceinline__ void epi_store_row(const uint32_t (&r)[32], int row, int cb0, int n_cols, T* __restrict__ C,
                                               int ldc, const T* __restrict__ bias, const Epi& epi) {
+  float f[CH];
+#pragma unroll
+  for (int i = 0; i < CH; ++i) f[i] = __uint_as_float(r[i]);
+  if (bias) {
+#pragma unroll
+    for (int i = 0; i < CH; ++i) f[i] += cb0 + i < n_cols ? to_f(bias[cb0 + i]) : 0.f;
+  }
+  epi_activate16_n<CH>(f, epi.code & kEpiActMask, epi.act);
+  T* dst = C + (size_t)row * ldc + cb0;
 #pragma unroll
   for (int v = 0; v < CH / 8; ++v) {
-    const int col = cb0 + v * 8;
-    const size_t at = (size_t)row * ldc + col;
-    if (col + 8 <= n_cols) {
-      float f[8];
+    if (cb0 + v * 8 + 8 <= n_cols) {
+      float g[8];
 #pragma unroll
-      for (int i = 0; i < 8; ++i) f[i] = __uint_as_float(r[v * 8 + i]);
-      if (bias) {
-        float b[8];
-        unpack8<T>(*reinterpret_cast<const uint4*>(bias + col), b);
-#pragma unroll
-        for (int i = 0; i < 8; ++i) f[i] += b[i];
-      }
-#pragma unroll
-      for (int i = 0; i < 8; ++i) f[i] = epi_activate(f[i], epi.code & kEpiActMask, epi.act);
-      if (epi.code & kEpiF32) {
-        float4* d = reinterpret_cast<float4*>(reinterpret_cast<float*>(C) + at);
-        d[0] = make_float4(f[0], f[1], f[2], f[3]);
-        d[1] = make_float4(f[4], f[5], f[6], f[7]);
-      } else {
-        *reinterpret_cast<uint4*>(C + at) = pack8<T>(f);
-      }
+      for (int i = 0; i < 8; ++i) g[i] = f[v * 8 + i];
+      *reinterpret_cast<uint4*>(dst + v * 8) = pack8<T>(g);
     } else {
+#pragma unroll
       for (int i = 0; i < 8; ++i)
-        if (col + i < n_cols)
-          epi_store1<T>(C, at + i, __uint_as_float(r[v * 8 + i]) + (bias ? to_f(bias[col + i]) : 0.f), epi);
+        if (cb0 + v * 8 + i < n_cols) dst[v * 8 + i] = from_f<T>(f[v * 8 + i]);
     }
   }
 }
 
+// fp32 output, 32 rows x 32 columns of a warp (lane = row, register = column), through a padded shared-memory square so
+// that every store is one row of 128 bytes.  The whole warp calls this; `stage` is the warp's own.
+template <typename T>
+__device__ __forceinline__ void epi_store_block_f32(const uint32_t (&r)[32], float (&stage)[32][33], int row0, int rows,
+                                                    int cb0, int n_cols, T* __restrict__ C, int ldc,
+                                                    const T* __restrict__ bias, const Epi& epi) {
+  const int lane = threadIdx.x & 31;
+#pragma unroll
+  for (int i = 0; i < 32; ++i) stage[lane][i] = __uint_as_float(r[i]);
+  __syncwarp();
+  const int col = cb0 + lane;
+  if (col < n_cols) {
+    const float b = bias ? to_f(bias[col]) : 0.f;
+    float* dst = reinterpret_cast<float*>(C) + (size_t)row0 * ldc + col;
+    const int n = min(32, rows - row0);
+    if ((epi.code & kEpiActMask) == 0) {
+#pragma unroll 8
+      for (int i = 0; i < n; ++i) dst[(size_t)i * ldc] = stage[i][lane] + b;
+    } else {
+#pragma unroll 1
+      for (int i = 0; i < n; ++i)
+        dst[(size_t)i * ldc] = epi_activate(stage[i][lane] + b, epi.code & kEpiActMask, epi.act);
+    }
+  }
+  __syncwarp();
+}
+
 // r[0..CH): accumulators of columns cb0..cb0+CH of row `row`; n_cols = number of valid columns.
+template <typename T, int CH>
+__device__ __forceinline__ void store_row_segment_f32(const uint32_t (&r)[32], int row, int cb0, int n_cols,
+                                                      T* __restrict__ C, int ldc, const T* __restrict__ bias, const Epi& epi) {
+  float f[CH];
+#pragma unroll
+  for (int i = 0; i < CH; ++i)
+    f[i] = __uint_as_float(r[i]) + ((bias && cb0 + i < n_cols) ? to_f(bias[cb0 + i]) : 0.f);
+  epi_activate16_n<CH>(f, epi.code & kEpiActMask, epi.act);
+  float* dst = reinterpret_cast<float*>(C) + (size_t)row * ldc + cb0;
+#pragma unroll
+  for (int i = 0; i < CH; ++i)
+    if (cb0 + i < n_cols) dst[i] = f[i];
+}
+
 template <typename T, int CH>
 __device__ __forceinline__ void store_row_segment(const uint32_t (&r)[32], int row, int cb0, int n_cols,
                                                   T* __restrict__ C, int ldc, const T* __restrict__ bias,
                                                   const T* __restrict__ residual, int ldr, const Epi& epi) {
   if (epi.code > 1) {
-    epi_store_row<T, CH>(r, row, cb0, n_cols, C, ldc, bias, epi);
+    if (epi.code & kEpiF32) store_row_segment_f32<T, CH>(r, row, cb0, n_cols, C, ldc, bias, epi);
+    else epi_store_row<T, CH>(r, row, cb0, n_cols, C, ldc, bias, epi);
     return;
   }
   if (epi.code == 1) {

@@ -199,7 +199,7 @@ void gemm_grouped(const void* A, int max_rows, int lda, const void* W, int E, in
                   void* status) {
   if (max_rows <= 0 || N <= 0) return;
   StatusWord* st = reinterpret_cast<StatusWord*>(status);
-  const bool wide = N >= 1024;
+  const bool wide = N >= 1024 || (N >= 512 && N % 256 == 0);
   if (dtype == 0) {
     if (wide) launch_grouped<__nv_bfloat16, 256, 4>(A, max_rows, lda, W, E, N, K, C, ldc, block_expert, total_padded, epi, stream, st);
     else launch_grouped<__nv_bfloat16, 128, 6>(A, max_rows, lda, W, E, N, K, C, ldc, block_expert, total_padded, epi, stream, st);

@@ -69,6 +69,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
   uint64_t* tmem_empty = tmem_full + 2;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(tmem_empty + 2);
 
+  __shared__ float f32_stage[BULK ? 1 : 4][32][33];   // fp32 outputs: one square per epilogue warp
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const uint32_t rank = cluster_ctarank();       // 0 = leader
   const int cluster_id = blockIdx.x >> 1;
@@ -226,6 +227,12 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
         uint32_t r[32];
         tmem_ld_32x32b_x32(taddr + c, r);
         tmem_ld_wait();
+        if constexpr (!BULK) {
+          if (epi.code & kEpiF32) {
+            epi_store_block_f32<T>(r, f32_stage[warp & 3], row - lane, M, tn * kPairBN + c, N, C, ldc, bias, epi);
+            continue;
+          }
+        }
         if (row < M) {
           if (sc.tp > 0) {
             // the row goes to the receive slot of the rank that owns it (a peer store over NVLink for d != me)
@@ -278,7 +285,7 @@ static void launch_pair(const void* A, const void* W, void* C, const void* bias,
   CUtensorMap tmA = make_tmap_2d(A, dt, 2, M, K, lda, 128, kPairBK);
   CUtensorMap tmB = make_tmap_2d(W, dt, 2, N, K, ldw, 128, kPairBK);
   using L = PairSmem<STAGES, BULK>;
-  static_assert(L::kDyn <= 232448, "shared memory budget exceeded");
+  static_assert(L::kDyn + (BULK ? 1 : 4) * 32 * 33 * 4 <= 232448, "shared memory budget exceeded");
   auto kern = gemm_pair_kernel<T, STAGES, BULK>;
   // kernel attributes and SM counts are per device
   static bool set[64] = {};

@@ -292,9 +292,13 @@ gemm_streamk_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_consta
               if (ra + 3 < sh.N) *reinterpret_cast<uint32_t*>(crow + (ra >> 1)) = *reinterpret_cast<const uint32_t*>(o2);
               else if (ra + 1 < sh.N) crow[ra >> 1] = o2[0];
             } else if (epi.code > 1) {
+              epi_activate16_n<4>(f, epi.code & kEpiActMask, epi.act);
 #pragma unroll
-              for (int e = 0; e < 4; ++e)
-                if (ra + e < sh.N) epi_store1<T>(C, (size_t)tok * ldc + ra + e, f[e], epi);
+              for (int e = 0; e < 4; ++e) {
+                if (ra + e >= sh.N) break;
+                if (epi.code & kEpiF32) reinterpret_cast<float*>(C)[(size_t)tok * ldc + ra + e] = f[e];
+                else C[(size_t)tok * ldc + ra + e] = from_f<T>(f[e]);
+              }
             } else {
               if (residual && sc.tp == 0) {
 #pragma unroll
@@ -336,8 +340,8 @@ gemm_streamk_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_consta
           } else if (epi.code > 1) {
             if (ra_ok) {
 #pragma unroll
-              for (int i = 0; i < 16; ++i)
-                if (tok0 + i < sh.M) epi_store1<T>(C, (size_t)(tok0 + i) * ldc + ra, a[i] + bv, epi);
+              for (int i = 0; i < 16; ++i) a[i] += bv;
+              epi_store_tokens<T, 16>(a, C, ra, tok0, sh.M, ldc, epi);
             }
           } else if (ra_ok) {
 #pragma unroll

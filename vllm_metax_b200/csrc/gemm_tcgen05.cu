@@ -63,6 +63,7 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmA,   // 128-row operand
   uint64_t* tmem_empty = tmem_full + 2;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(tmem_empty + 2);
 
+  __shared__ float f32_stage[SWAP ? 1 : 4][32][33];        // fp32 outputs: one square per epilogue warp
   const int warp = threadIdx.x >> 5;
   const int lane = threadIdx.x & 31;
   const int num_a = ceil_div(rows_a, kBM);
@@ -198,7 +199,10 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmA,   // 128-row operand
         const int cb0 = tb * BN + c;  // first index in the BN-row operand
         if constexpr (!SWAP) {
           // row = token (ra), columns = output features cb0..cb0+CH
-          if (epi.code > 1) {
+          if (epi.code & kEpiF32) {
+            if constexpr (CH == 32)
+              epi_store_block_f32<T>(r, f32_stage[quarter], ra - lane, rows_a, cb0, rows_b, C, ldc, bias, epi);
+          } else if (epi.code > 1) {
             if (ra < rows_a) epi_store_row<T, CH>(r, ra, cb0, rows_b, C, ldc, bias, epi);
           } else if (ra < rows_a && epi.code == 1) {
             // columns hold interleaved (gate, up) pairs: out[:, j] = silu(gate_j) * up_j
@@ -275,9 +279,10 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmA,   // 128-row operand
             }
           } else if (epi.code > 1) {
             if (ra < rows_a) {
+              float f[CH];
 #pragma unroll
-              for (int i = 0; i < CH; ++i)
-                if (cb0 + i < rows_b) epi_store1<T>(C, (size_t)(cb0 + i) * ldc + ra, __uint_as_float(r[i]) + bv, epi);
+              for (int i = 0; i < CH; ++i) f[i] = __uint_as_float(r[i]) + bv;
+              epi_store_tokens<T, CH>(f, C, ra, cb0, rows_b, ldc, epi);
             }
           } else if (ra < rows_a) {
 #pragma unroll
@@ -321,7 +326,7 @@ static void launch_cfg(const void* a_op, int rows_a, int lda, const void* b_op, 
                        const void* bias, const void* residual, int K, int ldc, int ldr, Epi epi, cudaStream_t stream,
                        StatusWord* status) {
   using L = GemmSmemLayout<BN, STAGES>;
-  static_assert(L::kDynSmem <= 232448, "shared memory budget exceeded");
+  static_assert(L::kDynSmem + (SWAP ? 1 : 4) * 32 * 33 * 4 <= 232448, "shared memory budget exceeded");
   const CUtensorMapDataType dt =
       std::is_same<T, __half>::value ? CU_TENSOR_MAP_DATA_TYPE_FLOAT16 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
   CUtensorMap tmA = make_tmap_2d(a_op, dt, 2, rows_a, K, lda, kBM, kBK);

@@ -21,43 +21,90 @@ __device__ __forceinline__ void rotate_pair(float& u, float& v, float pos, float
   v = b;
 }
 
-template <typename T>
+// V consecutive elements (V = 1, or 16 bytes of them)
+template <typename T, int V>
+__device__ __forceinline__ void ld_v(const T* p, float (&f)[V]) {
+  if constexpr (V == 1) {
+    f[0] = to_f(*p);
+  } else {
+    const uint4 r = *reinterpret_cast<const uint4*>(p);
+    const T* e = reinterpret_cast<const T*>(&r);
+#pragma unroll
+    for (int k = 0; k < V; ++k) f[k] = to_f(e[k]);
+  }
+}
+template <typename T, int V>
+__device__ __forceinline__ void st_v(T* p, const float (&f)[V]) {
+  if constexpr (V == 1) {
+    *p = from_f<T>(f[0]);
+  } else {
+    alignas(16) T e[V];
+#pragma unroll
+    for (int k = 0; k < V; ++k) e[k] = from_f<T>(f[k]);
+    *reinterpret_cast<uint4*>(p) = *reinterpret_cast<const uint4*>(e);
+  }
+}
+
+// V > 1: every size, offset and pitch is a multiple of V.
+template <typename T, int V>
 __global__ void __launch_bounds__(128)
 latent_insert_kernel(const LatentInsertParams p) {
-  __shared__ float red[32];
+  __shared__ float red[2][4];
   const int64_t t = blockIdx.x;
   const T* row = reinterpret_cast<const T*>(p.a) + t * p.a_stride;
   const T* aq = row + p.q_off;
   const T* ak = row + p.kv_off;
+  const int tid = threadIdx.x;
   float sq = 0.f, sk = 0.f;
-  for (int i = threadIdx.x; i < p.q_rank; i += blockDim.x) { const float v = to_f(aq[i]); sq = fmaf(v, v, sq); }
-  for (int i = threadIdx.x; i < p.kv_rank; i += blockDim.x) { const float v = to_f(ak[i]); sk = fmaf(v, v, sk); }
-  sq = block_sum(sq, red);
-  sk = block_sum(sk, red);
-  const float iq = 1.f / sqrtf(sq / (float)p.q_rank + p.eps), ik = 1.f / sqrtf(sk / (float)p.kv_rank + p.eps);
-  T* cq = reinterpret_cast<T*>(p.cq) + t * p.q_rank;
-  const T* wq = reinterpret_cast<const T*>(p.q_w);
-  for (int i = threadIdx.x; i < p.q_rank; i += blockDim.x) cq[i] = from_f<T>(to_f(aq[i]) * iq * to_f(wq[i]));
+  auto squares = [&](const T* src, int n) {
+    float ss = 0.f;
+#pragma unroll 4
+    for (int i = tid * V; i < n; i += 128 * V) {
+      float v[V];
+      ld_v<T, V>(src + i, v);
+#pragma unroll
+      for (int k = 0; k < V; ++k) ss = fmaf(v[k], v[k], ss);
+    }
+    return ss;
+  };
+  sq = warp_sum(squares(aq, p.q_rank));
+  sk = warp_sum(squares(ak, p.kv_rank));
+  if ((tid & 31) == 0) { red[0][tid >> 5] = sq; red[1][tid >> 5] = sk; }
+  __syncthreads();
+  sq = red[0][0] + red[0][1] + red[0][2] + red[0][3];
+  sk = red[1][0] + red[1][1] + red[1][2] + red[1][3];
+  auto scaled = [&](T* dst, const T* src, const T* w, int n, float inv) {
+#pragma unroll 4
+    for (int i = tid * V; i < n; i += 128 * V) {
+      float v[V], g[V];
+      ld_v<T, V>(src + i, v);
+      ld_v<T, V>(w + i, g);
+#pragma unroll
+      for (int k = 0; k < V; ++k) v[k] = v[k] * inv * g[k];
+      st_v<T, V>(dst + i, v);
+    }
+  };
+  scaled(reinterpret_cast<T*>(p.cq) + t * p.q_rank, aq, reinterpret_cast<const T*>(p.q_w), p.q_rank,
+         1.f / sqrtf(sq / (float)p.q_rank + p.eps));
   const int64_t slot = p.slots[t];
   if (slot < 0) return;
   if (slot >= p.num_slots) {
-    if (threadIdx.x == 0) report_status(p.status, kBadIndex, 120, (int)p.num_slots, (int)slot);
+    if (tid == 0) report_status(p.status, kBadIndex, 120, (int)p.num_slots, (int)slot);
     return;
   }
   T* dst = reinterpret_cast<T*>(p.cache) + slot * p.row_elems;
-  const T* wk = reinterpret_cast<const T*>(p.kv_w);
-  for (int i = threadIdx.x; i < p.kv_rank; i += blockDim.x) dst[i] = from_f<T>(to_f(ak[i]) * ik * to_f(wk[i]));
+  scaled(dst, ak, reinterpret_cast<const T*>(p.kv_w), p.kv_rank, 1.f / sqrtf(sk / (float)p.kv_rank + p.eps));
   const T* kr = ak + p.kv_rank;
   const int half = p.rot_dims / 2;
   const float pos = (float)p.positions[t];
-  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+  for (int i = tid; i < half; i += 128) {
     float u = to_f(kr[i]), v = to_f(kr[i + half]);
     rotate_pair(u, v, pos, p.inv_freq[i]);
     dst[p.kv_rank + i] = from_f<T>(u);
     dst[p.kv_rank + half + i] = from_f<T>(v);
   }
-  for (int i = 2 * half + threadIdx.x; i < p.rot_dim; i += blockDim.x) dst[p.kv_rank + i] = kr[i];
-  for (int i = p.kv_rank + p.rot_dim + threadIdx.x; i < p.row_elems; i += blockDim.x) dst[i] = from_f<T>(0.f);
+  for (int i = 2 * half + tid; i < p.rot_dim; i += 128) dst[p.kv_rank + i] = kr[i];
+  for (int i = p.kv_rank + p.rot_dim + tid; i < p.row_elems; i += 128) dst[i] = from_f<T>(0.f);
 }
 
 template <typename T>
@@ -168,7 +215,16 @@ latent_attn_simt_kernel(const MlaDecodeParams p) {
 
 int latent_insert(const LatentInsertParams& p, int dtype, cudaStream_t stream) {
   if (p.tokens <= 0) return 0;
-  BY_DTYPE((latent_insert_kernel<T><<<p.tokens, 128, 0, stream>>>(p)))
+  const int v = dtype == 2 ? 4 : 8;
+  auto aligned = [](const void* x) { return reinterpret_cast<uintptr_t>(x) % 16 == 0; };
+  const bool vec = p.q_rank % v == 0 && p.kv_rank % v == 0 && p.row_elems % v == 0 && p.a_stride % v == 0 &&
+                   p.q_off % v == 0 && p.kv_off % v == 0 && aligned(p.a) && aligned(p.cq) && aligned(p.cache) &&
+                   aligned(p.q_w) && aligned(p.kv_w);
+  if (vec) {
+    BY_DTYPE((latent_insert_kernel<T, 16 / (int)sizeof(T)><<<p.tokens, 128, 0, stream>>>(p)))
+  } else {
+    BY_DTYPE((latent_insert_kernel<T, 1><<<p.tokens, 128, 0, stream>>>(p)))
+  }
   return 0;
 }
 

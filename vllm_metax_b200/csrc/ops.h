@@ -318,14 +318,17 @@ struct GlaParams {
   const void* z_bias;          // [heads * dim] or null
   const void* norm_w;          // [vdim]
   float* state;                // [slots, heads, dim, vdim]
-  float* o_raw;                // [tokens, heads * vdim] scratch of the split form (columns of a head over several CTAs)
+  float* o_raw;                // set from the scratch: [tokens, heads * vdim] raw outputs of heads split over CTAs
+  float* seg_state;            // set from the scratch: [segments, heads, dim, vdim] ...
+  float* seg_decay;            // ... and [segments, heads, dim], or null
   void* out;                   // [tokens, heads * vdim]
   const int* qsl; const int* state_idx; const int* has_init;
   int batch, tokens, heads, dim, vdim, col_block;
   float scale, inv_tau, eps;
 };
-int gla_recurrent(GlaParams p, int max_query_len, int sms, int dtype, cudaStream_t stream);
-bool gla_needs_scratch(int batch, int heads, int dim, int vdim, int max_query_len, int sms);
+struct GlaScratch { int64_t raw, segments; };
+GlaScratch gla_scratch(int batch, int tokens, int heads, int dim, int vdim, int max_query_len, int sms);
+int gla_recurrent(GlaParams p, float* scratch, int max_query_len, int sms, int dtype, cudaStream_t stream);
 // ---- rglru.cu (real-gated linear recurrent unit)
 struct RgLruParams {
   const void* u; int64_t u_stride;       // [tokens, width] recurrence input

@@ -7,11 +7,14 @@
 // x, x_new and the convolution's carry [slots, K-1, D] (the last K-1 values of x_new, oldest first) are fp32.  The gain is
 // one number or one per channel.  A null x means x_new = y (the embedding in front of the first layer).
 //
-// One CTA = up to kTok consecutive tokens of one sequence, all channels; a thread keeps its C channels' last taps in
-// registers and walks the tokens, one barrier per token (the row's sum of squares).  The taps before the CTA's first token
-// are recomputed from x and y (x is read-only: x_new is another buffer), or come from the carry at the start of a step.
-// Only the CTA of a sequence's first tile reads the carry and the same CTA rewrites it afterwards, so no CTA waits for
-// another.  Tile i of sequence b is CTA floor(qsl[b] / kTok) + b + i: always enough of them, found by bisection.
+// One CTA = up to kTok consecutive tokens of one sequence.  First its warps form the rows' root mean squares (several warps
+// share a row when there are few), then, after the only barrier, every thread walks the tokens of its 4 channels with the
+// last taps in registers; a wide row is several such passes.  The taps before the CTA's first token are recomputed from x
+// and y (x is read-only: x_new is another buffer), or come from the carry at the start of a step.  Only the CTA of a
+// sequence's first tile reads the carry and the same threads rewrite it afterwards, so no CTA waits for another.
+// Tile i of sequence b is CTA floor(qsl[b] / kTok) + b + i: always enough of them, found by bisection.
+#include <type_traits>
+
 #include "common.cuh"
 #include "ops.h"
 
@@ -20,9 +23,9 @@ namespace {
 
 constexpr int kTok = 16;
 
-template <typename T, int C>
-__device__ __forceinline__ void load_row(const T* __restrict__ p, int c0, int D, bool vec, float (&f)[C]) {
-  if (vec && c0 + C <= D) {
+template <typename T, int C, bool VEC>
+__device__ __forceinline__ void load_row(const T* __restrict__ p, int c0, int D, float (&f)[C]) {
+  if constexpr (VEC) {
     constexpr int kBytes = C * (int)sizeof(T);
     if constexpr (kBytes % 16 == 0) {
       uint4 r[kBytes / 16];
@@ -43,9 +46,9 @@ __device__ __forceinline__ void load_row(const T* __restrict__ p, int c0, int D,
   }
 }
 
-template <typename T, int C>
-__device__ __forceinline__ void store_row(T* __restrict__ p, int c0, int D, bool vec, const float (&f)[C]) {
-  if (vec && c0 + C <= D) {
+template <typename T, int C, bool VEC>
+__device__ __forceinline__ void store_row(T* __restrict__ p, int c0, int D, const float (&f)[C]) {
+  if constexpr (VEC) {
     constexpr int kBytes = C * (int)sizeof(T);
     alignas(16) T e[C];
 #pragma unroll
@@ -63,20 +66,15 @@ __device__ __forceinline__ void store_row(T* __restrict__ p, int c0, int D, bool
   }
 }
 
-// Sum over the CTA with one barrier; the caller alternates between two buffers.
-__device__ __forceinline__ float row_sum(float v, float* red) {
-  v = warp_sum(v);
-  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
-  __syncthreads();
-  const int nw = blockDim.x >> 5;
-  const float s = (int)(threadIdx.x & 31) < nw ? red[threadIdx.x & 31] : 0.f;
-  return warp_sum(s);
-}
+constexpr int kThreads = 256, kRows = kTok + 8;
+constexpr int C = 4;                                       // channels of a thread
 
-template <typename T, int C, int KT>
-__global__ void __launch_bounds__(512)
+// VEC: the width is a multiple of 8, every row starts on 16 bytes.
+template <typename T, int KT, bool VEC>
+__global__ void __launch_bounds__(kThreads, KT == 4 && VEC ? 4 : 1)
 residual_conv_kernel(const ResidualConvParams p) {
-  __shared__ float red[2][32];
+  __shared__ float s_part[kRows][kThreads / 32];
+  __shared__ float s_inv[kRows];
   const int D = p.D, K = p.K;
   // the sequence of this CTA: largest b with qsl[b] / kTok + b <= blockIdx.x
   int b = 0;
@@ -89,152 +87,170 @@ residual_conv_kernel(const ResidualConvParams p) {
   const int i0 = tile * kTok;                              // first token of the tile within the step's tokens of b
   if (i0 >= n) return;
   const int i1 = min(n, i0 + kTok);
-  const int c0 = threadIdx.x * C;
-  const bool vec = p.vec != 0;
+  const int first = tile == 0 ? 0 : i0 - (K - 1);          // (kTok >= K - 1: these belong to this step)
+  const int slot = p.state_idx ? p.state_idx[b] : -1;
+  float* carry = (tile == 0 && slot >= 0 && p.carry != nullptr) ? p.carry + (int64_t)slot * (K - 1) * D : nullptr;
+  const bool tail = carry != nullptr && n > kTok;          // the step's last tokens, for the new carry, are in another tile
   const T* y = reinterpret_cast<const T*>(p.y);
+
+  if (p.x != nullptr) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = kThreads / 32;
+    const int n1 = i1 - first, rows = n1 + (tail ? K - 1 : 0);
+    const int parts = max(1, min(nw, nw / rows));          // warps that share a row
+    for (int u = warp; u < rows * parts; u += nw) {
+      const int r = u / parts, part = u % parts;
+      const T* row = y + (int64_t)(s0 + (r < n1 ? first + r : n - (K - 1) + r - n1)) * D;
+      float ss = 0.f;
+#pragma unroll 4
+      for (int c = (part * 32 + lane) * 8; c < D; c += parts * 256) {
+        float v[8];
+        load_row<T, 8, VEC>(row, c, D, v);
+#pragma unroll
+        for (int k = 0; k < 8; ++k) ss = fmaf(v[k], v[k], ss);
+      }
+      ss = warp_sum(ss);
+      if (lane == 0) s_part[r][part] = ss;
+    }
+    __syncthreads();
+    if ((int)threadIdx.x < rows) {
+      float t = 0.f;
+      for (int i = 0; i < parts; ++i) t += s_part[threadIdx.x][i];
+      s_inv[threadIdx.x] = 1.f / sqrtf(t / (float)D + p.eps);
+    }
+    __syncthreads();
+  }
+
   T* h = reinterpret_cast<T*>(p.h);
   const T* w = reinterpret_cast<const T*>(p.w);
-  float wt[C][KT];                                         // taps, aligned to the current token in the last column
+  const T* gp = reinterpret_cast<const T*>(p.gain);
+  for (int c0 = threadIdx.x * C; c0 < D; c0 += kThreads * C) {
+    float wt[C][KT], gain[C], hist[KT][C];                 // taps aligned right; hist[KT-1] = the current token
 #pragma unroll
-  for (int i = 0; i < C; ++i)
+    for (int i = 0; i < C; ++i) {
+      gain[i] = gp == nullptr ? 1.f : p.gain_per_channel ? (c0 + i < D ? to_f(gp[c0 + i]) : 0.f) : to_f(gp[0]);
 #pragma unroll
-    for (int j = 0; j < KT; ++j) {
-      const int jj = j - (KT - K);
-      wt[i][j] = (jj >= 0 && c0 + i < D) ? to_f(w[(int64_t)(c0 + i) * K + jj]) : 0.f;
+      for (int j = 0; j < KT; ++j) {
+        const int jj = j - (KT - K);
+        wt[i][j] = (jj >= 0 && c0 + i < D) ? to_f(w[(int64_t)(c0 + i) * K + jj]) : 0.f;
+        hist[j][i] = 0.f;
+      }
     }
-  float gain[C];
-#pragma unroll
-  for (int i = 0; i < C; ++i) gain[i] = 1.f;
-  if (p.gain != nullptr) {
-    const T* g = reinterpret_cast<const T*>(p.gain);
-#pragma unroll
-    for (int i = 0; i < C; ++i) gain[i] = p.gain_per_channel ? (c0 + i < D ? to_f(g[c0 + i]) : 0.f) : to_f(g[0]);
-  }
-  const float inv_d = 1.f / (float)D;
-  int flip = 0;
-  auto x_new = [&](int i, float (&v)[C]) {                 // every thread of the CTA calls this together
-    const int64_t row = (int64_t)(s0 + i) * D;
-    load_row<T, C>(y + row, c0, D, vec, v);
-    if (p.x == nullptr) return;
-    float xv[C];
-    load_row<float, C>(p.x + row, c0, D, vec, xv);
-    float ss = 0.f;
-#pragma unroll
-    for (int k = 0; k < C; ++k) ss = fmaf(v[k], v[k], ss);
-    ss = row_sum(ss, red[flip]);
-    flip ^= 1;
-    const float inv = 1.f / sqrtf(ss * inv_d + p.eps);
-#pragma unroll
-    for (int k = 0; k < C; ++k) v[k] = fmaf(v[k] * inv, gain[k], xv[k]);
-  };
-  const int slot = p.state_idx ? p.state_idx[b] : -1;
-  float* carry = (slot >= 0 && p.carry != nullptr) ? p.carry + (int64_t)slot * (K - 1) * D : nullptr;
-  float hist[KT][C];                                       // hist[KT-1] = current token
-#pragma unroll
-  for (int j = 0; j < KT; ++j)
-#pragma unroll
-    for (int i = 0; i < C; ++i) hist[j][i] = 0.f;
-  if (tile == 0) {
     if (carry != nullptr && p.has_init != nullptr && p.has_init[b] != 0) {
 #pragma unroll
-      for (int j = 1; j < KT; ++j) {                       // the values K-1 .. 1 tokens before the step's first token
-        const int back = KT - j;
-        if (back <= K - 1) load_row<float, C>(carry + (int64_t)(K - 1 - back) * D, c0, D, vec, hist[j]);
+      for (int j = 1; j < KT; ++j) {                       // the values K-1 .. 1 tokens before the step's first token,
+        const int back = KT - j;                           // one place to the right of where the first push puts them
+        if (back <= K - 1) load_row<float, C, VEC>(carry + (int64_t)(K - 1 - back) * D, c0, D, hist[j]);
       }
     }
-  } else {
+    // G tokens from i on, whose inverse norms start at s_inv[at]: the loads of all of them first
+    auto step = [&](auto width, int i, int at, bool emit) {
+      constexpr int G = decltype(width)::value;
+      float v[G][C], xv[G][C];
 #pragma unroll
-    for (int j = 1; j < KT; ++j) {
-      const int back = KT - j;
-      if (back <= K - 1) x_new(i0 - back, hist[j]);        // kTok >= K - 1: these tokens belong to this step
-    }
-  }
-  for (int i = i0; i < i1; ++i) {
+      for (int g = 0; g < G; ++g) {
+        load_row<T, C, VEC>(y + (int64_t)(s0 + i + g) * D, c0, D, v[g]);
+        if (p.x != nullptr) load_row<float, C, VEC>(p.x + (int64_t)(s0 + i + g) * D, c0, D, xv[g]);
+      }
 #pragma unroll
-    for (int j = 0; j + 1 < KT; ++j)
+      for (int g = 0; g < G; ++g) {
+        if (p.x != nullptr) {
+          const float inv = s_inv[at + g];
 #pragma unroll
-      for (int k = 0; k < C; ++k) hist[j][k] = hist[j + 1][k];
-    x_new(i, hist[KT - 1]);
-    const int64_t row = (int64_t)(s0 + i) * D;
-    store_row<float, C>(p.x_out + row, c0, D, vec, hist[KT - 1]);
-    float o[C];
+          for (int k = 0; k < C; ++k) v[g][k] = fmaf(v[g][k] * inv, gain[k], xv[g][k]);
+        }
 #pragma unroll
-    for (int k = 0; k < C; ++k) {
-      float a = 0.f;
+        for (int j = 0; j + 1 < KT; ++j)
 #pragma unroll
-      for (int j = 0; j < KT; ++j) a = fmaf(wt[k][j], hist[j][k], a);
-      o[k] = hist[KT - 1][k] + a;
-    }
-    store_row<T, C>(h + row, c0, D, vec, o);
-  }
-  if (tile == 0 && carry != nullptr) {
-    if (n > kTok) {                                        // the step's last tokens are in another tile: recompute them
+          for (int k = 0; k < C; ++k) hist[j][k] = hist[j + 1][k];
+#pragma unroll
+        for (int k = 0; k < C; ++k) hist[KT - 1][k] = v[g][k];
+        if (!emit) continue;
+        const int64_t row = (int64_t)(s0 + i + g) * D;
+        store_row<float, C, VEC>(p.x_out + row, c0, D, v[g]);
+        float o[C];
+#pragma unroll
+        for (int k = 0; k < C; ++k) {
+          float a = 0.f;
+#pragma unroll
+          for (int j = 0; j < KT; ++j) a = fmaf(wt[k][j], hist[j][k], a);
+          o[k] = v[g][k] + a;
+        }
+        store_row<T, C, VEC>(h + row, c0, D, o);
+      }
+    };
+    using One = std::integral_constant<int, 1>;
+    using Many = std::integral_constant<int, 2>;
+#pragma unroll 1
+    for (int i = first; i < i0; ++i) step(One{}, i, i - first, false);
+    int i = i0;
+#pragma unroll 1
+    for (; i + 2 <= i1; i += 2) step(Many{}, i, i - first, true);
+#pragma unroll 1
+    for (; i < i1; ++i) step(One{}, i, i - first, true);
+    if (carry != nullptr) {
+      if (tail) {
+#pragma unroll 1
+        for (int t = 0; t < K - 1; ++t) step(One{}, n - (K - 1) + t, i1 - first + t, false);
+      }
 #pragma unroll
       for (int j = 1; j < KT; ++j) {
-        const int back = KT - 1 - j;                       // hist[KT-1] = the last token
-        if (back <= K - 2) x_new(n - 1 - back, hist[j]);
+        const int at = j - (KT - (K - 1));
+        if (at >= 0) store_row<float, C, VEC>(carry + (int64_t)at * D, c0, D, hist[j]);
       }
-    }
-#pragma unroll
-    for (int j = 1; j < KT; ++j) {
-      const int at = j - (KT - (K - 1));
-      if (at >= 0) store_row<float, C>(carry + (int64_t)at * D, c0, D, vec, hist[j]);
     }
   }
 }
 
+// Sum over the CTA with one barrier; the caller alternates between two buffers.
+__device__ __forceinline__ float row_sum(float v, float* red) {
+  v = warp_sum(v);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  const int nw = blockDim.x >> 5;
+  const float s = (int)(threadIdx.x & 31) < nw ? red[threadIdx.x & 31] : 0.f;
+  return warp_sum(s);
+}
+
 // out = norm2(x + norm1(y)): the last boundary, in front of the LM head.  One CTA per token.
-template <typename T, int C>
+template <typename T, int CN, bool VEC>
 __global__ void __launch_bounds__(512)
 residual_norm_kernel(T* __restrict__ out, const float* __restrict__ x, const T* __restrict__ y,
-                     const T* __restrict__ gain, const T* __restrict__ gain2, int gain_n, int gain2_n, float eps, int D,
-                     int vec_i) {
+                     const T* __restrict__ gain, const T* __restrict__ gain2, int gain_n, int gain2_n, float eps, int D) {
   __shared__ float red[2][32];
-  const int c0 = threadIdx.x * C;
-  const bool vec = vec_i != 0;
+  const int c0 = threadIdx.x * CN;
   const int64_t row = (int64_t)blockIdx.x * D;
-  float v[C], xv[C];
-  load_row<T, C>(y + row, c0, D, vec, v);
+  float v[CN] = {}, xv[CN] = {};
+  if (c0 < D) load_row<T, CN, VEC>(y + row, c0, D, v);
   const float inv_d = 1.f / (float)D;
   if (x != nullptr) {
-    load_row<float, C>(x + row, c0, D, vec, xv);
+    if (c0 < D) load_row<float, CN, VEC>(x + row, c0, D, xv);
     float ss = 0.f;
 #pragma unroll
-    for (int k = 0; k < C; ++k) ss = fmaf(v[k], v[k], ss);
+    for (int k = 0; k < CN; ++k) ss = fmaf(v[k], v[k], ss);
     const float inv = 1.f / sqrtf(row_sum(ss, red[0]) * inv_d + eps);
 #pragma unroll
-    for (int k = 0; k < C; ++k)
+    for (int k = 0; k < CN; ++k)
       v[k] = fmaf(v[k] * inv, c0 + k < D ? to_f(gain[gain_n > 1 ? c0 + k : 0]) : 0.f, xv[k]);
   }
   float ss = 0.f;
 #pragma unroll
-  for (int k = 0; k < C; ++k) ss = fmaf(v[k], v[k], ss);
+  for (int k = 0; k < CN; ++k) ss = fmaf(v[k], v[k], ss);
   const float inv = 1.f / sqrtf(row_sum(ss, red[1]) * inv_d + eps);
 #pragma unroll
-  for (int k = 0; k < C; ++k) v[k] = v[k] * inv * (c0 + k < D ? to_f(gain2[gain2_n > 1 ? c0 + k : 0]) : 0.f);
-  store_row<T, C>(out + row, c0, D, vec, v);
+  for (int k = 0; k < CN; ++k) v[k] = v[k] * inv * (c0 + k < D ? to_f(gain2[gain2_n > 1 ? c0 + k : 0]) : 0.f);
+  if (c0 < D) store_row<T, CN, VEC>(out + row, c0, D, v);
 }
 
-int threads_for(int D, int C) { return (D + C * 32 - 1) / (C * 32) * 32; }
+int threads_for(int D, int c) { return (D + c * 32 - 1) / (c * 32) * 32; }
 
 template <typename T>
 int launch_boundary(const ResidualConvParams& p, cudaStream_t stream) {
   const int grid = p.tokens / kTok + p.batch;
-  const bool wide = p.D > 2048;
-  const int C = wide ? 8 : 4, th = threads_for(p.D, C);
-  if (th > 512) {
-    if (p.D > 16 * 512) return 1;
-    const int t16 = threads_for(p.D, 16);
-    if (p.K <= 4) residual_conv_kernel<T, 16, 4><<<grid, t16, 0, stream>>>(p);
-    else residual_conv_kernel<T, 16, 8><<<grid, t16, 0, stream>>>(p);
-    return 0;
-  }
-  if (wide) {
-    if (p.K <= 4) residual_conv_kernel<T, 8, 4><<<grid, th, 0, stream>>>(p);
-    else residual_conv_kernel<T, 8, 8><<<grid, th, 0, stream>>>(p);
+  if (p.vec) {
+    if (p.K <= 4) residual_conv_kernel<T, 4, true><<<grid, kThreads, 0, stream>>>(p);
+    else residual_conv_kernel<T, 8, true><<<grid, kThreads, 0, stream>>>(p);
   } else {
-    if (p.K <= 4) residual_conv_kernel<T, 4, 4><<<grid, th, 0, stream>>>(p);
-    else residual_conv_kernel<T, 4, 8><<<grid, th, 0, stream>>>(p);
+    residual_conv_kernel<T, 8, false><<<grid, kThreads, 0, stream>>>(p);
   }
   return 0;
 }
@@ -242,20 +258,20 @@ int launch_boundary(const ResidualConvParams& p, cudaStream_t stream) {
 template <typename T>
 int launch_norm(void* out, const float* x, const void* y, const void* g, const void* g2, int gn, int g2n, float eps,
                 int tokens, int D, int vec, cudaStream_t stream) {
-#define RN(C)                                                                                                      \
-  residual_norm_kernel<T, C><<<tokens, threads_for(D, C), 0, stream>>>((T*)out, x, (const T*)y, (const T*)g,        \
-                                                                       (const T*)g2, gn, g2n, eps, D, vec)
-  if (D <= 2048) RN(4);
-  else if (D <= 8 * 512) RN(8);
-  else if (D <= 16 * 512) RN(16);
-  else return 1;
+#define RN(CN, VEC)                                                                                                  \
+  residual_norm_kernel<T, CN, VEC><<<tokens, threads_for(D, CN), 0, stream>>>((T*)out, x, (const T*)y, (const T*)g,   \
+                                                                              (const T*)g2, gn, g2n, eps, D)
+  if (D > 16 * 512) return 1;
+  if (vec && D <= 2048) RN(8, true);
+  else if (vec) RN(16, true);
+  else RN(16, false);
 #undef RN
   return 0;
 }
 
 }  // namespace
 
-// Returns 1 for sizes the kernel does not take (width above 8192, more than 8 taps).
+// Returns 1 for more than 8 taps.
 int residual_conv(const ResidualConvParams& p, int dtype, cudaStream_t stream) {
   if (p.K < 1 || p.K > 8) return 1;
   if (p.tokens <= 0 || p.batch <= 0) return 0;

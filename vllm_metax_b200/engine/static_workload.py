@@ -47,11 +47,21 @@ class StaticWorkload:
                 num_tokens=T, num_reqs=k, num_decodes=0, num_decode_tokens=0, query_start_loc=qsl,
                 seq_lens=torch.full((k,), prompt_len, dtype=torch.int32, device=dev), block_table=bt,
                 slot_mapping=slots, max_query_len=prompt_len, max_seq_len=prompt_len, block_size=bs,
-                prefill_query_start_loc=qsl, max_prefill_query_len=prompt_len)
+                prefill_query_start_loc=qsl, max_prefill_query_len=prompt_len,
+                seq_lens_cpu=torch.full((k,), prompt_len, dtype=torch.int32), query_start_loc_cpu=qsl.cpu())
+            md.extra["prefill_no_context"] = True
+            self._state_slots(md, s0, k, False)
             last = (qsl[1:] - 1).long()
             self.prefill_steps.append((s0, k, self.tokens[s0:s0 + k].reshape(-1), positions, md, last))
         self.graph = None
         self.phase_events = None     # [start, prefill done, decode done] of the latest run()
+
+    def _state_slots(self, md, first: int, n: int, has_history: bool) -> None:
+        """Request i of the workload owns state slot i (models with recurrent layers)."""
+        if self.r.state_slots is not None:
+            dev = self.r.device
+            md.extra["state_indices"] = torch.arange(first, first + n, dtype=torch.int32, device=dev)
+            md.extra["state_has_init"] = torch.full((n,), int(has_history), dtype=torch.int32, device=dev)
 
     # ------------------------------------------------------------------ decode graph
     def capture(self) -> None:
@@ -63,13 +73,14 @@ class StaticWorkload:
             seq_lens=r.seq_lens[:N], block_table=r.block_table[:N], slot_mapping=r.slot_mapping[:N],
             max_query_len=1, max_seq_len=self.P + self.O, block_size=r.block_size,
             prefill_query_start_loc=r.prefill_qsl[:1], max_prefill_query_len=0)
-        md.decode_num_splits = ops.decode_num_splits(N, r.model.kv_cache_spec().get("num_kv_heads", 1),
-                                                     self.P + self.O, 1, r.sms)
+        if r.model.kv_cache_spec()["kind"] == "gqa":          # other caches choose in their own attention op
+            md.decode_num_splits = ops.decode_num_splits(N, r.model.kv_cache_spec()["num_kv_heads"], self.P + self.O, 1, r.sms)
         if md.decode_num_splits > 1:
             spec = r.model.kv_cache_spec()
             hq = r.cfg.model.num_attention_heads // max(1, r.cfg.parallel.tensor_parallel_size)
             md.decode_workspace = torch.empty(md.decode_num_splits * N * hq * (spec["head_size"] + 1),
                                               dtype=torch.float32, device=dev)
+        self._state_slots(md, 0, N, True)
         self.decode_md = md
         self.col = torch.zeros(1, dtype=torch.int64, device=dev)
         self._reset_decode_inputs()
@@ -100,6 +111,7 @@ class StaticWorkload:
         r.block_table[:N].zero_()
         r.block_table[:N, : self.bps] = self.block_table_all
         r.positions[:N].fill_(self.P)
+        r.query_start_loc[:N + 1] = torch.arange(N + 1, dtype=torch.int32, device=r.device)
         r.seq_lens[:N].fill_(self.P + 1)
         blk = self.block_table_all[:, self.P // bs].long()
         r.slot_mapping[:N] = blk * bs + self.P % bs

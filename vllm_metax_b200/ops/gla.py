@@ -58,8 +58,9 @@ def gated_linear_attention(qkvg: torch.Tensor, offsets: Sequence[int], z: torch.
     out = torch.empty(T, H * V, dtype=qkvg.dtype, device=qkvg.device)
     B = query_start_loc.numel() - 1
     scratch = None
-    if torch.ops.b200.gla_needs_scratch(qkvg, B, H, D, V, max_query_len):
-        scratch = torch.empty(T, H * V, dtype=torch.float32, device=qkvg.device)
+    need = torch.ops.b200.gla_scratch_floats(qkvg, B, H, D, V, max_query_len)
+    if need:                               # split heads or segments: further launches
+        scratch = torch.empty(need, dtype=torch.float32, device=qkvg.device)
         ops._launches += 1
     torch.ops.b200.gla_recurrent(out, state, qkvg, *offsets, z, z_bias, norm_w, scratch, query_start_loc, state_indices,
                                  has_initial_state, scale, 1.0 / tau, eps, max_query_len)
