@@ -15,6 +15,8 @@ iterations).  Two measurements per run:
   per-step pinned-memory H2D of the step inputs and D2H of the sampled tokens.
 
 `python bench.py --gpus N --steps K --warmup W`; for N > 1 launch under torchrun.
+`--hybrid` instead prints one JSON line with the layer-list hybrid (Naguzen) beside its closest models at equal sizes:
+prefill and decode throughput, and every kernel of it against its roofline (utils/bench_hybrid.py; one GPU).
 `--impl reference` reports that the reference cannot be installed on this machine.
 """
 from __future__ import annotations
@@ -115,6 +117,18 @@ class ClockSampler:
                 "reasons": sorted(reasons), "samples": len(sm)}
 
 
+def hybrid(args) -> None:
+    from vllm_metax_b200.utils.bench_hybrid import SIZES, kernel_rows, model_rows
+
+    sampler = ClockSampler(0)
+    sampler.start()
+    rows = model_rows(steps=max(1, args.steps), warmup=max(3, args.warmup))
+    kernels = [r for size in SIZES for r in kernel_rows(size)]
+    print(json.dumps({"metric": "hybrid decoder beside its closest models (device-timed, random weights)", "n_gpus": 1,
+                      "steps": args.steps, "warmup": max(3, args.warmup), "dtype": "bf16", "data": "synthetic",
+                      "models": rows, "kernels": kernels, "clocks": sampler.stop()}))
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -131,7 +145,11 @@ def main() -> None:
                     help="pipeline stages (the other gpus / pp ranks of a stage are tensor parallel); the value is then "
                          "the end-to-end number through LLM.generate, device-timed, because the device-resident "
                          "workload driver is tensor-parallel only")
+    ap.add_argument("--hybrid", action="store_true",
+                    help="hybrid decoder (Naguzen) beside its closest models: throughput and kernel rooflines, one GPU")
     args = ap.parse_args()
+    if args.hybrid:
+        return hybrid(args)
     conf = CONFIGS[args.config]
     MODEL = conf["model"]
     args.num_reqs = args.num_reqs or conf["workload"][0]

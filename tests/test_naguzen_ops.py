@@ -120,13 +120,13 @@ def test_gated_linear_attention_over_portions(device, dt, H, D, V, tau, long):
     widths = [H * D, H * D, H * V, H * V]
     off = [8, 8 + widths[0], 8 + 2 * widths[0], 8 + 2 * widths[0] + widths[2]]
     rows = [rnd(n, off[3] + widths[3] + 5, dt=dt, seed=n) for n in lens]
-    zs = [rnd(n, H * D, seed=50 + n) * 2 for n in lens]
-    zb, nw = rnd(H * D, dt=dt) + 3, rnd(V, dt=dt) + 1
+    zs = [O.sigmoid(rnd(n, H * D, seed=50 + n).double() * 2 + 3) ** (1 / tau) for n in lens]
+    nw = rnd(V, dt=dt) + 1
     want = []
     for r, z in zip(rows, zs):
         n, p = r.shape[0], r.double()
         part = lambda i, w: p[:, off[i]: off[i] + widths[i]].reshape(n, H, w)
-        alpha = O.sigmoid(z.double() + zb.double()).view(n, H, D) ** (1 / tau)
+        alpha = z.float().double().view(n, H, D)
         o = O.gated_linear_recurrence(part(0, D) * D ** -0.5, part(1, D), part(2, V), alpha)
         g = p[:, off[3]: off[3] + widths[3]]
         want.append((O.unit_rms(o, eps) * nw.double()).reshape(n, H * V) * g * O.sigmoid(g))
@@ -134,8 +134,8 @@ def test_gated_linear_attention_over_portions(device, dt, H, D, V, tau, long):
     for step in split_steps(lens, cuts):
         qsl, idx, init = step_args(step, SLOTS, device)
         x = torch.cat([rows[s][lo:hi] for s, lo, hi in step]).to(device)
-        z = torch.cat([zs[s][lo:hi] for s, lo, hi in step]).to(device)
-        got = gated_linear_attention(x, off, z, zb.to(device), nw.to(device), state, qsl, idx, init, D ** -0.5, tau, eps,
+        z = torch.cat([zs[s][lo:hi] for s, lo, hi in step]).float().to(device)
+        got = gated_linear_attention(x, off, z, nw.to(device), state, qsl, idx, init, D ** -0.5, eps,
                                      max(hi - lo for _, lo, hi in step))
         close(got, torch.cat([want[s][lo:hi] for s, lo, hi in step]), dt, 2.0)
 
@@ -184,6 +184,9 @@ def test_product_epilogues(device, dt, M, N, K):
     close(ops.gemm(ad, wd, act="gelu"), O.gelu_erf(z), dt)
     close(ops.gemm(ad, wd, act="gelu_tanh"), O.gelu_tanh(z), dt)
     close(ops.gemm(ad, wd, act="xielu", act_params=coef), O.xielu(z, p, q), dt)
+    b = rnd(N, dt=dt) + 2
+    y = ops.gemm(ad, wd, b.to(device), act="decay", act_params=torch.full((1,), 1 / 16, device=device), out_dtype=torch.float32)
+    close(y, O.sigmoid(z + b.double()) ** (1 / 16), torch.float32)
     y = ops.gemm(ad, wd, out_dtype=torch.float32)
     assert y.dtype == torch.float32
     close(y, z, torch.float32)

@@ -27,7 +27,7 @@ _loaded_units = ""
 ACT_CODES = {"silu": 0, "gelu": 1, "gelu_tanh": 2, "fatrelu": 3, "relu2": 4, "mul_silu": 5, "swigluoai": 6,
              "swiglustep": 7, "gelu_new": 8, "gelu_fast": 9, "gelu_quick": 10}
 # GEMM epilogues (csrc/gemm_epilogue.cuh)
-EPI_CODES = {None: 0, "silu_gate": 1, "gelu": 2, "gelu_tanh": 3, "xielu": 4}
+EPI_CODES = {None: 0, "silu_gate": 1, "gelu": 2, "gelu_tanh": 3, "xielu": 4, "decay": 5}
 CACHE_KIND = {"same": 0, "fp8_static": 1, "int8_dyn": 2, "fp8_dyn": 3}
 
 
@@ -117,7 +117,7 @@ def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
          force_bn: int = 0, act: Optional[str] = None, act_params: Optional[torch.Tensor] = None,
          out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
     """``act(a [M,K] @ w [N,K]^T (+bias)) (+residual)``.  ``act``: None, gelu, gelu_tanh, xielu (``act_params`` = its two
-    fp32 coefficients), applied to the fp32 accumulators in the epilogue; ``out_dtype=torch.float32`` stores those."""
+    fp32 coefficients), decay (``sigmoid(x)^act_params[0]``), applied to the fp32 accumulators in the epilogue; ``out_dtype=torch.float32`` stores those."""
     if _use_cuda(a):
         if out is None:
             out = torch.empty(a.shape[0], w.shape[0], dtype=out_dtype or a.dtype, device=a.device)

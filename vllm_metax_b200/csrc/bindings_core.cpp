@@ -12,16 +12,16 @@ using namespace b200_bind;
 // ------------------------------------------------------------------ GEMM
 // `act`: epilogue code (csrc/gemm_epilogue.cuh); an fp32 `out` of 16-bit operands adds the fp32-store flag.
 b200::Epi make_epi(const Tensor& out, const Tensor& a, int64_t act, const optional<Tensor>& act_params) {
-  TORCH_CHECK(act >= 0 && act <= b200::kEpiXielu, "unknown epilogue ", act);
+  TORCH_CHECK(act >= 0 && act <= b200::kEpiDecay, "unknown epilogue ", act);
   int code = (int)act;
   if (out.scalar_type() != a.scalar_type()) {
     TORCH_CHECK(out.scalar_type() == at::kFloat && act != 1, "the output is of the operands' type or fp32");
     code |= b200::kEpiF32;
   }
   const float* prm = nullptr;
-  if (act == b200::kEpiXielu) {
-    TORCH_CHECK(act_params.has_value() && act_params->scalar_type() == at::kFloat && act_params->numel() == 2 &&
-                act_params->is_contiguous(), "xIELU needs its two fp32 coefficients");
+  if (act == b200::kEpiXielu || act == b200::kEpiDecay) {
+    TORCH_CHECK(act_params.has_value() && act_params->scalar_type() == at::kFloat && act_params->is_contiguous() &&
+                act_params->numel() == (act == b200::kEpiXielu ? 2 : 1), "the epilogue needs its fp32 parameters");
     prm = act_params->data_ptr<float>();
   }
   return b200::Epi(code, prm);
@@ -500,19 +500,18 @@ int64_t gla_scratch_floats(const Tensor& like, int64_t batch, int64_t heads, int
 
 // qkvg [T, >= ...]: q, k at [q_off, k_off], v at v_off, gate at g_off (each heads * size wide)
 void gla_recurrent(Tensor& out, Tensor& state, const Tensor& qkvg, int64_t q_off, int64_t k_off, int64_t v_off,
-                   int64_t g_off, const Tensor& z, const optional<Tensor>& z_bias, const Tensor& norm_w,
+                   int64_t g_off, const Tensor& alpha, const Tensor& norm_w,
                    const optional<Tensor>& scratch, const Tensor& qsl, const optional<Tensor>& state_idx,
-                   const optional<Tensor>& has_init, double scale, double inv_tau, double eps, int64_t max_query_len) {
-  on_device_of(qkvg, {&out, &state, &z, &norm_w, &qsl}, {&z_bias, &scratch, &state_idx, &has_init});
+                   const optional<Tensor>& has_init, double scale, double eps, int64_t max_query_len) {
+  on_device_of(qkvg, {&out, &state, &alpha, &norm_w, &qsl}, {&scratch, &state_idx, &has_init});
   TORCH_CHECK(state.dim() == 4 && state.is_contiguous() && state.scalar_type() == at::kFloat);
   const int64_t T = qkvg.size(0), H = state.size(1), D = state.size(2), V = state.size(3);
   TORCH_CHECK(qkvg.dim() == 2 && qkvg.stride(1) == 1 && out.is_contiguous() && out.size(0) == T && out.size(1) == H * V &&
               out.scalar_type() == qkvg.scalar_type());
   const int64_t W = qkvg.size(1);
   TORCH_CHECK(q_off + H * D <= W && k_off + H * D <= W && v_off + H * V <= W && g_off + H * V <= W);
-  TORCH_CHECK(z.is_contiguous() && z.scalar_type() == at::kFloat && z.numel() == T * H * D);
+  TORCH_CHECK(alpha.is_contiguous() && alpha.scalar_type() == at::kFloat && alpha.numel() == T * H * D);
   TORCH_CHECK(norm_w.numel() == V && norm_w.scalar_type() == qkvg.scalar_type());
-  if (z_bias.has_value()) TORCH_CHECK(z_bias->numel() == H * D && z_bias->scalar_type() == qkvg.scalar_type());
   const StepRefs s = step_refs(qsl, state_idx, has_init);
   const int sms = device_sms(qkvg);
   const int64_t need = gla_scratch_floats(qkvg, s.batch, H, D, V, max_query_len);
@@ -522,11 +521,11 @@ void gla_recurrent(Tensor& out, Tensor& state, const Tensor& qkvg, int64_t q_off
   b200::GlaParams p{};
   p.qkvg = qkvg.data_ptr(); p.row_stride = qkvg.stride(0);
   p.q_off = q_off; p.k_off = k_off; p.v_off = v_off; p.g_off = g_off;
-  p.z = z.data_ptr<float>(); p.z_bias = ptr(z_bias); p.norm_w = norm_w.data_ptr(); p.state = state.data_ptr<float>();
+  p.alpha = alpha.data_ptr<float>(); p.norm_w = norm_w.data_ptr(); p.state = state.data_ptr<float>();
   p.out = out.data_ptr();
   p.qsl = s.qsl; p.state_idx = s.idx; p.has_init = s.init; p.batch = s.batch; p.tokens = T;
   p.heads = H; p.dim = D; p.vdim = V;
-  p.scale = (float)scale; p.inv_tau = (float)inv_tau; p.eps = (float)eps;
+  p.scale = (float)scale; p.eps = (float)eps;
   const c10::cuda::CUDAGuard guard(qkvg.device());
   TORCH_CHECK(b200::gla_recurrent(p, ptr<float>(scratch), (int)max_query_len, sms, dtype_code(qkvg), cur_stream()) == 0,
               "gla_recurrent: key dimension up to 256");
@@ -607,7 +606,7 @@ TORCH_LIBRARY(b200, m) {
   m.def("residual_conv(Tensor(a!) x_out, Tensor(b!) h, Tensor y, Tensor? x, Tensor? gain, Tensor w, Tensor(c!)? carry, Tensor query_start_loc, Tensor? state_idx, Tensor? has_initial, float eps) -> ()", &residual_conv);
   m.def("residual_norm(Tensor(a!) out, Tensor y, Tensor? x, Tensor? gain, Tensor gain2, float eps) -> ()", &residual_norm);
   m.def("gla_scratch_floats(Tensor like, int batch, int heads, int dim, int vdim, int max_query_len) -> int", &gla_scratch_floats);
-  m.def("gla_recurrent(Tensor(a!) out, Tensor(b!) state, Tensor qkvg, int q_off, int k_off, int v_off, int g_off, Tensor z, Tensor? z_bias, Tensor norm_w, Tensor(c!)? scratch, Tensor query_start_loc, Tensor? state_idx, Tensor? has_initial, float scale, float inv_tau, float eps, int max_query_len) -> ()", &gla_recurrent);
+  m.def("gla_recurrent(Tensor(a!) out, Tensor(b!) state, Tensor qkvg, int q_off, int k_off, int v_off, int g_off, Tensor alpha, Tensor norm_w, Tensor(c!)? scratch, Tensor query_start_loc, Tensor? state_idx, Tensor? has_initial, float scale, float eps, int max_query_len) -> ()", &gla_recurrent);
   m.def("rglru_chunk() -> int", &rglru_chunk);
   m.def("rglru_scan(Tensor(a!) out, Tensor(b!) state, Tensor(c!) gates, Tensor u, Tensor y, Tensor r_bias, Tensor i_bias, Tensor decay, int block_width, Tensor(d!)? summary, Tensor query_start_loc, Tensor? state_idx, Tensor? has_initial, int max_query_len) -> ()", &rglru_scan);
   m.def("latent_insert(Tensor(a!) cq, Tensor(b!) cache, Tensor a, int q_off, int kv_off, Tensor q_w, Tensor kv_w, int rot_dim, Tensor inv_freq, Tensor positions, Tensor slot_mapping, float eps) -> ()", &latent_insert);

@@ -3,7 +3,7 @@
 
 namespace b200 {
 
-constexpr int kEpiGelu = 2, kEpiGeluTanh = 3, kEpiXielu = 4;
+constexpr int kEpiGelu = 2, kEpiGeluTanh = 3, kEpiXielu = 4, kEpiDecay = 5;
 constexpr int kEpiActMask = 0xf, kEpiF32 = 0x10;
 
 struct Epi {

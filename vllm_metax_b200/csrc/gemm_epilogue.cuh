@@ -3,7 +3,7 @@
 // SiLU-gate over interleaved (gate, up) columns, converts and stores.
 //
 // Epilogue codes (``Epi::code``): 0 plain, 1 SiLU-gate over interleaved pairs, 2 gelu (erf), 3 gelu (tanh), 4 xIELU with
-// the two numbers ``act[0], act[1]`` (the quadratic and the exponential coefficient); kEpiF32 added to a code makes the
+// the two numbers ``act[0], act[1]`` (the quadratic and the exponential coefficient), 5 a decay sigmoid(x)^act[0]; kEpiF32 added to a code makes the
 // output matrix fp32 (``C`` then points at floats and ``ldc`` counts floats).
 #pragma once
 #include "common.cuh"
@@ -37,6 +37,11 @@ __device__ __forceinline__ float epi_activate16(float f, int act, const float* _
   return f;
 }
 
+// sigmoid(x)^e through the logarithm: log sigmoid(x) = min(x, 0) - log1p(exp(-|x|))
+__device__ __forceinline__ float decay_of(float x, float e) {
+  return expf((fminf(x, 0.f) - log1pf(expf(-fabsf(x)))) * e);
+}
+
 // N elements at once: one branch on the activation outside the element loop (a branch per element multiplies the code of
 // the unrolled epilogue until it no longer fits the instruction cache).
 template <int N>
@@ -48,6 +53,10 @@ __device__ __forceinline__ void epi_activate16_n(float (&f)[N], int act, const f
       const float neg = cn * (__expf(fminf(f[i], 0.f)) - 1.f - f[i]), pos = cp * f[i] * f[i];
       f[i] = fmaf(0.5f, f[i], f[i] > 0.f ? pos : neg);
     }
+  } else if (act == kEpiDecay) {
+    const float e = __ldg(prm);
+#pragma unroll
+    for (int i = 0; i < N; ++i) f[i] = decay_of(f[i], e);
   } else if (act == kEpiGelu) {
 #pragma unroll
     for (int i = 0; i < N; ++i) f[i] = 0.5f * f[i] * (1.f + erf_as(f[i] * 0.70710678118654752f));
@@ -64,6 +73,7 @@ __device__ __forceinline__ float epi_activate(float f, int act, const float* __r
     if (f > 0.f) return fmaf(__ldg(prm) * f, f, 0.5f * f);
     return fmaf(__ldg(prm + 1), expm1f(f) - f, 0.5f * f);
   }
+  if (act == kEpiDecay) return decay_of(f, __ldg(prm));
   return f;
 }
 
@@ -138,6 +148,10 @@ __device__ __forceinline__ void epi_store_block_f32(const uint32_t (&r)[32], flo
     if ((epi.code & kEpiActMask) == 0) {
 #pragma unroll 8
       for (int i = 0; i < n; ++i) dst[(size_t)i * ldc] = stage[i][lane] + b;
+    } else if (epi.code == (kEpiDecay | kEpiF32)) {
+      const float e = __ldg(epi.act);
+#pragma unroll 4
+      for (int i = 0; i < n; ++i) dst[(size_t)i * ldc] = decay_of(stage[i][lane] + b, e);
     } else {
 #pragma unroll 1
       for (int i = 0; i < n; ++i)

@@ -1,16 +1,19 @@
 // Gated linear attention, recurrent form, with a decay per key channel:
 //
-//   alpha_t = sigmoid(z_t + bias)^(1 / tau)                        [dim]        (fp32)
-//   S_t     = diag(alpha_t) S_(t-1) + k_t v_t^T                    [dim, vdim]  (fp32, carried per request and head)
-//   o_t     = S_t^T (scale q_t)
-//   out_t   = o_t / sqrt(mean(o_t^2) + eps) * w * silu(g_t)        (per head over vdim)
+//   S_t   = diag(alpha_t) S_(t-1) + k_t v_t^T                      [dim, vdim]  (fp32, carried per request and head)
+//   o_t   = S_t^T (scale q_t)
+//   out_t = o_t / sqrt(mean(o_t^2) + eps) * w * silu(g_t)          (per head over vdim)
+//
+// alpha [dim] per token and head comes in fp32 (the decay epilogue of the product in front, gemm_epilogue.cuh).
 //
 // One CTA = one (sequence, head, block of value columns).  RL lanes share a column group: lane r holds rows r*4 + 4*RL*i
-// (i = 0 ..) of 4 columns in registers, so a token costs NR * 4 * 3 fused operations per thread, a few 16-byte
-// shared-memory reads (conflict-free: the lanes of a group read consecutive float4) and 4-5 shuffles; no barrier.
-// Tokens are staged kChunk at a time: q, k and the decays (computed once per channel) as fp32 in shared memory, the
-// outputs collected there and normalised, gated and stored a warp per token.  The same kernel serves a decode step (one
-// token: the state's read and write are the traffic) and a prompt portion of any length.
+// (i = 0 ..) of 4 columns in registers, pairs of rows packed for the two-wide fp32 instructions, so a token costs
+// NR * 4 * 3 / 2 of them per thread, a few 16-byte shared-memory reads (conflict-free: the lanes of a group read
+// consecutive float4) and 4-5 shuffles; no barrier.
+// Tokens are staged kChunk at a time: the next chunk's raw q, k, v and alpha arrive by cp.async while this one is computed;
+// q, k, v become fp32 in shared memory once per chunk; outputs are collected there and normalised, gated and stored a warp
+// per token.  The same kernel serves a decode step (one token: the state's read and write are the traffic) and a prompt
+// portion of any length.
 // Few long sequences would leave most SMs idle: their tokens are then cut into segments of kSeg.
 //   1. every segment but a sequence's last runs the state update alone from zero and keeps its end state and the product
 //      of its decays,
@@ -46,7 +49,60 @@ __device__ __forceinline__ void head_out(const GlaParams& p, int64_t t, int h, c
   for (int c = lane; c < p.vdim; c += 32) out[c] = from_f<T>(o[c] * inv * to_f(w[c]) * silu(to_f(g[c])));
 }
 
-template <typename T, int RL, int NR, int MODE>
+__device__ __forceinline__ uint64_t pack2f(float lo, float hi) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+  return r;
+}
+__device__ __forceinline__ void unpack2f(uint64_t v, float& lo, float& hi) {
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
+}
+__device__ __forceinline__ uint64_t mul2f(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ uint64_t fma2f(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ void cp16(void* smem, const void* gmem) {
+  const uint32_t s = static_cast<uint32_t>(__cvta_generic_to_shared(smem));
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(s), "l"(gmem) : "memory");
+}
+
+// n x width elements from rows of `stride` to rows of `pitch` in shared memory; VEC: 16 bytes at a time, asynchronously.
+template <typename E, bool VEC>
+__device__ __forceinline__ void copy_rows(E* dst, int pitch, const E* src, int64_t stride, int n, int width) {
+  if constexpr (VEC) {
+    constexpr int V = 16 / (int)sizeof(E);
+    const int per = width / V;
+    for (int i = threadIdx.x; i < n * per; i += blockDim.x)
+      cp16(dst + (i / per) * pitch + (i % per) * V, src + (i / per) * stride + (i % per) * V);
+  } else {
+    for (int i = threadIdx.x; i < n * width; i += blockDim.x) dst[(i / width) * pitch + i % width] = src[(i / width) * stride + i % width];
+  }
+}
+
+// Two stages of raw chunks (alpha needs no conversion), then the fp32 chunk and the outputs.
+template <typename T, int DP>
+struct GlaSmem {
+  int q, k, v, stage, fq, fk, fv, fo, total;               // q, k, v within a stage (alpha comes first)
+  __host__ __device__ explicit GlaSmem(int cb) {
+    q = kChunk * DP * 4;
+    k = q + kChunk * DP * (int)sizeof(T);
+    v = k + kChunk * DP * (int)sizeof(T);
+    stage = v + kChunk * cb * (int)sizeof(T);              // (16 tokens: multiples of 16 bytes throughout)
+    fq = 2 * stage;
+    fk = fq + kChunk * DP * 4;
+    fv = fk + kChunk * DP * 4;
+    fo = fv + kChunk * cb * 4;
+    total = fo + kChunk * cb * 4;
+  }
+};
+
+template <typename T, int RL, int NR, int MODE, bool VEC>
 __global__ void __launch_bounds__(RL * kMaxCols / 4, RL == 8 ? 2 : 1)
 gla_kernel(const GlaParams p) {
   constexpr int DP = RL * NR;                                // padded rows
@@ -66,93 +122,118 @@ gla_kernel(const GlaParams p) {
   if (t1 <= t0) return;
   const bool last = t1 == s1, alone = MODE == kWhole || s1 - s0 <= kSeg;
   if (MODE == kLocal && last) return;
-  extern __shared__ __align__(16) float sm[];
-  float* s_q = sm;                                           // [kChunk][DP]
-  float* s_k = s_q + kChunk * DP;
-  float* s_a = s_k + kChunk * DP;
-  float* s_v = s_a + kChunk * DP;                            // [kChunk][col_block]
-  float* s_o = s_v + kChunk * p.col_block;                   // [kChunk][col_block]
+  extern __shared__ __align__(16) uint8_t sm[];
+  const GlaSmem<T, DP> L(p.col_block);
+  float *s_q = reinterpret_cast<float*>(sm + L.fq), *s_k = reinterpret_cast<float*>(sm + L.fk),
+        *s_v = reinterpret_cast<float*>(sm + L.fv), *s_o = reinterpret_cast<float*>(sm + L.fo);
   const int tid = threadIdx.x, nthr = blockDim.x;
   const int rl = tid % RL, cg = tid / RL;                    // row lane, group of 4 columns
   const int c4 = cg * 4;
   const T* base = reinterpret_cast<const T*>(p.qkvg);
-  const T* zb = reinterpret_cast<const T*>(p.z_bias);
   const int slot = p.state_idx ? p.state_idx[b] : -1;
   float* st = slot >= 0 ? p.state + ((int64_t)slot * p.heads + h) * p.dim * p.vdim + col0 : nullptr;
   float* sg = MODE == kWhole ? nullptr : p.seg_state + ((int64_t)blockIdx.x * p.heads + h) * p.dim * p.vdim + col0;
   const float* from = MODE == kLocal ? nullptr : alone ? st : sg;
   const bool vec = (p.vdim & 3) == 0 && (col0 & 3) == 0;
-  float S[NR][4];
+  uint64_t S[NR / 2][4];                                     // rows 2i, 2i + 1 of the thread's NR, four columns
   const bool init = from != nullptr && (!alone || p.has_init == nullptr || p.has_init[b] != 0);
-  float decay[MODE == kLocal ? NR : 1];
+  uint64_t decay[MODE == kLocal ? NR / 2 : 1];
   if constexpr (MODE == kLocal) {
 #pragma unroll
-    for (int i = 0; i < NR; ++i) decay[i] = 1.f;
+    for (int i = 0; i < NR / 2; ++i) decay[i] = pack2f(1.f, 1.f);
   }
-#pragma unroll
-  for (int i = 0; i < NR; ++i) {
-    const int row = (i / 4) * (RL * 4) + rl * 4 + (i % 4);
-    S[i][0] = S[i][1] = S[i][2] = S[i][3] = 0.f;
-    if (init && row < p.dim) {
-      const float* r = from + (int64_t)row * p.vdim + c4;
-      if (vec && c4 + 4 <= cols) {
-        const float4 v = *reinterpret_cast<const float4*>(r);
-        S[i][0] = v.x; S[i][1] = v.y; S[i][2] = v.z; S[i][3] = v.w;
-      } else {
-#pragma unroll
-        for (int j = 0; j < 4; ++j) if (c4 + j < cols) S[i][j] = r[j];
-      }
-    }
-  }
-  const bool whole = gridDim.z == 1;
-  for (int tc = t0; tc < t1; tc += kChunk) {
+  // raw chunk of the tokens from tc on; what lies behind dim and behind the columns stays zero
+  auto stage = [&](int tc, int buf) {
     const int n = min(kChunk, t1 - tc);
-    for (int i = tid; i < n * DP; i += nthr) {
-      const int t = i / DP, d = i % DP;
-      float q = 0.f, k = 0.f, a = 0.f;
-      if (d < p.dim) {
-        const int64_t row = (int64_t)(tc + t) * p.row_stride + h * p.dim + d;
-        if (MODE != kLocal) q = to_f(base[row + p.q_off]) * p.scale;
-        k = to_f(base[row + p.k_off]);
-        const float z = p.z[((int64_t)(tc + t) * p.heads + h) * p.dim + d] + (zb ? to_f(zb[h * p.dim + d]) : 0.f);
-        // log sigmoid(z) = min(z, 0) - log1p(exp(-|z|))
-        a = expf((fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * p.inv_tau);
+    const T* row = base + (int64_t)tc * p.row_stride;
+    copy_rows<float, VEC>(reinterpret_cast<float*>(sm + buf * L.stage), DP, p.alpha + ((int64_t)tc * p.heads + h) * p.dim,
+                          (int64_t)p.heads * p.dim, n, p.dim);
+    if (MODE != kLocal) copy_rows<T, VEC>(reinterpret_cast<T*>(sm + buf * L.stage + L.q), DP, row + p.q_off + h * p.dim, p.row_stride, n, p.dim);
+    copy_rows<T, VEC>(reinterpret_cast<T*>(sm + buf * L.stage + L.k), DP, row + p.k_off + h * p.dim, p.row_stride, n, p.dim);
+    copy_rows<T, VEC>(reinterpret_cast<T*>(sm + buf * L.stage + L.v), p.col_block, row + p.v_off + h * p.vdim + col0, p.row_stride, n, cols);
+    if constexpr (VEC) asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  if (p.dim < DP || cols < p.col_block) {
+    for (int i = tid * 4; i < L.fq; i += nthr * 4) *reinterpret_cast<uint32_t*>(sm + i) = 0u;
+    __syncthreads();
+  }
+  stage(t0, 0);
+  auto row_of = [&](int i) { return (i / 4) * (RL * 4) + rl * 4 + (i % 4); };
+#pragma unroll
+  for (int i = 0; i < NR; i += 2) {
+    float x[2][4] = {};
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int row = row_of(i + e);
+      if (init && row < p.dim) {
+        const float* r = from + (int64_t)row * p.vdim + c4;
+        if (vec && c4 + 4 <= cols) {
+          const float4 v = *reinterpret_cast<const float4*>(r);
+          x[e][0] = v.x; x[e][1] = v.y; x[e][2] = v.z; x[e][3] = v.w;
+        } else {
+#pragma unroll
+          for (int j = 0; j < 4; ++j) if (c4 + j < cols) x[e][j] = r[j];
+        }
       }
-      if (MODE != kLocal) s_q[i] = q;
-      s_k[i] = k; s_a[i] = a;
     }
-    for (int i = tid; i < n * p.col_block; i += nthr) {
-      const int t = i / p.col_block, c = i % p.col_block;
-      s_v[i] = c < cols ? to_f(base[(int64_t)(tc + t) * p.row_stride + p.v_off + h * p.vdim + col0 + c]) : 0.f;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) S[i / 2][j] = pack2f(x[0][j], x[1][j]);
+  }
+  int buf = 0;
+  const bool whole = gridDim.z == 1;
+  for (int tc = t0; tc < t1; tc += kChunk, buf ^= 1) {
+    const int n = min(kChunk, t1 - tc);
+    if constexpr (VEC) asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();                                         // the chunk is here; the previous one has been used up
+    if (tc + kChunk < t1) stage(tc + kChunk, buf ^ 1);
+    const float* s_a = reinterpret_cast<const float*>(sm + buf * L.stage);
+    {
+      const T *rq = reinterpret_cast<const T*>(sm + buf * L.stage + L.q), *rk = reinterpret_cast<const T*>(sm + buf * L.stage + L.k),
+              *rv = reinterpret_cast<const T*>(sm + buf * L.stage + L.v);
+      for (int i = tid * 4; i < n * DP; i += nthr * 4) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          if (MODE != kLocal) s_q[i + e] = to_f(rq[i + e]) * p.scale;
+          s_k[i + e] = to_f(rk[i + e]);
+        }
+      }
+      for (int i = tid * 4; i < n * p.col_block; i += nthr * 4) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s_v[i + e] = to_f(rv[i + e]);
+      }
     }
     __syncthreads();
 #pragma unroll 2
     for (int t = 0; t < n; ++t) {
-      const float4 v = *reinterpret_cast<const float4*>(s_v + t * p.col_block + c4);
-      float o0 = 0.f, o1 = 0.f, o2 = 0.f, o3 = 0.f;
+      const float4 v4 = *reinterpret_cast<const float4*>(s_v + t * p.col_block + c4);
+      const uint64_t v[4] = {pack2f(v4.x, v4.x), pack2f(v4.y, v4.y), pack2f(v4.z, v4.z), pack2f(v4.w, v4.w)};
+      uint64_t o[4] = {0, 0, 0, 0};
 #pragma unroll
       for (int i4 = 0; i4 < NR / 4; ++i4) {
         const int off = t * DP + i4 * (RL * 4) + rl * 4;
-        const float4 a4 = *reinterpret_cast<const float4*>(s_a + off), k4 = *reinterpret_cast<const float4*>(s_k + off);
-        float4 q4 = make_float4(0.f, 0.f, 0.f, 0.f);
-        if constexpr (MODE != kLocal) q4 = *reinterpret_cast<const float4*>(s_q + off);
-        const float a[4] = {a4.x, a4.y, a4.z, a4.w}, k[4] = {k4.x, k4.y, k4.z, k4.w}, q[4] = {q4.x, q4.y, q4.z, q4.w};
+        const ulonglong2 a4 = *reinterpret_cast<const ulonglong2*>(s_a + off), k4 = *reinterpret_cast<const ulonglong2*>(s_k + off);
+        ulonglong2 q4 = make_ulonglong2(0, 0);
+        if constexpr (MODE != kLocal) q4 = *reinterpret_cast<const ulonglong2*>(s_q + off);
+        const uint64_t a[2] = {a4.x, a4.y}, k[2] = {k4.x, k4.y}, q[2] = {q4.x, q4.y};
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          float* s = S[i4 * 4 + e];
-          s[0] = fmaf(a[e], s[0], k[e] * v.x);
-          s[1] = fmaf(a[e], s[1], k[e] * v.y);
-          s[2] = fmaf(a[e], s[2], k[e] * v.z);
-          s[3] = fmaf(a[e], s[3], k[e] * v.w);
+        for (int e = 0; e < 2; ++e) {
+          uint64_t* s = S[i4 * 2 + e];
+#pragma unroll
+          for (int c = 0; c < 4; ++c) s[c] = fma2f(a[e], s[c], mul2f(k[e], v[c]));
           if constexpr (MODE == kLocal) {
-            decay[i4 * 4 + e] *= a[e];
+            decay[i4 * 2 + e] = mul2f(decay[i4 * 2 + e], a[e]);
           } else {
-            o0 = fmaf(q[e], s[0], o0);
-            o1 = fmaf(q[e], s[1], o1);
-            o2 = fmaf(q[e], s[2], o2);
-            o3 = fmaf(q[e], s[3], o3);
+#pragma unroll
+            for (int c = 0; c < 4; ++c) o[c] = fma2f(q[e], s[c], o[c]);
           }
         }
+      }
+      float o0, o1, o2, o3;
+      {
+        float x[4], y[4];
+#pragma unroll
+        for (int c = 0; c < 4; ++c) unpack2f(o[c], x[c], y[c]);
+        o0 = x[0] + y[0]; o1 = x[1] + y[1]; o2 = x[2] + y[2]; o3 = x[3] + y[3];
       }
       if constexpr (MODE == kLocal) continue;
       // sum the RL row lanes: two halving exchanges leave one column per lane pair, then plain butterflies
@@ -176,23 +257,30 @@ gla_kernel(const GlaParams p) {
         p.o_raw[((int64_t)(tc + t) * p.heads + h) * p.vdim + col0 + c] = s_o[t * p.col_block + c];
       }
     }
-    // (the next chunk's staging writes s_q .. s_v only, and its outputs come after its own barrier: s_o is safe)
+    // (the next chunk is converted after a barrier, and its outputs come after another: s_o is safe)
   }
   float* to = MODE == kLocal ? sg : last ? st : nullptr;
   if (to != nullptr) {
 #pragma unroll
-    for (int i = 0; i < NR; ++i) {
-      const int row = (i / 4) * (RL * 4) + rl * 4 + (i % 4);
-      if (row >= p.dim) continue;
-      if constexpr (MODE == kLocal) {
-        if (cg == 0 && col0 == 0) p.seg_decay[((int64_t)blockIdx.x * p.heads + h) * p.dim + row] = decay[i];
-      }
-      float* r = to + (int64_t)row * p.vdim + c4;
-      if (vec && c4 + 4 <= cols) {
-        *reinterpret_cast<float4*>(r) = make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
-      } else {
+    for (int i = 0; i < NR; i += 2) {
+      float x[2][4], d[2] = {1.f, 1.f};
 #pragma unroll
-        for (int j = 0; j < 4; ++j) if (c4 + j < cols) r[j] = S[i][j];
+      for (int j = 0; j < 4; ++j) unpack2f(S[i / 2][j], x[0][j], x[1][j]);
+      if constexpr (MODE == kLocal) unpack2f(decay[i / 2], d[0], d[1]);
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int row = row_of(i + e);
+        if (row >= p.dim) continue;
+        if constexpr (MODE == kLocal) {
+          if (cg == 0 && col0 == 0) p.seg_decay[((int64_t)blockIdx.x * p.heads + h) * p.dim + row] = d[e];
+        }
+        float* r = to + (int64_t)row * p.vdim + c4;
+        if (vec && c4 + 4 <= cols) {
+          *reinterpret_cast<float4*>(r) = make_float4(x[e][0], x[e][1], x[e][2], x[e][3]);
+        } else {
+#pragma unroll
+          for (int j = 0; j < 4; ++j) if (c4 + j < cols) r[j] = x[e][j];
+        }
       }
     }
   }
@@ -229,10 +317,14 @@ __global__ void gla_head_out_kernel(const GlaParams p) {
 template <typename T, int RL, int NR, int MODE>
 void launch_mode(const GlaParams& p, int grid_x, cudaStream_t stream) {
   const int threads = RL * p.col_block / 4;                // col_block is a multiple of 16: whole warps
-  const int smem = (3 * kChunk * RL * NR + 2 * kChunk * p.col_block) * (int)sizeof(float);
-  auto kern = gla_kernel<T, RL, NR, MODE>;
-  cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-  kern<<<dim3(grid_x, p.heads, (p.vdim + p.col_block - 1) / p.col_block), threads, smem, stream>>>(p);
+  const int smem = GlaSmem<T, RL * NR>(p.col_block).total;
+  const dim3 grid(grid_x, p.heads, (p.vdim + p.col_block - 1) / p.col_block);
+  auto go = [&](auto kern) {
+    cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    kern<<<grid, threads, smem, stream>>>(p);
+  };
+  if (p.vec) go(gla_kernel<T, RL, NR, MODE, true>);
+  else go(gla_kernel<T, RL, NR, MODE, false>);
 }
 
 template <typename T, int RL, int NR>
@@ -299,6 +391,9 @@ int gla_recurrent(GlaParams p, float* scratch, int max_query_len, int sms, int d
     p.seg_state = scratch + (g.raw + 3) / 4 * 4;
     p.seg_decay = p.seg_state + g.segments / (p.vdim + 1) * p.vdim;
   }
+  // 16-byte copies: every head's rows start and end on them
+  p.vec = p.dim % 8 == 0 && p.vdim % 8 == 0 && p.row_stride % 8 == 0 && p.q_off % 8 == 0 && p.k_off % 8 == 0 &&
+          p.v_off % 8 == 0 && reinterpret_cast<uintptr_t>(p.qkvg) % 16 == 0 && reinterpret_cast<uintptr_t>(p.alpha) % 16 == 0;
   if (dtype == 0) return dispatch<__nv_bfloat16>(p, stream);
   if (dtype == 1) return dispatch<__half>(p, stream);
   return dispatch<float>(p, stream);

@@ -314,8 +314,7 @@ struct GlaParams {
   const void* qkvg;            // [tokens, row_stride]: q | k | v | gate at the given element offsets
   int64_t row_stride;
   int q_off, k_off, v_off, g_off;
-  const float* z;              // [tokens, heads * dim] decay logits without their bias
-  const void* z_bias;          // [heads * dim] or null
+  const float* alpha;          // [tokens, heads * dim] decays
   const void* norm_w;          // [vdim]
   float* state;                // [slots, heads, dim, vdim]
   float* o_raw;                // set from the scratch: [tokens, heads * vdim] raw outputs of heads split over CTAs
@@ -323,8 +322,8 @@ struct GlaParams {
   float* seg_decay;            // ... and [segments, heads, dim], or null
   void* out;                   // [tokens, heads * vdim]
   const int* qsl; const int* state_idx; const int* has_init;
-  int batch, tokens, heads, dim, vdim, col_block;
-  float scale, inv_tau, eps;
+  int batch, tokens, heads, dim, vdim, col_block, vec;
+  float scale, eps;
 };
 struct GlaScratch { int64_t raw, segments; };
 GlaScratch gla_scratch(int batch, int tokens, int heads, int dim, int vdim, int max_query_len, int sms);

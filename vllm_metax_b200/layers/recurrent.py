@@ -77,7 +77,8 @@ class GatedLinearAttention(nn.Module):
     def __init__(self, width: int, heads: int, dim: int, vdim: int, decay_rank: int, tau: float, eps: float,
                  dtype=torch.bfloat16):
         super().__init__()
-        self.heads, self.dim, self.vdim, self.tau, self.eps, self.dtype = heads, dim, vdim, tau, eps, dtype
+        self.heads, self.dim, self.vdim, self.eps, self.dtype = heads, dim, vdim, eps, dtype
+        self.register_buffer("inv_tau", torch.full((1,), 1.0 / tau, dtype=torch.float32), persistent=False)
         self.in_proj = StackedLinear(width, {"q": heads * dim, "k": heads * dim, "v": heads * vdim, "g": heads * vdim,
                                              "a1": decay_rank}, dtype=dtype)
         self.decay_proj = _param(heads * dim, decay_rank, dtype=dtype)
@@ -93,11 +94,11 @@ class GatedLinearAttention(nn.Module):
     def forward(self, positions, h):
         md = get_forward_context().attn_metadata
         p = self.in_proj(h)
-        z = ops.gemm(self.in_proj.part(p, "a1"), self.decay_proj, out_dtype=torch.float32)
+        alpha = ops.gemm(self.in_proj.part(p, "a1"), self.decay_proj, self.decay_bias, act="decay", act_params=self.inv_tau,
+                         out_dtype=torch.float32)
         off = [self.in_proj.offsets[n] for n in ("q", "k", "v", "g")]
-        o = gated_linear_attention(p, off, z, self.decay_bias, self.head_norm, self.state, md.query_start_loc,
-                                   md.extra["state_indices"], md.extra["state_has_init"], self.dim ** -0.5, self.tau,
-                                   self.eps, md.max_query_len)
+        o = gated_linear_attention(p, off, alpha, self.head_norm, self.state, md.query_start_loc, md.extra["state_indices"],
+                                   md.extra["state_has_init"], self.dim ** -0.5, self.eps, md.max_query_len)
         return ops.gemm(o, self.out_proj)
 
 

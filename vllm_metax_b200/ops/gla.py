@@ -1,11 +1,11 @@
 """Gated linear attention with a decay per key channel (``csrc/gla.cu``), with its fp32 PyTorch statement.
 
-    alpha = sigmoid(z + z_bias)^(1/tau);  S <- diag(alpha) S + k v^T;  o = S^T (scale q)
-    out   = o / sqrt(mean(o^2) + eps) * norm_w * silu(g)            per head over its value columns
+    S <- diag(alpha) S + k v^T;  o = S^T (scale q)
+    out = o / sqrt(mean(o^2) + eps) * norm_w * silu(g)              per head over its value columns
 
-``qkvg [T, *]`` is the merged projection's output with q, k, v and g (heads side by side) at column offsets; ``z`` is fp32
-``[T, H * dim]``; ``state [slots, H, dim, vdim]`` (fp32) is read where ``has_initial_state`` says so and always written back
-at ``state_indices``.
+``qkvg [T, *]`` is the merged projection's output with q, k, v and g (heads side by side) at column offsets; ``alpha`` is
+fp32 ``[T, H * dim]``; ``state [slots, H, dim, vdim]`` (fp32) is read where ``has_initial_state`` says so and always written
+back at ``state_indices``.
 """
 from __future__ import annotations
 
@@ -15,8 +15,8 @@ import torch
 import torch.nn.functional as F
 
 
-def gated_linear_attention_ref(qkvg, offsets, z, z_bias, norm_w, state, query_start_loc, state_indices,
-                               has_initial_state, scale, tau, eps):
+def gated_linear_attention_ref(qkvg, offsets, alpha, norm_w, state, query_start_loc, state_indices, has_initial_state,
+                               scale, eps):
     H, D, V = state.shape[1:]
     T = qkvg.shape[0]
     qo, ko, vo, go = offsets
@@ -24,10 +24,7 @@ def gated_linear_attention_ref(qkvg, offsets, z, z_bias, norm_w, state, query_st
     k = qkvg[:, ko: ko + H * D].float().reshape(T, H, D)
     v = qkvg[:, vo: vo + H * V].float().reshape(T, H, V)
     g = qkvg[:, go: go + H * V].float()
-    zf = z.float().reshape(T, H * D)
-    if z_bias is not None:
-        zf = zf + z_bias.float()
-    alpha = torch.exp(F.logsigmoid(zf) / tau).reshape(T, H, D)
+    alpha = alpha.float().reshape(T, H, D)
     o = torch.zeros(T, H, V, dtype=torch.float32, device=qkvg.device)
     qsl = query_start_loc.tolist()
     for b in range(len(qsl) - 1):
@@ -43,16 +40,16 @@ def gated_linear_attention_ref(qkvg, offsets, z, z_bias, norm_w, state, query_st
     return (o.reshape(T, H * V) * F.silu(g)).to(qkvg.dtype)
 
 
-def gated_linear_attention(qkvg: torch.Tensor, offsets: Sequence[int], z: torch.Tensor, z_bias: Optional[torch.Tensor],
-                           norm_w: torch.Tensor, state: torch.Tensor, query_start_loc: torch.Tensor,
-                           state_indices: Optional[torch.Tensor], has_initial_state: Optional[torch.Tensor], scale: float,
-                           tau: float, eps: float, max_query_len: int) -> torch.Tensor:
+def gated_linear_attention(qkvg: torch.Tensor, offsets: Sequence[int], alpha: torch.Tensor, norm_w: torch.Tensor,
+                           state: torch.Tensor, query_start_loc: torch.Tensor, state_indices: Optional[torch.Tensor],
+                           has_initial_state: Optional[torch.Tensor], scale: float, eps: float,
+                           max_query_len: int) -> torch.Tensor:
     """``offsets`` = columns of (q, k, v, g) in ``qkvg``.  Returns ``[T, H * vdim]``; ``state`` is updated in place."""
     from .. import _custom_ops as ops
 
     if not ops._use_cuda(qkvg):
-        return gated_linear_attention_ref(qkvg, offsets, z, z_bias, norm_w, state, query_start_loc, state_indices,
-                                          has_initial_state, scale, tau, eps)
+        return gated_linear_attention_ref(qkvg, offsets, alpha, norm_w, state, query_start_loc, state_indices,
+                                          has_initial_state, scale, eps)
     H, D, V = state.shape[1:]
     T = qkvg.shape[0]
     out = torch.empty(T, H * V, dtype=qkvg.dtype, device=qkvg.device)
@@ -62,6 +59,6 @@ def gated_linear_attention(qkvg: torch.Tensor, offsets: Sequence[int], z: torch.
     if need:                               # split heads or segments: further launches
         scratch = torch.empty(need, dtype=torch.float32, device=qkvg.device)
         ops._launches += 1
-    torch.ops.b200.gla_recurrent(out, state, qkvg, *offsets, z, z_bias, norm_w, scratch, query_start_loc, state_indices,
-                                 has_initial_state, scale, 1.0 / tau, eps, max_query_len)
+    torch.ops.b200.gla_recurrent(out, state, qkvg, *offsets, alpha, norm_w, scratch, query_start_loc, state_indices,
+                                 has_initial_state, scale, eps, max_query_len)
     return out

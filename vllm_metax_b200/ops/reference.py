@@ -330,6 +330,8 @@ def epilogue_activation(y: torch.Tensor, act: str, params: Optional[torch.Tensor
         return torch.nn.functional.gelu(y)
     if act == "gelu_tanh":
         return torch.nn.functional.gelu(y, approximate="tanh")
+    if act == "decay":
+        return torch.exp(torch.nn.functional.logsigmoid(y) * params.float()[0])
     a, b = params.float()
     return torch.where(y > 0, a * y * y, b * (torch.expm1(y.clamp(max=0)) - y)) + 0.5 * y
 

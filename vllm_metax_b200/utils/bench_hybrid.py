@@ -177,7 +177,7 @@ def kernel_rows(size: str = "w2048", only: str = "") -> list:
         row(f"residual_norm, {phase}", lambda: residual_norm(y, x, g1, g1, 1e-6), 8.0 * T * W, 0, norm_like)
         # -- gated linear attention
         n = H * D
-        p, z, zb, hn = rn(T, 4 * n + 16), rn(T, n, dt=torch.float32), rn(n), rn(V)
+        p, al, hn = rn(T, 4 * n + 16), torch.rand(T, n, device=dev), rn(V)
         st = torch.zeros(B, H, D, V, device=dev)
         state_bytes = 4.0 * B * H * D * V * (1 + (T == B))
         q, k, v = rn(T, H, D), rn(T, H, D), rn(T, H, V)
@@ -185,7 +185,7 @@ def kernel_rows(size: str = "w2048", only: str = "") -> list:
         gdn_bytes = T * H * (2.0 * (2 * D + 2 * V) + 8) + state_bytes
         gdn_like = ("gdn_recurrent", lambda: gated_delta_rule(q, k, v, gg, bb, qsl, st, idx, init), gdn_bytes, 0)
         row(f"gla_recurrent, {phase}",
-            lambda: gated_linear_attention(p, (0, n, 2 * n, 3 * n), z, zb, hn, st, qsl, idx, init, D ** -0.5, 16.0, 1e-6, per),
+            lambda: gated_linear_attention(p, (0, n, 2 * n, 3 * n), al, hn, st, qsl, idx, init, D ** -0.5, 1e-6, per),
             T * n * (2.0 * 5 + 4) + state_bytes, 0, gdn_like)
         # -- RG-LRU
         gates, u, yy = rn(T, 16, 2, W // 16, dt=torch.float32), rn(T, W), rn(T, 2 * W)[:, :W]
@@ -255,8 +255,8 @@ def kernel_rows(size: str = "w2048", only: str = "") -> list:
         rw = rn(E, W)
         row(f"router product (fp32 out), {phase}", lambda: ops.gemm(y, rw, out_dtype=torch.float32), 2.0 * (T * W + E * W + 2 * T * E),
             2.0 * T * W * E, ("router product (bf16 out)", lambda: ops.gemm(y, rw), 2.0 * (T * W + E * W + T * E), 2.0 * T * W * E))
-        a1, a2 = rn(T, 16), rn(n, 16)
-        row(f"decay product (fp32 out), {phase}", lambda: ops.gemm(a1, a2, out_dtype=torch.float32), 4.0 * T * n,
+        a1, a2, ab, it = rn(T, 16), rn(n, 16), rn(n), torch.full((1,), 1 / 16, device=dev)
+        row(f"decay product, {phase}", lambda: ops.gemm(a1, a2, ab, act="decay", act_params=it, out_dtype=torch.float32), 4.0 * T * n,
             2.0 * T * n * 16, ("bf16 out", lambda: ops.gemm(a1, a2), 2.0 * T * n, 2.0 * T * n * 16))
     ops.check_kernel_status(0)
     return rows
