@@ -36,7 +36,7 @@ CUMEM_LIB = ROOT / "cumem_allocator.so"
 CORE_UNITS = ("attn_prefill_pingpong", "attn_prefill_tcgen05", "causal_conv1d", "fused_misc", "gemm_grouped_tcgen05",
               "gemm_pair_tcgen05", "gemm_simt", "gemm_splitk_tcgen05", "gemm_streamk_tcgen05", "gemm_tcgen05", "gla",
               "latent_attn", "mla_decode", "mla_decode_tcgen05", "moe", "residual_conv", "rglru", "sampling")
-# units whose arithmetic is 32-bit by contract (recurrences, norms, angles, fp32 products): no fast-math substitutions
+# units that compute in true 32-bit (recurrences, norms, angles, fp32 products): no fast-math substitutions
 PRECISE_UNITS = ("gemm_simt", "gla", "latent_attn", "residual_conv", "rglru")
 
 NVCC_FLAGS = [

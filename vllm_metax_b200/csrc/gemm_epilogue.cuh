@@ -176,11 +176,13 @@ __device__ __forceinline__ void store_row_segment_f32(const uint32_t (&r)[32], i
     if (cb0 + i < n_cols) dst[i] = f[i];
 }
 
-template <typename T, int CH>
+// (EXT: built with the activations and the fp32 output.  The GEMM kernels exist in both forms, so that plain and gated
+// products keep their short epilogue.)
+template <typename T, int CH, bool EXT = false>
 __device__ __forceinline__ void store_row_segment(const uint32_t (&r)[32], int row, int cb0, int n_cols,
                                                   T* __restrict__ C, int ldc, const T* __restrict__ bias,
                                                   const T* __restrict__ residual, int ldr, const Epi& epi) {
-  if (epi.code > 1) {
+  if (EXT && epi.code > 1) {
     if (epi.code & kEpiF32) store_row_segment_f32<T, CH>(r, row, cb0, n_cols, C, ldc, bias, epi);
     else epi_store_row<T, CH>(r, row, cb0, n_cols, C, ldc, bias, epi);
     return;

@@ -32,7 +32,7 @@ struct GgSmem {
   static constexpr int kDyn = kBarOffset + (2 * STAGES + 4) * 8 + 16 + 1024;
 };
 
-template <typename T, int BN, int STAGES>
+template <typename T, int BN, int STAGES, bool EXT>
 __global__ void __launch_bounds__(192, 1)
 gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmW,
                     T* __restrict__ C, const int* __restrict__ block_expert, const int* __restrict__ total_padded,
@@ -152,7 +152,7 @@ gemm_grouped_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
         uint32_t r[32];
         tmem_ld_32x32b_x32(taddr + c, r);
         tmem_ld_wait();
-        if (row < rows) store_row_segment<T, 32>(r, row, tn * BN + c, N, C, ldc, nullptr, nullptr, 0, epi);
+        if (row < rows) store_row_segment<T, 32, EXT>(r, row, tn * BN + c, N, C, ldc, nullptr, nullptr, 0, epi);
       }
       tc_fence_before_sync();
       mbar_arrive(&tmem_empty[acc]);
@@ -178,7 +178,7 @@ static void launch_grouped(const void* A, int max_rows, int lda, const void* W, 
   uint64_t ws[2] = {(uint64_t)K * 2, (uint64_t)N * K * 2};
   uint32_t wb[3] = {(uint32_t)kGgBK, (uint32_t)BN, 1};
   CUtensorMap tmW = make_tmap_nd(W, dt, 3, wd, ws, wb, CU_TENSOR_MAP_SWIZZLE_128B);
-  auto kern = gemm_grouped_kernel<T, BN, STAGES>;
+  auto kern = epi.code > 1 ? gemm_grouped_kernel<T, BN, STAGES, true> : gemm_grouped_kernel<T, BN, STAGES, false>;
   // a per-device attribute of the kernel: set on every launch (cheap) rather than once per process
   cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kDyn);
   static int sms = 0;

@@ -54,7 +54,7 @@ __device__ __forceinline__ void bulk_store_1d(void* gdst, const void* ssrc, uint
 // BULK epilogue (used with the row scatter): a thread converts its output row of the tile into shared memory and
 // sends it as ONE bulk copy of up to 512 bytes, so rows that cross NVLink travel as large writes instead of
 // 16-byte stores.
-template <typename T, int STAGES, bool BULK>
+template <typename T, int STAGES, bool BULK, bool EXT>
 __global__ void __launch_bounds__(192, 1)
 gemm_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB,
                  T* __restrict__ C, const T* __restrict__ bias, const T* __restrict__ residual, int M, int N, int K,
@@ -69,7 +69,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
   uint64_t* tmem_empty = tmem_full + 2;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(tmem_empty + 2);
 
-  __shared__ float f32_stage[BULK ? 1 : 4][32][33];   // fp32 outputs: one square per epilogue warp
+  __shared__ float f32_stage[EXT ? 4 : 1][32][33];   // fp32 outputs: one square per epilogue warp
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const uint32_t rank = cluster_ctarank();       // 0 = leader
   const int cluster_id = blockIdx.x >> 1;
@@ -227,7 +227,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
         uint32_t r[32];
         tmem_ld_32x32b_x32(taddr + c, r);
         tmem_ld_wait();
-        if constexpr (!BULK) {
+        if constexpr (EXT) {
           if (epi.code & kEpiF32) {
             epi_store_block_f32<T>(r, f32_stage[warp & 3], row - lane, M, tn * kPairBN + c, N, C, ldc, bias, epi);
             continue;
@@ -237,11 +237,11 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
           if (sc.tp > 0) {
             // the row goes to the receive slot of the rank that owns it (a peer store over NVLink for d != me)
             const int owner = row / sc.rows_per_rank;
-            store_row_segment<T, 32>(r, sc.src_rank * sc.rows_cap + (row - owner * sc.rows_per_rank),
+            store_row_segment<T, 32, EXT>(r, sc.src_rank * sc.rows_cap + (row - owner * sc.rows_per_rank),
                                      tn * kPairBN + c, N, reinterpret_cast<T*>(sc.recv[owner]), ldc, bias, nullptr, 0,
                                      epi);
           } else {
-            store_row_segment<T, 32>(r, row, tn * kPairBN + c, N, C, ldc, bias, residual, ldr, epi);
+            store_row_segment<T, 32, EXT>(r, row, tn * kPairBN + c, N, C, ldc, bias, residual, ldr, epi);
           }
         }
       }
@@ -286,16 +286,17 @@ static void launch_pair(const void* A, const void* W, void* C, const void* bias,
   CUtensorMap tmB = make_tmap_2d(W, dt, 2, N, K, ldw, 128, kPairBK);
   using L = PairSmem<STAGES, BULK>;
   static_assert(L::kDyn + (BULK ? 1 : 4) * 32 * 33 * 4 <= 232448, "shared memory budget exceeded");
-  auto kern = gemm_pair_kernel<T, STAGES, BULK>;
+  const int ext = !BULK && epi.code > 1;
+  auto kern = ext ? gemm_pair_kernel<T, STAGES, BULK, !BULK> : gemm_pair_kernel<T, STAGES, BULK, false>;
   // kernel attributes and SM counts are per device
-  static bool set[64] = {};
+  static bool set[2][64] = {};
   static int sms_dev[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
   dev = dev < 0 || dev >= 64 ? 0 : dev;
-  if (!set[dev]) {
+  if (!set[ext][dev]) {
     cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kDyn);
-    set[dev] = true;
+    set[ext][dev] = true;
   }
   if (sms_dev[dev] == 0) cudaDeviceGetAttribute(&sms_dev[dev], cudaDevAttrMultiProcessorCount, dev);
   const int sms = sms_dev[dev];

@@ -1,5 +1,5 @@
 // GEMM on the CUDA cores for what the tensor-core kernels do not take: fp32 operands (a model served in 32-bit) and
-// 16-bit shapes whose contraction length, pitches or addresses break the 16-byte rules of TMA.
+// 16-bit shapes whose depth, pitches or addresses break the 16-byte rules of TMA.
 //
 //     C[z][M,N] = act( A[z][M,K] . W[z][N,K]^T + bias[N] )        fp32 accumulation, any M, N, K, pitch, alignment
 //

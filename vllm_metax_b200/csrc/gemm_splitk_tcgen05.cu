@@ -37,7 +37,7 @@ __device__ __forceinline__ float4 ld_shared_v4(uint32_t addr) {
   return v;
 }
 
-template <typename T>
+template <typename T, bool EXT>
 __global__ void __launch_bounds__(192, 1)
 gemm_splitk_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB,
                    T* __restrict__ C, const T* __restrict__ bias, const T* __restrict__ residual, int M, int N, int K,
@@ -183,7 +183,7 @@ gemm_splitk_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constan
           r[4 * q + 3] = __float_as_uint(__uint_as_float(r[4 * q + 3]) + v.w);
         }
       }
-      if (row < M) store_row_segment<T, 32>(r, row, tn * kSkBN + c, N, C, ldc, bias, residual, ldr, epi);
+      if (row < M) store_row_segment<T, 32, EXT>(r, row, tn * kSkBN + c, N, C, ldc, bias, residual, ldr, epi);
     }
   }
   tc_fence_before_sync();
@@ -201,7 +201,7 @@ static void launch_sk(const void* A, const void* W, void* C, const void* bias, c
       std::is_same<T, __half>::value ? CU_TENSOR_MAP_DATA_TYPE_FLOAT16 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
   CUtensorMap tmA = make_tmap_2d(A, dt, 2, M, K, lda, kSkBM, kSkBK);
   CUtensorMap tmB = make_tmap_2d(W, dt, 2, N, K, ldw, kSkBN, kSkBK);
-  auto kern = gemm_splitk_kernel<T>;
+  auto kern = epi.code > 1 ? gemm_splitk_kernel<T, true> : gemm_splitk_kernel<T, false>;
   // a per-device attribute of the kernel: set on every launch (cheap) rather than once per process
   cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SkSmem::kDyn);
   const int tiles = ceil_div(M, kSkBM) * ceil_div(N, kSkBN);

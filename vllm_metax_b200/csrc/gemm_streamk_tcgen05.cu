@@ -62,7 +62,7 @@ __host__ __device__ __forceinline__ int stk_cluster_of(long long units, int clus
 
 __device__ __forceinline__ void stk_bar_epilogue() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
 
-template <typename T>
+template <typename T, bool EXT>
 __global__ void __launch_bounds__(192, 1)
 gemm_streamk_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmX,
                     T* __restrict__ C, const T* __restrict__ bias, const T* __restrict__ residual, const StkShape sh,
@@ -291,7 +291,7 @@ gemm_streamk_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_consta
               }
               if (ra + 3 < sh.N) *reinterpret_cast<uint32_t*>(crow + (ra >> 1)) = *reinterpret_cast<const uint32_t*>(o2);
               else if (ra + 1 < sh.N) crow[ra >> 1] = o2[0];
-            } else if (epi.code > 1) {
+            } else if (EXT && epi.code > 1) {
               epi_activate16_n<4>(f, epi.code & kEpiActMask, epi.act);
 #pragma unroll
               for (int e = 0; e < 4; ++e) {
@@ -337,7 +337,7 @@ gemm_streamk_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_consta
               if ((lane & 1) == 0 && ra_ok && tok0 + i < sh.M)
                 C[(size_t)(tok0 + i) * ldc + (ra >> 1)] = from_f<T>(g / (1.f + __expf(-g)) * up);
             }
-          } else if (epi.code > 1) {
+          } else if (EXT && epi.code > 1) {
             if (ra_ok) {
 #pragma unroll
               for (int i = 0; i < 16; ++i) a[i] += bv;
@@ -418,13 +418,14 @@ static void launch_stk(const void* A, const void* W, void* C, const void* bias, 
       std::is_same<T, __half>::value ? CU_TENSOR_MAP_DATA_TYPE_FLOAT16 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
   CUtensorMap tmW = make_tmap_2d(W, dt, 2, sh.N, sh.K, ldw, 128, kStkBK);
   CUtensorMap tmX = make_tmap_2d(A, dt, 2, sh.M, sh.K, lda, sh.TN / 2, kStkBK);
-  auto kern = gemm_streamk_kernel<T>;
-  static bool set[64] = {};
+  const int ext = epi.code > 1;
+  auto kern = ext ? gemm_streamk_kernel<T, true> : gemm_streamk_kernel<T, false>;
+  static bool set[2][64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
-  if (dev >= 0 && dev < 64 && !set[dev]) {
+  if (dev >= 0 && dev < 64 && !set[ext][dev]) {
     cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, StkSmem::kDyn);
-    set[dev] = true;
+    set[ext][dev] = true;
   }
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(2 * sh.clusters, 1, 1);

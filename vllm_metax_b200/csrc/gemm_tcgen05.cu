@@ -47,7 +47,7 @@ struct GemmSmemLayout {
 
 // BATCHED: both operand maps are 3-D and the tile index runs over `batches` products of one shape (C advances by
 // `c_batch` elements from one to the next).
-template <typename T, int BN, int STAGES, bool SWAP, bool BATCHED>
+template <typename T, int BN, int STAGES, bool SWAP, bool BATCHED, bool EXT>
 __global__ void __launch_bounds__(192, 1)
 gemm_tn_kernel(const __grid_constant__ CUtensorMap tmA,   // 128-row operand
                const __grid_constant__ CUtensorMap tmB,   // BN-row operand
@@ -63,7 +63,7 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmA,   // 128-row operand
   uint64_t* tmem_empty = tmem_full + 2;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(tmem_empty + 2);
 
-  __shared__ float f32_stage[SWAP ? 1 : 4][32][33];        // fp32 outputs: one square per epilogue warp
+  __shared__ float f32_stage[EXT && !SWAP ? 4 : 1][32][33];        // fp32 outputs: one square per epilogue warp
   const int warp = threadIdx.x >> 5;
   const int lane = threadIdx.x & 31;
   const int num_a = ceil_div(rows_a, kBM);
@@ -172,7 +172,7 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmA,   // 128-row operand
       const int tz = BATCHED ? tile / per_batch : 0, tr = BATCHED ? tile % per_batch : tile;
       const int ta = tr % num_a, tb = tr / num_a;
       // (an fp32 output matrix counts its elements in floats)
-      T* const C = !BATCHED ? C0 : (epi.code & kEpiF32) ? reinterpret_cast<T*>(reinterpret_cast<float*>(C0) + tz * c_batch)
+      T* const C = !BATCHED ? C0 : (EXT && (epi.code & kEpiF32)) ? reinterpret_cast<T*>(reinterpret_cast<float*>(C0) + tz * c_batch)
                                                         : C0 + tz * c_batch;
       const int acc = it & 1;
       const uint32_t acc_phase = (it >> 1) & 1;
@@ -199,10 +199,10 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmA,   // 128-row operand
         const int cb0 = tb * BN + c;  // first index in the BN-row operand
         if constexpr (!SWAP) {
           // row = token (ra), columns = output features cb0..cb0+CH
-          if (epi.code & kEpiF32) {
+          if (EXT && (epi.code & kEpiF32)) {
             if constexpr (CH == 32)
               epi_store_block_f32<T>(r, f32_stage[quarter], ra - lane, rows_a, cb0, rows_b, C, ldc, bias, epi);
-          } else if (epi.code > 1) {
+          } else if (EXT && epi.code > 1) {
             if (ra < rows_a) epi_store_row<T, CH>(r, ra, cb0, rows_b, C, ldc, bias, epi);
           } else if (ra < rows_a && epi.code == 1) {
             // columns hold interleaved (gate, up) pairs: out[:, j] = silu(gate_j) * up_j
@@ -277,7 +277,7 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmA,   // 128-row operand
               if ((lane & 1) == 0 && ra < rows_a && tok < rows_b)
                 C[(size_t)tok * ldc + (ra >> 1)] = from_f<T>(g / (1.f + __expf(-g)) * u);
             }
-          } else if (epi.code > 1) {
+          } else if (EXT && epi.code > 1) {
             if (ra < rows_a) {
               float f[CH];
 #pragma unroll
@@ -331,7 +331,7 @@ static void launch_cfg(const void* a_op, int rows_a, int lda, const void* b_op, 
       std::is_same<T, __half>::value ? CU_TENSOR_MAP_DATA_TYPE_FLOAT16 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
   CUtensorMap tmA = make_tmap_2d(a_op, dt, 2, rows_a, K, lda, kBM, kBK);
   CUtensorMap tmB = make_tmap_2d(b_op, dt, 2, rows_b, K, ldb, BN, kBK);
-  auto kern = gemm_tn_kernel<T, BN, STAGES, SWAP, false>;
+  auto kern = epi.code > 1 ? gemm_tn_kernel<T, BN, STAGES, SWAP, false, true> : gemm_tn_kernel<T, BN, STAGES, SWAP, false, false>;
   // a per-device attribute of the kernel: set on every launch (cheap) rather than once per process
   cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kDynSmem);
   const int tiles = ceil_div(rows_a, kBM) * ceil_div(rows_b, BN);
@@ -355,7 +355,7 @@ static void launch_batched(const void* a_op, int rows_a, int lda, int64_t a_batc
   };
   CUtensorMap tmA = map3(a_op, rows_a, lda, a_batch, kBM);
   CUtensorMap tmB = map3(b_op, rows_b, ldb, b_batch, BN);
-  auto kern = gemm_tn_kernel<T, BN, STAGES, SWAP, true>;
+  auto kern = epi.code > 1 ? gemm_tn_kernel<T, BN, STAGES, SWAP, true, true> : gemm_tn_kernel<T, BN, STAGES, SWAP, true, false>;
   cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kDynSmem);
   const int tiles = ceil_div(rows_a, kBM) * ceil_div(rows_b, BN) * batches;
   const int grid = tiles < num_sms() ? tiles : num_sms();
