@@ -37,7 +37,7 @@ enum Mode { kWhole, kLocal, kFromSegment };                // see above: whole s
 __device__ __forceinline__ float silu(float x) { return x / (1.f + expf(-x)); }
 
 template <typename T>
-__device__ __forceinline__ void head_out(const GlaParams& p, int64_t t, int h, const float* o, int lane, bool from_shared) {
+__device__ __forceinline__ void head_out(const GlaParams& p, int64_t t, int h, const float* o, int lane) {
   // one warp: norm over vdim, weight, silu gate
   float ss = 0.f;
   for (int c = lane; c < p.vdim; c += 32) ss = fmaf(o[c], o[c], ss);
@@ -250,7 +250,7 @@ gla_kernel(const GlaParams p) {
     if constexpr (MODE == kLocal) continue;
     const int warp = tid >> 5, lane = tid & 31, nw = nthr >> 5;
     if (whole) {
-      for (int t = warp; t < n; t += nw) head_out<T>(p, tc + t, h, s_o + t * p.col_block, lane, true);
+      for (int t = warp; t < n; t += nw) head_out<T>(p, tc + t, h, s_o + t * p.col_block, lane);
     } else {
       for (int i = tid; i < n * cols; i += nthr) {
         const int t = i / cols, c = i % cols;
@@ -311,7 +311,7 @@ __global__ void gla_head_out_kernel(const GlaParams p) {
   if (w >= (int64_t)p.tokens * p.heads) return;
   const int64_t t = w / p.heads;
   const int h = (int)(w % p.heads);
-  head_out<T>(p, t, h, p.o_raw + (t * p.heads + h) * p.vdim, threadIdx.x & 31, false);
+  head_out<T>(p, t, h, p.o_raw + (t * p.heads + h) * p.vdim, threadIdx.x & 31);
 }
 
 template <typename T, int RL, int NR, int MODE>
