@@ -301,7 +301,7 @@ def test_config_and_weight_update(tmp_path):
     path, w = checkpoint(tmp_path, cfg)
     mc = ModelConfig.from_pretrained(path)
     assert (mc.architecture, mc.vocab_size, mc.hidden_size, mc.num_hidden_layers) == ("Naguzen", 200, 96, 5)
-    assert get_model_class("Naguzen").native_units == "core" and mc.dtype == torch.bfloat16
+    assert get_model_class("Naguzen").native_units == "hybrid" and mc.dtype == torch.bfloat16
     llm = LLM(path, device="cpu", dtype="float32", num_gpu_blocks=4, max_model_len=128, max_num_seqs=1)
     new = O.random_weights(dict(cfg, decay_rank=12), seed=99)
     part = {k: v for k, v in new.items() if k.startswith(("l1.", "l4.", "head"))}

@@ -7,7 +7,8 @@ from tests import naguzen_oracle as O
 from vllm_metax_b200 import _custom_ops as ops
 from vllm_metax_b200.ops.gdn import causal_conv1d
 from vllm_metax_b200.ops.gla import gated_linear_attention
-from vllm_metax_b200.ops.residual_conv import residual_conv, residual_norm
+from vllm_metax_b200.ops.residual_conv import residual_conv
+from vllm_metax_b200.ops.residual_norm import residual_norm
 from vllm_metax_b200.ops.rglru import rglru
 
 DEVICES = ["cpu", pytest.param("cuda", marks=pytest.mark.gpu)]

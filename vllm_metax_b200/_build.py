@@ -3,8 +3,8 @@
 The shared objects are produced next to this file:
 
 * ``_b200_C.so``            - CUDA kernels + ``torch.ops.b200`` bindings
-* ``_b200_core.so``         - the core set of them alone (``CORE_UNITS`` + ``bindings_core.cpp``): all that a model class
-  with ``native_units = "core"`` calls; built on demand where the full library does not exist yet
+* ``_b200_<group>.so``      - the core set and one group of ``UNIT_GROUPS``: all that a model class with
+  ``native_units = "<group>"`` calls; built on demand where the full library does not exist yet
 * ``cumem_allocator.so``    - sleep-mode VMM allocator (CPython module, driver API)
 
 Every ``.cu`` is compiled with ``-gencode arch=compute_100a,code=sm_100a`` by a
@@ -29,15 +29,19 @@ ROOT = Path(__file__).resolve().parent
 CSRC = ROOT / "csrc"
 OBJ = ROOT / "_obj"
 LIB = ROOT / "_b200_C.so"
-CORE_LIB = ROOT / "_b200_core.so"
 CUMEM_LIB = ROOT / "cumem_allocator.so"
 
-# the units behind bindings_core.cpp
-CORE_UNITS = ("attn_prefill_pingpong", "attn_prefill_tcgen05", "causal_conv1d", "fused_misc", "gemm_grouped_tcgen05",
-              "gemm_pair_tcgen05", "gemm_simt", "gemm_splitk_tcgen05", "gemm_streamk_tcgen05", "gemm_tcgen05", "gla",
-              "latent_attn", "mla_decode", "mla_decode_tcgen05", "moe", "residual_conv", "rglru", "sampling")
+# the units behind bindings_core.cpp, and what each group adds behind bindings_<group>.cpp
+CORE_UNITS = ("attn_prefill_pingpong", "attn_prefill_tcgen05", "gemm_grouped_tcgen05", "gemm_pair_tcgen05", "gemm_simt",
+              "gemm_splitk_tcgen05", "gemm_streamk_tcgen05", "gemm_tcgen05", "moe", "residual_norm", "sampling")
+UNIT_GROUPS = {
+    "gqa": ("attn_decode", "head_norm_rope", "paged_attn_simt"),
+    "hybrid": ("causal_conv1d", "fused_misc", "gla", "latent_attn", "mla_decode", "mla_decode_tcgen05", "residual_conv",
+               "rglru"),
+}
 # units that compute in true 32-bit (recurrences, norms, angles, fp32 products): no fast-math substitutions
-PRECISE_UNITS = ("gemm_simt", "gla", "latent_attn", "residual_conv", "rglru")
+PRECISE_UNITS = ("gemm_simt", "gla", "head_norm_rope", "latent_attn", "paged_attn_simt", "residual_conv", "residual_norm",
+                 "rglru")
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-std=c++17", "-O3", "-lineinfo",
@@ -70,10 +74,14 @@ def _unit_flags(unit: str) -> list[str]:
     return NVCC_FLAGS if unit in PRECISE_UNITS else NVCC_FLAGS + ["--use_fast_math"]
 
 
-def build(verbose: bool = False, force: bool = False, core_only: bool = False) -> Optional[Path]:
+def group_lib(group: str) -> Path:
+    return ROOT / f"_b200_{group}.so"
+
+
+def build(verbose: bool = False, force: bool = False, group: Optional[str] = None) -> Optional[Path]:
     """Compile ``csrc/*.cu`` for sm_100a and link ``_b200_C.so`` in-tree.  ``B200_TARGET_DEVICE=empty`` skips the
     native build (a CPU-only checkout that runs the PyTorch reference ops; the reference's ``VLLM_TARGET_DEVICE``).
-    ``core_only`` compiles the core units and links ``_b200_core.so`` instead."""
+    ``group`` compiles the core units and those of one group and links ``_b200_<group>.so`` instead."""
     if os.environ.get("B200_TARGET_DEVICE", "cuda").lower() in ("empty", "cpu"):
         return None
     import torch
@@ -85,13 +93,15 @@ def build(verbose: bool = False, force: bool = False, core_only: bool = False) -
     jobs = []
     objs = []
     for src in sources():
-        if core_only and src.stem not in CORE_UNITS:
+        if group is not None and src.stem not in CORE_UNITS + UNIT_GROUPS[group]:
             continue
         obj = OBJ / (src.stem + ".o")
         objs.append(obj)
         if force or _newer([src, *headers], obj):
             jobs.append([nvcc, *_unit_flags(src.stem), "-I", str(CSRC), "-c", str(src), "-o", str(obj)])
-    binds = [CSRC / "bindings_core.cpp"] + ([] if core_only else [CSRC / "bindings.cpp"])
+    binds = [CSRC / "bindings_core.cpp"] + [CSRC / f"bindings_{g}.cpp" for g in UNIT_GROUPS if group in (None, g)]
+    if group is None:
+        binds.append(CSRC / "bindings.cpp")
     inc = []
     for p in include_paths(device_type="cuda") if "device_type" in include_paths.__code__.co_varnames else include_paths(cuda=True):
         inc += ["-I", p]
@@ -104,7 +114,7 @@ def build(verbose: bool = False, force: bool = False, core_only: bool = False) -
             jobs.insert(0, ["g++", "-std=c++17", "-O2", "-fPIC", f"-D_GLIBCXX_USE_CXX11_ABI={cxx_abi}",
                             "-DTORCH_EXTENSION_NAME=_b200_C", *inc, "-I", str(CSRC), "-c", str(bind_src), "-o",
                             str(bind_obj)])
-    lib = CORE_LIB if core_only else LIB
+    lib = LIB if group is None else group_lib(group)
     if jobs:
         workers = int(os.environ.get("MAX_JOBS", "0")) or min(8, os.cpu_count() or 4)
         import json
@@ -133,7 +143,7 @@ def build(verbose: bool = False, force: bool = False, core_only: bool = False) -
             libdirs += ["-L", p, f"-Wl,-rpath,{p}"]
         _run(["g++", "-shared", "-o", str(lib), *map(str, objs), *libdirs, "-L", os.path.join(_cuda_home(), "lib64"),
               "-lc10", "-lc10_cuda", "-ltorch_cpu", "-ltorch_cuda", "-ltorch", "-lcudart"])
-    if not core_only:
+    if group is None:
         build_cumem(verbose=verbose, force=force)
     return lib
 

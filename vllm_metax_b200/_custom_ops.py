@@ -20,36 +20,36 @@ from . import envs
 from .ops import reference as ref
 
 _LIB = Path(__file__).resolve().parent / "_b200_C.so"
-_CORE_LIB = Path(__file__).resolve().parent / "_b200_core.so"
 _loaded = False
 _loaded_units = ""
 
 ACT_CODES = {"silu": 0, "gelu": 1, "gelu_tanh": 2, "fatrelu": 3, "relu2": 4, "mul_silu": 5, "swigluoai": 6,
              "swiglustep": 7, "gelu_new": 8, "gelu_fast": 9, "gelu_quick": 10}
 # GEMM epilogues (csrc/gemm_epilogue.cuh)
-EPI_CODES = {None: 0, "silu_gate": 1, "gelu": 2, "gelu_tanh": 3, "xielu": 4, "decay": 5}
+EPI_CODES = {None: 0, "silu_gate": 1, "gelu": 2, "gelu_tanh": 3, "xielu": 4, "decay": 5, "relu2": 6}
 CACHE_KIND = {"same": 0, "fp8_static": 1, "int8_dyn": 2, "fp8_dyn": 3}
 
 
 def load_native(build_if_missing: bool = True, units: str = "all") -> bool:
-    """Load ``_b200_C.so`` (building it in-tree when absent and allowed).  ``units="core"``: the caller needs the core set
-    only - where the full library has not been built, the core library is built and loaded instead."""
+    """Load ``_b200_C.so`` (building it in-tree when absent and allowed).  ``units`` other than "all": the caller needs the
+    core set and that unit group only - where the full library has not been built, the group's library is built and loaded
+    instead."""
     global _loaded, _loaded_units
-    if _loaded and (units == "core" or _loaded_units == "all"):
+    if _loaded and _loaded_units in (units, "all"):
         return True
     if _loaded:
-        raise RuntimeError("this process serves a model on the core kernel library; build the full one "
+        raise RuntimeError(f"this process serves a model on the {_loaded_units!r} kernel library; build the full one "
                            "(python -m vllm_metax_b200._build) to use other ops beside it")
     lib, got = _LIB, "all"
     if not _LIB.exists():
-        if units == "core":
-            lib, got = _CORE_LIB, "core"
+        from ._build import build, group_lib
+
+        if units != "all":
+            lib, got = group_lib(units), units
         if not lib.exists():
             if not build_if_missing or envs.B200_USE_PREBUILT_KERNELS:
                 return False
-            from ._build import build
-
-            build(core_only=got == "core")
+            build(group=None if got == "all" else got)
     torch.ops.load_library(str(lib))
     _loaded, _loaded_units = True, got
     return True
@@ -397,6 +397,12 @@ def silu_and_mul_per_block_quant(x, group_size=128, ue8m0=False, act: str = "sil
 _decode_ws: dict = {}
 
 
+def kv_views(kv_cache):
+    """``(K, V)`` as ``[num_blocks, block_size, kv_heads, head]`` views of a ``[num_blocks, 2, block_size, kv_heads, head]``
+    cache; a pair of such views passes through (heads whose keys and values differ in size)."""
+    return kv_cache if isinstance(kv_cache, tuple) else (kv_cache[:, 0], kv_cache[:, 1])
+
+
 def _decode_workspace(device, numel: int) -> torch.Tensor:
     ws = _decode_ws.get(device)
     if ws is None or ws.numel() < numel:
@@ -421,8 +427,11 @@ def batch_invariant() -> bool:
 _batch_invariant: Optional[bool] = None
 
 
-def decode_num_splits(batch: int, num_kv_heads: int, max_seq_len: int, row_tiles: int = 1, sms: int = 148) -> int:
-    """Enough KV splits to give every SM a CTA, never finer than 256 tokens per split."""
+def decode_num_splits(batch: int, num_kv_heads: int, max_seq_len: int, row_tiles: int = 1, sms: int = 148,
+                      window: int = -1) -> int:
+    """Enough KV splits to give every SM a CTA, never finer than 256 tokens per split (of those a window leaves)."""
+    if window > 0:
+        max_seq_len = min(max_seq_len, window)
     if batch_invariant():
         return 1                               # the split count follows the batch size: one pass per sequence instead
     ctas = max(1, batch * num_kv_heads * row_tiles)
@@ -437,18 +446,22 @@ def paged_attention_decode(q, kv_cache, block_table, seq_lens, scale, *, out=Non
                            sinks=None, lse_out=None, num_splits: int = 0, max_seq_len: int = 0, k_scale=1.0,
                            v_scale=1.0, causal=True, workspace=None, alibi_slopes=None):
     """Decode attention over the paged cache; ``q [T, Hq, D]``.  ``alibi_slopes [Hq]`` (f32) adds
-    ``slope * (kv position - query position)`` to the scores."""
+    ``slope * (kv position - query position)`` to the scores.  ``kv_cache``: the 5-D cache or a pair of ``kv_views``.
+    fp32 caches and 16-bit heads wider than 256 run on the CUDA cores."""
     if _use_cuda(q):
-        out = torch.empty(q.shape[0], q.shape[1], kv_cache.shape[-1], dtype=q.dtype, device=q.device) if out is None else out
+        k, v = kv_views(kv_cache)
+        out = torch.empty(q.shape[0], q.shape[1], v.shape[-1], dtype=q.dtype, device=q.device) if out is None else out
         B = seq_lens.shape[0]
-        Hkv = kv_cache.shape[3]
+        Hkv = k.shape[2]
         if num_splits <= 0:
             g = q.shape[1] // Hkv
-            num_splits = decode_num_splits(B, Hkv, max_seq_len or 4096, (max_q_len * g + 15) // 16)
+            num_splits = decode_num_splits(B, Hkv, max_seq_len or 4096, (max_q_len * g + 15) // 16, window=window)
+        if q.dtype == torch.float32 or max(k.shape[-1], v.shape[-1]) > 256:
+            num_splits = 1
         ws = workspace
         if num_splits > 1 and ws is None:
-            ws = _decode_workspace(q.device, num_splits * q.shape[0] * q.shape[1] * (q.shape[2] + 1))
-        torch.ops.b200.paged_attention_decode(out, q, kv_cache, kv_scales, block_table, seq_lens, query_start_loc,
+            ws = _decode_workspace(q.device, num_splits * q.shape[0] * q.shape[1] * (v.shape[-1] + 1))
+        torch.ops.b200.paged_attention_decode(out, q, k, v, kv_scales, block_table, seq_lens, query_start_loc,
                                               scale, window, softcap, sinks, lse_out, ws, num_splits, B, max_q_len,
                                               k_scale, v_scale, causal, alibi_slopes)
         return out
@@ -471,11 +484,11 @@ def paged_attention_prefill(q, kv_cache, block_table, seq_lens, query_start_loc,
                             k_scale=1.0, v_scale=1.0, causal=True, max_seq_len: int = 0, alibi_slopes=None):
     """Varlen prefill / chunked-prefill attention reading K, V from the paged cache."""
     if _use_cuda(q):
-        out = torch.empty(q.shape[0], q.shape[1], kv_cache.shape[-1], dtype=q.dtype, device=q.device) if out is None else out
+        k, v = kv_views(kv_cache)
+        out = torch.empty(q.shape[0], q.shape[1], v.shape[-1], dtype=q.dtype, device=q.device) if out is None else out
         B = seq_lens.shape[0]
-        D = q.shape[-1]
-        if kv_cache.dtype == q.dtype and D in (64, 128) and kv_scales is None:
-            torch.ops.b200.attention_prefill(out, q, kv_cache, None, block_table, seq_lens, query_start_loc, None,
+        if k.dtype == q.dtype and q.dtype != torch.float32 and k.shape[-1] <= 192 and v.shape[-1] <= 128 and kv_scales is None:
+            torch.ops.b200.attention_prefill(out, q, k, v, block_table, seq_lens, query_start_loc, None,
                                              scale, window, softcap, sinks, lse_out, B, max_q_len or q.shape[0], causal,
                                              alibi_slopes)
         else:
@@ -728,17 +741,22 @@ def gemm_grouped(a, w, block_expert, total_padded, epi: int = 0):
     return out
 
 
-def moe_combine(y, weights, inv_pos, tokens: int, shared=None):
-    """``out[t] = sum_k weights[t,k] * y[inv_pos[t,k]] (+ shared[t])``."""
+def moe_combine(y, weights, inv_pos, tokens: int, shared=None, identity=None):
+    """``out[t] = sum_k weights[t,k] * y[inv_pos[t,k]] (+ shared[t])``.  ``identity = (ids [tokens, k], x, first)``: pairs
+    whose expert id is at least ``first`` are identity experts and contribute ``weights[t,k] * x[t]``."""
     if _use_cuda(y):
         out = torch.empty(tokens, y.shape[1], dtype=y.dtype, device=y.device)
-        torch.ops.b200.moe_combine(out, y, weights.contiguous(), inv_pos, shared)
+        ids, x, first = identity if identity is not None else (None, None, 0)
+        torch.ops.b200.moe_combine(out, y, weights.contiguous(), inv_pos, shared, ids, x, first)
         return out
     topk = weights.shape[1]
     ip = inv_pos.reshape(tokens, topk).long()
     ok = ip >= 0
     g = y[ip.clamp(min=0)].float() * (weights.float() * ok)[..., None]
     out = g.sum(dim=1)
+    if identity is not None:
+        ids, x, first = identity
+        out = out + (weights.float() * (ids >= first)).sum(1, keepdim=True) * x.float()
     if shared is not None:
         out = out + shared.float()
     return out.to(y.dtype)
@@ -956,6 +974,34 @@ def mla_decode(q, mla_cache, block_table, seq_lens, scale, *, query_start_loc=No
         out.copy_(res)
         return out
     return res
+
+
+def head_norm_rope(qkv, offsets, q_weight, k_weight, heads: int, dim: int, inv_freq, positions, kv_cache, slot_mapping,
+                   eps: float, one_plus: bool = False):
+    """Epilogue of a merged q | k | v product whose parts start at the columns ``offsets``: per-head RMS norm (``one_plus``:
+    weights stored around zero) and rotation of queries and keys, keys and values written to the paged cache
+    (``kv_cache``: 5-D or a pair of ``kv_views``) at ``slot_mapping`` (-1: nowhere).  ``kv_cache=None``: the row holds queries
+    only.  Heads are ``len(weight)`` wide, of which ``dim`` are real; ``inv_freq`` is fp64.  Returns ``q [T, heads, width]``."""
+    T, width = qkv.shape[0], q_weight.numel()
+    k, v = kv_views(kv_cache) if kv_cache is not None else (None, None)
+    if _use_cuda(qkv):
+        q = torch.empty(T, heads, width, dtype=qkv.dtype, device=qkv.device)
+        torch.ops.b200.head_norm_rope(q, qkv, *offsets, k, v, q_weight, k_weight, dim, inv_freq, positions, slot_mapping,
+                                      eps, one_plus)
+        return q
+
+    def part(at, n, w):
+        x = ref.head_rms_norm(qkv[:, at: at + n * width].reshape(T, n, width), w, dim, eps, one_plus)
+        return ref.rotate_half(x, inv_freq, positions).to(qkv.dtype)
+
+    q = part(offsets[0], heads, q_weight)
+    if k is not None:
+        G, bs, dv = k.shape[2], k.shape[1], v.shape[-1]
+        ok = slot_mapping[:T] >= 0
+        slots = slot_mapping[:T][ok]
+        k[slots // bs, slots % bs] = part(offsets[1], G, k_weight)[ok]
+        v[slots // bs, slots % bs] = qkv[:, offsets[2]: offsets[2] + G * dv].reshape(T, G, dv)[ok]
+    return q
 
 
 def latent_insert(a, q_off: int, kv_off: int, q_weight, kv_weight, rot_dim: int, inv_freq, positions, cache, slot_mapping,

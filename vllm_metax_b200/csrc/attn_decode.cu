@@ -15,7 +15,9 @@
 // scales (dequantised on the fly: K scale multiplies the logit column, V scale is
 // folded into P); 3 = e4m3 with static per-tensor scales.
 //
-// Cache layout [num_blocks, 2, block_size, num_kv_heads, D]; block_size % 16 == 0.
+// A page holds K [block_size, num_kv_heads, dqk] and V [block_size, num_kv_heads, dv] (two base pointers and one page
+// stride); block_size % 16 == 0.  16-bit heads of any size that is a multiple of 8: tiles of 64 / 128 / 256 columns whose
+// tails are filled with zeros.  With a sliding window only the tiles that some row of the CTA can see are walked.
 // Replaces flash_attn_with_kvcache (vllm_metax/v1/attention/backends/flash_attn.py:1339-1355)
 // and the Triton unified_attention int8 path (triton_attn.py:688-725).
 #include <type_traits>
@@ -138,11 +140,16 @@ __global__ void __launch_bounds__(kDecWarps * 32, (D <= 128 ? 2 : 1)) paged_deco
     report_status(p.status, kBadIndex, 21, (int)(kv_cap > 0x7fffffff ? 0x7fffffff : kv_cap), kv_len);
     kv_len = kv_len < 0 ? 0 : (int)kv_cap;
   }
-  // tiles of this split
-  const int tiles_total = (kv_len + kDecTile - 1) / kDecTile;
+  // tiles that some row of this CTA can see, and this split's part of them
+  const int last_row = min(rows_total, row0 + 16) - 1;
+  const int hi_pos = p.causal ? kv_len - q_len + last_row / g + 1 : kv_len;
+  const int lo_pos = p.window > 0 ? max(0, (p.causal ? kv_len - q_len + row0 / g + 1 : kv_len) - p.window) : 0;
+  const int tile_lo = lo_pos / kDecTile;
+  const int tiles_total = max(0, (hi_pos + kDecTile - 1) / kDecTile - tile_lo);
   const int tiles_per_split = (tiles_total + p.num_splits - 1) / p.num_splits;
-  const int tile_begin = split * tiles_per_split;
-  const int tile_end = min(tiles_total, tile_begin + tiles_per_split);
+  const int tile_begin = tile_lo + split * tiles_per_split;
+  const int tile_end = min(tile_lo + tiles_total, tile_begin + tiles_per_split);
+  const int dqk = KIND == 0 ? p.dqk : D, dv = KIND == 0 ? p.dv : D;
 
   uint8_t* q_smem = smem;
   uint8_t* wbase = smem + S::kQBytes + warp * S::kWarpBytes;
@@ -155,9 +162,9 @@ __global__ void __launch_bounds__(kDecWarps * 32, (D <= 128 ? 2 : 1)) paged_deco
       const int r = idx / CPR, c = idx % CPR;
       const int rr = row0 + r;
       uint4 v = make_uint4(0, 0, 0, 0);
-      if (rr < rows_total) {
+      if (rr < rows_total && c * 8 < dqk) {
         const int tok = q_begin + rr / g, hq = hk * g + rr % g;
-        v = *reinterpret_cast<const uint4*>(qb + (int64_t)tok * p.q_stride + (int64_t)hq * D + c * 8);
+        v = *reinterpret_cast<const uint4*>(qb + (int64_t)tok * p.q_stride + (int64_t)hq * dqk + c * 8);
       }
       *reinterpret_cast<uint4*>(q_smem + r * S::kRowBytes + ((c ^ (r & 7)) * 16)) = v;
     }
@@ -208,14 +215,17 @@ __global__ void __launch_bounds__(kDecWarps * 32, (D <= 128 ? 2 : 1)) paged_deco
     }
     const int off0 = tok0 % p.block_size;
     constexpr int RAW_CPR = S::kRawRow / 16;
-    const uint8_t* cache = reinterpret_cast<const uint8_t*>(p.kv_cache);
+    constexpr int kElem = KIND == 0 ? 2 : 1;
 #pragma unroll
     for (int kv = 0; kv < 2; ++kv) {
-      const int64_t row_base = (((int64_t)page * 2 + kv) * p.block_size + off0) * p.num_kv_heads + hk;
+      const uint8_t* cache = reinterpret_cast<const uint8_t*>(kv ? p.v_cache : p.k_cache);
+      const int d = kv ? dv : dqk;
+      const uint8_t* rows = cache + ((int64_t)page * p.page_stride + ((int64_t)off0 * p.num_kv_heads + hk) * d) * kElem;
+      const int64_t row_bytes = (int64_t)p.num_kv_heads * d * kElem;
       for (int idx = lane; idx < kDecTile * RAW_CPR; idx += 32) {
         const int r = idx / RAW_CPR, c = idx % RAW_CPR;
-        const bool ok = tile_ok && (tok0 + r) < kv_len;
-        const uint8_t* src = cache + (row_base + (int64_t)r * p.num_kv_heads) * S::kRawRow + c * 16;
+        const bool ok = tile_ok && (tok0 + r) < kv_len && (KIND != 0 || c * 8 < d);
+        const uint8_t* src = rows + r * row_bytes + c * 16;
         // 16-bit tiles are stored swizzled directly; raw 8-bit tiles are stored linearly
         const int dst_c = (KIND == 0) ? (c ^ (r & 7)) : c;
         cp_async16(st + kv * S::kRawTile + r * S::kRawRow + dst_c * 16, ok ? src : cache, ok);
@@ -223,7 +233,7 @@ __global__ void __launch_bounds__(kDecWarps * 32, (D <= 128 ? 2 : 1)) paged_deco
       if constexpr (KIND == 1 || KIND == 2) {
         if (lane < kDecTile) {
           const bool ok = tile_ok && (tok0 + lane) < kv_len;
-          const float* src = p.kv_scales + row_base + (int64_t)lane * p.num_kv_heads;
+          const float* src = p.kv_scales + (((int64_t)page * 2 + kv) * p.block_size + off0 + lane) * p.num_kv_heads + hk;
           cp_async4(st + 2 * S::kRawTile + (kv * kDecTile + lane) * 4, ok ? src : p.kv_scales, ok);
         }
       }
@@ -398,7 +408,7 @@ __global__ void __launch_bounds__(kDecWarps * 32, (D <= 128 ? 2 : 1)) paged_deco
   for (int idx = threadIdx.x; idx < 16 * D; idx += blockDim.x) {
     const int r = idx / D, c = idx % D;
     const int rr = row0 + r;
-    if (rr >= rows_total) continue;
+    if (rr >= rows_total || c >= dv) continue;
     float M = -INFINITY;
 #pragma unroll
     for (int w = 0; w < kDecWarps; ++w) M = fmaxf(M, mm[w * 16 + r]);
@@ -415,12 +425,12 @@ __global__ void __launch_bounds__(kDecWarps * 32, (D <= 128 ? 2 : 1)) paged_deco
       float Lt = L;
       if (p.sinks) Lt += exp2f(p.sinks[hq] * 1.4426950408889634f - Ms);
       const float v = Lt > 0.f ? acc / Lt * out_scale : 0.f;
-      reinterpret_cast<T*>(p.out)[((int64_t)tok * p.num_q_heads + hq) * D + c] = from_f<T>(v);
+      reinterpret_cast<T*>(p.out)[((int64_t)tok * p.num_q_heads + hq) * dv + c] = from_f<T>(v);
       if (c == 0 && p.lse_out)
         p.lse_out[(int64_t)hq * p.total_tokens + tok] = Lt > 0.f ? (Ms * 0.6931471805599453f + logf(Lt)) : -INFINITY;
     } else {
       const int64_t prow = ((int64_t)split * p.total_tokens + tok) * p.num_q_heads + hq;
-      p.part_out[prow * D + c] = L > 0.f ? acc / L * out_scale : 0.f;
+      p.part_out[prow * dv + c] = L > 0.f ? acc / L * out_scale : 0.f;
       if (c == 0) p.part_lse[prow] = L > 0.f ? (Ms * 0.6931471805599453f + logf(L)) : -INFINITY;
     }
   }
@@ -467,7 +477,8 @@ static void launch_decode(const DecodeParams& p, int batch, int max_q_len, cudaS
   if (p.num_splits > 1) {
     const int64_t rows = (int64_t)p.total_tokens * p.num_q_heads;
     attn_split_reduce_kernel<T><<<(unsigned)rows, D <= 128 ? 128 : 256, 0, stream>>>(
-        (T*)p.out, p.lse_out, p.part_out, p.part_lse, p.sinks, p.num_splits, p.total_tokens, p.num_q_heads, D);
+        (T*)p.out, p.lse_out, p.part_out, p.part_lse, p.sinks, p.num_splits, p.total_tokens, p.num_q_heads,
+        KIND == 0 ? p.dv : D);
   }
 }
 
@@ -482,9 +493,11 @@ static void decode_kind(const DecodeParams& p, int kind, int batch, int max_q_le
 }
 
 // Returns 0 on success, -1 for an unsupported head size.
-int paged_attention_decode(const DecodeParams& p, int head_dim, int kv_kind, int dtype, int batch, int max_q_len,
-                           cudaStream_t stream) {
+int paged_attention_decode(const DecodeParams& p, int kv_kind, int dtype, int batch, int max_q_len, cudaStream_t stream) {
   if (batch <= 0) return 0;
+  int head_dim = p.dqk > p.dv ? p.dqk : p.dv;
+  if (kv_kind == 0 && p.dqk % 8 == 0 && p.dv % 8 == 0) head_dim = head_dim <= 64 ? 64 : head_dim <= 128 ? 128 : head_dim <= 256 ? 256 : -1;
+  else if (p.dqk != p.dv) return -1;
 #define DISPATCH_D(T)                                                             \
   if (head_dim == 64) decode_kind<T, 64>(p, kv_kind, batch, max_q_len, stream);   \
   else if (head_dim == 128) decode_kind<T, 128>(p, kv_kind, batch, max_q_len, stream); \

@@ -19,8 +19,8 @@
 //   The three warp groups re-balance the register file at start-up (setmaxnreg): the producer / issuer
 //   group gives registers up, the softmax groups take them so that a 128-wide row of S fits.
 //
-// Query heads must be 16-bit (bf16/fp16); the tiles are (D_qk, D_v) in {(128,128), (64,64), (192,128)}.  Contiguous K / V
-// may have smaller heads (multiples of 8): the TMA maps end at the real sizes and the fill pads the tile with zeros.
+// Query heads must be 16-bit (bf16/fp16); the tiles are (D_qk, D_v) in {(128,128), (64,64), (192,128)}.  Heads may be
+// smaller (multiples of 8): the TMA maps end at the real sizes and the fill pads the tile with zeros.
 // Causal offset: row token i of a sequence with q_len new tokens and kv_len total sits at position
 // kv_len - q_len + i.  Sliding window, soft-cap, ALiBi and attention sinks are supported; LSE can be
 // returned for later merges.  TMA loads touch this GPU's memory only.
@@ -199,7 +199,7 @@ attn_prefill_pp_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
               }
               for (int c = 0; c < nch; ++c)
                 tma_load_4d(dst + c * (BN * 128) + pg * rows_per_box * 128, which ? &tmV : &tmK, full, c * 64, hk,
-                            off, page * 2 + which);
+                            off, page);
             } else {
               for (int c = 0; c < nch; ++c)
                 tma_load_3d(dst + c * (BN * 128), which ? &tmV : &tmK, full, c * 64, hk, kv_begin + tok);
@@ -433,14 +433,16 @@ static void launch_prefill_pp(const PrefillParams& p, const void* q, int64_t q_s
   CUtensorMap tmQ = make_tmap_nd(q, dt, 3, qd, qs, qb, CU_TENSOR_MAP_SWIZZLE_128B);
   CUtensorMap tmK, tmV;
   if (p.paged) {
-    // cache [num_blocks, 2, block_size, Hkv, D] -> dims [D, Hkv, block_size, 2*num_blocks]
+    // a page: [block_size, Hkv, D] of K and of V -> dims [D, Hkv, block_size, num_blocks]
     const uint32_t rows = (uint32_t)(p.block_size < BN ? p.block_size : BN);
-    uint64_t kd[4] = {(uint64_t)DQK, (uint64_t)p.num_kv_heads, (uint64_t)p.block_size, (uint64_t)(2 * p.num_blocks)};
-    uint64_t ks[3] = {(uint64_t)DQK * 2, (uint64_t)p.num_kv_heads * DQK * 2,
-                      (uint64_t)p.block_size * p.num_kv_heads * DQK * 2};
     uint32_t kb[4] = {64, 1, rows, 1};
-    tmK = make_tmap_nd(k_src, dt, 4, kd, ks, kb, CU_TENSOR_MAP_SWIZZLE_128B);
-    tmV = tmK;
+    auto page_map = [&](const void* base, uint64_t d) {
+      uint64_t kd[4] = {d, (uint64_t)p.num_kv_heads, (uint64_t)p.block_size, (uint64_t)p.num_blocks};
+      uint64_t ks[3] = {d * 2, (uint64_t)p.num_kv_heads * d * 2, (uint64_t)p.page_stride * 2};
+      return make_tmap_nd(base, dt, 4, kd, ks, kb, CU_TENSOR_MAP_SWIZZLE_128B);
+    };
+    tmK = page_map(k_src, (uint64_t)p.dqk);
+    tmV = page_map(v_src, (uint64_t)p.dv);
   } else {
     uint64_t kd[3] = {(uint64_t)p.dqk, (uint64_t)p.num_kv_heads, (uint64_t)total_kv};
     uint64_t ks[2] = {(uint64_t)p.k_head_stride * 2, (uint64_t)kv_tok_stride_k * 2};
@@ -469,18 +471,16 @@ int attention_prefill_pp(const PrefillParams& p, const void* q, int64_t q_stride
                          int64_t k_tok_stride, int64_t v_tok_stride, int64_t total_kv, int dqk, int dv, int dtype,
                          int batch, int max_q_len, cudaStream_t stream) {
   if (batch <= 0 || max_q_len <= 0) return 0;
-  if (!p.paged) {                                // contiguous K / V: round the heads up to the tile sizes
-    if (dqk % 8 != 0 || dv % 8 != 0) return -1;
-    if (dqk <= 64 && dv <= 64) dqk = dv = 64;
-    else if (dqk <= 128 && dv <= 128) dqk = dv = 128;
-    else if (dqk <= 192 && dv <= 128) dqk = 192, dv = 128;
-  }
+  if (dqk % 8 != 0 || dv % 8 != 0) return -1;    // round the heads up to the tile sizes
+  if (dqk <= 64 && dv <= 64) dqk = dv = 64;
+  else if (dqk <= 128 && dv <= 128) dqk = dv = 128;
+  else if (dqk <= 192 && dv <= 128) dqk = 192, dv = 128;
 #define PF(T)                                                                                                        \
   if (dqk == 128 && dv == 128)                                                                                       \
     launch_prefill_pp<T, 128, 128, 128>(p, q, q_stride, k_src, v_src, k_tok_stride, v_tok_stride, total_kv, batch, max_q_len, stream); \
   else if (dqk == 64 && dv == 64)                                                                                    \
     launch_prefill_pp<T, 64, 64, 128>(p, q, q_stride, k_src, v_src, k_tok_stride, v_tok_stride, total_kv, batch, max_q_len, stream);   \
-  else if (dqk == 192 && dv == 128 && !p.paged)                                                                      \
+  else if (dqk == 192 && dv == 128)                                                                                  \
     launch_prefill_pp<T, 192, 128, 64>(p, q, q_stride, k_src, v_src, k_tok_stride, v_tok_stride, total_kv, batch, max_q_len, stream); \
   else                                                                                                               \
     return -1;

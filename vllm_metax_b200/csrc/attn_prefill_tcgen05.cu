@@ -7,7 +7,7 @@
 //             of one head.
 //   warp 0    TMA producer: Q tile once, then 128-token K and V tiles through
 //             2-stage rings.  K/V come either from the paged cache (4-D tensor
-//             map [D, kv_head, slot-in-block, 2*block+kv], one box per page) or
+//             maps [D, kv_head, slot-in-block, block] of K and V, one box per page) or
 //             from contiguous [T, H, D] tensors (3-D map).
 //   warp 1    MMA issuer: S = Q.K^T into one of two TMEM buffers (so the next
 //             tile's QK^T overlaps this tile's softmax), then O_tile = P.V with P
@@ -169,7 +169,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
               }
               for (int c = 0; c < nch; ++c)
                 tma_load_4d(dst + c * (BN * 128) + pg * rows_per_box * 128, which ? &tmV : &tmK, full, c * 64, hk,
-                            off, page * 2 + which);
+                            off, page);
             } else {
               for (int c = 0; c < nch; ++c)
                 tma_load_3d(dst + c * (BN * 128), which ? &tmV : &tmK, full, c * 64, hk, kv_begin + tok);
@@ -427,14 +427,16 @@ static void launch_prefill(const PrefillParams& p, const void* q, int64_t q_stri
   CUtensorMap tmQ = make_tmap_nd(q, dt, 3, qd, qs, qb, CU_TENSOR_MAP_SWIZZLE_128B);
   CUtensorMap tmK, tmV;
   if (p.paged) {
-    // cache [num_blocks, 2, block_size, Hkv, D] -> dims [D, Hkv, block_size, 2*num_blocks]
+    // a page: [block_size, Hkv, D] of K and of V -> dims [D, Hkv, block_size, num_blocks]
     const uint32_t rows = (uint32_t)(p.block_size < BN ? p.block_size : BN);
-    uint64_t kd[4] = {(uint64_t)DQK, (uint64_t)p.num_kv_heads, (uint64_t)p.block_size, (uint64_t)(2 * p.num_blocks)};
-    uint64_t ks[3] = {(uint64_t)DQK * 2, (uint64_t)p.num_kv_heads * DQK * 2,
-                      (uint64_t)p.block_size * p.num_kv_heads * DQK * 2};
     uint32_t kb[4] = {64, 1, rows, 1};
-    tmK = make_tmap_nd(k_src, dt, 4, kd, ks, kb, CU_TENSOR_MAP_SWIZZLE_128B);
-    tmV = tmK;
+    auto page_map = [&](const void* base, uint64_t d) {
+      uint64_t kd[4] = {d, (uint64_t)p.num_kv_heads, (uint64_t)p.block_size, (uint64_t)p.num_blocks};
+      uint64_t ks[3] = {d * 2, (uint64_t)p.num_kv_heads * d * 2, (uint64_t)p.page_stride * 2};
+      return make_tmap_nd(base, dt, 4, kd, ks, kb, CU_TENSOR_MAP_SWIZZLE_128B);
+    };
+    tmK = page_map(k_src, (uint64_t)DQK);
+    tmV = page_map(v_src, (uint64_t)DV);
   } else {
     uint64_t kd[3] = {(uint64_t)DQK, (uint64_t)p.num_kv_heads, (uint64_t)total_kv};
     uint64_t ks[2] = {(uint64_t)DQK * 2, (uint64_t)kv_tok_stride_k * 2};

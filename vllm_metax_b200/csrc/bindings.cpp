@@ -124,68 +124,6 @@ void act_and_mul_quant(Tensor& out_q, const optional<Tensor>& scale_out, const o
                           (float)p0, (float)p1, group, ue8m0, dtype16(x), cur_stream());
 }
 
-// ------------------------------------------------------------------ attention
-int64_t kv_kind_of(const Tensor& cache, bool has_scales) {
-  if (cache.scalar_type() == at::kChar) return 1;
-  if (cache.scalar_type() == at::kFloat8_e4m3fn) return has_scales ? 2 : 3;
-  return 0;
-}
-
-void paged_attention_decode(Tensor& out, const Tensor& q, const Tensor& kv_cache, const optional<Tensor>& kv_scales,
-                            const Tensor& block_table, const Tensor& seq_lens,
-                            const optional<Tensor>& query_start_loc, double scale, int64_t window, double softcap,
-                            const optional<Tensor>& sinks, const optional<Tensor>& lse_out,
-                            const optional<Tensor>& workspace, int64_t num_splits, int64_t batch, int64_t max_q_len,
-                            double k_scale, double v_scale, bool causal, const optional<Tensor>& alibi_slopes) {
-  TORCH_CHECK(q.dim() == 3 && q.stride(2) == 1 && q.stride(1) == q.size(2), "q must be [T, Hq, D] with packed heads");
-  TORCH_CHECK(kv_cache.dim() == 5 && kv_cache.is_contiguous());
-  TORCH_CHECK(block_table.scalar_type() == at::kInt && seq_lens.scalar_type() == at::kInt);
-  TORCH_CHECK(out.is_contiguous());
-  b200::DecodeParams p{};
-  const int T = q.size(0), Hq = q.size(1), D = q.size(2);
-  p.out = out.data_ptr();
-  p.q = q.data_ptr();
-  p.q_stride = q.stride(0);
-  p.kv_cache = kv_cache.data_ptr();
-  p.kv_scales = ptr<float>(kv_scales);
-  p.block_table = block_table.data_ptr<int>();
-  p.seq_lens = seq_lens.data_ptr<int>();
-  p.query_start_loc = ptr<int>(query_start_loc);
-  p.sinks = ptr<float>(sinks);
-  p.alibi_slopes = ptr<float>(alibi_slopes);
-  p.lse_out = ptr<float>(lse_out);
-  p.num_q_heads = Hq;
-  p.num_kv_heads = kv_cache.size(3);
-  p.block_size = kv_cache.size(2);
-  p.max_blocks = block_table.size(1);
-  p.num_blocks = kv_cache.size(0);
-  p.num_splits = std::max<int64_t>(1, num_splits);
-  p.total_tokens = T;
-  p.scale = (float)scale;
-  p.softcap = (float)softcap;
-  p.k_scale = (float)k_scale;
-  p.v_scale = (float)v_scale;
-  p.window = (int)window;
-  p.causal = causal;
-  TORCH_CHECK(p.block_size % 16 == 0, "block_size must be a multiple of 16");
-  if (p.num_splits > 1) {
-    TORCH_CHECK(workspace.has_value(), "split-KV decode needs a workspace");
-    const int64_t need = p.num_splits * (int64_t)T * Hq * (D + 1);
-    TORCH_CHECK(workspace->scalar_type() == at::kFloat && workspace->numel() >= need, "decode workspace too small");
-    p.part_out = workspace->data_ptr<float>();
-    p.part_lse = p.part_out + p.num_splits * (int64_t)T * Hq * D;
-  }
-  p.status = reinterpret_cast<b200::StatusWord*>(status_ptr(q));
-  const c10::cuda::CUDAGuard guard(q.device());
-  const int rc = b200::paged_attention_decode(p, D, kv_kind_of(kv_cache, kv_scales.has_value()), dtype16(q), batch,
-                                              max_q_len, cur_stream());
-  TORCH_CHECK(rc == 0, "paged_attention_decode: unsupported head_dim ", D);
-}
-
-
-
-
-
 // ------------------------------------------------------------------ quantisation
 void per_token_group_quant(Tensor& q, Tensor& scales, const Tensor& x, int64_t group, bool ue8m0, bool col_major,
                            double eps) {
@@ -1057,11 +995,5 @@ TORCH_LIBRARY_FRAGMENT(b200, m) {
       "act_and_mul_quant(Tensor(a!) out_q, Tensor(b!)? scale_out, Tensor? scale_in, Tensor x, int act, float p0, "
       "float p1, int group, bool ue8m0) -> ()",
       &act_and_mul_quant);
-  m.def(
-      "paged_attention_decode(Tensor(a!) out, Tensor q, Tensor kv_cache, Tensor? kv_scales, Tensor block_table, "
-      "Tensor seq_lens, Tensor? query_start_loc, float scale, int window, float softcap, Tensor? sinks, "
-      "Tensor(b!)? lse_out, Tensor(c!)? workspace, int num_splits, int batch, int max_q_len, float k_scale, "
-      "float v_scale, bool causal, Tensor? alibi_slopes=None) -> ()",
-      &paged_attention_decode);
   m.def("weak_ref_tensor(Tensor input) -> Tensor", &weak_ref_tensor);
 }

@@ -48,6 +48,20 @@ inline void on_device_of(const Tensor& ref, std::initializer_list<const Tensor*>
       TORCH_CHECK((*o)->device() == ref.device(), "tensors on ", (*o)->device(), " and ", ref.device());
 }
 
+// K [num_blocks, block_size, heads, dqk] and V [.., dv] of one paged cache: dense token rows inside a page, one page stride.
+struct PagedViews {
+  int64_t num_blocks, page_stride;
+  int block_size, heads, dqk, dv;
+};
+inline PagedViews paged_views(const Tensor& k, const Tensor& v) {
+  TORCH_CHECK(k.dim() == 4 && v.dim() == 4 && k.size(0) == v.size(0) && k.size(1) == v.size(1) && k.size(2) == v.size(2) &&
+              k.scalar_type() == v.scalar_type(), "paged K / V must be [num_blocks, block_size, kv_heads, head] views");
+  for (const Tensor* t : {&k, &v})
+    TORCH_CHECK(t->stride(3) == 1 && t->stride(2) == t->size(3) && t->stride(1) == t->size(2) * t->size(3) &&
+                t->stride(0) == k.stride(0), "paged K / V: dense token rows and one page stride");
+  return {k.size(0), k.stride(0), (int)k.size(1), (int)k.size(2), (int)k.size(3), (int)v.size(3)};
+}
+
 // One status word per device, zero-initialised on first use.
 inline Tensor& status_tensor(int device) {
   static std::vector<Tensor> words(64);

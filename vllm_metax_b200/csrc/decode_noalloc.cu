@@ -77,7 +77,12 @@ extern "C" int b200_paged_decode_noalloc(void* out, const void* q, const void* k
   p.out = out;
   p.q = q;
   p.q_stride = (int64_t)num_q_heads * head_dim;
-  p.kv_cache = kv_cache;
+  // a page: K [block_size, heads, head_dim], then V
+  const int64_t part = (int64_t)block_size * num_kv_heads * head_dim;
+  p.k_cache = kv_cache;
+  p.v_cache = static_cast<const uint8_t*>(kv_cache) + part * (cache_dtype == 0 ? 2 : 1);
+  p.page_stride = 2 * part;
+  p.dqk = p.dv = head_dim;
   p.kv_scales = kv_scales;
   p.block_table = block_table;
   p.seq_lens = seq_lens;
@@ -103,7 +108,7 @@ extern "C" int b200_paged_decode_noalloc(void* out, const void* q, const void* k
     p.part_lse = scratch + (uint64_t)num_splits * batch * num_q_heads * head_dim;
   }
   const int kind = cache_dtype == 0 ? 0 : (cache_dtype == 1 ? 1 : 2);
-  if (b200::paged_attention_decode(p, head_dim, kind, dtype, batch, 1, reinterpret_cast<cudaStream_t>(stream)) != 0)
+  if (b200::paged_attention_decode(p, kind, dtype, batch, 1, reinterpret_cast<cudaStream_t>(stream)) != 0)
     return fail(-5, "unsupported head_dim (64, 128 and 256 are built)");
   const cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) {

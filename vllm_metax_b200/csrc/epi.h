@@ -3,7 +3,8 @@
 
 namespace b200 {
 
-constexpr int kEpiGelu = 2, kEpiGeluTanh = 3, kEpiXielu = 4, kEpiDecay = 5;
+constexpr int kEpiGelu = 2, kEpiGeluTanh = 3, kEpiXielu = 4, kEpiDecay = 5, kEpiRelu2 = 6;
+constexpr int kEpiLast = kEpiRelu2;
 constexpr int kEpiActMask = 0xf, kEpiF32 = 0x10;
 
 struct Epi {

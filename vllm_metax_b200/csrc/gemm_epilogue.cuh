@@ -3,8 +3,8 @@
 // SiLU-gate over interleaved (gate, up) columns, converts and stores.
 //
 // Epilogue codes (``Epi::code``): 0 plain, 1 SiLU-gate over interleaved pairs, 2 gelu (erf), 3 gelu (tanh), 4 xIELU with
-// the two numbers ``act[0], act[1]`` (the quadratic and the exponential coefficient), 5 a decay sigmoid(x)^act[0]; kEpiF32 added to a code makes the
-// output matrix fp32 (``C`` then points at floats and ``ldc`` counts floats).
+// the two numbers ``act[0], act[1]`` (the quadratic and the exponential coefficient), 5 a decay sigmoid(x)^act[0],
+// 6 relu(x)^2; kEpiF32 added to a code makes the output matrix fp32 (``C`` then points at floats and ``ldc`` counts floats).
 #pragma once
 #include "common.cuh"
 #include "epi.h"
@@ -57,6 +57,9 @@ __device__ __forceinline__ void epi_activate16_n(float (&f)[N], int act, const f
     const float e = __ldg(prm);
 #pragma unroll
     for (int i = 0; i < N; ++i) f[i] = decay_of(f[i], e);
+  } else if (act == kEpiRelu2) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) f[i] = fmaxf(f[i], 0.f) * f[i];
   } else if (act == kEpiGelu) {
 #pragma unroll
     for (int i = 0; i < N; ++i) f[i] = 0.5f * f[i] * (1.f + erf_as(f[i] * 0.70710678118654752f));
@@ -74,6 +77,7 @@ __device__ __forceinline__ float epi_activate(float f, int act, const float* __r
     return fmaf(__ldg(prm + 1), expm1f(f) - f, 0.5f * f);
   }
   if (act == kEpiDecay) return decay_of(f, __ldg(prm));
+  if (act == kEpiRelu2) return fmaxf(f, 0.f) * f;
   return f;
 }
 

@@ -6,7 +6,8 @@
 //   moe_align          (token, k) pairs -> expert-contiguous order padded to `block` rows per
 //                      expert: sorted_token_ids, expert id per row block, padded total
 //   moe_gather         A_perm[i] = x[sorted_token_ids[i] / topk] (zero rows for padding)
-//   moe_combine        out[t] = sum_k w[t,k] * Y[position of (t,k)]  (+ optional shared-expert add)
+//   moe_combine        out[t] = sum_k w[t,k] * Y[position of (t,k)]  (+ optional shared-expert add; identity experts add
+//                      w[t,k] * x[t])
 //   moe_sum            out[t] = sum_k in[t,k,:]
 // Parity: csrc/moe/topk_softmax_kernels.cu:80-560, topk_softplus_sqrt_kernels.cu:90,
 // grouped_topk_kernels.cu:547, moe_align_sum_kernels.cu:25-369 of the reference.
@@ -297,11 +298,23 @@ __global__ void moe_gather_kernel(T* __restrict__ out, const T* __restrict__ x, 
   for (int v = threadIdx.x; v < hidden / 8; v += blockDim.x) dst[v] = src[v];
 }
 
-// out[t] = sum_k w[t,k] * y[inv_pos[t*topk+k]]  (+ shared[t]); pairs with inv_pos < 0 are skipped.
+// The row that (token, k) pair `i` of token t contributes: an expert's output row, the token's own row for an identity
+// expert, null for a pair that is computed elsewhere.
+template <typename T>
+__device__ __forceinline__ const T* combine_row(const T* y, const T* through, const int* __restrict__ expert_ids,
+                                                int identity_from, const int* __restrict__ inv_pos, size_t i, size_t t,
+                                                int hidden) {
+  const int pos = inv_pos[i];
+  if (pos >= 0) return y + (size_t)pos * hidden;
+  return through != nullptr && expert_ids[i] >= identity_from ? through + t * hidden : nullptr;
+}
+
+// out[t] = sum_k w[t,k] * row of pair (t, k)  (+ shared[t])
 template <typename T>
 __global__ void moe_combine_kernel(T* __restrict__ out, const T* __restrict__ y, const float* __restrict__ weights,
-                                   const int* __restrict__ inv_pos, const T* __restrict__ shared, int topk,
-                                   int hidden) {
+                                   const int* __restrict__ inv_pos, const T* __restrict__ shared,
+                                   const int* __restrict__ expert_ids, const T* __restrict__ through, int identity_from,
+                                   int topk, int hidden) {
   const int t = blockIdx.x;
   for (int v = threadIdx.x; v < hidden / 8; v += blockDim.x) {
     float acc[8];
@@ -309,11 +322,11 @@ __global__ void moe_combine_kernel(T* __restrict__ out, const T* __restrict__ y,
     for (int i = 0; i < 8; ++i) acc[i] = 0.f;
     if (shared) unpack8<T>(reinterpret_cast<const uint4*>(shared + (size_t)t * hidden)[v], acc);
     for (int k = 0; k < topk; ++k) {
-      const int pos = inv_pos[(size_t)t * topk + k];
-      if (pos < 0) continue;
+      const T* row = combine_row(y, through, expert_ids, identity_from, inv_pos, (size_t)t * topk + k, (size_t)t, hidden);
+      if (row == nullptr) continue;
       const float w = weights[(size_t)t * topk + k];
       float f[8];
-      unpack8<T>(reinterpret_cast<const uint4*>(y + (size_t)pos * hidden)[v], f);
+      unpack8<T>(reinterpret_cast<const uint4*>(row)[v], f);
 #pragma unroll
       for (int i = 0; i < 8; ++i) acc[i] += w * f[i];
     }
@@ -336,13 +349,14 @@ __global__ void moe_gather_scalar_kernel(T* __restrict__ out, const T* __restric
 template <typename T>
 __global__ void moe_combine_scalar_kernel(T* __restrict__ out, const T* __restrict__ y,
                                           const float* __restrict__ weights, const int* __restrict__ inv_pos,
-                                          const T* __restrict__ shared, int topk, int hidden) {
+                                          const T* __restrict__ shared, const int* __restrict__ expert_ids,
+                                          const T* __restrict__ through, int identity_from, int topk, int hidden) {
   const size_t t = blockIdx.x;
   for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
     float acc = shared ? to_f(shared[t * hidden + i]) : 0.f;
     for (int k = 0; k < topk; ++k) {
-      const int pos = inv_pos[t * topk + k];
-      if (pos >= 0) acc = fmaf(weights[t * topk + k], to_f(y[(size_t)pos * hidden + i]), acc);
+      const T* row = combine_row(y, through, expert_ids, identity_from, inv_pos, t * topk + k, t, hidden);
+      if (row != nullptr) acc = fmaf(weights[t * topk + k], to_f(row[i]), acc);
     }
     out[t * hidden + i] = from_f<T>(acc);
   }
@@ -408,21 +422,22 @@ void moe_gather(void* out, const void* x, const int* sorted_ids, const int* tota
     moe_gather_kernel<__half><<<max_padded, th, 0, stream>>>((__half*)out, (const __half*)x, sorted_ids, total_padded, numel, topk, hidden);
 }
 
-void moe_combine(void* out, const void* y, const float* weights, const int* inv_pos, const void* shared, int tokens,
-                 int topk, int hidden, int dtype, cudaStream_t stream) {
+void moe_combine(void* out, const void* y, const float* weights, const int* inv_pos, const void* shared,
+                 const int* expert_ids, const void* through, int identity_from, int tokens, int topk, int hidden, int dtype,
+                 cudaStream_t stream) {
   if (tokens <= 0) return;
+#define COMBINE(KERNEL, T, THREADS)                                                                                       \
+  KERNEL<T><<<tokens, THREADS, 0, stream>>>((T*)out, (const T*)y, weights, inv_pos, (const T*)shared, expert_ids,          \
+                                            (const T*)through, identity_from, topk, hidden)
   if (dtype == 2 || hidden % 8 != 0) {
-    DISPATCH_16(dtype,
-                (moe_combine_scalar_kernel<<<tokens, 128, 0, stream>>>((__nv_bfloat16*)out, (const __nv_bfloat16*)y, weights, inv_pos, (const __nv_bfloat16*)shared, topk, hidden)),
-                (moe_combine_scalar_kernel<<<tokens, 128, 0, stream>>>((__half*)out, (const __half*)y, weights, inv_pos, (const __half*)shared, topk, hidden)),
-                (moe_combine_scalar_kernel<<<tokens, 128, 0, stream>>>((float*)out, (const float*)y, weights, inv_pos, (const float*)shared, topk, hidden)))
+    DISPATCH_16(dtype, (COMBINE(moe_combine_scalar_kernel, __nv_bfloat16, 128)),
+                (COMBINE(moe_combine_scalar_kernel, __half, 128)), (COMBINE(moe_combine_scalar_kernel, float, 128)))
     return;
   }
   const int th = hidden / 8 < 256 ? (hidden / 8 < 32 ? 32 : hidden / 8) : 256;
-  if (dtype == 0)
-    moe_combine_kernel<__nv_bfloat16><<<tokens, th, 0, stream>>>((__nv_bfloat16*)out, (const __nv_bfloat16*)y, weights, inv_pos, (const __nv_bfloat16*)shared, topk, hidden);
-  else
-    moe_combine_kernel<__half><<<tokens, th, 0, stream>>>((__half*)out, (const __half*)y, weights, inv_pos, (const __half*)shared, topk, hidden);
+  if (dtype == 0) COMBINE(moe_combine_kernel, __nv_bfloat16, th);
+  else COMBINE(moe_combine_kernel, __half, th);
+#undef COMBINE
 }
 
 void moe_sum(void* out, const void* in, int tokens, int topk, int hidden, int dtype, cudaStream_t stream) {

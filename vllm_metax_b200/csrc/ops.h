@@ -15,7 +15,9 @@ struct DecodeParams {
   float* part_out;           // [splits, T, Hq, D]
   float* part_lse;           // [splits, T, Hq]
   const void* q;             // [T, Hq, D] with token stride q_stride (elements)
-  const void* kv_cache;
+  const void* k_cache;       // K of page 0; token rows of num_kv_heads * dqk elements
+  const void* v_cache;       // V of page 0; token rows of num_kv_heads * dv elements
+  int64_t page_stride;       // elements between two pages (of K and of V)
   const float* kv_scales;    // kinds 1, 2
   const int* block_table;    // [B, max_blocks]
   const int* seq_lens;       // [B]
@@ -26,6 +28,7 @@ struct DecodeParams {
   int64_t q_stride;
   int num_q_heads, num_kv_heads, block_size, max_blocks, num_splits, total_tokens;
   int64_t num_blocks;
+  int dqk, dv;               // head sizes (8-bit caches: both the tile size of the kernel)
   float scale, softcap, k_scale, v_scale;
   int window;                // <=0: none
   int causal;
@@ -49,6 +52,7 @@ struct PrefillParams {
   int window, causal, paged;
   int dqk, dv;                   // head sizes (the kernel's tiles are padded up to 64 / 128 / 192 by the TMA fill)
   int64_t k_head_stride, v_head_stride;   // contiguous mode, elements
+  int64_t page_stride;           // paged mode: elements between two pages (of K and of V)
   StatusWord* status;
 };
 
@@ -138,8 +142,9 @@ void activation(void* out, const void* x, int64_t n, int act, float p0, int dtyp
 void act_and_mul_quant(void* out_q, float* scale_out, const float* scale_in, const void* x, int tokens, int d, int act,
                        float p0, float p1, int group, int ue8m0, int dtype, cudaStream_t stream);
 // ---- attention
-int paged_attention_decode(const DecodeParams& p, int head_dim, int kv_kind, int dtype, int batch, int max_q_len,
-                           cudaStream_t stream);
+int paged_attention_decode(const DecodeParams& p, int kv_kind, int dtype, int batch, int max_q_len, cudaStream_t stream);
+// paged_attn_simt.cu: the same on the CUDA cores for fp32 caches and head sizes beyond the tensor-core kernels
+int paged_attn_simt(const DecodeParams& p, int dtype, int batch, cudaStream_t stream);
 int attention_prefill(const PrefillParams& p, const void* q, int64_t q_stride, const void* k_src, const void* v_src,
                       int64_t k_tok_stride, int64_t v_tok_stride, int64_t total_kv, int dqk, int dv, int dtype,
                       int batch, int max_q_len, cudaStream_t stream);
@@ -170,8 +175,10 @@ void moe_align(int* sorted_ids, int* block_expert, int* total_padded, int* inv_p
                const int* expert_map, int numel, int experts, int block, int max_padded, cudaStream_t stream);
 void moe_gather(void* out, const void* x, const int* sorted_ids, const int* total_padded, int max_padded, int numel,
                 int topk, int hidden, int dtype, cudaStream_t stream);
-void moe_combine(void* out, const void* y, const float* weights, const int* inv_pos, const void* shared, int tokens,
-                 int topk, int hidden, int dtype, cudaStream_t stream);
+// (expert_ids / through given: a pair whose expert id is at least identity_from adds its weight times the row of `through`)
+void moe_combine(void* out, const void* y, const float* weights, const int* inv_pos, const void* shared,
+                 const int* expert_ids, const void* through, int identity_from, int tokens, int topk, int hidden, int dtype,
+                 cudaStream_t stream);
 void moe_sum(void* out, const void* in, int tokens, int topk, int hidden, int dtype, cudaStream_t stream);
 void gemm_grouped(const void* A, int max_rows, int lda, const void* W, int E, int N, int K, void* C, int ldc,
                   const int* block_expert, const int* total_padded, Epi epi, int dtype, cudaStream_t stream,
@@ -307,8 +314,41 @@ struct ResidualConvParams {
   float eps;
 };
 int residual_conv(const ResidualConvParams& p, int dtype, cudaStream_t stream);
-int residual_norm(void* out, const float* x, const void* y, const void* gain, const void* gain2, int gain_n, int gain2_n,
-                  float eps, int tokens, int D, int vec, int dtype, cudaStream_t stream);
+// ---- residual_norm.cu (norm of a finished sublayer's output + residual add + norm in front of the next one)
+struct ResidualNormParams {
+  const void* y;           // [rows, D] sublayer output; its row for token t is t, ids[t], or a weighted sum (topk > 0)
+  const int64_t* ids;      // [tokens] rows of y (an embedding table of `rows` rows), or null
+  const float* weights;    // topk > 0: y holds expert-sorted rows, token t's is sum_k weights[t, k] * y[inv_pos[t, k]]
+  const int* inv_pos;      //   ... pairs with inv_pos < 0 are skipped,
+  const int* expert_ids;   //   ... unless expert_ids[t, k] >= identity_from: those add weights[t, k] * through[t]
+  const void* through;     // [tokens, D] or null
+  const void* shared;      // [tokens, D] added to the sum, or null
+  const float* x;          // [tokens, D] residual stream, or null: x' = scale * y
+  float* x_out;            // [tokens, D] new residual stream or null (may be x itself)
+  void* h;                 // [tokens, D] x' normed
+  const void* gain;        // norm of y: 1 or D numbers
+  const void* gain2;       // norm of x': 1 or D numbers
+  int gain_n, gain2_n, gain_f32;   // gain_f32: the gains are fp32 (else of y's type)
+  int tokens, D, vec, topk, identity_from;
+  int64_t rows;
+  float eps, scale;
+  StatusWord* status;
+};
+int residual_norm(const ResidualNormParams& p, int dtype, cudaStream_t stream);
+// ---- head_norm_rope.cu (epilogue of a merged q | k | v product: head norms, partial rotation, paged cache write)
+struct HeadNormRopeParams {
+  const void* qkv; int64_t row_stride; int q_off, k_off, v_off;   // [tokens, ...], heads packed from these columns on
+  void* q_out;                          // [tokens, heads, dim_pad]
+  void* k_cache; void* v_cache;         // K / V of page 0, or null: queries only
+  int64_t page_stride, num_slots;       // elements between two pages
+  const void* q_w; const void* k_w;     // [dim_pad] norm weights or null (no norm)
+  const double* inv_freq;               // [rot / 2]
+  const int64_t* positions; const int64_t* slots;
+  int tokens, heads, kv_heads, dim, dim_pad, vdim_pad, rot, block_size, one_plus, vec;
+  float eps;
+  StatusWord* status;
+};
+int head_norm_rope(const HeadNormRopeParams& p, int dtype, cudaStream_t stream);
 // ---- gla.cu (gated linear attention: decay per key channel)
 struct GlaParams {
   const void* qkvg;            // [tokens, row_stride]: q | k | v | gate at the given element offsets

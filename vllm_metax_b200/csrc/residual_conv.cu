@@ -15,56 +15,13 @@
 // Tile i of sequence b is CTA floor(qsl[b] / kTok) + b + i: always enough of them, found by bisection.
 #include <type_traits>
 
-#include "common.cuh"
 #include "ops.h"
+#include "row_vec.cuh"
 
 namespace b200 {
 namespace {
 
 constexpr int kTok = 16;
-
-template <typename T, int C, bool VEC>
-__device__ __forceinline__ void load_row(const T* __restrict__ p, int c0, int D, float (&f)[C]) {
-  if constexpr (VEC) {
-    constexpr int kBytes = C * (int)sizeof(T);
-    if constexpr (kBytes % 16 == 0) {
-      uint4 r[kBytes / 16];
-#pragma unroll
-      for (int i = 0; i < kBytes / 16; ++i) r[i] = reinterpret_cast<const uint4*>(p + c0)[i];
-      const T* e = reinterpret_cast<const T*>(r);
-#pragma unroll
-      for (int i = 0; i < C; ++i) f[i] = to_f(e[i]);
-    } else {
-      const uint2 r = *reinterpret_cast<const uint2*>(p + c0);
-      const T* e = reinterpret_cast<const T*>(&r);
-#pragma unroll
-      for (int i = 0; i < C; ++i) f[i] = to_f(e[i]);
-    }
-  } else {
-#pragma unroll
-    for (int i = 0; i < C; ++i) f[i] = c0 + i < D ? to_f(p[c0 + i]) : 0.f;
-  }
-}
-
-template <typename T, int C, bool VEC>
-__device__ __forceinline__ void store_row(T* __restrict__ p, int c0, int D, const float (&f)[C]) {
-  if constexpr (VEC) {
-    constexpr int kBytes = C * (int)sizeof(T);
-    alignas(16) T e[C];
-#pragma unroll
-    for (int i = 0; i < C; ++i) e[i] = from_f<T>(f[i]);
-    if constexpr (kBytes % 16 == 0) {
-#pragma unroll
-      for (int i = 0; i < kBytes / 16; ++i) reinterpret_cast<uint4*>(p + c0)[i] = reinterpret_cast<const uint4*>(e)[i];
-    } else {
-      *reinterpret_cast<uint2*>(p + c0) = *reinterpret_cast<const uint2*>(e);
-    }
-  } else {
-#pragma unroll
-    for (int i = 0; i < C; ++i)
-      if (c0 + i < D) p[c0 + i] = from_f<T>(f[i]);
-  }
-}
 
 constexpr int kThreads = 256, kRows = kTok + 8;
 constexpr int C = 4;                                       // channels of a thread
@@ -201,48 +158,6 @@ residual_conv_kernel(const ResidualConvParams p) {
   }
 }
 
-// Sum over the CTA with one barrier; the caller alternates between two buffers.
-__device__ __forceinline__ float row_sum(float v, float* red) {
-  v = warp_sum(v);
-  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
-  __syncthreads();
-  const int nw = blockDim.x >> 5;
-  const float s = (int)(threadIdx.x & 31) < nw ? red[threadIdx.x & 31] : 0.f;
-  return warp_sum(s);
-}
-
-// out = norm2(x + norm1(y)): the last boundary, in front of the LM head.  One CTA per token.
-template <typename T, int CN, bool VEC>
-__global__ void __launch_bounds__(512)
-residual_norm_kernel(T* __restrict__ out, const float* __restrict__ x, const T* __restrict__ y,
-                     const T* __restrict__ gain, const T* __restrict__ gain2, int gain_n, int gain2_n, float eps, int D) {
-  __shared__ float red[2][32];
-  const int c0 = threadIdx.x * CN;
-  const int64_t row = (int64_t)blockIdx.x * D;
-  float v[CN] = {}, xv[CN] = {};
-  if (c0 < D) load_row<T, CN, VEC>(y + row, c0, D, v);
-  const float inv_d = 1.f / (float)D;
-  if (x != nullptr) {
-    if (c0 < D) load_row<float, CN, VEC>(x + row, c0, D, xv);
-    float ss = 0.f;
-#pragma unroll
-    for (int k = 0; k < CN; ++k) ss = fmaf(v[k], v[k], ss);
-    const float inv = 1.f / sqrtf(row_sum(ss, red[0]) * inv_d + eps);
-#pragma unroll
-    for (int k = 0; k < CN; ++k)
-      v[k] = fmaf(v[k] * inv, c0 + k < D ? to_f(gain[gain_n > 1 ? c0 + k : 0]) : 0.f, xv[k]);
-  }
-  float ss = 0.f;
-#pragma unroll
-  for (int k = 0; k < CN; ++k) ss = fmaf(v[k], v[k], ss);
-  const float inv = 1.f / sqrtf(row_sum(ss, red[1]) * inv_d + eps);
-#pragma unroll
-  for (int k = 0; k < CN; ++k) v[k] = v[k] * inv * (c0 + k < D ? to_f(gain2[gain2_n > 1 ? c0 + k : 0]) : 0.f);
-  if (c0 < D) store_row<T, CN, VEC>(out + row, c0, D, v);
-}
-
-int threads_for(int D, int c) { return (D + c * 32 - 1) / (c * 32) * 32; }
-
 template <typename T>
 int launch_boundary(const ResidualConvParams& p, cudaStream_t stream) {
   const int grid = p.tokens / kTok + p.batch;
@@ -255,20 +170,6 @@ int launch_boundary(const ResidualConvParams& p, cudaStream_t stream) {
   return 0;
 }
 
-template <typename T>
-int launch_norm(void* out, const float* x, const void* y, const void* g, const void* g2, int gn, int g2n, float eps,
-                int tokens, int D, int vec, cudaStream_t stream) {
-#define RN(CN, VEC)                                                                                                  \
-  residual_norm_kernel<T, CN, VEC><<<tokens, threads_for(D, CN), 0, stream>>>((T*)out, x, (const T*)y, (const T*)g,   \
-                                                                              (const T*)g2, gn, g2n, eps, D)
-  if (D > 16 * 512) return 1;
-  if (vec && D <= 2048) RN(8, true);
-  else if (vec) RN(16, true);
-  else RN(16, false);
-#undef RN
-  return 0;
-}
-
 }  // namespace
 
 // Returns 1 for more than 8 taps.
@@ -278,15 +179,6 @@ int residual_conv(const ResidualConvParams& p, int dtype, cudaStream_t stream) {
   if (dtype == 0) return launch_boundary<__nv_bfloat16>(p, stream);
   if (dtype == 1) return launch_boundary<__half>(p, stream);
   return launch_boundary<float>(p, stream);
-}
-
-int residual_norm(void* out, const float* x, const void* y, const void* gain, const void* gain2, int gain_n, int gain2_n,
-                  float eps, int tokens, int D, int vec, int dtype, cudaStream_t stream) {
-  if (tokens <= 0) return 0;
-  if (dtype == 0)
-    return launch_norm<__nv_bfloat16>(out, x, y, gain, gain2, gain_n, gain2_n, eps, tokens, D, vec, stream);
-  if (dtype == 1) return launch_norm<__half>(out, x, y, gain, gain2, gain_n, gain2_n, eps, tokens, D, vec, stream);
-  return launch_norm<float>(out, x, y, gain, gain2, gain_n, gain2_n, eps, tokens, D, vec, stream);
 }
 
 }  // namespace b200

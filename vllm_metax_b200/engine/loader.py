@@ -118,6 +118,24 @@ def safetensors_shapes(path: str) -> dict[str, tuple]:
     return out
 
 
+def copy_to_slots(slots: dict, weights, complete: bool = True) -> set[str]:
+    """Copies a checkpoint's tensors to where a model's ``slots()`` say: name -> tensor, or (view, shape in the checkpoint).
+    Unknown names, shapes that do not fit and (``complete``) missing tensors are errors."""
+    loaded: set[str] = set()
+    for name, w in weights:
+        if name not in slots:
+            raise ValueError(f"unexpected tensor {name!r} in the checkpoint")
+        dst = slots[name]
+        dst, shape = dst if isinstance(dst, tuple) else (dst, dst.shape)
+        if w.numel() != dst.numel() or (w.dim() > 1 and len(shape) > 1 and tuple(w.shape) != tuple(shape)):
+            raise ValueError(f"tensor {name!r}: shape {tuple(w.shape)} does not fit {tuple(shape)}")
+        dst.copy_(w.reshape(dst.shape).to(dst.dtype))
+        loaded.add(name)
+    if complete and len(loaded) < len(slots):
+        raise ValueError(f"tensors missing from the checkpoint: {sorted(set(slots) - loaded)[:8]}")
+    return loaded
+
+
 def save_sharded_state(model: nn.Module, path: str, rank: int) -> None:
     from safetensors.torch import save_file
 

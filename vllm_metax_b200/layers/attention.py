@@ -18,6 +18,7 @@ import torch.nn as nn
 from .. import _custom_ops as ops
 from ..attention.metadata import get_forward_context
 from ..ops import turboquant as tq
+from .recurrent import StackedLinear, _param
 
 KV_DTYPES = {
     "auto": None, "bfloat16": torch.bfloat16, "float16": torch.float16, "fp8": torch.float8_e4m3fn,
@@ -27,7 +28,7 @@ KV_DTYPES = {
 
 class PagedGQABackend:
     name = "PAGED_GQA"
-    supported_head_sizes = (64, 128, 256)
+    supported_head_sizes = (64, 128, 256)      # 8-bit caches; 16-bit ones take every multiple of 8 up to 256
     supported_kv_cache_dtypes = tuple(KV_DTYPES)
 
     @staticmethod
@@ -41,6 +42,25 @@ class PagedGQABackend:
     @staticmethod
     def supported_block_sizes():
         return (16, 32, 64, 128, 256)
+
+    @staticmethod
+    def allocate_pages(num_blocks, block_size, num_kv_heads, head_size, v_head_size, dtype, device):
+        """Cache of a layer whose keys and values may differ in size: the usual 5-D tensor where they do not, otherwise one
+        row per page, ``[K of the page's tokens | V of them]``."""
+        if head_size == v_head_size:
+            shape = PagedGQABackend.get_kv_cache_shape(num_blocks, block_size, num_kv_heads, head_size)
+        else:
+            shape = (num_blocks, block_size * num_kv_heads * (head_size + v_head_size))
+        return torch.zeros(shape, dtype=dtype, device=device)
+
+    @staticmethod
+    def views(cache: torch.Tensor, block_size: int, num_kv_heads: int, head_size: int, v_head_size: int):
+        """``(K, V)`` views ``[num_blocks, block_size, num_kv_heads, size]`` of what ``allocate_pages`` returned."""
+        if cache.dim() == 5:
+            return cache[:, 0], cache[:, 1]
+        n = block_size * num_kv_heads
+        shape = (cache.shape[0], block_size, num_kv_heads)
+        return (cache[:, : n * head_size].view(*shape, head_size), cache[:, n * head_size:].view(*shape, v_head_size))
 
     @staticmethod
     def allocate(num_blocks, block_size, num_kv_heads, head_size, model_dtype, kv_cache_dtype: str, device):
@@ -103,10 +123,16 @@ class Attention(nn.Module):
         q3 = q.reshape(T, self.num_heads, self.head_size)
         if not q3.is_contiguous() and q3.stride(1) != self.head_size:
             q3 = q3.contiguous()
-        out = torch.empty(T, self.num_heads, self.head_size, dtype=q.dtype, device=q.device)
-        nd, ndt = md.num_decodes, md.num_decode_tokens
         if "cascade_blocks" in md.extra and self.window == -1 and self.alibi_slopes is None and self.sinks is None:
-            return self._forward_cascade(q3, out, md, kv_cache, kv_scales)
+            return self._forward_cascade(q3, md, kv_cache, kv_scales)
+        return self.attend(q3, md, kv_cache, kv_scales).reshape(T, self.num_heads * self.head_size)
+
+    def attend(self, q3: torch.Tensor, md, kv_cache, kv_scales=None) -> torch.Tensor:
+        """``q3 [T, heads, D]`` over the cache, which already holds this step's keys and values (written by this layer or by the
+        one whose cache it reads): decode rows, then prompt portions.  ``kv_cache``: 5-D or a pair of views."""
+        v_size = kv_cache[1].shape[-1] if isinstance(kv_cache, tuple) else self.head_size
+        out = torch.empty(q3.shape[0], self.num_heads, v_size, dtype=q3.dtype, device=q3.device)
+        nd, ndt = md.num_decodes, md.num_decode_tokens
         if nd > 0:
             ops.paged_attention_decode(q3[:ndt], kv_cache, md.block_table[:nd], md.seq_lens[:nd], self.scale,
                                        out=out[:ndt], kv_scales=kv_scales, window=self.window, softcap=self.softcap,
@@ -119,9 +145,9 @@ class Attention(nn.Module):
                                         max_q_len=md.max_prefill_query_len, window=self.window, softcap=self.softcap,
                                         sinks=self.sinks, k_scale=self.k_scale, v_scale=self.v_scale,
                                         max_seq_len=md.max_seq_len, alibi_slopes=self.alibi_slopes)
-        return out.reshape(T, self.num_heads * self.head_size)
+        return out
 
-    def _forward_cascade(self, q3, out, md, kv_cache, kv_scales) -> torch.Tensor:
+    def _forward_cascade(self, q3, md, kv_cache, kv_scales) -> torch.Tensor:
         """Shared-prefix (cascade) attention: the leading ``cascade_blocks`` cache blocks are the same physical blocks
         for every request of the step, so all of the step's query tokens attend them in ONE pass (one pseudo request,
         no causal mask: the prefix precedes every query), every request attends the rest of its own context, and the
@@ -261,3 +287,65 @@ class Attention(nn.Module):
                                  max_q_len=md.max_query_len, causal=True, window=self.window, softcap=self.softcap,
                                  sinks=self.sinks)
         return out.reshape(T, self.num_heads * self.head_size)
+
+
+class QKNormAttention(nn.Module):
+    """Grouped-query attention with RMS-normed, partially rotated queries and keys, key and value sizes of its own, an optional
+    sliding window, and optionally the keys and values of another layer (``kv_from``: that layer's module, which must come
+    earlier in the step) instead of projections and a cache of its own.
+
+        merged q | k | v product -> ``head_norm_rope`` (norms, rotation, cache write) -> paged attention -> output product
+
+    Head sizes are padded to multiples of 8 with zero rows of the projections (and zero columns of the output product)."""
+
+    def __init__(self, width: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, eps: float,
+                 inv_freq: torch.Tensor, cache_idx: int, window: Optional[int] = None,
+                 kv_from: Optional["QKNormAttention"] = None, dtype=torch.bfloat16):
+        super().__init__()
+        if heads % kv_heads:
+            raise ValueError(f"{heads} query heads over {kv_heads} key / value heads")
+        self.width, self.heads, self.kv_heads, self.dim, self.vdim, self.eps = width, heads, kv_heads, dim, vdim, eps
+        self.dim_pad, self.vdim_pad = -(-dim // 8) * 8, -(-vdim // 8) * 8
+        self.own_kv = kv_from is None
+        if kv_from is not None and (kv_from.kv_heads, kv_from.dim, kv_from.vdim) != (kv_heads, dim, vdim):
+            raise ValueError("a layer that reads another layer's keys and values has its key / value heads and sizes")
+        parts = {"q": heads * self.dim_pad}
+        if self.own_kv:
+            parts.update(k=kv_heads * self.dim_pad, v=kv_heads * self.vdim_pad)
+        self.proj = StackedLinear(width, parts, dtype=dtype)
+        self.offsets = tuple(self.proj.offsets.get(n, 0) for n in ("q", "k", "v"))
+        self.q_norm = _param(self.dim_pad, dtype=dtype)
+        self.k_norm = _param(self.dim_pad, dtype=dtype) if self.own_kv else None
+        self.out_proj = _param(width, heads * self.vdim_pad, dtype=dtype)
+        self.register_buffer("inv_freq", inv_freq.double().to(torch.get_default_device()), persistent=False)
+        self.attn = Attention(heads, self.dim_pad, scale, kv_heads, cache_idx, sliding_window=window)
+
+    def slots(self) -> dict:
+        """Tensor name -> (memory it is copied to, its shape in a checkpoint)."""
+        def heads(name, n, size, pad):
+            return self.proj.rows(name).view(n, pad, self.width)[:, :size], (n * size, self.width)
+
+        out = {"q": heads("q", self.heads, self.dim, self.dim_pad), "q.norm": self.q_norm.data[: self.dim],
+               "o": (self.out_proj.data.view(self.width, self.heads, self.vdim_pad)[..., : self.vdim],
+                     (self.width, self.heads * self.vdim))}
+        if self.own_kv:
+            out.update({"k": heads("k", self.kv_heads, self.dim, self.dim_pad), "k.norm": self.k_norm.data[: self.dim],
+                        "v": heads("v", self.kv_heads, self.vdim, self.vdim_pad)})
+        return out
+
+    def cache_elems_per_token(self) -> int:
+        return self.kv_heads * (self.dim_pad + self.vdim_pad) if self.own_kv else 0
+
+    def allocate_kv_cache(self, num_blocks: int, block_size: int, device):
+        return (PagedGQABackend.allocate_pages(num_blocks, block_size, self.kv_heads, self.dim_pad, self.vdim_pad,
+                                               self.q_norm.dtype, device), None)
+
+    def forward(self, positions: torch.Tensor, h: torch.Tensor) -> torch.Tensor:
+        ctx = get_forward_context()
+        md = ctx.attn_metadata
+        cache = ctx.kv_caches[self.attn.layer_idx][0]
+        kv = PagedGQABackend.views(cache, md.block_size, self.kv_heads, self.dim_pad, self.vdim_pad)
+        q = ops.head_norm_rope(self.proj(h), self.offsets, self.q_norm, self.k_norm, self.heads, self.dim, self.inv_freq,
+                               positions, kv if self.own_kv else None, md.slot_mapping, self.eps)
+        o = self.attn.attend(q, md, kv)
+        return ops.gemm(o.view(h.shape[0], self.heads * self.vdim_pad), self.out_proj)

@@ -14,6 +14,9 @@ Weights: ``w13 [E_local, 2I, H]`` with gate/up rows interleaved (row 2j = gate_j
 ``w2 [E_local, H, I]``.  Experts without a gate (``gated=False``) hold ``w13 [E_local, I, H]`` and apply their activation
 in the same epilogue.
 
+Identity experts (``num_identity``): the router's last outputs name experts that hand their input through.  They have no
+weights and no rows; the pairs routed to them add ``w_k * x`` where the rows are combined.
+
 Expert parallelism: experts are sharded over the EP group (``E_local = E / ep``).
 
 * One replica (``data_parallel_size == 1``): EP group = TP group.  Tokens are replicated across its ranks (SPMD,
@@ -44,6 +47,7 @@ import torch.nn as nn
 from .. import _custom_ops as ops
 from .. import envs
 from ..ops import reference as ref
+from ..ops.residual_norm import ExpertRows
 from ..parallel import state as ps
 from .linear import ReplicatedLinear
 
@@ -52,17 +56,27 @@ BLOCK_M = 128
 
 def fused_experts(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_weights: torch.Tensor,
                   topk_ids: torch.Tensor, num_local_experts: int, expert_map: Optional[torch.Tensor] = None,
-                  shared_out: Optional[torch.Tensor] = None, epi: int = ops.EPI_CODES["silu_gate"]) -> torch.Tensor:
+                  shared_out: Optional[torch.Tensor] = None, epi: int = ops.EPI_CODES["silu_gate"],
+                  identity_from: Optional[int] = None) -> torch.Tensor:
     """Expert MLPs for the pairs routed to this rank's experts; returns ``[T, H]`` (partial sum
-    when ``expert_map`` drops pairs owned by other ranks)."""
-    T, H = x.shape
+    when ``expert_map`` drops pairs owned by other ranks).  Pairs with ids from ``identity_from`` on hand ``x`` through."""
+    return expert_rows(x, w13, w2, topk_weights, topk_ids, num_local_experts, expert_map, shared_out, epi,
+                       identity_from).combined()
+
+
+def expert_rows(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_weights: torch.Tensor, topk_ids: torch.Tensor,
+                num_local_experts: int, expert_map: Optional[torch.Tensor] = None, shared_out: Optional[torch.Tensor] = None,
+                epi: int = ops.EPI_CODES["silu_gate"], identity_from: Optional[int] = None) -> ExpertRows:
+    """The experts' output rows before they are combined."""
     topk = topk_ids.shape[1]
     sorted_ids, block_expert, total, inv = ops.moe_align_block_size(topk_ids, BLOCK_M, num_local_experts,
                                                                     expert_map, want_inverse=True)
     a = ops.moe_gather(x, sorted_ids, total, topk)
     h = ops.gemm_grouped(a, w13, block_expert, total, epi=epi)
     y = ops.gemm_grouped(h, w2, block_expert, total, epi=0)
-    return ops.moe_combine(y, topk_weights, inv, T, shared_out)
+    ident = identity_from is not None
+    return ExpertRows(y, topk_weights.contiguous(), inv, topk_ids if ident else None, x if ident else None, identity_from or 0,
+                      shared_out)
 
 
 class FusedMoE(nn.Module):
@@ -71,8 +85,10 @@ class FusedMoE(nn.Module):
                  use_grouped_topk: bool = False, num_expert_group: int = 1, topk_group: int = 1,
                  routed_scaling_factor: float = 1.0, e_score_correction_bias: bool = False,
                  reduce_results: bool = True, quant_method=None, prefix: str = "",
-                 gated: bool = True, activation: str = "silu"):
+                 gated: bool = True, activation: str = "silu", num_identity: int = 0):
         super().__init__()
+        assert num_identity == 0 or quant_method is None, "identity experts beside unquantised ones"
+        self.num_identity = num_identity          # router outputs past the experts that hand the input through
         # gated: SiLU(gate) * up over interleaved rows; otherwise one up projection through `activation`
         assert not gated or activation == "silu", "gated experts use the SiLU gate"
         assert gated or quant_method is None, "quantised experts are gated"
@@ -104,10 +120,11 @@ class FusedMoE(nn.Module):
                                            requires_grad=False)
             self.w2_weight = nn.Parameter(torch.empty(self.num_local, hidden_size, intermediate_size, dtype=dtype),
                                           requires_grad=False)
-        self.e_score_correction_bias = (nn.Parameter(torch.zeros(num_experts, dtype=torch.float32), requires_grad=False)
+        assert num_identity == 0 or not (self.eplb or self.dp > 1), "identity experts: one replica, no load balancing"
+        self.e_score_correction_bias = (nn.Parameter(torch.zeros(num_experts + num_identity, dtype=torch.float32), requires_grad=False)
                                         if e_score_correction_bias else None)
         if self.ep > 1:
-            emap = torch.full((self.num_physical,), -1, dtype=torch.int32)
+            emap = torch.full((self.num_physical + num_identity,), -1, dtype=torch.int32)
             lo = self.ep_rank * self.num_local
             emap[lo: lo + self.num_local] = torch.arange(self.num_local, dtype=torch.int32)
             self.register_buffer("expert_map", emap, persistent=False)
@@ -292,9 +309,23 @@ class FusedMoE(nn.Module):
             return False
         if self.dp > 1:
             return True
-        if self._sp_config:
+        if self._sp_config and self.num_identity == 0:
             return True
-        return self._nvlink_exchange(x)
+        return self._nvlink_exchange(x) and self.num_identity == 0
+
+    def identity_from(self) -> Optional[int]:
+        """First identity expert id, where this rank adds their contribution (one rank of those that sum)."""
+        return self.num_experts if self.num_identity and self.ep_rank == 0 else None
+
+    def forward_rows(self, x: torch.Tensor, router_logits: torch.Tensor, shared_out: Optional[torch.Tensor] = None):
+        """Like ``forward`` for a consumer that combines the rows itself (``ops/residual_norm.py``): the experts' rows, or the
+        combined output where the layer needs more than one pass or rank."""
+        chunk = int(envs.B200_FUSED_MOE_CHUNK_SIZE)
+        if self.quant_method is not None or self.ep > 1 or self.dp > 1 or (0 < chunk < x.shape[0]):
+            return self.forward(x, router_logits, shared_out)
+        w, ids = self.route(router_logits)
+        return expert_rows(x, self.w13_weight, self.w2_weight, w, ids, self.num_local, self.expert_map, shared_out, self.epi,
+                           self.identity_from())
 
     def forward_reduced(self, x: torch.Tensor, router_logits: torch.Tensor,
                         shared_out: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -318,7 +349,8 @@ class FusedMoE(nn.Module):
         def experts(xs, ws, idss, shared):
             if self.quant_method is not None:
                 return self.quant_method.apply(self, xs, ws, idss, shared)
-            return fused_experts(xs, self.w13_weight, self.w2_weight, ws, idss, self.num_local, self.expert_map, shared, self.epi)
+            return fused_experts(xs, self.w13_weight, self.w2_weight, ws, idss, self.num_local, self.expert_map, shared, self.epi,
+                                 self.identity_from())
 
         chunk = int(envs.B200_FUSED_MOE_CHUNK_SIZE)
         T = x.shape[0]

@@ -53,6 +53,7 @@ _MODELS: dict[str, tuple[str, str]] = {
     "InternVLChatModel": ("internvl", "InternVLChatModel"),
     "InternS1ForConditionalGeneration": ("internvl", "InternVLForConditionalGeneration"),    # the same graph, other decoder
     "Naguzen": ("naguzen", "NaguzenForCausalLM"),
+    "Pupalorn": ("pupalorn", "PupalornForCausalLM"),
     "MambaForCausalLM": ("mamba", "MambaForCausalLM"),
     "Qwen3NextForCausalLM": ("qwen3_next", "Qwen3NextForCausalLM"),
     "Glm4MoeForCausalLM": ("moe_family", "Glm4MoeForCausalLM"),

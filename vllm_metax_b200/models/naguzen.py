@@ -23,11 +23,12 @@ import torch.nn.functional as F
 
 from .. import _custom_ops as ops
 from ..config import ModelConfig
+from ..engine.loader import copy_to_slots, safetensors_shapes
 from ..layers.basic import ParallelLMHead, VocabParallelEmbedding
 from ..layers.fused_moe import FusedMoE
 from ..layers.latent_attention import LatentAttention, LatentCache
 from ..layers.recurrent import GatedLinearAttention, InputConv, RGLRUMixer, _param
-from ..ops.residual_conv import residual_norm
+from ..ops.residual_norm import residual_norm
 from ..parallel import state as ps
 
 
@@ -146,7 +147,7 @@ class NaguzenLayer(nn.Module):
 
 class NaguzenForCausalLM(nn.Module):
     supports_prefix_caching = False        # a cached prefix has latent rows but no recurrent state to resume from
-    native_units = "core"
+    native_units = "hybrid"
 
     def __init__(self, cfg: ModelConfig):
         super().__init__()
@@ -219,18 +220,7 @@ class NaguzenForCausalLM(nn.Module):
         return out
 
     def load_weights(self, weights: Iterable[tuple[str, torch.Tensor]]) -> set[str]:
-        slots = self.slots()
-        loaded: set[str] = set()
-        for name, w in weights:
-            dst = slots.get(name)
-            if dst is None:
-                raise ValueError(f"unexpected tensor {name!r} in the checkpoint")
-            if w.numel() != dst.numel() or (w.dim() > 1 and dst.dim() > 1 and w.shape != dst.shape):
-                raise ValueError(f"tensor {name!r}: shape {tuple(w.shape)} does not fit {tuple(dst.shape)}")
-            dst.copy_(w.reshape(dst.shape).to(dst.dtype))
-            loaded.add(name)
-        if not self._complete and len(loaded) < len(slots):
-            raise ValueError(f"tensors missing from the checkpoint: {sorted(set(slots) - loaded)[:8]}")
+        loaded = copy_to_slots(self.slots(), weights, complete=not self._complete)
         self._complete = True                  # later calls may bring a subset (weight updates)
         self.finalize_weights()
         return loaded
@@ -242,7 +232,5 @@ def decay_ranks(cfg: ModelConfig) -> dict[int, int]:
     gla = [i for i, l in enumerate(cfg.hf_config["layers"]) if l["type"] == "gla"]
     if not gla or not cfg.model_path:
         return {}
-    from ..engine.loader import safetensors_shapes
-
     shapes = safetensors_shapes(cfg.model_path)
     return {i: shapes[f"l{i}.mix.a1"][0] for i in gla}

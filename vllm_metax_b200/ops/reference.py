@@ -53,6 +53,15 @@ def gemma_rms_norm(x, weight, eps):
     return (xf * torch.rsqrt(var + eps) * (1.0 + weight.float())).to(x.dtype)
 
 
+def head_rms_norm(x, weight, dim: int, eps: float, one_plus: bool = False):
+    """RMS norm of every head of ``x [T, H, width]`` whose first ``dim`` entries are real (zeros behind), fp32."""
+    xf = x.float()
+    if weight is None:
+        return xf
+    inv = torch.rsqrt(xf.square().sum(-1, keepdim=True) / dim + eps)
+    return xf * inv * (weight.float() + (1.0 if one_plus else 0.0))
+
+
 def rms_norm_gated(x, gate, weight, eps):
     """RMSNorm(x) * silu(gate) (Mamba2 / GDN style gated norm)."""
     return (rms_norm(x, weight, eps).float() * F.silu(gate.float())).to(x.dtype)
@@ -63,12 +72,8 @@ def layer_norm(x, weight, bias, eps):
 
 
 # --------------------------------------------------------------------------- rope
-def build_rope_cache(rot_dim: int, max_pos: int, base: float, dtype=torch.float32,
-                     scaling: Optional[dict] = None) -> torch.Tensor:
-    """cos/sin table ``[max_pos, rot_dim]`` = ``[cos(rot/2) | sin(rot/2)]``.
-
-    ``scaling`` supports ``{"type": "linear"|"llama3"|"yarn", ...}``.
-    """
+def rope_frequencies(rot_dim: int, base: float, scaling: Optional[dict] = None):
+    """``(inv_freq [rot_dim / 2] fp64, scale of cos and sin)``; ``scaling`` as in :func:`build_rope_cache`."""
     inv_freq = 1.0 / (base ** (torch.arange(0, rot_dim, 2, dtype=torch.float64) / rot_dim))
     mscale = 1.0
     if scaling:
@@ -110,6 +115,16 @@ def build_rope_cache(rot_dim: int, max_pos: int, base: float, dtype=torch.float3
                 mscale = get_mscale(factor, ms) / get_mscale(factor, ms_all) if ms_all else get_mscale(factor, ms)
             else:
                 mscale = get_mscale(factor, 1.0)
+    return inv_freq, mscale
+
+
+def build_rope_cache(rot_dim: int, max_pos: int, base: float, dtype=torch.float32,
+                     scaling: Optional[dict] = None) -> torch.Tensor:
+    """cos/sin table ``[max_pos, rot_dim]`` = ``[cos(rot/2) | sin(rot/2)]``.
+
+    ``scaling`` supports ``{"type": "linear"|"llama3"|"yarn", ...}``.
+    """
+    inv_freq, mscale = rope_frequencies(rot_dim, base, scaling)
     t_pos = torch.arange(max_pos, dtype=torch.float64)
     freqs = torch.outer(t_pos, inv_freq)
     return torch.cat([freqs.cos() * mscale, freqs.sin() * mscale], dim=-1).to(dtype)
@@ -332,15 +347,18 @@ def epilogue_activation(y: torch.Tensor, act: str, params: Optional[torch.Tensor
         return torch.nn.functional.gelu(y, approximate="tanh")
     if act == "decay":
         return torch.exp(torch.nn.functional.logsigmoid(y) * params.float()[0])
+    if act == "relu2":
+        return torch.relu(y).square()
     a, b = params.float()
     return torch.where(y > 0, a * y * y, b * (torch.expm1(y.clamp(max=0)) - y)) + 0.5 * y
 
 
 def rotate_half(x: torch.Tensor, inv_freq: torch.Tensor, positions: torch.Tensor) -> torch.Tensor:
-    """Rotation of the first ``2 * len(inv_freq)`` entries of ``x [T, H, D]``, pairs (i, i + half), angles in fp32."""
+    """Rotation of the first ``2 * len(inv_freq)`` entries of ``x [T, H, D]``, pairs (i, i + half), angles in the type of
+    ``inv_freq``."""
     half = inv_freq.numel()
-    a = positions[: x.shape[0]].float()[:, None] * inv_freq[None]
-    c, s = torch.cos(a)[:, None], torch.sin(a)[:, None]
+    a = positions[: x.shape[0]].to(inv_freq.dtype)[:, None] * inv_freq[None]
+    c, s = torch.cos(a).float()[:, None], torch.sin(a).float()[:, None]
     u, v = x[..., :half].float(), x[..., half: 2 * half].float()
     return torch.cat([(u * c - v * s).to(x.dtype), (v * c + u * s).to(x.dtype), x[..., 2 * half:]], -1)
 
@@ -415,7 +433,10 @@ def reshape_and_cache(key, value, kv_cache, slot_mapping, kv_scales=None, k_scal
 
 
 def gather_paged_kv(kv_cache, block_table_row, kv_len, kv_scales=None, k_scale=1.0, v_scale=1.0):
-    """Contiguous fp32 ``(K, V) [kv_len, Hkv, D]`` of one sequence."""
+    """Contiguous fp32 ``(K, V) [kv_len, Hkv, D]`` of one sequence (``kv_cache``: 5-D, or a pair of 4-D views)."""
+    if isinstance(kv_cache, tuple):
+        blocks = block_table_row[: -(-kv_len // kv_cache[0].shape[1])].long()
+        return tuple(c[blocks].float().flatten(0, 1)[:kv_len] for c in kv_cache)
     nb, _, bs, H, D = kv_cache.shape
     nblk = (kv_len + bs - 1) // bs
     blocks = block_table_row[:nblk].long()
@@ -501,7 +522,8 @@ def paged_attention(q, kv_cache, block_table, seq_lens, query_start_loc, scale, 
     at vllm_metax/v1/attention/backends/flash_attn.py:1302-1355.
     """
     T, Hq, D = q.shape
-    out = torch.zeros(T, Hq, kv_cache.shape[-1], dtype=torch.float32, device=q.device)
+    dv = kv_cache[1].shape[-1] if isinstance(kv_cache, tuple) else kv_cache.shape[-1]
+    out = torch.zeros(T, Hq, dv, dtype=torch.float32, device=q.device)
     lse_all = torch.full((Hq, T), float("-inf"), dtype=torch.float32, device=q.device)
     B = seq_lens.shape[0]
     qsl = query_start_loc.tolist()

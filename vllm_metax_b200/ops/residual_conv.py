@@ -1,5 +1,5 @@
 """Sublayer boundary of post-norm decoders with an fp32 residual stream and a short input convolution
-(``csrc/residual_conv.cu``), and the last boundary in front of the LM head.
+(``csrc/residual_conv.cu``).
 
     x' = x + gain * y / sqrt(mean(y^2) + eps)                    fp32
     h  = x' + sum_j w[:, j] * x'[t - (K-1) + j]                  the next sublayer's input, in y's dtype
@@ -14,14 +14,11 @@ from typing import Optional
 
 import torch
 
-
-def _normed(y: torch.Tensor, gain: torch.Tensor, eps: float) -> torch.Tensor:
-    yf = y.float()
-    return yf * torch.rsqrt(yf.pow(2).mean(-1, keepdim=True) + eps) * gain.float()
+from .residual_norm import normed
 
 
 def residual_conv_ref(y, x, gain, w, eps, carry, query_start_loc, state_indices, has_initial_state):
-    xn = y.float() if x is None else x + _normed(y, gain, eps)
+    xn = y.float() if x is None else x + normed(y, gain, eps)
     T, D = xn.shape
     K = w.shape[1]
     h = torch.empty_like(xn)
@@ -54,16 +51,3 @@ def residual_conv(y: torch.Tensor, x: Optional[torch.Tensor], gain: Optional[tor
     torch.ops.b200.residual_conv(x_out, h, y, x, None if x is None else gain, w, carry if w.shape[1] > 1 else None,
                                  query_start_loc, state_indices, has_initial_state, eps)
     return x_out, h
-
-
-def residual_norm(y: torch.Tensor, x: Optional[torch.Tensor], gain: Optional[torch.Tensor], gain_out: torch.Tensor,
-                  eps: float) -> torch.Tensor:
-    """``norm(x + norm(y))`` with gains ``gain_out`` and ``gain`` - the hidden states the LM head reads."""
-    from .. import _custom_ops as ops
-
-    if not ops._use_cuda(y):
-        xn = y.float() if x is None else x + _normed(y, gain, eps)
-        return _normed(xn, gain_out, eps).to(y.dtype)
-    out = torch.empty_like(y)
-    torch.ops.b200.residual_norm(out, y, x, None if x is None else gain, gain_out, eps)
-    return out

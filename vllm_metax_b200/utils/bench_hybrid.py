@@ -139,7 +139,8 @@ def kernel_rows(size: str = "w2048", only: str = "") -> list:
     """One row per new kernel and phase: time, roofline fraction, and the same for the like kernel of the closest model."""
     from ..ops.gdn import causal_conv1d, gated_delta_rule
     from ..ops.gla import gated_linear_attention
-    from ..ops.residual_conv import residual_conv, residual_norm
+    from ..ops.residual_conv import residual_conv
+    from ..ops.residual_norm import residual_norm
     from ..ops.rglru import rglru
 
     s = SIZES[size]
