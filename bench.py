@@ -17,6 +17,8 @@ iterations).  Two measurements per run:
 `python bench.py --gpus N --steps K --warmup W`; for N > 1 launch under torchrun.
 `--hybrid` instead prints one JSON line with the layer-list hybrid (Naguzen) beside its closest models at equal sizes:
 prefill and decode throughput, and every kernel of it against its roofline (utils/bench_hybrid.py; one GPU).
+`--shared-kv` does the same for the decoder with windowed, cross-layer-shared attention and identity experts (Pupalorn)
+beside Qwen3-MoE (utils/bench_shared_kv.py).
 `--impl reference` reports that the reference cannot be installed on this machine.
 """
 from __future__ import annotations
@@ -117,14 +119,17 @@ class ClockSampler:
                 "reasons": sorted(reasons), "samples": len(sm)}
 
 
-def hybrid(args) -> None:
-    from vllm_metax_b200.utils.bench_hybrid import SIZES, kernel_rows, model_rows
+def layer_list_bench(args) -> None:
+    if args.shared_kv:
+        from vllm_metax_b200.utils.bench_shared_kv import SIZES, TITLE, kernel_rows, model_rows
+    else:
+        from vllm_metax_b200.utils.bench_hybrid import SIZES, TITLE, kernel_rows, model_rows
 
     sampler = ClockSampler(0)
     sampler.start()
     rows = model_rows(steps=max(1, args.steps), warmup=max(3, args.warmup))
     kernels = [r for size in SIZES for r in kernel_rows(size)]
-    print(json.dumps({"metric": "hybrid decoder beside its closest models (device-timed, random weights)", "n_gpus": 1,
+    print(json.dumps({"metric": f"{TITLE} (device-timed, random weights)", "n_gpus": 1,
                       "steps": args.steps, "warmup": max(3, args.warmup), "dtype": "bf16", "data": "synthetic",
                       "models": rows, "kernels": kernels, "clocks": sampler.stop()}))
 
@@ -147,9 +152,11 @@ def main() -> None:
                          "workload driver is tensor-parallel only")
     ap.add_argument("--hybrid", action="store_true",
                     help="hybrid decoder (Naguzen) beside its closest models: throughput and kernel rooflines, one GPU")
+    ap.add_argument("--shared-kv", action="store_true",
+                    help="decoder with cross-layer-shared keys and values (Pupalorn) beside Qwen3-MoE, one GPU")
     args = ap.parse_args()
-    if args.hybrid:
-        return hybrid(args)
+    if args.hybrid or args.shared_kv:
+        return layer_list_bench(args)
     conf = CONFIGS[args.config]
     MODEL = conf["model"]
     args.num_reqs = args.num_reqs or conf["workload"][0]

@@ -167,8 +167,9 @@ def tensor_shapes(cfg):
     return out
 
 
-def random_weights(cfg, seed=0):
-    """bf16 tensors under the checkpoint's names; gains that are stored around zero stay there, others around one."""
+def random_weights(cfg, seed=0, decisive=False):
+    """bf16 tensors under the checkpoint's names; gains that are stored around zero stay there, others around one.
+    ``decisive``: corrections so far apart that they alone choose the experts."""
     g = torch.Generator().manual_seed(seed)
     out = {}
     for name, shape in tensor_shapes(cfg).items():
@@ -176,6 +177,8 @@ def random_weights(cfg, seed=0):
         leaf = name.split(".", 1)[-1]
         if leaf.endswith((".q.norm", ".k.norm")) or leaf in ("ls1", "ls2"):
             t = 1.0 + 0.3 * t
+        elif decisive and leaf.endswith("correction"):
+            t = 2.0 * torch.randperm(shape[0], generator=g)
         elif len(shape) == 1:
             t = (0.05 if leaf.endswith("correction") else 0.3) * t
         elif name != "embed":

@@ -655,6 +655,8 @@ class LLM:
 
         runner.execute = execute
         use_graphs, runner.use_graphs = runner.use_graphs, False      # every step must expose its hidden states
+        pool = self.engine.kv.pool                                    # ... and every token must be computed
+        prefix, pool.enable_prefix_caching = pool.enable_prefix_caching, False
         try:
             while any(r in self.engine.requests for r in rid_to_idx):
                 for r in self.engine.step():
@@ -662,6 +664,7 @@ class LLM:
                         self.foreign_finished.append(r)       # finished during these steps: handed back to it
         finally:
             runner.execute, runner.keep_hidden, runner.use_graphs = orig, prev_keep, use_graphs
+            pool.enable_prefix_caching = prefix
 
     def embed(self, prompts: Union[str, Sequence], pooling: str = "last", normalize: bool = True) -> torch.Tensor:
         """Sentence embeddings ``[n, hidden]`` (fp32, on CPU): the final hidden state of the last prompt token

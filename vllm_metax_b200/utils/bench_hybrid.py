@@ -17,6 +17,7 @@ import torch
 from .. import _custom_ops as ops
 from ..config import ModelConfig
 
+TITLE = "hybrid decoder beside its closest models"
 SIZES = {
     # width, heads, experts, top, expert ff (not gated), shared ff, dense ff
     "w2048": dict(width=2048, heads=16, experts=64, top=8, ff=768, shared=768, dense=8192),
@@ -69,14 +70,20 @@ def deepseek_config(s: dict, layers: int = 8) -> ModelConfig:
         norm_topk_prob=False, routed_scaling_factor=1.5)
 
 
-def model_rows(steps: int = 3, warmup: int = 2, sizes=("w2048", "w4096"), batches=((8, 1024), (64, 1024), (1, 8192))) -> list:
+MODELS = {"naguzen": naguzen_config, "qwen3_next": qwen3_next_config, "deepseek_v3": deepseek_config}
+
+
+def model_rows(steps: int = 3, warmup: int = 2, sizes=("w2048", "w4096"), batches=((8, 1024), (64, 1024), (1, 8192)),
+               models=None, table=None) -> list:
+    """``models``: label -> config of one entry of ``table`` (sizes by name)."""
     from ..engine.llm import LLM
     from ..engine.static_workload import StaticWorkload
 
     rows = []
     for name in sizes:
-        s = SIZES[name]
-        for label, cfg in (("naguzen", naguzen_config(s)), ("qwen3_next", qwen3_next_config(s)), ("deepseek_v3", deepseek_config(s))):
+        s = (table or SIZES)[name]
+        for label, make in (models or MODELS).items():
+            cfg = make(s)
             top_n = max(n for n, _ in batches)
             blocks = sum(-(-(p + 48) // 64) * n for n, p in batches) + 8
             llm = LLM(cfg, device="cuda", block_size=64, max_model_len=max(p for _, p in batches) + 128, max_num_seqs=top_n,
