@@ -97,10 +97,10 @@ def test_head_norm_rope(device, dt, H, G, dim, vdim, rot):
     pos = torch.tensor([0, 1, 2, 63, 64, 1000, 4097, 100000, 5])
     slots = torch.tensor([16, 17, 3, 79, 0, -1, 40, 41, 33])
     freqs = O.frequencies(rot, 9000.0)
-    inv = torch.tensor(freqs, dtype=torch.float64, device=device)
+    angles = ops.rope_angles(pos.to(device), torch.tensor(freqs, dtype=torch.float64, device=device), T)
     cache = torch.full_like(PagedGQABackend.allocate_pages(blocks, bs, G, dp, vp, dt, device), 7.0)
     kc, vc = PagedGQABackend.views(cache, bs, G, dp, vp)
-    got = ops.head_norm_rope(qkv, off, pad(wq, dp).to(device), pad(wk, dp).to(device), H, dim, inv, pos.to(device), (kc, vc),
+    got = ops.head_norm_rope(qkv, off, pad(wq, dp).to(device), pad(wk, dp).to(device), H, dim, angles, (kc, vc),
                              slots.to(device), eps)
     norm = lambda x, w: O.rotate(O.unit_rms(x.double(), eps) * w.double(), pos, rot, freqs)
     close(got[..., :dim], norm(q, wq), dt)
@@ -114,8 +114,8 @@ def test_head_norm_rope(device, dt, H, G, dim, vdim, rot):
     for s in range(blocks * bs):
         if s not in written:
             assert bool((kc[s // bs, s % bs] == 7).all()) and bool((vc[s // bs, s % bs] == 7).all())
-    only = ops.head_norm_rope(qkv[:, : H * dp].contiguous(), (0, 0, 0), pad(wq, dp).to(device), None, H, dim, inv,
-                              pos.to(device), None, slots.to(device), eps)
+    only = ops.head_norm_rope(qkv[:, : H * dp].contiguous(), (0, 0, 0), pad(wq, dp).to(device), None, H, dim, angles,
+                              None, slots.to(device), eps)
     assert torch.equal(only, got)
 
 
@@ -237,7 +237,7 @@ def test_identity_experts(device, dt, E, I, top, W, ff, T):
         layer.weight_loader(layer.w2_weight, w[f"x.e{e}.down"], e, "w2")
     layer.weight_loader(layer.e_score_correction_bias, w["x.correction"].float())
     hd = h.to(device)
-    logits = ops.gemm(hd, w["x.router"].to(device), out_dtype=torch.float32)
+    logits = ops.router_logits(hd, w["x.router"].to(device))
     close(layer(hd, logits), want, dt, 2.0)
     rows = layer.forward_rows(hd, logits)
     assert isinstance(rows, ExpertRows)

@@ -617,6 +617,13 @@ def embedding(table, ids, out=None, vocab_start: int = 0):
 
 
 # --------------------------------------------------------------------------- MoE routing / shuffling
+def router_logits(x, gate):
+    """fp32 ``x @ gate^T`` whose rows start on 16 bytes for any number of experts (the tensor-core products want that)."""
+    n = gate.shape[0]
+    out = torch.empty(x.shape[0], -(-n // 8) * 8, dtype=torch.float32, device=x.device)[:, :n] if x.is_cuda else None
+    return gemm(x, gate, out=out, out_dtype=torch.float32)
+
+
 _GATING_MODE = {"softmax": 0, "sigmoid": 1, "sqrtsoftplus": 2}
 
 
@@ -627,7 +634,7 @@ def topk_gating(gating, topk: int, renormalize: bool, scoring: str = "softmax", 
         T = gating.shape[0]
         w = torch.empty(T, topk, dtype=torch.float32, device=gating.device)
         ids = torch.empty(T, topk, dtype=torch.int32, device=gating.device)
-        torch.ops.b200.topk_gating(w, ids, gating.contiguous(), bias, _GATING_MODE[scoring], renormalize, scale)
+        torch.ops.b200.topk_gating(w, ids, gating if gating.stride(1) == 1 else gating.contiguous(), bias, _GATING_MODE[scoring], renormalize, scale)
         return w, ids
     if scoring == "softmax":
         w, ids = ref.topk_softmax(gating, topk, renormalize, bias)
@@ -976,23 +983,33 @@ def mla_decode(q, mla_cache, block_table, seq_lens, scale, *, query_start_loc=No
     return res
 
 
-def head_norm_rope(qkv, offsets, q_weight, k_weight, heads: int, dim: int, inv_freq, positions, kv_cache, slot_mapping,
-                   eps: float, one_plus: bool = False):
+def rope_angles(positions, inv_freq, tokens: int):
+    """Cosines and sines ``[tokens, 2, len(inv_freq)]`` (fp32) of ``position * inv_freq`` (fp64, whole turns taken off)."""
+    if _use_cuda(inv_freq):
+        out = torch.empty(tokens, 2, inv_freq.numel(), dtype=torch.float32, device=inv_freq.device)
+        torch.ops.b200.rope_angles(out, positions, inv_freq)
+        return out
+    a = positions[:tokens, None].double() * inv_freq[None]
+    return torch.stack([torch.cos(a), torch.sin(a)], 1).float()
+
+
+def head_norm_rope(qkv, offsets, q_weight, k_weight, heads: int, dim: int, angles, kv_cache, slot_mapping, eps: float,
+                   one_plus: bool = False):
     """Epilogue of a merged q | k | v product whose parts start at the columns ``offsets``: per-head RMS norm (``one_plus``:
     weights stored around zero) and rotation of queries and keys, keys and values written to the paged cache
     (``kv_cache``: 5-D or a pair of ``kv_views``) at ``slot_mapping`` (-1: nowhere).  ``kv_cache=None``: the row holds queries
-    only.  Heads are ``len(weight)`` wide, of which ``dim`` are real; ``inv_freq`` is fp64.  Returns ``q [T, heads, width]``."""
+    only.  Heads are ``len(weight)`` wide, of which ``dim`` are real; ``angles`` as ``rope_angles`` returns them.  Returns
+    ``q [T, heads, width]``."""
     T, width = qkv.shape[0], q_weight.numel()
     k, v = kv_views(kv_cache) if kv_cache is not None else (None, None)
     if _use_cuda(qkv):
         q = torch.empty(T, heads, width, dtype=qkv.dtype, device=qkv.device)
-        torch.ops.b200.head_norm_rope(q, qkv, *offsets, k, v, q_weight, k_weight, dim, inv_freq, positions, slot_mapping,
-                                      eps, one_plus)
+        torch.ops.b200.head_norm_rope(q, qkv, *offsets, k, v, q_weight, k_weight, dim, angles, slot_mapping, eps, one_plus)
         return q
 
     def part(at, n, w):
         x = ref.head_rms_norm(qkv[:, at: at + n * width].reshape(T, n, width), w, dim, eps, one_plus)
-        return ref.rotate_half(x, inv_freq, positions).to(qkv.dtype)
+        return ref.rotate_half_by(x, angles).to(qkv.dtype)
 
     q = part(offsets[0], heads, q_weight)
     if k is not None:

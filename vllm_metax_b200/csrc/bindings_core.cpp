@@ -146,11 +146,11 @@ void advance_step(Tensor& input_ids, Tensor& positions, Tensor& seq_lens, Tensor
 // ------------------------------------------------------------------ MoE
 void topk_gating(Tensor& weights, Tensor& ids, const Tensor& gating, const optional<Tensor>& bias, int64_t mode,
                  bool renorm, double scale) {
-  TORCH_CHECK(gating.dim() == 2 && gating.is_contiguous() && gating.size(1) <= 1024 && ids.size(1) <= 32);
+  TORCH_CHECK(gating.dim() == 2 && gating.stride(1) == 1 && gating.size(1) <= 1024 && ids.size(1) <= 32);
   TORCH_CHECK(weights.scalar_type() == at::kFloat && ids.scalar_type() == at::kInt);
   const c10::cuda::CUDAGuard guard(gating.device());
   b200::topk_gating(weights.data_ptr<float>(), ids.data_ptr<int>(), gating.data_ptr(), ptr<float>(bias),
-                    gating.size(0), gating.size(1), ids.size(1), mode, renorm, (float)scale, dtype_code(gating),
+                    gating.size(0), gating.size(1), gating.stride(0), ids.size(1), mode, renorm, (float)scale, dtype_code(gating),
                     cur_stream());
 }
 

@@ -85,16 +85,16 @@ void paged_attention_decode(Tensor& out, const Tensor& q, const Tensor& k_cache,
 // The epilogue of a merged q | k | v product (columns q_off, k_off, v_off); without caches: queries only.
 void head_norm_rope(Tensor& q_out, const Tensor& qkv, int64_t q_off, int64_t k_off, int64_t v_off,
                     const optional<Tensor>& k_cache, const optional<Tensor>& v_cache, const optional<Tensor>& q_w,
-                    const optional<Tensor>& k_w, int64_t dim, const Tensor& inv_freq, const Tensor& positions,
-                    const Tensor& slot_mapping, double eps, bool one_plus) {
-  on_device_of(qkv, {&q_out, &inv_freq, &positions, &slot_mapping}, {&k_cache, &v_cache, &q_w, &k_w});
+                    const optional<Tensor>& k_w, int64_t dim, const Tensor& angles, const Tensor& slot_mapping, double eps,
+                    bool one_plus) {
+  on_device_of(qkv, {&q_out, &angles, &slot_mapping}, {&k_cache, &v_cache, &q_w, &k_w});
   const int64_t T = qkv.size(0), H = q_out.size(1), DP = q_out.size(2);
   const auto dt = qkv.scalar_type();
   TORCH_CHECK(qkv.dim() == 2 && qkv.stride(1) == 1 && q_out.dim() == 3 && q_out.is_contiguous() && q_out.size(0) == T &&
               q_out.scalar_type() == dt && dim <= DP && q_off + H * DP <= qkv.size(1));
-  TORCH_CHECK(inv_freq.scalar_type() == at::kDouble && inv_freq.is_contiguous() && 2 * inv_freq.numel() <= dim);
-  TORCH_CHECK(positions.scalar_type() == at::kLong && positions.numel() >= T && positions.is_contiguous() &&
-              slot_mapping.scalar_type() == at::kLong && slot_mapping.numel() >= T && slot_mapping.is_contiguous());
+  TORCH_CHECK(angles.dim() == 3 && angles.size(0) == T && angles.size(1) == 2 && angles.scalar_type() == at::kFloat &&
+              angles.is_contiguous() && 2 * angles.size(2) <= dim, "angles [tokens, 2, half of the rotated entries]");
+  TORCH_CHECK(slot_mapping.scalar_type() == at::kLong && slot_mapping.numel() >= T && slot_mapping.is_contiguous());
   b200::HeadNormRopeParams p{};
   auto aligned = [](const void* a) { return reinterpret_cast<uintptr_t>(a) % 16 == 0; };
   const int64_t unit = 16 / (int64_t)qkv.element_size();
@@ -116,12 +116,23 @@ void head_norm_rope(Tensor& q_out, const Tensor& qkv, int64_t q_off, int64_t k_o
   }
   p.qkv = qkv.data_ptr(); p.row_stride = qkv.stride(0); p.q_off = q_off; p.k_off = k_off; p.v_off = v_off;
   p.q_out = q_out.data_ptr(); p.q_w = ptr(q_w); p.k_w = ptr(k_w);
-  p.inv_freq = inv_freq.data_ptr<double>(); p.positions = positions.data_ptr<int64_t>(); p.slots = slot_mapping.data_ptr<int64_t>();
-  p.tokens = T; p.heads = H; p.dim = dim; p.dim_pad = DP; p.rot = 2 * inv_freq.numel(); p.one_plus = one_plus;
+  p.angles = angles.data_ptr<float>(); p.slots = slot_mapping.data_ptr<int64_t>();
+  p.vec = p.vec && aligned(p.angles);
+  p.tokens = T; p.heads = H; p.dim = dim; p.dim_pad = DP; p.rot = 2 * (int)angles.size(2); p.one_plus = one_plus;
   p.eps = (float)eps;
   p.status = reinterpret_cast<b200::StatusWord*>(status_ptr(qkv));
   const c10::cuda::CUDAGuard guard(qkv.device());
-  TORCH_CHECK(b200::head_norm_rope(p, dtype_code(qkv), cur_stream()) == 0, "head_norm_rope: heads up to 1024, rotation up to 512 entries");
+  TORCH_CHECK(b200::head_norm_rope(p, dtype_code(qkv), cur_stream()) == 0, "head_norm_rope: heads up to 1024 wide");
+}
+
+void rope_angles(Tensor& out, const Tensor& positions, const Tensor& inv_freq) {
+  on_device_of(out, {&positions, &inv_freq});
+  TORCH_CHECK(out.dim() == 3 && out.size(1) == 2 && out.is_contiguous() && out.scalar_type() == at::kFloat);
+  TORCH_CHECK(inv_freq.scalar_type() == at::kDouble && inv_freq.is_contiguous() && inv_freq.numel() == out.size(2));
+  TORCH_CHECK(positions.scalar_type() == at::kLong && positions.is_contiguous() && positions.numel() >= out.size(0));
+  const c10::cuda::CUDAGuard guard(out.device());
+  b200::rope_angles(out.data_ptr<float>(), positions.data_ptr<int64_t>(), inv_freq.data_ptr<double>(), out.size(0),
+                    out.size(2), cur_stream());
 }
 
 }  // namespace
@@ -135,6 +146,7 @@ TORCH_LIBRARY_FRAGMENT(b200, m) {
       &paged_attention_decode);
   m.def(
       "head_norm_rope(Tensor(a!) q_out, Tensor qkv, int q_off, int k_off, int v_off, Tensor(b!)? k_cache, Tensor(c!)? v_cache, "
-      "Tensor? q_w, Tensor? k_w, int dim, Tensor inv_freq, Tensor positions, Tensor slot_mapping, float eps, bool one_plus) -> ()",
+      "Tensor? q_w, Tensor? k_w, int dim, Tensor angles, Tensor slot_mapping, float eps, bool one_plus) -> ()",
       &head_norm_rope);
+  m.def("rope_angles(Tensor(a!) out, Tensor positions, Tensor inv_freq) -> ()", &rope_angles);
 }

@@ -1,29 +1,30 @@
 // Epilogue of a merged q | k | v product, per token and head: RMS norm over the head (shared weights for all heads), rotation
 // of its first `rot` entries in pairs (i, i + rot / 2), then queries to a packed tensor and keys, together with the values,
-// to their paged cache row - one launch, one CTA per token.  Layers that read another layer's cache pass queries only.
+// to their paged cache row - one launch.  Layers that read another layer's cache pass queries only.
 //
-// Heads may be padded with zeros to a multiple of 8 (`dim_pad`); the mean runs over the `dim` real entries.  An angle is
-// position * frequency, reduced by whole turns in fp64 (one product per pair and token), so that far positions keep the
-// accuracy of near ones; everything else is fp32.
+// Heads may be padded with zeros to a multiple of 8 (`dim_pad`); the mean runs over the `dim` real entries.  Cosines and sines
+// come from a table of the step's tokens that all layers of one rotation share (`rope_angles`): an angle is position *
+// frequency, whole turns taken off in fp64, so that far positions keep the accuracy of near ones.  The rest is fp32.
 #include "ops.h"
 #include "row_vec.cuh"
 
 namespace b200 {
 namespace {
 
-constexpr int kMaxRot = 512, kThreads = 256;
+constexpr int kThreads = 256;
 
-struct Angles {
-  float c[kMaxRot / 2], s[kMaxRot / 2];
-};
-
-__device__ __forceinline__ void fill_angles(Angles& a, const HeadNormRopeParams& p, int64_t t) {
-  const double pos = (double)p.positions[t];
-  for (int i = threadIdx.x; i < p.rot / 2; i += blockDim.x) {
-    double turns = pos * p.inv_freq[i] * 0.15915494309189533577;       // angle / 2 pi
-    turns -= rint(turns);
-    sincosf((float)(turns * 6.28318530717958647693), &a.s[i], &a.c[i]);
-  }
+__global__ void rope_angles_kernel(float* __restrict__ out, const int64_t* __restrict__ positions,
+                                   const double* __restrict__ inv_freq, int64_t n, int half) {
+  const int64_t id = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (id >= n) return;
+  const int64_t t = id / half;
+  const int i = (int)(id % half);
+  double turns = (double)positions[t] * inv_freq[i] * 0.15915494309189533577;       // angle / 2 pi
+  turns -= rint(turns);
+  float s, c;
+  sincosf((float)(turns * 6.28318530717958647693), &s, &c);
+  out[(2 * t) * half + i] = c;
+  out[(2 * t + 1) * half + i] = s;
 }
 
 // Where head `item` (queries, then keys) of token t is read and written; dst is null where nothing is written.
@@ -50,7 +51,7 @@ __device__ __forceinline__ void cache_rows(const HeadNormRopeParams& p, int64_t 
   const int64_t slot = p.slots[t];
   if (slot < 0) return;
   if (slot >= p.num_slots) {
-    if (threadIdx.x == 0) report_status(p.status, kBadIndex, 140, (int)p.num_slots, (int)slot);
+    report_status(p.status, kBadIndex, 140, (int)p.num_slots, (int)slot);
     return;
   }
   const int64_t page = (slot / p.block_size) * p.page_stride, at = slot % p.block_size;
@@ -58,92 +59,84 @@ __device__ __forceinline__ void cache_rows(const HeadNormRopeParams& p, int64_t 
   v_row = page + at * p.kv_heads * p.vdim_pad;
 }
 
-template <typename T, bool VEC>
-__device__ __forceinline__ void copy_values(const HeadNormRopeParams& p, int64_t t, int64_t v_row) {
-  if (v_row < 0) return;
-  const T* src = reinterpret_cast<const T*>(p.qkv) + t * p.row_stride + p.v_off;
-  T* dst = reinterpret_cast<T*>(p.v_cache) + v_row;
-  const int n = p.kv_heads * p.vdim_pad;
-  if constexpr (VEC) {
-    constexpr int kPer = 16 / sizeof(T);
-    for (int i = threadIdx.x; i < n / kPer; i += blockDim.x)
-      reinterpret_cast<uint4*>(dst)[i] = reinterpret_cast<const uint4*>(src)[i];
-  } else {
-    for (int i = threadIdx.x; i < n; i += blockDim.x) dst[i] = src[i];
-  }
-}
-
-// Heads of up to 256 entries whose half rotation is a multiple of 8: `lanes` neighbouring lanes (a power of two) hold a head,
-// 8 entries each, and exchange rotation partners by shuffles.
+// Heads of up to 256 entries whose half rotation is a multiple of 8: `lanes` neighbouring lanes (a power of two) hold one head
+// of one token, 8 entries each, and exchange rotation partners by shuffles.  A token's items: queries, keys, then its values
+// in pieces of lanes * 8 entries.
 template <typename T>
 __global__ void __launch_bounds__(kThreads)
-head_norm_rope_vec_kernel(const HeadNormRopeParams p, int lanes) {
-  __shared__ Angles ang;
-  const int64_t t = blockIdx.x;
-  int64_t k_row, v_row;
-  cache_rows(p, t, k_row, v_row);
-  const int items = p.heads + (p.k_cache != nullptr ? p.kv_heads : 0);
-  const int lane = threadIdx.x & 31, per_warp = 32 / lanes, j = lane & (lanes - 1);
+head_norm_rope_vec_kernel(const HeadNormRopeParams p, int lanes, int value_items) {
+  const int lane = threadIdx.x & 31, j = lane & (lanes - 1);
+  const int normed = p.heads + (p.k_cache != nullptr ? p.kv_heads : 0), items = normed + value_items;
+  const int64_t id = ((int64_t)blockIdx.x * kThreads + threadIdx.x) / lanes;
+  const int64_t t = id / items;
+  const int item = (int)(id % items);
   const int c0 = j * 8, half = p.rot / 2;
-  const bool in_head = c0 < p.dim_pad;
-  const bool first = c0 < half, rotated = c0 < p.rot;
-  const int partner = (lane - j) + (first ? j + half / 8 : rotated ? j - half / 8 : j);
-  const int a0 = first ? c0 : c0 - half;
-  fill_angles(ang, p, t);
-  __syncthreads();
-  for (int base = (threadIdx.x >> 5) * per_warp; base < items; base += (blockDim.x >> 5) * per_warp) {   // warp-uniform
-    const int item = base + lane / lanes;
-    const bool live = item < items && in_head;
-    const T* src = nullptr;
-    T* dst = nullptr;
-    const T* w = nullptr;
-    float v[8] = {};
-    if (live) {
-      locate<T>(p, t, k_row, item, src, dst, w);
-      load_row<T, 8, true>(src, c0, p.dim_pad, v);
-    }
-    float ss = 0.f;
-#pragma unroll
-    for (int k = 0; k < 8; ++k) ss = fmaf(v[k], v[k], ss);
-    for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-    if (live && w != nullptr) {
-      const float inv = 1.f / sqrtf(ss / (float)p.dim + p.eps);
-      float g[8];
-      load_row<T, 8, true>(w, c0, p.dim_pad, g);
-#pragma unroll
-      for (int k = 0; k < 8; ++k) v[k] = v[k] * inv * (p.one_plus ? 1.f + g[k] : g[k]);
-    }
-    if (p.rot > 0) {
-#pragma unroll
-      for (int k = 0; k < 8; ++k) {
-        const float o = __shfl_sync(0xffffffffu, v[k], partner & 31);
-        if (rotated) {
-          const float c = ang.c[a0 + k], s = ang.s[a0 + k];
-          v[k] = first ? v[k] * c - o * s : v[k] * c + o * s;
-        }
+  const bool in_step = t < p.tokens, head = in_step && item < normed && c0 < p.dim_pad;
+  const T* src = nullptr;
+  T* dst = nullptr;
+  const T* w = nullptr;
+  float v[8] = {};
+  if (in_step && item >= p.heads) {
+    int64_t k_row, v_row;
+    cache_rows(p, t, k_row, v_row);
+    if (item >= normed) {                                    // values: copied as they are
+      const int at = ((item - normed) * lanes + j) * 8;
+      if (v_row >= 0 && at < p.kv_heads * p.vdim_pad) {
+        load_row<T, 8, true>(reinterpret_cast<const T*>(p.qkv) + t * p.row_stride + p.v_off, at, 0, v);
+        store_row<T, 8, true>(reinterpret_cast<T*>(p.v_cache) + v_row, at, 0, v);
       }
+    } else if (head) {
+      locate<T>(p, t, k_row, item, src, dst, w);
     }
-    if (live && dst != nullptr) store_row<T, 8, true>(dst, c0, p.dim_pad, v);
+  } else if (head) {
+    locate<T>(p, t, -1, item, src, dst, w);
   }
-  copy_values<T, true>(p, t, v_row);
+  const bool first = c0 < half, rotated = c0 < p.rot;
+  float c[8] = {}, s[8] = {}, g[8] = {};
+  if (head) {
+    load_row<T, 8, true>(src, c0, p.dim_pad, v);
+    if (w != nullptr) load_row<T, 8, true>(w, c0, p.dim_pad, g);
+    if (rotated) {
+      const float* a = p.angles + 2 * t * half;
+      load_row<float, 8, true>(a, first ? c0 : c0 - half, half, c);
+      load_row<float, 8, true>(a + half, first ? c0 : c0 - half, half, s);
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < 8; ++k) ss = fmaf(v[k], v[k], ss);
+  for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  if (w != nullptr) {
+    const float inv = 1.f / sqrtf(ss / (float)p.dim + p.eps);
+#pragma unroll
+    for (int k = 0; k < 8; ++k) v[k] = v[k] * inv * (p.one_plus ? 1.f + g[k] : g[k]);
+  }
+  if (p.rot > 0) {
+    const int partner = (lane - j) + (first ? j + half / 8 : rotated ? j - half / 8 : j);
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {
+      const float o = __shfl_sync(0xffffffffu, v[k], partner & 31);
+      if (rotated) v[k] = first ? v[k] * c[k] - o * s[k] : v[k] * c[k] + o * s[k];
+    }
+  }
+  if (dst != nullptr) store_row<T, 8, true>(dst, c0, p.dim_pad, v);
 }
 
-// Any sizes: a warp per head, the normed head staged in shared memory.
+// Any sizes: one CTA per token, a warp per head, the normed head staged in shared memory.
 constexpr int kMaxDim = 1024, kAnyWarps = 4;
 
 template <typename T>
 __global__ void __launch_bounds__(kAnyWarps * 32)
 head_norm_rope_kernel(const HeadNormRopeParams p) {
-  __shared__ Angles ang;
   __shared__ float stage[kAnyWarps][kMaxDim];
   const int64_t t = blockIdx.x;
   int64_t k_row, v_row;
   cache_rows(p, t, k_row, v_row);
   const int items = p.heads + (p.k_cache != nullptr ? p.kv_heads : 0);
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, half = p.rot / 2;
+  const float* cs = p.angles + 2 * t * half;
+  const float* sn = cs + half;
   float* buf = stage[warp];
-  fill_angles(ang, p, t);
-  __syncthreads();
   for (int item = warp; item < items; item += kAnyWarps) {
     const T* src;
     T* dst;
@@ -165,21 +158,27 @@ head_norm_rope_kernel(const HeadNormRopeParams p) {
     if (dst != nullptr)
       for (int i = lane; i < p.dim_pad; i += 32) {
         float f = buf[i];
-        if (i < half) f = f * ang.c[i] - buf[i + half] * ang.s[i];
-        else if (i < 2 * half) f = f * ang.c[i - half] + buf[i - half] * ang.s[i - half];
+        if (i < half) f = f * cs[i] - buf[i + half] * sn[i];
+        else if (i < 2 * half) f = f * cs[i - half] + buf[i - half] * sn[i - half];
         dst[i] = from_f<T>(f);
       }
   }
-  copy_values<T, false>(p, t, v_row);
+  if (v_row < 0) return;
+  const T* src = reinterpret_cast<const T*>(p.qkv) + t * p.row_stride + p.v_off;
+  T* dst = reinterpret_cast<T*>(p.v_cache) + v_row;
+  for (int i = threadIdx.x; i < p.kv_heads * p.vdim_pad; i += kAnyWarps * 32) dst[i] = src[i];
 }
 
 template <typename T>
 int launch(const HeadNormRopeParams& p, cudaStream_t stream) {
-  if (p.rot > kMaxRot || p.rot > p.dim || p.rot % 2 != 0 || p.dim_pad > kMaxDim) return 1;
+  if (p.rot > p.dim || p.rot % 2 != 0 || p.dim_pad > kMaxDim) return 1;
   if (p.vec && p.dim_pad <= 256 && p.rot % 16 == 0) {
     int lanes = 1;
     while (lanes * 8 < p.dim_pad) lanes *= 2;
-    head_norm_rope_vec_kernel<T><<<p.tokens, kThreads, 0, stream>>>(p, lanes);
+    const int values = p.k_cache != nullptr ? ceil_div(p.kv_heads * p.vdim_pad, lanes * 8) : 0;
+    const int items = p.heads + (p.k_cache != nullptr ? p.kv_heads : 0) + values;
+    const int64_t threads = (int64_t)p.tokens * items * lanes;
+    head_norm_rope_vec_kernel<T><<<(unsigned)((threads + kThreads - 1) / kThreads), kThreads, 0, stream>>>(p, lanes, values);
   } else {
     head_norm_rope_kernel<T><<<p.tokens, kAnyWarps * 32, 0, stream>>>(p);
   }
@@ -188,12 +187,18 @@ int launch(const HeadNormRopeParams& p, cudaStream_t stream) {
 
 }  // namespace
 
-// Returns 1 for heads wider than 1024 or more than 512 rotated entries.
+// Returns 1 for heads wider than 1024 or an odd number of rotated entries.
 int head_norm_rope(const HeadNormRopeParams& p, int dtype, cudaStream_t stream) {
   if (p.tokens <= 0) return 0;
   if (dtype == 0) return launch<__nv_bfloat16>(p, stream);
   if (dtype == 1) return launch<__half>(p, stream);
   return launch<float>(p, stream);
+}
+
+void rope_angles(float* out, const int64_t* positions, const double* inv_freq, int tokens, int half, cudaStream_t stream) {
+  const int64_t n = (int64_t)tokens * half;
+  if (n <= 0) return;
+  rope_angles_kernel<<<(unsigned)((n + kThreads - 1) / kThreads), kThreads, 0, stream>>>(out, positions, inv_freq, n, half);
 }
 
 }  // namespace b200

@@ -23,19 +23,20 @@ __device__ __forceinline__ float score_of(int mode, float x) {
   return x;                                                             // softmax handled by caller
 }
 
-// mode: 0 softmax, 1 sigmoid, 2 sqrt-softplus.  One warp per token.
-template <typename T>
+// mode: 0 softmax, 1 sigmoid, 2 sqrt-softplus.  One warp per token; PER
+// experts per lane (rows of `stride` elements).
+template <typename T, int PER>
 __global__ void topk_gating_kernel(float* __restrict__ weights, int* __restrict__ ids, const T* __restrict__ gating,
-                                   const float* __restrict__ bias, int tokens, int experts, int topk, int mode,
+                                   const float* __restrict__ bias, int tokens, int experts, int64_t stride, int topk, int mode,
                                    int renorm, float scale) {
   const int t = (blockIdx.x * blockDim.x + threadIdx.x) >> 5;
   const int lane = threadIdx.x & 31;
   if (t >= tokens) return;
-  const T* g = gating + (size_t)t * experts;
-  float sc[kMaxExpertsPerLane];   // scores of experts lane, lane+32, ...
+  const T* g = gating + t * stride;
+  float sc[PER];   // scores of experts lane, lane+32, ...
   float mx = -INFINITY;
 #pragma unroll
-  for (int j = 0; j < kMaxExpertsPerLane; ++j) {
+  for (int j = 0; j < PER; ++j) {
     const int e = lane + 32 * j;
     sc[j] = e < experts ? to_f(g[e]) : -INFINITY;
     mx = fmaxf(mx, sc[j]);
@@ -44,7 +45,7 @@ __global__ void topk_gating_kernel(float* __restrict__ weights, int* __restrict_
     mx = warp_max(mx);
     float sum = 0.f;
 #pragma unroll
-    for (int j = 0; j < kMaxExpertsPerLane; ++j) {
+    for (int j = 0; j < PER; ++j) {
       const int e = lane + 32 * j;
       sc[j] = e < experts ? __expf(sc[j] - mx) : 0.f;
       sum += sc[j];
@@ -52,18 +53,18 @@ __global__ void topk_gating_kernel(float* __restrict__ weights, int* __restrict_
     sum = warp_sum(sum);
     const float inv = 1.f / sum;
 #pragma unroll
-    for (int j = 0; j < kMaxExpertsPerLane; ++j) sc[j] *= inv;
+    for (int j = 0; j < PER; ++j) sc[j] *= inv;
   } else {
 #pragma unroll
-    for (int j = 0; j < kMaxExpertsPerLane; ++j) {
+    for (int j = 0; j < PER; ++j) {
       const int e = lane + 32 * j;
       sc[j] = e < experts ? score_of(mode, sc[j]) : 0.f;
     }
   }
   // selection value = score (+ bias); picked experts are marked by -inf in sel
-  float sel[kMaxExpertsPerLane];
+  float sel[PER];
 #pragma unroll
-  for (int j = 0; j < kMaxExpertsPerLane; ++j) {
+  for (int j = 0; j < PER; ++j) {
     const int e = lane + 32 * j;
     sel[j] = e < experts ? sc[j] + (bias ? bias[e] : 0.f) : -INFINITY;
   }
@@ -74,7 +75,7 @@ __global__ void topk_gating_kernel(float* __restrict__ weights, int* __restrict_
     float bv = -INFINITY;
     int be = 0x7fffffff;
 #pragma unroll
-    for (int j = 0; j < kMaxExpertsPerLane; ++j) {
+    for (int j = 0; j < PER; ++j) {
       const int e = lane + 32 * j;
       if (sel[j] > bv) { bv = sel[j]; be = e; }
     }
@@ -88,7 +89,7 @@ __global__ void topk_gating_kernel(float* __restrict__ weights, int* __restrict_
     float w = 0.f;
     if ((be & 31) == lane) {
 #pragma unroll
-      for (int j = 0; j < kMaxExpertsPerLane; ++j)
+      for (int j = 0; j < PER; ++j)
         if (j == (be >> 5)) { w = sc[j]; sel[j] = -INFINITY; }
     }
     w = __shfl_sync(0xffffffffu, w, be & 31);
@@ -376,14 +377,26 @@ __global__ void moe_sum_kernel(T* __restrict__ out, const T* __restrict__ in, in
 #define DISPATCH_16(dtype, CALL_BF16, CALL_F16, CALL_F32) \
   if (dtype == 0) { CALL_BF16; } else if (dtype == 1) { CALL_F16; } else { CALL_F32; }
 
-void topk_gating(float* weights, int* ids, const void* gating, const float* bias, int tokens, int experts, int topk,
-                 int mode, int renorm, float scale, int dtype, cudaStream_t stream) {
-  if (tokens <= 0) return;
+template <typename T>
+static void launch_topk(float* weights, int* ids, const T* gating, const float* bias, int tokens, int experts, int64_t stride,
+                        int topk, int mode, int renorm, float scale, cudaStream_t stream) {
   const int th = 128, blocks = ceil_div(tokens * 32, th);
+#define GATE(PER) \
+  topk_gating_kernel<T, PER><<<blocks, th, 0, stream>>>(weights, ids, gating, bias, tokens, experts, stride, topk, mode, renorm, scale)
+  if (experts <= 64) GATE(2);
+  else if (experts <= 128) GATE(4);
+  else if (experts <= 256) GATE(8);
+  else GATE(kMaxExpertsPerLane);
+#undef GATE
+}
+
+void topk_gating(float* weights, int* ids, const void* gating, const float* bias, int tokens, int experts, int64_t stride,
+                 int topk, int mode, int renorm, float scale, int dtype, cudaStream_t stream) {
+  if (tokens <= 0) return;
   DISPATCH_16(dtype,
-              (topk_gating_kernel<__nv_bfloat16><<<blocks, th, 0, stream>>>(weights, ids, (const __nv_bfloat16*)gating, bias, tokens, experts, topk, mode, renorm, scale)),
-              (topk_gating_kernel<__half><<<blocks, th, 0, stream>>>(weights, ids, (const __half*)gating, bias, tokens, experts, topk, mode, renorm, scale)),
-              (topk_gating_kernel<float><<<blocks, th, 0, stream>>>(weights, ids, (const float*)gating, bias, tokens, experts, topk, mode, renorm, scale)))
+              (launch_topk<__nv_bfloat16>(weights, ids, (const __nv_bfloat16*)gating, bias, tokens, experts, stride, topk, mode, renorm, scale, stream)),
+              (launch_topk<__half>(weights, ids, (const __half*)gating, bias, tokens, experts, stride, topk, mode, renorm, scale, stream)),
+              (launch_topk<float>(weights, ids, (const float*)gating, bias, tokens, experts, stride, topk, mode, renorm, scale, stream)))
 }
 
 void grouped_topk(float* weights, int* ids, const void* gating, const float* bias, int tokens, int experts, int topk,

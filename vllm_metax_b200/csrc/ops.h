@@ -167,8 +167,9 @@ void embedding(void* out, const void* table, const int64_t* ids, int tokens, int
                int64_t vocab_start, int dtype, cudaStream_t stream);
 
 // ---- moe.cu / gemm_grouped_tcgen05.cu
-void topk_gating(float* weights, int* ids, const void* gating, const float* bias, int tokens, int experts, int topk,
-                 int mode, int renorm, float scale, int dtype, cudaStream_t stream);
+// (rows of gating start `stride` elements apart)
+void topk_gating(float* weights, int* ids, const void* gating, const float* bias, int tokens, int experts, int64_t stride,
+                 int topk, int mode, int renorm, float scale, int dtype, cudaStream_t stream);
 void grouped_topk(float* weights, int* ids, const void* gating, const float* bias, int tokens, int experts, int topk,
                   int n_group, int topk_group, int sigmoid, int renorm, float scale, int dtype, cudaStream_t stream);
 void moe_align(int* sorted_ids, int* block_expert, int* total_padded, int* inv_pos, const int* topk_ids,
@@ -342,13 +343,15 @@ struct HeadNormRopeParams {
   void* k_cache; void* v_cache;         // K / V of page 0, or null: queries only
   int64_t page_stride, num_slots;       // elements between two pages
   const void* q_w; const void* k_w;     // [dim_pad] norm weights or null (no norm)
-  const double* inv_freq;               // [rot / 2]
-  const int64_t* positions; const int64_t* slots;
+  const float* angles;                  // [tokens, 2, rot / 2]: cosines, sines
+  const int64_t* slots;
   int tokens, heads, kv_heads, dim, dim_pad, vdim_pad, rot, block_size, one_plus, vec;
   float eps;
   StatusWord* status;
 };
 int head_norm_rope(const HeadNormRopeParams& p, int dtype, cudaStream_t stream);
+// cos and sin of position * inv_freq, [tokens, 2, half]; whole turns are taken off in fp64
+void rope_angles(float* out, const int64_t* positions, const double* inv_freq, int tokens, int half, cudaStream_t stream);
 // ---- gla.cu (gated linear attention: decay per key channel)
 struct GlaParams {
   const void* qkvg;            // [tokens, row_stride]: q | k | v | gate at the given element offsets

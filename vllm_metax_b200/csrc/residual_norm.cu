@@ -37,36 +37,52 @@ __device__ __forceinline__ void load_gain(const void* g, int n, int f32, int c0,
   }
 }
 
-template <typename T, int CN, bool VEC, bool COMBINE>
-__global__ void __launch_bounds__(512)
+// Four pairs of a token at once: their rows' loads are all in flight before the first is used.
+template <typename T, int CN, bool VEC>
+__device__ __forceinline__ void add_expert_rows(const ResidualNormParams& p, int64_t t, int c0, float (&v)[CN]) {
+  constexpr int kAhead = 4;
+  const T* y = reinterpret_cast<const T*>(p.y);
+  for (int k0 = 0; k0 < p.topk; k0 += kAhead) {
+    const T* row[kAhead];
+    float w[kAhead], f[kAhead][CN];
+#pragma unroll
+    for (int u = 0; u < kAhead; ++u) {
+      row[u] = nullptr;
+      w[u] = 0.f;
+      if (k0 + u < p.topk) {
+        const int64_t i = t * p.topk + k0 + u;
+        const int pos = p.inv_pos[i];
+        w[u] = p.weights[i];
+        if (pos >= 0) row[u] = y + (int64_t)pos * p.D;
+        else if (p.through != nullptr && p.expert_ids[i] >= p.identity_from)
+          row[u] = reinterpret_cast<const T*>(p.through) + t * p.D;
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < kAhead; ++u)
+      if (row[u] != nullptr) load_row<T, CN, VEC>(row[u], c0, p.D, f[u]);
+#pragma unroll
+    for (int u = 0; u < kAhead; ++u)
+      if (row[u] != nullptr)
+#pragma unroll
+        for (int j = 0; j < CN; ++j) v[j] = fmaf(w[u], f[u][j], v[j]);
+  }
+}
+
+template <typename T, int CN, bool VEC, bool COMBINE, int THREADS, int CTAS>
+__global__ void __launch_bounds__(THREADS, CTAS)
 residual_norm_kernel(const ResidualNormParams p) {
   __shared__ float red[2][32];
   const int64_t t = blockIdx.x;
   const int D = p.D, c0 = threadIdx.x * CN;
   const bool mine = c0 < D;
   const T* y = reinterpret_cast<const T*>(p.y);
-  float v[CN] = {}, xv[CN] = {}, g[CN] = {}, g2[CN] = {};
+  float v[CN] = {}, xv[CN] = {}, g[CN] = {};
   if (mine) {
-    if (p.x != nullptr) {
-      load_row<float, CN, VEC>(p.x + t * D, c0, D, xv);
-      load_gain<T, CN, VEC>(p.gain, p.gain_n, p.gain_f32, c0, D, g);
-    }
-    load_gain<T, CN, VEC>(p.gain2, p.gain2_n, p.gain_f32, c0, D, g2);
+    if (p.x != nullptr) load_row<float, CN, VEC>(p.x + t * D, c0, D, xv);
     if constexpr (COMBINE) {
       if (p.shared != nullptr) load_row<T, CN, VEC>(reinterpret_cast<const T*>(p.shared) + t * D, c0, D, v);
-      for (int k = 0; k < p.topk; ++k) {
-        const int64_t i = t * p.topk + k;
-        const int pos = p.inv_pos[i];
-        const T* row = nullptr;
-        if (pos >= 0) row = y + (int64_t)pos * D;
-        else if (p.through != nullptr && p.expert_ids[i] >= p.identity_from) row = reinterpret_cast<const T*>(p.through) + t * D;
-        if (row == nullptr) continue;
-        const float w = p.weights[i];
-        float f[CN];
-        load_row<T, CN, VEC>(row, c0, D, f);
-#pragma unroll
-        for (int j = 0; j < CN; ++j) v[j] = fmaf(w, f[j], v[j]);
-      }
+      add_expert_rows<T, CN, VEC>(p, t, c0, v);
     } else {
       const int64_t row = p.ids != nullptr ? p.ids[t] : t;
       if (row >= 0 && row < p.rows) load_row<T, CN, VEC>(y + row * D, c0, D, v);
@@ -79,6 +95,7 @@ residual_norm_kernel(const ResidualNormParams p) {
 #pragma unroll
     for (int k = 0; k < CN; ++k) ss = fmaf(v[k], v[k], ss);
     const float inv = 1.f / sqrtf(row_sum(ss, red[0]) * inv_d + p.eps);
+    if (mine) load_gain<T, CN, VEC>(p.gain, p.gain_n, p.gain_f32, c0, D, g);
 #pragma unroll
     for (int k = 0; k < CN; ++k) v[k] = fmaf(v[k] * inv, g[k], xv[k]);
   } else {
@@ -90,24 +107,29 @@ residual_norm_kernel(const ResidualNormParams p) {
 #pragma unroll
   for (int k = 0; k < CN; ++k) ss = fmaf(v[k], v[k], ss);
   const float inv = 1.f / sqrtf(row_sum(ss, red[1]) * inv_d + p.eps);
+  if (!mine) return;
+  load_gain<T, CN, VEC>(p.gain2, p.gain2_n, p.gain_f32, c0, D, g);
 #pragma unroll
-  for (int k = 0; k < CN; ++k) v[k] = v[k] * inv * g2[k];
-  if (mine) store_row<T, CN, VEC>(reinterpret_cast<T*>(p.h) + t * D, c0, D, v);
+  for (int k = 0; k < CN; ++k) v[k] = v[k] * inv * g[k];
+  store_row<T, CN, VEC>(reinterpret_cast<T*>(p.h) + t * D, c0, D, v);
 }
 
-template <typename T, int CN, bool VEC>
+template <typename T, int CN, bool VEC, int THREADS, int CTAS>
 void launch(const ResidualNormParams& p, cudaStream_t stream) {
   const int threads = (p.D + CN * 32 - 1) / (CN * 32) * 32;
-  if (p.topk > 0) residual_norm_kernel<T, CN, VEC, true><<<p.tokens, threads, 0, stream>>>(p);
-  else residual_norm_kernel<T, CN, VEC, false><<<p.tokens, threads, 0, stream>>>(p);
+  if (p.topk > 0)
+    residual_norm_kernel<T, CN, VEC, true, THREADS, CTAS / 2 + CTAS % 2><<<p.tokens, threads, 0, stream>>>(p);
+  else
+    residual_norm_kernel<T, CN, VEC, false, THREADS, CTAS><<<p.tokens, threads, 0, stream>>>(p);
 }
 
 template <typename T>
 int by_width(const ResidualNormParams& p, cudaStream_t stream) {
-  if (p.D > 16 * 512) return 1;
-  if (p.vec && p.D <= 2048) launch<T, 8, true>(p, stream);
-  else if (p.vec && p.D % 16 == 0) launch<T, 16, true>(p, stream);
-  else launch<T, 16, false>(p, stream);
+  if (p.D > 8 * 1024) return 1;
+  if (p.vec && p.D <= 2048) launch<T, 8, true, 256, 6>(p, stream);
+  else if (p.vec && p.D <= 4096) launch<T, 8, true, 512, 3>(p, stream);
+  else if (p.vec) launch<T, 8, true, 1024, 1>(p, stream);
+  else launch<T, 16, false, 512, 1>(p, stream);
   return 0;
 }
 

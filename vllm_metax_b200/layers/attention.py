@@ -317,6 +317,7 @@ class QKNormAttention(nn.Module):
         self.q_norm = _param(self.dim_pad, dtype=dtype)
         self.k_norm = _param(self.dim_pad, dtype=dtype) if self.own_kv else None
         self.out_proj = _param(width, heads * self.vdim_pad, dtype=dtype)
+        self.rotation = ("rope_angles", tuple(inv_freq.tolist()))
         self.register_buffer("inv_freq", inv_freq.double().to(torch.get_default_device()), persistent=False)
         self.attn = Attention(heads, self.dim_pad, scale, kv_heads, cache_idx, sliding_window=window)
 
@@ -345,7 +346,10 @@ class QKNormAttention(nn.Module):
         md = ctx.attn_metadata
         cache = ctx.kv_caches[self.attn.layer_idx][0]
         kv = PagedGQABackend.views(cache, md.block_size, self.kv_heads, self.dim_pad, self.vdim_pad)
-        q = ops.head_norm_rope(self.proj(h), self.offsets, self.q_norm, self.k_norm, self.heads, self.dim, self.inv_freq,
-                               positions, kv if self.own_kv else None, md.slot_mapping, self.eps)
+        angles = ctx.extra.get(self.rotation)                 # one table per step and rotation, shared by the layers
+        if angles is None:
+            angles = ctx.extra[self.rotation] = ops.rope_angles(positions, self.inv_freq, h.shape[0])
+        q = ops.head_norm_rope(self.proj(h), self.offsets, self.q_norm, self.k_norm, self.heads, self.dim, angles,
+                               kv if self.own_kv else None, md.slot_mapping, self.eps)
         o = self.attn.attend(q, md, kv)
         return ops.gemm(o.view(h.shape[0], self.heads * self.vdim_pad), self.out_proj)

@@ -88,7 +88,7 @@ class RoutedExperts(nn.Module):
 
     def forward(self, h):
         shared = self.shared(h) if self.shared is not None else None
-        return self.experts(h, ops.gemm(h, self.gate, out_dtype=torch.float32), shared)
+        return self.experts(h, ops.router_logits(h, self.gate), shared)
 
 
 class NaguzenLayer(nn.Module):

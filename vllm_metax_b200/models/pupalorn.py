@@ -65,7 +65,7 @@ class IdentityRoutedExperts(nn.Module):
         return out
 
     def forward(self, h):
-        return self.experts.forward_rows(h, ops.gemm(h, self.gate, out_dtype=torch.float32))
+        return self.experts.forward_rows(h, ops.router_logits(h, self.gate))
 
 
 def _rotation(rot: dict) -> torch.Tensor:

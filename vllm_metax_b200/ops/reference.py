@@ -354,11 +354,15 @@ def epilogue_activation(y: torch.Tensor, act: str, params: Optional[torch.Tensor
 
 
 def rotate_half(x: torch.Tensor, inv_freq: torch.Tensor, positions: torch.Tensor) -> torch.Tensor:
-    """Rotation of the first ``2 * len(inv_freq)`` entries of ``x [T, H, D]``, pairs (i, i + half), angles in the type of
-    ``inv_freq``."""
-    half = inv_freq.numel()
-    a = positions[: x.shape[0]].to(inv_freq.dtype)[:, None] * inv_freq[None]
-    c, s = torch.cos(a).float()[:, None], torch.sin(a).float()[:, None]
+    """Rotation of the first ``2 * len(inv_freq)`` entries of ``x [T, H, D]``, pairs (i, i + half), angles in fp32."""
+    a = positions[: x.shape[0]].float()[:, None] * inv_freq[None]
+    return rotate_half_by(x, torch.stack([torch.cos(a), torch.sin(a)], 1))
+
+
+def rotate_half_by(x: torch.Tensor, angles: torch.Tensor) -> torch.Tensor:
+    """The same by cosines and sines ``[T, 2, half]``."""
+    half = angles.shape[-1]
+    c, s = angles[:, :1], angles[:, 1:]
     u, v = x[..., :half].float(), x[..., half: 2 * half].float()
     return torch.cat([(u * c - v * s).to(x.dtype), (v * c + u * s).to(x.dtype), x[..., 2 * half:]], -1)
 

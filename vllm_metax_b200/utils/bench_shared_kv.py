@@ -105,6 +105,7 @@ def kernel_rows(size: str = "w2048", only: str = "") -> list:
         slots = bt.long()[torch.arange(T, device=dev) // per, pos // bs] * bs + pos % bs
         qkv, qw, kw = rn(T, (H + 2 * G) * D), rn(D), rn(D)
         freq = torch.rand(32, device=dev, dtype=torch.float64)
+        ang = ops.rope_angles(pos, freq, T)
         cs = torch.rand(16384, D, device=dev)
         q, k, v = qkv[:, : H * D], qkv[:, H * D: (H + G) * D], qkv[:, (H + G) * D:]
         kv = ops.kv_views(cache)
@@ -116,12 +117,13 @@ def kernel_rows(size: str = "w2048", only: str = "") -> list:
             ops.rope_and_cache(pos, q, k, v, D, cs, True, cache, slots)
 
         if B != 1:
+            row(f"rope_angles (once a step), {phase}", lambda: ops.rope_angles(pos, freq, T), 4.0 * T * 64)
             byts = 4.0 * T * (H + 2 * G) * D
-            row(f"head_norm_rope, {phase}", lambda: ops.head_norm_rope(qkv, off, qw, kw, H, D, freq, pos, kv, slots, 1e-6), byts, 0,
+            row(f"head_norm_rope, {phase}", lambda: ops.head_norm_rope(qkv, off, qw, kw, H, D, ang, kv, slots, 1e-6), byts, 0,
                 ("head_rms_norm x 2 + rope_and_cache", separate, byts, 0))
             qo = rn(T, H * D)
             row(f"head_norm_rope, queries only, {phase}",
-                lambda: ops.head_norm_rope(qo, (0, 0, 0), qw, None, H, D, freq, pos, None, slots, 1e-6), 4.0 * T * H * D, 0,
+                lambda: ops.head_norm_rope(qo, (0, 0, 0), qw, None, H, D, ang, None, slots, 1e-6), 4.0 * T * H * D, 0,
                 ("head_rms_norm", lambda: ops.head_rms_norm(qo, qw, 1e-6, H, D), 4.0 * T * H * D, 0))
         # -- attention
         q3 = rn(T, H, D)
@@ -130,8 +132,10 @@ def kernel_rows(size: str = "w2048", only: str = "") -> list:
             att = lambda w: (lambda: ops.paged_attention_decode(q3, cache, bt, lens, 0.09, window=w, max_seq_len=ctx))
             cost = lambda n: 4.0 * B * n * G * D + 4.0 * T * H * D
             for w in (win, 128):
+                short = torch.full((B,), w, dtype=torch.int32, device=dev)      # as many keys without a window
                 row(f"paged decode, window {w}, {phase}", att(w), cost(w), 4.0 * B * H * w * D,
-                    ("paged decode without a window", att(-1), cost(ctx), 4.0 * B * H * ctx * D))
+                    (f"paged decode, context {w}", lambda: ops.paged_attention_decode(q3, cache, bt, short, 0.09, max_seq_len=w),
+                     cost(w), 4.0 * B * H * w * D))
         else:
             qsl = torch.arange(B + 1, dtype=torch.int32, device=dev) * per
             att = lambda w: (lambda: ops.paged_attention_prefill(q3, cache, bt, lens, qsl, 0.09, max_q_len=per, window=w, max_seq_len=ctx))
@@ -145,7 +149,7 @@ def kernel_rows(size: str = "w2048", only: str = "") -> list:
         # -- experts
         E, I, top, ff, gf = s["experts"], s["identity"], s["top"], s["ff"], _gated(s["ff"])
         gate, bias = rn(E + I, W), rn(E + I, dt=torch.float32)
-        row(f"router product (fp32 out), {phase}", lambda: ops.gemm(y, gate, out_dtype=torch.float32),
+        row(f"router product (fp32 out), {phase}", lambda: ops.router_logits(y, gate),
             2.0 * (T * W + (E + I) * W) + 4.0 * T * (E + I), 2.0 * T * W * (E + I),
             ("router product (bf16 out)", lambda: ops.gemm(y, gate[:E]), 2.0 * (T * W + E * W + T * E), 2.0 * T * W * E))
         z, zb = rn(T, E + I, dt=torch.float32), rn(T, E)
