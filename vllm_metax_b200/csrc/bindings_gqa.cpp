@@ -110,6 +110,7 @@ void head_norm_rope(Tensor& q_out, const Tensor& qkv, int64_t q_off, int64_t k_o
     TORCH_CHECK(pv.dqk == DP && k_off + pv.heads * DP <= qkv.size(1) && v_off + pv.heads * pv.dv <= qkv.size(1));
     p.k_cache = k_cache->data_ptr(); p.v_cache = v_cache->data_ptr();
     p.page_stride = pv.page_stride; p.num_slots = pv.num_blocks * pv.block_size;
+    TORCH_CHECK(p.num_slots < (int64_t(1) << 31), "head_norm_rope: too many cache slots");
     p.kv_heads = pv.heads; p.vdim_pad = pv.dv; p.block_size = pv.block_size;
     p.vec = p.vec && pv.dv % 8 == 0 && k_off % unit == 0 && v_off % unit == 0 && pv.page_stride % unit == 0 &&
             aligned(p.k_cache) && aligned(p.v_cache);

@@ -11,7 +11,7 @@
 namespace b200 {
 namespace {
 
-constexpr int kThreads = 256;
+constexpr int kThreads = 256, kCtas = 8;           // kCtas: CTAs per SM that walk the tokens
 
 __global__ void rope_angles_kernel(float* __restrict__ out, const int64_t* __restrict__ positions,
                                    const double* __restrict__ inv_freq, int64_t n, int half) {
@@ -54,72 +54,81 @@ __device__ __forceinline__ void cache_rows(const HeadNormRopeParams& p, int64_t 
     report_status(p.status, kBadIndex, 140, (int)p.num_slots, (int)slot);
     return;
   }
-  const int64_t page = (slot / p.block_size) * p.page_stride, at = slot % p.block_size;
-  k_row = page + at * p.kv_heads * p.dim_pad;
-  v_row = page + at * p.kv_heads * p.vdim_pad;
+  const uint32_t block = (uint32_t)slot / (uint32_t)p.block_size, at = (uint32_t)slot % (uint32_t)p.block_size;
+  k_row = block * p.page_stride + (int64_t)at * p.kv_heads * p.dim_pad;
+  v_row = block * p.page_stride + (int64_t)at * p.kv_heads * p.vdim_pad;
 }
 
-// Heads of up to 256 entries whose half rotation is a multiple of 8: `lanes` neighbouring lanes (a power of two) hold one head
-// of one token, 8 entries each, and exchange rotation partners by shuffles.  A token's items: queries, keys, then its values
-// in pieces of lanes * 8 entries.
+// Heads of up to 256 entries whose half rotation is a multiple of 8: `1 << log_lanes` neighbouring lanes hold one head of one
+// token, 8 entries each, and exchange rotation partners by shuffles.  A token's items: queries, keys, then its values in
+// pieces of lanes * 8 entries.  A thread keeps its item and the norm weights of it and walks tokens.
 template <typename T>
 __global__ void __launch_bounds__(kThreads)
-head_norm_rope_vec_kernel(const HeadNormRopeParams p, int lanes, int value_items) {
-  const int lane = threadIdx.x & 31, j = lane & (lanes - 1);
-  const int normed = p.heads + (p.k_cache != nullptr ? p.kv_heads : 0), items = normed + value_items;
-  const int64_t id = ((int64_t)blockIdx.x * kThreads + threadIdx.x) / lanes;
-  const int64_t t = id / items;
-  const int item = (int)(id % items);
+head_norm_rope_vec_kernel(const HeadNormRopeParams p, int log_lanes, int items) {
+  const int lanes = 1 << log_lanes, lane = threadIdx.x & 31, j = lane & (lanes - 1);
+  const int item = (blockIdx.y * kThreads + threadIdx.x) >> log_lanes;
+  const int normed = p.heads + (p.k_cache != nullptr ? p.kv_heads : 0);
   const int c0 = j * 8, half = p.rot / 2;
-  const bool in_step = t < p.tokens, head = in_step && item < normed && c0 < p.dim_pad;
-  const T* src = nullptr;
-  T* dst = nullptr;
-  const T* w = nullptr;
-  float v[8] = {};
-  if (in_step && item >= p.heads) {
-    int64_t k_row, v_row;
-    cache_rows(p, t, k_row, v_row);
-    if (item >= normed) {                                    // values: copied as they are
-      const int at = ((item - normed) * lanes + j) * 8;
-      if (v_row >= 0 && at < p.kv_heads * p.vdim_pad) {
-        load_row<T, 8, true>(reinterpret_cast<const T*>(p.qkv) + t * p.row_stride + p.v_off, at, 0, v);
-        store_row<T, 8, true>(reinterpret_cast<T*>(p.v_cache) + v_row, at, 0, v);
+  const bool head = item < normed && c0 < p.dim_pad, is_q = item < p.heads;
+  const int h = is_q ? item : item - p.heads;
+  const int v_at = ((item - normed) * lanes + j) * 8;          // (of a value item)
+  const bool value = item >= normed && item < items && v_at < p.kv_heads * p.vdim_pad;
+  const bool first = c0 < half, rotated = c0 < p.rot;
+  const int partner = ((lane - j) + (first ? j + half / 8 : rotated ? j - half / 8 : j)) & 31;
+  const T* col = reinterpret_cast<const T*>(p.qkv) +
+                 (value ? p.v_off + v_at : (is_q ? p.q_off : p.k_off) + (int64_t)h * p.dim_pad + c0);
+  const T* w = reinterpret_cast<const T*>(is_q ? p.q_w : p.k_w);
+  const bool norm = p.q_w != nullptr;                          // (uniform: both weights or none)
+  const float* ang = p.angles + (first ? c0 : c0 - half);
+  float g[8];
+#pragma unroll
+  for (int k = 0; k < 8; ++k) g[k] = 1.f;
+  if (head && norm) {
+    load_row<T, 8, true>(w, c0, p.dim_pad, g);
+#pragma unroll
+    for (int k = 0; k < 8; ++k) g[k] += p.one_plus ? 1.f : 0.f;
+  }
+  const float inv_dim = 1.f / (float)p.dim;
+  for (int t = blockIdx.x; t < p.tokens; t += gridDim.x) {     // (uniform over the CTA: the shuffles below need whole warps)
+    float v[8] = {};
+    int64_t k_row = -1, v_row = -1;
+    if (item >= p.heads) cache_rows(p, t, k_row, v_row);
+    if (value) {                                               // copied as they are
+      if (v_row >= 0) {
+        load_row<T, 8, true>(col + t * p.row_stride, 0, 8, v);
+        store_row<T, 8, true>(reinterpret_cast<T*>(p.v_cache) + v_row + v_at, 0, 8, v);
       }
     } else if (head) {
-      locate<T>(p, t, k_row, item, src, dst, w);
+      load_row<T, 8, true>(col + t * p.row_stride, 0, 8, v);
     }
-  } else if (head) {
-    locate<T>(p, t, -1, item, src, dst, w);
-  }
-  const bool first = c0 < half, rotated = c0 < p.rot;
-  float c[8] = {}, s[8] = {}, g[8] = {};
-  if (head) {
-    load_row<T, 8, true>(src, c0, p.dim_pad, v);
-    if (w != nullptr) load_row<T, 8, true>(w, c0, p.dim_pad, g);
-    if (rotated) {
-      const float* a = p.angles + 2 * t * half;
-      load_row<float, 8, true>(a, first ? c0 : c0 - half, half, c);
-      load_row<float, 8, true>(a + half, first ? c0 : c0 - half, half, s);
+    float c[8] = {}, s[8] = {};
+    if (head && rotated) {
+      load_row<float, 8, true>(ang + (int64_t)(2 * t) * half, 0, 8, c);
+      load_row<float, 8, true>(ang + (int64_t)(2 * t + 1) * half, 0, 8, s);
     }
-  }
-  float ss = 0.f;
+    if (norm) {
+      float ss = 0.f;
 #pragma unroll
-  for (int k = 0; k < 8; ++k) ss = fmaf(v[k], v[k], ss);
-  for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-  if (w != nullptr) {
-    const float inv = 1.f / sqrtf(ss / (float)p.dim + p.eps);
+      for (int k = 0; k < 8; ++k) ss = fmaf(v[k], v[k], ss);
+      for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      const float inv = 1.f / sqrtf(ss * inv_dim + p.eps);
 #pragma unroll
-    for (int k = 0; k < 8; ++k) v[k] = v[k] * inv * (p.one_plus ? 1.f + g[k] : g[k]);
-  }
-  if (p.rot > 0) {
-    const int partner = (lane - j) + (first ? j + half / 8 : rotated ? j - half / 8 : j);
+      for (int k = 0; k < 8; ++k) v[k] = v[k] * inv * g[k];
+    }
+    if (p.rot > 0) {
 #pragma unroll
-    for (int k = 0; k < 8; ++k) {
-      const float o = __shfl_sync(0xffffffffu, v[k], partner & 31);
-      if (rotated) v[k] = first ? v[k] * c[k] - o * s[k] : v[k] * c[k] + o * s[k];
+      for (int k = 0; k < 8; ++k) {
+        const float o = __shfl_sync(0xffffffffu, v[k], partner);
+        if (head && rotated) v[k] = v[k] * c[k] + (first ? -o : o) * s[k];
+      }
+    }
+    if (head) {
+      if (is_q)
+        store_row<T, 8, true>(reinterpret_cast<T*>(p.q_out) + ((int64_t)t * p.heads + h) * p.dim_pad, c0, p.dim_pad, v);
+      else if (k_row >= 0)
+        store_row<T, 8, true>(reinterpret_cast<T*>(p.k_cache) + k_row + (int64_t)h * p.dim_pad, c0, p.dim_pad, v);
     }
   }
-  if (dst != nullptr) store_row<T, 8, true>(dst, c0, p.dim_pad, v);
 }
 
 // Any sizes: one CTA per token, a warp per head, the normed head staged in shared memory.
@@ -172,13 +181,15 @@ head_norm_rope_kernel(const HeadNormRopeParams p) {
 template <typename T>
 int launch(const HeadNormRopeParams& p, cudaStream_t stream) {
   if (p.rot > p.dim || p.rot % 2 != 0 || p.dim_pad > kMaxDim) return 1;
+  if (p.k_cache != nullptr && (p.q_w == nullptr) != (p.k_w == nullptr)) return 1;
   if (p.vec && p.dim_pad <= 256 && p.rot % 16 == 0) {
-    int lanes = 1;
-    while (lanes * 8 < p.dim_pad) lanes *= 2;
-    const int values = p.k_cache != nullptr ? ceil_div(p.kv_heads * p.vdim_pad, lanes * 8) : 0;
+    int log_lanes = 0;
+    while ((8 << log_lanes) < p.dim_pad) ++log_lanes;
+    const int values = p.k_cache != nullptr ? ceil_div(p.kv_heads * p.vdim_pad, 8 << log_lanes) : 0;
     const int items = p.heads + (p.k_cache != nullptr ? p.kv_heads : 0) + values;
-    const int64_t threads = (int64_t)p.tokens * items * lanes;
-    head_norm_rope_vec_kernel<T><<<(unsigned)((threads + kThreads - 1) / kThreads), kThreads, 0, stream>>>(p, lanes, values);
+    const int columns = ceil_div(items << log_lanes, kThreads);
+    const int rows = ceil_div(kCtas * 148, columns);
+    head_norm_rope_vec_kernel<T><<<dim3(p.tokens < rows ? p.tokens : rows, columns), kThreads, 0, stream>>>(p, log_lanes, items);
   } else {
     head_norm_rope_kernel<T><<<p.tokens, kAnyWarps * 32, 0, stream>>>(p);
   }
@@ -187,7 +198,7 @@ int launch(const HeadNormRopeParams& p, cudaStream_t stream) {
 
 }  // namespace
 
-// Returns 1 for heads wider than 1024 or an odd number of rotated entries.
+// Returns 1 for heads wider than 1024, an odd number of rotated entries, or key weights without query weights.
 int head_norm_rope(const HeadNormRopeParams& p, int dtype, cudaStream_t stream) {
   if (p.tokens <= 0) return 0;
   if (dtype == 0) return launch<__nv_bfloat16>(p, stream);
