@@ -689,6 +689,8 @@ class ModelRunner:
 
     def _decode_splits(self, batch: int) -> int:
         spec = self.model.kv_cache_spec()
+        if spec["kind"] == "layers":              # sizes and windows differ by layer: each chooses for itself
+            return 0
         if spec["kind"] != "gqa":
             return 1
         return ops.decode_num_splits(batch, spec["num_kv_heads"], self.cfg.scheduler.max_model_len, 1, self.sms)
@@ -718,6 +720,9 @@ class ModelRunner:
             hq = spec["num_kv_heads"] * (self.cfg.model.num_attention_heads // self.cfg.model.num_key_value_heads)
             md.decode_workspace = torch.empty(md.decode_num_splits * bucket * hq * (spec["head_size"] + 1),
                                               dtype=torch.float32, device=self.device)
+        elif spec["kind"] == "layers":            # (the graph keeps it: no other capture may grow or free it)
+            floats = self.model.decode_workspace_floats(bucket, self.cfg.scheduler.max_model_len)
+            md.decode_workspace = torch.empty(floats, dtype=torch.float32, device=self.device) if floats else None
         # safe dummy inputs for warm-up
         self.query_start_loc[:bucket + 1].copy_(torch.arange(bucket + 1, dtype=torch.int32))
         self.seq_lens[:bucket].fill_(1)

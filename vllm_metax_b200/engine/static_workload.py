@@ -80,6 +80,9 @@ class StaticWorkload:
             hq = r.cfg.model.num_attention_heads // max(1, r.cfg.parallel.tensor_parallel_size)
             md.decode_workspace = torch.empty(md.decode_num_splits * N * hq * (spec["head_size"] + 1),
                                               dtype=torch.float32, device=dev)
+        elif r.model.kv_cache_spec()["kind"] == "layers":
+            floats = r.model.decode_workspace_floats(N, self.P + self.O)
+            md.decode_workspace = torch.empty(floats, dtype=torch.float32, device=dev) if floats else None
         self._state_slots(md, 0, N, True)
         self.decode_md = md
         self.col = torch.zeros(1, dtype=torch.int64, device=dev)

@@ -334,6 +334,12 @@ class QKNormAttention(nn.Module):
                         "v": heads("v", self.kv_heads, self.vdim, self.vdim_pad)})
         return out
 
+    def decode_workspace_floats(self, batch: int, max_seq_len: int) -> int:
+        """What the split decode of ``batch`` rows needs for its partial results (0: it does not split)."""
+        tiles = -(-(self.heads // self.kv_heads) // 16)
+        n = ops.decode_num_splits(batch, self.kv_heads, max_seq_len, tiles, window=self.attn.window)
+        return n * batch * self.heads * (self.vdim_pad + 1) if n > 1 else 0
+
     def cache_elems_per_token(self) -> int:
         return self.kv_heads * (self.dim_pad + self.vdim_pad) if self.own_kv else 0
 

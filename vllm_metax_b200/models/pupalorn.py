@@ -151,6 +151,9 @@ class PupalornForCausalLM(nn.Module):
             raise ValueError(f"the cache is kept in the model's dtype, not {kv_cache_dtype}")
         return [m.allocate_kv_cache(num_blocks, block_size, device) for m in self._own()]
 
+    def decode_workspace_floats(self, batch: int, max_seq_len: int) -> int:
+        return max((l.mixer.decode_workspace_floats(batch, max_seq_len) for l in self.layers), default=0)
+
     def forward(self, input_ids, positions, intermediate=None):
         first = self.layers[0].in1 if len(self.layers) else self.final_norm
         x, h = embed_norm(self.embed.weight, input_ids, self.cfg.vocab_size, self.embed_scale, first.gain, self.eps)

@@ -141,9 +141,15 @@ def kernel_rows(size: str = "w2048", only: str = "") -> list:
             att = lambda w: (lambda: ops.paged_attention_prefill(q3, cache, bt, lens, qsl, 0.09, max_q_len=per, window=w, max_seq_len=ctx))
             pairs = lambda w: B * sum(min(i + 1, w) for i in range(per))
             byts = 4.0 * T * H * D + 4.0 * T * G * D
-            for w in (win, 128):
-                row(f"paged prompt attention, window {w}, {phase}", att(w), byts, 4.0 * H * pairs(w) * D,
-                    ("without a window", att(-1), byts, 4.0 * H * pairs(per) * D))
+            row(f"paged prompt attention, window {win}, {phase}", att(win), byts, 4.0 * H * pairs(win) * D,
+                ("without a window", att(-1), byts, 4.0 * H * pairs(per) * D))
+            # a short window against prompts as short as it: as many key tiles per query tile
+            n = T // 128
+            bt2 = torch.arange(2 * n, dtype=torch.int32, device=dev).view(n, 2)
+            len2, qsl2 = torch.full((n,), 128, dtype=torch.int32, device=dev), torch.arange(n + 1, dtype=torch.int32, device=dev) * 128
+            row(f"paged prompt attention, window 128, {phase}", att(128), byts, 4.0 * H * pairs(128) * D,
+                (f"prompts {n}x128 without a window", lambda: ops.paged_attention_prefill(
+                    q3, cache, bt2, len2, qsl2, 0.09, max_q_len=128, max_seq_len=128), byts, 4.0 * H * n * 128 * 129 / 2 * D))
         if B == 1:
             continue
         # -- experts
