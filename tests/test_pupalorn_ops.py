@@ -69,9 +69,9 @@ def test_embedding_boundary(device, dt, width):
 
 
 # ------------------------------------------------------------------ rotation frequencies
-@pytest.mark.parametrize("scaling", [None, dict(factor=8.0, low=1.0, high=4.0, original=512),
+@pytest.mark.parametrize("scaling", [None, dict(factor=5.0, low=1.0, high=3.0, original=300),
                                      dict(factor=3.0, low=2.0, high=2.5, original=100), dict(factor=1.0, low=1.0, high=4.0, original=64)])
-@pytest.mark.parametrize("dims,base", [(2, 500.0), (32, 10000.0), (96, 5e5)])
+@pytest.mark.parametrize("dims,base", [(2, 500.0), (40, 8000.0), (96, 5e5)])
 def test_frequencies(dims, base, scaling):
     hf = scaling and {"type": "llama3", "factor": scaling["factor"], "low_freq_factor": scaling["low"],
                       "high_freq_factor": scaling["high"], "original_max_position_embeddings": scaling["original"]}
@@ -204,7 +204,7 @@ def moe_weights(E, I, W, ff, dt, seed=0):
 
 
 @pytest.mark.parametrize("device", DEVICES)
-@pytest.mark.parametrize("E,I,top", [(16, 2, 2), (3, 5, 4), (8, 0, 1), (1, 1, 2), (40, 30, 6)])
+@pytest.mark.parametrize("E,I,top", [(12, 3, 2), (3, 5, 4), (8, 0, 1), (1, 1, 2), (40, 30, 6)])
 def test_routing(device, E, I, top):
     """Softmax over all outputs, the correction in the choice and not in the weights, no renormalisation."""
     T = 33

@@ -36,7 +36,7 @@ def pupalorn_config(s: dict, layers: int = 8, share: bool = True, window: bool =
             m["kv_from"] = layers // 2 - 1
         out.append({"type": "attention", "mixer": m, "mlp": mlp})
     return ModelConfig.from_layer_list({"architecture": "Pupalorn", "vocab": 32768, "width": s["width"], "norm": {"eps": 1e-6},
-                                        "embedding": {"scale": 12.0}, "residual_mult": 0.5, "layers": out})
+                                        "embedding": {"scale": 8.0}, "residual_mult": 0.4, "layers": out})
 
 
 def qwen3_moe_config(s: dict, layers: int = 8) -> ModelConfig:
@@ -95,7 +95,7 @@ def kernel_rows(size: str = "w2048", only: str = "") -> list:
             row(f"boundary_norm in front of the head, {phase}", lambda: boundary_norm(y, x, g1, g2, 1e-6, want_x=False),
                 8.0 * T * W, 0, norm_like)
             table, ids = rn(32768, W), torch.randint(0, 32768, (T,), device=dev)
-            row(f"embed_norm, {phase}", lambda: embed_norm(table, ids, 32768, 12.0, g2, 1e-6), 8.0 * T * W, 0,
+            row(f"embed_norm, {phase}", lambda: embed_norm(table, ids, 32768, 8.0, g2, 1e-6), 8.0 * T * W, 0,
                 ("embedding", lambda: ops.embedding(table, ids), 4.0 * T * W, 0))
         # -- projection epilogue
         bs, nb = 64, ctx // 64 + 1
