@@ -3,7 +3,7 @@
 The shared objects are produced next to this file:
 
 * ``_b200_C.so``            - CUDA kernels + ``torch.ops.b200`` bindings
-* ``_b200_<group>.so``      - the core set and one group of ``UNIT_GROUPS``: all that a model class with
+* ``_b200_<group>.so``      - the core set and the sets of one of ``UNIT_GROUPS``: all that a model class with
   ``native_units = "<group>"`` calls; built on demand where the full library does not exist yet
 * ``cumem_allocator.so``    - sleep-mode VMM allocator (CPython module, driver API)
 
@@ -31,17 +31,18 @@ OBJ = ROOT / "_obj"
 LIB = ROOT / "_b200_C.so"
 CUMEM_LIB = ROOT / "cumem_allocator.so"
 
-# the units behind bindings_core.cpp, and what each group adds behind bindings_<group>.cpp
+# the units behind bindings_core.cpp, what each set adds behind bindings_<set>.cpp, and the sets of each group
 CORE_UNITS = ("attn_prefill_pingpong", "attn_prefill_tcgen05", "gemm_grouped_tcgen05", "gemm_pair_tcgen05", "gemm_simt",
               "gemm_splitk_tcgen05", "gemm_streamk_tcgen05", "gemm_tcgen05", "moe", "residual_norm", "sampling")
-UNIT_GROUPS = {
+UNIT_SETS = {
     "gqa": ("attn_decode", "head_norm_rope", "paged_attn_simt"),
-    "hybrid": ("causal_conv1d", "fused_misc", "gla", "latent_attn", "mla_decode", "mla_decode_tcgen05", "residual_conv",
-               "rglru"),
+    "hybrid": ("fused_misc", "latent_attn", "mla_decode", "mla_decode_tcgen05", "residual_conv", "rglru"),
+    "recurrent": ("causal_conv1d", "channel_delta", "gla", "prenorm"),
 }
+UNIT_GROUPS = {"gqa": ("gqa",), "hybrid": ("hybrid", "recurrent"), "parallel": ("gqa", "recurrent")}
 # units that compute in true 32-bit (recurrences, norms, angles, fp32 products): no fast-math substitutions
-PRECISE_UNITS = ("gemm_simt", "gla", "head_norm_rope", "latent_attn", "paged_attn_simt", "residual_conv", "residual_norm",
-                 "rglru")
+PRECISE_UNITS = ("channel_delta", "gemm_simt", "gla", "head_norm_rope", "latent_attn", "paged_attn_simt", "prenorm",
+                 "residual_conv", "residual_norm", "rglru")
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-std=c++17", "-O3", "-lineinfo",
@@ -92,14 +93,16 @@ def build(verbose: bool = False, force: bool = False, group: Optional[str] = Non
     nvcc = os.path.join(_cuda_home(), "bin", "nvcc")
     jobs = []
     objs = []
+    sets = tuple(UNIT_SETS) if group is None else UNIT_GROUPS[group]
+    wanted = CORE_UNITS + tuple(u for s in sets for u in UNIT_SETS[s])
     for src in sources():
-        if group is not None and src.stem not in CORE_UNITS + UNIT_GROUPS[group]:
+        if group is not None and src.stem not in wanted:
             continue
         obj = OBJ / (src.stem + ".o")
         objs.append(obj)
         if force or _newer([src, *headers], obj):
             jobs.append([nvcc, *_unit_flags(src.stem), "-I", str(CSRC), "-c", str(src), "-o", str(obj)])
-    binds = [CSRC / "bindings_core.cpp"] + [CSRC / f"bindings_{g}.cpp" for g in UNIT_GROUPS if group in (None, g)]
+    binds = [CSRC / "bindings_core.cpp"] + [CSRC / f"bindings_{s}.cpp" for s in sets]
     if group is None:
         binds.append(CSRC / "bindings.cpp")
     inc = []

@@ -26,16 +26,19 @@ _loaded_units = ""
 ACT_CODES = {"silu": 0, "gelu": 1, "gelu_tanh": 2, "fatrelu": 3, "relu2": 4, "mul_silu": 5, "swigluoai": 6,
              "swiglustep": 7, "gelu_new": 8, "gelu_fast": 9, "gelu_quick": 10}
 # GEMM epilogues (csrc/gemm_epilogue.cuh)
-EPI_CODES = {None: 0, "silu_gate": 1, "gelu": 2, "gelu_tanh": 3, "xielu": 4, "decay": 5, "relu2": 6}
+EPI_CODES = {None: 0, "silu_gate": 1, "gelu": 2, "gelu_tanh": 3, "xielu": 4, "decay": 5, "relu2": 6, "gelu_tanh_gate": 7,
+             "clamped_swiglu_gate": 8, "softplus_decay": 9, "softcap": 10}
+EPI_NAMES = {v: k for k, v in EPI_CODES.items()}
+EPI_GATES = (1, 7, 8)                      # (gate, up) in adjacent columns, half as many come out
 CACHE_KIND = {"same": 0, "fp8_static": 1, "int8_dyn": 2, "fp8_dyn": 3}
 
 
 def load_native(build_if_missing: bool = True, units: str = "all") -> bool:
-    """Load ``_b200_C.so`` (building it in-tree when absent and allowed).  ``units`` other than "all": the caller needs the
-    core set and that unit group only - where the full library has not been built, the group's library is built and loaded
+    """Load ``_b200_C.so`` (building it in-tree when absent and allowed).  ``units`` other than "all" ("core": any library that is
+    loaded will do): the caller needs the core set and that unit group only - where the full library has not been built, the group's library is built and loaded
     instead."""
     global _loaded, _loaded_units
-    if _loaded and _loaded_units in (units, "all"):
+    if _loaded and (units == "core" or _loaded_units in (units, "all")):
         return True
     if _loaded:
         raise RuntimeError(f"this process serves a model on the {_loaded_units!r} kernel library; build the full one "
@@ -44,7 +47,7 @@ def load_native(build_if_missing: bool = True, units: str = "all") -> bool:
     if not _LIB.exists():
         from ._build import build, group_lib
 
-        if units != "all":
+        if units not in ("all", "core"):
             lib, got = group_lib(units), units
         if not lib.exists():
             if not build_if_missing or envs.B200_USE_PREBUILT_KERNELS:
@@ -117,11 +120,15 @@ def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
          force_bn: int = 0, act: Optional[str] = None, act_params: Optional[torch.Tensor] = None,
          out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
     """``act(a [M,K] @ w [N,K]^T (+bias)) (+residual)``.  ``act``: None, gelu, gelu_tanh, xielu (``act_params`` = its two
-    fp32 coefficients), decay (``sigmoid(x)^act_params[0]``), applied to the fp32 accumulators in the epilogue; ``out_dtype=torch.float32`` stores those."""
+    fp32 coefficients), decay (``sigmoid(x)^act_params[0]``), softplus_decay (``exp(-act_params[n] softplus(x))``), softcap
+    (``c tanh(x / c)``, c = ``act_params[0]``), or a gate over adjacent (gate, up) columns - gelu_tanh_gate,
+    clamped_swiglu_gate (``act_params`` = its limit and slope) - applied to the fp32 accumulators in the epilogue;
+    ``out_dtype=torch.float32`` stores those."""
+    gated = EPI_CODES[act] in EPI_GATES
     if _use_cuda(a):
         if out is None:
-            out = torch.empty(a.shape[0], w.shape[0], dtype=out_dtype or a.dtype, device=a.device)
-        if a.dtype == torch.float32 or a.shape[1] % 8 != 0 or not _tma_ok(a, w, out):
+            out = torch.empty(a.shape[0], w.shape[0] // (2 if gated else 1), dtype=out_dtype or a.dtype, device=a.device)
+        if a.dtype == torch.float32 or a.shape[1] % 8 != 0 or not _tma_ok(a, w, out) or (gated and w.shape[0] % 16 != 0):
             torch.ops.b200.gemm_simt(out, a, w, bias, EPI_CODES[act], act_params, None, None)
             if residual is not None:
                 out.add_(residual)
@@ -143,7 +150,7 @@ def gemm(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
         return out
     y = ref.gemm(a, w, bias, torch.float32 if act is not None else out_dtype)
     if act is not None:
-        y = ref.epilogue_activation(y, act, act_params).to(out_dtype or a.dtype)
+        y = (ref.epilogue_gate if gated else ref.epilogue_activation)(y, act, act_params).to(out_dtype or a.dtype)
     if residual is not None:
         y = (y.float() + residual.float()).to(a.dtype)
     if out is not None:
@@ -444,10 +451,13 @@ def decode_num_splits(batch: int, num_kv_heads: int, max_seq_len: int, row_tiles
 def paged_attention_decode(q, kv_cache, block_table, seq_lens, scale, *, out=None, kv_scales=None,
                            query_start_loc=None, max_q_len: int = 1, window: int = -1, softcap: float = 0.0,
                            sinks=None, lse_out=None, num_splits: int = 0, max_seq_len: int = 0, k_scale=1.0,
-                           v_scale=1.0, causal=True, workspace=None, alibi_slopes=None):
+                           v_scale=1.0, causal=True, workspace=None, alibi_slopes=None, distance_bias=None, gate=None,
+                           out_scale: float = 1.0):
     """Decode attention over the paged cache; ``q [T, Hq, D]``.  ``alibi_slopes [Hq]`` (f32) adds
-    ``slope * (kv position - query position)`` to the scores.  ``kv_cache``: the 5-D cache or a pair of ``kv_views``.
-    fp32 caches and 16-bit heads wider than 256 run on the CUDA cores."""
+    ``slope * (kv position - query position)`` to the scores, ``distance_bias [Hq, L]`` (f32) the entry of the distance (the
+    last one from L - 1 on).  The result is multiplied by ``out_scale`` and, with ``gate [T, Hq * Dv]`` (rows may be part of
+    wider ones), by its sigmoid; ``out``'s token rows may be part of wider ones too.  ``kv_cache``: the 5-D cache or a pair of
+    ``kv_views``.  fp32 caches and 16-bit heads wider than 256 run on the CUDA cores."""
     if _use_cuda(q):
         k, v = kv_views(kv_cache)
         out = torch.empty(q.shape[0], q.shape[1], v.shape[-1], dtype=q.dtype, device=q.device) if out is None else out
@@ -463,13 +473,14 @@ def paged_attention_decode(q, kv_cache, block_table, seq_lens, scale, *, out=Non
             ws = _decode_workspace(q.device, num_splits * q.shape[0] * q.shape[1] * (v.shape[-1] + 1))
         torch.ops.b200.paged_attention_decode(out, q, k, v, kv_scales, block_table, seq_lens, query_start_loc,
                                               scale, window, softcap, sinks, lse_out, ws, num_splits, B, max_q_len,
-                                              k_scale, v_scale, causal, alibi_slopes)
+                                              k_scale, v_scale, causal, alibi_slopes, distance_bias, gate, out_scale)
         return out
     B = seq_lens.shape[0]
     qsl = query_start_loc if query_start_loc is not None else torch.arange(B + 1, dtype=torch.int32, device=q.device)
     res = ref.paged_attention(q, kv_cache, block_table, seq_lens, qsl, scale, kv_scales=kv_scales, window=window,
                               softcap=softcap, sinks=sinks, k_scale=k_scale, v_scale=v_scale, causal=causal,
-                              return_lse=lse_out is not None, alibi_slopes=alibi_slopes)
+                              return_lse=lse_out is not None, alibi_slopes=alibi_slopes, distance_bias=distance_bias,
+                              gate=gate, out_scale=out_scale)
     if lse_out is not None:
         res, lse = res
         lse_out.copy_(lse)
@@ -481,8 +492,10 @@ def paged_attention_decode(q, kv_cache, block_table, seq_lens, scale, *, out=Non
 
 def paged_attention_prefill(q, kv_cache, block_table, seq_lens, query_start_loc, scale, *, out=None, kv_scales=None,
                             max_q_len: int = 0, window: int = -1, softcap: float = 0.0, sinks=None, lse_out=None,
-                            k_scale=1.0, v_scale=1.0, causal=True, max_seq_len: int = 0, alibi_slopes=None):
-    """Varlen prefill / chunked-prefill attention reading K, V from the paged cache."""
+                            k_scale=1.0, v_scale=1.0, causal=True, max_seq_len: int = 0, alibi_slopes=None,
+                            distance_bias=None, gate=None, out_scale: float = 1.0):
+    """Varlen prefill / chunked-prefill attention reading K, V from the paged cache (``distance_bias``, ``gate``,
+    ``out_scale`` as for decode)."""
     if _use_cuda(q):
         k, v = kv_views(kv_cache)
         out = torch.empty(q.shape[0], q.shape[1], v.shape[-1], dtype=q.dtype, device=q.device) if out is None else out
@@ -490,17 +503,19 @@ def paged_attention_prefill(q, kv_cache, block_table, seq_lens, query_start_loc,
         if k.dtype == q.dtype and q.dtype != torch.float32 and k.shape[-1] <= 192 and v.shape[-1] <= 128 and kv_scales is None:
             torch.ops.b200.attention_prefill(out, q, k, v, block_table, seq_lens, query_start_loc, None,
                                              scale, window, softcap, sinks, lse_out, B, max_q_len or q.shape[0], causal,
-                                             alibi_slopes)
+                                             alibi_slopes, distance_bias, gate, out_scale)
         else:
             # quantised caches / other head sizes: the split-KV kernel handles any query length in 16-row tiles
             paged_attention_decode(q, kv_cache, block_table, seq_lens, scale, out=out, kv_scales=kv_scales,
                                    query_start_loc=query_start_loc, max_q_len=max_q_len or q.shape[0], window=window,
                                    softcap=softcap, sinks=sinks, lse_out=lse_out, num_splits=1, k_scale=k_scale,
-                                   v_scale=v_scale, causal=causal, alibi_slopes=alibi_slopes)
+                                   v_scale=v_scale, causal=causal, alibi_slopes=alibi_slopes, distance_bias=distance_bias,
+                                   gate=gate, out_scale=out_scale)
         return out
     res = ref.paged_attention(q, kv_cache, block_table, seq_lens, query_start_loc, scale, kv_scales=kv_scales,
                               window=window, softcap=softcap, sinks=sinks, k_scale=k_scale, v_scale=v_scale,
-                              causal=causal, return_lse=lse_out is not None, alibi_slopes=alibi_slopes)
+                              causal=causal, return_lse=lse_out is not None, alibi_slopes=alibi_slopes,
+                              distance_bias=distance_bias, gate=gate, out_scale=out_scale)
     if lse_out is not None:
         res, lse = res
         lse_out.copy_(lse)
@@ -704,34 +719,38 @@ def moe_align_block_size(topk_ids, block_size: int, num_experts: int, expert_map
     return (sorted_ids, block_expert, total, inv) if want_inverse else (sorted_ids, block_expert, total)
 
 
-def moe_gather(x, sorted_ids, total_padded, topk: int):
-    """Rows of ``x [T,H]`` in expert-sorted order, zero rows for padding: ``[max_padded, H]``."""
+def moe_gather(x, sorted_ids, total_padded, topk: int, weights=None):
+    """Rows of ``x [T,H]`` in expert-sorted order, zero rows for padding: ``[max_padded, H]``.  ``weights [T, topk]`` (fp32):
+    each pair's row is multiplied by its weight."""
     if _use_cuda(x):
         out = torch.empty(sorted_ids.numel(), x.shape[1], dtype=x.dtype, device=x.device)
-        torch.ops.b200.moe_gather(out, x.contiguous(), sorted_ids, total_padded, topk)
+        torch.ops.b200.moe_gather(out, x.contiguous(), sorted_ids, total_padded, topk, weights)
         return out
     numel = x.shape[0] * topk
     sid = sorted_ids.long()
     valid = sid < numel
     out = torch.zeros(sid.numel(), x.shape[1], dtype=x.dtype)
     out[valid] = x[sid[valid] // topk]
+    if weights is not None:
+        out[valid] = (out[valid].float() * weights.reshape(-1)[sid[valid]][:, None]).to(x.dtype)
     return out
 
 
-def gemm_grouped(a, w, block_expert, total_padded, epi: int = 0):
-    """Per-row-block expert GEMM: ``a [R, K]`` (R multiple of 128), ``w [E, N, K]`` -> ``[R, N]`` (``N/2`` with the
-    SiLU-gate epilogue over row-interleaved gate/up weights).  ``epi``: a code of ``EPI_CODES``."""
+def gemm_grouped(a, w, block_expert, total_padded, epi: int = 0, act_params=None):
+    """Per-row-block expert GEMM: ``a [R, K]`` (R multiple of 128), ``w [E, N, K]`` -> ``[R, N]`` (``N/2`` with a gated
+    epilogue over row-interleaved gate/up weights).  ``epi``: a code of ``EPI_CODES``, ``act_params`` its numbers."""
+    gated = epi in EPI_GATES
     if _use_cuda(a):
-        n_out = w.shape[1] // 2 if epi == 1 else w.shape[1]
+        n_out = w.shape[1] // 2 if gated else w.shape[1]
         out = torch.empty(a.shape[0], n_out, dtype=a.dtype, device=a.device)
-        if a.dtype == torch.float32 or a.shape[1] % 8 != 0 or not _tma_ok(a, w, out):
-            torch.ops.b200.gemm_simt(out, a, w, None, epi, None, block_expert, total_padded)
+        if a.dtype == torch.float32 or a.shape[1] % 8 != 0 or not _tma_ok(a, w, out) or (gated and w.shape[1] % 16 != 0):
+            torch.ops.b200.gemm_simt(out, a, w, None, epi, act_params, block_expert, total_padded)
         else:
-            torch.ops.b200.gemm_grouped(out, a, w, block_expert, total_padded, epi)
+            torch.ops.b200.gemm_grouped(out, a, w, block_expert, total_padded, epi, act_params)
         return out
     R = a.shape[0]
     nblk = R // 128
-    n_out = w.shape[1] // 2 if epi == 1 else w.shape[1]
+    n_out = w.shape[1] // 2 if gated else w.shape[1]
     out = torch.zeros(R, n_out, dtype=a.dtype)
     valid_blocks = int(total_padded.item()) // 128
     for b in range(min(nblk, valid_blocks)):
@@ -742,8 +761,8 @@ def gemm_grouped(a, w, block_expert, total_padded, epi: int = 0):
         if epi == 1:
             y = (torch.nn.functional.silu(y[:, 0::2].float()) * y[:, 1::2].float()).to(a.dtype)
         elif epi > 1:
-            y = ref.epilogue_activation(ref.gemm(a[b * 128:(b + 1) * 128], w[e], out_dtype=torch.float32),
-                                        {v: k for k, v in EPI_CODES.items()}[epi], None).to(a.dtype)
+            fn = ref.epilogue_gate if gated else ref.epilogue_activation
+            y = fn(ref.gemm(a[b * 128:(b + 1) * 128], w[e], out_dtype=torch.float32), EPI_NAMES[epi], act_params).to(a.dtype)
         out[b * 128:(b + 1) * 128] = y
     return out
 
@@ -994,24 +1013,37 @@ def rope_angles(positions, inv_freq, tokens: int):
 
 
 def head_norm_rope(qkv, offsets, q_weight, k_weight, heads: int, dim: int, angles, kv_cache, slot_mapping, eps: float,
-                   one_plus: bool = False):
+                   one_plus: bool = False, whole_row: bool = False, interleaved: bool = False, q_temp=None):
     """Epilogue of a merged q | k | v product whose parts start at the columns ``offsets``: per-head RMS norm (``one_plus``:
-    weights stored around zero) and rotation of queries and keys, keys and values written to the paged cache
+    weights stored around zero; ``whole_row``: one norm over all heads, with a weight per head and entry) and rotation of
+    queries and keys (pairs (i, i + half), ``interleaved``: (2i, 2i + 1)), keys and values written to the paged cache
     (``kv_cache``: 5-D or a pair of ``kv_views``) at ``slot_mapping`` (-1: nowhere).  ``kv_cache=None``: the row holds queries
-    only.  Heads are ``len(weight)`` wide, of which ``dim`` are real; ``angles`` as ``rope_angles`` returns them.  Returns
-    ``q [T, heads, width]``."""
-    T, width = qkv.shape[0], q_weight.numel()
+    only.  Heads are as wide as their weights (of one head), of which ``dim`` are real; ``angles`` as ``rope_angles`` returns
+    them, or None.  ``q_temp = (positions, coef, every)`` multiplies queries by ``1 + coef * ln((p + 1) // every + 1)``.
+    Returns ``q [T, heads, width]``."""
+    T, width = qkv.shape[0], q_weight.numel() // (heads if whole_row else 1)
     k, v = kv_views(kv_cache) if kv_cache is not None else (None, None)
     if _use_cuda(qkv):
         q = torch.empty(T, heads, width, dtype=qkv.dtype, device=qkv.device)
-        torch.ops.b200.head_norm_rope(q, qkv, *offsets, k, v, q_weight, k_weight, dim, angles, slot_mapping, eps, one_plus)
+        torch.ops.b200.head_norm_rope(q, qkv, *offsets, k, v, q_weight, k_weight, dim, angles, slot_mapping, eps, one_plus,
+                                      whole_row, interleaved, *(q_temp or (None, 0.0, 1)))
         return q
 
-    def part(at, n, w):
-        x = ref.head_rms_norm(qkv[:, at: at + n * width].reshape(T, n, width), w, dim, eps, one_plus)
-        return ref.rotate_half_by(x, angles).to(qkv.dtype)
+    def part(at, n, w, temp=None):
+        x = qkv[:, at: at + n * width]
+        if whole_row:
+            x = ref.head_rms_norm(x[:, None], w, n * dim, eps, one_plus)
+        else:
+            x = ref.head_rms_norm(x.reshape(T, n, width), w, dim, eps, one_plus)
+        x = x.reshape(T, n, width)
+        if angles is not None:
+            x = ref.rotate_half_by(x, angles, interleaved)
+        if temp is not None:
+            pos, coef, every = temp
+            x = x * (1.0 + coef * torch.log(((pos[:T] + 1) // every).float() + 1.0))[:, None, None]
+        return x.to(qkv.dtype)
 
-    q = part(offsets[0], heads, q_weight)
+    q = part(offsets[0], heads, q_weight, q_temp)
     if k is not None:
         G, bs, dv = k.shape[2], k.shape[1], v.shape[-1]
         ok = slot_mapping[:T] >= 0

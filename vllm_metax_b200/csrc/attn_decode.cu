@@ -21,6 +21,7 @@
 // Replaces flash_attn_with_kvcache (vllm_metax/v1/attention/backends/flash_attn.py:1339-1355)
 // and the Triton unified_attention int8 path (triton_attn.py:688-725).
 #include <type_traits>
+#include "attn_score.cuh"
 #include "common.cuh"
 #include "ops.h"
 
@@ -170,6 +171,7 @@ __global__ void __launch_bounds__(kDecWarps * 32, (D <= 128 ? 2 : 1)) paged_deco
     }
   }
   __syncthreads();
+  const int rA0 = row0 + (lane >> 2);
   // Q fragments for all k-steps
   uint32_t qf[D / 16][4];
 #pragma unroll
@@ -179,6 +181,12 @@ __global__ void __launch_bounds__(kDecWarps * 32, (D <= 128 ? 2 : 1)) paged_deco
     const int c = 2 * ks + (mat >> 1);
     ldmatrix_x4(qf[ks], q_smem + r * S::kRowBytes + ((c ^ (r & 7)) * 16));
   }
+
+  // bias by distance: every key of a tile far enough away gets the last entry
+  const float* bsA = p.bias && rA0 < rows_total ? p.bias + (int64_t)(hk * g + rA0 % g) * p.bias_len : nullptr;
+  const float* bsB = p.bias && rA0 + 8 < rows_total ? p.bias + (int64_t)(hk * g + (rA0 + 8) % g) * p.bias_len : nullptr;
+  const float farA = bsA ? bsA[p.bias_len - 1] * 1.4426950408889634f : 0.f;
+  const float farB = bsB ? bsB[p.bias_len - 1] * 1.4426950408889634f : 0.f;
 
   // per-row causal limits: row r (token i = r / g) sees kv positions < limit
   const int rA = row0 + (lane >> 2), rB = rA + 8;
@@ -314,12 +322,17 @@ __global__ void __launch_bounds__(kDecWarps * 32, (D <= 128 ? 2 : 1)) paged_deco
         const int half = e >> 1;  // 0: row A, 1: row B
         float v = s[nt][e] * ksc[nt * 2 + (e & 1)];
         if (p.softcap > 0.f) {
-          v = p.softcap * tanhf(v * p.scale * ((KIND == 3) ? p.k_scale : 1.f) / p.softcap) * 1.4426950408889634f;
+          v = softcap_score(v * p.scale * ((KIND == 3) ? p.k_scale : 1.f), p.softcap) * 1.4426950408889634f;
         } else {
           v *= sm_scale_log2;
         }
         const int lim = half ? limB : limA, lo = half ? loB : loA;
         v += (half ? alB : alA) * (float)(col - (lim - 1));
+        if (p.bias) {
+          const float* bs = half ? bsB : bsA;
+          const int dist = lim - 1 - col;
+          v += (dist >= p.bias_len - 1 || bs == nullptr) ? (half ? farB : farA) : bs[max(0, dist)] * 1.4426950408889634f;
+        }
         if (col >= lim || col < lo) v = -INFINITY;
         s[nt][e] = v;
         mx[half] = fmaxf(mx[half], v);
@@ -405,6 +418,7 @@ __global__ void __launch_bounds__(kDecWarps * 32, (D <= 128 ? 2 : 1)) paged_deco
   }
   __syncthreads();
   const float out_scale = (KIND == 3) ? p.v_scale : 1.f;
+  const int64_t out_stride = p.out_stride ? p.out_stride : (int64_t)p.num_q_heads * dv;
   for (int idx = threadIdx.x; idx < 16 * D; idx += blockDim.x) {
     const int r = idx / D, c = idx % D;
     const int rr = row0 + r;
@@ -424,8 +438,8 @@ __global__ void __launch_bounds__(kDecWarps * 32, (D <= 128 ? 2 : 1)) paged_deco
     if (p.num_splits == 1) {
       float Lt = L;
       if (p.sinks) Lt += exp2f(p.sinks[hq] * 1.4426950408889634f - Ms);
-      const float v = Lt > 0.f ? acc / Lt * out_scale : 0.f;
-      reinterpret_cast<T*>(p.out)[((int64_t)tok * p.num_q_heads + hq) * dv + c] = from_f<T>(v);
+      const float v = (Lt > 0.f ? acc / Lt * out_scale : 0.f) * p.out_scale * gate_of<T>(p.gate, tok * p.gate_stride + hq * dv + c);
+      reinterpret_cast<T*>(p.out)[tok * out_stride + hq * dv + c] = from_f<T>(v);
       if (c == 0 && p.lse_out)
         p.lse_out[(int64_t)hq * p.total_tokens + tok] = Lt > 0.f ? (Ms * 0.6931471805599453f + logf(Lt)) : -INFINITY;
     } else {
@@ -441,7 +455,7 @@ template <typename T>
 __global__ void attn_split_reduce_kernel(T* __restrict__ out, float* __restrict__ lse_out,
                                          const float* __restrict__ part_out, const float* __restrict__ part_lse,
                                          const float* __restrict__ sinks, int num_splits, int total_tokens, int heads,
-                                         int D) {
+                                         int D, const void* gate, int64_t gate_stride, float out_scale, int64_t out_stride) {
   const int64_t row = blockIdx.x;  // token * heads + head
   const int hq = (int)(row % heads);
   const int64_t tok = row / heads;
@@ -458,7 +472,8 @@ __global__ void attn_split_reduce_kernel(T* __restrict__ out, float* __restrict_
     float acc = 0.f;
     for (int s = 0; s < num_splits; ++s)
       acc += part_out[(s * stride + row) * D + c] * __expf(part_lse[s * stride + row] - Ms);
-    out[row * D + c] = from_f<T>(L > 0.f ? acc / L : 0.f);
+    out[tok * out_stride + hq * D + c] =
+        from_f<T>((L > 0.f ? acc / L : 0.f) * out_scale * gate_of<T>(gate, tok * gate_stride + hq * D + c));
   }
   (void)Lk;
   if (threadIdx.x == 0 && lse_out) lse_out[(int64_t)hq * total_tokens + tok] = L > 0.f ? Ms + logf(L) : -INFINITY;
@@ -476,9 +491,10 @@ static void launch_decode(const DecodeParams& p, int batch, int max_q_len, cudaS
   kern<<<grid, kDecWarps * 32, S::kTotal, stream>>>(p);
   if (p.num_splits > 1) {
     const int64_t rows = (int64_t)p.total_tokens * p.num_q_heads;
+    const int dv = KIND == 0 ? p.dv : D;
     attn_split_reduce_kernel<T><<<(unsigned)rows, D <= 128 ? 128 : 256, 0, stream>>>(
-        (T*)p.out, p.lse_out, p.part_out, p.part_lse, p.sinks, p.num_splits, p.total_tokens, p.num_q_heads,
-        KIND == 0 ? p.dv : D);
+        (T*)p.out, p.lse_out, p.part_out, p.part_lse, p.sinks, p.num_splits, p.total_tokens, p.num_q_heads, dv, p.gate,
+        p.gate_stride, p.out_scale, p.out_stride ? p.out_stride : (int64_t)p.num_q_heads * dv);
   }
 }
 

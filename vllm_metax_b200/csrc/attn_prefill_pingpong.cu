@@ -28,6 +28,7 @@
 // Replaces flash_attn_varlen_func (vllm_metax/v1/attention/backends/flash_attn.py:1302-1322,
 // mla/prefill/flash_attn.py:157-163).
 #include <type_traits>
+#include "attn_score.cuh"
 #include "common.cuh"
 #include "ptx_sm100.cuh"
 #include "tma_host.h"
@@ -284,7 +285,9 @@ attn_prefill_pp_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     const int lo = (p.window > 0) ? max(0, lim - p.window) : 0;
     const float sl2 = p.scale * 1.4426950408889634f;
     const uint32_t lane_base = ((uint32_t)(quarter * 32)) << 16;
-    const bool plain = !(p.softcap > 0.f) && p.alibi_slopes == nullptr;
+    const bool plain = !(p.softcap > 0.f) && p.alibi_slopes == nullptr && p.bias == nullptr;
+    const float* bias = p.bias != nullptr ? p.bias + (int64_t)hq * p.bias_len : nullptr;      // by distance
+    const float bias_far = bias != nullptr ? bias[p.bias_len - 1] * 1.4426950408889634f : 0.f;
     const float alibi2 = (p.alibi_slopes && row_valid) ? p.alibi_slopes[hq] * 1.4426950408889634f : 0.f;
     const float mul = plain ? sl2 : 1.f;            // scores are kept raw on the plain path
     const int n_mine = t ? n_b : n_a;
@@ -310,9 +313,15 @@ attn_prefill_pp_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       if (!plain) {
 #pragma unroll
         for (int i = 0; i < BN; ++i) {
-          const float base =
-              (p.softcap > 0.f) ? p.softcap * tanhf(s[i] * p.scale / p.softcap) * 1.4426950408889634f : s[i] * sl2;
-          s[i] = base + alibi2 * (float)(t0 + i - pos);
+          const float base = (p.softcap > 0.f) ? softcap_score(s[i] * p.scale, p.softcap) * 1.4426950408889634f : s[i] * sl2;
+          s[i] = base + alibi2 * (float)(t0 + i - pos) + bias_far;
+        }
+        if (bias != nullptr && pos - (t0 + BN - 1) < p.bias_len - 1) {      // some keys of the tile are near
+#pragma unroll
+          for (int i = 0; i < BN; ++i) {
+            const int dist = max(0, pos - (t0 + i));
+            if (dist < p.bias_len - 1) s[i] = fmaf(__ldg(bias + dist), 1.4426950408889634f, s[i] - bias_far);
+          }
         }
       }
       if ((t0 + BN > lim) || (t0 < lo)) {
@@ -375,7 +384,9 @@ attn_prefill_pp_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     float l_tot = l_run;
     const float m_safe = (m_run == -INFINITY) ? 0.f : m_run;
     if (p.sinks && row_valid) l_tot += exp2f(p.sinks[hq] * 1.4426950408889634f - m_safe);
-    if (l_tot > 0.f) o_acc_scale = 1.f / l_tot;
+    if (l_tot > 0.f) o_acc_scale = p.out_scale / l_tot;
+    const int64_t out_stride = p.out_stride ? p.out_stride : (int64_t)p.num_q_heads * p.dv;
+    const T* gate = p.gate != nullptr ? reinterpret_cast<const T*>(p.gate) + (int64_t)(q_begin + tok) * p.gate_stride + hq * p.dv : nullptr;
     if (ok && n_mine > 0) {
       if (!mbar_wait(&o_done[t], (n_mine - 1) & 1)) {
         report_status(p.status, kWaitTimeout, 52, n_mine, t);
@@ -384,7 +395,7 @@ attn_prefill_pp_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       tc_fence_after_sync();
     }
     if (ok && n_mine > 0) {
-      T* dst = reinterpret_cast<T*>(p.out) + ((int64_t)(q_begin + tok) * p.num_q_heads + hq) * p.dv;
+      T* dst = reinterpret_cast<T*>(p.out) + (q_begin + tok) * out_stride + hq * p.dv;
 #pragma unroll 1
       for (int c = 0; c < DV; c += 32) {
         uint32_t v[32];
@@ -396,13 +407,19 @@ attn_prefill_pp_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
             float f[8];
 #pragma unroll
             for (int i = 0; i < 8; ++i) f[i] = __uint_as_float(v[g8 * 8 + i]) * o_acc_scale;
+            if (gate != nullptr && c + g8 * 8 < p.dv) {
+              float z[8];
+              unpack8<T>(*reinterpret_cast<const uint4*>(gate + c + g8 * 8), z);
+#pragma unroll
+              for (int i = 0; i < 8; ++i) f[i] *= __fdividef(1.f, 1.f + __expf(-z[i]));
+            }
             if (c + g8 * 8 < p.dv) *reinterpret_cast<uint4*>(dst + c + g8 * 8) = pack8<T>(f);
           }
         }
       }
     } else if (ok && row_valid) {
       // a row whose tile sees no key at all (empty context): zeros
-      T* dst = reinterpret_cast<T*>(p.out) + ((int64_t)(q_begin + tok) * p.num_q_heads + hq) * p.dv;
+      T* dst = reinterpret_cast<T*>(p.out) + (q_begin + tok) * out_stride + hq * p.dv;
       for (int c = 0; c < p.dv; c += 8) *reinterpret_cast<uint4*>(dst + c) = make_uint4(0, 0, 0, 0);
     }
     if (ok && row_valid && p.lse_out)

@@ -25,6 +25,7 @@
 // Replaces flash_attn_varlen_func (vllm_metax/v1/attention/backends/flash_attn.py:1302-1322,
 // mla/prefill/flash_attn.py:157-163).
 #include <type_traits>
+#include "attn_score.cuh"
 #include "common.cuh"
 #include "ptx_sm100.cuh"
 #include "tma_host.h"
@@ -263,7 +264,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     bool ok = true;
     const float alibi2 = (p.alibi_slopes && row_valid) ? p.alibi_slopes[hq] * 1.4426950408889634f : 0.f;
     auto fx = [&](float s, int col) -> float {
-      const float base = (p.softcap > 0.f) ? p.softcap * tanhf(s * p.scale / p.softcap) * 1.4426950408889634f : s * sl2;
+      const float base = (p.softcap > 0.f) ? softcap_score(s * p.scale, p.softcap) * 1.4426950408889634f : s * sl2;
       return base + alibi2 * (float)(col - pos);     // ALiBi bias (0 without slopes)
     };
     for (int j = 0; j < n_tiles; ++j) {

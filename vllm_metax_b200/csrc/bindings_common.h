@@ -62,6 +62,52 @@ inline PagedViews paged_views(const Tensor& k, const Tensor& v) {
   return {k.size(0), k.stride(0), (int)k.size(1), (int)k.size(2), (int)k.size(3), (int)v.size(3)};
 }
 
+// The sequences of a step and their state slots.
+struct StepRefs {
+  const int* qsl; const int* idx; const int* init;
+  int batch;
+};
+inline StepRefs step_refs(const Tensor& qsl, const optional<Tensor>& idx, const optional<Tensor>& init) {
+  TORCH_CHECK(qsl.scalar_type() == at::kInt && qsl.is_contiguous());
+  const int64_t B = qsl.numel() - 1;
+  for (const auto* x : {&idx, &init})
+    if (x->has_value()) TORCH_CHECK((*x)->scalar_type() == at::kInt && (*x)->is_contiguous() && (*x)->numel() >= B);
+  return {qsl.data_ptr<int>(), ptr<int>(idx), ptr<int>(init), (int)B};
+}
+
+inline int device_sms(const Tensor& t) {
+  static int sms[64] = {};
+  const int d = t.get_device();
+  if (sms[d] == 0) cudaDeviceGetAttribute(&sms[d], cudaDevAttrMultiProcessorCount, d);
+  return sms[d];
+}
+
+// Output rows, distance bias, output gate and factor of an attention call (DecodeParams, PrefillParams).
+template <typename P>
+inline void attn_extras(P& p, const Tensor& out, const optional<Tensor>& distance_bias, const optional<Tensor>& gate,
+                        double out_scale) {
+  const int64_t H = out.size(1), D = out.size(2), unit = 16 / (int64_t)out.element_size();
+  auto rows_ok = [&](const Tensor& t) {
+    return t.stride(0) % unit == 0 && reinterpret_cast<uintptr_t>(t.data_ptr()) % 16 == 0;
+  };
+  TORCH_CHECK(out.dim() == 3 && out.stride(2) == 1 && (out.size(1) == 1 || out.stride(1) == D) && (D % unit != 0 || rows_ok(out)),
+              "attention output: packed heads, token rows that start on 16 bytes");
+  p.out_stride = out.stride(0);
+  p.out_scale = (float)out_scale;
+  if (distance_bias.has_value()) {
+    TORCH_CHECK(distance_bias->dim() == 2 && distance_bias->is_contiguous() && distance_bias->size(0) == H &&
+                distance_bias->size(1) > 0 && distance_bias->scalar_type() == at::kFloat, "distance bias: fp32 [heads, distances]");
+    p.bias = distance_bias->template data_ptr<float>();
+    p.bias_len = (int)distance_bias->size(1);
+  }
+  if (gate.has_value()) {
+    TORCH_CHECK(gate->dim() == 2 && gate->stride(1) == 1 && gate->size(0) == out.size(0) && gate->size(1) == H * D &&
+                gate->scalar_type() == out.scalar_type() && (D % unit != 0 || rows_ok(*gate)), "attention gate: [tokens, heads * size]");
+    p.gate = gate->data_ptr();
+    p.gate_stride = gate->stride(0);
+  }
+}
+
 // One status word per device, zero-initialised on first use.
 inline Tensor& status_tensor(int device) {
   static std::vector<Tensor> words(64);

@@ -15,13 +15,16 @@ b200::Epi make_epi(const Tensor& out, const Tensor& a, int64_t act, const option
   TORCH_CHECK(act >= 0 && act <= b200::kEpiLast, "unknown epilogue ", act);
   int code = (int)act;
   if (out.scalar_type() != a.scalar_type()) {
-    TORCH_CHECK(out.scalar_type() == at::kFloat && act != 1, "the output is of the operands' type or fp32");
+    TORCH_CHECK(out.scalar_type() == at::kFloat && !b200::epi_is_gate((int)act), "the output is of the operands' type or fp32");
     code |= b200::kEpiF32;
   }
   const float* prm = nullptr;
-  if (act == b200::kEpiXielu || act == b200::kEpiDecay) {
+  const int64_t need = act == b200::kEpiXielu || act == b200::kEpiClampGate ? 2
+                       : act == b200::kEpiDecay || act == b200::kEpiSoftcap ? 1
+                       : act == b200::kEpiSoftplusDecay ? out.size(-1) : 0;
+  if (need > 0) {
     TORCH_CHECK(act_params.has_value() && act_params->scalar_type() == at::kFloat && act_params->is_contiguous() &&
-                act_params->numel() == (act == b200::kEpiXielu ? 2 : 1), "the epilogue needs its fp32 parameters");
+                act_params->numel() == need, "the epilogue needs its fp32 parameters");
     prm = act_params->data_ptr<float>();
   }
   return b200::Epi(code, prm);
@@ -35,9 +38,10 @@ void gemm(Tensor& out, const Tensor& a, const Tensor& w, const optional<Tensor>&
   const int M = a.size(0), K = a.size(1), N = w.size(0);
   const b200::Epi epi_arg = make_epi(out, a, act, act_params);
   const int epi = epi_arg.code;
+  const bool gate = b200::epi_is_gate(epi);
   TORCH_CHECK(epi < 2 || !residual.has_value(), "gemm: an activation or an fp32 output takes no residual");
-  TORCH_CHECK(w.size(1) == K && out.size(0) == M && out.size(1) == (epi == 1 ? N / 2 : N), "gemm shape mismatch");
-  TORCH_CHECK(epi != 1 || (!residual.has_value() && N % 16 == 0), "gated epilogue: no residual, N % 16 == 0");
+  TORCH_CHECK(w.size(1) == K && out.size(0) == M && out.size(1) == (gate ? N / 2 : N), "gemm shape mismatch");
+  TORCH_CHECK(!gate || (!residual.has_value() && N % 16 == 0), "gated epilogue: no residual, N % 16 == 0");
   TORCH_CHECK(K % 8 == 0 && a.stride(0) % 8 == 0 && w.stride(0) % 8 == 0 && out.stride(0) % 8 == 0,
               "gemm: K and row pitches must be multiples of 8 elements");
   TORCH_CHECK(a.scalar_type() == w.scalar_type(), "gemm dtype mismatch");
@@ -174,11 +178,14 @@ void moe_align(Tensor& sorted_ids, Tensor& block_expert, Tensor& total_padded, c
                   sorted_ids.numel(), cur_stream());
 }
 
-void moe_gather(Tensor& out, const Tensor& x, const Tensor& sorted_ids, const Tensor& total_padded, int64_t topk) {
+void moe_gather(Tensor& out, const Tensor& x, const Tensor& sorted_ids, const Tensor& total_padded, int64_t topk,
+                const optional<Tensor>& weights) {
   TORCH_CHECK(x.is_contiguous() && out.is_contiguous());
+  if (weights.has_value())
+    TORCH_CHECK(weights->is_contiguous() && weights->scalar_type() == at::kFloat && weights->numel() == x.size(0) * topk);
   const c10::cuda::CUDAGuard guard(x.device());
   b200::moe_gather(out.data_ptr(), x.data_ptr(), sorted_ids.data_ptr<int>(), total_padded.data_ptr<int>(),
-                   out.size(0), x.size(0) * topk, topk, x.size(1), dtype_code(x), cur_stream());
+                   ptr<float>(weights), out.size(0), x.size(0) * topk, topk, x.size(1), dtype_code(x), cur_stream());
 }
 
 void moe_combine(Tensor& out, const Tensor& y, const Tensor& weights, const Tensor& inv_pos,
@@ -202,12 +209,14 @@ void moe_sum(Tensor& out, const Tensor& in) {
 }
 
 void gemm_grouped(Tensor& out, const Tensor& a, const Tensor& w, const Tensor& block_expert,
-                  const Tensor& total_padded, int64_t act) {
-  on_device_of(a, {&out, &w, &block_expert, &total_padded});
-  const b200::Epi epi = make_epi(out, a, act, c10::nullopt);
+                  const Tensor& total_padded, int64_t act, const optional<Tensor>& act_params) {
+  on_device_of(a, {&out, &w, &block_expert, &total_padded}, {&act_params});
+  const b200::Epi epi = make_epi(out, a, act, act_params);
+  const bool gate = b200::epi_is_gate((int)act);
+  TORCH_CHECK(!gate || w.size(1) % 16 == 0, "gated epilogue: N % 16 == 0");
   TORCH_CHECK(a.dim() == 2 && w.dim() == 3 && a.stride(1) == 1 && w.is_contiguous() && out.stride(1) == 1);
   TORCH_CHECK(a.size(0) % 128 == 0 && a.size(1) == w.size(2) && a.size(1) % 8 == 0 && a.stride(0) % 8 == 0);
-  TORCH_CHECK(out.size(0) == a.size(0) && out.size(1) == (act == 1 ? w.size(1) / 2 : w.size(1)));
+  TORCH_CHECK(out.size(0) == a.size(0) && out.size(1) == (gate ? w.size(1) / 2 : w.size(1)));
   const c10::cuda::CUDAGuard guard(a.device());
   b200::gemm_grouped(a.data_ptr(), a.size(0), a.stride(0), w.data_ptr(), w.size(0), w.size(1), w.size(2),
                      out.data_ptr(), out.stride(0), block_expert.data_ptr<int>(), total_padded.data_ptr<int>(), epi,
@@ -219,9 +228,12 @@ void attention_prefill(Tensor& out, const Tensor& q, const Tensor& k_src, const 
                        const Tensor& query_start_loc, const optional<Tensor>& kv_start_loc, double scale,
                        int64_t window, double softcap, const optional<Tensor>& sinks,
                        const optional<Tensor>& lse_out, int64_t batch, int64_t max_q_len, bool causal,
-                       const optional<Tensor>& alibi_slopes) {
+                       const optional<Tensor>& alibi_slopes, const optional<Tensor>& distance_bias,
+                       const optional<Tensor>& gate, double out_scale) {
   TORCH_CHECK(q.dim() == 3 && q.stride(2) == 1 && q.stride(1) == q.size(2));
+  on_device_of(q, {&out, &k_src, &query_start_loc}, {&v_src, &distance_bias, &gate});
   b200::PrefillParams p{};
+  attn_extras(p, out, distance_bias, gate, out_scale);
   p.alibi_slopes = ptr<float>(alibi_slopes);
   const int T = q.size(0), Hq = q.size(1), DQK = q.size(2);
   const bool paged = block_table.has_value();
@@ -278,7 +290,7 @@ void attention_prefill(Tensor& out, const Tensor& q, const Tensor& k_src, const 
   p.causal = causal;
   p.paged = paged;
   p.status = reinterpret_cast<b200::StatusWord*>(status_ptr(q));
-  TORCH_CHECK(out.is_contiguous() && out.size(-1) == DV);
+  TORCH_CHECK(out.size(0) == T && out.size(1) == Hq && out.size(2) == DV);
   TORCH_CHECK(q.stride(0) % 8 == 0, "q token stride must be a multiple of 8 elements");
   const c10::cuda::CUDAGuard guard(q.device());
   // B200_ATTN_PREFILL_SINGLE=1 selects the one-tile-per-CTA kernel (P through shared memory)
@@ -286,7 +298,8 @@ void attention_prefill(Tensor& out, const Tensor& q, const Tensor& k_src, const 
     const char* e = std::getenv("B200_ATTN_PREFILL_SINGLE");
     return e != nullptr && std::atoi(e) != 0;
   }();
-  const bool packed = paged ? DQK == DV && (DQK == 64 || DQK == 128)                // the one-tile kernel wants that
+  const bool extras = distance_bias.has_value() || gate.has_value() || out_scale != 1.0 || !out.is_contiguous();
+  const bool packed = extras ? false : paged ? DQK == DV && (DQK == 64 || DQK == 128)                // the one-tile kernel wants that
                             : p.k_head_stride == DQK && p.v_head_stride == DV;
   const int rc = single_tile && packed
                      ? b200::attention_prefill(p, q.data_ptr(), q.stride(0), kptr, vptr, ks, vs, total_kv, DQK, DV,
@@ -322,14 +335,14 @@ void gemm_simt(Tensor& out, const Tensor& a, const Tensor& w, const optional<Ten
   const bool grouped = block_expert.has_value();
   TORCH_CHECK(a.dim() == out.dim() && (grouped ? (a.dim() == 2 && w.dim() == 3) : w.dim() == a.dim()));
   TORCH_CHECK(a.stride(-1) == 1 && w.stride(-1) == 1 && out.stride(-1) == 1 && a.scalar_type() == w.scalar_type());
-  TORCH_CHECK(act != 1, "the gated epilogue is not built on the CUDA cores");
+  const bool gate = b200::epi_is_gate((int)act);
   b200::SimtGemmParams p{};
   p.A = a.data_ptr(); p.W = w.data_ptr(); p.C = out.data_ptr();
   p.bias = ptr(bias);
   const bool b3 = a.dim() == 3;
   p.batches = b3 ? a.size(0) : 1;
   p.M = a.size(-2); p.K = a.size(-1); p.N = w.size(-2);
-  TORCH_CHECK(w.size(-1) == p.K && out.size(-2) == p.M && out.size(-1) == p.N && (!b3 || (w.size(0) == p.batches && out.size(0) == p.batches)));
+  TORCH_CHECK(w.size(-1) == p.K && out.size(-2) == p.M && out.size(-1) == (gate ? p.N / 2 : p.N) && (!gate || p.N % 2 == 0) && (!b3 || (w.size(0) == p.batches && out.size(0) == p.batches)));
   if (bias.has_value()) TORCH_CHECK(bias->numel() == p.N && bias->is_contiguous() && bias->scalar_type() == a.scalar_type());
   p.lda = a.stride(-2); p.ldw = w.stride(-2); p.ldc = out.stride(-2);
   p.a_batch = b3 ? a.stride(0) : 0; p.c_batch = b3 ? out.stride(0) : 0; p.w_batch = w.dim() == 3 ? w.stride(0) : 0;
@@ -436,17 +449,18 @@ TORCH_LIBRARY(b200, m) {
   m.def("topk_gating(Tensor(a!) weights, Tensor(b!) ids, Tensor gating, Tensor? bias, int mode, bool renorm, float scale) -> ()", &topk_gating);
   m.def("grouped_topk(Tensor(a!) weights, Tensor(b!) ids, Tensor gating, Tensor? bias, int n_group, int topk_group, bool sigmoid, bool renorm, float scale) -> ()", &grouped_topk);
   m.def("moe_align(Tensor(a!) sorted_ids, Tensor(b!) block_expert, Tensor(c!) total_padded, Tensor(d!)? inv_pos, Tensor topk_ids, Tensor? expert_map, int experts, int block) -> ()", &moe_align);
-  m.def("moe_gather(Tensor(a!) out, Tensor x, Tensor sorted_ids, Tensor total_padded, int topk) -> ()", &moe_gather);
+  m.def("moe_gather(Tensor(a!) out, Tensor x, Tensor sorted_ids, Tensor total_padded, int topk, Tensor? weights=None) -> ()", &moe_gather);
   m.def(
       "moe_combine(Tensor(a!) out, Tensor y, Tensor weights, Tensor inv_pos, Tensor? shared, Tensor? expert_ids=None, "
       "Tensor? through=None, int identity_from=0) -> ()",
       &moe_combine);
   m.def("moe_sum(Tensor(a!) out, Tensor inp) -> ()", &moe_sum);
-  m.def("gemm_grouped(Tensor(a!) out, Tensor a, Tensor w, Tensor block_expert, Tensor total_padded, int epi) -> ()", &gemm_grouped);
+  m.def("gemm_grouped(Tensor(a!) out, Tensor a, Tensor w, Tensor block_expert, Tensor total_padded, int epi, Tensor? act_params=None) -> ()", &gemm_grouped);
   m.def(
       "attention_prefill(Tensor(a!) out, Tensor q, Tensor k_src, Tensor? v_src, Tensor? block_table, "
       "Tensor? seq_lens, Tensor query_start_loc, Tensor? kv_start_loc, float scale, int window, float softcap, "
-      "Tensor? sinks, Tensor(b!)? lse_out, int batch, int max_q_len, bool causal, Tensor? alibi_slopes=None) -> ()",
+      "Tensor? sinks, Tensor(b!)? lse_out, int batch, int max_q_len, bool causal, Tensor? alibi_slopes=None, "
+      "Tensor? distance_bias=None, Tensor? gate=None, float out_scale=1.0) -> ()",
       &attention_prefill);
   m.def("get_status(int device) -> Tensor", &get_status);
 }

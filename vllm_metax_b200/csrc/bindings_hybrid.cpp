@@ -1,38 +1,9 @@
-// torch.ops.b200.* of the hybrid group: short convolutions, gated linear recurrences, latent attention of any sizes.
+// torch.ops.b200.* of the hybrid set: latent attention of any sizes, the post-norm boundary with a convolution, RG-LRU.
 #include "bindings_common.h"
 
 namespace {
 
 using namespace b200_bind;
-
-// x [T, C] (row pitch free), w [C, K], state [slots, K-1, C] (in / out), all of one dtype (bf16 / fp16 / fp32)
-void causal_conv1d(Tensor& out, const Tensor& x, const Tensor& w, const optional<Tensor>& bias,
-                   const optional<Tensor>& state, const Tensor& query_start_loc, const optional<Tensor>& state_idx,
-                   const optional<Tensor>& has_initial, bool silu) {
-  on_device_of(x, {&out, &w, &query_start_loc}, {&bias, &state, &state_idx, &has_initial});
-  TORCH_CHECK(x.dim() == 2 && x.stride(1) == 1 && out.is_contiguous() && out.sizes() == x.sizes() &&
-              out.scalar_type() == x.scalar_type());
-  const int64_t T = x.size(0), C = x.size(1), K = w.size(1);
-  TORCH_CHECK(w.dim() == 2 && w.size(0) == C && w.is_contiguous() && w.scalar_type() == x.scalar_type());
-  if (bias.has_value()) TORCH_CHECK(bias->is_contiguous() && bias->numel() == C && bias->scalar_type() == x.scalar_type());
-  TORCH_CHECK(query_start_loc.scalar_type() == at::kInt && query_start_loc.is_contiguous());
-  const int64_t B = query_start_loc.numel() - 1;
-  if (state.has_value()) {
-    TORCH_CHECK(state_idx.has_value(), "a carry needs state indices");
-    TORCH_CHECK(state->is_contiguous() && state->dim() == 3 && state->size(1) == K - 1 && state->size(2) == C &&
-                state->scalar_type() == x.scalar_type());
-  }
-  if (state_idx.has_value()) TORCH_CHECK(state_idx->scalar_type() == at::kInt && state_idx->numel() >= B);
-  if (has_initial.has_value()) TORCH_CHECK(has_initial->scalar_type() == at::kInt && has_initial->numel() >= B);
-  const c10::cuda::CUDAGuard guard(x.device());
-  const int rc = b200::causal_conv1d(out.data_ptr(), x.data_ptr(), x.stride(0), w.data_ptr(),
-                                     bias.has_value() ? bias->data_ptr() : nullptr,
-                                     state.has_value() ? state->data_ptr() : nullptr, query_start_loc.data_ptr<int>(),
-                                     state_idx.has_value() ? state_idx->data_ptr<int>() : nullptr,
-                                     has_initial.has_value() ? has_initial->data_ptr<int>() : nullptr, (int)B, (int)T,
-                                     (int)C, (int)K, silu ? 1 : 0, dtype_code(x), cur_stream());
-  TORCH_CHECK(rc == 0, "causal_conv1d: kernel width must be 1..8");
-}
 
 // ------------------------------------------------------------------ MLA
 void mla_decode(Tensor& out, const Tensor& q, const Tensor& cache, const Tensor& block_table, const Tensor& seq_lens,
@@ -99,18 +70,6 @@ void gather_mla_cache(Tensor& dst, const Tensor& cache, const Tensor& block_tabl
 }
 
 // ------------------------------------------------------------------ post-norm residual + input convolution
-struct StepRefs {
-  const int* qsl; const int* idx; const int* init;
-  int batch;
-};
-StepRefs step_refs(const Tensor& qsl, const optional<Tensor>& idx, const optional<Tensor>& init) {
-  TORCH_CHECK(qsl.scalar_type() == at::kInt && qsl.is_contiguous());
-  const int64_t B = qsl.numel() - 1;
-  for (const auto* x : {&idx, &init})
-    if (x->has_value()) TORCH_CHECK((*x)->scalar_type() == at::kInt && (*x)->is_contiguous() && (*x)->numel() >= B);
-  return {qsl.data_ptr<int>(), ptr<int>(idx), ptr<int>(init), (int)B};
-}
-
 void residual_conv(Tensor& x_out, Tensor& h, const Tensor& y, const optional<Tensor>& x, const optional<Tensor>& gain,
                    const Tensor& w, const optional<Tensor>& carry, const Tensor& qsl, const optional<Tensor>& state_idx,
                    const optional<Tensor>& has_init, double eps) {
@@ -139,52 +98,6 @@ void residual_conv(Tensor& x_out, Tensor& h, const Tensor& y, const optional<Ten
 }
 
 // ------------------------------------------------------------------ recurrences
-int device_sms(const Tensor& t) {
-  static int sms[64] = {};
-  const int d = t.get_device();
-  if (sms[d] == 0) cudaDeviceGetAttribute(&sms[d], cudaDevAttrMultiProcessorCount, d);
-  return sms[d];
-}
-
-int64_t gla_scratch_floats(const Tensor& like, int64_t batch, int64_t heads, int64_t dim, int64_t vdim, int64_t max_query_len) {
-  const b200::GlaScratch g = b200::gla_scratch((int)batch, (int)like.size(0), (int)heads, (int)dim, (int)vdim,
-                                               (int)max_query_len, device_sms(like));
-  return g.raw + g.segments + 4 * ((g.raw + g.segments) > 0);
-}
-
-// qkvg [T, >= ...]: q, k at [q_off, k_off], v at v_off, gate at g_off (each heads * size wide)
-void gla_recurrent(Tensor& out, Tensor& state, const Tensor& qkvg, int64_t q_off, int64_t k_off, int64_t v_off,
-                   int64_t g_off, const Tensor& alpha, const Tensor& norm_w,
-                   const optional<Tensor>& scratch, const Tensor& qsl, const optional<Tensor>& state_idx,
-                   const optional<Tensor>& has_init, double scale, double eps, int64_t max_query_len) {
-  on_device_of(qkvg, {&out, &state, &alpha, &norm_w, &qsl}, {&scratch, &state_idx, &has_init});
-  TORCH_CHECK(state.dim() == 4 && state.is_contiguous() && state.scalar_type() == at::kFloat);
-  const int64_t T = qkvg.size(0), H = state.size(1), D = state.size(2), V = state.size(3);
-  TORCH_CHECK(qkvg.dim() == 2 && qkvg.stride(1) == 1 && out.is_contiguous() && out.size(0) == T && out.size(1) == H * V &&
-              out.scalar_type() == qkvg.scalar_type());
-  const int64_t W = qkvg.size(1);
-  TORCH_CHECK(q_off + H * D <= W && k_off + H * D <= W && v_off + H * V <= W && g_off + H * V <= W);
-  TORCH_CHECK(alpha.is_contiguous() && alpha.scalar_type() == at::kFloat && alpha.numel() == T * H * D);
-  TORCH_CHECK(norm_w.numel() == V && norm_w.scalar_type() == qkvg.scalar_type());
-  const StepRefs s = step_refs(qsl, state_idx, has_init);
-  const int sms = device_sms(qkvg);
-  const int64_t need = gla_scratch_floats(qkvg, s.batch, H, D, V, max_query_len);
-  if (need > 0)
-    TORCH_CHECK(scratch.has_value() && scratch->scalar_type() == at::kFloat && scratch->numel() >= need &&
-                reinterpret_cast<uintptr_t>(scratch->data_ptr()) % 16 == 0, "gla scratch");
-  b200::GlaParams p{};
-  p.qkvg = qkvg.data_ptr(); p.row_stride = qkvg.stride(0);
-  p.q_off = q_off; p.k_off = k_off; p.v_off = v_off; p.g_off = g_off;
-  p.alpha = alpha.data_ptr<float>(); p.norm_w = norm_w.data_ptr(); p.state = state.data_ptr<float>();
-  p.out = out.data_ptr();
-  p.qsl = s.qsl; p.state_idx = s.idx; p.has_init = s.init; p.batch = s.batch; p.tokens = T;
-  p.heads = H; p.dim = D; p.vdim = V;
-  p.scale = (float)scale; p.eps = (float)eps;
-  const c10::cuda::CUDAGuard guard(qkvg.device());
-  TORCH_CHECK(b200::gla_recurrent(p, ptr<float>(scratch), (int)max_query_len, sms, dtype_code(qkvg), cur_stream()) == 0,
-              "gla_recurrent: key dimension up to 256");
-}
-
 int64_t rglru_chunk() { return b200::rglru_chunk(); }
 
 void rglru_scan(Tensor& out, Tensor& state, Tensor& gates, const Tensor& u, const Tensor& y, const Tensor& r_bias,
@@ -256,13 +169,10 @@ void latent_rope(Tensor& dst, const Tensor& src, const Tensor& inv_freq, const T
 
 TORCH_LIBRARY_FRAGMENT(b200, m) {
   m.def("residual_conv(Tensor(a!) x_out, Tensor(b!) h, Tensor y, Tensor? x, Tensor? gain, Tensor w, Tensor(c!)? carry, Tensor query_start_loc, Tensor? state_idx, Tensor? has_initial, float eps) -> ()", &residual_conv);
-  m.def("gla_scratch_floats(Tensor like, int batch, int heads, int dim, int vdim, int max_query_len) -> int", &gla_scratch_floats);
-  m.def("gla_recurrent(Tensor(a!) out, Tensor(b!) state, Tensor qkvg, int q_off, int k_off, int v_off, int g_off, Tensor alpha, Tensor norm_w, Tensor(c!)? scratch, Tensor query_start_loc, Tensor? state_idx, Tensor? has_initial, float scale, float eps, int max_query_len) -> ()", &gla_recurrent);
   m.def("rglru_chunk() -> int", &rglru_chunk);
   m.def("rglru_scan(Tensor(a!) out, Tensor(b!) state, Tensor(c!) gates, Tensor u, Tensor y, Tensor r_bias, Tensor i_bias, Tensor decay, int block_width, Tensor(d!)? summary, Tensor query_start_loc, Tensor? state_idx, Tensor? has_initial, int max_query_len) -> ()", &rglru_scan);
   m.def("latent_insert(Tensor(a!) cq, Tensor(b!) cache, Tensor a, int q_off, int kv_off, Tensor q_w, Tensor kv_w, int rot_dim, Tensor inv_freq, Tensor positions, Tensor slot_mapping, float eps) -> ()", &latent_insert);
   m.def("latent_rope(Tensor(a!) dst, Tensor src, Tensor inv_freq, Tensor positions, int rot_dim, int pad) -> ()", &latent_rope);
-  m.def("causal_conv1d(Tensor(a!) out, Tensor x, Tensor w, Tensor? bias, Tensor(b!)? state, Tensor query_start_loc, Tensor? state_idx, Tensor? has_initial, bool silu) -> ()", &causal_conv1d);
   m.def("mla_decode(Tensor(a!) out, Tensor q, Tensor cache, Tensor block_table, Tensor seq_lens, Tensor? query_start_loc, Tensor? topk_indices, float scale, Tensor(b!)? lse_out, Tensor(c!)? workspace, int num_splits, int impl=1, int window=0) -> ()", &mla_decode);
   m.def("gather_mla_cache(Tensor(a!) dst, Tensor cache, Tensor block_table, Tensor cu_seq_lens, Tensor? seq_starts) -> ()", &gather_mla_cache);
 }

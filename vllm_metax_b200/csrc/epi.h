@@ -3,9 +3,12 @@
 
 namespace b200 {
 
-constexpr int kEpiGelu = 2, kEpiGeluTanh = 3, kEpiXielu = 4, kEpiDecay = 5, kEpiRelu2 = 6;
-constexpr int kEpiLast = kEpiRelu2;
+constexpr int kEpiSiluGate = 1, kEpiGelu = 2, kEpiGeluTanh = 3, kEpiXielu = 4, kEpiDecay = 5, kEpiRelu2 = 6;
+constexpr int kEpiGeluTanhGate = 7, kEpiClampGate = 8, kEpiSoftplusDecay = 9, kEpiSoftcap = 10;
+constexpr int kEpiLast = kEpiSoftcap;
 constexpr int kEpiActMask = 0xf, kEpiF32 = 0x10;
+// (gate, up) in adjacent columns, half as many columns come out
+constexpr bool epi_is_gate(int code) { return code == kEpiSiluGate || code == kEpiGeluTanhGate || code == kEpiClampGate; }
 
 struct Epi {
   int code;

@@ -4,7 +4,8 @@
 //
 // Epilogue codes (``Epi::code``): 0 plain, 1 SiLU-gate over interleaved pairs, 2 gelu (erf), 3 gelu (tanh), 4 xIELU with
 // the two numbers ``act[0], act[1]`` (the quadratic and the exponential coefficient), 5 a decay sigmoid(x)^act[0],
-// 6 relu(x)^2; kEpiF32 added to a code makes the output matrix fp32 (``C`` then points at floats and ``ldc`` counts floats).
+// 6 relu(x)^2, 9 a decay exp(-act[column] softplus(x)), 10 act[0] tanh(x / act[0]); gates over interleaved pairs beside 1:
+// 7 gelu_tanh(gate) * up, 8 g sigmoid(act[1] g) (u + 1) with g = min(gate, act[0]), u = up held within +-act[0].  kEpiF32 added to a code makes the output matrix fp32 (``C`` then points at floats and ``ldc`` counts floats).
 #pragma once
 #include "common.cuh"
 #include "epi.h"
@@ -42,10 +43,44 @@ __device__ __forceinline__ float decay_of(float x, float e) {
   return expf((fminf(x, 0.f) - log1pf(expf(-fabsf(x)))) * e);
 }
 
+// exp(-rate softplus(x))
+__device__ __forceinline__ float softplus_decay_of(float x, float rate) {
+  return expf(-rate * (fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)))));
+}
+
+// c tanh(x / c) with an absolute error of some 1e-7 c
+__device__ __forceinline__ float softcap_of(float x, float c) {
+  return c - 2.f * c * __fdividef(1.f, 1.f + __expf(2.f * x / c));
+}
+
+__device__ __forceinline__ float epi_gate(float g, float u, int act, const float* __restrict__ prm) {
+  if (act == kEpiGeluTanhGate) return epi_activate16(g, kEpiGeluTanh, prm) * u;
+  if (act == kEpiClampGate) {
+    const float lim = __ldg(prm);
+    g = fminf(g, lim);
+    u = fminf(fmaxf(u, -lim), lim);
+    return __fdividef(g, 1.f + __expf(-__ldg(prm + 1) * g)) * (u + 1.f);
+  }
+  return __fdividef(g, 1.f + __expf(-g)) * u;
+}
+
+// The same for fp32 results.
+__device__ __forceinline__ float epi_gate32(float g, float u, int act, const float* __restrict__ prm) {
+  if (act == kEpiGeluTanhGate) return 0.5f * g * (1.f + tanhf(0.79788456080286536f * (g + 0.044715f * g * g * g))) * u;
+  if (act == kEpiClampGate) {
+    const float lim = __ldg(prm);
+    g = fminf(g, lim);
+    return g / (1.f + expf(-__ldg(prm + 1) * g)) * (fminf(fmaxf(u, -lim), lim) + 1.f);
+  }
+  return g / (1.f + expf(-g)) * u;
+}
+
 // N elements at once: one branch on the activation outside the element loop (a branch per element multiplies the code of
 // the unrolled epilogue until it no longer fits the instruction cache).
+// Element i belongs to output column col0 + i * step (of n_cols; further ones are not stored).
 template <int N>
-__device__ __forceinline__ void epi_activate16_n(float (&f)[N], int act, const float* __restrict__ prm) {
+__device__ __forceinline__ void epi_activate16_n(float (&f)[N], int act, const float* __restrict__ prm, int col0, int step,
+                                                 int n_cols) {
   if (act == kEpiXielu) {
     const float cp = __ldg(prm), cn = __ldg(prm + 1);
 #pragma unroll
@@ -60,6 +95,13 @@ __device__ __forceinline__ void epi_activate16_n(float (&f)[N], int act, const f
   } else if (act == kEpiRelu2) {
 #pragma unroll
     for (int i = 0; i < N; ++i) f[i] = fmaxf(f[i], 0.f) * f[i];
+  } else if (act == kEpiSoftplusDecay) {
+#pragma unroll 4
+    for (int i = 0; i < N; ++i) f[i] = softplus_decay_of(f[i], __ldg(prm + min(col0 + i * step, n_cols - 1)));
+  } else if (act == kEpiSoftcap) {
+    const float c = __ldg(prm);
+#pragma unroll
+    for (int i = 0; i < N; ++i) f[i] = softcap_of(f[i], c);
   } else if (act == kEpiGelu) {
 #pragma unroll
     for (int i = 0; i < N; ++i) f[i] = 0.5f * f[i] * (1.f + erf_as(f[i] * 0.70710678118654752f));
@@ -69,7 +111,7 @@ __device__ __forceinline__ void epi_activate16_n(float (&f)[N], int act, const f
   }
 }
 
-__device__ __forceinline__ float epi_activate(float f, int act, const float* __restrict__ prm) {
+__device__ __forceinline__ float epi_activate(float f, int act, const float* __restrict__ prm, int col) {
   if (act == kEpiGelu) return 0.5f * f * (1.f + erff(f * 0.70710678118654752f));
   if (act == kEpiGeluTanh) return 0.5f * f * (1.f + tanhf(0.79788456080286536f * (f + 0.044715f * f * f * f)));
   if (act == kEpiXielu) {
@@ -78,13 +120,15 @@ __device__ __forceinline__ float epi_activate(float f, int act, const float* __r
   }
   if (act == kEpiDecay) return decay_of(f, __ldg(prm));
   if (act == kEpiRelu2) return fmaxf(f, 0.f) * f;
+  if (act == kEpiSoftplusDecay) return softplus_decay_of(f, __ldg(prm + col));
+  if (act == kEpiSoftcap) return __ldg(prm) * tanhf(f / __ldg(prm));
   return f;
 }
 
-// One element of an epilogue with an activation and / or an fp32 output matrix.
+// One element (output column col) of an epilogue with an activation and / or an fp32 output matrix.
 template <typename T>
-__device__ __forceinline__ void epi_store1(T* __restrict__ C, size_t idx, float f, const Epi& epi) {
-  f = epi_activate(f, epi.code & kEpiActMask, epi.act);
+__device__ __forceinline__ void epi_store1(T* __restrict__ C, size_t idx, float f, const Epi& epi, int col) {
+  f = epi_activate(f, epi.code & kEpiActMask, epi.act, col);
   if (epi.code & kEpiF32) reinterpret_cast<float*>(C)[idx] = f;
   else C[idx] = from_f<T>(f);
 }
@@ -92,8 +136,8 @@ __device__ __forceinline__ void epi_store1(T* __restrict__ C, size_t idx, float 
 // N tokens of one output feature (transposed tiles: lane = feature): element k goes to C[(tok0 + k) * ldc + feature].
 template <typename T, int N>
 __device__ __forceinline__ void epi_store_tokens(float (&f)[N], T* __restrict__ C, int feature, int tok0, int tokens, int ldc,
-                                                 const Epi& epi) {
-  epi_activate16_n<N>(f, epi.code & kEpiActMask, epi.act);
+                                                 int features, const Epi& epi) {
+  epi_activate16_n<N>(f, epi.code & kEpiActMask, epi.act, feature, 0, features);
   const size_t at = (size_t)tok0 * ldc + feature;
   if (epi.code & kEpiF32) {
 #pragma unroll
@@ -103,6 +147,19 @@ __device__ __forceinline__ void epi_store_tokens(float (&f)[N], T* __restrict__ 
 #pragma unroll
     for (int k = 0; k < N; ++k)
       if (tok0 + k < tokens) C[at + (size_t)k * ldc] = from_f<T>(f[k]);
+  }
+}
+
+// Tokens of one output feature under a gated epilogue: even lanes hold gates, odd lanes the ups beside them.  The whole warp
+// calls this.
+template <typename T, int N>
+__device__ __forceinline__ void epi_gate_tokens(const float (&f)[N], T* __restrict__ C, int feature, int tok0, int tokens, int ldc,
+                                                int features, const Epi& epi) {
+  const bool mine = (threadIdx.x & 1) == 0 && feature < features;
+#pragma unroll
+  for (int k = 0; k < N; ++k) {
+    const float u = __shfl_down_sync(0xffffffffu, f[k], 1);
+    if (mine && tok0 + k < tokens) C[(size_t)(tok0 + k) * ldc + (feature >> 1)] = from_f<T>(epi_gate(f[k], u, epi.code, epi.act));
   }
 }
 
@@ -117,7 +174,19 @@ __device__ __forceinline__ void epi_store_row(const uint32_t (&r)[32], int row, 
 #pragma unroll
     for (int i = 0; i < CH; ++i) f[i] += cb0 + i < n_cols ? to_f(bias[cb0 + i]) : 0.f;
   }
-  epi_activate16_n<CH>(f, epi.code & kEpiActMask, epi.act);
+  if (epi_is_gate(epi.code)) {                     // (n_cols % 16 == 0)
+    T* dst = C + (size_t)row * ldc + (cb0 >> 1);
+#pragma unroll
+    for (int v = 0; v < CH / 8; ++v) {
+      if (cb0 + v * 8 >= n_cols) break;
+      T o4[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) o4[i] = from_f<T>(epi_gate(f[v * 8 + 2 * i], f[v * 8 + 2 * i + 1], epi.code, epi.act));
+      *reinterpret_cast<uint2*>(dst + v * 4) = *reinterpret_cast<const uint2*>(o4);
+    }
+    return;
+  }
+  epi_activate16_n<CH>(f, epi.code & kEpiActMask, epi.act, cb0, 1, n_cols);
   T* dst = C + (size_t)row * ldc + cb0;
 #pragma unroll
   for (int v = 0; v < CH / 8; ++v) {
@@ -156,10 +225,18 @@ __device__ __forceinline__ void epi_store_block_f32(const uint32_t (&r)[32], flo
       const float e = __ldg(epi.act);
 #pragma unroll 4
       for (int i = 0; i < n; ++i) dst[(size_t)i * ldc] = decay_of(stage[i][lane] + b, e);
+    } else if (epi.code == (kEpiSoftplusDecay | kEpiF32)) {
+      const float e = __ldg(epi.act + col);
+#pragma unroll 4
+      for (int i = 0; i < n; ++i) dst[(size_t)i * ldc] = softplus_decay_of(stage[i][lane] + b, e);
+    } else if (epi.code == (kEpiSoftcap | kEpiF32)) {
+      const float e = __ldg(epi.act);
+#pragma unroll 4
+      for (int i = 0; i < n; ++i) dst[(size_t)i * ldc] = softcap_of(stage[i][lane] + b, e);
     } else {
 #pragma unroll 1
       for (int i = 0; i < n; ++i)
-        dst[(size_t)i * ldc] = epi_activate(stage[i][lane] + b, epi.code & kEpiActMask, epi.act);
+        dst[(size_t)i * ldc] = epi_activate(stage[i][lane] + b, epi.code & kEpiActMask, epi.act, col);
     }
   }
   __syncwarp();
@@ -173,7 +250,7 @@ __device__ __forceinline__ void store_row_segment_f32(const uint32_t (&r)[32], i
 #pragma unroll
   for (int i = 0; i < CH; ++i)
     f[i] = __uint_as_float(r[i]) + ((bias && cb0 + i < n_cols) ? to_f(bias[cb0 + i]) : 0.f);
-  epi_activate16_n<CH>(f, epi.code & kEpiActMask, epi.act);
+  epi_activate16_n<CH>(f, epi.code & kEpiActMask, epi.act, cb0, 1, n_cols);
   float* dst = reinterpret_cast<float*>(C) + (size_t)row * ldc + cb0;
 #pragma unroll
   for (int i = 0; i < CH; ++i)

@@ -58,12 +58,22 @@ gemm_simt_kernel(const SimtGemmParams p) {
   for (int i = 0; i < 4; ++i) {
     const int m = m0 + ty * 4 + i;
     if (m >= rows) break;
+    if (epi_is_gate(p.epi.code)) {                     // (N is even)
+#pragma unroll
+      for (int j = 0; j < 4; j += 2) {
+        const int n = n0 + tx * 4 + j;
+        if (n >= p.N) break;
+        const float g = acc[i][j] + (bias ? to_f(bias[n]) : 0.f), u = acc[i][j + 1] + (bias ? to_f(bias[n + 1]) : 0.f);
+        reinterpret_cast<T*>(p.C)[z * p.c_batch + (int64_t)m * p.ldc + n / 2] = from_f<T>(epi_gate32(g, u, p.epi.code, p.epi.act));
+      }
+      continue;
+    }
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
       if (n < p.N)
         epi_store1<T>(reinterpret_cast<T*>(p.C), z * p.c_batch + (int64_t)m * p.ldc + n,
-                      acc[i][j] + (bias ? to_f(bias[n]) : 0.f), p.epi);
+                      acc[i][j] + (bias ? to_f(bias[n]) : 0.f), p.epi, n);
     }
   }
 }

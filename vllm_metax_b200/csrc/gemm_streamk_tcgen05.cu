@@ -292,7 +292,13 @@ gemm_streamk_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_consta
               if (ra + 3 < sh.N) *reinterpret_cast<uint32_t*>(crow + (ra >> 1)) = *reinterpret_cast<const uint32_t*>(o2);
               else if (ra + 1 < sh.N) crow[ra >> 1] = o2[0];
             } else if (EXT && epi.code > 1) {
-              epi_activate16_n<4>(f, epi.code & kEpiActMask, epi.act);
+              if (epi_is_gate(epi.code)) {
+#pragma unroll
+                for (int e = 0; e < 2; ++e)
+                  if (ra + 2 * e + 1 < sh.N) crow[(ra >> 1) + e] = from_f<T>(epi_gate(f[2 * e], f[2 * e + 1], epi.code, epi.act));
+                continue;
+              }
+              epi_activate16_n<4>(f, epi.code & kEpiActMask, epi.act, ra, 1, sh.N);
 #pragma unroll
               for (int e = 0; e < 4; ++e) {
                 if (ra + e >= sh.N) break;
@@ -338,11 +344,10 @@ gemm_streamk_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_consta
                 C[(size_t)(tok0 + i) * ldc + (ra >> 1)] = from_f<T>(g / (1.f + __expf(-g)) * up);
             }
           } else if (EXT && epi.code > 1) {
-            if (ra_ok) {
 #pragma unroll
-              for (int i = 0; i < 16; ++i) a[i] += bv;
-              epi_store_tokens<T, 16>(a, C, ra, tok0, sh.M, ldc, epi);
-            }
+            for (int i = 0; i < 16; ++i) a[i] += bv;
+            if (epi_is_gate(epi.code)) epi_gate_tokens<T, 16>(a, C, ra, tok0, sh.M, ldc, sh.N, epi);
+            else if (ra_ok) epi_store_tokens<T, 16>(a, C, ra, tok0, sh.M, ldc, sh.N, epi);
           } else if (ra_ok) {
 #pragma unroll
             for (int i = 0; i < 16; ++i) {

@@ -278,12 +278,11 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmA,   // 128-row operand
                 C[(size_t)tok * ldc + (ra >> 1)] = from_f<T>(g / (1.f + __expf(-g)) * u);
             }
           } else if (EXT && epi.code > 1) {
-            if (ra < rows_a) {
-              float f[CH];
+            float f[CH];
 #pragma unroll
-              for (int i = 0; i < CH; ++i) f[i] = __uint_as_float(r[i]) + bv;
-              epi_store_tokens<T, CH>(f, C, ra, cb0, rows_b, ldc, epi);
-            }
+            for (int i = 0; i < CH; ++i) f[i] = __uint_as_float(r[i]) + bv;
+            if (epi_is_gate(epi.code)) epi_gate_tokens<T, CH>(f, C, ra, cb0, rows_b, ldc, rows_a, epi);
+            else if (ra < rows_a) epi_store_tokens<T, CH>(f, C, ra, cb0, rows_b, ldc, rows_a, epi);
           } else if (ra < rows_a) {
 #pragma unroll
             for (int i = 0; i < CH; ++i) {

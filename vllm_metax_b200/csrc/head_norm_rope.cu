@@ -1,6 +1,7 @@
-// Epilogue of a merged q | k | v product, per token and head: RMS norm over the head (shared weights for all heads), rotation
-// of its first `rot` entries in pairs (i, i + rot / 2), then queries to a packed tensor and keys, together with the values,
-// to their paged cache row - one launch.  Layers that read another layer's cache pass queries only.
+// Epilogue of a merged q | k | v product, per token and head: RMS norm over the head (shared weights for all heads) or over all
+// heads together, rotation of its first `rot` entries in pairs (i, i + rot / 2) or (2i, 2i + 1), a factor for queries that grows
+// with the position, then queries to a packed tensor and keys, together with the values, to their paged cache row - one launch.
+// Layers that read another layer's cache pass queries only.
 //
 // Heads may be padded with zeros to a multiple of 8 (`dim_pad`); the mean runs over the `dim` real entries.  Cosines and sines
 // come from a table of the step's tokens that all layers of one rotation share (`rope_angles`): an angle is position *
@@ -59,6 +60,26 @@ __device__ __forceinline__ void cache_rows(const HeadNormRopeParams& p, int64_t 
   v_row = block * p.page_stride + (int64_t)at * p.kv_heads * p.vdim_pad;
 }
 
+// What token t's queries are multiplied by.
+__device__ __forceinline__ float query_temp(const HeadNormRopeParams& p, int64_t t) {
+  if (p.positions == nullptr) return 1.f;
+  return 1.f + p.temp_coef * logf((float)((p.positions[t] + 1) / p.temp_every) + 1.f);
+}
+
+// Pairs (2i, 2i + 1) of 8 entries from c0 on; `cs`, `sn`: the token's cosines and sines.
+__device__ __forceinline__ void rotate_pairs8(float (&v)[8], int c0, int half, const float* __restrict__ cs,
+                                              const float* __restrict__ sn) {
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const int i = c0 / 2 + j;
+    if (i < half) {
+      const float c = cs[i], s = sn[i], a = v[2 * j], b = v[2 * j + 1];
+      v[2 * j] = a * c - b * s;
+      v[2 * j + 1] = b * c + a * s;
+    }
+  }
+}
+
 // Heads of up to 256 entries whose half rotation is a multiple of 8: `1 << log_lanes` neighbouring lanes hold one head of one
 // token, 8 entries each, and exchange rotation partners by shuffles.  A token's items: queries, keys, then its values in
 // pieces of lanes * 8 entries.  A thread keeps its item and the norm weights of it and walks tokens.
@@ -102,7 +123,7 @@ head_norm_rope_vec_kernel(const HeadNormRopeParams p, int log_lanes, int items) 
       load_row<T, 8, true>(col + t * p.row_stride, 0, 8, v);
     }
     float c[8] = {}, s[8] = {};
-    if (head && rotated) {
+    if (head && rotated && !p.interleaved) {
       load_row<float, 8, true>(ang + (int64_t)(2 * t) * half, 0, 8, c);
       load_row<float, 8, true>(ang + (int64_t)(2 * t + 1) * half, 0, 8, s);
     }
@@ -115,12 +136,19 @@ head_norm_rope_vec_kernel(const HeadNormRopeParams p, int log_lanes, int items) 
 #pragma unroll
       for (int k = 0; k < 8; ++k) v[k] = v[k] * inv * g[k];
     }
-    if (p.rot > 0) {
+    if (p.interleaved) {
+      if (head && rotated) rotate_pairs8(v, c0, half, p.angles + 2 * (int64_t)t * half, p.angles + (2 * (int64_t)t + 1) * half);
+    } else if (p.rot > 0) {
 #pragma unroll
       for (int k = 0; k < 8; ++k) {
         const float o = __shfl_sync(0xffffffffu, v[k], partner);
         if (head && rotated) v[k] = v[k] * c[k] + (first ? -o : o) * s[k];
       }
+    }
+    if (head && is_q) {
+      const float temp = query_temp(p, t);
+#pragma unroll
+      for (int k = 0; k < 8; ++k) v[k] *= temp;
     }
     if (head) {
       if (is_q)
@@ -164,12 +192,15 @@ head_norm_rope_kernel(const HeadNormRopeParams p) {
       buf[i] = f;
     }
     __syncwarp();
+    const float temp = item < p.heads ? query_temp(p, t) : 1.f;
     if (dst != nullptr)
       for (int i = lane; i < p.dim_pad; i += 32) {
         float f = buf[i];
-        if (i < half) f = f * cs[i] - buf[i + half] * sn[i];
+        if (p.interleaved) {
+          if (i < p.rot) f = f * cs[i >> 1] + (i & 1 ? buf[i - 1] : -buf[i + 1]) * sn[i >> 1];
+        } else if (i < half) f = f * cs[i] - buf[i + half] * sn[i];
         else if (i < 2 * half) f = f * cs[i - half] + buf[i - half] * sn[i - half];
-        dst[i] = from_f<T>(f);
+        dst[i] = from_f<T>(f * temp);
       }
   }
   if (v_row < 0) return;
@@ -178,11 +209,93 @@ head_norm_rope_kernel(const HeadNormRopeParams p) {
   for (int i = threadIdx.x; i < p.kv_heads * p.vdim_pad; i += kAnyWarps * 32) dst[i] = src[i];
 }
 
+// One norm over all heads: a CTA per token, 8 entries of a head per thread and trip; the rows are read twice.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(kThreads)
+row_norm_rope_kernel(const HeadNormRopeParams p) {
+  __shared__ float red[2][kThreads / 32];
+  const int64_t t = blockIdx.x;
+  int64_t k_row, v_row;
+  cache_rows(p, t, k_row, v_row);
+  const int per = p.dim_pad / 8, nq = p.heads * per, nk = p.k_cache != nullptr ? p.kv_heads * per : 0;
+  const T* row = reinterpret_cast<const T*>(p.qkv) + t * p.row_stride;
+  float ss[2] = {0.f, 0.f};
+  for (int u = threadIdx.x; u < nq + nk; u += kThreads) {
+    float v[8], s = 0.f;
+    load_row<T, 8, VEC>(u < nq ? row + p.q_off + u * 8 : row + p.k_off + (u - nq) * 8, 0, 8, v);
+#pragma unroll
+    for (int k = 0; k < 8; ++k) s = fmaf(v[k], v[k], s);
+    if (u < nq) ss[0] += s; else ss[1] += s;
+  }
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    ss[i] = warp_sum(ss[i]);
+    if (lane == 0) red[i][warp] = ss[i];
+  }
+  __syncthreads();
+  float inv[2];
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    float s = 0.f;
+    for (int w = 0; w < kThreads / 32; ++w) s += red[i][w];
+    inv[i] = 1.f / sqrtf(s / ((float)(i ? p.kv_heads : p.heads) * (float)p.dim) + p.eps);
+  }
+  const int half = p.rot / 2;
+  const float *cs = p.angles + 2 * t * half, *sn = cs + half;
+  const float temp = query_temp(p, t);
+  for (int u = threadIdx.x; u < nq + nk; u += kThreads) {
+    const bool is_q = u < nq;
+    if (!is_q && k_row < 0) break;
+    const int h = (is_q ? u : u - nq) / per, c0 = ((is_q ? u : u - nq) % per) * 8;
+    const T* src = row + (is_q ? p.q_off : p.k_off) + (int64_t)h * p.dim_pad;
+    const T* w = reinterpret_cast<const T*>(is_q ? p.q_w : p.k_w) + (int64_t)h * p.dim_pad;
+    const float one = p.one_plus ? 1.f : 0.f, scale = is_q ? inv[0] : inv[1];
+    float v[8], g[8];
+    load_row<T, 8, VEC>(src + c0, 0, 8, v);
+    load_row<T, 8, VEC>(w + c0, 0, 8, g);
+#pragma unroll
+    for (int k = 0; k < 8; ++k) v[k] = v[k] * scale * (g[k] + one);
+    if (p.interleaved) {
+      rotate_pairs8(v, c0, half, cs, sn);
+    } else {
+#pragma unroll
+      for (int k = 0; k < 8; ++k) {
+        const int i = c0 + k, j = i < half ? i + half : i - half;
+        if (i < p.rot) {
+          const float o = to_f(src[j]) * scale * (to_f(w[j]) + one);
+          v[k] = i < half ? v[k] * cs[i] - o * sn[i] : v[k] * cs[j] + o * sn[j];
+        }
+      }
+    }
+    if (is_q) {
+#pragma unroll
+      for (int k = 0; k < 8; ++k) v[k] *= temp;
+      store_row<T, 8, VEC>(reinterpret_cast<T*>(p.q_out) + (t * p.heads + h) * p.dim_pad + c0, 0, 8, v);
+    } else {
+      store_row<T, 8, VEC>(reinterpret_cast<T*>(p.k_cache) + k_row + (int64_t)h * p.dim_pad + c0, 0, 8, v);
+    }
+  }
+  if (v_row < 0) return;
+  const int nv = p.kv_heads * p.vdim_pad;
+  for (int i = threadIdx.x * 8; i < nv; i += kThreads * 8) {
+    float v[8];
+    load_row<T, 8, VEC>(row + p.v_off, i, nv, v);
+    store_row<T, 8, VEC>(reinterpret_cast<T*>(p.v_cache) + v_row, i, nv, v);
+  }
+}
+
 template <typename T>
 int launch(const HeadNormRopeParams& p, cudaStream_t stream) {
   if (p.rot > p.dim || p.rot % 2 != 0 || p.dim_pad > kMaxDim) return 1;
   if (p.k_cache != nullptr && (p.q_w == nullptr) != (p.k_w == nullptr)) return 1;
-  if (p.vec && p.dim_pad <= 256 && p.rot % 16 == 0) {
+  if (p.whole_row) {
+    if (p.q_w == nullptr || p.dim_pad % 8 != 0) return 1;
+    if (p.vec) row_norm_rope_kernel<T, true><<<p.tokens, kThreads, 0, stream>>>(p);
+    else row_norm_rope_kernel<T, false><<<p.tokens, kThreads, 0, stream>>>(p);
+    return 0;
+  }
+  if (p.vec && p.dim_pad <= 256 && (p.interleaved || p.rot % 16 == 0)) {
     int log_lanes = 0;
     while ((8 << log_lanes) < p.dim_pad) ++log_lanes;
     const int values = p.k_cache != nullptr ? ceil_div(p.kv_heads * p.vdim_pad, 8 << log_lanes) : 0;

@@ -286,7 +286,8 @@ moe_align_kernel(int* __restrict__ sorted_ids, int* __restrict__ block_expert, i
 
 template <typename T>
 __global__ void moe_gather_kernel(T* __restrict__ out, const T* __restrict__ x, const int* __restrict__ sorted_ids,
-                                  const int* __restrict__ total_padded, int numel, int topk, int hidden) {
+                                  const int* __restrict__ total_padded, const float* __restrict__ weights, int numel, int topk,
+                                  int hidden) {
   const int row = blockIdx.x;
   if (row >= *total_padded) return;
   const int id = sorted_ids[row];
@@ -296,6 +297,17 @@ __global__ void moe_gather_kernel(T* __restrict__ out, const T* __restrict__ x, 
     return;
   }
   const uint4* src = reinterpret_cast<const uint4*>(x + (size_t)(id / topk) * hidden);
+  if (weights != nullptr) {
+    const float w = weights[id];
+    for (int v = threadIdx.x; v < hidden / 8; v += blockDim.x) {
+      float f[8];
+      unpack8<T>(src[v], f);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) f[i] *= w;
+      dst[v] = pack8<T>(f);
+    }
+    return;
+  }
   for (int v = threadIdx.x; v < hidden / 8; v += blockDim.x) dst[v] = src[v];
 }
 
@@ -339,12 +351,13 @@ __global__ void moe_combine_kernel(T* __restrict__ out, const T* __restrict__ y,
 template <typename T>
 __global__ void moe_gather_scalar_kernel(T* __restrict__ out, const T* __restrict__ x,
                                          const int* __restrict__ sorted_ids, const int* __restrict__ total_padded,
-                                         int numel, int topk, int hidden) {
+                                         const float* __restrict__ weights, int numel, int topk, int hidden) {
   const int row = blockIdx.x;
   if (row >= *total_padded) return;
   const int id = sorted_ids[row];
+  const float w = weights != nullptr && id < numel ? weights[id] : 1.f;
   for (int i = threadIdx.x; i < hidden; i += blockDim.x)
-    out[(size_t)row * hidden + i] = id < numel ? x[(size_t)(id / topk) * hidden + i] : from_f<T>(0.f);
+    out[(size_t)row * hidden + i] = from_f<T>(id < numel ? w * to_f(x[(size_t)(id / topk) * hidden + i]) : 0.f);
 }
 
 template <typename T>
@@ -418,21 +431,21 @@ void moe_align(int* sorted_ids, int* block_expert, int* total_padded, int* inv_p
                                             numel, experts, block, max_padded);
 }
 
-void moe_gather(void* out, const void* x, const int* sorted_ids, const int* total_padded, int max_padded, int numel,
-                int topk, int hidden, int dtype, cudaStream_t stream) {
+void moe_gather(void* out, const void* x, const int* sorted_ids, const int* total_padded, const float* weights, int max_padded,
+                int numel, int topk, int hidden, int dtype, cudaStream_t stream) {
   if (max_padded <= 0) return;
   if (dtype == 2 || hidden % 8 != 0) {
     DISPATCH_16(dtype,
-                (moe_gather_scalar_kernel<<<max_padded, 128, 0, stream>>>((__nv_bfloat16*)out, (const __nv_bfloat16*)x, sorted_ids, total_padded, numel, topk, hidden)),
-                (moe_gather_scalar_kernel<<<max_padded, 128, 0, stream>>>((__half*)out, (const __half*)x, sorted_ids, total_padded, numel, topk, hidden)),
-                (moe_gather_scalar_kernel<<<max_padded, 128, 0, stream>>>((float*)out, (const float*)x, sorted_ids, total_padded, numel, topk, hidden)))
+                (moe_gather_scalar_kernel<<<max_padded, 128, 0, stream>>>((__nv_bfloat16*)out, (const __nv_bfloat16*)x, sorted_ids, total_padded, weights, numel, topk, hidden)),
+                (moe_gather_scalar_kernel<<<max_padded, 128, 0, stream>>>((__half*)out, (const __half*)x, sorted_ids, total_padded, weights, numel, topk, hidden)),
+                (moe_gather_scalar_kernel<<<max_padded, 128, 0, stream>>>((float*)out, (const float*)x, sorted_ids, total_padded, weights, numel, topk, hidden)))
     return;
   }
   const int th = hidden / 8 < 256 ? (hidden / 8 < 32 ? 32 : hidden / 8) : 256;
   if (dtype == 0)
-    moe_gather_kernel<__nv_bfloat16><<<max_padded, th, 0, stream>>>((__nv_bfloat16*)out, (const __nv_bfloat16*)x, sorted_ids, total_padded, numel, topk, hidden);
+    moe_gather_kernel<__nv_bfloat16><<<max_padded, th, 0, stream>>>((__nv_bfloat16*)out, (const __nv_bfloat16*)x, sorted_ids, total_padded, weights, numel, topk, hidden);
   else
-    moe_gather_kernel<__half><<<max_padded, th, 0, stream>>>((__half*)out, (const __half*)x, sorted_ids, total_padded, numel, topk, hidden);
+    moe_gather_kernel<__half><<<max_padded, th, 0, stream>>>((__half*)out, (const __half*)x, sorted_ids, total_padded, weights, numel, topk, hidden);
 }
 
 void moe_combine(void* out, const void* y, const float* weights, const int* inv_pos, const void* shared,

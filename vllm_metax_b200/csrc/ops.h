@@ -10,6 +10,16 @@
 
 namespace b200 {
 
+// What follows the read-outs o of a linear-attention recurrence:
+// out = out_scale * unit_rms(o) * norm_w * act(gate), act = sigmoid or silu.
+struct GatedNormOut {
+  const void* gate; int64_t gate_stride;      // [tokens, heads * vdim]
+  const void* norm_w; int w_head_stride;      // [vdim] (stride 0) or [heads * vdim]
+  void* out; int64_t out_stride;              // [tokens, heads * vdim]
+  float eps, out_scale;
+  int sigmoid_gate;
+};
+
 struct DecodeParams {
   void* out;                 // [T, Hq, D] (T dtype)
   float* part_out;           // [splits, T, Hq, D]
@@ -33,6 +43,13 @@ struct DecodeParams {
   int window;                // <=0: none
   int causal;
   StatusWord* status;
+  // what happens to scores and results beyond that (all optional)
+  const float* bias = nullptr;   // [Hq, bias_len]: added to the scaled (and capped) score of a key by its distance
+  int bias_len = 0;              //   ... from bias_len - 1 on: the last entry
+  const void* gate = nullptr;    // [T, Hq * dv] (token stride gate_stride): the result is multiplied by its sigmoid
+  int64_t gate_stride = 0;
+  float out_scale = 1.f;
+  int64_t out_stride = 0;        // elements between two tokens of out (0: packed)
 };
 
 struct PrefillParams {
@@ -54,6 +71,13 @@ struct PrefillParams {
   int64_t k_head_stride, v_head_stride;   // contiguous mode, elements
   int64_t page_stride;           // paged mode: elements between two pages (of K and of V)
   StatusWord* status;
+  // what happens to scores and results beyond that (all optional)
+  const float* bias = nullptr;   // [Hq, bias_len]: added to the scaled (and capped) score of a key by its distance
+  int bias_len = 0;              //   ... from bias_len - 1 on: the last entry
+  const void* gate = nullptr;    // [T, Hq * dv] (token stride gate_stride): the result is multiplied by its sigmoid
+  int64_t gate_stride = 0;
+  float out_scale = 1.f;
+  int64_t out_stride = 0;        // elements between two tokens of out (0: packed)
 };
 
 struct MlaDecodeParams {
@@ -174,8 +198,9 @@ void grouped_topk(float* weights, int* ids, const void* gating, const float* bia
                   int n_group, int topk_group, int sigmoid, int renorm, float scale, int dtype, cudaStream_t stream);
 void moe_align(int* sorted_ids, int* block_expert, int* total_padded, int* inv_pos, const int* topk_ids,
                const int* expert_map, int numel, int experts, int block, int max_padded, cudaStream_t stream);
-void moe_gather(void* out, const void* x, const int* sorted_ids, const int* total_padded, int max_padded, int numel,
-                int topk, int hidden, int dtype, cudaStream_t stream);
+// (weights given: a pair's row is multiplied by its weight)
+void moe_gather(void* out, const void* x, const int* sorted_ids, const int* total_padded, const float* weights, int max_padded,
+                int numel, int topk, int hidden, int dtype, cudaStream_t stream);
 // (expert_ids / through given: a pair whose expert id is at least identity_from adds its weight times the row of `through`)
 void moe_combine(void* out, const void* y, const float* weights, const int* inv_pos, const void* shared,
                  const int* expert_ids, const void* through, int identity_from, int tokens, int topk, int hidden, int dtype,
@@ -336,6 +361,26 @@ struct ResidualNormParams {
   StatusWord* status;
 };
 int residual_norm(const ResidualNormParams& p, int dtype, cudaStream_t stream);
+// ---- prenorm.cu (residual add + layer norm in front of the next sublayer, or the operand of a loop's entry product)
+struct PrenormParams {
+  const void* y;           // [rows, D] as in ResidualNormParams; y_f32: fp32 rows
+  const int64_t* ids;      // [tokens] rows of y, or null
+  const float* weights;    // topk > 0: expert-sorted rows; null weights: ones
+  const int* inv_pos;
+  const void* shared;      // [tokens, D] or null
+  const float* x;          // [tokens, D] or null
+  const void* add;         // [D] or null
+  float* x_out;            // [tokens, D] or null
+  void* h;                 // [tokens, D]; with `table`: [tokens, 3 D] = x' in two 16-bit parts | table row (fp32: [tokens, 2 D])
+  const void* gain;        // [D]
+  const void* table;       // loop operand: rows of the embedding table ...
+  const int64_t* table_ids;
+  int tokens, D, vec, topk, y_f32;
+  int64_t rows, table_rows;
+  float eps;
+  StatusWord* status;
+};
+int prenorm(const PrenormParams& p, int dtype, cudaStream_t stream);
 // ---- head_norm_rope.cu (epilogue of a merged q | k | v product: head norms, partial rotation, paged cache write)
 struct HeadNormRopeParams {
   const void* qkv; int64_t row_stride; int q_off, k_off, v_off;   // [tokens, ...], heads packed from these columns on
@@ -346,31 +391,62 @@ struct HeadNormRopeParams {
   const float* angles;                  // [tokens, 2, rot / 2]: cosines, sines
   const int64_t* slots;
   int tokens, heads, kv_heads, dim, dim_pad, vdim_pad, rot, block_size, one_plus, vec;
+  int whole_row, interleaved;           // one norm over all heads (weights [heads, dim_pad]); pairs (2i, 2i + 1)
+  const int64_t* positions;             // with temp_coef: queries times 1 + temp_coef * ln((position + 1) / temp_every + 1)
+  float temp_coef; int temp_every;
   float eps;
   StatusWord* status;
 };
 int head_norm_rope(const HeadNormRopeParams& p, int dtype, cudaStream_t stream);
 // cos and sin of position * inv_freq, [tokens, 2, half]; whole turns are taken off in fp64
 void rope_angles(float* out, const int64_t* positions, const double* inv_freq, int tokens, int half, cudaStream_t stream);
-// ---- gla.cu (gated linear attention: decay per key channel)
+// ---- gla.cu (linear attention with a decay)
 struct GlaParams {
-  const void* qkvg;            // [tokens, row_stride]: q | k | v | gate at the given element offsets
+  const void* qkvg;            // [tokens, row_stride]: q | k | v at the given element offsets
   int64_t row_stride;
-  int q_off, k_off, v_off, g_off;
-  const float* alpha;          // [tokens, heads * dim] decays
-  const void* norm_w;          // [vdim]
+  int q_off, k_off, v_off;
+  const float* alpha;          // [tokens, heads * dim] decays per key channel, or null:
+  const float* decay_tok;      // [tokens, heads], or null:
+  const float* decay_head;     // [heads]
+  const float* k_mul;          // matrix memory: [tokens, heads] factors of k,
+  const float* floor;          //   [tokens, heads] least absolute value of the divisor,
+  float* norm_state;           //   [slots, heads, ceil(vdim / 16), dim] (equal copies), or null
+  GatedNormOut out;
   float* state;                // [slots, heads, dim, vdim]
   float* o_raw;                // set from the scratch: [tokens, heads * vdim] raw outputs of heads split over CTAs
   float* seg_state;            // set from the scratch: [segments, heads, dim, vdim] ...
-  float* seg_decay;            // ... and [segments, heads, dim], or null
-  void* out;                   // [tokens, heads * vdim]
+  float* seg_decay;            // ... and [segments, heads, dim] ...
+  float* seg_norm;             // ... twice, or null
   const int* qsl; const int* state_idx; const int* has_init;
-  int batch, tokens, heads, dim, vdim, col_block, vec;
-  float scale, eps;
+  int batch, tokens, heads, dim, vdim, col_block, vec, chunk, silu_qkv, whole_row;
+  float scale;
 };
 struct GlaScratch { int64_t raw, segments; };
-GlaScratch gla_scratch(int batch, int tokens, int heads, int dim, int vdim, int max_query_len, int sms);
+GlaScratch gla_scratch(int batch, int tokens, int heads, int dim, int vdim, int max_query_len, int sms, bool whole_row);
 int gla_recurrent(GlaParams p, float* scratch, int max_query_len, int sms, int dtype, cudaStream_t stream);
+struct MemoryGatesParams {
+  const float* logits; int64_t stride;   // [tokens, >= 2 heads]: input gates, forget gates
+  const float* bias;                     // [2 heads]
+  float* top;                            // [slots, heads]
+  float* out;                            // [3, tokens, heads]: decay, k_mul, floor
+  const int* qsl; const int* state_idx; const int* has_init;
+  int batch, tokens, heads;
+  float cap;
+};
+void memory_gates(const MemoryGatesParams& p, int max_query_len, cudaStream_t stream);
+// ---- channel_delta.cu (gated delta rule with a decay per key channel)
+struct ChannelDeltaParams {
+  const void* qkv; int64_t row_stride; int q_off, k_off, v_off;
+  const float* g; int64_t g_stride;            // [tokens, heads * dim] decays
+  const float* beta; int64_t beta_stride;      // [tokens, heads] logits of the step sizes
+  GatedNormOut out;
+  float* state;                                // [slots, heads, dim, vdim]
+  float* o_raw;                                // [tokens, heads * vdim] scratch where heads are split over CTAs
+  const int* qsl; const int* state_idx; const int* has_init;
+  int batch, tokens, heads, kv_heads, dim, vdim, col_block, vec, chunk;
+};
+int64_t channel_delta_scratch(int batch, int tokens, int heads, int vdim, int max_query_len, int sms);
+int channel_delta(ChannelDeltaParams p, float* scratch, int max_query_len, int sms, int dtype, cudaStream_t stream);
 // ---- rglru.cu (real-gated linear recurrent unit)
 struct RgLruParams {
   const void* u; int64_t u_stride;       // [tokens, width] recurrence input

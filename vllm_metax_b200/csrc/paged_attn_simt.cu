@@ -3,7 +3,7 @@
 // of query tokens per sequence.
 //
 // One CTA per (query token, head): 128 keys at a time, eight lanes per key for the scores (coalesced rows), then a thread per
-// value column.  Online softmax in fp32.
+// value column.  Online softmax in fp32, with the soft-cap, distance bias, sinks and output gate of the tensor-core kernels.
 #include "ops.h"
 #include "row_vec.cuh"
 
@@ -65,7 +65,12 @@ paged_attn_simt_kernel(const DecodeParams p, int batch) {
       }
 #pragma unroll
       for (int o = 4; o > 0; o >>= 1) d += __shfl_xor_sync(0xffffffffu, d, o);
-      if ((threadIdx.x & 7) == 0) s_p[k] = r >= 0 ? d * p.scale : -INFINITY;
+      if ((threadIdx.x & 7) == 0) {
+        d *= p.scale;
+        if (p.softcap > 0.f) d = p.softcap * tanhf(d / p.softcap);
+        if (p.bias != nullptr) d += p.bias[(int64_t)h * p.bias_len + min(max(pos - 1 - (k0 + k), 0), p.bias_len - 1)];
+        s_p[k] = r >= 0 ? d : -INFINITY;
+      }
     }
     __syncthreads();
     const float s = s_p[threadIdx.x];
@@ -88,12 +93,19 @@ paged_attn_simt_kernel(const DecodeParams p, int batch) {
       }
     }
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
-  T* out = reinterpret_cast<T*>(p.out) + ((int64_t)t * p.num_q_heads + h) * p.dv;
+  float scale_o = 1.f;
+  if (p.sinks != nullptr) {                                  // one more term of the denominator (and of its maximum)
+    const float z = p.sinks[h], mn = fmaxf(m, z);
+    scale_o = m == -INFINITY ? 0.f : expf(m - mn);
+    l = l * scale_o + expf(z - mn);
+  }
+  const float inv = l > 0.f ? p.out_scale * scale_o / l : 0.f;
+  T* out = reinterpret_cast<T*>(p.out) + t * (p.out_stride ? p.out_stride : (int64_t)p.num_q_heads * p.dv) + h * p.dv;
+  const T* gate = p.gate != nullptr ? reinterpret_cast<const T*>(p.gate) + t * p.gate_stride + h * p.dv : nullptr;
 #pragma unroll
   for (int i = 0; i < kCols; ++i) {
     const int c = threadIdx.x + i * kKeys;
-    if (c < p.dv) out[c] = from_f<T>(acc[i] * inv);
+    if (c < p.dv) out[c] = from_f<T>(acc[i] * inv * (gate != nullptr ? 1.f / (1.f + expf(-to_f(gate[c]))) : 1.f));
   }
 }
 

@@ -8,21 +8,11 @@
 // multiplier folded together).  Token t's y is row t, row ids[t] of a table, or - straight from the grouped expert products,
 // so that the combined rows never reach memory - the weighted sum of its expert-sorted rows, where identity experts
 // contribute the token's own row.  One CTA per token, a row in registers.
+#include "boundary_rows.cuh"
 #include "ops.h"
-#include "row_vec.cuh"
 
 namespace b200 {
 namespace {
-
-// Sum over the CTA with one barrier; the caller alternates between two buffers.
-__device__ __forceinline__ float row_sum(float v, float* red) {
-  v = warp_sum(v);
-  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
-  __syncthreads();
-  const int nw = blockDim.x >> 5;
-  const float s = (int)(threadIdx.x & 31) < nw ? red[threadIdx.x & 31] : 0.f;
-  return warp_sum(s);
-}
 
 template <typename T, int CN, bool VEC>
 __device__ __forceinline__ void load_gain(const void* g, int n, int f32, int c0, int D, float (&out)[CN]) {
@@ -34,38 +24,6 @@ __device__ __forceinline__ void load_gain(const void* g, int n, int f32, int c0,
     load_row<float, CN, VEC>(reinterpret_cast<const float*>(g), c0, D, out);
   } else {
     load_row<T, CN, VEC>(reinterpret_cast<const T*>(g), c0, D, out);
-  }
-}
-
-// Four pairs of a token at once: their rows' loads are all in flight before the first is used.
-template <typename T, int CN, bool VEC>
-__device__ __forceinline__ void add_expert_rows(const ResidualNormParams& p, int64_t t, int c0, float (&v)[CN]) {
-  constexpr int kAhead = 4;
-  const T* y = reinterpret_cast<const T*>(p.y);
-  for (int k0 = 0; k0 < p.topk; k0 += kAhead) {
-    const T* row[kAhead];
-    float w[kAhead], f[kAhead][CN];
-#pragma unroll
-    for (int u = 0; u < kAhead; ++u) {
-      row[u] = nullptr;
-      w[u] = 0.f;
-      if (k0 + u < p.topk) {
-        const int64_t i = t * p.topk + k0 + u;
-        const int pos = p.inv_pos[i];
-        w[u] = p.weights[i];
-        if (pos >= 0) row[u] = y + (int64_t)pos * p.D;
-        else if (p.through != nullptr && p.expert_ids[i] >= p.identity_from)
-          row[u] = reinterpret_cast<const T*>(p.through) + t * p.D;
-      }
-    }
-#pragma unroll
-    for (int u = 0; u < kAhead; ++u)
-      if (row[u] != nullptr) load_row<T, CN, VEC>(row[u], c0, p.D, f[u]);
-#pragma unroll
-    for (int u = 0; u < kAhead; ++u)
-      if (row[u] != nullptr)
-#pragma unroll
-        for (int j = 0; j < CN; ++j) v[j] = fmaf(w[u], f[u][j], v[j]);
   }
 }
 
@@ -82,7 +40,8 @@ residual_norm_kernel(const ResidualNormParams p) {
     if (p.x != nullptr) load_row<float, CN, VEC>(p.x + t * D, c0, D, xv);
     if constexpr (COMBINE) {
       if (p.shared != nullptr) load_row<T, CN, VEC>(reinterpret_cast<const T*>(p.shared) + t * D, c0, D, v);
-      add_expert_rows<T, CN, VEC>(p, t, c0, v);
+      add_expert_rows<T, CN, VEC>(y, p.weights, p.inv_pos, p.expert_ids, reinterpret_cast<const T*>(p.through), p.identity_from,
+                                  p.topk, t, c0, D, v);
     } else {
       const int64_t row = p.ids != nullptr ? p.ids[t] : t;
       if (row >= 0 && row < p.rows) load_row<T, CN, VEC>(y + row * D, c0, D, v);

@@ -10,6 +10,7 @@ vllm_metax/v1/attention/backends/flash_attn.py:1302-1355 (VLLM_METAX_ENABLE_FA_S
 """
 from __future__ import annotations
 
+import math
 from typing import Optional
 
 import torch
@@ -91,6 +92,8 @@ class Attention(nn.Module):
         self.softcap = softcap
         self.sinks = sinks
         self.k_scale, self.v_scale = k_scale, v_scale
+        self.distance_bias: Optional[torch.Tensor] = None      # f32 [num_heads, L]: bias by distance, the last entry from L - 1 on
+        self.out_scale = 1.0
 
     def forward(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, positions: Optional[torch.Tensor] = None,
                 rope=None) -> torch.Tensor:
@@ -127,24 +130,29 @@ class Attention(nn.Module):
             return self._forward_cascade(q3, md, kv_cache, kv_scales)
         return self.attend(q3, md, kv_cache, kv_scales).reshape(T, self.num_heads * self.head_size)
 
-    def attend(self, q3: torch.Tensor, md, kv_cache, kv_scales=None) -> torch.Tensor:
+    def attend(self, q3: torch.Tensor, md, kv_cache, kv_scales=None, out=None, gate=None) -> torch.Tensor:
         """``q3 [T, heads, D]`` over the cache, which already holds this step's keys and values (written by this layer or by the
-        one whose cache it reads): decode rows, then prompt portions.  ``kv_cache``: 5-D or a pair of views."""
-        v_size = kv_cache[1].shape[-1] if isinstance(kv_cache, tuple) else self.head_size
-        out = torch.empty(q3.shape[0], self.num_heads, v_size, dtype=q3.dtype, device=q3.device)
+        one whose cache it reads): decode rows, then prompt portions.  ``kv_cache``: 5-D or a pair of views.  ``out`` and
+        ``gate``: as in ``ops.paged_attention_decode``."""
+        if out is None:
+            v_size = kv_cache[1].shape[-1] if isinstance(kv_cache, tuple) else self.head_size
+            out = torch.empty(q3.shape[0], self.num_heads, v_size, dtype=q3.dtype, device=q3.device)
         nd, ndt = md.num_decodes, md.num_decode_tokens
+        gates = (None, None) if gate is None else (gate[:ndt], gate[ndt:])
         if nd > 0:
             ops.paged_attention_decode(q3[:ndt], kv_cache, md.block_table[:nd], md.seq_lens[:nd], self.scale,
                                        out=out[:ndt], kv_scales=kv_scales, window=self.window, softcap=self.softcap,
                                        sinks=self.sinks, num_splits=md.decode_num_splits, max_seq_len=md.max_seq_len,
                                        k_scale=self.k_scale, v_scale=self.v_scale, workspace=md.decode_workspace,
-                                       alibi_slopes=self.alibi_slopes)
+                                       alibi_slopes=self.alibi_slopes, distance_bias=self.distance_bias, gate=gates[0],
+                                       out_scale=self.out_scale)
         if md.num_prefills > 0:
             ops.paged_attention_prefill(q3[ndt:], kv_cache, md.block_table[nd:], md.seq_lens[nd:],
                                         md.prefill_query_start_loc, self.scale, out=out[ndt:], kv_scales=kv_scales,
                                         max_q_len=md.max_prefill_query_len, window=self.window, softcap=self.softcap,
                                         sinks=self.sinks, k_scale=self.k_scale, v_scale=self.v_scale,
-                                        max_seq_len=md.max_seq_len, alibi_slopes=self.alibi_slopes)
+                                        max_seq_len=md.max_seq_len, alibi_slopes=self.alibi_slopes,
+                                        distance_bias=self.distance_bias, gate=gates[1], out_scale=self.out_scale)
         return out
 
     def _forward_cascade(self, q3, md, kv_cache, kv_scales) -> torch.Tensor:
@@ -290,17 +298,26 @@ class Attention(nn.Module):
 
 
 class QKNormAttention(nn.Module):
-    """Grouped-query attention with RMS-normed, partially rotated queries and keys, key and value sizes of its own, an optional
-    sliding window, and optionally the keys and values of another layer (``kv_from``: that layer's module, which must come
-    earlier in the step) instead of projections and a cache of its own.
+    """Grouped-query attention with RMS-normed queries and keys, key and value sizes of its own, an optional sliding window, and
+    optionally the keys and values of another layer (``kv_from``: that layer's module, which must come earlier in the step)
+    instead of projections and a cache of its own.
 
         merged q | k | v product -> ``head_norm_rope`` (norms, rotation, cache write) -> paged attention -> output product
 
-    Head sizes are padded to multiples of 8 with zero rows of the projections (and zero columns of the output product)."""
+    ``whole_row_norm``: one norm over all heads.  ``inv_freq=None``: no rotation; ``interleaved``: pairs (2i, 2i + 1).
+    ``q_temp = (coef, every)``: queries grow with the position.  ``bias_far`` and ``bias_rows``: a learned bias by distance, one
+    row per bucket (``distance_buckets``).  ``gated``: the heads' outputs times the sigmoid of another projection.
+
+    Head sizes are padded to multiples of 8 with zero rows of the projections (and zero columns of the output product).
+    ``standalone=False``: a branch of a :class:`layers.mixer.ProjectedMixer`, which owns the products.  ``runs``: how often a
+    step passes through the layer; every pass has a cache of its own, from ``cache_idx`` on."""
 
     def __init__(self, width: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, eps: float,
-                 inv_freq: torch.Tensor, cache_idx: int, window: Optional[int] = None,
-                 kv_from: Optional["QKNormAttention"] = None, dtype=torch.bfloat16):
+                 inv_freq: Optional[torch.Tensor], cache_idx: int, window: Optional[int] = None,
+                 kv_from: Optional["QKNormAttention"] = None, dtype=torch.bfloat16, *, standalone: bool = True, runs: int = 1,
+                 whole_row_norm: bool = False, interleaved: bool = False, q_temp: Optional[tuple] = None, softcap: float = 0.0,
+                 sinks: bool = False, bias_rows: int = 0, bias_far: int = 0, gated: bool = False, proj_bias: bool = False,
+                 out_scale: float = 1.0):
         super().__init__()
         if heads % kv_heads:
             raise ValueError(f"{heads} query heads over {kv_heads} key / value heads")
@@ -309,31 +326,87 @@ class QKNormAttention(nn.Module):
         self.own_kv = kv_from is None
         if kv_from is not None and (kv_from.kv_heads, kv_from.dim, kv_from.vdim) != (kv_heads, dim, vdim):
             raise ValueError("a layer that reads another layer's keys and values has its key / value heads and sizes")
-        parts = {"q": heads * self.dim_pad}
-        if self.own_kv:
-            parts.update(k=kv_heads * self.dim_pad, v=kv_heads * self.vdim_pad)
-        self.proj = StackedLinear(width, parts, dtype=dtype)
-        self.offsets = tuple(self.proj.offsets.get(n, 0) for n in ("q", "k", "v"))
-        self.q_norm = _param(self.dim_pad, dtype=dtype)
-        self.k_norm = _param(self.dim_pad, dtype=dtype) if self.own_kv else None
-        self.out_proj = _param(width, heads * self.vdim_pad, dtype=dtype)
-        self.rotation = ("rope_angles", tuple(inv_freq.tolist()))
-        self.register_buffer("inv_freq", inv_freq.double().to(torch.get_default_device()), persistent=False)
-        self.attn = Attention(heads, self.dim_pad, scale, kv_heads, cache_idx, sliding_window=window)
+        self.runs, self.whole_row_norm, self.interleaved, self.q_temp = runs, whole_row_norm, interleaved, q_temp
+        self.proj_bias, self.gated = proj_bias, gated
+        self.out_width = heads * self.vdim_pad
+        rows = (heads, kv_heads) if whole_row_norm else (1, 1)
+        self.q_norm = _param(rows[0] * self.dim_pad, dtype=dtype)
+        self.k_norm = _param(rows[1] * self.dim_pad, dtype=dtype) if self.own_kv else None
+        self.rotation = None
+        if inv_freq is not None:
+            self.rotation = ("rope_angles", tuple(inv_freq.tolist()))
+            self.register_buffer("inv_freq", inv_freq.double().to(torch.get_default_device()), persistent=False)
+        self.attn = Attention(heads, self.dim_pad, scale, kv_heads, cache_idx, sliding_window=window, softcap=softcap)
+        self.attn.out_scale = out_scale
+        self.sinks = _param(heads, dtype=torch.float32) if sinks else None
+        self.attn.sinks = self.sinks
+        self.rel = None
+        if bias_rows:
+            index = distance_buckets(bias_rows, bias_far)
+            self.rel = _param(bias_rows, heads, dtype=dtype)
+            self.register_buffer("distance_bias", torch.zeros(heads, len(index), dtype=torch.float32), persistent=False)
+            self.buckets = index
+            self.attn.distance_bias = self.distance_bias
+        if standalone:
+            self.proj = StackedLinear(width, self.in_parts(), ("q", "k", "v") if proj_bias else (), dtype=dtype)
+            self.attach(self.proj)
+            self.out_proj = _param(width, self.out_width, dtype=dtype)
 
-    def slots(self) -> dict:
-        """Tensor name -> (memory it is copied to, its shape in a checkpoint)."""
+    # ---- the products around it -----------------------------------------------------------------------------------
+    def in_parts(self) -> dict:
+        parts = {"q": self.heads * self.dim_pad}
+        if self.own_kv:
+            parts.update(k=self.kv_heads * self.dim_pad, v=self.kv_heads * self.vdim_pad)
+        if self.gated:
+            parts["g"] = self.out_width
+        return parts
+
+    def attach(self, proj: StackedLinear, prefix: str = "") -> None:
+        """The product that yields q, k, v (and g) as its parts ``prefix + name``."""
+        self.prefix = prefix
+        self.offsets = tuple(proj.offsets.get(prefix + n, 0) for n in ("q", "k", "v"))
+        self.gate_offset = proj.offsets.get(prefix + "g", 0)
+
+    def finalize_weights(self) -> None:
+        if self.rel is not None:
+            self.distance_bias.copy_(self.rel.data.float()[self.buckets].t())
+
+    def in_slots(self, proj: StackedLinear) -> dict:
+        """Tensor name -> (memory it is copied to, its shape in a checkpoint), without the output product."""
         def heads(name, n, size, pad):
-            return self.proj.rows(name).view(n, pad, self.width)[:, :size], (n * size, self.width)
+            return proj.rows(self.prefix + name).view(n, pad, self.width)[:, :size], (n * size, self.width)
 
-        out = {"q": heads("q", self.heads, self.dim, self.dim_pad), "q.norm": self.q_norm.data[: self.dim],
-               "o": (self.out_proj.data.view(self.width, self.heads, self.vdim_pad)[..., : self.vdim],
-                     (self.width, self.heads * self.vdim))}
+        def bias(name, n, size, pad):
+            return proj.bias_rows(self.prefix + name).view(n, pad)[:, :size], (n * size,)
+
+        def norm(w, n):
+            return (w.data.view(n, self.dim_pad)[:, : self.dim], (n * self.dim,)) if self.whole_row_norm else w.data[: self.dim]
+
+        sizes = {"q": (self.heads, self.dim, self.dim_pad)}
+        out = {"q.norm": norm(self.q_norm, self.heads)}
         if self.own_kv:
-            out.update({"k": heads("k", self.kv_heads, self.dim, self.dim_pad), "k.norm": self.k_norm.data[: self.dim],
-                        "v": heads("v", self.kv_heads, self.vdim, self.vdim_pad)})
+            sizes.update(k=(self.kv_heads, self.dim, self.dim_pad), v=(self.kv_heads, self.vdim, self.vdim_pad))
+            out["k.norm"] = norm(self.k_norm, self.kv_heads)
+        for name, s in sizes.items():
+            out[name] = heads(name, *s)
+            if self.proj_bias:
+                out[name + ".b"] = bias(name, *s)
+        if self.gated:
+            out["g"] = heads("g", self.heads, self.vdim, self.vdim_pad)
+        if self.sinks is not None:
+            out["sink"] = self.sinks.data
+        if self.rel is not None:
+            out["rel"] = self.rel.data
         return out
 
+    def out_slot(self, weight: torch.Tensor) -> tuple:
+        """The same for the output product, whose columns for this layer are ``weight [width, out_width]``."""
+        return (weight.unflatten(1, (self.heads, self.vdim_pad))[..., : self.vdim], (self.width, self.heads * self.vdim))
+
+    def slots(self) -> dict:
+        return {**self.in_slots(self.proj), "o": self.out_slot(self.out_proj.data)}
+
+    # ---- cache ------------------------------------------------------------------------------------------------------
     def decode_workspace_floats(self, batch: int, max_seq_len: int) -> int:
         """What the split decode of ``batch`` rows needs for its partial results (0: it does not split)."""
         tiles = -(-(self.heads // self.kv_heads) // 16)
@@ -341,21 +414,49 @@ class QKNormAttention(nn.Module):
         return n * batch * self.heads * (self.vdim_pad + 1) if n > 1 else 0
 
     def cache_elems_per_token(self) -> int:
-        return self.kv_heads * (self.dim_pad + self.vdim_pad) if self.own_kv else 0
+        return self.runs * self.kv_heads * (self.dim_pad + self.vdim_pad) if self.own_kv else 0
 
     def allocate_kv_cache(self, num_blocks: int, block_size: int, device):
         return (PagedGQABackend.allocate_pages(num_blocks, block_size, self.kv_heads, self.dim_pad, self.vdim_pad,
                                                self.q_norm.dtype, device), None)
 
-    def forward(self, positions: torch.Tensor, h: torch.Tensor) -> torch.Tensor:
+    # ---- forward ----------------------------------------------------------------------------------------------------
+    def mix(self, positions: torch.Tensor, h: torch.Tensor, p: torch.Tensor, out: torch.Tensor, run: int = 0) -> None:
+        """From the input product's rows ``p`` to the output product's operand ``out [T, out_width]``."""
         ctx = get_forward_context()
         md = ctx.attn_metadata
-        cache = ctx.kv_caches[self.attn.layer_idx][0]
+        T = p.shape[0]
+        cache = ctx.kv_caches[self.attn.layer_idx + run][0]
         kv = PagedGQABackend.views(cache, md.block_size, self.kv_heads, self.dim_pad, self.vdim_pad)
-        angles = ctx.extra.get(self.rotation)                 # one table per step and rotation, shared by the layers
-        if angles is None:
-            angles = ctx.extra[self.rotation] = ops.rope_angles(positions, self.inv_freq, h.shape[0])
-        q = ops.head_norm_rope(self.proj(h), self.offsets, self.q_norm, self.k_norm, self.heads, self.dim, angles,
-                               kv if self.own_kv else None, md.slot_mapping, self.eps)
-        o = self.attn.attend(q, md, kv)
-        return ops.gemm(o.view(h.shape[0], self.heads * self.vdim_pad), self.out_proj)
+        angles = None
+        if self.rotation is not None:                         # one table per step and rotation, shared by the layers
+            angles = ctx.extra.get(self.rotation)
+            if angles is None:
+                angles = ctx.extra[self.rotation] = ops.rope_angles(positions, self.inv_freq, T)
+        q = ops.head_norm_rope(p, self.offsets, self.q_norm, self.k_norm, self.heads, self.dim, angles,
+                               kv if self.own_kv else None, md.slot_mapping, self.eps, whole_row=self.whole_row_norm,
+                               interleaved=self.interleaved, q_temp=(positions, *self.q_temp) if self.q_temp else None)
+        gate = None
+        if self.gated:
+            gate = p[:, self.gate_offset: self.gate_offset + self.out_width]
+        self.attn.attend(q, md, kv, out=out.unflatten(1, (self.heads, self.vdim_pad)), gate=gate)
+
+    def forward(self, positions: torch.Tensor, h: torch.Tensor) -> torch.Tensor:
+        o = torch.empty(h.shape[0], self.out_width, dtype=h.dtype, device=h.device)
+        self.mix(positions, h, self.proj(h), o)
+        return ops.gemm(o, self.out_proj)
+
+
+def distance_buckets(rows: int, far: int) -> list:
+    """Row of a learned distance bias for every distance 0, 1, ... up to the first that has the last row, which all larger ones
+    share: ``rows / 2`` rows for single distances, the others on a logarithmic scale that ends at ``far``."""
+    half = rows // 2
+    if half < 1 or far <= half:
+        raise ValueError(f"a distance bias of {rows} rows up to distance {far}")
+    out = list(range(half))
+    while out[-1] != rows - 1:
+        n = len(out)
+        x = math.log(n / half) / math.log(far / half) * (rows - half)
+        whole = round(x)                               # a quotient of logarithms that is a whole number, up to rounding
+        out.append(min(rows - 1, half + (whole if abs(x - whole) < 1e-9 else math.floor(x))))
+    return out

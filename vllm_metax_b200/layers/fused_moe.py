@@ -12,7 +12,8 @@ Data flow on one rank (bf16):
 
 Weights: ``w13 [E_local, 2I, H]`` with gate/up rows interleaved (row 2j = gate_j, 2j+1 = up_j),
 ``w2 [E_local, H, I]``.  Experts without a gate (``gated=False``) hold ``w13 [E_local, I, H]`` and apply their activation
-in the same epilogue.
+in the same epilogue.  ``weight_input``: the routing weight multiplies the expert's input (in the gather) and the outputs are
+added as they are.
 
 Identity experts (``num_identity``): the router's last outputs name experts that hand their input through.  They have no
 weights and no rows; the pairs routed to them add ``w_k * x`` where the rows are combined.
@@ -57,26 +58,29 @@ BLOCK_M = 128
 def fused_experts(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_weights: torch.Tensor,
                   topk_ids: torch.Tensor, num_local_experts: int, expert_map: Optional[torch.Tensor] = None,
                   shared_out: Optional[torch.Tensor] = None, epi: int = ops.EPI_CODES["silu_gate"],
-                  identity_from: Optional[int] = None) -> torch.Tensor:
+                  identity_from: Optional[int] = None, epi_params: Optional[torch.Tensor] = None,
+                  weight_input: bool = False) -> torch.Tensor:
     """Expert MLPs for the pairs routed to this rank's experts; returns ``[T, H]`` (partial sum
     when ``expert_map`` drops pairs owned by other ranks).  Pairs with ids from ``identity_from`` on hand ``x`` through."""
     return expert_rows(x, w13, w2, topk_weights, topk_ids, num_local_experts, expert_map, shared_out, epi,
-                       identity_from).combined()
+                       identity_from, epi_params, weight_input).combined()
 
 
 def expert_rows(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_weights: torch.Tensor, topk_ids: torch.Tensor,
                 num_local_experts: int, expert_map: Optional[torch.Tensor] = None, shared_out: Optional[torch.Tensor] = None,
-                epi: int = ops.EPI_CODES["silu_gate"], identity_from: Optional[int] = None) -> ExpertRows:
+                epi: int = ops.EPI_CODES["silu_gate"], identity_from: Optional[int] = None,
+                epi_params: Optional[torch.Tensor] = None, weight_input: bool = False) -> ExpertRows:
     """The experts' output rows before they are combined."""
     topk = topk_ids.shape[1]
     sorted_ids, block_expert, total, inv = ops.moe_align_block_size(topk_ids, BLOCK_M, num_local_experts,
                                                                     expert_map, want_inverse=True)
-    a = ops.moe_gather(x, sorted_ids, total, topk)
-    h = ops.gemm_grouped(a, w13, block_expert, total, epi=epi)
+    topk_weights = topk_weights.contiguous()
+    a = ops.moe_gather(x, sorted_ids, total, topk, topk_weights if weight_input else None)
+    h = ops.gemm_grouped(a, w13, block_expert, total, epi=epi, act_params=epi_params)
     y = ops.gemm_grouped(h, w2, block_expert, total, epi=0)
     ident = identity_from is not None
-    return ExpertRows(y, topk_weights.contiguous(), inv, topk_ids if ident else None, x if ident else None, identity_from or 0,
-                      shared_out)
+    return ExpertRows(y, None if weight_input else topk_weights, inv, topk_ids if ident else None, x if ident else None,
+                      identity_from or 0, shared_out, topk)
 
 
 class FusedMoE(nn.Module):
@@ -85,15 +89,21 @@ class FusedMoE(nn.Module):
                  use_grouped_topk: bool = False, num_expert_group: int = 1, topk_group: int = 1,
                  routed_scaling_factor: float = 1.0, e_score_correction_bias: bool = False,
                  reduce_results: bool = True, quant_method=None, prefix: str = "",
-                 gated: bool = True, activation: str = "silu", num_identity: int = 0):
+                 gated: bool = True, activation: str = "silu", num_identity: int = 0,
+                 activation_params: tuple = (), weight_input: bool = False):
         super().__init__()
+        assert not weight_input or (quant_method is None and num_identity == 0), "weighted inputs: unquantised experts"
+        self.weight_input = weight_input          # the routing weight multiplies the expert's input, not its output
         assert num_identity == 0 or quant_method is None, "identity experts beside unquantised ones"
         self.num_identity = num_identity          # router outputs past the experts that hand the input through
-        # gated: SiLU(gate) * up over interleaved rows; otherwise one up projection through `activation`
-        assert not gated or activation == "silu", "gated experts use the SiLU gate"
-        assert gated or quant_method is None, "quantised experts are gated"
+        # gated: activation(gate, up) over interleaved rows; otherwise one up projection through `activation`
+        assert quant_method is None or (gated and activation == "silu"), "quantised experts use the SiLU gate"
         self.gated = gated
-        self.epi = ops.EPI_CODES["silu_gate" if gated else activation]
+        self.epi = ops.EPI_CODES[activation + "_gate" if gated else activation]
+        if activation_params:
+            self.register_buffer("epi_params", torch.tensor(activation_params, dtype=torch.float32), persistent=False)
+        else:
+            self.epi_params = None
         self.num_experts, self.top_k = num_experts, top_k
         self.hidden_size, self.intermediate_size = hidden_size, intermediate_size
         self.renormalize, self.scoring_func = renormalize, scoring_func
@@ -121,6 +131,7 @@ class FusedMoE(nn.Module):
             self.w2_weight = nn.Parameter(torch.empty(self.num_local, hidden_size, intermediate_size, dtype=dtype),
                                           requires_grad=False)
         assert num_identity == 0 or not (self.eplb or self.dp > 1), "identity experts: one replica, no load balancing"
+        assert not weight_input or self.dp == 1, "weighted inputs: one replica"
         self.e_score_correction_bias = (nn.Parameter(torch.zeros(num_experts + num_identity, dtype=torch.float32), requires_grad=False)
                                         if e_score_correction_bias else None)
         if self.ep > 1:
@@ -141,7 +152,8 @@ class FusedMoE(nn.Module):
             self.register_buffer("expert_load", torch.zeros(num_experts, dtype=torch.int64), persistent=False)
 
     # ---- load balancing ---------------------------------------------------------
-    _EPLB_BUFFERS = ("phy2log", "log2phy", "logcnt", "expert_load", "expert_map", "e_score_correction_bias")
+    _EPLB_BUFFERS = ("phy2log", "log2phy", "logcnt", "expert_load", "expert_map", "e_score_correction_bias",
+                     "epi_params")
 
     def _local_slots(self, expert_id: int) -> list:
         """Local slot indices that hold logical expert ``expert_id`` on this rank."""
@@ -240,7 +252,7 @@ class FusedMoE(nn.Module):
         qm = self.quant_method
         if qm is not None:
             return qm.apply_sorted(self, a, a_scale, block_expert, total)
-        h = ops.gemm_grouped(a, self.w13_weight, block_expert, total, epi=self.epi)
+        h = ops.gemm_grouped(a, self.w13_weight, block_expert, total, epi=self.epi, act_params=self.epi_params)
         return ops.gemm_grouped(h, self.w2_weight, block_expert, total)
 
     def _forward_sp(self, x: torch.Tensor, router_logits: torch.Tensor,
@@ -287,7 +299,8 @@ class FusedMoE(nn.Module):
                 part = qm.apply(self, h_all, w_all, ids_all.to(torch.int32), None)
             else:
                 part = fused_experts(h_all, self.w13_weight, self.w2_weight, w_all, ids_all.to(torch.int32),
-                                     self.num_local, self.expert_map, None, self.epi)
+                                     self.num_local, self.expert_map, None, self.epi, epi_params=self.epi_params,
+                                     weight_input=self.weight_input)
             mine = mgr.combine(part)
         y = tpg.all_gatherv(mine.contiguous(), sizes)
         if shared_out is not None:       # shared experts are tensor-parallel: their partial sums still need the reduction
@@ -307,6 +320,8 @@ class FusedMoE(nn.Module):
         ``B200_MOE_A2A=1`` for the NVLink kernels, or ``use_sequence_parallel_moe`` with either backend)."""
         if self.ep == 1:
             return False
+        if self.weight_input:
+            return False
         if self.dp > 1:
             return True
         if self._sp_config and self.num_identity == 0:
@@ -325,7 +340,7 @@ class FusedMoE(nn.Module):
             return self.forward(x, router_logits, shared_out)
         w, ids = self.route(router_logits)
         return expert_rows(x, self.w13_weight, self.w2_weight, w, ids, self.num_local, self.expert_map, shared_out, self.epi,
-                           self.identity_from())
+                           self.identity_from(), self.epi_params, self.weight_input)
 
     def forward_reduced(self, x: torch.Tensor, router_logits: torch.Tensor,
                         shared_out: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -350,7 +365,7 @@ class FusedMoE(nn.Module):
             if self.quant_method is not None:
                 return self.quant_method.apply(self, xs, ws, idss, shared)
             return fused_experts(xs, self.w13_weight, self.w2_weight, ws, idss, self.num_local, self.expert_map, shared, self.epi,
-                                 self.identity_from())
+                                 self.identity_from(), self.epi_params, self.weight_input)
 
         chunk = int(envs.B200_FUSED_MOE_CHUNK_SIZE)
         T = x.shape[0]

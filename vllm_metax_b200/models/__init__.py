@@ -54,6 +54,7 @@ _MODELS: dict[str, tuple[str, str]] = {
     "InternS1ForConditionalGeneration": ("internvl", "InternVLForConditionalGeneration"),    # the same graph, other decoder
     "Naguzen": ("naguzen", "NaguzenForCausalLM"),
     "Pupalorn": ("pupalorn", "PupalornForCausalLM"),
+    "Luluzen": ("luluzen", "LuluzenForCausalLM"),
     "MambaForCausalLM": ("mamba", "MambaForCausalLM"),
     "Qwen3NextForCausalLM": ("qwen3_next", "Qwen3NextForCausalLM"),
     "Glm4MoeForCausalLM": ("moe_family", "Glm4MoeForCausalLM"),

@@ -349,8 +349,24 @@ def epilogue_activation(y: torch.Tensor, act: str, params: Optional[torch.Tensor
         return torch.exp(torch.nn.functional.logsigmoid(y) * params.float()[0])
     if act == "relu2":
         return torch.relu(y).square()
+    if act == "softcap":
+        return params.float() * torch.tanh(y / params.float())
+    if act == "softplus_decay":
+        return torch.exp(-params.float() * torch.nn.functional.softplus(y, threshold=50.0))
     a, b = params.float()
     return torch.where(y > 0, a * y * y, b * (torch.expm1(y.clamp(max=0)) - y)) + 0.5 * y
+
+
+def epilogue_gate(y: torch.Tensor, act: str, params: Optional[torch.Tensor]) -> torch.Tensor:
+    """The gated GEMM epilogues over interleaved (gate, up) columns, fp32."""
+    g, u = y[:, 0::2].float(), y[:, 1::2].float()
+    if act == "silu_gate":
+        return torch.nn.functional.silu(g) * u
+    if act == "gelu_tanh_gate":
+        return torch.nn.functional.gelu(g, approximate="tanh") * u
+    limit, alpha = params.float()
+    g = torch.minimum(g, limit)
+    return g * torch.sigmoid(alpha * g) * (torch.maximum(torch.minimum(u, limit), -limit) + 1.0)
 
 
 def rotate_half(x: torch.Tensor, inv_freq: torch.Tensor, positions: torch.Tensor) -> torch.Tensor:
@@ -359,10 +375,14 @@ def rotate_half(x: torch.Tensor, inv_freq: torch.Tensor, positions: torch.Tensor
     return rotate_half_by(x, torch.stack([torch.cos(a), torch.sin(a)], 1))
 
 
-def rotate_half_by(x: torch.Tensor, angles: torch.Tensor) -> torch.Tensor:
-    """The same by cosines and sines ``[T, 2, half]``."""
+def rotate_half_by(x: torch.Tensor, angles: torch.Tensor, interleaved: bool = False) -> torch.Tensor:
+    """The same by cosines and sines ``[T, 2, half]``; ``interleaved``: pairs (2i, 2i + 1)."""
     half = angles.shape[-1]
     c, s = angles[:, :1], angles[:, 1:]
+    if interleaved:
+        u, v = x[..., 0: 2 * half: 2].float(), x[..., 1: 2 * half: 2].float()
+        pairs = torch.stack([u * c - v * s, v * c + u * s], -1).flatten(-2)
+        return torch.cat([pairs.to(x.dtype), x[..., 2 * half:]], -1)
     u, v = x[..., :half].float(), x[..., half: 2 * half].float()
     return torch.cat([(u * c - v * s).to(x.dtype), (v * c + u * s).to(x.dtype), x[..., 2 * half:]], -1)
 
@@ -473,7 +493,7 @@ def convert_fp8(dst, src, scale: float = 1.0):
 # --------------------------------------------------------------------------- attention
 def attention_core(q, k, v, scale, causal_offset: Optional[int] = None, window: int = -1,
                    softcap: float = 0.0, sinks: Optional[torch.Tensor] = None,
-                   alibi_slopes: Optional[torch.Tensor] = None):
+                   alibi_slopes: Optional[torch.Tensor] = None, distance_bias: Optional[torch.Tensor] = None):
     """Dense softmax attention for one sequence.
 
     ``q [Lq, Hq, D]``, ``k [Lk, Hkv, D]``, ``v [Lk, Hkv, Dv]`` (fp32).  Query row i
@@ -497,6 +517,8 @@ def attention_core(q, k, v, scale, causal_offset: Optional[int] = None, window: 
         qpos = torch.full((Lq, 1), Lk - 1, device=q.device)
     if alibi_slopes is not None:
         s = s + alibi_slopes.float()[:, None, None] * (kpos - qpos)[None].float()
+    if distance_bias is not None:
+        s = s + distance_bias.float()[:, (qpos - kpos).clamp(0, distance_bias.shape[1] - 1)]
     mask = torch.zeros(Lq, Lk, dtype=torch.bool, device=q.device)
     if causal_offset is not None:
         mask |= kpos > qpos
@@ -516,7 +538,8 @@ def attention_core(q, k, v, scale, causal_offset: Optional[int] = None, window: 
 
 def paged_attention(q, kv_cache, block_table, seq_lens, query_start_loc, scale, *, kv_scales=None,
                     window: int = -1, softcap: float = 0.0, sinks=None, alibi_slopes=None,
-                    k_scale: float = 1.0, v_scale: float = 1.0, causal: bool = True, return_lse: bool = False):
+                    k_scale: float = 1.0, v_scale: float = 1.0, causal: bool = True, return_lse: bool = False,
+                    distance_bias=None, gate=None, out_scale: float = 1.0):
     """Varlen attention over the paged cache (prefill, chunked prefill and decode).
 
     ``q [T, Hq, D]`` holds the new tokens of every sequence back to back
@@ -539,10 +562,13 @@ def paged_attention(q, kv_cache, block_table, seq_lens, query_start_loc, scale, 
         k, v = gather_paged_kv(kv_cache, block_table[b], sl[b], kv_scales, k_scale, v_scale)
         o, lse = attention_core(q[s0:s1].float(), k, v, scale,
                                 causal_offset=(sl[b] - (s1 - s0)) if causal else None,
-                                window=window, softcap=softcap, sinks=sinks, alibi_slopes=alibi_slopes)
+                                window=window, softcap=softcap, sinks=sinks, alibi_slopes=alibi_slopes,
+                                distance_bias=distance_bias)
         out[s0:s1] = o
         lse_all[:, s0:s1] = lse
-    out = out.to(q.dtype)
+    if gate is not None:
+        out = out * torch.sigmoid(gate.float()).reshape(out.shape)
+    out = (out * out_scale).to(q.dtype)
     return (out, lse_all) if return_lse else out
 
 

@@ -20,18 +20,30 @@ class ExpertRows:
     """What the grouped expert products left: the rows of pair (t, k) is ``rows[inv_pos[t * topk + k]]``; pairs whose id is at
     least ``identity_from`` are identity experts and stand for the token's own row of ``through``."""
     rows: torch.Tensor                       # [R, width], expert-sorted
-    weights: torch.Tensor                    # fp32 [T, topk]
+    weights: Optional[torch.Tensor]          # fp32 [T, topk]; None: the rows are added as they are (weighted inputs)
     inv_pos: torch.Tensor                    # int32 [T * topk], -1: computed elsewhere
     ids: Optional[torch.Tensor] = None       # int32 [T, topk]
     through: Optional[torch.Tensor] = None   # [T, width]
     identity_from: int = 0
     shared: Optional[torch.Tensor] = None    # [T, width]
+    top: int = 0                             # pairs per token (where there are no weights to tell)
+
+    @property
+    def topk(self) -> int:
+        return self.top if self.weights is None else self.weights.shape[1]
+
+    @property
+    def tokens(self) -> int:
+        return self.inv_pos.numel() // self.topk
 
     def combined(self) -> torch.Tensor:
         from .. import _custom_ops as ops
 
         identity = None if self.through is None else (self.ids, self.through, self.identity_from)
-        return ops.moe_combine(self.rows, self.weights, self.inv_pos, self.weights.shape[0], self.shared, identity)
+        w = self.weights
+        if w is None:
+            w = torch.ones(self.tokens, self.topk, dtype=torch.float32, device=self.rows.device)
+        return ops.moe_combine(self.rows, w, self.inv_pos, self.tokens, self.shared, identity)
 
 
 def normed(y: torch.Tensor, gain: torch.Tensor, eps: float) -> torch.Tensor:
@@ -46,7 +58,7 @@ def boundary_norm(y: Union[torch.Tensor, ExpertRows], x: Optional[torch.Tensor],
 
     late = isinstance(y, ExpertRows)
     rows = y.rows if late else y
-    T = y.weights.shape[0] if late else y.shape[0]
+    T = y.tokens if late else y.shape[0]
     if not ops._use_cuda(rows):
         yt = y.combined() if late else y
         xn = yt.float() if x is None else x + normed(yt, gain, eps)
