@@ -131,16 +131,21 @@ def gated_window_attention(h, w, pre, m, eps):
 
 
 # ------------------------------------------------------------------ recurrences
+def decayed_states(q, k, v, decay):
+    """``q, k [T, H, D]``, ``v [T, H, V]``, ``decay [H]``: S <- decay S + k v^T, read-out S^T q."""
+    S, o = torch.zeros(q.shape[1], q.shape[2], v.shape[2], dtype=F64), []
+    for t in range(q.shape[0]):
+        S = decay[:, None, None] * S + k[t][:, :, None] * v[t][:, None, :]
+        o.append(torch.einsum("hdv,hd->hv", S, q[t]))
+    return torch.stack(o)
+
+
 def lightning(h, w, pre, m, eps):
     T, H = h.shape[0], m["heads"]
     q, k = (silu(linear(w, pre + n, h)).view(T, H, m["dim"]) for n in "qk")
     v = silu(linear(w, pre + "v", h)).view(T, H, m["vdim"])
-    decay = torch.tensor(m["decay"], dtype=F64)[:, None, None]
-    S, o = torch.zeros(H, m["dim"], m["vdim"], dtype=F64), []
-    for t in range(T):
-        S = decay * S + k[t][:, :, None] * v[t][:, None, :]
-        o.append(torch.einsum("hdv,hd->hv", S, q[t]))
-    o = unit_rms(torch.stack(o).reshape(T, -1), eps) * get(w, pre + "norm")
+    o = decayed_states(q, k, v, torch.tensor(m["decay"], dtype=F64))
+    o = unit_rms(o.reshape(T, -1), eps) * get(w, pre + "norm")
     return linear(w, pre + "o", o * sigmoid(linear(w, pre + "g", h)))
 
 
@@ -177,13 +182,10 @@ def gated_delta(h, w, pre, m, eps):
     return linear(w, pre + "o", o.reshape(T, -1) * gate)
 
 
-def matrix_memory(h, w, pre, m, eps):
-    T, H, D, V = h.shape[0], m["heads"], m["dim"], m["vdim"]
-    q = linear(w, pre + "q", h).view(T, H, D) * D ** -0.5
-    k, v = linear(w, pre + "k", h).view(T, H, D), linear(w, pre + "v", h).view(T, H, V)
-    i = cap(linear(w, pre + "i", h), m["gate_cap"])
-    f = -softplus(-cap(linear(w, pre + "f", h), m["gate_cap"]))
-    S, n, top, out = torch.zeros(H, D, V, dtype=F64), torch.zeros(H, D, dtype=F64), torch.zeros(H, dtype=F64), []
+def memory_states(q, k, v, i, f):
+    """``q, k [T, H, D]``, ``v [T, H, V]``, log gates ``i, f [T, H]``: the stabilised matrix memory with its normaliser."""
+    T, H, D = q.shape
+    S, n, top, out = torch.zeros(H, D, v.shape[2], dtype=F64), torch.zeros(H, D, dtype=F64), torch.zeros(H, dtype=F64), []
     for t in range(T):
         new = torch.maximum(f[t] + top, i[t])
         keep, add, top = torch.exp(f[t] + top - new), torch.exp(i[t] - new), new
@@ -191,7 +193,16 @@ def matrix_memory(h, w, pre, m, eps):
         n = keep[:, None] * n + add[:, None] * k[t]
         den = torch.maximum((n * q[t]).sum(-1).abs(), torch.exp(-top)) + 1e-6
         out.append(torch.einsum("hdv,hd->hv", S, q[t]) / den[:, None])
-    o = unit_rms(torch.stack(out), eps).reshape(T, -1) * get(w, pre + "norm")
+    return torch.stack(out)
+
+
+def matrix_memory(h, w, pre, m, eps):
+    T, H, D, V = h.shape[0], m["heads"], m["dim"], m["vdim"]
+    q = linear(w, pre + "q", h).view(T, H, D) * D ** -0.5
+    k, v = linear(w, pre + "k", h).view(T, H, D), linear(w, pre + "v", h).view(T, H, V)
+    i = cap(linear(w, pre + "i", h), m["gate_cap"])
+    f = -softplus(-cap(linear(w, pre + "f", h), m["gate_cap"]))
+    o = unit_rms(memory_states(q, k, v, i, f), eps).reshape(T, -1) * get(w, pre + "norm")
     return linear(w, pre + "o", o * sigmoid(linear(w, pre + "g", h)))
 
 
@@ -262,3 +273,80 @@ def forward(tokens, w, cfg, residuals=None):
         if residuals is not None:
             residuals.append(x)
     return cap(layer_norm(x, w["final.norm"], eps) @ get(w, "embed").t(), float(cfg["logit_softcap"]))
+
+
+# ------------------------------------------------------------------ checkpoints for tests
+def tensor_shapes(cfg, low=lambda i: (6 + 2 * i, 5 + i, 11)):
+    """``low(i)``: what the config does not carry - rows of layer i's distance bias, ranks of its decay and gate projections."""
+    W = cfg["width"]
+    out = {"embed": (cfg["vocab"], W), "final.norm": (W,)}
+    if cfg.get("loop"):
+        out.update({"loop.in": (W, 2 * W), "loop.step": (cfg["loop"]["times"], W)})
+    for i, l in enumerate(cfg["layers"]):
+        p, m, f = f"l{i}.", l["mixer"], l.get("mlp")
+        out[p + "norm1"] = (W,)
+
+        def linear_attention(pre, m, gated=True):
+            k, v = m["heads"] * m["dim"], m["heads"] * m["vdim"]
+            out.update({pre + "q": (k, W), pre + "k": (k, W), pre + "v": (v, W), pre + "g": (v, W), pre + "o": (W, v),
+                        pre + "norm": (v,)})
+
+        if l["type"] == "lightning":
+            linear_attention(p + "mix.", m)
+        else:
+            a, r, pre = m["left"], m["right"], p + "mix.left."
+            q, k, v, o = a["heads"] * a["dim"], a["kv_heads"] * a["dim"], a["kv_heads"] * a["vdim"], a["heads"] * a["vdim"]
+            out.update({pre + "q": (q, W), pre + "k": (k, W), pre + "v": (v, W), pre + "o": (W, o)})
+            rows, ra, rg = low(i)
+            if l["type"] == "parallel":
+                out.update({pre + "q.b": (q,), pre + "k.b": (k,), pre + "v.b": (v,), pre + "q.norm": (a["dim"],),
+                            pre + "k.norm": (a["dim"],), pre + "rel": (rows, a["heads"])})
+                pre = p + "mix.right."
+                H, k, v = r["heads"], r["kv_heads"] * r["dim"], r["heads"] * r["vdim"]
+                out.update({pre + "q": (k, W), pre + "k": (k, W), pre + "v": (v, W), pre + "q.conv": (k, r["conv"]),
+                            pre + "k.conv": (k, r["conv"]), pre + "v.conv": (v, r["conv"]), pre + "b": (H, W),
+                            pre + "A_log": (H,), pre + "norm": (r["vdim"],), pre + "a1": (ra, W), pre + "a2": (H * r["dim"], ra),
+                            pre + "dt_bias": (H * r["dim"],), pre + "g1": (rg, W), pre + "g2": (v, rg), pre + "o": (W, v)})
+            else:
+                out.update({pre + "q.norm": (q,), pre + "k.norm": (k,), pre + "sink": (a["heads"],), pre + "g": (o, W)})
+                pre, H = p + "mix.right.", r["heads"]
+                linear_attention(pre, r)
+                out.update({pre + "i": (H, W), pre + "i.b": (H,), pre + "f": (H, W), pre + "f.b": (H,)})
+        if f is not None:
+            out[p + "norm2"] = (W,)
+            if f["kind"] == "dense":
+                out.update({p + "mlp.gate": (f["ff"], W), p + "mlp.up": (f["ff"], W), p + "mlp.down": (W, f["ff"])})
+            else:
+                out[p + "mlp.router"] = (f["router"]["experts"], W)
+                for e in range(f["router"]["experts"]):
+                    ff, q = f["expert"]["ff"], f"{p}mlp.e{e}."
+                    out.update({q + "gate": (ff, W), q + "up": (ff, W), q + "down": (W, ff)})
+    return out
+
+
+def random_weights(cfg, seed=0, **kw):
+    """bf16 tensors under the checkpoint's names; norm weights around one, biases of the forget gates that keep states alive,
+    sinks and distance biases of the size of scores."""
+    g = torch.Generator().manual_seed(seed)
+    out = {}
+    for name, shape in tensor_shapes(cfg, **kw).items():
+        t = torch.randn(*shape, generator=g)
+        leaf = name.split(".")[-1]
+        if "norm" in leaf:
+            t = 1.0 + 0.3 * t
+        elif leaf == "A_log":
+            t = 0.5 * t - 1.0
+        elif leaf == "dt_bias":
+            t = t - 2.0
+        elif name.endswith(".f.b"):
+            t = t + 4.0
+        elif leaf == "conv":
+            t = 0.5 * t
+        elif leaf in ("rel", "sink"):
+            t = 1.5 * t
+        elif leaf in ("step", "b") and len(shape) < 2 or name == "loop.step":
+            t = 0.3 * t
+        elif name != "embed":
+            t = t * shape[-1] ** -0.5 * (2.0 if leaf == "router" else 1.0)
+        out[name] = t.to(torch.bfloat16)
+    return out

@@ -58,7 +58,7 @@ inline PagedViews paged_views(const Tensor& k, const Tensor& v) {
               k.scalar_type() == v.scalar_type(), "paged K / V must be [num_blocks, block_size, kv_heads, head] views");
   for (const Tensor* t : {&k, &v})
     TORCH_CHECK(t->stride(3) == 1 && t->stride(2) == t->size(3) && t->stride(1) == t->size(2) * t->size(3) &&
-                t->stride(0) == k.stride(0), "paged K / V: dense token rows and one page stride");
+                (t->size(0) == 1 || t->stride(0) == k.stride(0)), "paged K / V: dense token rows and one page stride");
   return {k.size(0), k.stride(0), (int)k.size(1), (int)k.size(2), (int)k.size(3), (int)v.size(3)};
 }
 
