@@ -18,7 +18,8 @@ iterations).  Two measurements per run:
 `--hybrid` instead prints one JSON line with the layer-list hybrid (Naguzen) beside its closest models at equal sizes:
 prefill and decode throughput, and every kernel of it against its roofline (utils/bench_hybrid.py; one GPU).
 `--shared-kv` does the same for the decoder with windowed, cross-layer-shared attention and identity experts (Pupalorn)
-beside Qwen3-MoE (utils/bench_shared_kv.py).
+beside Qwen3-MoE (utils/bench_shared_kv.py), and `--parallel` for the looped decoder with two mixers side by side (Luluzen)
+beside Qwen3-Next and Naguzen (utils/bench_parallel.py).
 `--impl reference` reports that the reference cannot be installed on this machine.
 """
 from __future__ import annotations
@@ -122,6 +123,8 @@ class ClockSampler:
 def layer_list_bench(args) -> None:
     if args.shared_kv:
         from vllm_metax_b200.utils.bench_shared_kv import SIZES, TITLE, kernel_rows, model_rows
+    elif args.parallel:
+        from vllm_metax_b200.utils.bench_parallel import SIZES, TITLE, kernel_rows, model_rows
     else:
         from vllm_metax_b200.utils.bench_hybrid import SIZES, TITLE, kernel_rows, model_rows
 
@@ -154,8 +157,10 @@ def main() -> None:
                     help="hybrid decoder (Naguzen) beside its closest models: throughput and kernel rooflines, one GPU")
     ap.add_argument("--shared-kv", action="store_true",
                     help="decoder with cross-layer-shared keys and values (Pupalorn) beside Qwen3-MoE, one GPU")
+    ap.add_argument("--parallel", action="store_true",
+                    help="looped decoder with two mixers side by side (Luluzen) beside Qwen3-Next and Naguzen, one GPU")
     args = ap.parse_args()
-    if args.hybrid or args.shared_kv:
+    if args.hybrid or args.shared_kv or args.parallel:
         return layer_list_bench(args)
     conf = CONFIGS[args.config]
     MODEL = conf["model"]
