@@ -490,20 +490,31 @@ def paged_attention_decode(q, kv_cache, block_table, seq_lens, scale, *, out=Non
     return res
 
 
+def distance_bias_tiles(bias, group: int):
+    """``bias [Hq, L]`` by distance in the layout of the prompt kernel: entries in the order of the keys (distances from L + 126
+    down to -127, clamped), times log2(e), the heads of a ``group`` that share a key head side by side."""
+    H, L = bias.shape
+    gp = group if 128 % group == 0 else 1
+    d = (L + 126 - torch.arange(L + 254, device=bias.device)).clamp(0, L - 1)
+    return (bias[:, d] * 1.4426950408889634).view(H // gp, gp, L + 254).transpose(1, 2).contiguous()
+
+
 def paged_attention_prefill(q, kv_cache, block_table, seq_lens, query_start_loc, scale, *, out=None, kv_scales=None,
                             max_q_len: int = 0, window: int = -1, softcap: float = 0.0, sinks=None, lse_out=None,
                             k_scale=1.0, v_scale=1.0, causal=True, max_seq_len: int = 0, alibi_slopes=None,
-                            distance_bias=None, gate=None, out_scale: float = 1.0):
+                            distance_bias=None, bias_tiles=None, gate=None, out_scale: float = 1.0):
     """Varlen prefill / chunked-prefill attention reading K, V from the paged cache (``distance_bias``, ``gate``,
-    ``out_scale`` as for decode)."""
+    ``out_scale`` as for decode; ``bias_tiles``: what ``distance_bias_tiles`` makes of the bias, where it is at hand)."""
     if _use_cuda(q):
         k, v = kv_views(kv_cache)
         out = torch.empty(q.shape[0], q.shape[1], v.shape[-1], dtype=q.dtype, device=q.device) if out is None else out
         B = seq_lens.shape[0]
         if k.dtype == q.dtype and q.dtype != torch.float32 and k.shape[-1] <= 192 and v.shape[-1] <= 128 and kv_scales is None:
+            if distance_bias is not None and bias_tiles is None:
+                bias_tiles = distance_bias_tiles(distance_bias, q.shape[1] // k.shape[2])
             torch.ops.b200.attention_prefill(out, q, k, v, block_table, seq_lens, query_start_loc, None,
                                              scale, window, softcap, sinks, lse_out, B, max_q_len or q.shape[0], causal,
-                                             alibi_slopes, distance_bias, gate, out_scale)
+                                             alibi_slopes, distance_bias, bias_tiles, gate, out_scale)
         else:
             # quantised caches / other head sizes: the split-KV kernel handles any query length in 16-row tiles
             paged_attention_decode(q, kv_cache, block_table, seq_lens, scale, out=out, kv_scales=kv_scales,

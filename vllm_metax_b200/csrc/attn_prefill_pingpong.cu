@@ -285,11 +285,10 @@ attn_prefill_pp_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     const int lo = (p.window > 0) ? max(0, lim - p.window) : 0;
     const float sl2 = p.scale * 1.4426950408889634f;
     const uint32_t lane_base = ((uint32_t)(quarter * 32)) << 16;
-    const bool plain = !(p.softcap > 0.f) && p.alibi_slopes == nullptr && p.bias == nullptr;
-    const float* bias = p.bias != nullptr ? p.bias + (int64_t)hq * p.bias_len : nullptr;      // by distance
-    const float bias_far = bias != nullptr ? bias[p.bias_len - 1] * 1.4426950408889634f : 0.f;
+    // bias by distance (log2 units): rows of the table lie as the keys do, the gp heads of a tile side by side
+    const float* bias = p.bias_tiles != nullptr ? p.bias_tiles + (int64_t)hg * (p.bias_len + 254) * p.gp + r % p.gp : nullptr;
+    const float bias_far = bias != nullptr ? bias[0] : 0.f;
     const float alibi2 = (p.alibi_slopes && row_valid) ? p.alibi_slopes[hq] * 1.4426950408889634f : 0.f;
-    const float mul = plain ? sl2 : 1.f;            // scores are kept raw on the plain path
     const int n_mine = t ? n_b : n_a;
     const uint32_t tmem_St = (t ? tmem_S1 : tmem_S0) + lane_base, tmem_Ot = (t ? tmem_O1 : tmem_O0) + lane_base;
     float m_run = -INFINITY, l_run = 0.f;
@@ -310,18 +309,30 @@ attn_prefill_pp_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       float s[BN];
 #pragma unroll
       for (int i = 0; i < BN; ++i) s[i] = __uint_as_float(sv[i]);
-      if (!plain) {
+      // the score of key i is s[i] * mul + off: raw scores keep their scale until the exponential
+      float mul = sl2, off = 0.f;
+      if (p.softcap > 0.f) {
+        softcap_row(s, p.scale, p.softcap);
+        mul = 1.f;
+      }
+      if (p.alibi_slopes != nullptr) {
 #pragma unroll
-        for (int i = 0; i < BN; ++i) {
-          const float base = (p.softcap > 0.f) ? softcap_score(s[i] * p.scale, p.softcap) * 1.4426950408889634f : s[i] * sl2;
-          s[i] = base + alibi2 * (float)(t0 + i - pos) + bias_far;
-        }
-        if (bias != nullptr && pos - (t0 + BN - 1) < p.bias_len - 1) {      // some keys of the tile are near
+        for (int i = 0; i < BN; ++i) s[i] = fmaf(s[i], mul, alibi2 * (float)(t0 + i - pos));
+        mul = 1.f;
+      }
+      if (bias != nullptr) {
+        // entry y of the table belongs to distance bias_len + 126 - y; everything from bias_len - 1 on is the far entry
+        if (__any_sync(0xffffffffu, pos - (t0 + BN - 1) < p.bias_len - 1)) {
+          const int y0 = min(max(p.bias_len + 126 - (pos - t0), 0), p.bias_len + 254 - BN);
+          const float* row = bias + (int64_t)y0 * p.gp;
 #pragma unroll
           for (int i = 0; i < BN; ++i) {
-            const int dist = max(0, pos - (t0 + i));
-            if (dist < p.bias_len - 1) s[i] = fmaf(__ldg(bias + dist), 1.4426950408889634f, s[i] - bias_far);
+            s[i] = fmaf(s[i], mul, __ldg(row));
+            row += p.gp;
           }
+          mul = 1.f;
+        } else {
+          off = bias_far;
         }
       }
       if ((t0 + BN > lim) || (t0 < lo)) {
@@ -334,7 +345,7 @@ attn_prefill_pp_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       float mx = s[0];
 #pragma unroll
       for (int i = 1; i < BN; ++i) mx = fmaxf(mx, s[i]);
-      mx *= mul;                                     // scale > 0: the maximum commutes with it
+      mx = fmaf(mx, mul, off);                       // scale > 0: the maximum commutes with it
       // lazy maximum: move it only when a row outgrows the exponent range the packed P can carry
       const bool grow = mx > m_run + kPpLazy;        // also true for the first finite maximum
       float corr = 1.f;
@@ -360,7 +371,7 @@ attn_prefill_pp_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
           tmem_st_32x32b_x32(tmem_Ot + c, v);
         }
       }
-      const float m_off = (m_run == -INFINITY) ? 0.f : m_run;
+      const float m_off = ((m_run == -INFINITY) ? 0.f : m_run) - off;
       float rs = 0.f;
 #pragma unroll
       for (int c = 0; c < BN; c += 64) {
@@ -387,6 +398,13 @@ attn_prefill_pp_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     if (l_tot > 0.f) o_acc_scale = p.out_scale / l_tot;
     const int64_t out_stride = p.out_stride ? p.out_stride : (int64_t)p.num_q_heads * p.dv;
     const T* gate = p.gate != nullptr ? reinterpret_cast<const T*>(p.gate) + (int64_t)(q_begin + tok) * p.gate_stride + hq * p.dv : nullptr;
+    // the row's gates, all loads in flight while the last product runs
+    uint4 z[DV / 8];
+    if (gate != nullptr) {
+#pragma unroll
+      for (int i = 0; i < DV / 8; ++i)
+        z[i] = row_valid && i * 8 < p.dv ? __ldg(reinterpret_cast<const uint4*>(gate) + i) : make_uint4(0, 0, 0, 0);
+    }
     if (ok && n_mine > 0) {
       if (!mbar_wait(&o_done[t], (n_mine - 1) & 1)) {
         report_status(p.status, kWaitTimeout, 52, n_mine, t);
@@ -396,7 +414,7 @@ attn_prefill_pp_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     }
     if (ok && n_mine > 0) {
       T* dst = reinterpret_cast<T*>(p.out) + (q_begin + tok) * out_stride + hq * p.dv;
-#pragma unroll 1
+#pragma unroll
       for (int c = 0; c < DV; c += 32) {
         uint32_t v[32];
         tmem_ld_32x32b_x32(tmem_Ot + c, v);     // warp-collective: every lane takes part
@@ -407,11 +425,11 @@ attn_prefill_pp_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
             float f[8];
 #pragma unroll
             for (int i = 0; i < 8; ++i) f[i] = __uint_as_float(v[g8 * 8 + i]) * o_acc_scale;
-            if (gate != nullptr && c + g8 * 8 < p.dv) {
-              float z[8];
-              unpack8<T>(*reinterpret_cast<const uint4*>(gate + c + g8 * 8), z);
+            if (gate != nullptr) {
+              float x[8];
+              unpack8<T>(z[(c + g8 * 8) / 8], x);
 #pragma unroll
-              for (int i = 0; i < 8; ++i) f[i] *= __fdividef(1.f, 1.f + __expf(-z[i]));
+              for (int i = 0; i < 8; ++i) f[i] *= __fdividef(1.f, 1.f + __expf(-x[i]));
             }
             if (c + g8 * 8 < p.dv) *reinterpret_cast<uint4*>(dst + c + g8 * 8) = pack8<T>(f);
           }

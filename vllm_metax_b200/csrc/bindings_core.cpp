@@ -229,9 +229,9 @@ void attention_prefill(Tensor& out, const Tensor& q, const Tensor& k_src, const 
                        int64_t window, double softcap, const optional<Tensor>& sinks,
                        const optional<Tensor>& lse_out, int64_t batch, int64_t max_q_len, bool causal,
                        const optional<Tensor>& alibi_slopes, const optional<Tensor>& distance_bias,
-                       const optional<Tensor>& gate, double out_scale) {
+                       const optional<Tensor>& bias_tiles, const optional<Tensor>& gate, double out_scale) {
   TORCH_CHECK(q.dim() == 3 && q.stride(2) == 1 && q.stride(1) == q.size(2));
-  on_device_of(q, {&out, &k_src, &query_start_loc}, {&v_src, &distance_bias, &gate});
+  on_device_of(q, {&out, &k_src, &query_start_loc}, {&v_src, &distance_bias, &bias_tiles, &gate});
   b200::PrefillParams p{};
   attn_extras(p, out, distance_bias, gate, out_scale);
   p.alibi_slopes = ptr<float>(alibi_slopes);
@@ -283,6 +283,12 @@ void attention_prefill(Tensor& out, const Tensor& q, const Tensor& k_src, const 
   p.num_kv_heads = Hkv;
   const int g = Hq / Hkv;
   p.gp = (128 % g == 0) ? g : 1;
+  if (p.bias != nullptr) {
+    TORCH_CHECK(bias_tiles.has_value() && bias_tiles->dim() == 3 && bias_tiles->is_contiguous() &&
+                bias_tiles->scalar_type() == at::kFloat && bias_tiles->size(0) == Hq / p.gp &&
+                bias_tiles->size(1) == p.bias_len + 254 && bias_tiles->size(2) == p.gp, "distance bias in the prompt kernel's layout");
+    p.bias_tiles = ptr<float>(bias_tiles);
+  }
   p.total_q = T;
   p.scale = (float)scale;
   p.softcap = (float)softcap;
@@ -460,7 +466,7 @@ TORCH_LIBRARY(b200, m) {
       "attention_prefill(Tensor(a!) out, Tensor q, Tensor k_src, Tensor? v_src, Tensor? block_table, "
       "Tensor? seq_lens, Tensor query_start_loc, Tensor? kv_start_loc, float scale, int window, float softcap, "
       "Tensor? sinks, Tensor(b!)? lse_out, int batch, int max_q_len, bool causal, Tensor? alibi_slopes=None, "
-      "Tensor? distance_bias=None, Tensor? gate=None, float out_scale=1.0) -> ()",
+      "Tensor? distance_bias=None, Tensor? bias_tiles=None, Tensor? gate=None, float out_scale=1.0) -> ()",
       &attention_prefill);
   m.def("get_status(int device) -> Tensor", &get_status);
 }

@@ -128,14 +128,16 @@ void memory_gates(Tensor& out, Tensor& top, const Tensor& logits, const Tensor& 
 }
 
 // ------------------------------------------------------------------ delta rule with a decay per key channel
-int64_t channel_delta_scratch_floats(const Tensor& like, int64_t batch, int64_t heads, int64_t vdim, int64_t max_query_len) {
-  return b200::channel_delta_scratch((int)batch, (int)like.size(0), (int)heads, (int)vdim, (int)max_query_len, device_sms(like));
+int64_t channel_delta_scratch_floats(const Tensor& like, int64_t batch, int64_t heads, int64_t kv_heads, int64_t dim, int64_t vdim,
+                                     int64_t max_query_len, int64_t shape) {
+  return b200::channel_delta_scratch((int)batch, (int)like.size(0), (int)heads, (int)kv_heads, (int)dim, (int)vdim,
+                                     (int)max_query_len, device_sms(like), (int)shape);
 }
 
 void channel_delta(Tensor& out, Tensor& state, const Tensor& qkv, int64_t q_off, int64_t k_off, int64_t v_off, int64_t kv_heads,
                    const Tensor& g, const Tensor& beta, const Tensor& gate, const Tensor& norm_w, const optional<Tensor>& scratch,
                    const Tensor& qsl, const optional<Tensor>& state_idx, const optional<Tensor>& has_init, double eps,
-                   double out_scale, int64_t max_query_len) {
+                   double out_scale, int64_t max_query_len, int64_t shape) {
   on_device_of(qkv, {&out, &state, &g, &beta, &gate, &norm_w, &qsl}, {&scratch, &state_idx, &has_init});
   TORCH_CHECK(state.dim() == 4 && state.is_contiguous() && state.scalar_type() == at::kFloat);
   const int64_t T = qkv.size(0), H = state.size(1), D = state.size(2), V = state.size(3), G = kv_heads, W = qkv.size(1);
@@ -145,9 +147,10 @@ void channel_delta(Tensor& out, Tensor& state, const Tensor& qkv, int64_t q_off,
   TORCH_CHECK(beta.dim() == 2 && beta.stride(1) == 1 && beta.scalar_type() == at::kFloat && beta.size(0) == T && beta.size(1) >= H);
   const StepRefs s = step_refs(qsl, state_idx, has_init);
   const int sms = device_sms(qkv);
-  const int64_t need = channel_delta_scratch_floats(qkv, s.batch, H, V, max_query_len);
+  const int64_t need = channel_delta_scratch_floats(qkv, s.batch, H, G, D, V, max_query_len, shape);
   if (need > 0)
-    TORCH_CHECK(scratch.has_value() && scratch->scalar_type() == at::kFloat && scratch->numel() >= need, "channel_delta scratch");
+    TORCH_CHECK(scratch.has_value() && scratch->scalar_type() == at::kFloat && scratch->numel() >= need &&
+                reinterpret_cast<uintptr_t>(scratch->data_ptr()) % 16 == 0, "channel_delta scratch");
   b200::ChannelDeltaParams p{};
   p.qkv = qkv.data_ptr(); p.row_stride = qkv.stride(0); p.q_off = q_off; p.k_off = k_off; p.v_off = v_off;
   p.g = g.data_ptr<float>(); p.g_stride = g.stride(0); p.beta = beta.data_ptr<float>(); p.beta_stride = beta.stride(0);
@@ -156,7 +159,7 @@ void channel_delta(Tensor& out, Tensor& state, const Tensor& qkv, int64_t q_off,
   p.qsl = s.qsl; p.state_idx = s.idx; p.has_init = s.init; p.batch = s.batch; p.tokens = T;
   p.heads = H; p.kv_heads = G; p.dim = D; p.vdim = V;
   const c10::cuda::CUDAGuard guard(qkv.device());
-  TORCH_CHECK(b200::channel_delta(p, ptr<float>(scratch), (int)max_query_len, sms, dtype_code(qkv), cur_stream()) == 0,
+  TORCH_CHECK(b200::channel_delta(p, ptr<float>(scratch), (int)max_query_len, sms, (int)shape, dtype_code(qkv), cur_stream()) == 0,
               "channel_delta: key dimension up to 256");
 }
 
@@ -237,11 +240,11 @@ TORCH_LIBRARY_FRAGMENT(b200, m) {
       "memory_gates(Tensor(a!) out, Tensor(b!) top, Tensor logits, Tensor bias, float cap, Tensor query_start_loc, "
       "Tensor? state_idx, Tensor? has_initial, int max_query_len) -> ()",
       &memory_gates);
-  m.def("channel_delta_scratch_floats(Tensor like, int batch, int heads, int vdim, int max_query_len) -> int", &channel_delta_scratch_floats);
+  m.def("channel_delta_scratch_floats(Tensor like, int batch, int heads, int kv_heads, int dim, int vdim, int max_query_len, int shape) -> int", &channel_delta_scratch_floats);
   m.def(
       "channel_delta(Tensor(a!) out, Tensor(b!) state, Tensor qkv, int q_off, int k_off, int v_off, int kv_heads, Tensor g, "
       "Tensor beta, Tensor gate, Tensor norm_w, Tensor(c!)? scratch, Tensor query_start_loc, Tensor? state_idx, "
-      "Tensor? has_initial, float eps, float out_scale, int max_query_len) -> ()",
+      "Tensor? has_initial, float eps, float out_scale, int max_query_len, int shape) -> ()",
       &channel_delta);
   m.def(
       "prenorm(Tensor(a!) h, Tensor(b!)? x_out, Tensor y, Tensor? x, Tensor? add, Tensor? gain, float eps, Tensor? ids, "

@@ -14,16 +14,20 @@
 // (i = 0 ..) of 4 columns in registers, pairs of rows packed for the two-wide fp32 instructions.  Of the 8 partial sums of a
 // group (4 columns, two products) three halving exchanges leave one per lane.  Columns are independent of one another, which is
 // where few long sequences find their parallelism; tokens follow one another.
-// Tokens are staged up to kChunk at a time: the next chunk's raw rows arrive by cp.async while this one is computed; a warp per
-// token forms the unit vectors, their products with the decays and q . k once per chunk.
+// Tokens are staged up to kChunk at a time: the next chunk's raw rows arrive by cp.async while this one is computed, and become
+// unit vectors and their products with the decays once per chunk.  For portions of prompts a small kernel in front forms the
+// lengths and q . k of all tokens, which would otherwise wait for one another's sums here.
+// RL = 8, 16 or 32: the more lanes share a column, the shorter a token takes and the more shared-memory reads it costs - few
+// sequences want short tokens.
 // A decode step is the same kernel with chunks of one token: the state's read and write are the traffic.
 #include "linear_attn.cuh"
 #include "ops.h"
+#include "row_vec.cuh"
 
 namespace b200 {
 namespace {
 
-constexpr int kChunk = 16;
+constexpr int kChunk = 8;
 constexpr int kMaxCols = 128;
 
 // Two stages of raw chunks, then the fp32 rows of a chunk: k, g k, g q, v, o.
@@ -44,8 +48,36 @@ struct DeltaSmem {
   }
 };
 
-template <typename T, int RL, int NR, bool VEC>
-__global__ void __launch_bounds__(RL * kMaxCols / 4, RL == 8 ? 2 : 1)
+__device__ __forceinline__ void cp4(void* smem, const void* gmem) {
+  const uint32_t s = static_cast<uint32_t>(__cvta_generic_to_shared(smem));
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(s), "l"(gmem) : "memory");
+}
+
+// A warp per (token, key head): 1 / |q| (times dim^(-1/2)), 1 / |k| and q . k of the unit vectors.
+template <typename T>
+__global__ void __launch_bounds__(256)
+channel_delta_lengths_kernel(const ChannelDeltaParams p) {
+  const int64_t w = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (w >= (int64_t)p.tokens * p.kv_heads) return;
+  const int lane = threadIdx.x & 31;
+  const T* row = reinterpret_cast<const T*>(p.qkv) + (w / p.kv_heads) * p.row_stride + (w % p.kv_heads) * p.dim;
+  float qq = 0.f, kk = 0.f, qk = 0.f;
+  for (int i = lane; i < p.dim; i += 32) {
+    const float q = to_f(row[p.q_off + i]), k = to_f(row[p.k_off + i]);
+    qq = fmaf(q, q, qq);
+    kk = fmaf(k, k, kk);
+    qk = fmaf(q, k, qk);
+  }
+  qq = warp_sum(qq); kk = warp_sum(kk); qk = warp_sum(qk);
+  if (lane == 0) {
+    const float iq = 1.f / (sqrtf((float)p.dim) * sqrtf(qq + 1e-6f)), ik = 1.f / sqrtf(kk + 1e-6f);
+    p.lengths[w] = make_float4(iq, ik, qk * iq * ik, 0.f);
+  }
+}
+
+// LEN: the lengths are there (portions of prompts).
+template <typename T, int RL, int NR, bool VEC, bool LEN>
+__global__ void __launch_bounds__(256, RL == 32 ? 3 : 2)
 channel_delta_kernel(const ChannelDeltaParams p) {
   constexpr int DP = RL * NR;                                // padded rows
   const int b = blockIdx.x, h = blockIdx.y, hk = h / (p.heads / p.kv_heads), col0 = blockIdx.z * p.col_block;
@@ -54,6 +86,8 @@ channel_delta_kernel(const ChannelDeltaParams p) {
   if (t1 <= t0) return;
   extern __shared__ __align__(16) uint8_t sm[];
   __shared__ float s_beta[kChunk], s_qk[kChunk];
+  __shared__ float4 s_len[2][kChunk];
+  __shared__ float s_logit[2][kChunk];
   const DeltaSmem<T, DP> L(p.col_block, chunk);
   float *s_k = reinterpret_cast<float*>(sm + L.fk), *s_gk = reinterpret_cast<float*>(sm + L.fgk),
         *s_gq = reinterpret_cast<float*>(sm + L.fgq), *s_v = reinterpret_cast<float*>(sm + L.fv),
@@ -74,7 +108,13 @@ channel_delta_kernel(const ChannelDeltaParams p) {
     copy_rows<T, VEC>(reinterpret_cast<T*>(s + L.q), DP, row + p.q_off + hk * p.dim, p.row_stride, n, p.dim);
     copy_rows<T, VEC>(reinterpret_cast<T*>(s + L.k), DP, row + p.k_off + hk * p.dim, p.row_stride, n, p.dim);
     copy_rows<T, VEC>(reinterpret_cast<T*>(s + L.v), p.col_block, row + p.v_off + h * p.vdim + col0, p.row_stride, n, cols);
-    if constexpr (VEC) asm volatile("cp.async.commit_group;" ::: "memory");
+    if constexpr (LEN) {
+      if (tid < n) {
+        cp16(&s_len[buf][tid], p.lengths + (int64_t)(tc + tid) * p.kv_heads + hk);
+        cp4(&s_logit[buf][tid], p.beta + (int64_t)(tc + tid) * p.beta_stride + h);
+      }
+    }
+    if constexpr (VEC || LEN) asm volatile("cp.async.commit_group;" ::: "memory");
   };
   if (p.dim < DP || cols < p.col_block) {
     for (int i = tid * 4; i < L.fk; i += nthr * 4) *reinterpret_cast<uint32_t*>(sm + i) = 0u;
@@ -108,14 +148,33 @@ channel_delta_kernel(const ChannelDeltaParams p) {
   const float q_scale = 1.f / sqrtf((float)p.dim);
   for (int tc = t0; tc < t1; tc += chunk, buf ^= 1) {
     const int n = min(chunk, t1 - tc);
-    if constexpr (VEC) asm volatile("cp.async.wait_group 0;" ::: "memory");
+    if constexpr (VEC || LEN) asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();                                         // the chunk is here; the previous one has been used up
     if (tc + chunk < t1) stage(tc + chunk, buf ^ 1);
     const uint8_t* raw = sm + buf * L.stage;
     const float* s_g = reinterpret_cast<const float*>(raw);
     const T *rq = reinterpret_cast<const T*>(raw + L.q), *rk = reinterpret_cast<const T*>(raw + L.k),
             *rv = reinterpret_cast<const T*>(raw + L.v);
-    for (int t = warp; t < n; t += nw) {
+    if constexpr (LEN) {
+      for (int i = tid * 4; i < n * DP; i += nthr * 4) {
+        const float4 len = s_len[buf][i / DP];
+        const float4 g = *reinterpret_cast<const float4*>(s_g + i);
+        float qv[4], kv[4];
+        load_row<T, 4, true>(rq, i, 0, qv);
+        load_row<T, 4, true>(rk, i, 0, kv);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) kv[e] *= len.y;
+        *reinterpret_cast<float4*>(s_k + i) = make_float4(kv[0], kv[1], kv[2], kv[3]);
+        *reinterpret_cast<float4*>(s_gk + i) = make_float4(g.x * kv[0], g.y * kv[1], g.z * kv[2], g.w * kv[3]);
+        *reinterpret_cast<float4*>(s_gq + i) = make_float4(g.x * (qv[0] * len.x), g.y * (qv[1] * len.x), g.z * (qv[2] * len.x),
+                                                           g.w * (qv[3] * len.x));
+      }
+      if (tid < n) {
+        s_qk[tid] = s_len[buf][tid].z;
+        s_beta[tid] = sigmoid_precise(s_logit[buf][tid]);
+      }
+    }
+    for (int t = LEN ? n : warp; t < n; t += nw) {
       float qv[DP / 32], kv[DP / 32], qq = 0.f, kk = 0.f, qk = 0.f;
 #pragma unroll
       for (int i = 0; i < DP / 32; ++i) {
@@ -176,7 +235,8 @@ channel_delta_kernel(const ChannelDeltaParams p) {
 #pragma unroll
         for (int c = 0; c < 2; ++c) z[c] = (h2 ? y[2 + c] : y[c]) + __shfl_xor_sync(0xffffffffu, h2 ? y[c] : y[2 + c], 2);
         r = (h1 ? z[1] : z[0]) + __shfl_xor_sync(0xffffffffu, h1 ? z[0] : z[1], 1);
-        if constexpr (RL == 16) r += __shfl_xor_sync(0xffffffffu, r, 8);
+        if constexpr (RL >= 16) r += __shfl_xor_sync(0xffffffffu, r, 8);
+        if constexpr (RL == 32) r += __shfl_xor_sync(0xffffffffu, r, 16);
       }
       const float4 v4 = *reinterpret_cast<const float4*>(s_v + t * p.col_block + c4);
       const float v[4] = {v4.x, v4.y, v4.z, v4.w};
@@ -253,8 +313,15 @@ void launch(const ChannelDeltaParams& p, cudaStream_t stream) {
     cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     kern<<<grid, threads, smem, stream>>>(p);
   };
-  if (p.vec) go(channel_delta_kernel<T, RL, NR, true>);
-  else go(channel_delta_kernel<T, RL, NR, false>);
+  if (p.lengths != nullptr) {
+    const int64_t warps = (int64_t)p.tokens * p.kv_heads;
+    channel_delta_lengths_kernel<T><<<(unsigned)((warps + 7) / 8), 256, 0, stream>>>(p);
+    if (p.vec) go(channel_delta_kernel<T, RL, NR, true, true>);
+    else go(channel_delta_kernel<T, RL, NR, false, true>);
+  } else {
+    if (p.vec) go(channel_delta_kernel<T, RL, NR, true, false>);
+    else go(channel_delta_kernel<T, RL, NR, false, false>);
+  }
 }
 
 template <typename T>
@@ -262,6 +329,8 @@ int dispatch(const ChannelDeltaParams& p, cudaStream_t stream) {
   if (p.dim <= 32) launch<T, 8, 4>(p, stream);
   else if (p.dim <= 64) launch<T, 8, 8>(p, stream);
   else if (p.dim <= 96) launch<T, 8, 12>(p, stream);
+  else if (p.dim <= 128 && p.lanes == 32) launch<T, 32, 4>(p, stream);
+  else if (p.dim <= 128 && p.lanes == 16) launch<T, 16, 8>(p, stream);
   else if (p.dim <= 128) launch<T, 8, 16>(p, stream);
   else if (p.dim <= 192) launch<T, 16, 12>(p, stream);
   else if (p.dim <= 256) launch<T, 16, 16>(p, stream);
@@ -274,26 +343,39 @@ int dispatch(const ChannelDeltaParams& p, cudaStream_t stream) {
 }
 
 // Value columns per CTA: a whole head up to 128 columns; fewer when a long step would leave SMs without CTAs.
-int col_block_for(int batch, int heads, int vdim, int max_query_len, int sms) {
+// Keys of more than 64 channels: 16 or 32 lanes per column (`lanes`) take blocks of at most 64 or 32 columns.
+struct Shape { int col_block, lanes; };
+
+Shape shape_for(int batch, int heads, int dim, int vdim, int max_query_len, int sms) {
   int cb = vdim < kMaxCols ? (vdim + 15) / 16 * 16 : kMaxCols;
-  if (max_query_len < 64) return cb;
+  if (max_query_len < 64) return {dim > 128 && cb > 64 ? 64 : cb, 8};
   const int64_t rows = (int64_t)batch * heads;
-  while (cb > 16 && rows * ((vdim + cb - 1) / cb) < 2 * (int64_t)sms) cb = (cb / 2 + 15) / 16 * 16;
-  return cb;
+  while (cb > 16 && 2 * rows * ((vdim + cb - 1) / cb) < 3 * (int64_t)sms) cb = (cb / 2 + 15) / 16 * 16;
+  if (dim > 128) return {cb > 64 ? 64 : cb, 16};
+  const int64_t warps = rows * ((vdim + cb - 1) / cb) * (cb / 16);     // with 8 lanes
+  const int lanes = warps >= 6 * (int64_t)sms ? 8 : warps >= 3 * (int64_t)sms ? 16 : 32;
+  return {lanes == 32 && cb > 32 ? 32 : lanes == 16 && cb > 64 ? 64 : cb, lanes};
 }
 
 }  // namespace
 
 // Floats of scratch a call needs (0: none): raw outputs of heads that are split over several CTAs.
-int64_t channel_delta_scratch(int batch, int tokens, int heads, int vdim, int max_query_len, int sms) {
-  return col_block_for(batch, heads, vdim, max_query_len, sms) < vdim ? (int64_t)tokens * heads * vdim : 0;
+// ... and, in front of them, the lengths of the tokens of prompts.
+int64_t channel_delta_scratch(int batch, int tokens, int heads, int kv_heads, int dim, int vdim, int max_query_len, int sms,
+                              int shape) {
+  const int cb = shape ? shape % 1000 : shape_for(batch, heads, dim, vdim, max_query_len, sms).col_block;
+  return (max_query_len > 1 ? (int64_t)tokens * kv_heads * 4 : 0) + (cb < vdim ? (int64_t)tokens * heads * vdim : 0);
 }
 
-// Returns 1 when the key dimension is above 256.
-int channel_delta(ChannelDeltaParams p, float* scratch, int max_query_len, int sms, int dtype, cudaStream_t stream) {
+// `shape` (0: chosen here) pins lanes * 1000 + columns per CTA.  Returns 1 when the key dimension is above 256.
+int channel_delta(ChannelDeltaParams p, float* scratch, int max_query_len, int sms, int shape, int dtype, cudaStream_t stream) {
   if (p.tokens <= 0 || p.batch <= 0) return 0;
-  p.col_block = col_block_for(p.batch, p.heads, p.vdim, max_query_len, sms);
-  p.o_raw = p.col_block < p.vdim ? scratch : nullptr;
+  const Shape s = shape ? Shape{shape % 1000, shape / 1000} : shape_for(p.batch, p.heads, p.dim, p.vdim, max_query_len, sms);
+  if (s.col_block < 16 || s.col_block % 16 != 0 || s.col_block > (s.lanes == 8 && p.dim <= 128 ? kMaxCols : s.lanes == 32 ? 32 : 64)) return 1;
+  p.col_block = s.col_block;
+  p.lanes = s.lanes;
+  p.lengths = max_query_len > 1 ? reinterpret_cast<float4*>(scratch) : nullptr;
+  p.o_raw = p.col_block < p.vdim ? scratch + (max_query_len > 1 ? (int64_t)p.tokens * p.kv_heads * 4 : 0) : nullptr;
   p.chunk = max_query_len < kChunk ? max_query_len : kChunk;
   p.vec = p.dim % 8 == 0 && p.vdim % 8 == 0 && p.row_stride % 8 == 0 && p.q_off % 8 == 0 && p.k_off % 8 == 0 &&
           p.v_off % 8 == 0 && p.g_stride % 4 == 0 && reinterpret_cast<uintptr_t>(p.qkv) % 16 == 0 &&

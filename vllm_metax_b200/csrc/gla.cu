@@ -404,9 +404,10 @@ bool use_segments(int batch, int heads, int max_query_len, int sms) {
 
 // Value columns per CTA: a whole head up to 128 columns; fewer when a long step would leave SMs without a CTA.
 // (a multiple of 16 columns keeps whole warps)
-int col_block_for(int batch, int heads, int vdim, int max_query_len, int sms) {
+// With a second kernel for the outputs anyway (`raw`), single tokens take small blocks: their time is the state's traffic.
+int col_block_for(int batch, int heads, int vdim, int max_query_len, int sms, bool raw) {
   int cb = vdim < kMaxCols ? (vdim + 15) / 16 * 16 : kMaxCols;
-  if (max_query_len < 64) return cb;
+  if (max_query_len < 64) return raw && cb > 32 ? 32 : cb;
   const int64_t rows = (int64_t)batch * heads * (use_segments(batch, heads, max_query_len, sms) ? (max_query_len + kSeg - 1) / kSeg : 1);
   while (cb > 32 && rows * ((vdim + cb - 1) / cb) * 2 <= sms) cb = (cb / 2 + 15) / 16 * 16;
   return cb;
@@ -478,7 +479,7 @@ void memory_gates(const MemoryGatesParams& p, int max_query_len, cudaStream_t st
 // Floats of scratch a call needs: raw outputs of split heads, then segment states and decays (0: none of that kind).
 GlaScratch gla_scratch(int batch, int tokens, int heads, int dim, int vdim, int max_query_len, int sms, bool whole_row) {
   GlaScratch g{0, 0};
-  if (whole_row || col_block_for(batch, heads, vdim, max_query_len, sms) < vdim) g.raw = (int64_t)tokens * heads * vdim;
+  if (whole_row || col_block_for(batch, heads, vdim, max_query_len, sms, whole_row) < vdim) g.raw = (int64_t)tokens * heads * vdim;
   if (use_segments(batch, heads, max_query_len, sms)) g.segments = (int64_t)(tokens / kSeg + batch) * heads * dim * (vdim + 2);
   return g;
 }
@@ -486,7 +487,7 @@ GlaScratch gla_scratch(int batch, int tokens, int heads, int dim, int vdim, int 
 // Returns 1 when the key dimension is above 256.
 int gla_recurrent(GlaParams p, float* scratch, int max_query_len, int sms, int dtype, cudaStream_t stream) {
   if (p.tokens <= 0 || p.batch <= 0) return 0;
-  p.col_block = col_block_for(p.batch, p.heads, p.vdim, max_query_len, sms);
+  p.col_block = col_block_for(p.batch, p.heads, p.vdim, max_query_len, sms, p.whole_row);
   const GlaScratch g = gla_scratch(p.batch, p.tokens, p.heads, p.dim, p.vdim, max_query_len, sms, p.whole_row);
   p.chunk = max_query_len < kChunk ? max_query_len : kChunk;
   p.o_raw = g.raw ? scratch : nullptr;

@@ -46,6 +46,8 @@ struct DecodeParams {
   // what happens to scores and results beyond that (all optional)
   const float* bias = nullptr;   // [Hq, bias_len]: added to the scaled (and capped) score of a key by its distance
   int bias_len = 0;              //   ... from bias_len - 1 on: the last entry
+  const float* bias_tiles = nullptr;   // prompt kernel: [Hq / gp, bias_len + 254, gp], the same times log2(e): entry y of a head
+                                       //   is that of distance clamp(bias_len + 126 - y, 0, bias_len - 1)
   const void* gate = nullptr;    // [T, Hq * dv] (token stride gate_stride): the result is multiplied by its sigmoid
   int64_t gate_stride = 0;
   float out_scale = 1.f;
@@ -74,6 +76,8 @@ struct PrefillParams {
   // what happens to scores and results beyond that (all optional)
   const float* bias = nullptr;   // [Hq, bias_len]: added to the scaled (and capped) score of a key by its distance
   int bias_len = 0;              //   ... from bias_len - 1 on: the last entry
+  const float* bias_tiles = nullptr;   // prompt kernel: [Hq / gp, bias_len + 254, gp], the same times log2(e): entry y of a head
+                                       //   is that of distance clamp(bias_len + 126 - y, 0, bias_len - 1)
   const void* gate = nullptr;    // [T, Hq * dv] (token stride gate_stride): the result is multiplied by its sigmoid
   int64_t gate_stride = 0;
   float out_scale = 1.f;
@@ -441,12 +445,14 @@ struct ChannelDeltaParams {
   const float* beta; int64_t beta_stride;      // [tokens, heads] logits of the step sizes
   GatedNormOut out;
   float* state;                                // [slots, heads, dim, vdim]
-  float* o_raw;                                // [tokens, heads * vdim] scratch where heads are split over CTAs
+  float4* lengths;                             // set from the scratch: [tokens, kv_heads] 1 / |q|, 1 / |k|, q . k, or null
+  float* o_raw;                                // set from the scratch: [tokens, heads * vdim] where heads are split over CTAs
   const int* qsl; const int* state_idx; const int* has_init;
-  int batch, tokens, heads, kv_heads, dim, vdim, col_block, vec, chunk;
+  int batch, tokens, heads, kv_heads, dim, vdim, col_block, lanes, vec, chunk;
 };
-int64_t channel_delta_scratch(int batch, int tokens, int heads, int vdim, int max_query_len, int sms);
-int channel_delta(ChannelDeltaParams p, float* scratch, int max_query_len, int sms, int dtype, cudaStream_t stream);
+int64_t channel_delta_scratch(int batch, int tokens, int heads, int kv_heads, int dim, int vdim, int max_query_len, int sms,
+                              int shape);
+int channel_delta(ChannelDeltaParams p, float* scratch, int max_query_len, int sms, int shape, int dtype, cudaStream_t stream);
 // ---- rglru.cu (real-gated linear recurrent unit)
 struct RgLruParams {
   const void* u; int64_t u_stride;       // [tokens, width] recurrence input

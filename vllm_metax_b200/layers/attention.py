@@ -93,6 +93,7 @@ class Attention(nn.Module):
         self.sinks = sinks
         self.k_scale, self.v_scale = k_scale, v_scale
         self.distance_bias: Optional[torch.Tensor] = None      # f32 [num_heads, L]: bias by distance, the last entry from L - 1 on
+        self.bias_tiles: Optional[torch.Tensor] = None         # the same for the prompt kernel (ops.distance_bias_tiles)
         self.out_scale = 1.0
 
     def forward(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, positions: Optional[torch.Tensor] = None,
@@ -152,7 +153,8 @@ class Attention(nn.Module):
                                         max_q_len=md.max_prefill_query_len, window=self.window, softcap=self.softcap,
                                         sinks=self.sinks, k_scale=self.k_scale, v_scale=self.v_scale,
                                         max_seq_len=md.max_seq_len, alibi_slopes=self.alibi_slopes,
-                                        distance_bias=self.distance_bias, gate=gates[1], out_scale=self.out_scale)
+                                        distance_bias=self.distance_bias, bias_tiles=self.bias_tiles, gate=gates[1],
+                                        out_scale=self.out_scale)
         return out
 
     def _forward_cascade(self, q3, md, kv_cache, kv_scales) -> torch.Tensor:
@@ -347,6 +349,8 @@ class QKNormAttention(nn.Module):
             self.register_buffer("distance_bias", torch.zeros(heads, len(index), dtype=torch.float32), persistent=False)
             self.buckets = index
             self.attn.distance_bias = self.distance_bias
+            self.register_buffer("bias_tiles", ops.distance_bias_tiles(self.distance_bias, heads // kv_heads), persistent=False)
+            self.attn.bias_tiles = self.bias_tiles
         if standalone:
             self.proj = StackedLinear(width, self.in_parts(), ("q", "k", "v") if proj_bias else (), dtype=dtype)
             self.attach(self.proj)
@@ -370,6 +374,7 @@ class QKNormAttention(nn.Module):
     def finalize_weights(self) -> None:
         if self.rel is not None:
             self.distance_bias.copy_(self.rel.data.float()[self.buckets].t())
+            self.bias_tiles.copy_(ops.distance_bias_tiles(self.distance_bias, self.heads // self.kv_heads))
 
     def in_slots(self, proj: StackedLinear) -> dict:
         """Tensor name -> (memory it is copied to, its shape in a checkpoint), without the output product."""

@@ -43,9 +43,9 @@ def channel_delta_rule_ref(qkv, offsets, kv_heads, g, beta, gate, norm_w, state,
 
 def channel_delta_rule(qkv: torch.Tensor, offsets: Sequence[int], kv_heads: int, g: torch.Tensor, beta: torch.Tensor,
                        gate: torch.Tensor, norm_w: torch.Tensor, state: torch.Tensor, steps: Steps, eps: float,
-                       out_scale: float = 1.0, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+                       out_scale: float = 1.0, out: Optional[torch.Tensor] = None, shape: int = 0) -> torch.Tensor:
     """``offsets`` = columns of (q, k, v).  Returns ``[T, H * vdim]`` (``out``: rows may be part of wider ones); ``state`` is
-    updated in place."""
+    updated in place.  ``shape``: pins the kernel's lanes per column * 1000 + columns per CTA (0: chosen from the sizes)."""
     from .. import _custom_ops as ops
 
     if not ops._use_cuda(qkv):
@@ -55,9 +55,9 @@ def channel_delta_rule(qkv: torch.Tensor, offsets: Sequence[int], kv_heads: int,
     T, B = qkv.shape[0], steps.query_start_loc.numel() - 1
     if out is None:
         out = torch.empty(T, H * V, dtype=qkv.dtype, device=qkv.device)
-    need = torch.ops.b200.channel_delta_scratch_floats(qkv, B, H, V, steps.max_query_len)
+    need = torch.ops.b200.channel_delta_scratch_floats(qkv, B, H, kv_heads, D, V, steps.max_query_len, shape)
     scratch = torch.empty(need, dtype=torch.float32, device=qkv.device) if need else None
     ops._launches += need > 0
     torch.ops.b200.channel_delta(out, state, qkv, *offsets, kv_heads, g, beta, gate, norm_w, scratch, *steps[:3], eps, out_scale,
-                                 steps.max_query_len)
+                                 steps.max_query_len, shape)
     return out

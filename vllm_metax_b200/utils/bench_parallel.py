@@ -131,6 +131,7 @@ def kernel_rows(size: str = "w2048", only: str = "") -> list:
         q3 = rn(T, H, D)
         lens = torch.full((B,), ctx, dtype=torch.int32, device=dev)
         bias = rn(32, H, dt=f32)[distance_buckets(32, 512)].t().contiguous()
+        tiles = {} if decode else {"bias_tiles": ops.distance_bias_tiles(bias, H // G)}
         sink = rn(H, dt=f32)
         wide = rn(T, 2 * n)
         ot = wide[:, :n].unflatten(1, (H, D))
@@ -142,7 +143,7 @@ def kernel_rows(size: str = "w2048", only: str = "") -> list:
             cost = lambda w: 4.0 * T * n + 4.0 * T * G * D
             flp = lambda w: 4.0 * H * B * sum(min(i + 1, w) for i in range(per)) * D
         plain = lambda w: (f"plain, window {w}" if w < ctx else "plain", att(window=w if w < ctx else -1), cost(min(w, ctx)), flp(w))
-        row(f"attention with a distance bias, {phase}", att(distance_bias=bias, out=ot, out_scale=0.8), cost(ctx), flp(ctx), plain(ctx))
+        row(f"attention with a distance bias, {phase}", att(distance_bias=bias, out=ot, out_scale=0.8, **tiles), cost(ctx), flp(ctx), plain(ctx))
         row(f"capped window attention, sink and gate, {phase}",
             att(window=win, softcap=50.0, sinks=sink, gate=gate, out=ot, out_scale=0.8), cost(min(win, ctx)) + 2.0 * T * n, flp(win), plain(win))
         # -- the rest does not care how the tokens are cut
