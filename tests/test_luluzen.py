@@ -28,7 +28,7 @@ def lightning(heads, dim, vdim, decay, mlp=None):
     return {"type": "lightning", "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "decay": decay}, "mlp": mlp}
 
 
-def delta(left, right, scales=(0.7, 1.2), mlp=None, scale=None, temp=(0.3, 20), far=40):
+def delta(left, right, scales=(0.7, 1.2), mlp=None, scale=None, temp=(0.35, 20), far=40):
     H, G, D, V = left
     h, g, d, v, conv = right
     return {"type": "parallel", "mlp": mlp, "mixer": {
