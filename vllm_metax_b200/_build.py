@@ -33,16 +33,19 @@ CUMEM_LIB = ROOT / "cumem_allocator.so"
 
 # the units behind bindings_core.cpp, what each set adds behind bindings_<set>.cpp, and the sets of each group
 CORE_UNITS = ("attn_prefill_pingpong", "attn_prefill_tcgen05", "gemm_grouped_tcgen05", "gemm_pair_tcgen05", "gemm_simt",
-              "gemm_splitk_tcgen05", "gemm_streamk_tcgen05", "gemm_tcgen05", "moe", "residual_norm", "sampling")
+              "gemm_splitk_tcgen05", "gemm_streamk_tcgen05", "gemm_tcgen05", "moe", "residual_norm", "rope_angles", "sampling")
 UNIT_SETS = {
     "gqa": ("attn_decode", "head_norm_rope", "paged_attn_simt"),
-    "hybrid": ("fused_misc", "latent_attn", "mla_decode", "mla_decode_tcgen05", "residual_conv", "rglru"),
+    "hybrid": ("residual_conv", "rglru"),
+    "latent": ("fused_misc", "latent_attn", "mla_decode", "mla_decode_tcgen05"),
     "recurrent": ("causal_conv1d", "channel_delta", "gla", "prenorm"),
+    "streams": ("stream_norm",),
 }
-UNIT_GROUPS = {"gqa": ("gqa",), "hybrid": ("hybrid", "recurrent"), "parallel": ("gqa", "recurrent")}
+UNIT_GROUPS = {"gqa": ("gqa",), "hybrid": ("latent", "hybrid", "recurrent"), "parallel": ("gqa", "recurrent"),
+               "streams": ("gqa", "latent", "streams")}
 # units that compute in true 32-bit (recurrences, norms, angles, fp32 products): no fast-math substitutions
 PRECISE_UNITS = ("channel_delta", "gemm_simt", "gla", "head_norm_rope", "latent_attn", "paged_attn_simt", "prenorm",
-                 "residual_conv", "residual_norm", "rglru")
+                 "residual_conv", "residual_norm", "rglru", "rope_angles", "stream_norm")
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-std=c++17", "-O3", "-lineinfo",

@@ -402,6 +402,7 @@ def silu_and_mul_per_block_quant(x, group_size=128, ue8m0=False, act: str = "sil
 
 # --------------------------------------------------------------------------- attention
 _decode_ws: dict = {}
+_outgrown_ws: list = []
 
 
 def kv_views(kv_cache):
@@ -413,7 +414,9 @@ def kv_views(kv_cache):
 def _decode_workspace(device, numel: int) -> torch.Tensor:
     ws = _decode_ws.get(device)
     if ws is None or ws.numel() < numel:
-        ws = torch.empty(max(numel, 1 << 20), dtype=torch.float32, device=device)
+        if ws is not None:
+            _outgrown_ws.append(ws)            # captured graphs may still write there
+        ws = torch.empty(max(numel, 1 << 20, 0 if ws is None else 2 * ws.numel()), dtype=torch.float32, device=device)
         _decode_ws[device] = ws
     return ws
 
@@ -435,10 +438,11 @@ _batch_invariant: Optional[bool] = None
 
 
 def decode_num_splits(batch: int, num_kv_heads: int, max_seq_len: int, row_tiles: int = 1, sms: int = 148,
-                      window: int = -1) -> int:
-    """Enough KV splits to give every SM a CTA, never finer than 256 tokens per split (of those a window leaves)."""
-    if window > 0:
-        max_seq_len = min(max_seq_len, window)
+                      window: int = -1, chunk: int = 0) -> int:
+    """Enough KV splits to give every SM a CTA, never finer than 256 tokens per split (of those a window or chunk leaves)."""
+    for reach in (window, chunk):
+        if reach > 0:
+            max_seq_len = min(max_seq_len, reach)
     if batch_invariant():
         return 1                               # the split count follows the batch size: one pass per sequence instead
     ctas = max(1, batch * num_kv_heads * row_tiles)
@@ -452,12 +456,14 @@ def paged_attention_decode(q, kv_cache, block_table, seq_lens, scale, *, out=Non
                            query_start_loc=None, max_q_len: int = 1, window: int = -1, softcap: float = 0.0,
                            sinks=None, lse_out=None, num_splits: int = 0, max_seq_len: int = 0, k_scale=1.0,
                            v_scale=1.0, causal=True, workspace=None, alibi_slopes=None, distance_bias=None, gate=None,
-                           out_scale: float = 1.0):
+                           out_scale: float = 1.0, chunk: int = 0, sigmoid_shift=None):
     """Decode attention over the paged cache; ``q [T, Hq, D]``.  ``alibi_slopes [Hq]`` (f32) adds
     ``slope * (kv position - query position)`` to the scores, ``distance_bias [Hq, L]`` (f32) the entry of the distance (the
-    last one from L - 1 on).  The result is multiplied by ``out_scale`` and, with ``gate [T, Hq * Dv]`` (rows may be part of
-    wider ones), by its sigmoid; ``out``'s token rows may be part of wider ones too.  ``kv_cache``: the 5-D cache or a pair of
-    ``kv_views``.  fp32 caches and 16-bit heads wider than 256 run on the CUDA cores."""
+    last one from L - 1 on).  ``chunk`` > 0: a position sees its own chunk of that many, counted from 0.  ``sigmoid_shift [Hq]``
+    (f32): no softmax, a key's weight is ``sigmoid(score + shift)``.  The result is multiplied by ``out_scale`` and, with ``gate
+    [T, Hq * Dv]`` or ``[T, Hq]`` (rows may be part of wider ones), by its sigmoid; ``out``'s token rows may be part of wider
+    ones too.  ``kv_cache``: the 5-D cache or a pair of ``kv_views``.  fp32 caches and 16-bit heads wider than 256 run on the
+    CUDA cores."""
     if _use_cuda(q):
         k, v = kv_views(kv_cache)
         out = torch.empty(q.shape[0], q.shape[1], v.shape[-1], dtype=q.dtype, device=q.device) if out is None else out
@@ -465,7 +471,8 @@ def paged_attention_decode(q, kv_cache, block_table, seq_lens, scale, *, out=Non
         Hkv = k.shape[2]
         if num_splits <= 0:
             g = q.shape[1] // Hkv
-            num_splits = decode_num_splits(B, Hkv, max_seq_len or 4096, (max_q_len * g + 15) // 16, window=window)
+            num_splits = decode_num_splits(B, Hkv, max_seq_len or 4096, (max_q_len * g + 15) // 16, window=window,
+                                           chunk=chunk)
         if q.dtype == torch.float32 or max(k.shape[-1], v.shape[-1]) > 256:
             num_splits = 1
         ws = workspace
@@ -473,14 +480,15 @@ def paged_attention_decode(q, kv_cache, block_table, seq_lens, scale, *, out=Non
             ws = _decode_workspace(q.device, num_splits * q.shape[0] * q.shape[1] * (v.shape[-1] + 1))
         torch.ops.b200.paged_attention_decode(out, q, k, v, kv_scales, block_table, seq_lens, query_start_loc,
                                               scale, window, softcap, sinks, lse_out, ws, num_splits, B, max_q_len,
-                                              k_scale, v_scale, causal, alibi_slopes, distance_bias, gate, out_scale)
+                                              k_scale, v_scale, causal, alibi_slopes, distance_bias, gate, out_scale,
+                                              chunk, sigmoid_shift)
         return out
     B = seq_lens.shape[0]
     qsl = query_start_loc if query_start_loc is not None else torch.arange(B + 1, dtype=torch.int32, device=q.device)
     res = ref.paged_attention(q, kv_cache, block_table, seq_lens, qsl, scale, kv_scales=kv_scales, window=window,
                               softcap=softcap, sinks=sinks, k_scale=k_scale, v_scale=v_scale, causal=causal,
                               return_lse=lse_out is not None, alibi_slopes=alibi_slopes, distance_bias=distance_bias,
-                              gate=gate, out_scale=out_scale)
+                              gate=gate, out_scale=out_scale, chunk=chunk, sigmoid_shift=sigmoid_shift)
     if lse_out is not None:
         res, lse = res
         lse_out.copy_(lse)
@@ -502,9 +510,10 @@ def distance_bias_tiles(bias, group: int):
 def paged_attention_prefill(q, kv_cache, block_table, seq_lens, query_start_loc, scale, *, out=None, kv_scales=None,
                             max_q_len: int = 0, window: int = -1, softcap: float = 0.0, sinks=None, lse_out=None,
                             k_scale=1.0, v_scale=1.0, causal=True, max_seq_len: int = 0, alibi_slopes=None,
-                            distance_bias=None, bias_tiles=None, gate=None, out_scale: float = 1.0):
+                            distance_bias=None, bias_tiles=None, gate=None, out_scale: float = 1.0, chunk: int = 0,
+                            sigmoid_shift=None):
     """Varlen prefill / chunked-prefill attention reading K, V from the paged cache (``distance_bias``, ``gate``,
-    ``out_scale`` as for decode; ``bias_tiles``: what ``distance_bias_tiles`` makes of the bias, where it is at hand)."""
+    ``out_scale``, ``chunk``, ``sigmoid_shift`` as for decode; ``bias_tiles``: what ``distance_bias_tiles`` makes of the bias, where it is at hand)."""
     if _use_cuda(q):
         k, v = kv_views(kv_cache)
         out = torch.empty(q.shape[0], q.shape[1], v.shape[-1], dtype=q.dtype, device=q.device) if out is None else out
@@ -514,19 +523,20 @@ def paged_attention_prefill(q, kv_cache, block_table, seq_lens, query_start_loc,
                 bias_tiles = distance_bias_tiles(distance_bias, q.shape[1] // k.shape[2])
             torch.ops.b200.attention_prefill(out, q, k, v, block_table, seq_lens, query_start_loc, None,
                                              scale, window, softcap, sinks, lse_out, B, max_q_len or q.shape[0], causal,
-                                             alibi_slopes, distance_bias, bias_tiles, gate, out_scale)
+                                             alibi_slopes, distance_bias, bias_tiles, gate, out_scale, chunk, sigmoid_shift)
         else:
             # quantised caches / other head sizes: the split-KV kernel handles any query length in 16-row tiles
             paged_attention_decode(q, kv_cache, block_table, seq_lens, scale, out=out, kv_scales=kv_scales,
                                    query_start_loc=query_start_loc, max_q_len=max_q_len or q.shape[0], window=window,
                                    softcap=softcap, sinks=sinks, lse_out=lse_out, num_splits=1, k_scale=k_scale,
                                    v_scale=v_scale, causal=causal, alibi_slopes=alibi_slopes, distance_bias=distance_bias,
-                                   gate=gate, out_scale=out_scale)
+                                   gate=gate, out_scale=out_scale, chunk=chunk, sigmoid_shift=sigmoid_shift)
         return out
     res = ref.paged_attention(q, kv_cache, block_table, seq_lens, query_start_loc, scale, kv_scales=kv_scales,
                               window=window, softcap=softcap, sinks=sinks, k_scale=k_scale, v_scale=v_scale,
                               causal=causal, return_lse=lse_out is not None, alibi_slopes=alibi_slopes,
-                              distance_bias=distance_bias, gate=gate, out_scale=out_scale)
+                              distance_bias=distance_bias, gate=gate, out_scale=out_scale, chunk=chunk,
+                              sigmoid_shift=sigmoid_shift)
     if lse_out is not None:
         res, lse = res
         lse_out.copy_(lse)
@@ -972,14 +982,26 @@ def wna16_gemm(x, qweight, scales, zeros, bits: int, group: int, *, bias=None, b
 
 
 # --------------------------------------------------------------------------- MLA
+def mla_decode_num_splits(tokens: int, heads: int, kv: int, window: int = 0, fp8: bool = False, tcgen05: bool = False) -> int:
+    # heads per CTA as chosen by the kernel launcher (csrc/mla_decode.cu:mla_decode_heads_per_cta)
+    hpc = 16 if heads <= 16 else (32 if (heads <= 32 or fp8) else 64)
+    ctas = tokens * ((heads + hpc - 1) // hpc)
+    if tcgen05:
+        ctas = 2 * tokens * ((heads + 127) // 128)           # 128 heads x half the latent per CTA
+    if window > 0:
+        kv = min(kv, window)
+    return 1 if ctas >= 148 else max(1, min((296 + ctas - 1) // ctas, kv // 256, 16))
+
+
 def mla_decode(q, mla_cache, block_table, seq_lens, scale, *, query_start_loc=None, topk_indices=None, out=None,
                lse_out=None, num_splits: int = 0, max_seq_len: int = 0, impl: int = 0, window: int = 0,
-               kv_rank: int = 512):
+               kv_rank: int = 512, workspace=None):
     """Absorbed MLA over the latent cache (dense, or sparse with ``topk_indices [T, topk]``).
     ``q [T, H, 576]`` -> ``[T, H, 512]``.  ``impl``: 0 = choose, 1 = mma.sync kernel, 2 = tcgen05 kernel (dense 16-bit
     caches; csrc/mla_decode_tcgen05.cu) or fail.  "Choose" takes the tcgen05 kernel for 64 heads per rank or more only
     with ``B200_MLA_TCGEN05=1``.  Other sizes: cache rows ``[kv_rank latent | rotated part | padding]``, queries of the same
-    row length, output ``[T, H, kv_rank]``.  ``window`` > 0: only the last ``window`` visible positions."""
+    row length, output ``[T, H, kv_rank]``.  ``window`` > 0: only the last ``window`` visible positions.  ``workspace``: for
+    the partial results of splits, where the caller owns it (fp32)."""
     if _use_cuda(q):
         T, H, _ = q.shape
         if q.dtype == torch.float32 or kv_rank > 512:      # CUDA-core kernel: one pass
@@ -990,16 +1012,12 @@ def mla_decode(q, mla_cache, block_table, seq_lens, scale, *, query_start_loc=No
         if num_splits <= 0 and batch_invariant():
             num_splits = 1
         if num_splits <= 0:
-            # heads per CTA as chosen by the kernel launcher (csrc/mla_decode.cu:mla_decode_heads_per_cta)
-            hpc = 16 if H <= 16 else (32 if (H <= 32 or mla_cache.dtype == torch.uint8) else 64)
-            ctas = T * ((H + hpc - 1) // hpc)
-            if impl != 1 and topk_indices is None and mla_cache.dtype != torch.uint8 and (impl == 2 or H >= 64):
-                ctas = 2 * T * ((H + 127) // 128)            # tcgen05 kernel: 128 heads x half the latent per CTA
             kv = topk_indices.shape[1] if topk_indices is not None else (max_seq_len or 4096)
-            if window > 0:
-                kv = min(kv, window)
-            num_splits = 1 if ctas >= 148 else max(1, min((296 + ctas - 1) // ctas, kv // 256, 16))
-        ws = _decode_workspace(q.device, num_splits * T * H * (kv_rank + 1)) if num_splits > 1 else None
+            tcgen05 = impl != 1 and topk_indices is None and mla_cache.dtype != torch.uint8 and (impl == 2 or H >= 64)
+            num_splits = mla_decode_num_splits(T, H, kv, window, mla_cache.dtype == torch.uint8, tcgen05)
+        ws = workspace
+        if num_splits > 1 and (ws is None or ws.numel() < num_splits * T * H * (kv_rank + 1)):
+            ws = _decode_workspace(q.device, num_splits * T * H * (kv_rank + 1))
         torch.ops.b200.mla_decode(out, q, mla_cache, block_table, seq_lens, query_start_loc, topk_indices, scale,
                                   lse_out, ws, num_splits, impl, window)
         return out
@@ -1024,27 +1042,36 @@ def rope_angles(positions, inv_freq, tokens: int):
 
 
 def head_norm_rope(qkv, offsets, q_weight, k_weight, heads: int, dim: int, angles, kv_cache, slot_mapping, eps: float,
-                   one_plus: bool = False, whole_row: bool = False, interleaved: bool = False, q_temp=None):
+                   one_plus: bool = False, whole_row: bool = False, interleaved: bool = False, q_temp=None, q_scale=None,
+                   normed: bool = True, width: int = 0):
     """Epilogue of a merged q | k | v product whose parts start at the columns ``offsets``: per-head RMS norm (``one_plus``:
     weights stored around zero; ``whole_row``: one norm over all heads, with a weight per head and entry) and rotation of
     queries and keys (pairs (i, i + half), ``interleaved``: (2i, 2i + 1)), keys and values written to the paged cache
     (``kv_cache``: 5-D or a pair of ``kv_views``) at ``slot_mapping`` (-1: nowhere).  ``kv_cache=None``: the row holds queries
-    only.  Heads are as wide as their weights (of one head), of which ``dim`` are real; ``angles`` as ``rope_angles`` returns
-    them, or None.  ``q_temp = (positions, coef, every)`` multiplies queries by ``1 + coef * ln((p + 1) // every + 1)``.
-    Returns ``q [T, heads, width]``."""
-    T, width = qkv.shape[0], q_weight.numel() // (heads if whole_row else 1)
+    only.  Heads are as wide as their weights (of one head; without weights ``width``), of which ``dim`` are real; ``angles`` as
+    ``rope_angles`` returns them, or None.  ``q_temp = (positions, coef, every)`` multiplies queries by ``1 + coef * ln((p + 1)
+    // every + 1)``, ``q_scale [heads]`` (fp32) by a number per head.  ``normed=False``: no norm; queries that nothing is done
+    to are returned as they lie in ``qkv``.  Returns ``q [T, heads, width]``."""
+    T, width = qkv.shape[0], width or q_weight.numel() // (heads if whole_row else 1)
     k, v = kv_views(kv_cache) if kv_cache is not None else (None, None)
+    as_is = not normed and angles is None and q_temp is None and q_scale is None
+    q_rows = qkv[:, offsets[0]: offsets[0] + heads * width].unflatten(1, (heads, width))
+    if as_is and k is None:
+        return q_rows
     if _use_cuda(qkv):
-        q = torch.empty(T, heads, width, dtype=qkv.dtype, device=qkv.device)
-        torch.ops.b200.head_norm_rope(q, qkv, *offsets, k, v, q_weight, k_weight, dim, angles, slot_mapping, eps, one_plus,
-                                      whole_row, interleaved, *(q_temp or (None, 0.0, 1)))
-        return q
+        q = None if as_is else torch.empty(T, heads, width, dtype=qkv.dtype, device=qkv.device)
+        torch.ops.b200.head_norm_rope(q, qkv, *offsets, k, v, q_weight, k_weight, dim, angles, slot_mapping, eps, normed,
+                                      one_plus, whole_row, interleaved, *(q_temp or (None, 0.0, 1)), q_scale)
+        return q_rows if as_is else q
 
-    def part(at, n, w, temp=None):
+    def part(at, n, w, temp=None, scale=None):
         x = qkv[:, at: at + n * width]
-        if whole_row:
+        if normed and w is None:
+            x = x.reshape(T, n, width).float()
+            x = x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) / dim + eps)
+        elif normed and whole_row:
             x = ref.head_rms_norm(x[:, None], w, n * dim, eps, one_plus)
-        else:
+        elif normed:
             x = ref.head_rms_norm(x.reshape(T, n, width), w, dim, eps, one_plus)
         x = x.reshape(T, n, width)
         if angles is not None:
@@ -1052,9 +1079,11 @@ def head_norm_rope(qkv, offsets, q_weight, k_weight, heads: int, dim: int, angle
         if temp is not None:
             pos, coef, every = temp
             x = x * (1.0 + coef * torch.log(((pos[:T] + 1) // every).float() + 1.0))[:, None, None]
+        if scale is not None:
+            x = x * scale[:, None]
         return x.to(qkv.dtype)
 
-    q = part(offsets[0], heads, q_weight, q_temp)
+    q = q_rows if as_is else part(offsets[0], heads, q_weight, q_temp, q_scale)
     if k is not None:
         G, bs, dv = k.shape[2], k.shape[1], v.shape[-1]
         ok = slot_mapping[:T] >= 0
@@ -1064,31 +1093,33 @@ def head_norm_rope(qkv, offsets, q_weight, k_weight, heads: int, dim: int, angle
     return q
 
 
-def latent_insert(a, q_off: int, kv_off: int, q_weight, kv_weight, rot_dim: int, inv_freq, positions, cache, slot_mapping,
-                  eps: float):
-    """Epilogue of the merged latent down-projection ``a``: returns the normed query latent ``[T, q_rank]`` and writes
-    ``[normed key latent | rotated key part]`` into the paged cache rows ``slot_mapping`` names (-1: none)."""
-    T, qr, kr = a.shape[0], q_weight.numel(), kv_weight.numel()
+def latent_insert(a, q_off: int, kv_off: int, q_weight, kv_weight, rot_dim: int, angles, cache, slot_mapping, eps: float,
+                  interleaved: bool = False):
+    """Epilogue of the merged latent down-projection ``a``: returns the normed query latent ``[T, q_rank]`` (None without
+    ``q_weight``) and writes ``[normed key latent | rotated key part]`` into the paged cache rows ``slot_mapping`` names (-1:
+    none).  ``angles``: as ``rope_angles`` returns them; pairs (i, i + half), ``interleaved``: (2i, 2i + 1)."""
+    T, kr = a.shape[0], kv_weight.numel()
+    qr = 0 if q_weight is None else q_weight.numel()
     if _use_cuda(a):
-        cq = torch.empty(T, qr, dtype=a.dtype, device=a.device)
-        torch.ops.b200.latent_insert(cq, cache, a, q_off, kv_off, q_weight, kv_weight, rot_dim, inv_freq, positions,
+        cq = torch.empty(T, qr, dtype=a.dtype, device=a.device) if qr else None
+        torch.ops.b200.latent_insert(cq, cache, a, q_off, kv_off, q_weight, kv_weight, rot_dim, angles, interleaved,
                                      slot_mapping, eps)
         return cq
-    cq = ref.rms_norm(a[:, q_off: q_off + qr], q_weight, eps)
+    cq = ref.rms_norm(a[:, q_off: q_off + qr], q_weight, eps) if qr else None
     rows = torch.zeros(T, cache.shape[-1], dtype=a.dtype, device=a.device)
     rows[:, :kr] = ref.rms_norm(a[:, kv_off: kv_off + kr], kv_weight, eps)
-    rows[:, kr: kr + rot_dim] = ref.rotate_half(a[:, kv_off + kr: kv_off + kr + rot_dim][:, None], inv_freq, positions)[:, 0]
+    rows[:, kr: kr + rot_dim] = ref.rotate_half_by(a[:, kv_off + kr: kv_off + kr + rot_dim][:, None], angles, interleaved)[:, 0]
     ok = slot_mapping[:T] >= 0
     cache.view(-1, cache.shape[-1])[slot_mapping[:T][ok]] = rows[ok]
     return cq
 
 
-def latent_rope(dst, src, inv_freq, positions, rot_dim: int, pad: int = 0):
+def latent_rope(dst, src, angles, rot_dim: int, pad: int = 0, interleaved: bool = False):
     """Rotates ``src [T, H, rot_dim]`` into ``dst`` (may be the same memory) and zeroes ``pad`` entries behind."""
     if _use_cuda(src):
-        torch.ops.b200.latent_rope(dst, src, inv_freq, positions, rot_dim, pad)
+        torch.ops.b200.latent_rope(dst, src, angles, interleaved, rot_dim, pad)
         return dst
-    dst[..., :rot_dim] = ref.rotate_half(src[..., :rot_dim], inv_freq, positions)
+    dst[..., :rot_dim] = ref.rotate_half_by(src[..., :rot_dim], angles, interleaved)
     dst[..., rot_dim: rot_dim + pad] = 0
     return dst
 

@@ -144,7 +144,8 @@ __global__ void __launch_bounds__(kDecWarps * 32, (D <= 128 ? 2 : 1)) paged_deco
   // tiles that some row of this CTA can see, and this split's part of them
   const int last_row = min(rows_total, row0 + 16) - 1;
   const int hi_pos = p.causal ? kv_len - q_len + last_row / g + 1 : kv_len;
-  const int lo_pos = p.window > 0 ? max(0, (p.causal ? kv_len - q_len + row0 / g + 1 : kv_len) - p.window) : 0;
+  const int first_lim = p.causal ? kv_len - q_len + row0 / g + 1 : kv_len;
+  const int lo_pos = first_key(first_lim, p.window, p.chunk);
   const int tile_lo = lo_pos / kDecTile;
   const int tiles_total = max(0, (hi_pos + kDecTile - 1) / kDecTile - tile_lo);
   const int tiles_per_split = (tiles_total + p.num_splits - 1) / p.num_splits;
@@ -195,14 +196,18 @@ __global__ void __launch_bounds__(kDecWarps * 32, (D <= 128 ? 2 : 1)) paged_deco
     return p.causal ? (kv_len - q_len + r / g + 1) : kv_len;
   };
   const int limA = row_limit(rA), limB = row_limit(rB);
-  const int loA = (p.window > 0) ? max(0, limA - p.window) : 0;
-  const int loB = (p.window > 0) ? max(0, limB - p.window) : 0;
+  const int loA = first_key(limA, p.window, p.chunk), loB = first_key(limB, p.window, p.chunk);
   // ALiBi: bias = slope[head of the row] * (kv position - query position), in log2 units like the scores
   const float alA = (p.alibi_slopes && rA < rows_total) ? p.alibi_slopes[hk * g + rA % g] * 1.4426950408889634f : 0.f;
   const float alB = (p.alibi_slopes && rB < rows_total) ? p.alibi_slopes[hk * g + rB % g] * 1.4426950408889634f : 0.f;
 
   const float sm_scale_log2 = p.scale * 1.4426950408889634f * ((KIND == 3) ? p.k_scale : 1.f);
-  float m_run[2] = {-INFINITY, -INFINITY};
+  // sigmoid weights need no maximum and no sum: the recurrence below runs at a maximum of zero
+  const bool sigmoid = p.sigmoid_shift != nullptr;
+  const float shA = sigmoid && rA < rows_total ? p.sigmoid_shift[hk * g + rA % g] * 1.4426950408889634f : 0.f;
+  const float shB = sigmoid && rB < rows_total ? p.sigmoid_shift[hk * g + rB % g] * 1.4426950408889634f : 0.f;
+  const float m_start = sigmoid ? 0.f : -INFINITY;
+  float m_run[2] = {m_start, m_start};
   float l_run[2] = {0.f, 0.f};
   float o[D / 8][4];
 #pragma unroll
@@ -346,7 +351,7 @@ __global__ void __launch_bounds__(kDecWarps * 32, (D <= 128 ? 2 : 1)) paged_deco
     float corr[2], msafe[2];
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
-      const float mnew = fmaxf(m_run[h], mx[h]);
+      const float mnew = sigmoid ? 0.f : fmaxf(m_run[h], mx[h]);
       msafe[h] = (mnew == -INFINITY) ? 0.f : mnew;
       corr[h] = exp2f(m_run[h] - msafe[h]);  // m_run = -inf -> 0
       m_run[h] = mnew;
@@ -359,7 +364,7 @@ __global__ void __launch_bounds__(kDecWarps * 32, (D <= 128 ? 2 : 1)) paged_deco
       for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const float pe = exp2f(s[nt][e] - msafe[e >> 1]);
+          const float pe = sigmoid ? __fdividef(1.f, 1.f + exp2f(-s[nt][e] - (e >> 1 ? shB : shA))) : exp2f(s[nt][e] - msafe[e >> 1]);
           rs[e >> 1] += pe;
           pv[nt][e] = pe * vsc[nt * 2 + (e & 1)];
         }
@@ -436,26 +441,30 @@ __global__ void __launch_bounds__(kDecWarps * 32, (D <= 128 ? 2 : 1)) paged_deco
     }
     const int tok = q_begin + rr / g, hq = hk * g + rr % g;
     if (p.num_splits == 1) {
-      float Lt = L;
+      float Lt = sigmoid ? 1.f : L;
       if (p.sinks) Lt += exp2f(p.sinks[hq] * 1.4426950408889634f - Ms);
-      const float v = (Lt > 0.f ? acc / Lt * out_scale : 0.f) * p.out_scale * gate_of<T>(p.gate, tok * p.gate_stride + hq * dv + c);
+      const float v = (Lt > 0.f ? acc / Lt * out_scale : 0.f) * p.out_scale *
+                      gate_of<T>(p.gate, tok * p.gate_stride + (p.gate_per_head ? hq : hq * dv + c));
       reinterpret_cast<T*>(p.out)[tok * out_stride + hq * dv + c] = from_f<T>(v);
       if (c == 0 && p.lse_out)
         p.lse_out[(int64_t)hq * p.total_tokens + tok] = Lt > 0.f ? (Ms * 0.6931471805599453f + logf(Lt)) : -INFINITY;
     } else {
       const int64_t prow = ((int64_t)split * p.total_tokens + tok) * p.num_q_heads + hq;
-      p.part_out[prow * dv + c] = L > 0.f ? acc / L * out_scale : 0.f;
-      if (c == 0) p.part_lse[prow] = L > 0.f ? (Ms * 0.6931471805599453f + logf(L)) : -INFINITY;
+      const float Lp = sigmoid ? 1.f : L;
+      p.part_out[prow * dv + c] = Lp > 0.f ? acc / Lp * out_scale : 0.f;
+      if (c == 0) p.part_lse[prow] = Lp > 0.f ? (Ms * 0.6931471805599453f + logf(Lp)) : -INFINITY;
     }
   }
 }
 
-// out[t,h,:] = sum_s part_out[s,t,h,:] * exp(lse_s - LSE), LSE = logsumexp_s (+ sink)
+// out[t,h,:] = sum_s part_out[s,t,h,:] * exp(lse_s - LSE), LSE = logsumexp_s (+ sink); sigmoid weights: the plain sum (every
+// lse_s is 0)
 template <typename T>
 __global__ void attn_split_reduce_kernel(T* __restrict__ out, float* __restrict__ lse_out,
                                          const float* __restrict__ part_out, const float* __restrict__ part_lse,
                                          const float* __restrict__ sinks, int num_splits, int total_tokens, int heads,
-                                         int D, const void* gate, int64_t gate_stride, float out_scale, int64_t out_stride) {
+                                         int D, const void* gate, int64_t gate_stride, int gate_per_head, bool sum, float out_scale,
+                                         int64_t out_stride) {
   const int64_t row = blockIdx.x;  // token * heads + head
   const int hq = (int)(row % heads);
   const int64_t tok = row / heads;
@@ -466,16 +475,15 @@ __global__ void attn_split_reduce_kernel(T* __restrict__ out, float* __restrict_
   const float Ms = (M == -INFINITY) ? 0.f : M;
   float L = 0.f;
   for (int s = 0; s < num_splits; ++s) L += __expf(part_lse[s * stride + row] - Ms);
-  const float Lk = L;
+  if (sum) L = 1.f;
   if (sinks) L += __expf(sinks[hq] - Ms);
   for (int c = threadIdx.x; c < D; c += blockDim.x) {
     float acc = 0.f;
     for (int s = 0; s < num_splits; ++s)
       acc += part_out[(s * stride + row) * D + c] * __expf(part_lse[s * stride + row] - Ms);
     out[tok * out_stride + hq * D + c] =
-        from_f<T>((L > 0.f ? acc / L : 0.f) * out_scale * gate_of<T>(gate, tok * gate_stride + hq * D + c));
+        from_f<T>((L > 0.f ? acc / L : 0.f) * out_scale * gate_of<T>(gate, tok * gate_stride + (gate_per_head ? hq : hq * D + c)));
   }
-  (void)Lk;
   if (threadIdx.x == 0 && lse_out) lse_out[(int64_t)hq * total_tokens + tok] = L > 0.f ? Ms + logf(L) : -INFINITY;
 }
 
@@ -494,7 +502,7 @@ static void launch_decode(const DecodeParams& p, int batch, int max_q_len, cudaS
     const int dv = KIND == 0 ? p.dv : D;
     attn_split_reduce_kernel<T><<<(unsigned)rows, D <= 128 ? 128 : 256, 0, stream>>>(
         (T*)p.out, p.lse_out, p.part_out, p.part_lse, p.sinks, p.num_splits, p.total_tokens, p.num_q_heads, dv, p.gate,
-        p.gate_stride, p.out_scale, p.out_stride ? p.out_stride : (int64_t)p.num_q_heads * dv);
+        p.gate_stride, p.gate_per_head, p.sigmoid_shift != nullptr, p.out_scale, p.out_stride ? p.out_stride : (int64_t)p.num_q_heads * dv);
   }
 }
 

@@ -22,8 +22,10 @@
 // Query heads must be 16-bit (bf16/fp16); the tiles are (D_qk, D_v) in {(128,128), (64,64), (192,128)}.  Heads may be
 // smaller (multiples of 8): the TMA maps end at the real sizes and the fill pads the tile with zeros.
 // Causal offset: row token i of a sequence with q_len new tokens and kv_len total sits at position
-// kv_len - q_len + i.  Sliding window, soft-cap, ALiBi and attention sinks are supported; LSE can be
+// kv_len - q_len + i.  Sliding window, chunks, soft-cap, ALiBi and attention sinks are supported; LSE can be
 // returned for later merges.  TMA loads touch this GPU's memory only.
+// SIGMOID: a key's weight is the sigmoid of its score.  Without a softmax there is no running maximum and no sum: the weights
+// go straight to the product, whose accumulators are never rescaled.
 //
 // Replaces flash_attn_varlen_func (vllm_metax/v1/attention/backends/flash_attn.py:1302-1322,
 // mla/prefill/flash_attn.py:157-163).
@@ -74,7 +76,7 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return y;
 }
 
-template <typename T, int DQK, int DV, int BN>
+template <typename T, int DQK, int DV, int BN, bool SIGMOID>
 __global__ void __launch_bounds__(384, 1)
 attn_prefill_pp_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                        const __grid_constant__ CUtensorMap tmV, const PrefillParams p) {
@@ -109,8 +111,7 @@ attn_prefill_pp_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   const int h0 = hg * p.gp;                                   // first query head of the tiles
   const int hk = h0 / (p.num_q_heads / p.num_kv_heads);       // kv head
   const int pos0 = kv_len - q_len + tok0;                     // position of tile A's first token
-  int kv_lo = 0;
-  if (p.window > 0) kv_lo = max(0, pos0 + 1 - p.window);
+  const int kv_lo = first_key(pos0 + 1, p.window, p.chunk);
   const int tile_lo = kv_lo / BN;
   // number of K/V tiles each query tile walks (0: the tile holds no token of this sequence)
   auto tiles_of = [&](int t) -> int {
@@ -282,13 +283,14 @@ attn_prefill_pp_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     const bool row_valid = tok < q_len;
     const int pos = kv_len - q_len + tok;           // absolute position of this row
     const int lim = row_valid ? (p.causal ? pos + 1 : kv_len) : 0;  // sees kv < lim
-    const int lo = (p.window > 0) ? max(0, lim - p.window) : 0;
+    const int lo = first_key(lim, p.window, p.chunk);
     const float sl2 = p.scale * 1.4426950408889634f;
     const uint32_t lane_base = ((uint32_t)(quarter * 32)) << 16;
     // bias by distance (log2 units): rows of the table lie as the keys do, the gp heads of a tile side by side
     const float* bias = p.bias_tiles != nullptr ? p.bias_tiles + (int64_t)hg * (p.bias_len + 254) * p.gp + r % p.gp : nullptr;
     const float bias_far = bias != nullptr ? bias[0] : 0.f;
     const float alibi2 = (p.alibi_slopes && row_valid) ? p.alibi_slopes[hq] * 1.4426950408889634f : 0.f;
+    const float shift2 = SIGMOID && row_valid ? p.sigmoid_shift[hq] * 1.4426950408889634f : 0.f;
     const int n_mine = t ? n_b : n_a;
     const uint32_t tmem_St = (t ? tmem_S1 : tmem_S0) + lane_base, tmem_Ot = (t ? tmem_O1 : tmem_O0) + lane_base;
     float m_run = -INFINITY, l_run = 0.f;
@@ -316,8 +318,9 @@ attn_prefill_pp_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         mul = 1.f;
       }
       if (p.alibi_slopes != nullptr) {
+        const float at0 = alibi2 * (float)(t0 - pos);
 #pragma unroll
-        for (int i = 0; i < BN; ++i) s[i] = fmaf(s[i], mul, alibi2 * (float)(t0 + i - pos));
+        for (int i = 0; i < BN; ++i) s[i] = fmaf(s[i], mul, fmaf(alibi2, (float)i, at0));
         mul = 1.f;
       }
       if (bias != nullptr) {
@@ -335,12 +338,26 @@ attn_prefill_pp_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
           off = bias_far;
         }
       }
+      if constexpr (SIGMOID) sigmoid_row(s, mul, off + shift2);
       if ((t0 + BN > lim) || (t0 < lo)) {
 #pragma unroll
         for (int i = 0; i < BN; ++i) {
           const int col = t0 + i;
-          if (col >= lim || col < lo) s[i] = -INFINITY;
+          if (col >= lim || col < lo) s[i] = SIGMOID ? 0.f : -INFINITY;
         }
+      }
+      if constexpr (SIGMOID) {
+#pragma unroll
+        for (int c = 0; c < BN; c += 64) {
+          uint32_t pk[32];
+#pragma unroll
+          for (int i = 0; i < 32; ++i) pk[i] = pack2<T>(s[c + 2 * i], s[c + 2 * i + 1]);
+          tmem_st_32x32b_x32(tmem_St + (c >> 1), pk);
+        }
+        tmem_st_wait();
+        tc_fence_before_sync();
+        mbar_arrive(&p_full[t]);
+        continue;
       }
       float mx = s[0];
 #pragma unroll
@@ -395,9 +412,11 @@ attn_prefill_pp_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     float l_tot = l_run;
     const float m_safe = (m_run == -INFINITY) ? 0.f : m_run;
     if (p.sinks && row_valid) l_tot += exp2f(p.sinks[hq] * 1.4426950408889634f - m_safe);
+    if (SIGMOID) l_tot = 1.f;
     if (l_tot > 0.f) o_acc_scale = p.out_scale / l_tot;
+    if (p.gate_per_head && row_valid) o_acc_scale *= gate_of<T>(p.gate, (int64_t)(q_begin + tok) * p.gate_stride + hq);
     const int64_t out_stride = p.out_stride ? p.out_stride : (int64_t)p.num_q_heads * p.dv;
-    const T* gate = p.gate != nullptr ? reinterpret_cast<const T*>(p.gate) + (int64_t)(q_begin + tok) * p.gate_stride + hq * p.dv : nullptr;
+    const T* gate = p.gate != nullptr && !p.gate_per_head ? reinterpret_cast<const T*>(p.gate) + (int64_t)(q_begin + tok) * p.gate_stride + hq * p.dv : nullptr;
     // the row's gates, all loads in flight while the last product runs
     uint4 z[DV / 8];
     if (gate != nullptr) {
@@ -452,7 +471,7 @@ attn_prefill_pp_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   }
 }
 
-template <typename T, int DQK, int DV, int BN>
+template <typename T, int DQK, int DV, int BN, bool SIGMOID>
 static void launch_prefill_pp(const PrefillParams& p, const void* q, int64_t q_stride, const void* k_src,
                               const void* v_src, int64_t kv_tok_stride_k, int64_t kv_tok_stride_v, int64_t total_kv,
                               int batch, int max_q_len, cudaStream_t stream) {
@@ -487,7 +506,7 @@ static void launch_prefill_pp(const PrefillParams& p, const void* q, int64_t q_s
     uint64_t vs[2] = {(uint64_t)p.v_head_stride * 2, (uint64_t)kv_tok_stride_v * 2};
     tmV = make_tmap_nd(v_src, dt, 3, vd, vs, kb, CU_TENSOR_MAP_SWIZZLE_128B);
   }
-  auto kern = attn_prefill_pp_kernel<T, DQK, DV, BN>;
+  auto kern = attn_prefill_pp_kernel<T, DQK, DV, BN, SIGMOID>;
   // the shared-memory limit is a per-device attribute of the kernel
   static bool set[64] = {};
   int dev = 0;
@@ -510,17 +529,20 @@ int attention_prefill_pp(const PrefillParams& p, const void* q, int64_t q_stride
   if (dqk <= 64 && dv <= 64) dqk = dv = 64;
   else if (dqk <= 128 && dv <= 128) dqk = dv = 128;
   else if (dqk <= 192 && dv <= 128) dqk = 192, dv = 128;
-#define PF(T)                                                                                                        \
-  if (dqk == 128 && dv == 128)                                                                                       \
-    launch_prefill_pp<T, 128, 128, 128>(p, q, q_stride, k_src, v_src, k_tok_stride, v_tok_stride, total_kv, batch, max_q_len, stream); \
-  else if (dqk == 64 && dv == 64)                                                                                    \
-    launch_prefill_pp<T, 64, 64, 128>(p, q, q_stride, k_src, v_src, k_tok_stride, v_tok_stride, total_kv, batch, max_q_len, stream);   \
-  else if (dqk == 192 && dv == 128)                                                                                  \
-    launch_prefill_pp<T, 192, 128, 64>(p, q, q_stride, k_src, v_src, k_tok_stride, v_tok_stride, total_kv, batch, max_q_len, stream); \
-  else                                                                                                               \
-    return -1;
-  if (dtype == 0) { PF(__nv_bfloat16) } else { PF(__half) }
+#define PF1(T, DQK, DV, BN, SIG) \
+  launch_prefill_pp<T, DQK, DV, BN, SIG>(p, q, q_stride, k_src, v_src, k_tok_stride, v_tok_stride, total_kv, batch, max_q_len, stream)
+#define PF(T, SIG)                                                   \
+  if (dqk == 128 && dv == 128) PF1(T, 128, 128, 128, SIG);           \
+  else if (dqk == 64 && dv == 64) PF1(T, 64, 64, 128, SIG);          \
+  else if (dqk == 192 && dv == 128) PF1(T, 192, 128, 64, SIG);       \
+  else return -1;
+  if (p.sigmoid_shift != nullptr) {
+    if (dtype == 0) { PF(__nv_bfloat16, true) } else { PF(__half, true) }
+  } else {
+    if (dtype == 0) { PF(__nv_bfloat16, false) } else { PF(__half, false) }
+  }
 #undef PF
+#undef PF1
   return 0;
 }
 

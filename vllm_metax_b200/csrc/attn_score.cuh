@@ -1,9 +1,17 @@
-// What the attention kernels share beyond the plain softmax: capped scores and gated results.
+// What the attention kernels share beyond the plain softmax: which keys are seen, capped scores, sigmoid weights, gated results.
 #pragma once
 #include "common.cuh"
 #include "f32x2.cuh"
 
 namespace b200 {
+
+// The first key of a query that sees keys below `lim` (its own position is lim - 1 where that matters): the last `window` of
+// them, those of its own chunk of `chunk` positions counted from 0, or both (0: no such limit).
+__host__ __device__ __forceinline__ int first_key(int lim, int window, int chunk) {
+  int lo = window > 0 ? lim - window : 0;
+  if (chunk > 0 && lim > 0) lo = lo > (lim - 1) / chunk * chunk ? lo : (lim - 1) / chunk * chunk;
+  return lo > 0 ? lo : 0;
+}
 
 // cap * tanh(s / cap) with an absolute error of some 1e-7 * cap: (1 + tanh(u)) / 2 = 1 / (1 + exp(-2 u))
 __device__ __forceinline__ float softcap_score(float s, float cap) {
@@ -45,6 +53,25 @@ __device__ __forceinline__ void softcap_row(float (&s)[N], float scale, float ca
   } else {
 #pragma unroll
     for (int i = 0; i < N; ++i) s[i] = softcap_score(s[i] * scale, cap) * kLog2e;
+  }
+}
+
+// s[i] <- sigmoid of s[i] * mul + off, which is in units of log2.  Two neighbours share a reciprocal: 1 / a = b / (a b).  Weights
+// below 2^-60 stay there, so that the product is finite.
+template <int N>
+__device__ __forceinline__ void sigmoid_row(float (&s)[N], float mul, float off) {
+#pragma unroll
+  for (int i = 0; i < N; i += 2) {
+    float e[2];
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      const float z = fminf(-fmaf(s[i + k], mul, off), 60.f);
+      asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e[k]) : "f"(z));
+      e[k] += 1.f;
+    }
+    const float r = __fdividef(1.f, e[0] * e[1]);
+    s[i] = e[1] * r;
+    s[i + 1] = e[0] * r;
   }
 }
 

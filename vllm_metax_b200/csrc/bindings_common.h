@@ -82,10 +82,11 @@ inline int device_sms(const Tensor& t) {
   return sms[d];
 }
 
-// Output rows, distance bias, output gate and factor of an attention call (DecodeParams, PrefillParams).
+// Output rows, distance bias, output gate and factor, chunks and sigmoid weights of an attention call (DecodeParams,
+// PrefillParams).
 template <typename P>
 inline void attn_extras(P& p, const Tensor& out, const optional<Tensor>& distance_bias, const optional<Tensor>& gate,
-                        double out_scale) {
+                        double out_scale, int64_t chunk, const optional<Tensor>& sigmoid_shift, bool causal) {
   const int64_t H = out.size(1), D = out.size(2), unit = 16 / (int64_t)out.element_size();
   auto rows_ok = [&](const Tensor& t) {
     return t.stride(0) % unit == 0 && reinterpret_cast<uintptr_t>(t.data_ptr()) % 16 == 0;
@@ -101,10 +102,19 @@ inline void attn_extras(P& p, const Tensor& out, const optional<Tensor>& distanc
     p.bias_len = (int)distance_bias->size(1);
   }
   if (gate.has_value()) {
-    TORCH_CHECK(gate->dim() == 2 && gate->stride(1) == 1 && gate->size(0) == out.size(0) && gate->size(1) == H * D &&
-                gate->scalar_type() == out.scalar_type() && (D % unit != 0 || rows_ok(*gate)), "attention gate: [tokens, heads * size]");
+    p.gate_per_head = gate->dim() == 2 && gate->size(1) == H && D != 1;
+    TORCH_CHECK(gate->dim() == 2 && gate->stride(1) == 1 && gate->size(0) == out.size(0) && gate->scalar_type() == out.scalar_type() &&
+                (p.gate_per_head || (gate->size(1) == H * D && (D % unit != 0 || rows_ok(*gate)))),
+                "attention gate: [tokens, heads * size] or [tokens, heads]");
     p.gate = gate->data_ptr();
     p.gate_stride = gate->stride(0);
+  }
+  TORCH_CHECK(chunk <= 0 || causal, "attention over chunks is causal");
+  p.chunk = chunk > 0 ? (int)chunk : 0;
+  if (sigmoid_shift.has_value()) {
+    TORCH_CHECK(sigmoid_shift->scalar_type() == at::kFloat && sigmoid_shift->is_contiguous() && sigmoid_shift->numel() == H,
+                "sigmoid weights: one fp32 number per head");
+    p.sigmoid_shift = sigmoid_shift->template data_ptr<float>();
   }
 }
 

@@ -229,11 +229,13 @@ void attention_prefill(Tensor& out, const Tensor& q, const Tensor& k_src, const 
                        int64_t window, double softcap, const optional<Tensor>& sinks,
                        const optional<Tensor>& lse_out, int64_t batch, int64_t max_q_len, bool causal,
                        const optional<Tensor>& alibi_slopes, const optional<Tensor>& distance_bias,
-                       const optional<Tensor>& bias_tiles, const optional<Tensor>& gate, double out_scale) {
+                       const optional<Tensor>& bias_tiles, const optional<Tensor>& gate, double out_scale, int64_t chunk,
+                       const optional<Tensor>& sigmoid_shift) {
   TORCH_CHECK(q.dim() == 3 && q.stride(2) == 1 && q.stride(1) == q.size(2));
-  on_device_of(q, {&out, &k_src, &query_start_loc}, {&v_src, &distance_bias, &bias_tiles, &gate});
+  on_device_of(q, {&out, &k_src, &query_start_loc}, {&v_src, &alibi_slopes, &distance_bias, &bias_tiles, &gate, &sigmoid_shift});
   b200::PrefillParams p{};
-  attn_extras(p, out, distance_bias, gate, out_scale);
+  attn_extras(p, out, distance_bias, gate, out_scale, chunk, sigmoid_shift, causal);
+  TORCH_CHECK(!sigmoid_shift.has_value() || !(sinks.has_value() || lse_out.has_value()), "sigmoid weights have no denominator");
   p.alibi_slopes = ptr<float>(alibi_slopes);
   const int T = q.size(0), Hq = q.size(1), DQK = q.size(2);
   const bool paged = block_table.has_value();
@@ -304,7 +306,7 @@ void attention_prefill(Tensor& out, const Tensor& q, const Tensor& k_src, const 
     const char* e = std::getenv("B200_ATTN_PREFILL_SINGLE");
     return e != nullptr && std::atoi(e) != 0;
   }();
-  const bool extras = distance_bias.has_value() || gate.has_value() || out_scale != 1.0 || !out.is_contiguous();
+  const bool extras = distance_bias.has_value() || gate.has_value() || p.chunk > 0 || sigmoid_shift.has_value() || out_scale != 1.0 || !out.is_contiguous();
   const bool packed = extras ? false : paged ? DQK == DV && (DQK == 64 || DQK == 128)                // the one-tile kernel wants that
                             : p.k_head_stride == DQK && p.v_head_stride == DV;
   const int rc = single_tile && packed
@@ -361,6 +363,17 @@ void gemm_simt(Tensor& out, const Tensor& a, const Tensor& w, const optional<Ten
   p.epi = make_epi(out, a, act, act_params);
   const c10::cuda::CUDAGuard guard(a.device());
   TORCH_CHECK(b200::gemm_simt(p, dtype_code(a), cur_stream()) == 0, "gemm_simt: too many rows or batches");
+}
+
+// ------------------------------------------------------------------ rotation
+void rope_angles(Tensor& out, const Tensor& positions, const Tensor& inv_freq) {
+  on_device_of(out, {&positions, &inv_freq});
+  TORCH_CHECK(out.dim() == 3 && out.size(1) == 2 && out.is_contiguous() && out.scalar_type() == at::kFloat);
+  TORCH_CHECK(inv_freq.scalar_type() == at::kDouble && inv_freq.is_contiguous() && inv_freq.numel() == out.size(2));
+  TORCH_CHECK(positions.scalar_type() == at::kLong && positions.is_contiguous() && positions.numel() >= out.size(0));
+  const c10::cuda::CUDAGuard guard(out.device());
+  b200::rope_angles(out.data_ptr<float>(), positions.data_ptr<int64_t>(), inv_freq.data_ptr<double>(), out.size(0),
+                    out.size(2), cur_stream());
 }
 
 // ------------------------------------------------------------------ boundary of decoders that norm both sides of a sublayer
@@ -466,7 +479,9 @@ TORCH_LIBRARY(b200, m) {
       "attention_prefill(Tensor(a!) out, Tensor q, Tensor k_src, Tensor? v_src, Tensor? block_table, "
       "Tensor? seq_lens, Tensor query_start_loc, Tensor? kv_start_loc, float scale, int window, float softcap, "
       "Tensor? sinks, Tensor(b!)? lse_out, int batch, int max_q_len, bool causal, Tensor? alibi_slopes=None, "
-      "Tensor? distance_bias=None, Tensor? bias_tiles=None, Tensor? gate=None, float out_scale=1.0) -> ()",
+      "Tensor? distance_bias=None, Tensor? bias_tiles=None, Tensor? gate=None, float out_scale=1.0, int chunk=0, "
+      "Tensor? sigmoid_shift=None) -> ()",
       &attention_prefill);
+  m.def("rope_angles(Tensor(a!) out, Tensor positions, Tensor inv_freq) -> ()", &rope_angles);
   m.def("get_status(int device) -> Tensor", &get_status);
 }

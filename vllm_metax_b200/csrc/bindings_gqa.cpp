@@ -19,14 +19,16 @@ void paged_attention_decode(Tensor& out, const Tensor& q, const Tensor& k_cache,
                             const optional<Tensor>& sinks, const optional<Tensor>& lse_out,
                             const optional<Tensor>& workspace, int64_t num_splits, int64_t batch, int64_t max_q_len,
                             double k_scale, double v_scale, bool causal, const optional<Tensor>& alibi_slopes,
-                            const optional<Tensor>& distance_bias, const optional<Tensor>& gate, double out_scale) {
+                            const optional<Tensor>& distance_bias, const optional<Tensor>& gate, double out_scale, int64_t chunk,
+                            const optional<Tensor>& sigmoid_shift) {
   TORCH_CHECK(q.dim() == 3 && q.stride(2) == 1 && q.stride(1) == q.size(2), "q must be [T, Hq, D] with packed heads");
   on_device_of(q, {&out, &k_cache, &v_cache, &block_table, &seq_lens},
-               {&kv_scales, &query_start_loc, &sinks, &lse_out, &workspace, &alibi_slopes, &distance_bias, &gate});
+               {&kv_scales, &query_start_loc, &sinks, &lse_out, &workspace, &alibi_slopes, &distance_bias, &gate, &sigmoid_shift});
   const PagedViews pv = paged_views(k_cache, v_cache);
   TORCH_CHECK(block_table.scalar_type() == at::kInt && seq_lens.scalar_type() == at::kInt);
   b200::DecodeParams p{};
-  attn_extras(p, out, distance_bias, gate, out_scale);
+  attn_extras(p, out, distance_bias, gate, out_scale, chunk, sigmoid_shift, causal);
+  TORCH_CHECK(!sigmoid_shift.has_value() || !(sinks.has_value() || lse_out.has_value()), "sigmoid weights have no denominator");
   const int T = q.size(0), Hq = q.size(1), D = pv.dv;
   TORCH_CHECK(q.size(2) == pv.dqk && out.size(0) == T && out.size(1) == Hq && out.size(2) == D && Hq % pv.heads == 0);
   p.out = out.data_ptr();
@@ -62,8 +64,8 @@ void paged_attention_decode(Tensor& out, const Tensor& q, const Tensor& k_cache,
   auto aligned = [](const Tensor& t) { return reinterpret_cast<uintptr_t>(t.data_ptr()) % 16 == 0; };
   const bool simt = dtype_code(q) == 2 || std::max(pv.dqk, pv.dv) > 256;
   if (simt) {                                  // fp32, or wider heads than the tensor-core kernels' tiles
-    TORCH_CHECK(k_cache.scalar_type() == q.scalar_type() && !alibi_slopes.has_value() && !lse_out.has_value(),
-                "fp32 / wide-head paged attention: a cache of q's type, no ALiBi, no log-sum-exps");
+    TORCH_CHECK(k_cache.scalar_type() == q.scalar_type() && !lse_out.has_value(),
+                "fp32 / wide-head paged attention: a cache of q's type, no log-sum-exps");
     TORCH_CHECK(b200::paged_attn_simt(p, dtype_code(q), batch, cur_stream()) == 0, "paged attention: heads up to 1024 wide");
     return;
   }
@@ -84,16 +86,22 @@ void paged_attention_decode(Tensor& out, const Tensor& q, const Tensor& k_cache,
 }
 
 // The epilogue of a merged q | k | v product (columns q_off, k_off, v_off); without caches: queries only.
-void head_norm_rope(Tensor& q_out, const Tensor& qkv, int64_t q_off, int64_t k_off, int64_t v_off,
+// (null q_out: keys and values only).
+void head_norm_rope(const optional<Tensor>& q_out, const Tensor& qkv, int64_t q_off, int64_t k_off, int64_t v_off,
                     const optional<Tensor>& k_cache, const optional<Tensor>& v_cache, const optional<Tensor>& q_w,
                     const optional<Tensor>& k_w, int64_t dim, const optional<Tensor>& angles, const Tensor& slot_mapping,
-                    double eps, bool one_plus, bool whole_row, bool interleaved, const optional<Tensor>& positions,
-                    double temp_coef, int64_t temp_every) {
-  on_device_of(qkv, {&q_out, &slot_mapping}, {&k_cache, &v_cache, &q_w, &k_w, &angles, &positions});
-  const int64_t T = qkv.size(0), H = q_out.size(1), DP = q_out.size(2);
+                    double eps, bool normed, bool one_plus, bool whole_row, bool interleaved, const optional<Tensor>& positions,
+                    double temp_coef, int64_t temp_every, const optional<Tensor>& q_scale) {
+  on_device_of(qkv, {&slot_mapping}, {&q_out, &k_cache, &v_cache, &q_w, &k_w, &angles, &positions, &q_scale});
+  TORCH_CHECK(q_out.has_value() || k_cache.has_value());
+  const int64_t T = qkv.size(0), H = q_out.has_value() ? q_out->size(1) : 0, DP = q_out.has_value() ? q_out->size(2) : k_cache->size(3);
   const auto dt = qkv.scalar_type();
-  TORCH_CHECK(qkv.dim() == 2 && qkv.stride(1) == 1 && q_out.dim() == 3 && q_out.is_contiguous() && q_out.size(0) == T &&
-              q_out.scalar_type() == dt && dim <= DP && q_off + H * DP <= qkv.size(1));
+  TORCH_CHECK(qkv.dim() == 2 && qkv.stride(1) == 1 && dim <= DP && q_off + H * DP <= qkv.size(1));
+  if (q_out.has_value())
+    TORCH_CHECK(q_out->dim() == 3 && q_out->is_contiguous() && q_out->size(0) == T && q_out->scalar_type() == dt);
+  TORCH_CHECK(normed || !(q_w.has_value() || k_w.has_value()), "norm weights without a norm");
+  if (q_scale.has_value())
+    TORCH_CHECK(q_scale->scalar_type() == at::kFloat && q_scale->is_contiguous() && q_scale->numel() == H, "one fp32 factor per query head");
   if (angles.has_value())
     TORCH_CHECK(angles->dim() == 3 && angles->size(0) == T && angles->size(1) == 2 && angles->scalar_type() == at::kFloat &&
                 angles->is_contiguous() && 2 * angles->size(2) <= dim, "angles [tokens, 2, half of the rotated entries]");
@@ -103,7 +111,7 @@ void head_norm_rope(Tensor& q_out, const Tensor& qkv, int64_t q_off, int64_t k_o
   b200::HeadNormRopeParams p{};
   auto aligned = [](const void* a) { return reinterpret_cast<uintptr_t>(a) % 16 == 0; };
   const int64_t unit = 16 / (int64_t)qkv.element_size();
-  p.vec = DP % 8 == 0 && q_off % unit == 0 && qkv.stride(0) % unit == 0 && aligned(qkv.data_ptr()) && aligned(q_out.data_ptr());
+  p.vec = DP % 8 == 0 && q_off % unit == 0 && qkv.stride(0) % unit == 0 && aligned(qkv.data_ptr()) && aligned(ptr(q_out));
   for (const auto* w : {&q_w, &k_w})
     if (w->has_value()) {
       const int64_t rows = !whole_row ? 1 : w == &q_w ? H : k_cache.has_value() ? k_cache->size(2) : 1;
@@ -123,7 +131,7 @@ void head_norm_rope(Tensor& q_out, const Tensor& qkv, int64_t q_off, int64_t k_o
             aligned(p.k_cache) && aligned(p.v_cache);
   }
   p.qkv = qkv.data_ptr(); p.row_stride = qkv.stride(0); p.q_off = q_off; p.k_off = k_off; p.v_off = v_off;
-  p.q_out = q_out.data_ptr(); p.q_w = ptr(q_w); p.k_w = ptr(k_w);
+  p.q_out = ptr(q_out); p.q_w = ptr(q_w); p.k_w = ptr(k_w); p.normed = normed; p.q_scale = ptr<float>(q_scale);
   p.angles = ptr<float>(angles); p.slots = slot_mapping.data_ptr<int64_t>();
   p.vec = p.vec && aligned(p.angles);
   p.tokens = T; p.heads = H; p.dim = dim; p.dim_pad = DP; p.rot = angles.has_value() ? 2 * (int)angles->size(2) : 0;
@@ -135,16 +143,6 @@ void head_norm_rope(Tensor& q_out, const Tensor& qkv, int64_t q_off, int64_t k_o
   TORCH_CHECK(b200::head_norm_rope(p, dtype_code(qkv), cur_stream()) == 0, "head_norm_rope: heads up to 1024 wide");
 }
 
-void rope_angles(Tensor& out, const Tensor& positions, const Tensor& inv_freq) {
-  on_device_of(out, {&positions, &inv_freq});
-  TORCH_CHECK(out.dim() == 3 && out.size(1) == 2 && out.is_contiguous() && out.scalar_type() == at::kFloat);
-  TORCH_CHECK(inv_freq.scalar_type() == at::kDouble && inv_freq.is_contiguous() && inv_freq.numel() == out.size(2));
-  TORCH_CHECK(positions.scalar_type() == at::kLong && positions.is_contiguous() && positions.numel() >= out.size(0));
-  const c10::cuda::CUDAGuard guard(out.device());
-  b200::rope_angles(out.data_ptr<float>(), positions.data_ptr<int64_t>(), inv_freq.data_ptr<double>(), out.size(0),
-                    out.size(2), cur_stream());
-}
-
 }  // namespace
 
 TORCH_LIBRARY_FRAGMENT(b200, m) {
@@ -153,12 +151,11 @@ TORCH_LIBRARY_FRAGMENT(b200, m) {
       "Tensor seq_lens, Tensor? query_start_loc, float scale, int window, float softcap, Tensor? sinks, "
       "Tensor(b!)? lse_out, Tensor(c!)? workspace, int num_splits, int batch, int max_q_len, float k_scale, "
       "float v_scale, bool causal, Tensor? alibi_slopes=None, Tensor? distance_bias=None, Tensor? gate=None, "
-      "float out_scale=1.0) -> ()",
+      "float out_scale=1.0, int chunk=0, Tensor? sigmoid_shift=None) -> ()",
       &paged_attention_decode);
   m.def(
-      "head_norm_rope(Tensor(a!) q_out, Tensor qkv, int q_off, int k_off, int v_off, Tensor(b!)? k_cache, Tensor(c!)? v_cache, "
-      "Tensor? q_w, Tensor? k_w, int dim, Tensor? angles, Tensor slot_mapping, float eps, bool one_plus, bool whole_row, "
-      "bool interleaved, Tensor? positions, float temp_coef, int temp_every) -> ()",
+      "head_norm_rope(Tensor(a!)? q_out, Tensor qkv, int q_off, int k_off, int v_off, Tensor(b!)? k_cache, Tensor(c!)? v_cache, "
+      "Tensor? q_w, Tensor? k_w, int dim, Tensor? angles, Tensor slot_mapping, float eps, bool normed, bool one_plus, "
+      "bool whole_row, bool interleaved, Tensor? positions, float temp_coef, int temp_every, Tensor? q_scale) -> ()",
       &head_norm_rope);
-  m.def("rope_angles(Tensor(a!) out, Tensor positions, Tensor inv_freq) -> ()", &rope_angles);
 }

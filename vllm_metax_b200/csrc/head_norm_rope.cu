@@ -1,11 +1,11 @@
 // Epilogue of a merged q | k | v product, per token and head: RMS norm over the head (shared weights for all heads) or over all
-// heads together, rotation of its first `rot` entries in pairs (i, i + rot / 2) or (2i, 2i + 1), a factor for queries that grows
-// with the position, then queries to a packed tensor and keys, together with the values, to their paged cache row - one launch.
-// Layers that read another layer's cache pass queries only.
+// heads together (with weights or without), rotation of its first `rot` entries in pairs (i, i + rot / 2) or (2i, 2i + 1), a
+// factor for queries that grows with the position or one per head, then queries to a packed tensor and keys, together with the
+// values, to their paged cache row - one launch.  Layers that read another layer's cache pass queries only; queries that stay
+// as they are need no launch, and then keys and values pass alone (heads = 0).
 //
 // Heads may be padded with zeros to a multiple of 8 (`dim_pad`); the mean runs over the `dim` real entries.  Cosines and sines
-// come from a table of the step's tokens that all layers of one rotation share (`rope_angles`): an angle is position *
-// frequency, whole turns taken off in fp64, so that far positions keep the accuracy of near ones.  The rest is fp32.
+// come from a table of the step's tokens that all layers of one rotation share (rope_angles.cu).  The arithmetic is fp32.
 #include "ops.h"
 #include "row_vec.cuh"
 
@@ -13,20 +13,6 @@ namespace b200 {
 namespace {
 
 constexpr int kThreads = 256, kCtas = 8;           // kCtas: CTAs per SM that walk the tokens
-
-__global__ void rope_angles_kernel(float* __restrict__ out, const int64_t* __restrict__ positions,
-                                   const double* __restrict__ inv_freq, int64_t n, int half) {
-  const int64_t id = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
-  if (id >= n) return;
-  const int64_t t = id / half;
-  const int i = (int)(id % half);
-  double turns = (double)positions[t] * inv_freq[i] * 0.15915494309189533577;       // angle / 2 pi
-  turns -= rint(turns);
-  float s, c;
-  sincosf((float)(turns * 6.28318530717958647693), &s, &c);
-  out[(2 * t) * half + i] = c;
-  out[(2 * t + 1) * half + i] = s;
-}
 
 // Where head `item` (queries, then keys) of token t is read and written; dst is null where nothing is written.
 template <typename T>
@@ -60,10 +46,11 @@ __device__ __forceinline__ void cache_rows(const HeadNormRopeParams& p, int64_t 
   v_row = block * p.page_stride + (int64_t)at * p.kv_heads * p.vdim_pad;
 }
 
-// What token t's queries are multiplied by.
-__device__ __forceinline__ float query_temp(const HeadNormRopeParams& p, int64_t t) {
-  if (p.positions == nullptr) return 1.f;
-  return 1.f + p.temp_coef * logf((float)((p.positions[t] + 1) / p.temp_every) + 1.f);
+// What head h of token t's queries is multiplied by.
+__device__ __forceinline__ float query_temp(const HeadNormRopeParams& p, int64_t t, int h) {
+  const float f = p.q_scale != nullptr ? p.q_scale[h] : 1.f;
+  if (p.positions == nullptr) return f;
+  return f * (1.f + p.temp_coef * logf((float)((p.positions[t] + 1) / p.temp_every) + 1.f));
 }
 
 // Pairs (2i, 2i + 1) of 8 entries from c0 on; `cs`, `sn`: the token's cosines and sines.
@@ -99,12 +86,12 @@ head_norm_rope_vec_kernel(const HeadNormRopeParams p, int log_lanes, int items) 
   const T* col = reinterpret_cast<const T*>(p.qkv) +
                  (value ? p.v_off + v_at : (is_q ? p.q_off : p.k_off) + (int64_t)h * p.dim_pad + c0);
   const T* w = reinterpret_cast<const T*>(is_q ? p.q_w : p.k_w);
-  const bool norm = p.q_w != nullptr;                          // (uniform: both weights or none)
+  const bool norm = p.normed, weighted = p.q_w != nullptr;     // (uniform: both weights or none)
   const float* ang = p.angles + (first ? c0 : c0 - half);
   float g[8];
 #pragma unroll
   for (int k = 0; k < 8; ++k) g[k] = 1.f;
-  if (head && norm) {
+  if (head && weighted) {
     load_row<T, 8, true>(w, c0, p.dim_pad, g);
 #pragma unroll
     for (int k = 0; k < 8; ++k) g[k] += p.one_plus ? 1.f : 0.f;
@@ -146,7 +133,7 @@ head_norm_rope_vec_kernel(const HeadNormRopeParams p, int log_lanes, int items) 
       }
     }
     if (head && is_q) {
-      const float temp = query_temp(p, t);
+      const float temp = query_temp(p, t, h);
 #pragma unroll
       for (int k = 0; k < 8; ++k) v[k] *= temp;
     }
@@ -188,11 +175,11 @@ head_norm_rope_kernel(const HeadNormRopeParams p) {
     __syncwarp();
     for (int i = lane; i < p.dim_pad; i += 32) {
       float f = to_f(src[i]);
-      if (w != nullptr) f = f * inv * (p.one_plus ? 1.f + to_f(w[i]) : to_f(w[i]));
+      if (p.normed) f = f * inv * (w == nullptr ? 1.f : p.one_plus ? 1.f + to_f(w[i]) : to_f(w[i]));
       buf[i] = f;
     }
     __syncwarp();
-    const float temp = item < p.heads ? query_temp(p, t) : 1.f;
+    const float temp = item < p.heads ? query_temp(p, t, item) : 1.f;
     if (dst != nullptr)
       for (int i = lane; i < p.dim_pad; i += 32) {
         float f = buf[i];
@@ -243,7 +230,6 @@ row_norm_rope_kernel(const HeadNormRopeParams p) {
   }
   const int half = p.rot / 2;
   const float *cs = p.angles + 2 * t * half, *sn = cs + half;
-  const float temp = query_temp(p, t);
   for (int u = threadIdx.x; u < nq + nk; u += kThreads) {
     const bool is_q = u < nq;
     if (!is_q && k_row < 0) break;
@@ -269,6 +255,7 @@ row_norm_rope_kernel(const HeadNormRopeParams p) {
       }
     }
     if (is_q) {
+      const float temp = query_temp(p, t, h);
 #pragma unroll
       for (int k = 0; k < 8; ++k) v[k] *= temp;
       store_row<T, 8, VEC>(reinterpret_cast<T*>(p.q_out) + (t * p.heads + h) * p.dim_pad + c0, 0, 8, v);
@@ -287,8 +274,8 @@ row_norm_rope_kernel(const HeadNormRopeParams p) {
 
 template <typename T>
 int launch(const HeadNormRopeParams& p, cudaStream_t stream) {
-  if (p.rot > p.dim || p.rot % 2 != 0 || p.dim_pad > kMaxDim) return 1;
-  if (p.k_cache != nullptr && (p.q_w == nullptr) != (p.k_w == nullptr)) return 1;
+  if (p.rot > p.dim || p.rot % 2 != 0 || p.dim_pad > kMaxDim || p.heads + p.kv_heads == 0) return 1;
+  if (p.heads > 0 && p.k_cache != nullptr && (p.q_w == nullptr) != (p.k_w == nullptr)) return 1;
   if (p.whole_row) {
     if (p.q_w == nullptr || p.dim_pad % 8 != 0) return 1;
     if (p.vec) row_norm_rope_kernel<T, true><<<p.tokens, kThreads, 0, stream>>>(p);
@@ -317,12 +304,6 @@ int head_norm_rope(const HeadNormRopeParams& p, int dtype, cudaStream_t stream) 
   if (dtype == 0) return launch<__nv_bfloat16>(p, stream);
   if (dtype == 1) return launch<__half>(p, stream);
   return launch<float>(p, stream);
-}
-
-void rope_angles(float* out, const int64_t* positions, const double* inv_freq, int tokens, int half, cudaStream_t stream) {
-  const int64_t n = (int64_t)tokens * half;
-  if (n <= 0) return;
-  rope_angles_kernel<<<(unsigned)((n + kThreads - 1) / kThreads), kThreads, 0, stream>>>(out, positions, inv_freq, n, half);
 }
 
 }  // namespace b200

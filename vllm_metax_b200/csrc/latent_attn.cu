@@ -6,16 +6,14 @@
 //                     (decode path), one warp per (token, head)
 //   latent_attn_simt  absorbed attention on the CUDA cores: fp32 caches, and 16-bit sizes the tensor-core kernel
 //                     (mla_decode.cu) does not take
-// Angles are position * inv_freq in fp32; pairs are (i, i + rot_dims / 2).
+// Cosines and sines come from the step's table (head_norm_rope.cu:rope_angles); pairs are (i, i + rot_dims / 2) or (2i, 2i + 1).
 #include "common.cuh"
 #include "ops.h"
 
 namespace b200 {
 namespace {
 
-__device__ __forceinline__ void rotate_pair(float& u, float& v, float pos, float f) {
-  float s, c;
-  sincosf(pos * f, &s, &c);
+__device__ __forceinline__ void rotate_pair(float& u, float& v, float c, float s) {
   const float a = u * c - v * s, b = v * c + u * s;
   u = a;
   v = b;
@@ -95,13 +93,14 @@ latent_insert_kernel(const LatentInsertParams p) {
   T* dst = reinterpret_cast<T*>(p.cache) + slot * p.row_elems;
   scaled(dst, ak, reinterpret_cast<const T*>(p.kv_w), p.kv_rank, 1.f / sqrtf(sk / (float)p.kv_rank + p.eps));
   const T* kr = ak + p.kv_rank;
-  const int half = p.rot_dims / 2;
-  const float pos = (float)p.positions[t];
+  const int half = p.rot_dims / 2, step = p.interleaved ? 2 : 1, apart = p.interleaved ? 1 : half;
+  const float* cs = p.angles + 2 * t * half;
   for (int i = tid; i < half; i += 128) {
-    float u = to_f(kr[i]), v = to_f(kr[i + half]);
-    rotate_pair(u, v, pos, p.inv_freq[i]);
-    dst[p.kv_rank + i] = from_f<T>(u);
-    dst[p.kv_rank + half + i] = from_f<T>(v);
+    const int at = i * step;
+    float u = to_f(kr[at]), v = to_f(kr[at + apart]);
+    rotate_pair(u, v, cs[i], cs[half + i]);
+    dst[p.kv_rank + at] = from_f<T>(u);
+    dst[p.kv_rank + at + apart] = from_f<T>(v);
   }
   for (int i = 2 * half + tid; i < p.rot_dim; i += 128) dst[p.kv_rank + i] = kr[i];
   for (int i = p.kv_rank + p.rot_dim + tid; i < p.row_elems; i += 128) dst[i] = from_f<T>(0.f);
@@ -109,22 +108,22 @@ latent_insert_kernel(const LatentInsertParams p) {
 
 template <typename T>
 __global__ void latent_rope_kernel(const T* src, int64_t src_tok, int64_t src_head, T* dst, int64_t dst_tok,
-                                   int64_t dst_head, const int64_t* __restrict__ positions,
-                                   const float* __restrict__ inv_freq, int tokens, int heads, int rot_dim, int rot_dims,
-                                   int pad) {
+                                   int64_t dst_head, const float* __restrict__ angles, int tokens, int heads, int rot_dim,
+                                   int rot_dims, int pad, int interleaved) {
   const int64_t w = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
   if (w >= (int64_t)tokens * heads) return;
   const int64_t t = w / heads, h = w % heads;
   const T* s = src + t * src_tok + h * src_head;
   T* d = dst + t * dst_tok + h * dst_head;
-  const int half = rot_dims / 2;
-  const float pos = (float)positions[t];
+  const int half = rot_dims / 2, step = interleaved ? 2 : 1, apart = interleaved ? 1 : half;
+  const float* cs = angles + 2 * t * half;
   for (int i = lane; i < half; i += 32) {
-    float u = to_f(s[i]), v = to_f(s[i + half]);
-    rotate_pair(u, v, pos, inv_freq[i]);
-    d[i] = from_f<T>(u);
-    d[i + half] = from_f<T>(v);
+    const int at = i * step;
+    float u = to_f(s[at]), v = to_f(s[at + apart]);
+    rotate_pair(u, v, cs[i], cs[half + i]);
+    d[at] = from_f<T>(u);
+    d[at + apart] = from_f<T>(v);
   }
   if (s != d)
     for (int i = 2 * half + lane; i < rot_dim; i += 32) d[i] = s[i];
@@ -229,13 +228,13 @@ int latent_insert(const LatentInsertParams& p, int dtype, cudaStream_t stream) {
 }
 
 int latent_rope(const void* src, int64_t src_tok, int64_t src_head, void* dst, int64_t dst_tok, int64_t dst_head,
-                const int64_t* positions, const float* inv_freq, int tokens, int heads, int rot_dim, int rot_dims, int pad,
-                int dtype, cudaStream_t stream) {
+                const float* angles, int tokens, int heads, int rot_dim, int rot_dims, int pad, bool interleaved, int dtype,
+                cudaStream_t stream) {
   const int64_t warps = (int64_t)tokens * heads;
   if (warps <= 0) return 0;
   BY_DTYPE((latent_rope_kernel<T><<<(unsigned)((warps + 3) / 4), 128, 0, stream>>>(
-      (const T*)src, src_tok, src_head, (T*)dst, dst_tok, dst_head, positions, inv_freq, tokens, heads, rot_dim, rot_dims,
-      pad)))
+      (const T*)src, src_tok, src_head, (T*)dst, dst_tok, dst_head, angles, tokens, heads, rot_dim, rot_dims, pad,
+      interleaved)))
   return 0;
 }
 

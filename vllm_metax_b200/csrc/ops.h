@@ -50,8 +50,11 @@ struct DecodeParams {
                                        //   is that of distance clamp(bias_len + 126 - y, 0, bias_len - 1)
   const void* gate = nullptr;    // [T, Hq * dv] (token stride gate_stride): the result is multiplied by its sigmoid
   int64_t gate_stride = 0;
+  int gate_per_head = 0;         //   ... [T, Hq]: one number per head
   float out_scale = 1.f;
   int64_t out_stride = 0;        // elements between two tokens of out (0: packed)
+  int chunk = 0;                 // > 0 (causal): a position sees its own chunk of this many positions, counted from 0
+  const float* sigmoid_shift = nullptr;   // [Hq]: a key's weight is sigmoid(score + shift), no softmax over the keys
 };
 
 struct PrefillParams {
@@ -80,8 +83,11 @@ struct PrefillParams {
                                        //   is that of distance clamp(bias_len + 126 - y, 0, bias_len - 1)
   const void* gate = nullptr;    // [T, Hq * dv] (token stride gate_stride): the result is multiplied by its sigmoid
   int64_t gate_stride = 0;
+  int gate_per_head = 0;         //   ... [T, Hq]: one number per head
   float out_scale = 1.f;
   int64_t out_stride = 0;        // elements between two tokens of out (0: packed)
+  int chunk = 0;                 // > 0 (causal): a position sees its own chunk of this many positions, counted from 0
+  const float* sigmoid_shift = nullptr;   // [Hq]: a key's weight is sigmoid(score + shift), no softmax over the keys
 };
 
 struct MlaDecodeParams {
@@ -385,13 +391,30 @@ struct PrenormParams {
   StatusWord* status;
 };
 int prenorm(const PrenormParams& p, int dtype, cudaStream_t stream);
+// ---- stream_norm.cu (sublayer boundary of decoders whose residual is several streams)
+constexpr int kMaxStreams = 8;
+struct StreamNormParams {
+  const void* y;           // [tokens, D] the finished sublayer's output, or null in front of the first one
+  const float* x;          // [tokens, streams, D], or null: every stream is scale * table[ids]
+  const void* table; const int64_t* ids; int64_t rows; float scale;
+  const float* coef;       // [streams] read | [streams] write | [streams, streams] mix (from, to)
+  const float* gain;       // [D]
+  float* x_out;            // [tokens, streams, D] (may be x) or null
+  void* h;                 // [tokens, D]
+  int tokens, D, streams, vec;
+  float eps;
+  StatusWord* status;
+};
+int stream_norm(const StreamNormParams& p, int dtype, cudaStream_t stream);
 // ---- head_norm_rope.cu (epilogue of a merged q | k | v product: head norms, partial rotation, paged cache write)
 struct HeadNormRopeParams {
   const void* qkv; int64_t row_stride; int q_off, k_off, v_off;   // [tokens, ...], heads packed from these columns on
-  void* q_out;                          // [tokens, heads, dim_pad]
+  void* q_out;                          // [tokens, heads, dim_pad] (heads = 0: keys and values only)
   void* k_cache; void* v_cache;         // K / V of page 0, or null: queries only
   int64_t page_stride, num_slots;       // elements between two pages
-  const void* q_w; const void* k_w;     // [dim_pad] norm weights or null (no norm)
+  const void* q_w; const void* k_w;     // [dim_pad] norm weights or null
+  int normed;                           // 0: no norm (without weights a norm multiplies by one)
+  const float* q_scale;                 // [heads]: factors of the queries, or null
   const float* angles;                  // [tokens, 2, rot / 2]: cosines, sines
   const int64_t* slots;
   int tokens, heads, kv_heads, dim, dim_pad, vdim_pad, rot, block_size, one_plus, vec;
@@ -471,19 +494,20 @@ int rglru_scan(const RgLruParams& p, int max_query_len, int dtype, cudaStream_t 
 struct LatentInsertParams {
   const void* a; int64_t a_stride; int q_off, kv_off;   // [tokens, ...]: query latent | key latent, rotated key part
   const void* q_w; const void* kv_w;                    // norm weights
-  void* cq;                                             // [tokens, q_rank]
+  void* cq;                                             // [tokens, q_rank] (q_rank = 0: no query latent)
   void* cache; int64_t row_elems, num_slots;            // [slots, row_elems]
-  const int64_t* slots; const int64_t* positions;
-  const float* inv_freq;                                // [rot_dims / 2]
+  const int64_t* slots;
+  const float* angles;                                  // [tokens, 2, rot_dims / 2]: cosines, sines
   int tokens, q_rank, kv_rank, rot_dim, rot_dims;
+  int interleaved;                                      // pairs (2i, 2i + 1) instead of (i, i + rot_dims / 2)
   float eps;
   StatusWord* status;
 };
 int latent_insert(const LatentInsertParams& p, int dtype, cudaStream_t stream);
 // Rotates the first rot_dims of the rot_dim entries at src (per token and head) into dst and zeroes `pad` entries behind.
 int latent_rope(const void* src, int64_t src_tok, int64_t src_head, void* dst, int64_t dst_tok, int64_t dst_head,
-                const int64_t* positions, const float* inv_freq, int tokens, int heads, int rot_dim, int rot_dims, int pad,
-                int dtype, cudaStream_t stream);
+                const float* angles, int tokens, int heads, int rot_dim, int rot_dims, int pad, bool interleaved, int dtype,
+                cudaStream_t stream);
 int latent_attn_simt(const MlaDecodeParams& p, int dtype, cudaStream_t stream);
 // ---- tq_cache.cu (TurboQuant KV cache, head_dim 128)
 int tq_slot_bytes(int kbits, int vbits);

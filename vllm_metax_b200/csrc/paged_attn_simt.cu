@@ -3,7 +3,9 @@
 // of query tokens per sequence.
 //
 // One CTA per (query token, head): 128 keys at a time, eight lanes per key for the scores (coalesced rows), then a thread per
-// value column.  Online softmax in fp32, with the soft-cap, distance bias, sinks and output gate of the tensor-core kernels.
+// value column.  Online softmax in fp32 (or sigmoid weights), with the soft-cap, distance biases, sinks, chunks and output gate of
+// the tensor-core kernels.
+#include "attn_score.cuh"
 #include "ops.h"
 #include "row_vec.cuh"
 
@@ -33,7 +35,9 @@ paged_attn_simt_kernel(const DecodeParams p, int batch) {
   const int q0 = p.query_start_loc ? p.query_start_loc[b] : b, q1 = p.query_start_loc ? p.query_start_loc[b + 1] : b + 1;
   const int len = p.seq_lens[b], pos = len - (q1 - q0) + (t - q0) + 1;
   const int lim = p.causal ? pos : len;
-  const int first = p.window > 0 ? max(0, lim - p.window) : 0;
+  const int first = first_key(lim, p.window, p.chunk);
+  const bool sigmoid = p.sigmoid_shift != nullptr;
+  const float slope = p.alibi_slopes != nullptr ? p.alibi_slopes[h] : 0.f, shift = sigmoid ? p.sigmoid_shift[h] : 0.f;
   const int* btab = p.block_table + (int64_t)b * p.max_blocks;
   const T* q = reinterpret_cast<const T*>(p.q) + (int64_t)t * p.q_stride + (int64_t)h * p.dqk;
   for (int i = threadIdx.x; i < p.dqk; i += kKeys) s_q[i] = to_f(q[i]);
@@ -69,16 +73,22 @@ paged_attn_simt_kernel(const DecodeParams p, int batch) {
         d *= p.scale;
         if (p.softcap > 0.f) d = p.softcap * tanhf(d / p.softcap);
         if (p.bias != nullptr) d += p.bias[(int64_t)h * p.bias_len + min(max(pos - 1 - (k0 + k), 0), p.bias_len - 1)];
+        d = fmaf(slope, (float)(k0 + k - (pos - 1)), d);
         s_p[k] = r >= 0 ? d : -INFINITY;
       }
     }
     __syncthreads();
     const float s = s_p[threadIdx.x];
-    const float mx = block_max(s, red);
-    const float mn = fmaxf(m, mx), ms = mn == -INFINITY ? 0.f : mn;
-    const float corr = m == -INFINITY ? 0.f : expf(m - ms);
-    const float e = s == -INFINITY ? 0.f : expf(s - ms);
-    m = mn;
+    float corr = 1.f, e;
+    if (sigmoid) {
+      e = s == -INFINITY ? 0.f : 1.f / (1.f + expf(-(s + shift)));
+    } else {
+      const float mx = block_max(s, red);
+      const float mn = fmaxf(m, mx), ms = mn == -INFINITY ? 0.f : mn;
+      corr = m == -INFINITY ? 0.f : expf(m - ms);
+      e = s == -INFINITY ? 0.f : expf(s - ms);
+      m = mn;
+    }
     s_p[threadIdx.x] = e;
     l = l * corr + block_sum(e, red);                        // (its barriers publish s_p)
     const int nk = min(kKeys, lim - k0);
@@ -94,6 +104,7 @@ paged_attn_simt_kernel(const DecodeParams p, int batch) {
     }
   }
   float scale_o = 1.f;
+  if (sigmoid) l = 1.f;
   if (p.sinks != nullptr) {                                  // one more term of the denominator (and of its maximum)
     const float z = p.sinks[h], mn = fmaxf(m, z);
     scale_o = m == -INFINITY ? 0.f : expf(m - mn);
@@ -101,11 +112,11 @@ paged_attn_simt_kernel(const DecodeParams p, int batch) {
   }
   const float inv = l > 0.f ? p.out_scale * scale_o / l : 0.f;
   T* out = reinterpret_cast<T*>(p.out) + t * (p.out_stride ? p.out_stride : (int64_t)p.num_q_heads * p.dv) + h * p.dv;
-  const T* gate = p.gate != nullptr ? reinterpret_cast<const T*>(p.gate) + t * p.gate_stride + h * p.dv : nullptr;
+  const T* gate = p.gate != nullptr ? reinterpret_cast<const T*>(p.gate) + t * p.gate_stride + (p.gate_per_head ? h : h * p.dv) : nullptr;
 #pragma unroll
   for (int i = 0; i < kCols; ++i) {
     const int c = threadIdx.x + i * kKeys;
-    if (c < p.dv) out[c] = from_f<T>(acc[i] * inv * (gate != nullptr ? 1.f / (1.f + expf(-to_f(gate[c]))) : 1.f));
+    if (c < p.dv) out[c] = from_f<T>(acc[i] * inv * (gate != nullptr ? 1.f / (1.f + expf(-to_f(gate[p.gate_per_head ? 0 : c]))) : 1.f));
   }
 }
 

@@ -20,6 +20,7 @@ from .. import _custom_ops as ops
 from ..attention.metadata import get_forward_context
 from ..ops import turboquant as tq
 from .recurrent import StackedLinear, _param
+from .rotation import Rotation
 
 KV_DTYPES = {
     "auto": None, "bfloat16": torch.bfloat16, "float16": torch.float16, "fp8": torch.float8_e4m3fn,
@@ -95,6 +96,8 @@ class Attention(nn.Module):
         self.distance_bias: Optional[torch.Tensor] = None      # f32 [num_heads, L]: bias by distance, the last entry from L - 1 on
         self.bias_tiles: Optional[torch.Tensor] = None         # the same for the prompt kernel (ops.distance_bias_tiles)
         self.out_scale = 1.0
+        self.chunk = 0                                         # a position sees its own chunk of this many (0: no chunks)
+        self.sigmoid_shift: Optional[torch.Tensor] = None      # f32 [num_heads]: weights are sigmoid(score + shift), no softmax
 
     def forward(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, positions: Optional[torch.Tensor] = None,
                 rope=None) -> torch.Tensor:
@@ -146,7 +149,7 @@ class Attention(nn.Module):
                                        sinks=self.sinks, num_splits=md.decode_num_splits, max_seq_len=md.max_seq_len,
                                        k_scale=self.k_scale, v_scale=self.v_scale, workspace=md.decode_workspace,
                                        alibi_slopes=self.alibi_slopes, distance_bias=self.distance_bias, gate=gates[0],
-                                       out_scale=self.out_scale)
+                                       out_scale=self.out_scale, chunk=self.chunk, sigmoid_shift=self.sigmoid_shift)
         if md.num_prefills > 0:
             ops.paged_attention_prefill(q3[ndt:], kv_cache, md.block_table[nd:], md.seq_lens[nd:],
                                         md.prefill_query_start_loc, self.scale, out=out[ndt:], kv_scales=kv_scales,
@@ -154,7 +157,7 @@ class Attention(nn.Module):
                                         sinks=self.sinks, k_scale=self.k_scale, v_scale=self.v_scale,
                                         max_seq_len=md.max_seq_len, alibi_slopes=self.alibi_slopes,
                                         distance_bias=self.distance_bias, bias_tiles=self.bias_tiles, gate=gates[1],
-                                        out_scale=self.out_scale)
+                                        out_scale=self.out_scale, chunk=self.chunk, sigmoid_shift=self.sigmoid_shift)
         return out
 
     def _forward_cascade(self, q3, md, kv_cache, kv_scales) -> torch.Tensor:
@@ -300,15 +303,19 @@ class Attention(nn.Module):
 
 
 class QKNormAttention(nn.Module):
-    """Grouped-query attention with RMS-normed queries and keys, key and value sizes of its own, an optional sliding window, and
-    optionally the keys and values of another layer (``kv_from``: that layer's module, which must come earlier in the step)
+    """Grouped-query attention, by default with RMS-normed queries and keys, with key and value sizes of its own, an optional
+    sliding window or chunks, and optionally the keys and values of another layer (``kv_from``: that layer's module, which must come earlier in the step)
     instead of projections and a cache of its own.
 
         merged q | k | v product -> ``head_norm_rope`` (norms, rotation, cache write) -> paged attention -> output product
 
-    ``whole_row_norm``: one norm over all heads.  ``inv_freq=None``: no rotation; ``interleaved``: pairs (2i, 2i + 1).
-    ``q_temp = (coef, every)``: queries grow with the position.  ``bias_far`` and ``bias_rows``: a learned bias by distance, one
-    row per bucket (``distance_buckets``).  ``gated``: the heads' outputs times the sigmoid of another projection.
+    ``norm``: "weighted", "unit" (without weights) or "none"; ``whole_row_norm``: one norm over all heads.  ``inv_freq=None``: no
+    rotation; ``interleaved``: pairs (2i, 2i + 1).  ``q_temp = (coef, every)``: queries grow with the position; ``head_temp``:
+    scores are multiplied by a learned number per head.  ``bias_far`` and ``bias_rows``: a learned bias by distance, one row per
+    bucket (``distance_buckets``).  ``alibi_slopes``: a fixed slope per head.  ``log_bias``: ``r1 ln(1 + r2 distance)`` with
+    two learned numbers per head is taken off (the keys must be near: a window or chunks).  ``sigmoid``: weights are the sigmoid
+    of the score plus a learned number per head, without a softmax.  ``gated``: the heads' outputs times the sigmoid of another
+    projection, an entry each, or ("head") one number per head.
 
     Head sizes are padded to multiples of 8 with zero rows of the projections (and zero columns of the output product).
     ``standalone=False``: a branch of a :class:`layers.mixer.ProjectedMixer`, which owns the products.  ``runs``: how often a
@@ -318,9 +325,14 @@ class QKNormAttention(nn.Module):
                  inv_freq: Optional[torch.Tensor], cache_idx: int, window: Optional[int] = None,
                  kv_from: Optional["QKNormAttention"] = None, dtype=torch.bfloat16, *, standalone: bool = True, runs: int = 1,
                  whole_row_norm: bool = False, interleaved: bool = False, q_temp: Optional[tuple] = None, softcap: float = 0.0,
-                 sinks: bool = False, bias_rows: int = 0, bias_far: int = 0, gated: bool = False, proj_bias: bool = False,
-                 out_scale: float = 1.0):
+                 sinks: bool = False, bias_rows: int = 0, bias_far: int = 0, gated=False, proj_bias: bool = False,
+                 out_scale: float = 1.0, norm: str = "weighted", chunk: int = 0, head_temp: bool = False,
+                 alibi_slopes: Optional[list] = None, log_bias: bool = False, sigmoid: bool = False):
         super().__init__()
+        if norm not in ("weighted", "unit", "none") or (whole_row_norm and norm != "weighted"):
+            raise ValueError(f"norm {norm!r}" + (" over whole rows" if whole_row_norm else ""))
+        if sigmoid and sinks:
+            raise ValueError("a sink belongs to a softmax")
         if heads % kv_heads:
             raise ValueError(f"{heads} query heads over {kv_heads} key / value heads")
         self.width, self.heads, self.kv_heads, self.dim, self.vdim, self.eps = width, heads, kv_heads, dim, vdim, eps
@@ -332,22 +344,32 @@ class QKNormAttention(nn.Module):
         self.proj_bias, self.gated = proj_bias, gated
         self.out_width = heads * self.vdim_pad
         rows = (heads, kv_heads) if whole_row_norm else (1, 1)
-        self.q_norm = _param(rows[0] * self.dim_pad, dtype=dtype)
-        self.k_norm = _param(rows[1] * self.dim_pad, dtype=dtype) if self.own_kv else None
-        self.rotation = None
-        if inv_freq is not None:
-            self.rotation = ("rope_angles", tuple(inv_freq.tolist()))
-            self.register_buffer("inv_freq", inv_freq.double().to(torch.get_default_device()), persistent=False)
+        self.norm, self.dtype = norm, dtype
+        self.q_norm = _param(rows[0] * self.dim_pad, dtype=dtype) if norm == "weighted" else None
+        self.k_norm = _param(rows[1] * self.dim_pad, dtype=dtype) if norm == "weighted" and self.own_kv else None
+        self.rotation = Rotation(inv_freq) if inv_freq is not None else None
+        self.head_temp = _param(heads, dtype=torch.float32) if head_temp else None
         self.attn = Attention(heads, self.dim_pad, scale, kv_heads, cache_idx, sliding_window=window, softcap=softcap)
-        self.attn.out_scale = out_scale
+        self.attn.out_scale, self.attn.chunk = out_scale, chunk
+        if alibi_slopes is not None:
+            self.register_buffer("slopes", torch.tensor(alibi_slopes, dtype=torch.float32), persistent=False)
+            self.attn.alibi_slopes = self.slopes
+        self.shift = _param(heads, dtype=torch.float32) if sigmoid else None
+        self.attn.sigmoid_shift = self.shift
         self.sinks = _param(heads, dtype=torch.float32) if sinks else None
         self.attn.sinks = self.sinks
-        self.rel = None
+        self.rel = self.log_bias = None
+        reach = 0                                  # distances of the bias table
         if bias_rows:
-            index = distance_buckets(bias_rows, bias_far)
-            self.rel = _param(bias_rows, heads, dtype=dtype)
-            self.register_buffer("distance_bias", torch.zeros(heads, len(index), dtype=torch.float32), persistent=False)
-            self.buckets = index
+            self.buckets = distance_buckets(bias_rows, bias_far)
+            self.rel, reach = _param(bias_rows, heads, dtype=dtype), len(self.buckets)
+        elif log_bias:
+            reach = min((n for n in (window, chunk) if n), default=0)
+            if not reach:
+                raise ValueError("a logarithmic distance bias needs a window or chunks")
+            self.log_bias = _param(2, heads, dtype=torch.float32)
+        if reach:
+            self.register_buffer("distance_bias", torch.zeros(heads, reach, dtype=torch.float32), persistent=False)
             self.attn.distance_bias = self.distance_bias
             self.register_buffer("bias_tiles", ops.distance_bias_tiles(self.distance_bias, heads // kv_heads), persistent=False)
             self.attn.bias_tiles = self.bias_tiles
@@ -362,8 +384,12 @@ class QKNormAttention(nn.Module):
         if self.own_kv:
             parts.update(k=self.kv_heads * self.dim_pad, v=self.kv_heads * self.vdim_pad)
         if self.gated:
-            parts["g"] = self.out_width
+            parts["g"] = self.gate_width
         return parts
+
+    @property
+    def gate_width(self) -> int:
+        return self.heads if self.gated == "head" else self.out_width
 
     def attach(self, proj: StackedLinear, prefix: str = "") -> None:
         """The product that yields q, k, v (and g) as its parts ``prefix + name``."""
@@ -374,6 +400,11 @@ class QKNormAttention(nn.Module):
     def finalize_weights(self) -> None:
         if self.rel is not None:
             self.distance_bias.copy_(self.rel.data.float()[self.buckets].t())
+        if self.log_bias is not None:
+            r1, r2 = self.log_bias.data.double()[..., None]
+            far = torch.arange(self.distance_bias.shape[1], dtype=torch.float64, device=r1.device)
+            self.distance_bias.copy_(-r1 * torch.log1p(r2 * far))
+        if self.attn.distance_bias is not None:
             self.bias_tiles.copy_(ops.distance_bias_tiles(self.distance_bias, self.heads // self.kv_heads))
 
     def in_slots(self, proj: StackedLinear) -> dict:
@@ -388,20 +419,27 @@ class QKNormAttention(nn.Module):
             return (w.data.view(n, self.dim_pad)[:, : self.dim], (n * self.dim,)) if self.whole_row_norm else w.data[: self.dim]
 
         sizes = {"q": (self.heads, self.dim, self.dim_pad)}
-        out = {"q.norm": norm(self.q_norm, self.heads)}
+        out = {"q.norm": norm(self.q_norm, self.heads)} if self.q_norm is not None else {}
         if self.own_kv:
             sizes.update(k=(self.kv_heads, self.dim, self.dim_pad), v=(self.kv_heads, self.vdim, self.vdim_pad))
+        if self.k_norm is not None:
             out["k.norm"] = norm(self.k_norm, self.kv_heads)
         for name, s in sizes.items():
             out[name] = heads(name, *s)
             if self.proj_bias:
                 out[name + ".b"] = bias(name, *s)
         if self.gated:
-            out["g"] = heads("g", self.heads, self.vdim, self.vdim_pad)
+            out["g"] = proj.rows(self.prefix + "g") if self.gated == "head" else heads("g", self.heads, self.vdim, self.vdim_pad)
         if self.sinks is not None:
             out["sink"] = self.sinks.data
         if self.rel is not None:
             out["rel"] = self.rel.data
+        if self.log_bias is not None:
+            out["r1"], out["r2"] = self.log_bias.data
+        if self.head_temp is not None:
+            out["temp"] = self.head_temp.data
+        if self.shift is not None:
+            out["pb"] = self.shift.data
         return out
 
     def out_slot(self, weight: torch.Tensor) -> tuple:
@@ -415,7 +453,7 @@ class QKNormAttention(nn.Module):
     def decode_workspace_floats(self, batch: int, max_seq_len: int) -> int:
         """What the split decode of ``batch`` rows needs for its partial results (0: it does not split)."""
         tiles = -(-(self.heads // self.kv_heads) // 16)
-        n = ops.decode_num_splits(batch, self.kv_heads, max_seq_len, tiles, window=self.attn.window)
+        n = ops.decode_num_splits(batch, self.kv_heads, max_seq_len, tiles, window=self.attn.window, chunk=self.attn.chunk)
         return n * batch * self.heads * (self.vdim_pad + 1) if n > 1 else 0
 
     def cache_elems_per_token(self) -> int:
@@ -423,7 +461,7 @@ class QKNormAttention(nn.Module):
 
     def allocate_kv_cache(self, num_blocks: int, block_size: int, device):
         return (PagedGQABackend.allocate_pages(num_blocks, block_size, self.kv_heads, self.dim_pad, self.vdim_pad,
-                                               self.q_norm.dtype, device), None)
+                                               self.dtype, device), None)
 
     # ---- forward ----------------------------------------------------------------------------------------------------
     def mix(self, positions: torch.Tensor, h: torch.Tensor, p: torch.Tensor, out: torch.Tensor, run: int = 0) -> None:
@@ -433,17 +471,14 @@ class QKNormAttention(nn.Module):
         T = p.shape[0]
         cache = ctx.kv_caches[self.attn.layer_idx + run][0]
         kv = PagedGQABackend.views(cache, md.block_size, self.kv_heads, self.dim_pad, self.vdim_pad)
-        angles = None
-        if self.rotation is not None:                         # one table per step and rotation, shared by the layers
-            angles = ctx.extra.get(self.rotation)
-            if angles is None:
-                angles = ctx.extra[self.rotation] = ops.rope_angles(positions, self.inv_freq, T)
+        angles = self.rotation.angles(positions, T) if self.rotation is not None else None
         q = ops.head_norm_rope(p, self.offsets, self.q_norm, self.k_norm, self.heads, self.dim, angles,
                                kv if self.own_kv else None, md.slot_mapping, self.eps, whole_row=self.whole_row_norm,
-                               interleaved=self.interleaved, q_temp=(positions, *self.q_temp) if self.q_temp else None)
+                               interleaved=self.interleaved, q_temp=(positions, *self.q_temp) if self.q_temp else None,
+                               q_scale=self.head_temp, normed=self.norm != "none", width=self.dim_pad)
         gate = None
         if self.gated:
-            gate = p[:, self.gate_offset: self.gate_offset + self.out_width]
+            gate = p[:, self.gate_offset: self.gate_offset + self.gate_width]
         self.attn.attend(q, md, kv, out=out.unflatten(1, (self.heads, self.vdim_pad)), gate=gate)
 
     def forward(self, positions: torch.Tensor, h: torch.Tensor) -> torch.Tensor:

@@ -38,6 +38,22 @@ class GemmaRMSNorm(RMSNorm):
         self.weight.data.zero_()
 
 
+class NormAroundOne(nn.Module):
+    """The gain ``factor * scale * (1 + weight)`` of an RMS norm, folded into one fp32 vector for the boundary kernels.
+    ``scale`` is a layer scale (one number per channel) or absent."""
+
+    def __init__(self, width: int, dtype, factor: float = 1.0, scaled: bool = False):
+        super().__init__()
+        self.weight = nn.Parameter(torch.zeros(width, dtype=dtype), requires_grad=False)
+        self.scale = nn.Parameter(torch.zeros(width, dtype=dtype), requires_grad=False) if scaled else None
+        self.factor = factor
+        self.register_buffer("gain", torch.zeros(width, dtype=torch.float32), persistent=False)
+
+    def finalize_weights(self) -> None:
+        g = self.factor * (1.0 + self.weight.data.float())
+        self.gain.copy_(g if self.scale is None else g * self.scale.data.float())
+
+
 class RMSNormGated(nn.Module):
     def __init__(self, hidden_size, eps=1e-6, dtype=torch.bfloat16):
         super().__init__()

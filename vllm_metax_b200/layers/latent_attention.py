@@ -4,7 +4,8 @@ sparse and distributed variants; both run the same attention kernels).
 Cache: one row per token and layer, ``[latent kv_rank | rotated key part rot_dim | zeros to a multiple of 8]``, paged like
 every KV cache; the rotated part is shared by the heads.
 
-    down      one product for both latents -> ``latent_insert``: norms, rotation of the key part, cache write
+    down      one product for both latents (or the queries themselves and the key latent) -> ``latent_insert``: norms, rotation of
+              the key part, cache write
     decode    absorbed form: q . W_UK per head (batched product), attention over the cached rows (``mla_decode``), . W_UV
     prompts   the cached rows a portion can see (its own tokens and up to window - 1 before it) are gathered and multiplied
               with ONE matrix that yields, head by head, [unrotated key | rotated key | value] - the rotated columns are an
@@ -20,7 +21,9 @@ import torch.nn as nn
 
 from .. import _custom_ops as ops
 from ..attention.metadata import get_forward_context
+from ..ops.reference import rope_frequencies
 from .recurrent import StackedLinear, _param
+from .rotation import Rotation
 
 # A portion takes the up-projected path unless the context rows to up-project outnumber its tokens by more than this.
 CONTEXT_PER_TOKEN = 4
@@ -57,23 +60,25 @@ def prompt_spans(md, window: int):
 
 
 class LatentAttention(nn.Module):
-    def __init__(self, width: int, heads: int, dim: int, rot_dim: int, vdim: int, q_rank: int, kv_rank: int, scale: float,
-                 window: int, rot_base: float, rot_dims: int, eps: float, cache_idx: int, dtype=torch.bfloat16):
+    def __init__(self, width: int, heads: int, dim: int, rot_dim: int, vdim: int, q_rank: Optional[int], kv_rank: int,
+                 scale: float, window: int, rot_base: float, rot_dims: int, eps: float, cache_idx: int, dtype=torch.bfloat16,
+                 interleaved: bool = False):
+        """``q_rank=None``: queries straight from the input.  ``window`` 0: none.  ``interleaved``: rotation in pairs (2i, 2i + 1)
+        instead of (i, i + half)."""
         super().__init__()
         self.heads, self.dim, self.rot_dim, self.vdim = heads, dim, rot_dim, vdim
         self.q_rank, self.kv_rank, self.scale, self.window, self.eps = q_rank, kv_rank, scale, window, eps
         self.cache_idx, self.dtype = cache_idx, dtype
         self.row = LatentCache.row_elems(kv_rank, rot_dim)
-        self.down = StackedLinear(width, {"dq": q_rank, "dkv": kv_rank + rot_dim}, dtype=dtype)
-        self.q_norm = _param(q_rank, dtype=dtype)
+        self.interleaved, q_rows = interleaved, heads * (dim + rot_dim)
+        self.down = StackedLinear(width, {"dq" if q_rank else "q": q_rank or q_rows, "dkv": kv_rank + rot_dim}, dtype=dtype)
+        self.q_norm = _param(q_rank, dtype=dtype) if q_rank else None
         self.kv_norm = _param(kv_rank, dtype=dtype)
-        self.up_q = _param(heads * (dim + rot_dim), q_rank, dtype=dtype)
+        self.up_q = _param(q_rows, q_rank, dtype=dtype) if q_rank else None
         self.up_k = _param(heads * dim, kv_rank, dtype=dtype)
         self.up_v = _param(heads * vdim, kv_rank, dtype=dtype)
         self.out_proj = _param(width, heads * vdim, dtype=dtype)
-        i = torch.arange(rot_dims // 2, dtype=torch.float64, device="cpu")
-        freq = (float(rot_base) ** (-2.0 * i / rot_dims)).float().to(torch.get_default_device())
-        self.register_buffer("inv_freq", freq, persistent=False)
+        self.rotation = Rotation(rope_frequencies(int(rot_dims), float(rot_base))[0])
         # filled by finalize_weights: W_UK transposed per head, and the prompt path's [k | rotated k | v] matrix
         self.register_buffer("absorb_k", torch.zeros(heads, kv_rank, dim, dtype=dtype), persistent=False)
         qk = dim + rot_dim
@@ -91,15 +96,36 @@ class LatentAttention(nn.Module):
             self.up_kv[:, D: D + R, K: K + R] = torch.eye(R, dtype=self.dtype, device=uk.device)
             self.up_kv[:, D + R:, :K] = self.up_v.data.view(H, self.vdim, K)
 
-    def _absorbed(self, q, positions, cache, md, n_req: int, out) -> None:
+    def slots(self) -> dict:
+        """Tensor name -> the memory it is copied to."""
+        out = {"dkv": self.down.rows("dkv"), "dkv.norm": self.kv_norm.data, "uk": self.up_k.data, "uv": self.up_v.data,
+               "o": self.out_proj.data}
+        if self.q_rank:
+            return {"dq": self.down.rows("dq"), "dq.norm": self.q_norm.data, "uq": self.up_q.data, **out}
+        return {"q": self.down.rows("q"), **out}
+
+    # ---- cache ------------------------------------------------------------------------------------------------------
+    def cache_elems_per_token(self) -> int:
+        return self.row
+
+    def allocate_kv_cache(self, num_blocks: int, block_size: int, device) -> torch.Tensor:
+        return LatentCache.allocate(num_blocks, block_size, self.kv_rank, self.rot_dim, self.dtype, device)
+
+    def decode_workspace_floats(self, batch: int, max_seq_len: int) -> int:
+        """What the split decode of ``batch`` rows needs for its partial results (0: it does not split)."""
+        n = ops.mla_decode_num_splits(batch, self.heads, max_seq_len, self.window)
+        return n * batch * self.heads * (self.kv_rank + 1) if n > 1 else 0
+
+    # ---- forward ----------------------------------------------------------------------------------------------------
+    def _absorbed(self, q, angles, cache, md, n_req: int, out) -> None:
         """Rows [0, len(q)) of the step, which belong to its first ``n_req`` requests."""
         m, H, D, K = q.shape[0], self.heads, self.dim, self.kv_rank
         qa = torch.empty(m, H, self.row, dtype=q.dtype, device=q.device)
         ops.gemm_batched(q[..., :D].transpose(0, 1), self.absorb_k, out=qa[..., :K].transpose(0, 1))
-        ops.latent_rope(qa[..., K:], q[..., D:], self.inv_freq, positions, self.rot_dim, self.row - K - self.rot_dim)
+        ops.latent_rope(qa[..., K:], q[..., D:], angles, self.rot_dim, self.row - K - self.rot_dim, self.interleaved)
         lat = ops.mla_decode(qa, cache, md.block_table[:n_req], md.seq_lens[:n_req], self.scale,
                              query_start_loc=md.query_start_loc[:n_req + 1], max_seq_len=md.max_seq_len,
-                             window=self.window, kv_rank=K)
+                             window=self.window, kv_rank=K, workspace=md.decode_workspace)
         ops.gemm_batched(lat.transpose(0, 1), self.up_v.view(H, self.vdim, K), out=out.transpose(0, 1))
 
     def forward(self, positions, h):
@@ -107,10 +133,10 @@ class LatentAttention(nn.Module):
         md = ctx.attn_metadata
         cache = ctx.kv_caches[self.cache_idx]
         T, H, D, R, V = h.shape[0], self.heads, self.dim, self.rot_dim, self.vdim
-        a = self.down(h)
-        cq = ops.latent_insert(a, self.down.offsets["dq"], self.down.offsets["dkv"], self.q_norm, self.kv_norm, R,
-                               self.inv_freq, positions, cache, md.slot_mapping, self.eps)
-        q = ops.gemm(cq, self.up_q).view(T, H, D + R)
+        a, angles = self.down(h), self.rotation.angles(positions, T)
+        cq = ops.latent_insert(a, self.down.offsets.get("dq", 0), self.down.offsets["dkv"], self.q_norm, self.kv_norm, R,
+                               angles, cache, md.slot_mapping, self.eps, self.interleaved)
+        q = (ops.gemm(cq, self.up_q) if self.q_rank else self.down.part(a, "q")).unflatten(1, (H, D + R))
         out = torch.empty(T, H, V, dtype=h.dtype, device=h.device)
         nd, ndt = md.num_decodes, md.num_decode_tokens
         mha = self.prompt_kernel and h.is_cuda and md.num_prefills > 0
@@ -118,12 +144,12 @@ class LatentAttention(nn.Module):
             cu_rows, first, total = prompt_spans(md, self.window)
             mha = total <= CONTEXT_PER_TOKEN * (T - ndt)
         if not mha:
-            self._absorbed(q, positions, cache, md, md.num_reqs, out)
+            self._absorbed(q, angles, cache, md, md.num_reqs, out)
         else:
             if ndt > 0:
-                self._absorbed(q[:ndt], positions[:ndt], cache, md, nd, out[:ndt])
+                self._absorbed(q[:ndt], angles[:ndt], cache, md, nd, out[:ndt])
             qp = q[ndt:]
-            ops.latent_rope(qp[..., D:], qp[..., D:], self.inv_freq, positions[ndt:], R, 0)
+            ops.latent_rope(qp[..., D:], qp[..., D:], angles[ndt:], R, 0, self.interleaved)
             rows = ops.gather_mla_cache(cache, md.block_table[nd:], cu_rows, first, total)
             kv = ops.gemm(rows, self.up_kv.view(H * (D + R + V), self.row)).view(total, H, D + R + V)
             ops.varlen_attention(qp, kv[..., : D + R], kv[..., D + R:], md.prefill_query_start_loc, cu_rows, self.scale,

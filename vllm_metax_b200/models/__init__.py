@@ -55,6 +55,7 @@ _MODELS: dict[str, tuple[str, str]] = {
     "Naguzen": ("naguzen", "NaguzenForCausalLM"),
     "Pupalorn": ("pupalorn", "PupalornForCausalLM"),
     "Luluzen": ("luluzen", "LuluzenForCausalLM"),
+    "Vetipel": ("vetipel", "VetipelForCausalLM"),
     "MambaForCausalLM": ("mamba", "MambaForCausalLM"),
     "Qwen3NextForCausalLM": ("qwen3_next", "Qwen3NextForCausalLM"),
     "Glm4MoeForCausalLM": ("moe_family", "Glm4MoeForCausalLM"),

@@ -26,7 +26,7 @@ from ..config import ModelConfig
 from ..engine.loader import copy_to_slots, safetensors_shapes
 from ..layers.basic import ParallelLMHead, VocabParallelEmbedding
 from ..layers.fused_moe import FusedMoE
-from ..layers.latent_attention import LatentAttention, LatentCache
+from ..layers.latent_attention import LatentAttention
 from ..layers.recurrent import GatedLinearAttention, InputConv, RGLRUMixer, _param
 from ..ops.residual_norm import residual_norm
 from ..parallel import state as ps
@@ -125,9 +125,7 @@ class NaguzenLayer(nn.Module):
         out = {"norm1": self.out1_norm.weight.data, "canon1": self.conv1.weight.data}
         m = self.mixer
         if self.kind == "latent_attention":
-            out.update({"mix.dq": m.down.rows("dq"), "mix.dq.norm": m.q_norm.data, "mix.uq": m.up_q.data,
-                        "mix.dkv": m.down.rows("dkv"), "mix.dkv.norm": m.kv_norm.data, "mix.uk": m.up_k.data,
-                        "mix.uv": m.up_v.data, "mix.o": m.out_proj.data})
+            out.update({f"mix.{k}": v for k, v in m.slots().items()})
         elif self.kind == "gla":
             out.update({f"mix.{n}": m.in_proj.rows(n) for n in ("q", "k", "v", "g", "a1")})
             out.update({"mix.a2": m.decay_proj.data, "mix.a2.b": m.decay_bias.data, "mix.norm": m.head_norm.data,
@@ -181,13 +179,12 @@ class NaguzenForCausalLM(nn.Module):
         return {"kind": "latent"}
 
     def kv_bytes_per_block(self, block_size: int, kv_cache_dtype: str) -> int:
-        return sum(m.row for m in self._latent()) * block_size * torch.empty((), dtype=self.cfg.dtype).element_size()
+        return sum(m.cache_elems_per_token() for m in self._latent()) * block_size * torch.empty((), dtype=self.cfg.dtype).element_size()
 
     def allocate_kv_cache(self, num_blocks: int, block_size: int, kv_cache_dtype: str, device) -> list:
         if kv_cache_dtype not in ("auto", "bfloat16", "float16"):
             raise ValueError(f"the latent cache is kept in the model's dtype, not {kv_cache_dtype}")
-        return [LatentCache.allocate(num_blocks, block_size, m.kv_rank, m.rot_dim, self.cfg.dtype, device)
-                for m in self._latent()]
+        return [m.allocate_kv_cache(num_blocks, block_size, device) for m in self._latent()]
 
     def allocate_state(self, slots: int, device) -> int:
         return sum(m.allocate_state(slots, device) for m in self.modules() if m is not self and hasattr(m, "allocate_state"))

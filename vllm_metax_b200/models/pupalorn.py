@@ -23,28 +23,12 @@ from .. import _custom_ops as ops
 from ..config import ModelConfig
 from ..engine.loader import copy_to_slots
 from ..layers.attention import QKNormAttention
-from ..layers.basic import ParallelLMHead, VocabParallelEmbedding
+from ..layers.basic import NormAroundOne, ParallelLMHead, VocabParallelEmbedding
 from ..layers.fused_moe import FusedMoE
 from ..layers.recurrent import _param
 from ..ops.reference import rope_frequencies
 from ..ops.residual_norm import boundary_norm, embed_norm
 from ..parallel import state as ps
-
-
-class NormAroundOne(nn.Module):
-    """The gain ``factor * scale * (1 + weight)`` of an RMS norm, folded into one fp32 vector for the boundary kernels.
-    ``scale`` is a layer scale (one number per channel) or absent."""
-
-    def __init__(self, width: int, dtype, factor: float = 1.0, scaled: bool = False):
-        super().__init__()
-        self.weight = _param(width, dtype=dtype)
-        self.scale = _param(width, dtype=dtype) if scaled else None
-        self.factor = factor
-        self.register_buffer("gain", torch.zeros(width, dtype=torch.float32), persistent=False)
-
-    def finalize_weights(self) -> None:
-        g = self.factor * (1.0 + self.weight.data.float())
-        self.gain.copy_(g if self.scale is None else g * self.scale.data.float())
 
 
 class IdentityRoutedExperts(nn.Module):

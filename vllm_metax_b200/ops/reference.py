@@ -493,8 +493,9 @@ def convert_fp8(dst, src, scale: float = 1.0):
 # --------------------------------------------------------------------------- attention
 def attention_core(q, k, v, scale, causal_offset: Optional[int] = None, window: int = -1,
                    softcap: float = 0.0, sinks: Optional[torch.Tensor] = None,
-                   alibi_slopes: Optional[torch.Tensor] = None, distance_bias: Optional[torch.Tensor] = None):
-    """Dense softmax attention for one sequence.
+                   alibi_slopes: Optional[torch.Tensor] = None, distance_bias: Optional[torch.Tensor] = None,
+                   chunk: int = 0, sigmoid_shift: Optional[torch.Tensor] = None):
+    """Dense softmax (or, with ``sigmoid_shift [Hq]``, sigmoid-weighted) attention for one sequence.
 
     ``q [Lq, Hq, D]``, ``k [Lk, Hkv, D]``, ``v [Lk, Hkv, Dv]`` (fp32).  Query row i
     sits at absolute position ``causal_offset + i`` and sees keys ``<=`` that
@@ -524,7 +525,12 @@ def attention_core(q, k, v, scale, causal_offset: Optional[int] = None, window: 
         mask |= kpos > qpos
     if window is not None and window > 0:
         mask |= kpos <= qpos - window
+    if chunk > 0:
+        mask |= kpos < qpos // chunk * chunk
     s = s.masked_fill(mask[None], float("-inf"))
+    if sigmoid_shift is not None:
+        p = torch.sigmoid(s + sigmoid_shift.float()[:, None, None])
+        return torch.einsum("hqk,khd->qhd", p, vv), torch.zeros(Hq, Lq, device=q.device)
     if sinks is not None:
         s_ext = torch.cat([s, sinks.float()[:, None, None].expand(Hq, Lq, 1)], dim=-1)
         lse = torch.logsumexp(s_ext, dim=-1)
@@ -539,7 +545,7 @@ def attention_core(q, k, v, scale, causal_offset: Optional[int] = None, window: 
 def paged_attention(q, kv_cache, block_table, seq_lens, query_start_loc, scale, *, kv_scales=None,
                     window: int = -1, softcap: float = 0.0, sinks=None, alibi_slopes=None,
                     k_scale: float = 1.0, v_scale: float = 1.0, causal: bool = True, return_lse: bool = False,
-                    distance_bias=None, gate=None, out_scale: float = 1.0):
+                    distance_bias=None, gate=None, out_scale: float = 1.0, chunk: int = 0, sigmoid_shift=None):
     """Varlen attention over the paged cache (prefill, chunked prefill and decode).
 
     ``q [T, Hq, D]`` holds the new tokens of every sequence back to back
@@ -563,11 +569,11 @@ def paged_attention(q, kv_cache, block_table, seq_lens, query_start_loc, scale, 
         o, lse = attention_core(q[s0:s1].float(), k, v, scale,
                                 causal_offset=(sl[b] - (s1 - s0)) if causal else None,
                                 window=window, softcap=softcap, sinks=sinks, alibi_slopes=alibi_slopes,
-                                distance_bias=distance_bias)
+                                distance_bias=distance_bias, chunk=chunk, sigmoid_shift=sigmoid_shift)
         out[s0:s1] = o
         lse_all[:, s0:s1] = lse
     if gate is not None:
-        out = out * torch.sigmoid(gate.float()).reshape(out.shape)
+        out = out * torch.sigmoid(gate.float()).reshape(T, Hq, -1)
     out = (out * out_scale).to(q.dtype)
     return (out, lse_all) if return_lse else out
 
