@@ -184,3 +184,61 @@ def forward(tokens, w, cfg, residuals=None):
         if last and residuals is not None:
             residuals.append(sum(streams))
     return norm(w, "final.norm", sum(streams), eps) @ get(w, "head").t()
+
+
+# ------------------------------------------------------------------ checkpoints for tests
+def tensor_shapes(cfg):
+    W, S = cfg["width"], cfg["streams"]
+    out = {"embed": (cfg["vocab"], W), "final.norm": (W,), "head": (cfg["vocab"], W)}
+    for i, l in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", l["mixer"]
+        subs, pre, H = [1] if l.get("mlp") is None else [1, 2], p + "mix.", m["heads"]
+        for q in subs:
+            out.update({f"{p}norm{q}": (W,), f"{p}hc{q}.in": (S,), f"{p}hc{q}.out": (S,), f"{p}hc{q}.mix": (S, S)})
+        if l["type"] == "latent_attention":
+            K = m["kv_rank"]
+            out.update({pre + "q": (H * (m["dim"] + m["rot_dim"]), W), pre + "dkv": (K + m["rot_dim"], W), pre + "dkv.norm": (K,),
+                        pre + "uk": (H * m["dim"], K), pre + "uv": (H * m["vdim"], K)})
+        else:
+            G = m["kv_heads"]
+            rows = {"q": H * m["dim"], "k": G * m["dim"], "v": G * m["vdim"], "g": H}
+            out.update({pre + n: (r, W) for n, r in rows.items()})
+            if l["type"] == "attention":
+                out[pre + "pb"] = (H,)
+            else:
+                out.update({f"{pre}{n}.b": (rows[n],) for n in "qkv"})
+                out.update({pre + n: (H,) for n in ("r1", "r2", "temp", "sink")})
+        out[pre + "o"] = (W, H * m["vdim"])
+        if l.get("mlp") is not None:
+            out.update({p + "mlp.up": (l["mlp"]["ff"], W), p + "mlp.down": (W, l["mlp"]["ff"])})
+    return out
+
+
+def random_weights(cfg, seed=0):
+    """bf16 tensors under the checkpoint's names; stored norm weights around zero (the latent's around one), mixes around the
+    identity, biases of the size of scores."""
+    g = torch.Generator().manual_seed(seed)
+    out = {}
+    for name, shape in tensor_shapes(cfg).items():
+        t = torch.randn(*shape, generator=g)
+        leaf = name.split(".")[-1]
+        if name.endswith("dkv.norm"):
+            t = 1.0 + 0.3 * t
+        elif "norm" in leaf or leaf == "b":
+            t = 0.3 * t
+        elif leaf == "in":
+            t = 1.0 / cfg["streams"] + 0.3 * t
+        elif leaf in ("out", "temp"):
+            t = 1.0 + 0.4 * t
+        elif leaf == "mix":
+            t = 0.8 * torch.eye(shape[0]) + 0.3 * t
+        elif leaf in ("r1", "r2"):
+            t = t.abs() + 0.1
+        elif leaf == "pb":
+            t = 0.7 * t - 2.0
+        elif leaf == "sink":
+            t = 1.5 * t
+        elif name != "embed":
+            t = t * shape[-1] ** -0.5
+        out[name] = t.to(torch.bfloat16)
+    return out

@@ -215,12 +215,12 @@ def kernel_rows(size: str = "w2048", only: str = "") -> list:
         cache = rn(B * nb, bs, K + R)
         table = torch.arange(B * nb, dtype=torch.int32, device=dev).view(B, nb)
         a, qw, kvw = rn(T, 1536 + K + R), rn(1536), rn(K)
-        freq = torch.rand(R // 2, device=dev)
         pos = (torch.arange(T, device=dev) % per) + (ctx - 1 if T == B else 0)
         blk = torch.arange(T, device=dev) // per
         slots = (table.long()[blk, pos // bs] * bs + pos % bs)
+        angles = ops.rope_angles(pos, torch.rand(R // 2, device=dev, dtype=torch.float64), T)
         row(f"latent_insert, {phase}",
-            lambda: ops.latent_insert(a, 0, 1536, qw, kvw, R, freq, pos, cache, slots, 1e-6),
+            lambda: ops.latent_insert(a, 0, 1536, qw, kvw, R, angles, cache, slots, 1e-6),
             2.0 * T * (1536 + K + R) * 2, 0, ("rms_norm (query latent only)", lambda: ops.rms_norm(y, nw, 1e-6), 4.0 * T * W, 0))
         qn, absorb, lat_q = rn(T, H, D + R), rn(H, K, D), rn(T, H, K + R)
         if T == B:
