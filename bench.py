@@ -19,7 +19,8 @@ iterations).  Two measurements per run:
 prefill and decode throughput, and every kernel of it against its roofline (utils/bench_hybrid.py; one GPU).
 `--shared-kv` does the same for the decoder with windowed, cross-layer-shared attention and identity experts (Pupalorn)
 beside Qwen3-MoE (utils/bench_shared_kv.py), and `--parallel` for the looped decoder with two mixers side by side (Luluzen)
-beside Qwen3-Next and Naguzen (utils/bench_parallel.py).
+beside Qwen3-Next and Naguzen (utils/bench_parallel.py), and `--streams` for the decoder over several residual streams
+(Vetipel) beside Llama and DeepSeek-V3 (utils/bench_streams.py).
 `--impl reference` reports that the reference cannot be installed on this machine.
 """
 from __future__ import annotations
@@ -125,6 +126,8 @@ def layer_list_bench(args) -> None:
         from vllm_metax_b200.utils.bench_shared_kv import SIZES, TITLE, kernel_rows, model_rows
     elif args.parallel:
         from vllm_metax_b200.utils.bench_parallel import SIZES, TITLE, kernel_rows, model_rows
+    elif args.streams:
+        from vllm_metax_b200.utils.bench_streams import SIZES, TITLE, kernel_rows, model_rows
     else:
         from vllm_metax_b200.utils.bench_hybrid import SIZES, TITLE, kernel_rows, model_rows
 
@@ -159,8 +162,10 @@ def main() -> None:
                     help="decoder with cross-layer-shared keys and values (Pupalorn) beside Qwen3-MoE, one GPU")
     ap.add_argument("--parallel", action="store_true",
                     help="looped decoder with two mixers side by side (Luluzen) beside Qwen3-Next and Naguzen, one GPU")
+    ap.add_argument("--streams", action="store_true",
+                    help="decoder over several residual streams (Vetipel) beside Llama and DeepSeek-V3, one GPU")
     args = ap.parse_args()
-    if args.hybrid or args.shared_kv or args.parallel:
+    if args.hybrid or args.shared_kv or args.parallel or args.streams:
         return layer_list_bench(args)
     conf = CONFIGS[args.config]
     MODEL = conf["model"]

@@ -9,6 +9,8 @@ constexpr int kEpiLast = kEpiSoftcap;
 constexpr int kEpiActMask = 0xf, kEpiF32 = 0x10;
 // (gate, up) in adjacent columns, half as many columns come out
 constexpr bool epi_is_gate(int code) { return code == kEpiSiluGate || code == kEpiGeluTanhGate || code == kEpiClampGate; }
+// What store_row_segment's short form does not have; a squared relu is two instructions and does.
+constexpr bool epi_extended(int code) { return code > 1 && code != kEpiRelu2; }
 
 struct Epi {
   int code;

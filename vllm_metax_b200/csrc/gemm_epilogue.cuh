@@ -257,8 +257,8 @@ __device__ __forceinline__ void store_row_segment_f32(const uint32_t (&r)[32], i
     if (cb0 + i < n_cols) dst[i] = f[i];
 }
 
-// (EXT: built with the activations and the fp32 output.  The GEMM kernels exist in both forms, so that plain and gated
-// products keep their short epilogue.)
+// (EXT: built with the activations and the fp32 output.  The GEMM kernels exist in both forms, so that plain, gated and
+// squared-relu products keep their short epilogue.)
 template <typename T, int CH, bool EXT = false>
 __device__ __forceinline__ void store_row_segment(const uint32_t (&r)[32], int row, int cb0, int n_cols,
                                                   T* __restrict__ C, int ldc, const T* __restrict__ bias,
@@ -294,8 +294,42 @@ __device__ __forceinline__ void store_row_segment(const uint32_t (&r)[32], int r
     }
     return;
   }
+  const bool relu2 = epi.code == kEpiRelu2;
   T* dst = C + (size_t)row * ldc + cb0;
   const T* res = residual ? residual + (size_t)row * ldr + cb0 : nullptr;
+  if (cb0 + CH <= n_cols) {                        // the whole segment: every load is on its way before the first is used
+    uint4 b[CH / 8], x[CH / 8];
+    if (bias) {
+#pragma unroll
+      for (int v = 0; v < CH / 8; ++v) b[v] = __ldg(reinterpret_cast<const uint4*>(bias + cb0) + v);
+    }
+    if (res) {
+#pragma unroll
+      for (int v = 0; v < CH / 8; ++v) x[v] = reinterpret_cast<const uint4*>(res)[v];
+    }
+#pragma unroll
+    for (int v = 0; v < CH / 8; ++v) {
+      float f[8], g[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) f[i] = __uint_as_float(r[v * 8 + i]);
+      if (bias) {
+        unpack8<T>(b[v], g);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) f[i] += g[i];
+      }
+      if (res) {
+        unpack8<T>(x[v], g);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) f[i] += g[i];
+      }
+      if (relu2) {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) f[i] *= fmaxf(f[i], 0.f);
+      }
+      *reinterpret_cast<uint4*>(dst + v * 8) = pack8<T>(f);
+    }
+    return;
+  }
 #pragma unroll
   for (int v = 0; v < CH / 8; ++v) {
     const int col = cb0 + v * 8;
@@ -315,6 +349,10 @@ __device__ __forceinline__ void store_row_segment(const uint32_t (&r)[32], int r
 #pragma unroll
         for (int i = 0; i < 8; ++i) f[i] += b[i];
       }
+      if (relu2) {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) f[i] *= fmaxf(f[i], 0.f);
+      }
       *reinterpret_cast<uint4*>(dst + v * 8) = pack8<T>(f);
     } else {
       for (int i = 0; i < 8; ++i) {
@@ -322,6 +360,7 @@ __device__ __forceinline__ void store_row_segment(const uint32_t (&r)[32], int r
           float f = __uint_as_float(r[v * 8 + i]);
           if (bias) f += to_f(bias[col + i]);
           if (res) f += to_f(res[v * 8 + i]);
+          if (relu2) f *= fmaxf(f, 0.f);
           dst[v * 8 + i] = from_f<T>(f);
         }
       }

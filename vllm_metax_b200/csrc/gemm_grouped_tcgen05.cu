@@ -178,7 +178,7 @@ static void launch_grouped(const void* A, int max_rows, int lda, const void* W, 
   uint64_t ws[2] = {(uint64_t)K * 2, (uint64_t)N * K * 2};
   uint32_t wb[3] = {(uint32_t)kGgBK, (uint32_t)BN, 1};
   CUtensorMap tmW = make_tmap_nd(W, dt, 3, wd, ws, wb, CU_TENSOR_MAP_SWIZZLE_128B);
-  auto kern = epi.code > 1 ? gemm_grouped_kernel<T, BN, STAGES, true> : gemm_grouped_kernel<T, BN, STAGES, false>;
+  auto kern = epi_extended(epi.code) ? gemm_grouped_kernel<T, BN, STAGES, true> : gemm_grouped_kernel<T, BN, STAGES, false>;
   // a per-device attribute of the kernel: set on every launch (cheap) rather than once per process
   cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kDyn);
   static int sms = 0;

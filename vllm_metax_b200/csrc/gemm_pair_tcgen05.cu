@@ -286,7 +286,7 @@ static void launch_pair(const void* A, const void* W, void* C, const void* bias,
   CUtensorMap tmB = make_tmap_2d(W, dt, 2, N, K, ldw, 128, kPairBK);
   using L = PairSmem<STAGES, BULK>;
   static_assert(L::kDyn + (BULK ? 1 : 4) * 32 * 33 * 4 <= 232448, "shared memory budget exceeded");
-  const int ext = !BULK && epi.code > 1;
+  const int ext = !BULK && epi_extended(epi.code);
   auto kern = ext ? gemm_pair_kernel<T, STAGES, BULK, !BULK> : gemm_pair_kernel<T, STAGES, BULK, false>;
   // kernel attributes and SM counts are per device
   static bool set[2][64] = {};

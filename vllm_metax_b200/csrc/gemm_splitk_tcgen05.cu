@@ -201,7 +201,7 @@ static void launch_sk(const void* A, const void* W, void* C, const void* bias, c
       std::is_same<T, __half>::value ? CU_TENSOR_MAP_DATA_TYPE_FLOAT16 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
   CUtensorMap tmA = make_tmap_2d(A, dt, 2, M, K, lda, kSkBM, kSkBK);
   CUtensorMap tmB = make_tmap_2d(W, dt, 2, N, K, ldw, kSkBN, kSkBK);
-  auto kern = epi.code > 1 ? gemm_splitk_kernel<T, true> : gemm_splitk_kernel<T, false>;
+  auto kern = epi_extended(epi.code) ? gemm_splitk_kernel<T, true> : gemm_splitk_kernel<T, false>;
   // a per-device attribute of the kernel: set on every launch (cheap) rather than once per process
   cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SkSmem::kDyn);
   const int tiles = ceil_div(M, kSkBM) * ceil_div(N, kSkBN);

@@ -106,6 +106,58 @@ latent_insert_kernel(const LatentInsertParams p) {
   for (int i = p.kv_rank + p.rot_dim + tid; i < p.row_elems; i += 128) dst[i] = from_f<T>(0.f);
 }
 
+// Without a query latent, 16-byte pieces: a warp per token, whose latent (up to 32 * V * PIECES entries) stays in registers.
+template <typename T, int V, int PIECES>
+__global__ void __launch_bounds__(128)
+latent_insert_rows_kernel(const LatentInsertParams p) {
+  const int64_t t = (int64_t)blockIdx.x * 4 + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (t >= p.tokens) return;
+  const int64_t slot = p.slots[t];
+  if (slot < 0) return;
+  if (slot >= p.num_slots) {
+    if (lane == 0) report_status(p.status, kBadIndex, 120, (int)p.num_slots, (int)slot);
+    return;
+  }
+  const T* src = reinterpret_cast<const T*>(p.a) + t * p.a_stride + p.kv_off;
+  T* dst = reinterpret_cast<T*>(p.cache) + slot * p.row_elems;
+  const T* kr = src + p.kv_rank;
+  float v[PIECES][V], ss = 0.f;
+#pragma unroll
+  for (int r = 0; r < PIECES; ++r) {
+    const int i = (r * 32 + lane) * V;
+    if (i < p.kv_rank) ld_v<T, V>(src + i, v[r]);
+  }
+  const int half = p.rot_dims / 2, step = p.interleaved ? 2 : 1, apart = p.interleaved ? 1 : half;
+  const float* cs = p.angles + 2 * t * half;
+  for (int i = lane; i < half; i += 32) {
+    const int at = i * step;
+    float a = to_f(kr[at]), b = to_f(kr[at + apart]);
+    rotate_pair(a, b, cs[i], cs[half + i]);
+    dst[p.kv_rank + at] = from_f<T>(a);
+    dst[p.kv_rank + at + apart] = from_f<T>(b);
+  }
+  for (int i = 2 * half + lane; i < p.rot_dim; i += 32) dst[p.kv_rank + i] = kr[i];
+  for (int i = p.kv_rank + p.rot_dim + lane; i < p.row_elems; i += 32) dst[i] = from_f<T>(0.f);
+#pragma unroll
+  for (int r = 0; r < PIECES; ++r)
+    if ((r * 32 + lane) * V < p.kv_rank)
+#pragma unroll
+      for (int k = 0; k < V; ++k) ss = fmaf(v[r][k], v[r][k], ss);
+  const float inv = 1.f / sqrtf(warp_sum(ss) / (float)p.kv_rank + p.eps);
+#pragma unroll
+  for (int r = 0; r < PIECES; ++r) {
+    const int i = (r * 32 + lane) * V;
+    if (i < p.kv_rank) {
+      float g[V];
+      ld_v<T, V>(reinterpret_cast<const T*>(p.kv_w) + i, g);
+#pragma unroll
+      for (int k = 0; k < V; ++k) v[r][k] = v[r][k] * inv * g[k];
+      st_v<T, V>(dst + i, v[r]);
+    }
+  }
+}
+
 template <typename T>
 __global__ void latent_rope_kernel(const T* src, int64_t src_tok, int64_t src_head, T* dst, int64_t dst_tok,
                                    int64_t dst_head, const float* __restrict__ angles, int tokens, int heads, int rot_dim,
@@ -219,7 +271,14 @@ int latent_insert(const LatentInsertParams& p, int dtype, cudaStream_t stream) {
   const bool vec = p.q_rank % v == 0 && p.kv_rank % v == 0 && p.row_elems % v == 0 && p.a_stride % v == 0 &&
                    p.q_off % v == 0 && p.kv_off % v == 0 && aligned(p.a) && aligned(p.cq) && aligned(p.cache) &&
                    aligned(p.q_w) && aligned(p.kv_w);
-  if (vec) {
+  if (vec && p.q_rank == 0 && p.kv_rank <= 1024) {
+    const int rows = (p.tokens + 3) / 4;
+    if (p.kv_rank <= 512) {
+      BY_DTYPE((latent_insert_rows_kernel<T, 16 / (int)sizeof(T), 4 * (int)sizeof(T) / 4><<<rows, 128, 0, stream>>>(p)))
+    } else {
+      BY_DTYPE((latent_insert_rows_kernel<T, 16 / (int)sizeof(T), 8 * (int)sizeof(T) / 4><<<rows, 128, 0, stream>>>(p)))
+    }
+  } else if (vec) {
     BY_DTYPE((latent_insert_kernel<T, 16 / (int)sizeof(T)><<<p.tokens, 128, 0, stream>>>(p)))
   } else {
     BY_DTYPE((latent_insert_kernel<T, 1><<<p.tokens, 128, 0, stream>>>(p)))

@@ -14,47 +14,54 @@
 namespace b200 {
 namespace {
 
-// S: streams, or (8) room for p.streams of them.  A thread owns CN columns in each of TRIPS pieces of the row.
-template <typename T, int S, int CN, int TRIPS, bool VEC, int THREADS, int CTAS>
+// S: streams, or (8) room for p.streams of them.  A thread owns CN columns in each of TRIPS pieces of the row.  FIRST: the streams
+// are the embedding row, so that one load and the columns' sums of the mix stand for them all.
+template <typename T, int S, int CN, int TRIPS, bool VEC, bool FIRST, int THREADS, int CTAS>
 __global__ void __launch_bounds__(THREADS, CTAS)
 stream_norm_kernel(const StreamNormParams p) {
   __shared__ float red[2][32];
+  constexpr int R = FIRST ? 1 : S;                 // distinct streams
   const int D = p.D, n = S < kMaxStreams ? S : p.streams, piece = blockDim.x * CN;
-  float read[S], write[S], mix[S][S];
+  float read[S], write[S], mix[R][S];
 #pragma unroll
   for (int t = 0; t < S; ++t) {
     read[t] = t < n ? p.coef[t] : 0.f;
     write[t] = t < n && p.y != nullptr ? p.coef[n + t] : 0.f;
 #pragma unroll
-    for (int s = 0; s < S; ++s) mix[s][t] = p.y == nullptr ? (s == t ? 1.f : 0.f) : s < n && t < n ? p.coef[2 * n + s * n + t] : 0.f;
+    for (int s = 0; s < R; ++s) mix[s][t] = 0.f;
+#pragma unroll
+    for (int s = 0; s < S; ++s)
+      if (s < n && t < n) mix[FIRST ? 0 : s][t] += p.y != nullptr ? p.coef[2 * n + s * n + t] : s == t ? 1.f : 0.f;
   }
   const float inv_d = 1.f / (float)D;
   int turn = 0;
   for (int64_t tok = blockIdx.x; tok < p.tokens; tok += gridDim.x, turn ^= 1) {
     float u[TRIPS][CN], ss = 0.f;
+    const T* row = nullptr;
+    float scale = 1.f;
+    if constexpr (FIRST) {
+      const int64_t id = p.ids[tok];
+      const bool ok = id >= 0 && id < p.rows;
+      if (!ok && threadIdx.x == 0) report_status(p.status, kBadIndex, 160, (int)p.rows, (int)id);
+      row = reinterpret_cast<const T*>(p.table) + (ok ? id : 0) * D;
+      scale = ok ? p.scale : 0.f;
+    }
 #pragma unroll
     for (int r = 0; r < TRIPS; ++r) {
       const int c0 = r * piece + threadIdx.x * CN;
 #pragma unroll
       for (int k = 0; k < CN; ++k) u[r][k] = 0.f;
       if (c0 >= D) continue;
-      float x[S][CN], y[CN] = {};
+      float x[R][CN], y[CN] = {};
       if (p.y != nullptr) load_row<T, CN, VEC>(reinterpret_cast<const T*>(p.y) + tok * D, c0, D, y);
-      if (p.x != nullptr) {
+      if constexpr (FIRST) {
+        load_row<T, CN, VEC>(row, c0, D, x[0]);
+#pragma unroll
+        for (int k = 0; k < CN; ++k) x[0][k] *= scale;
+      } else {
 #pragma unroll
         for (int s = 0; s < S; ++s)
           if (s < n) load_row<float, CN, VEC>(p.x + (tok * n + s) * D, c0, D, x[s]);
-      } else {
-        const int64_t row = p.ids[tok];
-        const bool ok = row >= 0 && row < p.rows;
-        if (!ok && threadIdx.x == 0 && r == 0) report_status(p.status, kBadIndex, 160, (int)p.rows, (int)row);
-        load_row<T, CN, VEC>(reinterpret_cast<const T*>(p.table) + (ok ? row : 0) * D, c0, D, x[0]);
-#pragma unroll
-        for (int k = 0; k < CN; ++k) {
-          x[0][k] *= ok ? p.scale : 0.f;
-#pragma unroll
-          for (int s = 1; s < S; ++s) x[s][k] = x[0][k];
-        }
       }
 #pragma unroll
       for (int t = 0; t < S; ++t) {
@@ -64,7 +71,7 @@ stream_norm_kernel(const StreamNormParams p) {
           for (int k = 0; k < CN; ++k) {
             v[k] = write[t] * y[k];
 #pragma unroll
-            for (int s = 0; s < S; ++s)
+            for (int s = 0; s < R; ++s)
               if (s < n) v[k] = fmaf(mix[s][t], x[s][k], v[k]);
             u[r][k] = fmaf(read[t], v[k], u[r][k]);
           }
@@ -90,9 +97,16 @@ stream_norm_kernel(const StreamNormParams p) {
 
 template <typename T, int S, int CN, int TRIPS, bool VEC, int THREADS, int CTAS>
 void launch(const StreamNormParams& p, cudaStream_t stream) {
-  const int piece = ceil_div(p.D, TRIPS), threads = ceil_div(piece, CN * 32) * 32;
-  const int ctas = 148 * CTAS * (THREADS / threads);
-  stream_norm_kernel<T, S, CN, TRIPS, VEC, THREADS, CTAS><<<p.tokens < ctas ? p.tokens : ctas, threads, 0, stream>>>(p);
+  const int threads = ceil_div(ceil_div(p.D, TRIPS), CN * 32) * 32;
+  auto grid = [&](int ctas) {
+    ctas *= 148 * (THREADS / threads);
+    return p.tokens < ctas ? p.tokens : ctas;
+  };
+  constexpr int kFirst = 1024 / THREADS;           // (one row in registers: room for more CTAs)
+  if (p.x == nullptr)
+    stream_norm_kernel<T, S, CN, TRIPS, VEC, true, THREADS, kFirst><<<grid(kFirst), threads, 0, stream>>>(p);
+  else
+    stream_norm_kernel<T, S, CN, TRIPS, VEC, false, THREADS, CTAS><<<grid(CTAS), threads, 0, stream>>>(p);
 }
 
 template <typename T, int S>
