@@ -41,7 +41,7 @@ def read_streams(streams, weights):
 
 
 def write_streams(streams, mix, out, y):
-    """All streams at once from the old ones: ``mix[s, t]`` is what stream t takes of stream s."""
+    """The new streams, each made of all the streams before: ``mix[s, t]`` is what stream t takes of stream s."""
     return [sum(float(mix[s, t]) * x for s, x in enumerate(streams)) + float(out[t]) * y for t in range(len(streams))]
 
 

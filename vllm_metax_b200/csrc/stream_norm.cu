@@ -1,7 +1,7 @@
 // Sublayer boundary of decoders whose residual is several fp32 streams (hyper-connections with fixed weights) - everything between
 // one sublayer's last product and the next one's first, in one launch:
 //
-//     x'_t = sum_s mix[s, t] x_s + write[t] y          all streams at once from the old ones
+//     x'_t = sum_s mix[s, t] x_s + write[t] y          (x: the streams before)
 //     u    = sum_t read[t] x'_t
 //     h    = gain * u / sqrt(mean(u^2) + eps)          (in y's type: the next product's operand, or the LM head's)
 //

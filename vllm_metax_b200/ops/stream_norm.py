@@ -1,6 +1,6 @@
 """Sublayer boundary of decoders whose residual is several fp32 streams (``csrc/stream_norm.cu``).
 
-    x'_t = sum_s mix[s, t] x_s + write[t] y          all streams at once from the old ones
+    x'_t = sum_s mix[s, t] x_s + write[t] y          (x: the streams before)
     u    = sum_t read[t] x'_t
     h    = gain * u / sqrt(mean(u^2) + eps)          the next sublayer's input
 
